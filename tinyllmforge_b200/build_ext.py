@@ -94,10 +94,12 @@ def build(force: bool = False, verbose: bool = False) -> str:
     if force or jobs or not os.path.exists(out) or not os.path.exists(stamp) or open(stamp).read() != link_tag:
         torch_lib = os.path.join(os.path.dirname(torch.__file__), "lib")
         cuda_lib = os.path.join(os.path.dirname(cuda_inc), "lib64")
-        cmd = ["g++", "-shared", "-o", out] + objs + [
+        part = out + ".part"                      # complete before it gets its name: another process may be looking for it
+        cmd = ["g++", "-shared", "-o", part] + objs + [
             f"-L{torch_lib}", f"-L{cuda_lib}", "-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-ltorch_python",
             "-lcudart", f"-Wl,-rpath,{torch_lib}", f"-Wl,-rpath,{cuda_lib}"]
         _run(cmd, verbose)
+        os.replace(part, out)
         with open(stamp, "w") as f:
             f.write(link_tag)
     return out

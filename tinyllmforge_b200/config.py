@@ -114,9 +114,18 @@ class ModelConfig:
         if self.head_dim % 2:
             raise ValueError("head_dim must be even for rotary embedding")
 
+    def validate_tp(self, size: int) -> None:
+        if self.num_key_value_heads % size or self.num_attention_heads % size:
+            raise ValueError("attention heads and KV heads must divide evenly by tensor_parallel_size")
+        if self.vocab_size % size:
+            raise ValueError("vocab_size must divide evenly by tensor_parallel_size")
+
     @property
     def dtype(self) -> torch.dtype:
         return parse_dtype(self.torch_dtype)
+
+    prefix_cacheable = True          # every block of the KV cache is a function of the tokens before it alone
+    num_recurrent_runs = 0           # layer runs that keep a per-sequence state beside the paged cache
 
 
 # Architectures named by the benchmark definition; weights are random-init.
@@ -139,10 +148,11 @@ PRESETS = {
 }
 
 
-def preset(name: str, **overrides) -> ModelConfig:
+def preset(name: str, **overrides):
     if name not in PRESETS:
         raise KeyError(f"unknown preset {name!r}; known: {sorted(PRESETS)}")
-    return ModelConfig.from_dict({**PRESETS[name], **overrides})
+    from .models import registry
+    return registry.config_from_dict({**PRESETS[name], **overrides})
 
 
 @dataclass
@@ -154,7 +164,7 @@ class Config:
     gpu_memory_utilization: float = 0.9
     tensor_parallel_size: int = 1
     enforce_eager: bool = False
-    hf_config: Optional[ModelConfig] = None
+    hf_config: Optional[Any] = None          # a configuration class of models/registry.py (ModelConfig, GoselixConfig) or its dict
     eos: int = -1
     kvcache_block_size: int = 256
     num_kvcache_blocks: int = -1
@@ -173,22 +183,20 @@ class Config:
     extra: dict = field(default_factory=dict)
 
     def __post_init__(self):
+        from .models import registry
         if self.hf_config is None:
             if not os.path.isdir(self.model):
                 raise FileNotFoundError(f"model directory not found: {self.model}")
-            self.hf_config = ModelConfig.from_dir(self.model)
+            self.hf_config = registry.config_from_dir(self.model)
         elif isinstance(self.hf_config, dict):
-            self.hf_config = ModelConfig.from_dict(self.hf_config)
+            self.hf_config = registry.config_from_dict(self.hf_config)
         bs = self.kvcache_block_size
         if bs < 8 or bs & (bs - 1):
             raise ValueError(f"kvcache_block_size must be a power of two >= 8, got {bs}")
         if not 1 <= self.tensor_parallel_size <= 8:
             raise ValueError("tensor_parallel_size must be in [1, 8] (single host)")
         hf = self.hf_config
-        if hf.num_key_value_heads % self.tensor_parallel_size or hf.num_attention_heads % self.tensor_parallel_size:
-            raise ValueError("attention heads and KV heads must divide evenly by tensor_parallel_size")
-        if hf.vocab_size % self.tensor_parallel_size:
-            raise ValueError("vocab_size must divide evenly by tensor_parallel_size")
+        hf.validate_tp(self.tensor_parallel_size)
         self.max_model_len = min(self.max_model_len, hf.max_position_embeddings)
         if self.max_num_batched_tokens < self.max_model_len and not self.chunked_prefill:
             raise ValueError("max_num_batched_tokens must be >= max_model_len (prompts are prefilled whole; "
@@ -209,6 +217,8 @@ class Config:
             raise ValueError("quantization must be None or 'fp8_block'")
         if self.load_format not in ("auto", "dummy"):
             raise ValueError("load_format must be 'auto' or 'dummy'")
+        if self.quantization is not None and not getattr(hf, "quantizable", True):
+            raise ValueError(f"quantization={self.quantization!r} is not available for {type(hf).__name__}")
         self.dtype = parse_dtype(self.dtype) if self.dtype is not None else hf.dtype
         if self.eos < 0 and hf.eos_token_id is not None:
             self.eos = hf.eos_token_id

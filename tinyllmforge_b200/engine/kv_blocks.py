@@ -19,6 +19,10 @@ insertion-ordered dict, so reviving a specific freed block is O(1) (the
 reference's ``deque.remove`` is O(free blocks)); the number of cached tokens
 is capped at ``len(request) - 1`` so a fully cached prompt still computes its
 last token (the reference produces an empty query in that case).
+
+Models with recurrent layers keep one state per sequence beside the paged cache.  Its slot
+is taken and given back together with the request's blocks (``StateSlots``), and prefix
+reuse is off for them: a state cannot be picked up in the middle of a prompt.
 """
 from __future__ import annotations
 
@@ -52,10 +56,27 @@ def chain_hash(token_ids, parent: int = -1) -> int:
     return _hash64(parent, struct.pack(f"<{len(token_ids)}q", *token_ids))
 
 
+class StateSlots:
+    """Free list of recurrent-state slots.  A slot needs no clearing: a sequence's first token starts from zero."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self.free = list(range(num_slots - 1, -1, -1))
+
+    def take(self) -> int:
+        return self.free.pop()
+
+    def give(self, slot: int) -> None:
+        assert 0 <= slot < self.num_slots and slot not in self.free
+        self.free.append(slot)
+
+
 class KVBlockPool:
-    def __init__(self, num_blocks: int, block_size: int):
+    def __init__(self, num_blocks: int, block_size: int, prefix_caching: bool = True, num_state_slots: int = 0):
         if num_blocks <= 0:
             raise ValueError("the KV pool needs at least one block")
+        self.prefix_caching = prefix_caching
+        self.state_slots = StateSlots(num_state_slots) if num_state_slots > 0 else None
         self.num_blocks = num_blocks
         self.block_size = block_size
         self.ref_count = [0] * num_blocks
@@ -97,6 +118,8 @@ class KVBlockPool:
 
     # ------------------------------------------------------------------ prefill
     def can_admit(self, req: Request) -> bool:
+        if self.state_slots is not None and not self.state_slots.free:
+            return False
         return len(self.free) >= self.blocks_needed(len(req))
 
     def admit(self, req: Request, seal_upto: int | None = None) -> None:
@@ -106,6 +129,8 @@ class KVBlockPool:
         a block must not be found by other requests before the step that computes it has been scheduled);
         ``seal_computed`` registers the rest later."""
         assert not req.block_table, "request already holds blocks"
+        if self.state_slots is not None:
+            req.state_slot = self.state_slots.take()
         bs = self.block_size
         n = len(req)
         if seal_upto is None:
@@ -116,7 +141,7 @@ class KVBlockPool:
         cached = 0
         for i in range(self.blocks_needed(n)):
             chunk = tuple(toks[i * bs:(i + 1) * bs])
-            full = len(chunk) == bs
+            full = len(chunk) == bs and self.prefix_caching
             h = chain_hash(chunk, parent) if full else -1
             block_id = -1
             if not missed and full:
@@ -150,6 +175,9 @@ class KVBlockPool:
             self._seal_block(req, index, (index + 1) * bs)
 
     def release(self, req: Request) -> None:
+        if req.state_slot >= 0:
+            self.state_slots.give(req.state_slot)
+            req.state_slot = -1
         for block_id in reversed(req.block_table):
             self.ref_count[block_id] -= 1
             assert self.ref_count[block_id] >= 0
@@ -182,6 +210,8 @@ class KVBlockPool:
 
     def _seal_block(self, req: Request, index: int, end: int) -> None:
         """Hash and register block ``index`` of ``req``, whose last token is token ``end - 1``."""
+        if not self.prefix_caching:
+            return
         block_id = req.block_table[index]
         if self.block_hash[block_id] != -1 or self.ref_count[block_id] != 1:
             return
@@ -191,11 +221,26 @@ class KVBlockPool:
         chunk = tuple(req.token_ids[end - self.block_size:end])
         self._seal(block_id, chain_hash(chunk, parent), chunk)
 
+    def extend(self, req: Request) -> None:
+        """Blocks for all tokens of ``req`` (any number of new ones), without sealing any: a caller that feeds a request's
+        tokens in portions of its own choice."""
+        if not req.block_table and self.state_slots is not None and req.state_slot < 0:
+            if not self.state_slots.free:
+                raise RuntimeError("no recurrent-state slot is free")
+            req.state_slot = self.state_slots.take()
+        need = self.blocks_needed(len(req)) - len(req.block_table)
+        if need > len(self.free):
+            raise RuntimeError(f"the KV cache has {len(self.free)} free blocks, {need} are needed")
+        for _ in range(need):
+            req.block_table.append(self._take_oldest())
+
     # ------------------------------------------------------------------ checks (tests)
     def check_invariants(self) -> None:
         used = {i for i, r in enumerate(self.ref_count) if r > 0}
         free = set(self.free)
         assert used.isdisjoint(free)
         assert used | free == set(range(self.num_blocks))
+        if self.state_slots is not None:
+            assert len(set(self.state_slots.free)) == len(self.state_slots.free)
         for h, b in self.hash_to_block.items():
             assert self.block_hash[b] == h

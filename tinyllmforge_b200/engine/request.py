@@ -22,7 +22,7 @@ class RequestStatus(Enum):
 
 class Request:
     __slots__ = ("req_id", "status", "token_ids", "num_prompt_tokens", "num_cached_tokens", "num_computed_tokens", "prefill_end",
-                 "block_table", "temperature", "max_tokens", "ignore_eos", "num_preemptions")
+                 "block_table", "state_slot", "temperature", "max_tokens", "ignore_eos", "num_preemptions")
 
     _ids = count()
 
@@ -40,6 +40,7 @@ class Request:
         self.num_computed_tokens = -1
         self.prefill_end = -1
         self.block_table: list[int] = []
+        self.state_slot = -1                # row of the recurrent-state arrays (models with recurrent layers), -1: none
         self.temperature = float(sampling_params.temperature)
         self.max_tokens = int(sampling_params.max_tokens)
         self.ignore_eos = bool(sampling_params.ignore_eos)

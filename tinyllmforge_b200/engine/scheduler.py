@@ -36,7 +36,9 @@ class Scheduler:
         self.max_num_seqs = config.max_num_seqs
         self.max_num_batched_tokens = config.max_num_batched_tokens
         self.eos = config.eos
-        self.pool = KVBlockPool(config.num_kvcache_blocks, config.kvcache_block_size)
+        hf = config.hf_config
+        self.pool = KVBlockPool(config.num_kvcache_blocks, config.kvcache_block_size, prefix_caching=hf.prefix_cacheable,
+                                num_state_slots=config.max_num_seqs if hf.num_recurrent_runs else 0)
         self.waiting: deque[Request] = deque()
         self.running: deque[Request] = deque()
         self.num_preemptions = 0

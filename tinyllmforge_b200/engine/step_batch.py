@@ -15,13 +15,20 @@ graph always finds its inputs at the same device addresses.
 Layout (all int32 words, every section starts on a 16-byte boundary):
 
     header[16]   magic, is_prefill, num_seqs, num_tokens, padded_seqs, padded_tokens,
-                 table_width, max_seqlen_q, max_seqlen_k, step_index, seed_lo, seed_hi, 0...
+                 table_width, max_seqlen_q, max_seqlen_k, step_index, seed_lo, seed_hi, num_single, kv_rows, 0...
     input_ids[padded_tokens] positions[padded_tokens] slot_mapping[padded_tokens]
     cu_seqlens_q[padded_seqs + 1] context_lens[padded_seqs] last_index[padded_seqs]
     temperatures[padded_seqs] (float32 bit patterns)
     block_tables[padded_seqs * table_width]
     src_rows[padded_seqs]    decode only: >= 0 -> this sequence's input token is row src_rows[i] of the PREVIOUS step's
                              sampled tokens, still on the device (pipelined engine loop); -1 -> input_ids[i] is valid
+    state_slots[padded_seqs] row of the recurrent-state arrays that belongs to the sequence; -1: none (padding, or a model
+                             without recurrent layers)
+    cu_seqlens_k[padded_seqs + 1]  running sum of the keys visible to the sequences from ``num_single`` on (0 before)
+
+A prefill step may mix portions of prompts with single tokens of running requests.  ``num_single`` counts its LEADING
+sequences with one query token: a model may give them to its decode kernels and the rest to its prefill kernels;
+``kv_rows`` is the last entry of cu_seqlens_k.
 
 Padding rows use slot -1 (the KV store skips them), context length 0 and block id -1.
 Decode positions are ``len - 1``: the index of the token whose KV entry is being
@@ -33,10 +40,10 @@ import numpy as np
 
 MAGIC = 0x464F5247  # "FORG"
 HEADER_WORDS = 16
-H_MAGIC, H_PREFILL, H_NSEQ, H_NTOK, H_PSEQ, H_PTOK, H_WIDTH, H_MAXQ, H_MAXK, H_STEP, H_SEEDLO, H_SEEDHI = range(12)
+H_MAGIC, H_PREFILL, H_NSEQ, H_NTOK, H_PSEQ, H_PTOK, H_WIDTH, H_MAXQ, H_MAXK, H_STEP, H_SEEDLO, H_SEEDHI, H_NSINGLE, H_KVROWS = range(14)
 
 SECTIONS = ("input_ids", "positions", "slot_mapping", "cu_seqlens_q", "context_lens", "last_index",
-            "temperatures", "block_tables", "src_rows")
+            "temperatures", "block_tables", "src_rows", "state_slots", "cu_seqlens_k")
 
 
 def _align4(n: int) -> int:
@@ -49,6 +56,7 @@ def section_offsets(padded_tokens: int, padded_seqs: int, table_width: int) -> t
         "input_ids": padded_tokens, "positions": padded_tokens, "slot_mapping": padded_tokens,
         "cu_seqlens_q": padded_seqs + 1, "context_lens": padded_seqs, "last_index": padded_seqs,
         "temperatures": padded_seqs, "block_tables": padded_seqs * table_width, "src_rows": padded_seqs,
+        "state_slots": padded_seqs, "cu_seqlens_k": padded_seqs + 1,
     }
     off = HEADER_WORDS
     out = {}
@@ -75,6 +83,7 @@ class StepBatch:
         self.max_seqlen_q = int(buf[H_MAXQ])
         self.max_seqlen_k = int(buf[H_MAXK])
         self.step_index = int(buf[H_STEP])
+        self.num_single, self.kv_rows = int(buf[H_NSINGLE]), int(buf[H_KVROWS])
         self.seed = (int(buf[H_SEEDLO]) & 0xFFFFFFFF) | ((int(buf[H_SEEDHI]) & 0xFFFFFFFF) << 32)
         self.offsets, self.num_words = section_offsets(self.padded_tokens, self.padded_seqs, self.table_width)
         assert self.num_words <= buf.shape[0]
@@ -118,7 +127,8 @@ def _new(is_prefill, num_seqs, num_tokens, padded_seqs, padded_tokens, width, ma
 
 def build_prefill(reqs, block_size: int, step_index: int = 0, seed: int = 0) -> StepBatch:
     """Prefill step: every request contributes its not-yet-cached tokens (or, for a prompt prefilled in chunks, the
-    tokens [num_computed_tokens, prefill_end); the keys it sees then end at prefill_end)."""
+    tokens [num_computed_tokens, prefill_end); the keys it sees then end at prefill_end).  A range of one token is a
+    decode step of that request; put such requests first (``num_single``)."""
     S = len(reqs)
     starts = [r.num_computed_tokens if r.num_computed_tokens >= 0 else r.num_cached_tokens for r in reqs]
     ends = [r.prefill_end if r.prefill_end >= 0 else len(r) for r in reqs]
@@ -153,6 +163,12 @@ def build_prefill(reqs, block_size: int, step_index: int = 0, seed: int = 0) -> 
     sec("last_index")[:] = cu[1:] - 1
     sec("temperatures").view(np.float32)[:] = [r.temperature for r in reqs]
     sec("src_rows")[:] = -1
+    sec("state_slots")[:] = [r.state_slot for r in reqs]
+    longer = np.nonzero(q_lens != 1)[0]
+    num_single = int(longer[0]) if longer.size else S
+    cu_k = sec("cu_seqlens_k")
+    np.cumsum(k_lens[num_single:], out=cu_k[num_single + 1:])
+    buf[H_NSINGLE], buf[H_KVROWS] = num_single, cu_k[-1]
     return StepBatch(buf)
 
 
@@ -185,6 +201,10 @@ def build_decode(reqs, block_size: int, step_index: int = 0, seed: int = 0,
         bt = r.block_table
         tables[i, :len(bt)] = bt
     sec("src_rows")[:] = -1
+    slots = sec("state_slots")
+    slots[:] = -1
+    slots[:S] = [r.state_slot for r in reqs]
+    buf[H_NSINGLE] = S
     return StepBatch(buf)
 
 

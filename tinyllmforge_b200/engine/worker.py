@@ -21,7 +21,7 @@ import numpy as np
 import torch
 
 from ..config import Config
-from ..models.qwen3 import Qwen3ForCausalLM
+from ..models.registry import model_class
 from ..ops.ref import RefOps
 from ..parallel.comm import TPGroup
 from ..utils.weights import init_dummy_weights, load_weights
@@ -38,6 +38,7 @@ class DeviceBatch:
         self.padded_seqs, self.padded_tokens = sb.padded_seqs, sb.padded_tokens
         self.table_width = sb.table_width
         self.max_seqlen_q, self.max_seqlen_k = sb.max_seqlen_q, sb.max_seqlen_k
+        self.num_single, self.kv_rows = sb.num_single, sb.kv_rows
         self.step_index, self.seed = sb.step_index, sb.seed
         self.words = words
         self.header = words[:HEADER_WORDS]
@@ -82,19 +83,12 @@ class Worker:
             ops = RefOps
         self.ops = ops
         with torch.inference_mode():
-            self.model = Qwen3ForCausalLM(hf, tp, config.dtype, self.device, ops, max_positions=config.max_model_len)
+            self.model = model_class(hf)(hf, tp, config.dtype, self.device, ops, max_positions=config.max_model_len)
             if config.load_format == "dummy":
                 init_dummy_weights(self.model, config.seed)
             else:
                 load_weights(self.model, config.model)
-            if (self.is_cuda and tp.size == 1 and config.quantization is None and config.dtype == torch.bfloat16
-                    and config.extra.get("fold_norms", True) and not hf.attention_bias):
-                self.model.fold_norm_weights()      # add + RMSNorm become GEMM epilogues (models/qwen3.py)
-            if config.quantization == "fp8_block":
-                from ..ops.quant import Fp8BlockWeight
-                for l in self.model.layers:          # the four projections of every block; embeddings and LM head stay bf16
-                    for lin in (l.qkv_proj, l.o_proj, l.gate_up_proj, l.down_proj):
-                        lin.weight = Fp8BlockWeight.quantize(lin.weight)
+            self.model.finish_loading(config)
             if self.is_cuda and tp.size > 1 and config.comm == "fused":
                 ops.enable_fused_comm(hf.hidden_size, config.max_num_batched_tokens, config.comm_timeout_s)
             # staging: the largest step is a full prefill (3 token-sized sections) or the widest decode bucket
@@ -125,11 +119,6 @@ class Worker:
             self.ops.launches = 0
 
     # ------------------------------------------------------------------ KV cache
-    def _kv_block_bytes(self) -> int:
-        hf = self.config.hf_config
-        kvh = hf.num_key_value_heads // self.tp.size
-        return 2 * hf.num_hidden_layers * self.block_size * kvh * hf.head_dim * torch.finfo(self.config.dtype).bits // 8
-
     def _warmup(self) -> None:
         """One full-budget prefill so the allocator's peak reflects the largest step
         (tinyvllm/engine/model_runner.py:108-116)."""
@@ -142,29 +131,32 @@ class Worker:
         for i in range(n):
             r = Request([0] * seq_len)
             r.block_table = list(range(i * nblk, (i + 1) * nblk))
+            r.state_slot = i if self.num_slots else -1
             reqs.append(r)
         self.run(build_prefill(reqs, self.block_size))
 
     def _allocate_kv_cache(self) -> None:
-        cfg, hf = self.config, self.config.hf_config
-        kvh = hf.num_key_value_heads // self.tp.size
-        block_bytes = self._kv_block_bytes()
+        cfg = self.config
+        block_bytes = self.model.kv_block_bytes(self.block_size)
+        self.num_slots = cfg.max_num_seqs if self.model.state_bytes() else 0        # one recurrent state per running request
         if cfg.num_kvcache_blocks <= 0:
             if self.is_cuda:
                 # temporary cache just large enough for the warm-up prefill
                 n_tmp = max(1, min(cfg.max_num_batched_tokens // min(cfg.max_model_len, cfg.max_num_batched_tokens), cfg.max_num_seqs)) * self.table_width
-                self.model.bind_kv_cache(torch.zeros(hf.num_hidden_layers, 2, n_tmp, kvh, self.block_size, hf.head_dim,
-                                                     dtype=cfg.dtype, device=self.device))
+                self.model.bind_cache(n_tmp, self.block_size, self.num_slots)
                 torch.cuda.reset_peak_memory_stats()
                 self._warmup()
                 torch.cuda.synchronize()
-                self.model.kv_cache = None
+                self.model.drop_cache()
                 torch.cuda.empty_cache()
                 free, total = torch.cuda.mem_get_info()
                 stats = torch.cuda.memory_stats()
                 peak, cur = stats["allocated_bytes.all.peak"], stats["allocated_bytes.all.current"]
-                budget = int(total * cfg.gpu_memory_utilization) - (total - free) - (peak - cur)
-                n = budget // block_bytes
+                budget = int(total * cfg.gpu_memory_utilization) - (total - free) - (peak - cur) - self.num_slots * self.model.state_bytes()
+                # a model whose layers are all recurrent pages nothing: the blocks then only bound the tokens of live requests
+                n = budget // block_bytes if block_bytes else cfg.max_num_seqs * self.table_width
+                if budget <= 0:
+                    n = 0
             else:
                 n = max(64, min(cfg.max_num_seqs, 16) * self.table_width)
             # every rank must agree on the pool size: take the minimum
@@ -175,8 +167,7 @@ class Worker:
             if n <= 0:
                 raise RuntimeError("no memory left for the KV cache; raise gpu_memory_utilization")
             cfg.num_kvcache_blocks = int(n)
-        self.model.bind_kv_cache(torch.zeros(hf.num_hidden_layers, 2, cfg.num_kvcache_blocks, kvh, self.block_size,
-                                             hf.head_dim, dtype=cfg.dtype, device=self.device))
+        self.model.bind_cache(cfg.num_kvcache_blocks, self.block_size, self.num_slots)
 
     # ------------------------------------------------------------------ execution
     def decode_padding(self, num_seqs: int) -> tuple[int | None, int | None]:
@@ -267,6 +258,16 @@ class Worker:
         return self.collect(self.launch(sb))
 
     @torch.inference_mode()
+    def logits(self, sb: StepBatch, rows: list[int]) -> torch.Tensor:
+        """Run one step without sampling; fp32 logits (on the host) of the step's tokens ``rows``."""
+        batch = self._stage(sb)
+        out = self.model.logits_at(batch, torch.tensor(rows, dtype=torch.int32, device=self.device)).float().cpu()
+        if self.is_cuda:
+            self.ops.check_status()
+        self.num_steps += 1
+        return out
+
+    @torch.inference_mode()
     def _capture_graphs(self) -> None:
         """One graph per decode bucket, largest first so they share one memory pool
         (tinyvllm/engine/model_runner.py:289-297).  Inputs are views of the static step buffer."""
@@ -278,6 +279,7 @@ class Worker:
             for i in range(b):
                 r = Request([0, 0])
                 r.block_table = [i % self.config.num_kvcache_blocks]
+                r.state_slot = i % self.num_slots if self.num_slots else -1
                 reqs.append(r)
             sb = build_decode(reqs, self.block_size, pad_to=b, table_width=self.table_width)
             batch = self._stage(sb)

@@ -1,0 +1,146 @@
+"""Building blocks of decoders whose layers are listed one by one: mixers and feed-forwards.
+
+A block owns its weights (all sizes and constants come from its spec), names them for the checkpoint loader, says what it
+keeps per token (paged cache) or per sequence (recurrent state), and issues its ops.  A model of another design uses the
+same blocks with other specs.
+
+    mixer        forward(ops, h, memory, batch) -> [tokens, width]; ``memory`` is what ``new_memory`` returned for this run
+    feed-forward forward(ops, h) -> [tokens, width], or the op set's own representation of a sum over experts
+"""
+from __future__ import annotations
+
+import torch
+
+
+def _empty(shape, dtype, device):
+    return torch.empty(shape, dtype=dtype, device=device)
+
+
+class LatentAttention:
+    """Attention whose keys and values are rebuilt from one low-rank latent per token; a rotated key part is shared by all
+    heads.  Cached per token: the normed latent and the rotated part."""
+    recurrent = False
+
+    def __init__(self, spec, width: int, eps: float, dtype, device, rope):
+        self.spec, self.eps = spec, eps
+        H = spec.heads
+        self.a_proj = _empty((spec.q_rank + spec.kv_rank + spec.rot_dim, width), dtype, device)     # dq | dkv
+        self.q_norm = _empty(spec.q_rank, dtype, device)
+        self.kv_norm = _empty(spec.kv_rank, dtype, device)
+        self.uq = _empty((H * (spec.dim + spec.rot_dim), spec.q_rank), dtype, device)
+        self.ukv = _empty((H * (spec.dim + spec.vdim), spec.kv_rank), dtype, device)                # uk | uv
+        self.o = _empty((width, H * spec.vdim), dtype, device)
+        self.uk_t = None                        # [heads, kv_rank, dim]: see finish_loading
+        self.rope = rope(spec.rot)
+
+    def named_parameters(self, p):
+        s = self.spec
+        yield p + "dq", self.a_proj[:s.q_rank]
+        yield p + "dkv", self.a_proj[s.q_rank:]
+        yield p + "dq.norm", self.q_norm
+        yield p + "dkv.norm", self.kv_norm
+        yield p + "uq", self.uq
+        yield p + "uk", self.ukv[:s.heads * s.dim]
+        yield p + "uv", self.ukv[s.heads * s.dim:]
+        yield p + "o", self.o
+
+    def finish_loading(self) -> None:
+        """Decode folds the key matrix into the query (q_h . W_h c = (W_h^T q_h) . c): keep each head's matrix transposed too."""
+        s = self.spec
+        self.uk_t = self.ukv[:s.heads * s.dim].view(s.heads, s.dim, s.kv_rank).transpose(1, 2).contiguous()
+
+    @property
+    def uv(self):
+        s = self.spec
+        return self.ukv[s.heads * s.dim:].view(s.heads, s.vdim, s.kv_rank)
+
+    def bytes_per_token(self) -> int:
+        return (self.spec.kv_rank + self.spec.rot_dim) * self.o.element_size()
+
+    def bytes_per_sequence(self) -> int:
+        return 0
+
+    def new_memory(self, num_blocks: int, block_size: int, num_slots: int):
+        return torch.zeros(num_blocks, block_size, self.spec.kv_rank + self.spec.rot_dim, dtype=self.o.dtype, device=self.o.device)
+
+    def forward(self, ops, h, cache, batch):
+        s = self.spec
+        proj = ops.linear(h, self.a_proj)
+        cq = ops.latent_prepare(proj, s.q_rank, s.kv_rank, self.q_norm, self.kv_norm, self.eps, self.rope, batch.positions,
+                                batch.slot_mapping, cache)
+        q = ops.linear(cq, self.uq)
+        return ops.linear(ops.latent_attention(q, self, cache, batch, self.rope, s), self.o)
+
+
+class Retention:
+    """Linear attention with a fixed decay per head and no denominator.  Kept per sequence: one fp32 matrix per head."""
+    recurrent = True
+
+    def __init__(self, spec, width: int, eps: float, dtype, device, rope):
+        self.spec, self.eps = spec, eps
+        H = spec.heads
+        self.qkvg = _empty((H * (2 * spec.dim + 2 * spec.vdim), width), dtype, device)
+        self.o = _empty((width, H * spec.vdim), dtype, device)
+        self.decay = torch.tensor(spec.decay, dtype=torch.float32, device=device)
+        self.rope = rope(spec.rot)
+
+    def named_parameters(self, p):
+        s, at = self.spec, 0
+        for name, d in (("q", s.dim), ("k", s.dim), ("v", s.vdim), ("g", s.vdim)):
+            yield p + name, self.qkvg[at:at + s.heads * d]
+            at += s.heads * d
+        yield p + "o", self.o
+
+    def finish_loading(self) -> None:
+        pass
+
+    def bytes_per_token(self) -> int:
+        return 0
+
+    def bytes_per_sequence(self) -> int:
+        return 4 * self.spec.heads * self.spec.dim * self.spec.vdim
+
+    def new_memory(self, num_blocks: int, block_size: int, num_slots: int):
+        s = self.spec
+        return torch.zeros(num_slots, s.heads, s.dim, s.vdim, dtype=torch.float32, device=self.o.device)
+
+    def forward(self, ops, h, state, batch):
+        y = ops.retention(ops.linear(h, self.qkvg), self.decay, state, batch, self.rope, self.spec, self.eps)
+        return ops.linear(y, self.o)
+
+
+class GatedFeedForward:
+    """down(silu(gate h) * (up h))"""
+
+    def __init__(self, spec, width: int, dtype, device):
+        self.ff = spec.ff
+        self.gate_up = _empty((2 * spec.ff, width), dtype, device)
+        self.down = _empty((width, spec.ff), dtype, device)
+
+    def named_parameters(self, p):
+        yield p + "gate", self.gate_up[:self.ff]
+        yield p + "up", self.gate_up[self.ff:]
+        yield p + "down", self.down
+
+    def forward(self, ops, h):
+        return ops.linear(ops.linear_silu_mul(h, self.gate_up), self.down)
+
+
+class RoutedFeedForward:
+    """Experts chosen per token by the largest sigmoid scores; the score multiplies the expert's input."""
+
+    def __init__(self, spec, width: int, dtype, device):
+        self.spec = spec
+        self.router = _empty((spec.experts, width), dtype, device)
+        self.gate_up = _empty((spec.experts, 2 * spec.ff, width), dtype, device)
+        self.down = _empty((spec.experts, width, spec.ff), dtype, device)
+
+    def named_parameters(self, p):
+        yield p + "router", self.router
+        for e in range(self.spec.experts):
+            yield f"{p}e{e}.gate", self.gate_up[e, :self.spec.ff]
+            yield f"{p}e{e}.up", self.gate_up[e, self.spec.ff:]
+            yield f"{p}e{e}.down", self.down[e]
+
+    def forward(self, ops, h):
+        return ops.moe(h, self.router, self.gate_up, self.down, self.spec.top)

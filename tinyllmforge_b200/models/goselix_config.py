@@ -1,0 +1,193 @@
+"""Configuration of Goselix, a decoder whose layers are listed one by one.
+
+``config.json`` gives, for every layer, the type and the sizes of its mixer (latent attention or retention) and its
+feed-forward (dense, mixture of experts, or none), optionally a range of layers that runs several times with the same
+weights (``loop``), and the model's vocabulary, width and norm constant.  Nothing here has a default taken from one
+checkpoint: a missing size is an error, an unknown key a warning.
+"""
+from __future__ import annotations
+
+import warnings
+from dataclasses import dataclass
+
+from ..config import parse_dtype
+
+
+def _take(d: dict, what: str, keys: dict) -> dict:
+    """The values of ``keys`` (name -> converter) in ``d``."""
+    missing = [k for k in keys if k not in d]
+    if missing:
+        raise ValueError(f"{what}: missing {missing}")
+    extra = sorted(set(d) - set(keys))
+    if extra:
+        warnings.warn(f"{what}: keys not used by this model: {extra}")
+    return {k: conv(d[k]) for k, conv in keys.items()}
+
+
+@dataclass(frozen=True)
+class Rotation:
+    """Pairs (i, i + dims / 2) of the first ``dims`` entries of a head, angle = position * base ** (-2 i / dims)."""
+    base: float
+    dims: int
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "Rotation":
+        r = cls(**_take(d, "rot", {"base": float, "dims": int}))
+        if r.dims < 0 or r.dims % 2:
+            raise ValueError("rot.dims must be even")
+        return r
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rot: Rotation
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "LatentAttentionSpec":
+        s = cls(**_take(d, "latent_attention", {"heads": int, "dim": int, "rot_dim": int, "vdim": int, "q_rank": int, "kv_rank": int,
+                                                "scale": float, "rot": Rotation.from_dict}))
+        if s.rot.dims != s.rot_dim:
+            raise ValueError("latent_attention: the whole rotated part is rotated (rot.dims == rot_dim)")
+        return s
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    rot: Rotation
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "RetentionSpec":
+        s = cls(**_take(d, "retention", {"heads": int, "dim": int, "vdim": int, "decay": lambda v: tuple(float(x) for x in v),
+                                         "rot": Rotation.from_dict}))
+        if len(s.decay) != s.heads:
+            raise ValueError("retention: one decay per head")
+        if not all(0.0 <= g <= 1.0 for g in s.decay):
+            raise ValueError("retention: decays lie between 0 and 1")
+        if s.rot.dims > s.dim:
+            raise ValueError("retention: rot.dims cannot exceed dim")
+        return s
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    ff: int
+
+
+@dataclass(frozen=True)
+class MoeSpec:
+    experts: int
+    top: int
+    ff: int
+
+
+def _mlp_from_dict(d):
+    if d is None:
+        return None
+    kind = d.get("kind")
+    if kind == "dense":
+        return DenseSpec(int(d["ff"]))
+    if kind == "moe":
+        router = _take(d["router"], "mlp.router", {"experts": int, "top": int})
+        spec = MoeSpec(router["experts"], router["top"], int(d["expert"]["ff"]))
+        if not 1 <= spec.top <= spec.experts:
+            raise ValueError("mlp.router: top must lie between 1 and experts")
+        return spec
+    raise ValueError(f"unknown feed-forward kind {kind!r}; known: dense, moe")
+
+
+MIXER_SPECS = {"latent_attention": LatentAttentionSpec, "retention": RetentionSpec}
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    type: str
+    mixer: object
+    mlp: object
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "LayerSpec":
+        if d.get("type") not in MIXER_SPECS:
+            raise ValueError(f"unknown layer type {d.get('type')!r}; known: {sorted(MIXER_SPECS)}")
+        return cls(d["type"], MIXER_SPECS[d["type"]].from_dict(d["mixer"]), _mlp_from_dict(d.get("mlp")))
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers start .. stop - 1 run ``times`` times in a row before the rest follow."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass
+class GoselixConfig:
+    vocab_size: int
+    hidden_size: int
+    rms_norm_eps: float
+    layers: tuple
+    loop: object = None
+    torch_dtype: str = "bfloat16"
+    eos_token_id: int = -1
+    max_position_embeddings: int = 1 << 20      # the design names no limit; rotary tables are built for max_model_len
+
+    quantizable = False
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "GoselixConfig":
+        for key in ("vocab", "width", "norm", "layers"):
+            if key not in d:
+                raise ValueError(f"Goselix config: missing {key!r}")
+        loop = d.get("loop")
+        cfg = cls(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), tuple(LayerSpec.from_dict(l) for l in d["layers"]),
+                  LoopSpec(**_take(loop, "loop", {"start": int, "stop": int, "times": int})) if loop else None,
+                  torch_dtype=str(d.get("torch_dtype") or d.get("dtype") or "bfloat16").replace("torch.", ""))
+        if d.get("eos_token_id") is not None:
+            eos = d["eos_token_id"]
+            cfg.eos_token_id = int(eos[0] if isinstance(eos, (list, tuple)) else eos)
+        if d.get("max_position_embeddings"):
+            cfg.max_position_embeddings = int(d["max_position_embeddings"])
+        cfg.validate()
+        return cfg
+
+    def validate(self) -> None:
+        if not self.layers:
+            raise ValueError("Goselix config: no layers")
+        if self.loop is not None and not (0 <= self.loop.start < self.loop.stop <= len(self.layers) and self.loop.times >= 1):
+            raise ValueError("Goselix config: loop must name a range of layers and at least one pass")
+
+    def validate_tp(self, size: int) -> None:
+        if size != 1:
+            raise ValueError("Goselix runs on one GPU (tensor_parallel_size=1)")
+
+    def layer_runs(self) -> list:
+        """[(layer, pass)] in the order of computation; pass is None for a layer outside the loop."""
+        n, loop = len(self.layers), self.loop
+        if loop is None:
+            return [(i, None) for i in range(n)]
+        return ([(i, None) for i in range(loop.start)]
+                + [(i, t) for t in range(loop.times) for i in range(loop.start, loop.stop)]
+                + [(i, None) for i in range(loop.stop, n)])
+
+    @property
+    def dtype(self):
+        return parse_dtype(self.torch_dtype)
+
+    @property
+    def num_recurrent_runs(self) -> int:
+        return sum(self.layers[i].type == "retention" for i, _ in self.layer_runs())
+
+    @property
+    def prefix_cacheable(self) -> bool:
+        """A recurrent state cannot be picked up in the middle of a prompt from cached blocks alone."""
+        return self.num_recurrent_runs == 0

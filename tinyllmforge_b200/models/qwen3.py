@@ -107,9 +107,35 @@ class Qwen3ForCausalLM:
                 total += t.numel() * t.element_size()
         return total
 
+    # ------------------------------------------------------------------ cache
+    def kv_block_bytes(self, block_size: int) -> int:
+        return 2 * len(self.layers) * block_size * self.num_kv_heads * self.head_dim * self.norm.element_size()
+
+    def state_bytes(self) -> int:
+        """Per-sequence state beside the paged cache: none."""
+        return 0
+
+    def bind_cache(self, num_blocks: int, block_size: int, num_slots: int = 0) -> None:
+        self.bind_kv_cache(torch.zeros(len(self.layers), 2, num_blocks, self.num_kv_heads, block_size, self.head_dim, dtype=self.dtype,
+                                       device=self.device))
+
+    def drop_cache(self) -> None:
+        self.kv_cache = None
+
     def bind_kv_cache(self, kv_cache: torch.Tensor) -> None:
         assert kv_cache.shape[0] == len(self.layers) and kv_cache.shape[1] == 2
         self.kv_cache = kv_cache
+
+    def finish_loading(self, config) -> None:
+        """What follows loading: norm folding (single GPU, bf16) or block-wise fp8 quantisation of the four projections."""
+        if (config.device == "cuda" and self.tp.size == 1 and config.quantization is None and config.dtype == torch.bfloat16
+                and config.extra.get("fold_norms", True) and not self.cfg.attention_bias):
+            self.fold_norm_weights()            # add + RMSNorm become GEMM epilogues
+        if config.quantization == "fp8_block":
+            from ..ops.quant import Fp8BlockWeight
+            for l in self.layers:               # embeddings and LM head stay bf16
+                for lin in (l.qkv_proj, l.o_proj, l.gate_up_proj, l.down_proj):
+                    lin.weight = Fp8BlockWeight.quantize(lin.weight)
 
     # ------------------------------------------------------------------ norm folding (single GPU, CUDA op set)
     def fold_norm_weights(self) -> None:
@@ -200,6 +226,10 @@ class Qwen3ForCausalLM:
         """This rank's logits shard for the last token of every sequence: ``[seqs, vocab / tp]``."""
         last = self.ops.select_rows(hidden, batch.last_index)
         return self.lm_head.forward(self.ops, last)
+
+    def logits_at(self, batch, rows: torch.Tensor) -> torch.Tensor:
+        """Logits of the batch's tokens ``rows`` (an index tensor)."""
+        return self.lm_head.forward(self.ops, self.ops.select_rows(self.forward(batch), rows))
 
     def sample(self, logits: torch.Tensor, batch) -> torch.Tensor:
         return self.ops.sample(logits, batch, self.lm_head.vocab_start, self.tp)

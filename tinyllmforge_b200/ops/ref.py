@@ -42,12 +42,13 @@ def add_rms_norm(x: torch.Tensor, residual: torch.Tensor | None, weight: torch.T
 
 
 # ----------------------------------------------------------------------------- rotary
-def rope_table(max_positions: int, head_dim: int, theta: float, device="cpu") -> torch.Tensor:
-    """fp32 table ``[max_positions, head_dim]`` = cat(cos, sin) of pos * theta^(-2i/d)."""
-    inv_freq = 1.0 / (theta ** (torch.arange(0, head_dim, 2, dtype=torch.float32) / head_dim))
-    t = torch.arange(max_positions, dtype=torch.float32)
+def rope_table(max_positions: int, head_dim: int, theta: float, device="cpu", angle_dtype=torch.float32) -> torch.Tensor:
+    """fp32 table ``[max_positions, head_dim]`` = cat(cos, sin) of pos * theta^(-2i/d).  ``angle_dtype=torch.float64``: the
+    angles carry no rounding of their own (in fp32 an angle of 1e4 rad is off by up to 5e-4)."""
+    inv_freq = 1.0 / (theta ** (torch.arange(0, head_dim, 2, dtype=angle_dtype) / max(head_dim, 1)))
+    t = torch.arange(max_positions, dtype=angle_dtype)
     freqs = torch.outer(t, inv_freq)
-    return torch.cat((freqs.cos(), freqs.sin()), dim=-1).to(device)
+    return torch.cat((freqs.cos(), freqs.sin()), dim=-1).float().to(device)
 
 
 def apply_rope(x: torch.Tensor, positions: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
@@ -147,6 +148,113 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_
         o = torch.bmm(p, v).reshape(H, ql, d).permute(1, 0, 2)
         out[a:b] = o.to(q.dtype)
     return out.reshape(T, H * d)
+
+
+# ----------------------------------------------------------------------------- 32-bit residual stream
+def stream_update(x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None):
+    """The residual stream between two layers: x += a + b (the two branches of a parallel layer), += embed[ids], += vec,
+    all in fp32; then one RMS norm per weight in ``norms``, each rounded once to ``dtype``.  ``start``: x begins at zero.
+    ``rows``: norms of these rows only, and x is left as it was."""
+    s = torch.zeros_like(x) if start else x
+    for term in (a, b):
+        if term is not None:
+            s = s + term.float()
+    if ids is not None:
+        s = s + F.embedding(ids.long(), embed).float()
+    if vec is not None:
+        s = s + vec.float()
+    if rows is None:
+        x.copy_(s)
+    else:
+        s = s[rows.long()]
+    inv = torch.rsqrt(s.pow(2).mean(dim=-1, keepdim=True) + eps)
+    return [(s * inv * w.float()).to(dtype) for w in norms]
+
+
+def apply_partial_rope(x: torch.Tensor, positions: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+    """fp32 [T, heads, d]; the first ``table.shape[1]`` entries of every head are rotated, the rest pass."""
+    n = table.shape[1]
+    return torch.cat((apply_rope(x[..., :n].float(), positions, table), x[..., n:].float()), dim=-1)
+
+
+# ----------------------------------------------------------------------------- latent attention
+def latent_prepare(proj, q_rank, kv_rank, q_norm, kv_norm, eps, table, positions, slot_mapping, cache):
+    """proj [T, q_rank + kv_rank + rot] -> the normed query latent; the normed key/value latent and the rotated shared key
+    part go to the paged cache [blocks, block_size, kv_rank + rot]."""
+    def norm(v, w):
+        v = v.float()
+        return v * torch.rsqrt(v.pow(2).mean(dim=-1, keepdim=True) + eps) * w.float()
+    cq = norm(proj[:, :q_rank], q_norm).to(proj.dtype)
+    c = norm(proj[:, q_rank:q_rank + kv_rank], kv_norm)
+    kr = apply_partial_rope(proj[:, None, q_rank + kv_rank:], positions, table)[:, 0]
+    slots = slot_mapping.long()
+    keep = slots >= 0
+    flat = cache.view(-1, cache.shape[-1])
+    flat[slots[keep]] = torch.cat((c, kr), dim=-1)[keep].to(cache.dtype)
+    return cq
+
+
+def latent_attention(q, wkv, cache, batch, table, spec):
+    """q [T, heads * (dim + rot)] before rotation; wkv [heads * (dim + vdim), kv_rank] = key rows, then value rows."""
+    H, d, r, dv, R = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
+    T = q.shape[0]
+    q = q.view(T, H, d + r).float()
+    q = torch.cat((q[..., :d], apply_partial_rope(q[..., d:], batch.positions, table)), dim=-1)
+    out = torch.zeros(T, H, dv, dtype=cache.dtype, device=cache.device)
+    w = wkv.float()
+    cu, lens = batch.cu_seqlens_q.tolist(), batch.context_lens.tolist()
+    bs = cache.shape[1]
+    for s in range(batch.num_seqs):
+        a, b = cu[s], cu[s + 1]
+        n = lens[s]
+        rows = cache[batch.block_tables[s, :(n + bs - 1) // bs].long()].reshape(-1, R + r)[:n].float()
+        kv = rows[:, :R] @ w.t()
+        k = torch.cat((kv[:, :H * d].view(n, H, d), rows[:, None, R:].expand(n, H, r)), dim=-1)
+        scores = torch.einsum("qhd,khd->hqk", q[a:b], k) * spec.scale
+        pos = batch.positions[a:b].long()
+        scores.masked_fill_(torch.arange(n, device=q.device)[None, None, :] > pos[None, :, None], float("-inf"))
+        out[a:b] = torch.einsum("hqk,khe->qhe", torch.softmax(scores, dim=-1), kv[:, H * d:].view(n, H, dv)).to(out.dtype)
+    return out.view(T, H * dv)
+
+
+# ----------------------------------------------------------------------------- retention
+def retention(qkvg, decay, state, batch, table, spec, eps):
+    """qkvg [T, heads * (2 dim + 2 vdim)] = q, k, v, gate.  state [slots, heads, dim, vdim] fp32 is read and updated in place
+    (a sequence's first token starts from zero).  Returns the gated, per-head normed output [T, heads * vdim]."""
+    H, d, dv = spec.heads, spec.dim, spec.vdim
+    T = qkvg.shape[0]
+    q, k, v, g = qkvg.float().split([H * d, H * d, H * dv, H * dv], dim=-1)
+    q = apply_partial_rope(q.reshape(T, H, d), batch.positions, table)
+    k = apply_partial_rope(k.reshape(T, H, d), batch.positions, table) * d ** -0.5
+    v = v.reshape(T, H, dv)
+    o = torch.zeros(T, H, dv, device=q.device)
+    cu, slots = batch.cu_seqlens_q.tolist(), batch.state_slots.tolist()
+    keep = decay.view(H, 1, 1)
+    for s in range(batch.num_seqs):
+        a, b = cu[s], cu[s + 1]
+        if int(batch.positions[a]) == 0:
+            state[slots[s]].zero_()
+        S = state[slots[s]]
+        for t in range(a, b):
+            S.mul_(keep).add_(k[t][:, :, None] * v[t][:, None, :])
+            o[t] = torch.einsum("hde,hd->he", S, q[t])
+    o = o * torch.rsqrt(o.pow(2).mean(dim=-1, keepdim=True) + eps)
+    return (o.reshape(T, H * dv) * F.silu(g)).to(qkvg.dtype)
+
+
+# ----------------------------------------------------------------------------- mixture of experts
+def moe(h, router, gate_up, down, top):
+    """Sigmoid-scored top-k experts; the score multiplies the expert's INPUT.  gate_up [experts, 2 ff, width], down [experts,
+    width, ff]."""
+    score = torch.sigmoid(h.float() @ router.float().t())
+    w, e = torch.sort(score, dim=-1, descending=True, stable=True)
+    out = torch.zeros(h.shape[0], down.shape[1], device=h.device)
+    for j in range(top):
+        for x in e[:, j].unique().tolist():
+            rows = (e[:, j] == x).nonzero()[:, 0]
+            hx = (h[rows].float() * w[rows, j, None]).to(h.dtype)
+            out[rows] += linear(linear_silu_mul(hx, gate_up[x]), down[x]).float()
+    return out
 
 
 # ----------------------------------------------------------------------------- embedding
@@ -264,6 +372,14 @@ class RefOps:
     add_rms_norm = staticmethod(add_rms_norm)
     rms_norm = staticmethod(rms_norm)
     qk_norm_rope_store = staticmethod(qk_norm_rope_store)
+    stream_update = staticmethod(stream_update)
+    latent_prepare = staticmethod(latent_prepare)
+    retention = staticmethod(retention)
+    moe = staticmethod(moe)
+
+    @staticmethod
+    def latent_attention(q, weights, cache, batch, table, spec):
+        return latent_attention(q, weights.ukv, cache, batch, table, spec)
 
     @staticmethod
     def attention(q, k_cache, v_cache, batch, scale):

@@ -29,7 +29,7 @@ def load_weights(model, path: str, strict: bool = True) -> None:
         with safe_open(file, "pt", "cpu") as f:
             for name in f.keys():
                 if name not in wanted:
-                    if name == "lm_head.weight" and model.cfg.tie_word_embeddings:
+                    if name == "lm_head.weight" and getattr(model.cfg, "tie_word_embeddings", False):
                         continue
                     if strict and "rotary_emb.inv_freq" not in name:
                         raise KeyError(f"unexpected tensor {name!r} in {file}")
@@ -59,7 +59,7 @@ def init_dummy_weights(model, seed: int = 0, std: float = 0.02) -> None:
     gen = torch.Generator(device=dev)
     gen.manual_seed(seed * 1000003 + model.tp.rank)
     for name, param, owner, _ in model.named_parameters():
-        if owner is None:
+        if owner is None and param.dim() == 1:
             param.fill_(1.0)
         elif name.endswith(".bias"):
             param.zero_()
