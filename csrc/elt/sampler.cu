@@ -35,9 +35,16 @@ __device__ __forceinline__ void load_group(const __nv_bfloat16* lrow, int g, int
   }
 }
 
+__device__ __forceinline__ void load_group(const float* lrow, int g, int vocab_start, int vocab, bool, float lv[kSampleGroup]) {
+  const int local0 = g * kSampleGroup - vocab_start;
+#pragma unroll
+  for (int j = 0; j < kSampleGroup; ++j) lv[j] = (local0 + j >= 0 && local0 + j < vocab) ? lrow[local0 + j] : -INFINITY;
+}
+
 // header: the packed step buffer's first words; [9] = step index, [10], [11] = seed low / high.
+template <typename L>
 __global__ void __launch_bounds__(kSampleThreads) sample_partial_kernel(
-    const __nv_bfloat16* __restrict__ logits, int ld, int vocab, int vocab_start, const float* __restrict__ temps,
+    const L* __restrict__ logits, int ld, int vocab, int vocab_start, const float* __restrict__ temps,
     const int* __restrict__ header, float* __restrict__ part_v, int* __restrict__ part_i, int nsplit) {
   __shared__ float sv[kSampleThreads / 32];
   __shared__ int si[kSampleThreads / 32];
@@ -55,7 +62,7 @@ __global__ void __launch_bounds__(kSampleThreads) sample_partial_kernel(
   const int per = (ngroups + nsplit - 1) / nsplit;
   const int gb = g_first + split * per;
   const int ge = min(gb + per, g_last + 1);
-  const __nv_bfloat16* lrow = logits + static_cast<size_t>(row) * ld;
+  const L* lrow = logits + static_cast<size_t>(row) * ld;
   const bool aligned = (reinterpret_cast<uintptr_t>(lrow) & 15) == 0 && (vocab_start & 7) == 0;   // groups start on 16-byte boundaries
   // level 1: every thread scores the groups it visits; `i` of the pair is the group index here
   Best best{-INFINITY, 0x7fffffff};
@@ -121,15 +128,18 @@ extern "C" int forge_sample_nsplit(int rows, int vocab) {
   return n < 1 ? 1 : (n > 64 ? 64 : n);
 }
 
-// logits [rows, vocab] bf16 (row stride ld); part_* are scratch of rows * nsplit entries.
-extern "C" int forge_sample(const void* logits, int ld, int rows, int vocab, int vocab_start, const float* temps,
+// logits [rows, vocab] bf16, or fp32 when the model runs in 32-bit (row stride ld); part_* are scratch of rows * nsplit entries.
+extern "C" int forge_sample(const void* logits, int fp32, int ld, int rows, int vocab, int vocab_start, const float* temps,
                             const int* header, float* part_v, int* part_i, int nsplit, int* out_i, float* out_v,
                             cudaStream_t stream) {
   if (rows <= 0) return 0;
   dim3 grid(nsplit, rows);
-  if (launch_kernel(sample_partial_kernel, grid, dim3(kSampleThreads), 0, stream, 0, static_cast<const __nv_bfloat16*>(logits), ld,
-                    vocab, vocab_start, temps, header, part_v, part_i, nsplit) != cudaSuccess)
-    return -2;
+  const cudaError_t e =
+      fp32 ? launch_kernel(sample_partial_kernel<float>, grid, dim3(kSampleThreads), 0, stream, 0, static_cast<const float*>(logits), ld,
+                           vocab, vocab_start, temps, header, part_v, part_i, nsplit)
+           : launch_kernel(sample_partial_kernel<__nv_bfloat16>, grid, dim3(kSampleThreads), 0, stream, 0,
+                           static_cast<const __nv_bfloat16*>(logits), ld, vocab, vocab_start, temps, header, part_v, part_i, nsplit);
+  if (e != cudaSuccess) return -2;
   return launch_kernel(sample_merge_kernel, dim3((rows + 3) / 4), dim3(128), 0, stream, 0, static_cast<const float*>(part_v),
                        static_cast<const int*>(part_i), nsplit, rows, out_i, out_v) == cudaSuccess ? 0 : -2;
 }

@@ -1,0 +1,174 @@
+// The fp32 residual stream between two layers of a decoder with parallel branches, in one pass over a row:
+//
+//   x += a + b                    both branches of the layer before (b dense, or the sum of a token's expert outputs)
+//   x += embed[id], x += vec      ahead of a pass of a looped range of layers (and at the start, where x begins at zero)
+//   h_i = rms_norm(x) * w_i       the norms of the layer after (they share the row's mean square)
+//
+// One CTA per row; the row stays in shared memory between the two halves.  With `rows` only those rows are normed and x is
+// left as it was (the last norm of a step: only rows whose logits are wanted).
+#include "../include/launch.cuh"
+#include "../include/scalar.cuh"
+
+namespace forge {
+
+template <typename T>
+struct StreamArgs {
+  float* x;
+  const T* a;
+  const T* b;
+  const int* b_rows;     // null: b is [rows][W]; else b is indexed by b_rows[row * top + j], j < top
+  int top;
+  const int* ids;
+  const T* embed;
+  int vocab;
+  const T* vec;
+  const T* w1;
+  const T* w2;
+  T* h1;
+  T* h2;
+  const int* rows;
+  int n_rows, W, start;
+  float eps;
+};
+
+template <typename T, int N>
+__global__ void __launch_bounds__(256) stream_update_kernel(const StreamArgs<T> p) {
+  extern __shared__ float srow[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  int r = blockIdx.x;
+  if (p.rows != nullptr) {
+    r = p.rows[r];
+    r = r < 0 ? 0 : (r >= p.n_rows ? p.n_rows - 1 : r);
+  }
+  const size_t base = static_cast<size_t>(r) * p.W;
+  const T* emb = nullptr;
+  if (p.ids != nullptr) {
+    int id = p.ids[r];
+    id = id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id);
+    emb = p.embed + static_cast<size_t>(id) * p.W;
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x * N; i < p.W; i += blockDim.x * N) {
+    float s[N], v[N];
+    if (p.start) {
+#pragma unroll
+      for (int e = 0; e < N; ++e) s[e] = 0.f;
+    } else {
+      load_n<N>(p.x + base + i, s);
+    }
+    if (p.a != nullptr) {
+      load_n<N>(p.a + base + i, v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) s[e] += v[e];
+    }
+    if (p.b != nullptr) {
+      if (p.b_rows == nullptr) {
+        load_n<N>(p.b + base + i, v);
+#pragma unroll
+        for (int e = 0; e < N; ++e) s[e] += v[e];
+      } else {
+        for (int j = 0; j < p.top; ++j) {
+          load_n<N>(p.b + static_cast<size_t>(p.b_rows[static_cast<size_t>(r) * p.top + j]) * p.W + i, v);
+#pragma unroll
+          for (int e = 0; e < N; ++e) s[e] += v[e];
+        }
+      }
+    }
+    if (emb != nullptr) {
+      load_n<N>(emb + i, v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) s[e] += v[e];
+    }
+    if (p.vec != nullptr) {
+      load_n<N>(p.vec + i, v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) s[e] += v[e];
+    }
+    if (p.rows == nullptr) store_n<N>(p.x + base + i, s);
+#pragma unroll
+    for (int e = 0; e < N; ++e) ss += s[e] * s[e];
+    store_n<N>(srow + i, s);
+  }
+  if (p.w1 == nullptr) return;
+  const float inv = rsqrtf(block_sum_f(ss, red) / static_cast<float>(p.W) + p.eps);
+  const size_t out = static_cast<size_t>(blockIdx.x) * p.W;
+  for (int i = threadIdx.x * N; i < p.W; i += blockDim.x * N) {
+    float s[N], w[N], y[N];
+    load_n<N>(srow + i, s);
+    load_n<N>(p.w1 + i, w);
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      s[e] *= inv;
+      y[e] = s[e] * w[e];
+    }
+    store_n<N>(p.h1 + out + i, y);
+    if (p.w2 != nullptr) {
+      load_n<N>(p.w2 + i, w);
+#pragma unroll
+      for (int e = 0; e < N; ++e) y[e] = s[e] * w[e];
+      store_n<N>(p.h2 + out + i, y);
+    }
+  }
+}
+
+template <typename T>
+static int stream_update(int out_rows, const StreamArgs<T>& p, cudaStream_t stream) {
+  const size_t smem = static_cast<size_t>(p.W) * 4;
+  if (smem > 200 * 1024) return -1;
+  const bool v4 = (p.W & 3) == 0;
+  int threads = ((p.W / (v4 ? 4 : 1) + 31) / 32) * 32;
+  threads = threads < 32 ? 32 : (threads > 256 ? 256 : threads);
+  if (v4) {
+    auto k = stream_update_kernel<T, 4>;
+    FORGE_ENSURE_DYN_SMEM(k, 200 * 1024);
+    return launch_kernel(k, dim3(out_rows), dim3(threads), smem, stream, 0, p) == cudaSuccess ? 0 : -2;
+  }
+  auto k = stream_update_kernel<T, 1>;
+  FORGE_ENSURE_DYN_SMEM(k, 200 * 1024);
+  return launch_kernel(k, dim3(out_rows), dim3(threads), smem, stream, 0, p) == cudaSuccess ? 0 : -2;
+}
+
+extern "C" int forge_stream_update(int fp32, float* x, const void* a, const void* b, const int* b_rows, int top, const int* ids,
+                                   const void* embed, int vocab, const void* vec, const void* w1, const void* w2, void* h1, void* h2,
+                                   const int* rows, int out_rows, int n_rows, int W, int start, float eps, cudaStream_t stream) {
+  if (out_rows <= 0) return 0;
+  if (fp32) {
+    using T = float;
+    const StreamArgs<T> p = {x, static_cast<const T*>(a), static_cast<const T*>(b), b_rows, top, ids, static_cast<const T*>(embed), vocab,
+                             static_cast<const T*>(vec), static_cast<const T*>(w1), static_cast<const T*>(w2), static_cast<T*>(h1),
+                             static_cast<T*>(h2), rows, n_rows, W, start, eps};
+    return stream_update<T>(out_rows, p, stream);
+  }
+  using T = bf16;
+  const StreamArgs<T> p = {x, static_cast<const T*>(a), static_cast<const T*>(b), b_rows, top, ids, static_cast<const T*>(embed), vocab,
+                           static_cast<const T*>(vec), static_cast<const T*>(w1), static_cast<const T*>(w2), static_cast<T*>(h1),
+                           static_cast<T*>(h2), rows, n_rows, W, start, eps};
+  return stream_update<T>(out_rows, p, stream);
+}
+
+// out[r, :I] = silu(x[r, :I]) * x[r, I:2I], any I, bf16 or fp32 (the fused epilogue of the tcgen05 GEMMs needs no such pass).
+template <typename T>
+__global__ void __launch_bounds__(256) silu_mul_any_kernel(const T* __restrict__ x, T* __restrict__ out, long long rows, int I) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long idx = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; idx < rows * I;
+       idx += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = idx / I;
+    const int c = static_cast<int>(idx % I);
+    store_f(out + idx, silu_t<T>(load_f(x + r * 2 * I + c)) * load_f(x + r * 2 * I + I + c));
+  }
+}
+
+extern "C" int forge_silu_mul_any(int fp32, const void* x, void* out, long long rows, int I, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  long long grid = (rows * I + 255) / 256;
+  if (grid > device_sm_count() * 16) grid = device_sm_count() * 16;
+  const dim3 g(static_cast<unsigned>(grid));
+  if (fp32)
+    return launch_kernel(silu_mul_any_kernel<float>, g, dim3(256), 0, stream, 0, static_cast<const float*>(x), static_cast<float*>(out), rows, I) == cudaSuccess ? 0 : -2;
+  return launch_kernel(silu_mul_any_kernel<bf16>, g, dim3(256), 0, stream, 0, static_cast<const bf16*>(x), static_cast<bf16*>(out), rows, I) == cudaSuccess ? 0 : -2;
+}
+
+}  // namespace forge

@@ -68,7 +68,7 @@ int forge_embedding(const int* ids, const void* w, void* out, int T, int H, int 
 int forge_gather_rows(const int* idx, const void* x, void* out, int S, int H, int x_rows, cudaStream_t stream);
 int forge_feed_tokens(int* ids, const int* src_rows, const int* prev_tokens, int n, int prev_n, cudaStream_t stream);
 int forge_sample_nsplit(int rows, int vocab);
-int forge_sample(const void* logits, int ld, int rows, int vocab, int vocab_start, const float* temps, const int* header,
+int forge_sample(const void* logits, int fp32, int ld, int rows, int vocab, int vocab_start, const float* temps, const int* header,
                  float* part_v, int* part_i, int nsplit, int* out_i, float* out_v, cudaStream_t stream);
 int forge_sample_merge_ranks(const float* vals, const int* ids, int ranks, int rows, int* out_i, cudaStream_t stream);
 int forge_decode_attention(const void* q, const void* kc, const void* vc, const int* bt, const int* lens, void* out,
@@ -326,10 +326,12 @@ void feed_tokens(Tensor& ids, const Tensor& src_rows, const Tensor& prev_tokens)
 
 int64_t sample_nsplit(int64_t rows, int64_t vocab) { return forge_sample_nsplit(static_cast<int>(rows), static_cast<int>(vocab)); }
 
-// logits [rows, vocab] bf16; header = first words of the packed step buffer (step index, seed) on the device.
+// logits [rows, vocab] bf16 or fp32; header = first words of the packed step buffer (step index, seed) on the device.
 void sample(const Tensor& logits, int64_t vocab_start, const Tensor& temps, const Tensor& header, Tensor& part_v, Tensor& part_i,
             Tensor& out_i, const c10::optional<Tensor>& out_v) {
-  CHECK_BF16(logits); CHECK_CUDA_CONTIG(temps); CHECK_F32(temps); CHECK_CUDA_CONTIG(header); CHECK_I32(header);
+  const bool fp32 = logits.scalar_type() == at::kFloat;
+  if (!fp32) CHECK_BF16(logits);
+  CHECK_CUDA_CONTIG(temps); CHECK_F32(temps); CHECK_CUDA_CONTIG(header); CHECK_I32(header);
   CHECK_CUDA_CONTIG(part_v); CHECK_F32(part_v); CHECK_CUDA_CONTIG(part_i); CHECK_I32(part_i); CHECK_CUDA_CONTIG(out_i); CHECK_I32(out_i);
   TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1, "logits must be [rows, vocab]");
   const int64_t rows = logits.size(0), vocab = logits.size(1);
@@ -339,7 +341,7 @@ void sample(const Tensor& logits, int64_t vocab_start, const Tensor& temps, cons
   float* ov = nullptr;
   if (out_v.has_value()) { CHECK_CUDA_CONTIG(*out_v); CHECK_F32(*out_v); TORCH_CHECK(out_v->numel() >= rows); ov = out_v->data_ptr<float>(); }
   const c10::cuda::CUDAGuard guard(logits.device());
-  check(forge_sample(logits.data_ptr(), static_cast<int>(logits.stride(0)), static_cast<int>(rows), static_cast<int>(vocab),
+  check(forge_sample(logits.data_ptr(), fp32 ? 1 : 0, static_cast<int>(logits.stride(0)), static_cast<int>(rows), static_cast<int>(vocab),
                      static_cast<int>(vocab_start), temps.data_ptr<float>(), header.data_ptr<int>(), part_v.data_ptr<float>(),
                      part_i.data_ptr<int>(), nsplit, out_i.data_ptr<int>(), ov, stream_of(logits)),
         "forge_sample");
@@ -665,8 +667,11 @@ void tp_sample_pairs(const Tensor& vals, const Tensor& ids, int64_t tp_rank, con
 
 }  // namespace
 
+void register_mixers(pybind11::module& m);      // bindings_mixers.cpp
+
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.doc() = "tinyllmforge_b200 sm_100a kernels";
+  register_mixers(m);
   m.def("gemm", &gemm);
   m.def("gemm_fused", &gemm_fused);
   m.def("gemm_sample", &gemm_sample);

@@ -1,0 +1,289 @@
+// Bindings of the ops of decoders with an fp32 residual stream, latent attention, retention and expert layers.  As in
+// bindings.cpp every argument is checked here (device, dtype, contiguity, shapes), so a malformed call raises in Python
+// instead of reaching a kernel.
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/extension.h>
+
+#include <cstdint>
+
+extern "C" {
+int forge_stream_update(int fp32, float* x, const void* a, const void* b, const int* b_rows, int top, const int* ids, const void* embed,
+                        int vocab, const void* vec, const void* w1, const void* w2, void* h1, void* h2, const int* rows, int out_rows,
+                        int n_rows, int W, int start, float eps, cudaStream_t stream);
+int forge_silu_mul_any(int fp32, const void* x, void* out, long long rows, int I, cudaStream_t stream);
+int forge_gemm_simt(int fp32, const void* x, long long ldx, long long x_batch, const void* w, long long ldw, long long w_batch, void* out,
+                    long long ldo, long long o_batch, int M, int N, int K, int batch, const int* tile_expert, cudaStream_t stream);
+int forge_latent_prepare(int fp32, const void* proj, int T, int q_rank, int kv_rank, int rot, const void* qw, const void* kw, float eps,
+                         const float* rope, int rope_rows, const int* positions, const int* slots, void* cq, void* cache,
+                         long long num_slots, unsigned* status, cudaStream_t stream);
+int forge_latent_rotate_q(int fp32, const void* q, void* qa, int tokens, int heads, int dim, int rot, int kv_rank, const float* rope,
+                          int rope_rows, const int* positions, cudaStream_t stream);
+int forge_latent_attend_any(int fp32, const void* qa, const void* cache, void* o, int tok0, int tokens, const int* cu, int num_seqs,
+                            const int* positions, const int* block_tables, int table_width, int num_blocks, int block_size, int heads,
+                            int kv_rank, int rot, float scale, unsigned* status, cudaStream_t stream);
+int forge_retention_decode(int fp32, const void* qkvg, int ld, const float* decay, float* state, const int* slots, const int* positions,
+                           const float* rope, int rope_rows, int rd, int seqs, int heads, int dk, int dv, int num_slots, void* y, float eps,
+                           unsigned* status, cudaStream_t stream);
+int forge_retention_scan(int fp32, const void* qkvg, int ld, const float* decay, float* state, const int* slots, const int* positions,
+                         const float* rope, int rope_rows, int rd, const int* cu, int seqs, int heads, int dk, int dv, int num_slots,
+                         float* o, unsigned* status, cudaStream_t stream);
+int forge_retention_gate(int fp32, const float* o, const void* qkvg, int ld, int gate_at, void* y, int tok0, int tokens, int heads, int dv,
+                         float eps, cudaStream_t stream);
+int forge_router(int fp32, const void* h, const void* w, int T, int W, int E, int top, int* experts, float* weights, cudaStream_t stream);
+int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles, cudaStream_t stream);
+int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs, cudaStream_t stream);
+}
+
+namespace {
+
+using torch::Tensor;
+using OptTensor = c10::optional<Tensor>;
+
+void check_rc(int rc, const char* what) { TORCH_CHECK(rc == 0, what, " failed with code ", rc); }
+cudaStream_t stream_of(const Tensor& t) { return at::cuda::getCurrentCUDAStream(t.get_device()).stream(); }
+unsigned* status_word(const Tensor& status) {
+  TORCH_CHECK(status.is_cuda() && status.scalar_type() == at::kInt && status.numel() >= 1, "status must be a CUDA int32 tensor");
+  return reinterpret_cast<unsigned*>(status.data_ptr<int>());
+}
+// 1: fp32, 0: bf16
+int elem(const Tensor& t) {
+  TORCH_CHECK(t.scalar_type() == at::kFloat || t.scalar_type() == at::kBFloat16, "element type must be bfloat16 or float32");
+  return t.scalar_type() == at::kFloat ? 1 : 0;
+}
+void need(const Tensor& t, at::ScalarType dtype, int64_t min_numel, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.scalar_type() == dtype, what, ": contiguous CUDA tensor of the right type expected");
+  TORCH_CHECK(t.numel() >= min_numel, what, ": too few elements (", t.numel(), " of ", min_numel, ")");
+}
+const int* ints(const Tensor& t, int64_t n, const char* what) {
+  need(t, at::kInt, n, what);
+  return t.data_ptr<int>();
+}
+float* floats(const Tensor& t, int64_t n, const char* what) {
+  need(t, at::kFloat, n, what);
+  return t.data_ptr<float>();
+}
+void* data(const Tensor& t, at::ScalarType dtype, int64_t n, const char* what) {
+  need(t, dtype, n, what);
+  return t.data_ptr();
+}
+int i32(int64_t v) {
+  TORCH_CHECK(v >= INT32_MIN && v <= INT32_MAX, "value does not fit 32 bits");
+  return static_cast<int>(v);
+}
+
+// x fp32 [rows, W]; a, b, embed, vec, w1, w2, h1, h2 of one element type.  b_rows (int32 [rows, top]): b is a buffer of expert
+// outputs whose rows b_rows[r, :] are summed.  rows (int32): norms of these rows only, x unchanged.
+void stream_update(Tensor& x, const OptTensor& a, const OptTensor& b, const OptTensor& b_rows, const OptTensor& ids, const OptTensor& embed,
+                   const OptTensor& vec, const OptTensor& w1, const OptTensor& w2, const OptTensor& h1, const OptTensor& h2,
+                   const OptTensor& rows, bool start, double eps, bool fp32) {
+  TORCH_CHECK(x.dim() == 2, "stream_update: x must be [rows, width]");
+  const int64_t R = x.size(0), W = x.size(1);
+  const auto dt = fp32 ? at::kFloat : at::kBFloat16;
+  float* xp = floats(x, R * W, "x");
+  const void *ap = nullptr, *bp = nullptr, *ep = nullptr, *vp = nullptr, *w1p = nullptr, *w2p = nullptr;
+  void *h1p = nullptr, *h2p = nullptr;
+  const int *brp = nullptr, *idp = nullptr, *rp = nullptr;
+  int64_t top = 0, vocab = 0, out_rows = R;
+  if (rows.has_value()) { rp = ints(*rows, 0, "rows"); out_rows = rows->numel(); }
+  if (a.has_value()) ap = data(*a, dt, R * W, "a");
+  if (b.has_value()) {
+    if (b_rows.has_value()) {
+      TORCH_CHECK(b_rows->dim() == 2 && b_rows->size(0) == R && b->dim() == 2 && b->size(1) == W, "stream_update: routed b");
+      top = b_rows->size(1);
+      brp = ints(*b_rows, R * top, "b_rows");
+      bp = data(*b, dt, W, "b");
+    } else {
+      bp = data(*b, dt, R * W, "b");
+    }
+  }
+  if (ids.has_value()) {
+    TORCH_CHECK(embed.has_value() && embed->dim() == 2 && embed->size(1) == W, "stream_update: embed");
+    idp = ints(*ids, R, "ids");
+    vocab = embed->size(0);
+    ep = data(*embed, dt, W, "embed");
+  }
+  if (vec.has_value()) vp = data(*vec, dt, W, "vec");
+  if (w1.has_value()) {
+    w1p = data(*w1, dt, W, "w1");
+    TORCH_CHECK(h1.has_value(), "stream_update: h1");
+    h1p = data(*h1, dt, out_rows * W, "h1");
+  }
+  if (w2.has_value()) {
+    TORCH_CHECK(w1.has_value() && h2.has_value(), "stream_update: h2");
+    w2p = data(*w2, dt, W, "w2");
+    h2p = data(*h2, dt, out_rows * W, "h2");
+  }
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_stream_update(fp32, xp, ap, bp, brp, i32(top), idp, ep, i32(vocab), vp, w1p, w2p, h1p, h2p, rp, i32(out_rows), i32(R), i32(W),
+                               start ? 1 : 0, static_cast<float>(eps), stream_of(x)),
+           "forge_stream_update");
+}
+
+void silu_mul_any(const Tensor& x, Tensor& out) {
+  const int f = elem(x);
+  TORCH_CHECK(x.dim() == 2 && x.size(1) % 2 == 0, "silu_mul_any: x [rows, 2 I]");
+  const int64_t rows = x.size(0), I = x.size(1) / 2;
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_silu_mul_any(f, data(x, x.scalar_type(), rows * 2 * I, "x"), data(out, x.scalar_type(), rows * I, "out"), rows, i32(I), stream_of(x)),
+           "forge_silu_mul_any");
+}
+
+// out[b] = x[b] w[b]^T for 3-D views [batch, M, K], [batch, N, K], [batch, M, N] with unit inner strides (2-D: one product).
+// tile_expert: w is [experts, N, K] and the 64-row tile i of the 2-D x uses matrix tile_expert[i].
+void gemm_simt(const Tensor& x, const Tensor& w, Tensor& out, const OptTensor& tile_expert) {
+  const int f = elem(x);
+  TORCH_CHECK(x.is_cuda() && w.is_cuda() && out.is_cuda() && w.scalar_type() == x.scalar_type() && out.scalar_type() == x.scalar_type(), "gemm_simt: operands");
+  TORCH_CHECK(x.dim() == out.dim() && (x.dim() == 2 || x.dim() == 3), "gemm_simt: ranks");
+  const bool three = x.dim() == 3, experts = tile_expert.has_value();
+  TORCH_CHECK(w.dim() == (three || experts ? 3 : 2) && !(three && experts), "gemm_simt: rank of w");
+  const int64_t batch = three ? x.size(0) : 1, M = x.size(-2), K = x.size(-1), N = w.size(-2);
+  TORCH_CHECK(w.size(-1) == K && out.size(-2) == M && out.size(-1) == N && (!three || (w.size(0) == batch && out.size(0) == batch)), "gemm_simt: shapes");
+  TORCH_CHECK(x.stride(-1) == 1 && w.stride(-1) == 1 && out.stride(-1) == 1, "gemm_simt: inner strides must be 1");
+  const int* te = nullptr;
+  if (experts) te = ints(*tile_expert, (M + 63) / 64, "tile_expert");
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_gemm_simt(f, x.data_ptr(), x.stride(-2), three ? x.stride(0) : 0, w.data_ptr(), w.stride(-2), w.dim() == 3 ? w.stride(0) : 0,
+                           out.data_ptr(), out.stride(-2), three ? out.stride(0) : 0, i32(M), i32(N), i32(K), i32(batch), te, stream_of(x)),
+           "forge_gemm_simt");
+}
+
+void latent_prepare(const Tensor& proj, int64_t q_rank, int64_t kv_rank, const Tensor& qw, const Tensor& kw, double eps, const Tensor& rope,
+                    const Tensor& positions, const Tensor& slots, Tensor& cq, Tensor& cache, const Tensor& status) {
+  const int f = elem(proj);
+  const auto dt = proj.scalar_type();
+  TORCH_CHECK(proj.dim() == 2 && cache.dim() == 3 && rope.dim() == 2, "latent_prepare: ranks");
+  const int64_t T = proj.size(0), rot = proj.size(1) - q_rank - kv_rank;
+  TORCH_CHECK(q_rank > 0 && kv_rank > 0 && rot >= 0 && cache.size(2) == kv_rank + rot && rope.size(1) == rot, "latent_prepare: sizes");
+  const c10::cuda::CUDAGuard guard(proj.device());
+  check_rc(forge_latent_prepare(f, data(proj, dt, 0, "proj"), i32(T), i32(q_rank), i32(kv_rank), i32(rot), data(qw, dt, q_rank, "qw"),
+                                data(kw, dt, kv_rank, "kw"), static_cast<float>(eps), floats(rope, 0, "rope"), i32(rope.size(0)),
+                                ints(positions, T, "positions"), ints(slots, T, "slots"), data(cq, dt, T * q_rank, "cq"),
+                                data(cache, dt, 0, "cache"), static_cast<long long>(cache.size(0)) * cache.size(1), status_word(status),
+                                stream_of(proj)),
+           "forge_latent_prepare");
+}
+
+// q [tokens, heads * (dim + rot)] -> the rotated parts in qa [tokens, heads, kv_rank + rot]
+void latent_rotate_q(const Tensor& q, Tensor& qa, int64_t dim, int64_t kv_rank, const Tensor& rope, const Tensor& positions) {
+  const int f = elem(q);
+  TORCH_CHECK(q.dim() == 2 && qa.dim() == 3 && rope.dim() == 2, "latent_rotate_q: ranks");
+  const int64_t T = q.size(0), H = qa.size(1), rot = rope.size(1);
+  TORCH_CHECK(qa.size(0) == T && q.size(1) == H * (dim + rot) && qa.size(2) == kv_rank + rot, "latent_rotate_q: sizes");
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_rc(forge_latent_rotate_q(f, data(q, q.scalar_type(), 0, "q"), data(qa, q.scalar_type(), 0, "qa"), i32(T), i32(H), i32(dim), i32(rot),
+                                 i32(kv_rank), floats(rope, 0, "rope"), i32(rope.size(0)), ints(positions, T, "positions"), stream_of(q)),
+           "forge_latent_rotate_q");
+}
+
+// qa [tokens, heads, kv_rank + rot] = the step's tokens tok0 .. tok0 + tokens; o [tokens, heads, kv_rank]
+void latent_attend_any(const Tensor& qa, const Tensor& cache, Tensor& o, int64_t tok0, const Tensor& cu, int64_t num_seqs,
+                       const Tensor& positions, const Tensor& block_tables, double scale, const Tensor& status) {
+  const int f = elem(qa);
+  TORCH_CHECK(qa.dim() == 3 && cache.dim() == 3 && o.dim() == 3 && block_tables.dim() == 2, "latent_attend_any: ranks");
+  const int64_t T = qa.size(0), H = qa.size(1), R = o.size(2), D = qa.size(2);
+  TORCH_CHECK(o.size(0) == T && o.size(1) == H && cache.size(2) == D && R <= D && block_tables.size(0) >= num_seqs, "latent_attend_any: sizes");
+  const c10::cuda::CUDAGuard guard(qa.device());
+  check_rc(forge_latent_attend_any(f, data(qa, qa.scalar_type(), 0, "qa"), data(cache, qa.scalar_type(), 0, "cache"),
+                                   data(o, qa.scalar_type(), 0, "o"), i32(tok0), i32(T), ints(cu, num_seqs + 1, "cu_seqlens_q"), i32(num_seqs),
+                                   ints(positions, tok0 + T, "positions"), ints(block_tables, 0, "block_tables"), i32(block_tables.size(1)),
+                                   i32(cache.size(0)), i32(cache.size(1)), i32(H), i32(R), i32(D - R), static_cast<float>(scale),
+                                   status_word(status), stream_of(qa)),
+           "forge_latent_attend_any");
+}
+
+struct Ret {
+  int64_t T, H, dk, dv, slots;
+};
+Ret retention_sizes(const Tensor& qkvg, const Tensor& decay, const Tensor& state, const Tensor& rope) {
+  TORCH_CHECK(qkvg.dim() == 2 && state.dim() == 4 && rope.dim() == 2, "retention: ranks");
+  const Ret r{qkvg.size(0), state.size(1), state.size(2), state.size(3), state.size(0)};
+  TORCH_CHECK(qkvg.size(1) == r.H * (2 * r.dk + 2 * r.dv) && decay.numel() == r.H && rope.size(1) <= r.dk && rope.size(1) % 2 == 0, "retention: sizes");
+  return r;
+}
+
+void retention_decode(const Tensor& qkvg, const Tensor& decay, Tensor& state, const Tensor& slots, const Tensor& positions, const Tensor& rope,
+                      int64_t seqs, Tensor& y, double eps, const Tensor& status) {
+  const int f = elem(qkvg);
+  const Ret r = retention_sizes(qkvg, decay, state, rope);
+  TORCH_CHECK(seqs <= r.T, "retention_decode: sequences");
+  const c10::cuda::CUDAGuard guard(qkvg.device());
+  check_rc(forge_retention_decode(f, data(qkvg, qkvg.scalar_type(), 0, "qkvg"), i32(qkvg.size(1)), floats(decay, r.H, "decay"),
+                                  floats(state, 0, "state"), ints(slots, seqs, "slots"), ints(positions, seqs, "positions"),
+                                  floats(rope, 0, "rope"), i32(rope.size(0)), i32(rope.size(1)), i32(seqs), i32(r.H), i32(r.dk), i32(r.dv),
+                                  i32(r.slots), data(y, qkvg.scalar_type(), seqs * r.H * r.dv, "y"), static_cast<float>(eps),
+                                  status_word(status), stream_of(qkvg)),
+           "forge_retention_decode");
+}
+
+void retention_scan(const Tensor& qkvg, const Tensor& decay, Tensor& state, const Tensor& slots, const Tensor& positions, const Tensor& rope,
+                    const Tensor& cu, int64_t seqs, Tensor& o, const Tensor& status) {
+  const int f = elem(qkvg);
+  const Ret r = retention_sizes(qkvg, decay, state, rope);
+  const c10::cuda::CUDAGuard guard(qkvg.device());
+  check_rc(forge_retention_scan(f, data(qkvg, qkvg.scalar_type(), 0, "qkvg"), i32(qkvg.size(1)), floats(decay, r.H, "decay"),
+                                floats(state, 0, "state"), ints(slots, seqs, "slots"), ints(positions, r.T, "positions"),
+                                floats(rope, 0, "rope"), i32(rope.size(0)), i32(rope.size(1)), ints(cu, seqs + 1, "cu"), i32(seqs), i32(r.H),
+                                i32(r.dk), i32(r.dv), i32(r.slots), floats(o, r.T * r.H * r.dv, "o"), status_word(status), stream_of(qkvg)),
+           "forge_retention_scan");
+}
+
+// o fp32 [T, heads * dv] -> y [T, heads * dv] for the tokens from tok0 on
+void retention_gate(const Tensor& o, const Tensor& qkvg, Tensor& y, int64_t tok0, int64_t heads, int64_t dv, double eps) {
+  const int f = elem(qkvg);
+  const int64_t T = qkvg.size(0), ld = qkvg.size(1);
+  TORCH_CHECK(qkvg.dim() == 2 && tok0 >= 0 && tok0 <= T && ld >= heads * dv, "retention_gate: sizes");
+  const c10::cuda::CUDAGuard guard(qkvg.device());
+  check_rc(forge_retention_gate(f, floats(o, T * heads * dv, "o"), data(qkvg, qkvg.scalar_type(), 0, "qkvg"), i32(ld), i32(ld - heads * dv),
+                                data(y, qkvg.scalar_type(), T * heads * dv, "y"), i32(tok0), i32(T - tok0), i32(heads), i32(dv),
+                                static_cast<float>(eps), stream_of(qkvg)),
+           "forge_retention_gate");
+}
+
+void router(const Tensor& h, const Tensor& w, Tensor& experts, Tensor& weights) {
+  const int f = elem(h);
+  TORCH_CHECK(h.dim() == 2 && w.dim() == 2 && w.size(1) == h.size(1) && experts.dim() == 2 && experts.size(0) == h.size(0), "router: shapes");
+  const int64_t T = h.size(0), W = h.size(1), E = w.size(0), top = experts.size(1);
+  const c10::cuda::CUDAGuard guard(h.device());
+  check_rc(forge_router(f, data(h, h.scalar_type(), 0, "h"), data(w, h.scalar_type(), 0, "w"), i32(T), i32(W), i32(E), i32(top),
+                        const_cast<int*>(ints(experts, T * top, "experts")), floats(weights, T * top, "weights"), stream_of(h)),
+           "forge_router");
+}
+
+void moe_plan(const Tensor& experts, int64_t E, int64_t tile, Tensor& pos, Tensor& tile_expert, Tensor& num_tiles) {
+  const int64_t n = experts.numel();
+  // an expert with c rows takes ceil(c / tile) tiles, at least one row each
+  const int64_t worst = std::min(n, n / tile + E);
+  const c10::cuda::CUDAGuard guard(experts.device());
+  check_rc(forge_moe_plan(ints(experts, n, "experts"), i32(n), i32(E), i32(tile), i32(tile_expert.numel()),
+                          const_cast<int*>(ints(pos, n, "pos")), const_cast<int*>(ints(tile_expert, worst, "tile_expert")),
+                          const_cast<int*>(ints(num_tiles, 1, "num_tiles")), stream_of(experts)),
+           "forge_moe_plan");
+}
+
+void moe_scatter(const Tensor& h, const Tensor& pos, const Tensor& weights, Tensor& xs) {
+  const int f = elem(h);
+  TORCH_CHECK(h.dim() == 2 && pos.dim() == 2 && pos.size(0) == h.size(0) && xs.dim() == 2 && xs.size(1) == h.size(1), "moe_scatter: shapes");
+  const int64_t n = pos.numel();
+  const c10::cuda::CUDAGuard guard(h.device());
+  check_rc(forge_moe_scatter(f, data(h, h.scalar_type(), 0, "h"), ints(pos, n, "pos"), floats(weights, n, "weights"), i32(n), i32(pos.size(1)),
+                             i32(h.size(1)), data(xs, h.scalar_type(), 0, "xs"), stream_of(h)),
+           "forge_moe_scatter");
+}
+
+}  // namespace
+
+void register_mixers(pybind11::module& m) {
+  m.def("stream_update", &stream_update);
+  m.def("silu_mul_any", &silu_mul_any);
+  m.def("gemm_simt", &gemm_simt);
+  m.def("latent_prepare", &latent_prepare);
+  m.def("latent_rotate_q", &latent_rotate_q);
+  m.def("latent_attend_any", &latent_attend_any);
+  m.def("retention_decode", &retention_decode);
+  m.def("retention_scan", &retention_scan);
+  m.def("retention_gate", &retention_gate);
+  m.def("router", &router);
+  m.def("moe_plan", &moe_plan);
+  m.def("moe_scatter", &moe_scatter);
+}

@@ -1,0 +1,151 @@
+// Mixture of experts: routing and the shuffling of rows.
+//
+//   router_scores   logits (fp32) -> sigmoid -> the `top` largest scores of a token (ties: the lower expert)
+//   moe_plan        (token, choice) -> row of the expert-sorted buffer; every expert's rows start on a multiple of `tile`, so
+//                   a tile of rows has one expert (tile_expert; -1 past the last tile in use)
+//   moe_scatter     row = score * token, the score in fp32: it multiplies the expert's INPUT
+//
+// Rows between an expert's last token and its next tile boundary are never written nor read back.
+#include "../include/launch.cuh"
+#include "../include/scalar.cuh"
+
+namespace forge {
+
+// CTA = one token; one warp per expert at a time.
+template <typename T, int N>
+__global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, const T* __restrict__ w, int W, int E, int top,
+                                                     int* __restrict__ experts, float* __restrict__ weights) {
+  extern __shared__ float score[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* row = h + t * W;
+  for (int e = warp; e < E; e += blockDim.x >> 5) {
+    const T* we = w + static_cast<size_t>(e) * W;
+    float z = 0.f;
+    for (int i = lane * N; i < W; i += 32 * N) {
+      float a[N], b[N];
+      load_n<N>(row + i, a);
+      load_n<N>(we + i, b);
+#pragma unroll
+      for (int q = 0; q < N; ++q) z = fmaf(a[q], b[q], z);
+    }
+    z = warp_sum_f(z);
+    if (lane == 0) score[e] = 1.f / (1.f + expf(-z));
+  }
+  __syncthreads();
+  if (warp != 0) return;
+  for (int j = 0; j < top; ++j) {
+    float best = -1.f;
+    int at = E;
+    for (int e = lane; e < E; e += 32)
+      if (score[e] > best) { best = score[e]; at = e; }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+      const float v = __shfl_xor_sync(0xffffffffu, best, off);
+      const int i = __shfl_xor_sync(0xffffffffu, at, off);
+      if (v > best || (v == best && i < at)) { best = v; at = i; }
+    }
+    if (at >= E) at = 0;                          // only if every score is NaN
+    if (lane == 0) {
+      experts[t * top + j] = at;
+      weights[t * top + j] = best;
+      score[at] = -2.f;
+    }
+    __syncwarp();
+  }
+}
+
+extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int W, int E, int top, int* experts, float* weights,
+                            cudaStream_t stream) {
+  if (T_ <= 0) return 0;
+  if (E > 4096 || top < 1 || top > E) return -1;
+  const bool v4 = (W & 3) == 0;
+  const size_t smem = static_cast<size_t>(E) * 4;
+  if (fp32) {
+    auto k = v4 ? router_kernel<float, 4> : router_kernel<float, 1>;
+    return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+  }
+  auto k = v4 ? router_kernel<bf16, 4> : router_kernel<bf16, 1>;
+  return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+}
+
+constexpr int kPlanThreads = 1024;
+
+// One CTA.  smem: counts [E], next row [E].
+__global__ void __launch_bounds__(kPlanThreads) moe_plan_kernel(const int* __restrict__ experts, int n, int E, int tile, int max_tiles,
+                                                                int* __restrict__ pos, int* __restrict__ tile_expert,
+                                                                int* __restrict__ num_tiles) {
+  extern __shared__ int sm_plan[];
+  int* count = sm_plan;
+  int* next = sm_plan + E;
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int e = threadIdx.x; e < E; e += kPlanThreads) count[e] = 0;
+  __syncthreads();
+  for (int i = threadIdx.x; i < n; i += kPlanThreads) atomicAdd(&count[experts[i]], 1);
+  __syncthreads();
+  if (threadIdx.x < 32) {                         // running sum of tiles, 32 experts at a time
+    int base = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int tiles = e < E ? (count[e] + tile - 1) / tile : 0;
+      int incl = tiles;
+#pragma unroll
+      for (int off = 1; off < 32; off <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, incl, off);
+        if (threadIdx.x >= off) incl += v;
+      }
+      if (e < E) next[e] = (base + incl - tiles) * tile;
+      base += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    if (threadIdx.x == 0) num_tiles[0] = base;
+  }
+  for (int i = threadIdx.x; i < max_tiles; i += kPlanThreads) tile_expert[i] = -1;
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += kPlanThreads)
+    for (int k = 0; k < (count[e] + tile - 1) / tile; ++k) tile_expert[next[e] / tile + k] = e;
+  __syncthreads();
+  for (int i = threadIdx.x; i < n; i += kPlanThreads) pos[i] = atomicAdd(&next[experts[i]], 1);
+}
+
+// max_tiles >= n / tile + E rounded up: the caller's buffer has max_tiles * tile rows.
+extern "C" int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles,
+                              cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (E > 4096 || tile < 1) return -1;
+  return launch_kernel(moe_plan_kernel, dim3(1), dim3(kPlanThreads), static_cast<size_t>(E) * 8, stream, 0, experts, n, E, tile, max_tiles,
+                       pos, tile_expert, num_tiles) == cudaSuccess ? 0 : -2;
+}
+
+template <typename T, int N>
+__global__ void __launch_bounds__(128) moe_scatter_kernel(const T* __restrict__ h, const int* __restrict__ pos,
+                                                          const float* __restrict__ weights, int top, int W, T* __restrict__ xs) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = blockIdx.x, t = i / top;
+  const float s = weights[i];
+  T* dst = xs + static_cast<size_t>(pos[i]) * W;
+  for (int c = threadIdx.x * N; c < W; c += blockDim.x * N) {
+    float v[N];
+    load_n<N>(h + t * W + c, v);
+#pragma unroll
+    for (int e = 0; e < N; ++e) v[e] *= s;
+    store_n<N>(dst + c, v);
+  }
+}
+
+extern "C" int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs,
+                                 cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const bool v4 = (W & 3) == 0;
+  if (fp32) {
+    auto k = v4 ? moe_scatter_kernel<float, 4> : moe_scatter_kernel<float, 1>;
+    return launch_kernel(k, dim3(n), dim3(128), 0, stream, 0, static_cast<const float*>(h), pos, weights, top, W, static_cast<float*>(xs)) == cudaSuccess ? 0 : -2;
+  }
+  auto k = v4 ? moe_scatter_kernel<bf16, 4> : moe_scatter_kernel<bf16, 1>;
+  return launch_kernel(k, dim3(n), dim3(128), 0, stream, 0, static_cast<const bf16*>(h), pos, weights, top, W, static_cast<bf16*>(xs)) == cudaSuccess ? 0 : -2;
+}
+
+}  // namespace forge

@@ -1,7 +1,7 @@
 """In-tree build of the CUDA extension ``tinyllmforge_b200/_C*.so`` for sm_100a.
 
 Kernels (``csrc/**/*.cu``) are compiled with nvcc directly (they do not include torch headers, so a file
-rebuilds in seconds); ``csrc/host/bindings.cpp`` is the only translation unit that sees torch.  Objects are
+rebuilds in seconds); only ``csrc/host/*.cpp`` see torch.  Objects are
 cached under ``build/`` by content hash of the source, its headers and the flags.  nvcc cross-compiles without
 a GPU, so this runs on a CPU-only machine.
 
@@ -64,7 +64,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
     os.makedirs(BUILD, exist_ok=True)
     headers = glob.glob(os.path.join(CSRC, "include", "*"))
     cu_files = sorted(glob.glob(os.path.join(CSRC, "**", "*.cu"), recursive=True))
-    cpp_files = [os.path.join(CSRC, "host", "bindings.cpp")]
+    cpp_files = sorted(glob.glob(os.path.join(CSRC, "host", "*.cpp")))
     cuda_inc = os.path.join(os.path.dirname(os.path.dirname(_nvcc())), "include") if os.path.sep in _nvcc() else "/usr/local/cuda/include"
 
     jobs, objs = [], []

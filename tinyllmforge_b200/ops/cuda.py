@@ -17,6 +17,7 @@ import torch
 
 from ..config import Config
 from ..parallel.comm import TPGroup
+from .cuda_mixers import MixerOps
 from .quant import Fp8BlockWeight
 
 try:
@@ -76,7 +77,7 @@ def _streamk_workspace(C, device, num_sms: int) -> None:
     _STREAMK_WS[key] = (ws, counters)
 
 
-class CudaOps:
+class CudaOps(MixerOps):
     name = "cuda"
 
     def __init__(self, config: Config | None = None, tp: TPGroup | None = None, device=None):
@@ -138,6 +139,8 @@ class CudaOps:
             if not self._expands_fp8(w, x.shape[0]):
                 return self.linear_fp8(x, w)
             w, force_deep = self._expand_fp8(w), force_deep | W_DYNAMIC
+        if not self.tma_ok(x, w):
+            return self.linear_simt(x, w)
         out = torch.empty(x.shape[0], w.shape[0], dtype=x.dtype, device=x.device)
         self.C.gemm(x, w, out, 0, force_mode, force_splits | (force_block_c << 8) | (force_deep << 16), self.status)
         return out
@@ -148,6 +151,8 @@ class CudaOps:
             if not self._expands_fp8(w_gate_up, x.shape[0]):
                 return self.silu_mul(self.linear_fp8(x, w_gate_up))
             w_gate_up, force_deep = self._expand_fp8(w_gate_up), force_deep | W_DYNAMIC
+        if not self.tma_ok(x, w_gate_up):
+            return self.silu_mul_any(self.linear_simt(x, w_gate_up))
         out = torch.empty(x.shape[0], w_gate_up.shape[0] // 2, dtype=x.dtype, device=x.device)
         self.C.gemm(x, w_gate_up, out, 1, force_mode, force_splits | (force_block_c << 8) | (force_deep << 16), self.status)
         return out
@@ -450,7 +455,8 @@ class CudaOps:
         """The LM-head GEMM can sample in its epilogue when it runs on the persistent token-tile kernel (many vocabulary
         tiles, at least 8 rows) over a bf16 shard; the shard must start on a multiple of 32 token ids (checked by the
         caller that knows the start)."""
-        return (self.sample_in_lm_head and not isinstance(weight, Fp8BlockWeight) and rows >= 8
+        return (self.sample_in_lm_head and not isinstance(weight, Fp8BlockWeight) and weight.dtype == torch.bfloat16 and rows >= 8
+                and weight.shape[1] % 8 == 0
                 and (weight.shape[0] + 127) // 128 >= 2 * self.num_sms)
 
     def lm_head_sample_shard(self, hidden, weight, temperatures, header, vocab_start):
