@@ -5,6 +5,7 @@
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
 
+#include <algorithm>
 #include <cstdint>
 
 extern "C" {
@@ -32,6 +33,26 @@ int forge_retention_gate(int fp32, const float* o, const void* qkvg, int ld, int
                          float eps, cudaStream_t stream);
 int forge_router(int fp32, const void* h, const void* w, int T, int W, int E, int top, int* experts, float* weights, cudaStream_t stream);
 int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles, cudaStream_t stream);
+int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int n_out, int K, int gated, int tile, const int* tile_expert,
+                       const int* num_tiles, int max_tiles, unsigned* status, cudaStream_t stream);
+int forge_head_linear(const void* x, long long x_tok, long long x_head, const void* w, void* out, long long o_tok, long long o_head, int M,
+                      int heads, int N, int K, cudaStream_t stream);
+int forge_latent_decode_ok(int R, int rot, int block_size);
+int forge_latent_decode(const void* qa, const void* cache, const int* block_tables, const int* lens, void* o, float* part_o, float* part_ml,
+                        int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size, int chunk, int max_chunks,
+                        int tile, float scale, unsigned* status, cudaStream_t stream);
+int forge_latent_prefill_qcols(int dim, int rot, int vdim);
+int forge_latent_prefill(const void* q, const void* kv, const void* kr, const int* cu_q, const int* cu_k, void* out, int tokens, int tok0,
+                         int keys, int num_seqs, int max_q, int heads, int dim, int rot, int vdim, float scale, unsigned* status,
+                         cudaStream_t stream);
+int forge_latent_gather(const void* cache, const int* cu_k, int num_seqs, const int* block_tables, int table_width, int num_blocks,
+                        int block_size, int R, int rot, int keys, void* c, void* kr, unsigned* status, cudaStream_t stream);
+int forge_latent_pack_q(const void* q, void* qp, int tokens, int heads, int dim, int rot, const float* rope, int rope_rows,
+                        const int* positions, cudaStream_t stream);
+int forge_retention_chunk_ok(int heads, int dk, int dv, int rd);
+int forge_retention_chunk(void* qkvg, int ld, const float* decay, float* state, const int* slots, const int* positions, const float* rope,
+                          int rope_rows, int rd, const int* cu, int seqs, int tok0, int tokens, int heads, int dk, int dv, int num_slots,
+                          float* o, float* ws, int segs, int seg_len, unsigned* status, cudaStream_t stream);
 int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs, cudaStream_t stream);
 }
 
@@ -271,6 +292,111 @@ void moe_scatter(const Tensor& h, const Tensor& pos, const Tensor& weights, Tens
            "forge_moe_scatter");
 }
 
+// ---- tensor-core kernels (bf16)
+constexpr auto kBf16 = at::kBFloat16;
+
+void grouped_gemm(const Tensor& x, const Tensor& w, Tensor& out, bool gated, int64_t tile, const Tensor& tile_expert, const Tensor& num_tiles,
+                  const Tensor& status) {
+  TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && out.dim() == 2 && w.size(2) == x.size(1), "grouped_gemm: ranks");
+  const int64_t rows = x.size(0), K = x.size(1), N = gated ? w.size(1) / 2 : w.size(1), tiles = tile_expert.numel();
+  TORCH_CHECK(rows == tiles * tile && out.size(0) == rows && out.size(1) == N, "grouped_gemm: shapes");
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_grouped_gemm(data(x, kBf16, 0, "x"), data(w, kBf16, 0, "w"), data(out, kBf16, 0, "out"), i32(w.size(0)), i32(N), i32(K),
+                              gated ? 1 : 0, i32(tile), ints(tile_expert, 0, "tile_expert"), ints(num_tiles, 1, "num_tiles"), i32(tiles),
+                              status_word(status), stream_of(x)),
+           "forge_grouped_gemm");
+}
+
+// x [tokens, heads, K] and out [tokens, heads, N] may be strided views; w [heads, N, K] contiguous
+void head_linear(const Tensor& x, const Tensor& w, Tensor& out) {
+  TORCH_CHECK(x.is_cuda() && out.is_cuda() && x.scalar_type() == kBf16 && out.scalar_type() == kBf16, "head_linear: operands");
+  TORCH_CHECK(x.dim() == 3 && w.dim() == 3 && out.dim() == 3 && x.stride(2) == 1 && out.stride(2) == 1, "head_linear: ranks");
+  TORCH_CHECK(x.size(0) == out.size(0) && x.size(1) == w.size(0) && out.size(1) == w.size(0) && w.size(2) == x.size(2) && w.size(1) == out.size(2),
+              "head_linear: shapes");
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_head_linear(x.data_ptr(), x.stride(0), x.stride(1), data(w, kBf16, 0, "w"), out.data_ptr(), out.stride(0), out.stride(1),
+                             i32(x.size(0)), i32(w.size(0)), i32(w.size(1)), i32(w.size(2)), stream_of(x)),
+           "forge_head_linear");
+}
+
+void latent_decode(const Tensor& qa, const Tensor& cache, const Tensor& block_tables, const Tensor& lens, Tensor& o, const OptTensor& part_o,
+                   const OptTensor& part_ml, int64_t chunk, int64_t max_chunks, int64_t tile, double scale, const Tensor& status) {
+  TORCH_CHECK(qa.dim() == 3 && cache.dim() == 3 && block_tables.dim() == 2 && o.dim() == 3, "latent_decode: ranks");
+  const int64_t B = qa.size(0), H = qa.size(1), D = qa.size(2), R = o.size(2);
+  TORCH_CHECK(cache.size(2) == D && R <= D && o.size(0) == B && o.size(1) == H && block_tables.size(0) >= B && max_chunks >= 1, "latent_decode: shapes");
+  float *po = nullptr, *pml = nullptr;
+  if (max_chunks > 1) {
+    TORCH_CHECK(part_o.has_value() && part_ml.has_value(), "latent_decode: scratch");
+    po = floats(*part_o, B * H * max_chunks * R, "part_o");
+    pml = floats(*part_ml, B * H * max_chunks * 2, "part_ml");
+  }
+  const c10::cuda::CUDAGuard guard(qa.device());
+  check_rc(forge_latent_decode(data(qa, kBf16, 0, "qa"), data(cache, kBf16, 0, "cache"), ints(block_tables, 0, "block_tables"), ints(lens, B, "lens"),
+                               data(o, kBf16, 0, "o"), po, pml, i32(B), i32(H), i32(R), i32(D - R), i32(block_tables.size(1)), i32(cache.size(0)),
+                               i32(cache.size(1)), i32(chunk), i32(max_chunks), i32(tile), static_cast<float>(scale), status_word(status),
+                               stream_of(qa)),
+           "forge_latent_decode");
+}
+
+// c [keys, R], kr [keys, rot] <- the cached rows of the sequences whose running key counts are cu_k
+void latent_gather(const Tensor& cache, const Tensor& cu_k, int64_t num_seqs, const Tensor& block_tables, Tensor& c, Tensor& kr, const Tensor& status) {
+  TORCH_CHECK(cache.dim() == 3 && block_tables.dim() == 2 && c.dim() == 2 && kr.dim() == 2, "latent_gather: ranks");
+  const int64_t keys = c.size(0), R = c.size(1), rot = kr.size(1);
+  TORCH_CHECK(kr.size(0) == keys && cache.size(2) == R + rot && block_tables.size(0) >= num_seqs, "latent_gather: shapes");
+  const c10::cuda::CUDAGuard guard(cache.device());
+  check_rc(forge_latent_gather(data(cache, kBf16, 0, "cache"), ints(cu_k, num_seqs + 1, "cu_k"), i32(num_seqs), ints(block_tables, 0, "block_tables"),
+                               i32(block_tables.size(1)), i32(cache.size(0)), i32(cache.size(1)), i32(R), i32(rot), i32(keys),
+                               data(c, kBf16, 0, "c"), data(kr, kBf16, 0, "kr"), status_word(status), stream_of(cache)),
+           "forge_latent_gather");
+}
+
+void latent_pack_q(const Tensor& q, Tensor& qp, int64_t heads, int64_t dim, const Tensor& rope, const Tensor& positions) {
+  TORCH_CHECK(q.dim() == 2 && qp.dim() == 3 && rope.dim() == 2, "latent_pack_q: ranks");
+  const int64_t T = q.size(0), rot = rope.size(1);
+  TORCH_CHECK(q.size(1) == heads * (dim + rot) && qp.size(0) == T && qp.size(1) == heads && qp.size(2) == 64 * ((dim + 63) / 64 + (rot + 63) / 64),
+              "latent_pack_q: shapes");
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_rc(forge_latent_pack_q(data(q, kBf16, 0, "q"), data(qp, kBf16, 0, "qp"), i32(T), i32(heads), i32(dim), i32(rot), floats(rope, 0, "rope"),
+                               i32(rope.size(0)), ints(positions, T, "positions"), stream_of(q)),
+           "forge_latent_pack_q");
+}
+
+// qp [tokens - tok0, heads, qcols], kv [keys, heads * (dim + vdim)], kr [keys, rot], out [tokens, heads * vdim]
+void latent_prefill(const Tensor& qp, const Tensor& kv, const Tensor& kr, const Tensor& cu_q, const Tensor& cu_k, Tensor& out, int64_t tok0,
+                    int64_t num_seqs, int64_t max_q, int64_t dim, int64_t vdim, double scale, const Tensor& status) {
+  TORCH_CHECK(qp.dim() == 3 && kv.dim() == 2 && kr.dim() == 2 && out.dim() == 2, "latent_prefill: ranks");
+  const int64_t H = qp.size(1), T = out.size(0), keys = kv.size(0), rot = kr.size(1);
+  TORCH_CHECK(qp.size(0) == T - tok0 && kv.size(1) == H * (dim + vdim) && kr.size(0) == keys && out.size(1) == H * vdim &&
+                  qp.size(2) == forge_latent_prefill_qcols(i32(dim), i32(rot), i32(vdim)),
+              "latent_prefill: shapes");
+  const c10::cuda::CUDAGuard guard(qp.device());
+  check_rc(forge_latent_prefill(data(qp, kBf16, 0, "qp"), data(kv, kBf16, 0, "kv"), data(kr, kBf16, 0, "kr"), ints(cu_q, num_seqs + 1, "cu_q"),
+                                ints(cu_k, num_seqs + 1, "cu_k"), data(out, kBf16, 0, "out"), i32(T), i32(tok0), i32(keys), i32(num_seqs),
+                                i32(max_q), i32(H), i32(dim), i32(rot), i32(vdim), static_cast<float>(scale), status_word(status),
+                                stream_of(qp)),
+           "forge_latent_prefill");
+}
+
+// q and k of qkvg are rotated in place (tokens from tok0 on); o fp32 [tokens, heads * dv]
+void retention_chunk(Tensor& qkvg, const Tensor& decay, Tensor& state, const Tensor& slots, const Tensor& positions, const Tensor& rope,
+                     const Tensor& cu, int64_t seqs, int64_t tok0, Tensor& o, const OptTensor& ws, int64_t segs, int64_t seg_len,
+                     const Tensor& status) {
+  const Ret r = retention_sizes(qkvg, decay, state, rope);
+  float* wp = nullptr;
+  if (segs > 1) {
+    TORCH_CHECK(ws.has_value(), "retention_chunk: scratch");
+    wp = floats(*ws, seqs * segs * r.H * r.dk * r.dv, "ws");
+    TORCH_CHECK(segs * seg_len >= r.T - tok0 || seqs > 1, "retention_chunk: segments do not cover the run");
+  }
+  const c10::cuda::CUDAGuard guard(qkvg.device());
+  check_rc(forge_retention_chunk(data(qkvg, kBf16, 0, "qkvg"), i32(qkvg.size(1)), floats(decay, r.H, "decay"), floats(state, 0, "state"),
+                                 ints(slots, seqs, "slots"), ints(positions, r.T, "positions"), floats(rope, 0, "rope"), i32(rope.size(0)),
+                                 i32(rope.size(1)), ints(cu, seqs + 1, "cu"), i32(seqs), i32(tok0), i32(r.T), i32(r.H), i32(r.dk), i32(r.dv),
+                                 i32(r.slots), floats(o, r.T * r.H * r.dv, "o"), wp, i32(segs), i32(seg_len), status_word(status),
+                                 stream_of(qkvg)),
+           "forge_retention_chunk");
+}
+
 }  // namespace
 
 void register_mixers(pybind11::module& m) {
@@ -286,4 +412,14 @@ void register_mixers(pybind11::module& m) {
   m.def("router", &router);
   m.def("moe_plan", &moe_plan);
   m.def("moe_scatter", &moe_scatter);
+  m.def("grouped_gemm", &grouped_gemm);
+  m.def("head_linear", &head_linear);
+  m.def("latent_decode", &latent_decode);
+  m.def("latent_decode_ok", [](int64_t R, int64_t rot, int64_t bs) { return forge_latent_decode_ok(i32(R), i32(rot), i32(bs)) != 0; });
+  m.def("latent_gather", &latent_gather);
+  m.def("latent_pack_q", &latent_pack_q);
+  m.def("latent_prefill", &latent_prefill);
+  m.def("latent_prefill_qcols", [](int64_t dim, int64_t rot, int64_t vdim) { return forge_latent_prefill_qcols(i32(dim), i32(rot), i32(vdim)); });
+  m.def("retention_chunk", &retention_chunk);
+  m.def("retention_chunk_ok", [](int64_t H, int64_t dk, int64_t dv, int64_t rd) { return forge_retention_chunk_ok(i32(H), i32(dk), i32(dv), i32(rd)) != 0; });
 }
