@@ -59,10 +59,10 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
   const int c0 = blockIdx.x * 64, h = blockIdx.y;
   const int seq = blockIdx.z / p.segs, seg = blockIdx.z % p.segs;
   const int run = p.cu[seq + 1] - p.cu[seq];
-  const int n_segs = p.segs == 1 ? 1 : (run + p.seg_len - 1) / p.seg_len;
+  const int n_segs = p.segs == 1 ? 1 : min((run + p.seg_len - 1) / p.seg_len, p.segs);
   if (run <= 0 || seg >= n_segs || (kStateOnly && seg == n_segs - 1)) return;
   const int t_begin = p.cu[seq] + seg * p.seg_len;
-  const int t_end = p.segs == 1 ? p.cu[seq + 1] : min(p.cu[seq + 1], t_begin + p.seg_len);
+  const int t_end = seg == n_segs - 1 ? p.cu[seq + 1] : t_begin + p.seg_len;
   const int slot = p.slots[seq];
   if (slot < 0 || slot >= p.num_slots) {
     if (threadIdx.x == 0) set_status(p.status, kStatusBadIndex);
@@ -272,7 +272,7 @@ __global__ void __launch_bounds__(256) retention_segments_kernel(const Retention
   const int run = p.cu[seq + 1] - p.cu[seq];
   const int slot = p.slots[seq];
   if (run <= 0 || slot < 0 || slot >= p.num_slots) return;
-  const int n_segs = (run + p.seg_len - 1) / p.seg_len;
+  const int n_segs = min((run + p.seg_len - 1) / p.seg_len, p.segs);
   const int n = p.dk * p.dv, i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (i >= n) return;
   const float g = powf(p.decay[h], static_cast<float>(p.seg_len));

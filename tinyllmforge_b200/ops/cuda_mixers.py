@@ -18,6 +18,8 @@ class Routed:
 class MixerOps:
     """Mixed into ``CudaOps`` (uses its ``C``, ``status``, ``device`` and GEMM methods)."""
 
+    latent_tile = 32                # keys per tile of the decode kernel (32: two CTAs per SM, 64: one)
+
     # ------------------------------------------------------------------ residual stream
     def stream_update(self, x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
@@ -48,7 +50,11 @@ class MixerOps:
 
     def head_linear(self, x, w, out) -> None:
         """out[:, h] = x[:, h] @ w[h].T for views x [tokens, heads, K], w [heads, N, K], out [tokens, heads, N]."""
-        self.C.gemm_simt(x.transpose(0, 1), w, out.transpose(0, 1), None)
+        if (x.dtype == torch.bfloat16 and not (x.shape[2] | x.stride(0) | x.stride(1)) % 8 and not (w.shape[1] | out.stride(0) | out.stride(1)) % 2
+                and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
+            self.C.head_linear(x, w, out)
+        else:
+            self.C.gemm_simt(x.transpose(0, 1), w, out.transpose(0, 1), None)
 
     # ------------------------------------------------------------------ latent attention
     def latent_prepare(self, proj, q_rank, kv_rank, q_norm, kv_norm, eps, table, positions, slot_mapping, cache):
@@ -57,25 +63,65 @@ class MixerOps:
         return cq
 
     def latent_attention(self, q, weights, cache, batch, table, spec):
+        """Single tokens go through the folded form (queries against the cached latents themselves), runs of tokens through
+        the expanded one (keys and values rebuilt per head)."""
         T = q.shape[0]
         out = torch.empty(T, spec.heads * spec.vdim, dtype=q.dtype, device=q.device)
-        self._latent_folded(q, weights, cache, batch, table, spec, out, 0, T)
+        n1 = T if not batch.is_prefill else batch.num_single
+        if T > n1 and not self._latent_expanded(q, weights, cache, batch, table, spec, out, n1):
+            n1 = T
+        self._latent_folded(q, weights, cache, batch, table, spec, out, n1)
         return out
 
-    def _latent_folded(self, q, weights, cache, batch, table, spec, out, tok0, tok1) -> None:
-        """Tokens [tok0, tok1) of the step through the folded form: queries against the cached latents themselves."""
+    def latent_chunking(self, seqs: int, heads: int, max_len: int) -> tuple[int, int]:
+        """(keys per chunk, chunks) of the decode kernel: enough chunks to fill the GPU, from shapes known at capture time."""
+        ctas = seqs * -(-heads // 16)
+        want = -(-2 * self.num_sms // ctas)                       # chunks per sequence for two CTAs per SM
+        chunk = 64
+        while chunk < 1024 and -(-max_len // (2 * chunk)) >= want:
+            chunk *= 2
+        return chunk, max(1, -(-max_len // chunk))
+
+    def _latent_folded(self, q, weights, cache, batch, table, spec, out, n) -> None:
+        """The first n tokens of the step."""
         H, d, r, dv, R = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
-        n = tok1 - tok0
         if n <= 0:
             return
-        q = q[tok0:tok1]
+        q = q[:n]
         qa = torch.empty(n, H, R + r, dtype=q.dtype, device=q.device)
         self.head_linear(q.view(n, H, d + r)[:, :, :d], weights.uk_t, qa[:, :, :R])
-        self.C.latent_rotate_q(q, qa, d, R, table, batch.positions[tok0:tok1])
+        self.C.latent_rotate_q(q, qa, d, R, table, batch.positions[:n])
         o = torch.empty(n, H, R, dtype=q.dtype, device=q.device)
-        self.C.latent_attend_any(qa, cache, o, tok0, batch.cu_seqlens_q, batch.padded_seqs, batch.positions, batch.block_tables,
+        singles = n == (batch.num_single if batch.is_prefill else batch.padded_seqs)
+        if singles and q.dtype == torch.bfloat16 and self.C.latent_decode_ok(R, r, cache.shape[1]):
+            chunk, chunks = self.latent_chunking(n, H, batch.table_width * cache.shape[1])
+            part_o = part_ml = None
+            if chunks > 1:
+                part_o = torch.empty(n * H * chunks * R, dtype=torch.float32, device=q.device)
+                part_ml = torch.empty(n * H * chunks * 2, dtype=torch.float32, device=q.device)
+            self.C.latent_decode(qa, cache, batch.block_tables, batch.context_lens, o, part_o, part_ml, chunk, chunks, self.latent_tile,
                                  spec.scale, self.status)
-        self.head_linear(o, weights.uv, out[tok0:tok1].view(n, H, dv))
+        else:
+            self.C.latent_attend_any(qa, cache, o, 0, batch.cu_seqlens_q, batch.padded_seqs, batch.positions, batch.block_tables,
+                                     spec.scale, self.status)
+        self.head_linear(o, weights.uv, out[:n].view(n, H, dv))
+
+    def _latent_expanded(self, q, weights, cache, batch, table, spec, out, n1) -> bool:
+        """The sequences from ``n1`` on (their tokens start at row n1).  False: these sizes have no kernel, nothing was done."""
+        H, d, r, dv, R = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
+        qcols = self.C.latent_prefill_qcols(d, r, dv)
+        if q.dtype != torch.bfloat16 or qcols == 0 or R % 8:
+            return False
+        T, seqs, keys = q.shape[0], batch.num_seqs - n1, batch.kv_rows
+        cu_q, cu_k, tables = batch.cu_seqlens_q[n1:], batch.cu_seqlens_k[n1:], batch.block_tables[n1:]
+        c = torch.empty(keys, R, dtype=q.dtype, device=q.device)
+        kr = torch.empty(keys, r, dtype=q.dtype, device=q.device)
+        self.C.latent_gather(cache, cu_k, seqs, tables, c, kr, self.status)
+        kv = self.linear(c, weights.ukv)
+        qp = torch.empty(T - n1, H, qcols, dtype=q.dtype, device=q.device)
+        self.C.latent_pack_q(q[n1:], qp, H, d, table, batch.positions[n1:])
+        self.C.latent_prefill(qp, kv, kr, cu_q, cu_k, out, n1, seqs, batch.max_seqlen_q, d, dv, spec.scale, self.status)
+        return True
 
     # ------------------------------------------------------------------ retention
     def retention(self, qkvg, decay, state, batch, table, spec, eps):
@@ -88,10 +134,23 @@ class MixerOps:
         rest = batch.num_seqs - n1
         if batch.is_prefill and rest > 0:
             o = torch.empty(T, H * dv, dtype=torch.float32, device=qkvg.device)
-            self.C.retention_scan(qkvg, decay, state, batch.state_slots[n1:], batch.positions, table, batch.cu_seqlens_q[n1:], rest, o,
-                                  self.status)
+            slots, cu = batch.state_slots[n1:], batch.cu_seqlens_q[n1:]
+            if qkvg.dtype == torch.bfloat16 and self.C.retention_chunk_ok(H, spec.dim, dv, table.shape[1]):
+                segs, seg_len = self.retention_segments(rest, H, dv, batch.max_seqlen_q)
+                ws = torch.empty(rest * segs * H * spec.dim * dv, dtype=torch.float32, device=qkvg.device) if segs > 1 else None
+                self.C.retention_chunk(qkvg, decay, state, slots, batch.positions, table, cu, rest, n1, o, ws, segs, seg_len, self.status)
+            else:
+                self.C.retention_scan(qkvg, decay, state, slots, batch.positions, table, cu, rest, o, self.status)
             self.C.retention_gate(o, qkvg, y, n1, H, dv, eps)
         return y
+
+    def retention_segments(self, seqs: int, heads: int, dv: int, longest: int) -> tuple[int, int]:
+        """(segments per run, tokens per segment): a run is cut when the batch alone does not give two CTAs per SM."""
+        want = 2 * self.num_sms // (seqs * heads * -(-dv // 64))
+        segs = max(1, min(want, longest // 256))
+        seg_len = -(-longest // segs)
+        seg_len = -(-seg_len // 64) * 64
+        return max(1, -(-longest // seg_len)), seg_len
 
     # ------------------------------------------------------------------ experts
     def moe(self, h, router, gate_up, down, top):
@@ -100,7 +159,10 @@ class MixerOps:
         experts = torch.empty(T, top, dtype=torch.int32, device=h.device)
         weights = torch.empty(T, top, dtype=torch.float32, device=h.device)
         self.C.router(h, router, experts, weights)
-        tile = 64
+        fast = h.dtype == torch.bfloat16 and W % 8 == 0 and down.shape[2] % 8 == 0
+        tile = 64                                   # rows per tile; the tensor-core kernel takes 16 to 128
+        if fast:
+            tile = next((t for t in (16, 32, 64) if n <= t * E), 128)
         tiles = min(n, n // tile + E)
         rows = torch.empty(T, top, dtype=torch.int32, device=h.device)
         tile_expert = torch.empty(tiles, dtype=torch.int32, device=h.device)
@@ -108,9 +170,13 @@ class MixerOps:
         self.C.moe_plan(experts, E, tile, rows, tile_expert, num_tiles)
         xs = torch.empty(tiles * tile, W, dtype=h.dtype, device=h.device)
         self.C.moe_scatter(h, rows, weights, xs)
-        gu = torch.empty(tiles * tile, gate_up.shape[1], dtype=h.dtype, device=h.device)
-        self.C.gemm_simt(xs, gate_up, gu, tile_expert)
-        g = self.silu_mul_any(gu)
         y = torch.empty(tiles * tile, W, dtype=h.dtype, device=h.device)
-        self.C.gemm_simt(g, down, y, tile_expert)
+        if fast:
+            g = torch.empty(tiles * tile, down.shape[2], dtype=h.dtype, device=h.device)
+            self.C.grouped_gemm(xs, gate_up, g, True, tile, tile_expert, num_tiles, self.status)
+            self.C.grouped_gemm(g, down, y, False, tile, tile_expert, num_tiles, self.status)
+        else:
+            gu = torch.empty(tiles * tile, gate_up.shape[1], dtype=h.dtype, device=h.device)
+            self.C.gemm_simt(xs, gate_up, gu, tile_expert)
+            self.C.gemm_simt(self.silu_mul_any(gu), down, y, tile_expert)
         return Routed(y, rows)
