@@ -18,7 +18,7 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(const T* __restrict
                                                              const int* __restrict__ positions, const int* __restrict__ slots,
                                                              T* __restrict__ cq, T* __restrict__ cache, long long num_slots,
                                                              unsigned* status) {
-  __shared__ float red[32];
+  __shared__ float red[8];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -36,8 +36,15 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(const T* __restrict
 #pragma unroll
     for (int e = 0; e < N; ++e) ssk += v[e] * v[e];
   }
-  const float inv_q = rsqrtf(block_sum_f(ssq, red) / static_cast<float>(q_rank) + eps);
-  const float inv_k = rsqrtf(block_sum_f(ssk, red) / static_cast<float>(kv_rank) + eps);
+  ssq = warp_sum_f(ssq);
+  ssk = warp_sum_f(ssk);
+  if ((threadIdx.x & 31) == 0) {
+    red[threadIdx.x >> 5] = ssq;
+    red[4 + (threadIdx.x >> 5)] = ssk;
+  }
+  __syncthreads();                                 // four warps
+  const float inv_q = rsqrtf((red[0] + red[1] + red[2] + red[3]) / static_cast<float>(q_rank) + eps);
+  const float inv_k = rsqrtf((red[4] + red[5] + red[6] + red[7]) / static_cast<float>(kv_rank) + eps);
   T* q_out = cq + static_cast<size_t>(t) * q_rank;
   for (int i = threadIdx.x * N; i < q_rank; i += blockDim.x * N) {
     float v[N], w[N];

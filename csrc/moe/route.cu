@@ -120,19 +120,21 @@ extern "C" int forge_moe_plan(const int* experts, int n, int E, int tile, int ma
 }
 
 template <typename T, int N>
-__global__ void __launch_bounds__(128) moe_scatter_kernel(const T* __restrict__ h, const int* __restrict__ pos,
+__global__ void __launch_bounds__(256) moe_scatter_kernel(const T* __restrict__ h, const int* __restrict__ pos,
                                                           const float* __restrict__ weights, int top, int W, T* __restrict__ xs) {
   pdl_launch_dependents();
   pdl_wait();
-  const size_t i = blockIdx.x, t = i / top;
-  const float s = weights[i];
-  T* dst = xs + static_cast<size_t>(pos[i]) * W;
+  const size_t t = blockIdx.x;
   for (int c = threadIdx.x * N; c < W; c += blockDim.x * N) {
     float v[N];
     load_n<N>(h + t * W + c, v);
+    for (int j = 0; j < top; ++j) {
+      const float s = weights[t * top + j];
+      float x[N];
 #pragma unroll
-    for (int e = 0; e < N; ++e) v[e] *= s;
-    store_n<N>(dst + c, v);
+      for (int e = 0; e < N; ++e) x[e] = s * v[e];
+      store_n<N>(xs + static_cast<size_t>(pos[t * top + j]) * W + c, x);
+    }
   }
 }
 
@@ -142,10 +144,10 @@ extern "C" int forge_moe_scatter(int fp32, const void* h, const int* pos, const 
   const bool v4 = (W & 3) == 0;
   if (fp32) {
     auto k = v4 ? moe_scatter_kernel<float, 4> : moe_scatter_kernel<float, 1>;
-    return launch_kernel(k, dim3(n), dim3(128), 0, stream, 0, static_cast<const float*>(h), pos, weights, top, W, static_cast<float*>(xs)) == cudaSuccess ? 0 : -2;
+    return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const float*>(h), pos, weights, top, W, static_cast<float*>(xs)) == cudaSuccess ? 0 : -2;
   }
   auto k = v4 ? moe_scatter_kernel<bf16, 4> : moe_scatter_kernel<bf16, 1>;
-  return launch_kernel(k, dim3(n), dim3(128), 0, stream, 0, static_cast<const bf16*>(h), pos, weights, top, W, static_cast<bf16*>(xs)) == cudaSuccess ? 0 : -2;
+  return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const bf16*>(h), pos, weights, top, W, static_cast<bf16*>(xs)) == cudaSuccess ? 0 : -2;
 }
 
 }  // namespace forge

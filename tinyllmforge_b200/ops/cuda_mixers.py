@@ -153,6 +153,11 @@ class MixerOps:
         return max(1, -(-longest // seg_len)), seg_len
 
     # ------------------------------------------------------------------ experts
+    @staticmethod
+    def expert_tile(rows: int, experts: int) -> int:
+        """Rows per tile of the tensor-core kernel (16 to 128): about what an expert gets."""
+        return next((t for t in (16, 32, 64) if rows <= t * experts), 128)
+
     def moe(self, h, router, gate_up, down, top):
         T, W = h.shape
         E, n = router.shape[0], T * top
@@ -160,9 +165,7 @@ class MixerOps:
         weights = torch.empty(T, top, dtype=torch.float32, device=h.device)
         self.C.router(h, router, experts, weights)
         fast = h.dtype == torch.bfloat16 and W % 8 == 0 and down.shape[2] % 8 == 0
-        tile = 64                                   # rows per tile; the tensor-core kernel takes 16 to 128
-        if fast:
-            tile = next((t for t in (16, 32, 64) if n <= t * E), 128)
+        tile = self.expert_tile(n, E) if fast else 64
         tiles = min(n, n // tile + E)
         rows = torch.empty(T, top, dtype=torch.int32, device=h.device)
         tile_expert = torch.empty(tiles, dtype=torch.int32, device=h.device)

@@ -7,7 +7,8 @@ decode_attention_g8 (64 x 2304, 64 / 8 heads: Qwen3-32B), prefill_attention, gem
 gemm_prefill_8b (8192 x 6144 x 4096), gemm_silu, gemm_fp8 (256 x 6144 x 4096, block-scaled e4m3 weights), gemm_residual (o_proj-like GEMM with the residual add + sums of squares
 epilogue), gemm_scaled (qkv-like GEMM with the folded-norm row scale), gemm_decode_8b_down (256 x 4096 x 12288 with the residual
 epilogue: K split over CTA pairs + the reduce kernel), lm_head_sample (LM head + sampling in one kernel),
-rms_norm, qk_norm_rope_store, sampler.
+rms_norm, qk_norm_rope_store, sampler; and those of ``mixer_cases.CASES`` (latent attention, retention, experts, residual
+stream).  Several cases may be given, separated by commas.
 ``--lib`` runs the library kernel the reference would use on the same case instead (cuBLAS through torch.matmul for the
 GEMMs, flash-attn 2 for the attention cases), for a same-box comparison.
 Prints the mean device time per launch (CUDA events) and the achieved fraction of the roofline denominator that applies:
@@ -21,6 +22,8 @@ import json
 import os
 
 import torch
+
+from .mixer_cases import CASES
 
 BF = torch.bfloat16
 
@@ -158,6 +161,8 @@ def build(case: str, ops, lib: bool = False):
         temps = torch.full((256,), 0.6, device="cuda")
         hdr = torch.zeros(16, dtype=torch.int32, device="cuda")
         return (lambda: ops.sample_shard(logits, temps, hdr, 0)), 256 * 151936 * 2, 0
+    if case in CASES and not lib:
+        return CASES[case](ops)
     raise SystemExit(f"unknown case {case!r}")
 
 
@@ -170,7 +175,12 @@ def main():
     args = ap.parse_args()
     from ..ops.cuda import CudaOps
     ops = CudaOps()
-    fn, nbytes, flops = build(args.case, ops, args.lib)
+    for case in args.case.split(","):
+        run_case(case, ops, args)
+
+
+def run_case(case, ops, args):
+    fn, nbytes, flops = build(case, ops, args.lib)
     for _ in range(3):
         fn()
     torch.cuda.synchronize()
@@ -183,14 +193,14 @@ def main():
     ops.check_status()
     us = e0.elapsed_time(e1) * 1e3 / args.iters
     hbm, tf, src = _peaks(args.peaks)
-    out = {"case": args.case + (" (library kernel)" if args.lib else ""), "us_per_launch": round(us, 2)}
+    out = {"case": case + (" (library kernel)" if args.lib else ""), "us_per_launch": round(us, 2)}
     if nbytes:
         out["GB_per_s"] = round(nbytes / us / 1e3, 1)
         out[f"fraction_of_{src}_copy_bandwidth"] = round(nbytes / us / 1e3 / hbm, 3)
     if flops:
         out["TFLOP_per_s"] = round(flops / us / 1e6, 1)
         out[f"fraction_of_{src}_bf16_gemm_rate"] = round(flops / us / 1e6 / tf, 3)
-    print(json.dumps(out))
+    print(json.dumps(out), flush=True)
 
 
 if __name__ == "__main__":
