@@ -8,7 +8,8 @@
 // accumulator registers; where it, the decayed scores or the decayed keys are operands of a product they enter as bf16
 // hi + lo halves (two products, 16 mantissa bits).  q and k come rotated (retention_rotate, in place).
 //
-// CTA = (64 columns of the values, head, sequence x segment), eight warps.  A long run is cut into segments so that a few long
+// CTA = (columns of the values, head, sequence x segment).  Two shapes: 16 warps over 128 columns with the next chunk's rows on
+// their way while this one is computed (heads up to 128 wide), or 8 warps over 64 columns.  A long run is cut into segments so that a few long
 // prompts fill the GPU: the segments' own end states are computed first, a scan over them gives every segment its initial
 // state, and then all segments compute their outputs at the same time.
 #include "../include/launch.cuh"
@@ -17,7 +18,7 @@
 
 namespace forge {
 
-constexpr int kRC = 64, kRThreads = 256, kRPitch = 72;     // tokens per chunk; 64 columns + 8 (odd number of 16-byte units)
+constexpr int kRC = 64, kRPP = kRC + 8;      // tokens per chunk; row pitch of the decayed scores (odd number of 16-byte units)
 
 struct RetentionChunk {
   const bf16* qkvg;         // [tokens][ld], q and k rotated
@@ -43,20 +44,21 @@ __device__ __forceinline__ void weigh_split(const uint32_t* a, float w0, float w
   }
 }
 
-template <int MT, bool kStateOnly>
-__global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_kernel(const RetentionChunk p) {
+// kWide: 16 warps, 128 columns, two stages; else 8 warps, 64 columns, one stage.  MT: 16-row tiles of the state per warp.
+template <int MT, bool kStateOnly, bool kWide>
+__global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) retention_chunk_kernel(const RetentionChunk p) {
+  constexpr int kWarps = kWide ? 16 : 8, kQuarters = kWarps / 4, kCols = 32 * kQuarters, kRPitch = kCols + 8, kStages = kWide ? 2 : 1;
+  constexpr int kKB = 8 / kQuarters;                                   // 8-key blocks of the scores per warp
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int kp = p.dk + 8;                                             // dk is a multiple of 16: an odd number of units
-  bf16* sq = reinterpret_cast<bf16*>(smem_raw);                        // [64][kp]
-  bf16* sk = sq + kRC * kp;                                            // [64][kp]
-  bf16* sv = sk + kRC * kp;                                            // [64][72]
-  bf16* sS = sv + kRC * kRPitch;                                       // [hi, lo][dk][72]
-  bf16* sP = sS + 2 * p.dk * kRPitch;                                  // [hi, lo][64][72]
-  float* pw = reinterpret_cast<float*>(sP + 2 * kRC * kRPitch);        // [65]: g^i
+  const int stage = kRC * (2 * kp + kRPitch);                          // elements: q [64][kp], k [64][kp], v [64][kRPitch]
+  bf16* sS = reinterpret_cast<bf16*>(smem_raw) + kStages * stage;      // [hi, lo][dk][kRPitch]
+  bf16* sP = sS + 2 * p.dk * kRPitch;                                  // [hi, lo][64][kRPP]
+  float* pw = reinterpret_cast<float*>(sP + 2 * kRC * kRPP);           // [65]: g^i
 
   pdl_launch_dependents();
   pdl_wait();
-  const int c0 = blockIdx.x * 64, h = blockIdx.y;
+  const int c0 = blockIdx.x * kCols, h = blockIdx.y;
   const int seq = blockIdx.z / p.segs, seg = blockIdx.z % p.segs;
   const int run = p.cu[seq + 1] - p.cu[seq];
   const int n_segs = p.segs == 1 ? 1 : min((run + p.seg_len - 1) / p.seg_len, p.segs);
@@ -73,17 +75,17 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
   if (threadIdx.x <= kRC) pw[threadIdx.x] = powf(p.decay[h], static_cast<float>(threadIdx.x));
 
   const int steps = p.dk >> 4;
-  const bool both = steps > 4;                     // a warp owns both column halves of its state rows, or one of them
+  const bool both = steps > 4;                     // a warp owns two 32-column parts of its state rows, or one
   const size_t head_state = static_cast<size_t>(p.dk) * p.dv;
   float* slot_state = p.state + (static_cast<size_t>(slot) * p.heads + h) * head_state;
   float* seg_state = p.segs == 1 ? nullptr : p.ws + ((static_cast<size_t>(seq) * p.segs + seg) * p.heads + h) * head_state;
   const bool fresh = p.positions[p.cu[seq]] == 0;
   const float* init = kStateOnly ? nullptr : (p.segs > 1 ? seg_state : (fresh ? nullptr : slot_state));
 
-  // state fragments: rows mt * 16 + g4 (+ 8), columns half * 32 + nb * 8 + q2 (+ 1)
+  // state fragments: rows row_tile * 16 + g4 (+ 8), columns col_part * 32 + nb * 8 + q2 (+ 1)
   float st[MT][2][4][4];
-  auto row_tile = [&](int m) { return both ? warp + 8 * m : (warp & 3); };
-  auto col_half = [&](int i) { return both ? i : (warp >> 2); };
+  auto row_tile = [&](int m) { return both ? (warp & 7) + 8 * m : (warp & 3); };
+  auto col_part = [&](int i) { return both ? (warp >> 3) * 2 + i : (warp >> 2); };
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -92,16 +94,17 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
       for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int r = row_tile(m) * 16 + g4 + (e >> 1) * 8, c = c0 + col_half(i) * 32 + nb * 8 + q2 + (e & 1);
+          const int r = row_tile(m) * 16 + g4 + (e >> 1) * 8, c = c0 + col_part(i) * 32 + nb * 8 + q2 + (e & 1);
           st[m][i][nb][e] = (init != nullptr && (both || i == 0) && r < p.dk && c < p.dv) ? init[static_cast<size_t>(r) * p.dv + c] : 0.f;
         }
 
   const int units = p.dk >> 3;
-  for (int t0 = t_begin; t0 < t_end; t0 += kRC) {
-    const int L = min(kRC, t_end - t0);
-    __syncthreads();                                                   // the chunk before is done with shared memory
-    for (int r = warp; r < kRC; r += 8) {
-      const bool in = r < L;
+  auto load_chunk = [&](int t0, int st) {
+    bf16* sq = reinterpret_cast<bf16*>(smem_raw) + st * stage;
+    bf16* sk = sq + kRC * kp;
+    bf16* sv = sk + kRC * kp;
+    for (int r = warp; r < kRC; r += kWarps) {
+      const bool in = t0 + r < t_end;
       const bf16* row = p.qkvg + static_cast<size_t>(in ? t0 + r : t0) * p.ld;
       const bf16* qr = row + h * p.dk;
       const bf16* kr = row + (p.heads + h) * p.dk;
@@ -110,12 +113,27 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
         if (!kStateOnly) cp_async16(smem_u32(sq + r * kp + u * 8), qr + u * 8, in ? 16 : 0);
         cp_async16(smem_u32(sk + r * kp + u * 8), kr + u * 8, in ? 16 : 0);
       }
-      if (lane < 8) {
+      if (lane < kCols / 8) {
         const bool vin = in && c0 + lane * 8 < p.dv;
         cp_async16(smem_u32(sv + r * kRPitch + lane * 8), vin ? vr + lane * 8 : row, vin ? 16 : 0);
       }
     }
+  };
+  if (kStages == 2) {
+    load_chunk(t_begin, 0);
     cp_async_commit();
+  }
+  int st_now = 0;
+  for (int t0 = t_begin; t0 < t_end; t0 += kRC) {
+    const int L = min(kRC, t_end - t0);
+    __syncthreads();                                                   // the chunk before is done with shared memory
+    if (kStages == 1) load_chunk(t0, 0);
+    else if (t0 + kRC < t_end) load_chunk(t0 + kRC, st_now ^ 1);
+    cp_async_commit();
+    const bf16* sq = reinterpret_cast<bf16*>(smem_raw) + st_now * stage;
+    const bf16* sk = sq + kRC * kp;
+    const bf16* sv = sk + kRC * kp;
+    st_now ^= kStages - 1;
     if (!kStateOnly) {                                                 // the state before this chunk as hi and lo operands
 #pragma unroll
       for (int m = 0; m < MT; ++m)
@@ -126,7 +144,7 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
           for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-              bf16* dst = sS + (row_tile(m) * 16 + g4 + e * 8) * kRPitch + col_half(i) * 32 + nb * 8 + q2;
+              bf16* dst = sS + (row_tile(m) * 16 + g4 + e * 8) * kRPitch + col_part(i) * 32 + nb * 8 + q2;
               const float x = st[m][i][nb][2 * e], y = st[m][i][nb][2 * e + 1];
               const uint32_t hi = pack_bf16x2(x, y);
               *reinterpret_cast<uint32_t*>(dst) = hi;
@@ -134,24 +152,24 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
             }
         }
     }
-    cp_async_wait<0>();
+    cp_async_wait<kStages - 1>();
     __syncthreads();
 
     if (!kStateOnly) {
-      const int mt = warp & 3, nh = warp >> 2;                         // 16 tokens; 32 keys, then 32 value columns
-      float s[4][4], o[4][4];
+      const int mt = warp & 3, nh = warp >> 2;                         // 16 tokens; 8 kKB keys, then 32 value columns
+      float s[kKB][4], o[4][4];
 #pragma unroll
       for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[nb][e] = o[nb][e] = 0.f;
-      const bool any_key = nh * 32 <= mt * 16 + 15;
+        for (int e = 0; e < 4; ++e) o[nb][e] = s[nb % kKB][e] = 0.f;
+      const bool any_key = nh * 8 * kKB <= mt * 16 + 15;
       for (int k = 0; k < steps; ++k) {
         uint32_t a[4], b[4];
         ldsm_x4(smem_u32(sq + (mt * 16 + (lane & 15)) * kp + k * 16 + (lane >> 4) * 8), a);
         if (any_key) {
 #pragma unroll
-          for (int nb = 0; nb < 4; nb += 2) {
-            ldsm_x4(smem_u32(sk + (nh * 32 + nb * 8 + (lane & 7) + (lane >> 4) * 8) * kp + k * 16 + ((lane >> 3) & 1) * 8), b);
+          for (int nb = 0; nb < kKB; nb += 2) {
+            ldsm_x4(smem_u32(sk + (nh * 8 * kKB + nb * 8 + (lane & 7) + (lane >> 4) * 8) * kp + k * 16 + ((lane >> 3) & 1) * 8), b);
             mma16816(s[nb], a, b[0], b[1]);
             mma16816(s[nb + 1], a, b[2], b[3]);
           }
@@ -168,25 +186,30 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
         }
       }
 #pragma unroll
-      for (int nb = 0; nb < 4; ++nb)
+      for (int e = 0; e < 2; ++e) {
+        const int i = mt * 16 + g4 + e * 8;
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int i = mt * 16 + g4 + e * 8, j = nh * 32 + nb * 8 + q2;
+        for (int nb = 0; nb < kKB; ++nb) {
+          const int j = nh * 8 * kKB + nb * 8 + q2;
           const float x = j <= i ? s[nb][2 * e] * (pw[i - j] * ks) : 0.f;
           const float y = j + 1 <= i ? s[nb][2 * e + 1] * (pw[i - j - 1] * ks) : 0.f;
           const uint32_t hi = pack_bf16x2(x, y);
-          bf16* dst = sP + i * kRPitch + j;
+          bf16* dst = sP + i * kRPP + j;
           *reinterpret_cast<uint32_t*>(dst) = hi;
-          *reinterpret_cast<uint32_t*>(dst + kRC * kRPitch) = pack_bf16x2(x - bf16_lo(hi), y - bf16_hi(hi));
+          *reinterpret_cast<uint32_t*>(dst + kRC * kRPP) = pack_bf16x2(x - bf16_lo(hi), y - bf16_hi(hi));
+        }
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) {
           o[nb][2 * e] *= pw[i + 1];
           o[nb][2 * e + 1] *= pw[i + 1];
         }
+      }
       __syncthreads();
       for (int k = 0; k <= mt; ++k) {                                  // keys up to this warp's last token
         uint32_t ah[4], al[4], b[4];
-        const uint32_t at = smem_u32(sP + (mt * 16 + (lane & 15)) * kRPitch + k * 16 + (lane >> 4) * 8);
+        const uint32_t at = smem_u32(sP + (mt * 16 + (lane & 15)) * kRPP + k * 16 + (lane >> 4) * 8);
         ldsm_x4(at, ah);
-        ldsm_x4(at + kRC * kRPitch * 2, al);
+        ldsm_x4(at + kRC * kRPP * 2, al);
         const bf16* vr = sv + (k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kRPitch + nh * 32 + (lane >> 4) * 8;
 #pragma unroll
         for (int nb = 0; nb < 4; nb += 2) {
@@ -237,7 +260,7 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
           if (!both && i == 1) continue;
 #pragma unroll
           for (int nb = 0; nb < 4; nb += 2) {
-            ldsm_x4_trans(smem_u32(vr + col_half(i) * 32 + nb * 8), b);
+            ldsm_x4_trans(smem_u32(vr + col_part(i) * 32 + nb * 8), b);
             mma16816(st[m][i][nb], ah, b[0], b[1]);
             mma16816(st[m][i][nb + 1], ah, b[2], b[3]);
             mma16816(st[m][i][nb], al, b[0], b[1]);
@@ -258,7 +281,7 @@ __global__ void __launch_bounds__(kRThreads, MT == 1 ? 2 : 1) retention_chunk_ke
       for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int r = row_tile(m) * 16 + g4 + e * 8, c = c0 + col_half(i) * 32 + nb * 8 + q2;
+          const int r = row_tile(m) * 16 + g4 + e * 8, c = c0 + col_part(i) * 32 + nb * 8 + q2;
           if ((both || i == 0) && r < p.dk && c < p.dv)
             *reinterpret_cast<float2*>(dst + static_cast<size_t>(r) * p.dv + c) = make_float2(st[m][i][nb][2 * e], st[m][i][nb][2 * e + 1]);
         }
@@ -317,9 +340,13 @@ __global__ void __launch_bounds__(128) retention_rotate_kernel(bf16* __restrict_
   }
 }
 
-static size_t retention_chunk_smem(int dk) {
-  return static_cast<size_t>(2 * kRC * (dk + 8) + kRC * kRPitch + 2 * dk * kRPitch + 2 * kRC * kRPitch) * 2 + (kRC + 1) * 4;
+static size_t retention_chunk_smem(int dk, bool wide) {
+  const int pitch = wide ? 136 : 72;
+  return static_cast<size_t>((wide ? 2 : 1) * kRC * (2 * (dk + 8) + pitch) + 2 * dk * pitch + 2 * kRC * kRPP) * 2 + (kRC + 1) * 4;
 }
+
+// Value columns per CTA for these sizes.
+extern "C" int forge_retention_chunk_cols(int dk, int dv) { return dk <= 128 && dv > 64 ? 128 : 64; }
 
 // 1 if the kernels take these sizes (else: retention_scan).
 extern "C" int forge_retention_chunk_ok(int heads, int dk, int dv, int rd) {
@@ -340,19 +367,21 @@ extern "C" int forge_retention_chunk(void* qkvg, int ld, const float* decay, flo
                               dk, rd, rope, rope_rows, positions) != cudaSuccess)
     return -2;
   const RetentionChunk p = {static_cast<const bf16*>(qkvg), ld, decay, state, slots, positions, cu, ws, o, heads, dk, dv, num_slots, segs, seg_len, status};
-  const dim3 grid((dv + 63) / 64, heads, seqs * segs);
-  const size_t smem = retention_chunk_smem(dk);
-#define FORGE_RC(MT, ONLY)                                                                                                 \
+  const int cols = forge_retention_chunk_cols(dk, dv);
+  const bool wide = cols == 128;
+  const dim3 grid((dv + cols - 1) / cols, heads, seqs * segs);
+  const size_t smem = retention_chunk_smem(dk, wide);
+#define FORGE_RC(MT, ONLY, WIDE)                                                                                           \
   {                                                                                                                        \
-    auto k = retention_chunk_kernel<MT, ONLY>;                                                                             \
-    FORGE_ENSURE_DYN_SMEM(k, static_cast<int>(retention_chunk_smem(128 * MT)));                                            \
-    if (launch_kernel(k, grid, dim3(kRThreads), smem, stream, 0, p) != cudaSuccess) return -2;                             \
+    auto k = retention_chunk_kernel<MT, ONLY, WIDE>;                                                                       \
+    FORGE_ENSURE_DYN_SMEM(k, static_cast<int>(retention_chunk_smem(128 * MT, WIDE)));                                      \
+    if (launch_kernel(k, grid, dim3(WIDE ? 512 : 256), smem, stream, 0, p) != cudaSuccess) return -2;                      \
   }
   if (segs > 1) {
-    if (dk <= 128) FORGE_RC(1, true) else FORGE_RC(2, true)
+    if (wide) FORGE_RC(1, true, true) else if (dk <= 128) FORGE_RC(1, true, false) else FORGE_RC(2, true, false)
     if (launch_kernel(retention_segments_kernel, dim3((dk * dv / 4 + 255) / 256, heads, seqs), dim3(256), 0, stream, 0, p) != cudaSuccess) return -2;
   }
-  if (dk <= 128) FORGE_RC(1, false) else FORGE_RC(2, false)
+  if (wide) FORGE_RC(1, false, true) else if (dk <= 128) FORGE_RC(1, false, false) else FORGE_RC(2, false, false)
 #undef FORGE_RC
   return 0;
 }

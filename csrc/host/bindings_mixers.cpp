@@ -50,6 +50,7 @@ int forge_latent_gather(const void* cache, const int* cu_k, int num_seqs, const 
 int forge_latent_pack_q(const void* q, void* qp, int tokens, int heads, int dim, int rot, const float* rope, int rope_rows,
                         const int* positions, cudaStream_t stream);
 int forge_retention_chunk_ok(int heads, int dk, int dv, int rd);
+int forge_retention_chunk_cols(int dk, int dv);
 int forge_retention_chunk(void* qkvg, int ld, const float* decay, float* state, const int* slots, const int* positions, const float* rope,
                           int rope_rows, int rd, const int* cu, int seqs, int tok0, int tokens, int heads, int dk, int dv, int num_slots,
                           float* o, float* ws, int segs, int seg_len, unsigned* status, cudaStream_t stream);
@@ -421,5 +422,6 @@ void register_mixers(pybind11::module& m) {
   m.def("latent_prefill", &latent_prefill);
   m.def("latent_prefill_qcols", [](int64_t dim, int64_t rot, int64_t vdim) { return forge_latent_prefill_qcols(i32(dim), i32(rot), i32(vdim)); });
   m.def("retention_chunk", &retention_chunk);
+  m.def("retention_chunk_cols", [](int64_t dk, int64_t dv) { return forge_retention_chunk_cols(i32(dk), i32(dv)); });
   m.def("retention_chunk_ok", [](int64_t H, int64_t dk, int64_t dv, int64_t rd) { return forge_retention_chunk_ok(i32(H), i32(dk), i32(dv), i32(rd)) != 0; });
 }

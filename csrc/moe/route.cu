@@ -1,15 +1,104 @@
 // Mixture of experts: routing and the shuffling of rows.
 //
-//   router_scores   logits (fp32) -> sigmoid -> the `top` largest scores of a token (ties: the lower expert)
+//   router          logits (fp32) -> sigmoid -> the `top` largest scores of a token (ties: the lower expert)
 //   moe_plan        (token, choice) -> row of the expert-sorted buffer; every expert's rows start on a multiple of `tile`, so
 //                   a tile of rows has one expert (tile_expert; -1 past the last tile in use)
 //   moe_scatter     row = score * token, the score in fp32: it multiplies the expert's INPUT
 //
 // Rows between an expert's last token and its next tile boundary are never written nor read back.
 #include "../include/launch.cuh"
+#include "../include/mma_sync.cuh"
 #include "../include/scalar.cuh"
 
 namespace forge {
+
+// The `top` largest of a token's scores, by one warp; the scores in shared memory are used up.
+__device__ __forceinline__ void choose_top(float* score, int E, int top, int lane, int* experts, float* weights) {
+  for (int j = 0; j < top; ++j) {
+    float best = -1.f;
+    int at = E;
+    for (int e = lane; e < E; e += 32)
+      if (score[e] > best) { best = score[e]; at = e; }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+      const float v = __shfl_xor_sync(0xffffffffu, best, off);
+      const int i = __shfl_xor_sync(0xffffffffu, at, off);
+      if (v > best || (v == best && i < at)) { best = v; at = i; }
+    }
+    if (at >= E) at = 0;                          // only if every score is NaN
+    if (lane == 0) {
+      experts[j] = at;
+      weights[j] = best;
+      score[at] = -2.f;
+    }
+    __syncwarp();
+  }
+}
+
+// bf16, W a multiple of 32, E <= 256: CTA = 16 MT tokens, the eight warps split W.  The order of the columns in a dot product is
+// free, so a lane loads eight consecutive columns of its row (16 bytes) and uses them as the four column pairs of two mma
+// k-steps, for tokens and experts alike: no shared memory on the way in.  The warps' partial logits are added in a fixed order.
+template <int MT>
+__global__ void __launch_bounds__(256) router_mma_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w, int T, int W, int E, int top,
+                                                         int* __restrict__ experts, float* __restrict__ weights) {
+  extern __shared__ float sm_part[];               // [8][16 MT][Ep]
+  constexpr int kTok = 16 * MT, kGroup = 8;        // 8-expert blocks per pass
+  const int Ep = (E + 7) & ~7;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
+  const int t0 = blockIdx.x * kTok;
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int e0 = 0; e0 < E; e0 += 8 * kGroup) {
+    float acc[MT][kGroup][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < kGroup; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
+    for (int c = warp * 32; c < W; c += 256) {
+      uint4 a[MT][2];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = t0 + m * 16 + r * 8 + g;
+          a[m][r] = t < T ? *reinterpret_cast<const uint4*>(h + static_cast<size_t>(t) * W + c + q * 8) : make_uint4(0, 0, 0, 0);
+        }
+#pragma unroll
+      for (int n = 0; n < kGroup; ++n) {
+        const int e = e0 + n * 8 + g;
+        if (e0 + n * 8 >= E) continue;
+        const uint4 b = e < E ? *reinterpret_cast<const uint4*>(w + static_cast<size_t>(e) * W + c + q * 8) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          const uint32_t lo[4] = {a[m][0].x, a[m][1].x, a[m][0].y, a[m][1].y}, hi[4] = {a[m][0].z, a[m][1].z, a[m][0].w, a[m][1].w};
+          mma16816(acc[m][n], lo, b.x, b.y);
+          mma16816(acc[m][n], hi, b.z, b.w);
+        }
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < kGroup; ++n) {
+        if (e0 + n * 8 >= E) continue;
+        float* dst = sm_part + (static_cast<size_t>(warp) * kTok + m * 16 + g) * Ep + e0 + n * 8 + 2 * q;
+        *reinterpret_cast<float2*>(dst) = make_float2(acc[m][n][0], acc[m][n][1]);
+        *reinterpret_cast<float2*>(dst + 8 * Ep) = make_float2(acc[m][n][2], acc[m][n][3]);
+      }
+  }
+  __syncthreads();
+  for (int t = warp; t < kTok && t0 + t < T; t += 8) {
+    float* score = sm_part + static_cast<size_t>(t) * Ep;
+    for (int e = lane; e < E; e += 32) {
+      float z = score[e];
+#pragma unroll
+      for (int k = 1; k < 8; ++k) z += score[static_cast<size_t>(k) * kTok * Ep + e];
+      score[e] = 1.f / (1.f + expf(-z));
+    }
+    __syncwarp();
+    choose_top(score, E, top, lane, experts + static_cast<size_t>(t0 + t) * top, weights + static_cast<size_t>(t0 + t) * top);
+  }
+}
 
 // CTA = one token; one warp per expert at a time.
 template <typename T, int N>
@@ -35,26 +124,7 @@ __global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, co
     if (lane == 0) score[e] = 1.f / (1.f + expf(-z));
   }
   __syncthreads();
-  if (warp != 0) return;
-  for (int j = 0; j < top; ++j) {
-    float best = -1.f;
-    int at = E;
-    for (int e = lane; e < E; e += 32)
-      if (score[e] > best) { best = score[e]; at = e; }
-#pragma unroll
-    for (int off = 16; off > 0; off >>= 1) {
-      const float v = __shfl_xor_sync(0xffffffffu, best, off);
-      const int i = __shfl_xor_sync(0xffffffffu, at, off);
-      if (v > best || (v == best && i < at)) { best = v; at = i; }
-    }
-    if (at >= E) at = 0;                          // only if every score is NaN
-    if (lane == 0) {
-      experts[t * top + j] = at;
-      weights[t * top + j] = best;
-      score[at] = -2.f;
-    }
-    __syncwarp();
-  }
+  if (warp == 0) choose_top(score, E, top, lane, experts + t * top, weights + t * top);
 }
 
 extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int W, int E, int top, int* experts, float* weights,
@@ -66,6 +136,18 @@ extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int 
   if (fp32) {
     auto k = v4 ? router_kernel<float, 4> : router_kernel<float, 1>;
     return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+  }
+  if (W % 32 == 0 && E <= 256 && (reinterpret_cast<uintptr_t>(h) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
+    const int Ep = (E + 7) & ~7;
+    const bool two = T_ > 2048 && E <= 128;        // more tokens per CTA halve the reads of the router matrix
+    const dim3 grid((T_ + (two ? 31 : 15)) / (two ? 32 : 16));
+    const size_t part = static_cast<size_t>(8) * (two ? 32 : 16) * Ep * 4;
+    if (two) {
+      FORGE_ENSURE_DYN_SMEM(router_mma_kernel<2>, 8 * 32 * 128 * 4);
+      return launch_kernel(router_mma_kernel<2>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+    }
+    FORGE_ENSURE_DYN_SMEM(router_mma_kernel<1>, 8 * 16 * 256 * 4);
+    return launch_kernel(router_mma_kernel<1>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
   }
   auto k = v4 ? router_kernel<bf16, 4> : router_kernel<bf16, 1>;
   return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, experts, weights) == cudaSuccess ? 0 : -2;

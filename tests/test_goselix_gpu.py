@@ -298,7 +298,7 @@ def test_retention_decode(ops, name, dtype):
 def test_retention_segments(ops, name):
     """One long run is cut into segments; the state crosses them.  The token scan of the oracle has no segments."""
     s = RETENTION[name]
-    assert ops.retention_segments(1, s.heads, s.vdim, 1500)[0] > 1
+    assert ops.retention_segments(1, s.heads, s.dim, s.vdim, 1500)[0] > 1
     retention_check(ops, s, BF, [(0, 1500)], seed=3)
     retention_check(ops, s, BF, [(11, 1211)], seed=4)
     retention_check(ops, s, BF, [(0, 1100), (64, 75), (2, 770)], seed=5)

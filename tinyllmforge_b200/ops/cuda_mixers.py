@@ -74,9 +74,10 @@ class MixerOps:
         return out
 
     def latent_chunking(self, seqs: int, heads: int, max_len: int) -> tuple[int, int]:
-        """(keys per chunk, chunks) of the decode kernel: enough chunks to fill the GPU, from shapes known at capture time."""
-        ctas = seqs * -(-heads // 16)
-        want = -(-2 * self.num_sms // ctas)                       # chunks per sequence for two CTAs per SM
+        """(keys per chunk, chunks) of the decode kernel: enough chunks to fill the GPU once or
+        twice, from shapes known at capture time."""
+        ctas = seqs * (-(-heads // 32) if heads > 16 else 1)      # 16 heads per CTA and two CTAs per SM, or 32 and one
+        want = -(-self.num_sms * (1 if heads > 16 else 2) // ctas)
         chunk = 64
         while chunk < 1024 and -(-max_len // (2 * chunk)) >= want:
             chunk *= 2
@@ -136,7 +137,7 @@ class MixerOps:
             o = torch.empty(T, H * dv, dtype=torch.float32, device=qkvg.device)
             slots, cu = batch.state_slots[n1:], batch.cu_seqlens_q[n1:]
             if qkvg.dtype == torch.bfloat16 and self.C.retention_chunk_ok(H, spec.dim, dv, table.shape[1]):
-                segs, seg_len = self.retention_segments(rest, H, dv, batch.max_seqlen_q)
+                segs, seg_len = self.retention_segments(rest, H, spec.dim, dv, batch.max_seqlen_q)
                 ws = torch.empty(rest * segs * H * spec.dim * dv, dtype=torch.float32, device=qkvg.device) if segs > 1 else None
                 self.C.retention_chunk(qkvg, decay, state, slots, batch.positions, table, cu, rest, n1, o, ws, segs, seg_len, self.status)
             else:
@@ -144,9 +145,10 @@ class MixerOps:
             self.C.retention_gate(o, qkvg, y, n1, H, dv, eps)
         return y
 
-    def retention_segments(self, seqs: int, heads: int, dv: int, longest: int) -> tuple[int, int]:
-        """(segments per run, tokens per segment): a run is cut when the batch alone does not give two CTAs per SM."""
-        want = 2 * self.num_sms // (seqs * heads * -(-dv // 64))
+    def retention_segments(self, seqs: int, heads: int, dk: int, dv: int, longest: int) -> tuple[int, int]:
+        """(segments per run, tokens per segment): a run is cut when the batch alone leaves half of the CTA places empty."""
+        cols = self.C.retention_chunk_cols(dk, dv)
+        want = (self.num_sms if cols == 128 or dk > 128 else 2 * self.num_sms) // (seqs * heads * -(-dv // cols))
         segs = max(1, min(want, longest // 256))
         seg_len = -(-longest // segs)
         seg_len = -(-seg_len // 64) * 64

@@ -64,7 +64,7 @@ def _retention_prefill(ops, S, n):
     decay = torch.linspace(0.9, 0.9999, s.heads, device="cuda")
     cu, slots, pos = _ints([i * n for i in range(S + 1)]), _ints(list(range(S))), _ints(list(range(n)) * S)
     o = torch.empty(T, s.heads * s.vdim, device="cuda")
-    segs, seg_len = ops.retention_segments(S, s.heads, s.vdim, n)
+    segs, seg_len = ops.retention_segments(S, s.heads, s.dim, s.vdim, n)
     ws = torch.empty(S * segs * s.heads * s.dim * s.vdim, device="cuda")
     table = _rope(n, 128)
     flops = T * s.heads * (4 * s.dim * s.vdim + C * (s.dim + s.vdim))
