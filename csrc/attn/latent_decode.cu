@@ -1,28 +1,27 @@
-// Latent attention of single query tokens on the tensor cores, straight over the paged latents [blocks][block_size][R + rot].
+// Latent attention of single query tokens on the 5th-generation tensor cores, straight over the paged latents
+// [blocks][block_size][R + rot].
 //
 // The queries come folded (W_k^T q | rotated part), so all heads of a token share one key row per cached token (its whole
-// latent row) and one value row (the first R entries of the SAME row): a tile of keys is read from memory once and serves
-// both products for 16 or 32 heads.  CTA = (context chunk, group of 16 kMT heads, sequence), eight warps:
+// latent row) and one value row (the first R entries of the SAME row): a tile of 128 keys is read from memory once and serves
+// both products for up to 32 heads.  The keys and latents are the UMMA's 128-row side, the heads ride the N side:
 //
-//   S = Q K^T    mma.sync m16n8k16, M = 16 heads.  Warp (slice, half) multiplies a quarter of the D columns of Q (held in
-//                registers for the whole chunk) with half of the tile's keys; the four partial sums meet in shared memory.
-//   softmax      fp32, 16 / kMT threads per head, running maximum and sum in registers.
-//   O += P V     every warp owns R / 8 columns.  P is fp32: it enters as bf16 hi + lo halves (two products), so the weights
-//                keep 16 mantissa bits.
+//   S^T = K Q^T     A = the key tile as TMA delivers it (K-major boxes of 64 columns), B = the queries
+//   O^T += V^T P^T  A = the same boxes read the other way (MN-major: rows = latent columns), B = the softmax weights.  They are
+//                   fp32 and enter as bf16 hi and lo halves side by side on N (16 mantissa bits); hi and lo sums meet at the end
 //
-// Key tiles come in by 16-byte cp.async through a ring of two or three stages (the chunk's block ids wait in shared memory); rows are padded to an odd number of 16-byte units, so ldmatrix is
-// free of bank conflicts.  Chunks are merged by a second kernel.
+// CTA = (context chunk, group of heads, sequence).  A tile is ceil((R + rot) / 128) units of two boxes; a ring of units runs
+// across tiles, and a unit is free again as soon as its 128 latent columns have been multiplied.  Warp roles (192 threads): warp
+// 0 = TMA producer, warp 1 = TMEM owner + UMMA issuer, warps 2..5 = softmax: scores go through shared memory to change from
+// one key per thread to a share of one head's keys per thread.  O is rescaled only when a head's maximum has grown by 2^8.
+// All waits are bounded (ptx.cuh).  Chunks are merged by a second kernel.
 #include "../include/launch.cuh"
-#include "../include/mma_sync.cuh"
 #include "../include/scalar.cuh"
 
 namespace forge {
 
-constexpr int kLdThreads = 256, kLdMaxSteps = 9, kLdMaxPairs = 4, kLdMaxChunk = 1024, kLdMaxBlocks = kLdMaxChunk / 16 + 1;
+constexpr int kLdKeys = 128, kLdThreads = 192, kLdBox = kLdKeys * 128, kLdUnit = 2 * kLdBox, kLdMaxD = 576;
 
 struct LatentDecodeArgs {
-  const bf16* qa;            // [seqs][heads][D]
-  const bf16* cache;
   const int* block_tables;   // [seqs][table_width]
   const int* lens;           // [seqs] keys visible, the token's own included
   bf16* o;                   // [seqs][heads][R]
@@ -33,229 +32,279 @@ struct LatentDecodeArgs {
   unsigned* status;
 };
 
-__host__ __device__ inline int latent_pitch(int D) { return (D / 8 | 1) * 8; }     // elements; odd number of 16-byte units
+template <int N>
+struct LatentDecodeCfg {
+  static constexpr int kSlots = N == 16 ? 6 : 5;
+  static constexpr int kTPitch = kLdKeys + 4;                        // floats per head of the transposed scores
+  static constexpr int kQBytes = (kLdMaxD / 64) * N * 128;
+  static constexpr int kTBytes = (N * kTPitch * 4 + 1023) / 1024 * 1024;      // also holds the weights: 2 boxes of 2N rows x 128 bytes
+  static constexpr int kSmem = kSlots * kLdUnit + kQBytes + kTBytes + 512 + 1024;
+  static_assert(kTBytes >= 2 * 2 * N * 128 && kSmem <= 227 * 1024, "shared memory");
+};
 
-template <int kTile, int kMT, int kStages>
-__global__ void __launch_bounds__(kLdThreads, kTile == 32 && kMT == 1 ? 2 : 1) latent_decode_kernel(const LatentDecodeArgs p) {
-  constexpr int kLdHeads = 16 * kMT, kRowThreads = kLdThreads / kLdHeads, kRowKeys = kTile / kRowThreads;
-  constexpr int kSPitch = kTile + 4, kPPitch = kTile + 8;
-  extern __shared__ __align__(16) uint8_t smem_raw[];
-  const int pitch = latent_pitch(p.D);
-  bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                        // [heads][pitch]
-  bf16* sKV = sQ + kLdHeads * pitch;                                   // [kStages][kTile][pitch]
-  float* sS = reinterpret_cast<float*>(sKV + kStages * kTile * pitch); // [4][heads][kTile + 4]
-  bf16* sP = reinterpret_cast<bf16*>(sS + 4 * kLdHeads * kSPitch);     // [hi, lo][heads][kTile + 8]
-  float* sAlpha = reinterpret_cast<float*>(sP + 2 * kLdHeads * kPPitch);       // [heads]
-  int* sBlk = reinterpret_cast<int*>(sAlpha + kLdHeads);               // [kLdMaxBlocks]
+// MN-major operand with the 128-byte swizzle: rows of 64 MN elements, 8 K rows 1024 bytes apart, the next 64 MN elements one box on.
+__device__ __forceinline__ uint64_t latent_v_desc(uint32_t smem_addr) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((smem_addr & 0x3FFFFu) >> 4);
+  d |= static_cast<uint64_t>((kLdBox >> 4) & 0x3FFF) << 16;
+  d |= static_cast<uint64_t>(1024 >> 4) << 32;
+  d |= static_cast<uint64_t>(1) << 46;
+  d |= static_cast<uint64_t>(2) << 61;
+  return d;
+}
+
+// tm_q: [seqs * heads, D], box N x 64; tm_kv: [blocks * block_size, D], box min(128, block_size) x 64.
+template <int N>
+__global__ void __launch_bounds__(kLdThreads, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const LatentDecodeArgs p) {
+  using Cfg = LatentDecodeCfg<N>;
+  constexpr int kHeadThreads = 128 / N, kHeadKeys = kLdKeys / kHeadThreads;   // 8 x 16 or 4 x 32
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* ring = smem;
+  uint8_t* sQ = ring + Cfg::kSlots * kLdUnit;
+  uint8_t* sTP = sQ + Cfg::kQBytes;                     // scores [N][kTPitch] fp32, then weights
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sTP + Cfg::kTBytes);
+  uint64_t* full = bars;                                // [kSlots]
+  uint64_t* empty = full + Cfg::kSlots;                 // [kSlots]
+  uint64_t* q_full = empty + Cfg::kSlots;
+  uint64_t* s_full = q_full + 1;
+  uint64_t* p_full = q_full + 2;                        // one arrival per softmax warp
+  uint64_t* o_full = q_full + 3;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 4);
+  int* s_grow = reinterpret_cast<int*>(tmem_slot + 1);  // [2]: some head's maximum has grown (by tile parity)
+  float* s_scale = reinterpret_cast<float*>(s_grow + 3);       // [N]
 
   pdl_launch_dependents();
   pdl_wait();
-  const int ch = blockIdx.x, h0 = blockIdx.y * kLdHeads, seq = blockIdx.z;
+  const int ch = blockIdx.x, h0 = blockIdx.y * N, seq = blockIdx.z;
   const int len = min(p.lens[seq], p.table_width << p.block_shift);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int k_begin = ch * p.chunk, k_end = min(len, k_begin + p.chunk);
-  const int row = threadIdx.x / kRowThreads, sub = threadIdx.x % kRowThreads;   // softmax: head row, lane within its threads
-  if (k_begin >= k_end) {
-    if (p.max_chunks == 1)                                             // padding of a graph bucket: defined values
-      for (int i = threadIdx.x; i < kLdHeads * p.R; i += kLdThreads)
+  if (k_begin >= k_end) {                               // uniform, before anything is allocated
+    if (p.max_chunks == 1)                              // padding of a graph bucket: defined values
+      for (int i = threadIdx.x; i < N * p.R; i += kLdThreads)
         if (h0 + i / p.R < p.heads) p.o[(static_cast<size_t>(seq) * p.heads + h0) * p.R + i] = __float2bfloat16_rn(0.f);
     return;
   }
-  const int units = p.D >> 3;                                          // 16-byte units per row
-  const int* table = p.block_tables + static_cast<size_t>(seq) * p.table_width;
-  const int blk0 = k_begin >> p.block_shift, n_blk = ((k_end - 1) >> p.block_shift) - blk0 + 1;
-  for (int i = threadIdx.x; i < n_blk; i += kLdThreads) {
-    int blk = table[blk0 + i];
-    if (blk < 0 || blk >= p.num_blocks) {
-      set_status(p.status, kStatusBadIndex);
-      blk = -1;
-    }
-    sBlk[i] = blk;
-  }
-  auto load_tile = [&](int t) {
-    bf16* dst = sKV + (t % kStages) * kTile * pitch;
-#pragma unroll
-    for (int i = 0; i < kTile / 8; ++i) {
-      const int r = warp + 8 * i, key = k_begin + t * kTile + r;
-      const int blk = key < k_end ? sBlk[(key >> p.block_shift) - blk0] : -1;
-      const uint32_t bytes = blk >= 0 ? 16 : 0;
-      const bf16* src = p.cache + (blk >= 0 ? ((static_cast<size_t>(blk) << p.block_shift) + (key & ((1 << p.block_shift) - 1))) * p.D : 0);
-      const uint32_t to = smem_u32(dst + r * pitch);
-      for (int u = lane; u < units; u += 32) cp_async16(to + u * 16, src + u * 8, bytes);
-    }
-  };
-  for (int r = warp; r < kLdHeads; r += kLdThreads / 32) {
-    const bool in = h0 + r < p.heads;
-    const bf16* src = p.qa + (static_cast<size_t>(seq) * p.heads + (in ? h0 + r : 0)) * p.D;
-    for (int u = lane; u < units; u += 32) cp_async16(smem_u32(sQ + r * pitch + u * 8), src + u * 8, in ? 16 : 0);
-  }
-  __syncthreads();                                                     // block ids
-#pragma unroll
-  for (int t = 0; t < kStages - 1; ++t) {
-    if (k_begin + t * kTile < k_end) load_tile(t);
-    cp_async_commit();
-  }
+  const int n_tiles = (k_end - k_begin + kLdKeys - 1) / kLdKeys;
+  const int boxes = (p.D + 63) >> 6, units = (boxes + 1) >> 1, m_tiles = (p.R + 127) >> 7;
 
-  const int slice = warp & 3, half = warp >> 2;
-  const int steps = p.D >> 4;
-  const int ks0 = slice * steps / 4, ksn = (slice + 1) * steps / 4 - ks0;
-  uint32_t qf[kMT][kLdMaxSteps][4];
-  float acc[kMT][kLdMaxPairs][2][4];
-#pragma unroll
-  for (int m = 0; m < kMT; ++m)
-#pragma unroll
-    for (int i = 0; i < kLdMaxPairs; ++i)
-#pragma unroll
-      for (int j = 0; j < 2; ++j) acc[m][i][j][0] = acc[m][i][j][1] = acc[m][i][j][2] = acc[m][i][j][3] = 0.f;
-  float m_run = -INFINITY, l_run = 0.f;
-  const int pairs = p.R >> 4;
-  const int n_tiles = (k_end - k_begin + kTile - 1) / kTile;
-
-  for (int t = 0; t < n_tiles; ++t) {
-    cp_async_wait<kStages - 2>();
-    __syncthreads();                       // tile t is here; everyone is done with tile t - 1, its stage may be filled again
-    if (t + kStages - 1 < n_tiles) load_tile(t + kStages - 1);
-    cp_async_commit();
-    const uint32_t kv = smem_u32(sKV + (t % kStages) * kTile * pitch);
-    if (t == 0) {
-#pragma unroll
-      for (int m = 0; m < kMT; ++m)
-#pragma unroll
-        for (int i = 0; i < kLdMaxSteps; ++i)
-          if (i < ksn) ldsm_x4(smem_u32(sQ) + ((m * 16 + (lane & 15)) * pitch + (ks0 + i) * 16 + (lane >> 4) * 8) * 2, qf[m][i]);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp == 0 && lane == 0) {
+    prefetch_tensormap(&tm_q);
+    prefetch_tensormap(&tm_kv);
+    for (int s = 0; s < Cfg::kSlots; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 1);
     }
-    {
-      constexpr int kNB = kTile / 16;                                  // 8-key blocks per warp
-      float s[kMT][kNB][4];
+    mbar_init(q_full, 1);
+    mbar_init(s_full, 1);
+    mbar_init(p_full, 4);
+    mbar_init(o_full, 1);
+    s_grow[0] = s_grow[1] = 0;
+    fence_mbar_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, 512);                         // S (N columns) | O: m_tiles x (hi N, lo N) from column 32
+    tmem_relinquish();
+  }
+  tcgen05_fence_before();
+  __syncthreads();
+  tcgen05_fence_after();
+  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 32;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      mbar_expect_tx(q_full, boxes * N * 128);
+      for (int b = 0; b < boxes; ++b) tma_load_2d(sQ + b * N * 128, &tm_q, q_full, b * 64, seq * p.heads + h0);
+      const int* table = p.block_tables + static_cast<size_t>(seq) * p.table_width;
+      const int box_rows = min(kLdKeys, 1 << p.block_shift);
+      int g = 0;
+      bool ok = true;
+      for (int t = 0; t < n_tiles && ok; ++t) {
+        int rows[8];                                    // cache row of every box_rows keys of the tile
 #pragma unroll
-      for (int m = 0; m < kMT; ++m)
-#pragma unroll
-        for (int nb = 0; nb < kNB; ++nb) s[m][nb][0] = s[m][nb][1] = s[m][nb][2] = s[m][nb][3] = 0.f;
-#pragma unroll
-      for (int i = 0; i < kLdMaxSteps; ++i) {
-        if (i < ksn) {
-#pragma unroll
-          for (int nb = 0; nb < kNB; nb += 2) {
-            uint32_t b[4];
-            const int r = half * (kTile / 2) + nb * 8 + (lane & 7) + (lane >> 4) * 8;
-            ldsm_x4(kv + (r * pitch + (ks0 + i) * 16 + ((lane >> 3) & 1) * 8) * 2, b);
-#pragma unroll
-            for (int m = 0; m < kMT; ++m) {
-              mma16816(s[m][nb], qf[m][i], b[0], b[1]);
-              mma16816(s[m][nb + 1], qf[m][i], b[2], b[3]);
+        for (int i = 0; i < 8; ++i) {
+          rows[i] = 0;
+          const int key = k_begin + t * kLdKeys + i * box_rows;
+          if (i * box_rows < kLdKeys && key < k_end) {  // past the end: any rows will do, their weights are zero
+            int blk = table[key >> p.block_shift];
+            if (blk < 0 || blk >= p.num_blocks) {
+              set_status(p.status, kStatusBadIndex);
+              blk = 0;
             }
+            rows[i] = (blk << p.block_shift) + (key & ((1 << p.block_shift) - 1));
           }
         }
-      }
-      float* dst = sS + slice * kLdHeads * kSPitch + half * (kTile / 2) + 2 * (lane & 3);
+        for (int u = 0; u < units && ok; ++u, ++g) {
+          const int s = g % Cfg::kSlots;
+          if (!mbar_wait_parked(&empty[s], ((g / Cfg::kSlots) & 1) ^ 1, p.status)) { ok = false; break; }
+          const int nb = min(2, boxes - 2 * u);
+          mbar_expect_tx(&full[s], nb * kLdBox);
+          for (int b = 0; b < nb; ++b)
 #pragma unroll
-      for (int m = 0; m < kMT; ++m)
-#pragma unroll
-        for (int nb = 0; nb < kNB; ++nb) {
-          *reinterpret_cast<float2*>(dst + (m * 16 + (lane >> 2)) * kSPitch + nb * 8) = make_float2(s[m][nb][0], s[m][nb][1]);
-          *reinterpret_cast<float2*>(dst + (m * 16 + (lane >> 2) + 8) * kSPitch + nb * 8) = make_float2(s[m][nb][2], s[m][nb][3]);
+            for (int i = 0; i < 8; ++i)
+              if (i * box_rows < kLdKeys)
+                tma_load_2d(ring + s * kLdUnit + b * kLdBox + i * box_rows * 128, &tm_kv, &full[s], (2 * u + b) * 64, rows[i]);
         }
+      }
     }
-    __syncthreads();
-    {
-      float s[kRowKeys], mx = -INFINITY;
-      const int left = k_end - k_begin - t * kTile;
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = umma_idesc(kLdKeys, N, 1, 1);
+      constexpr uint32_t idesc_o = umma_idesc(128, 2 * N, 1, 1) | (1u << 15);         // A (= V^T) MN-major
+      const uint32_t ring_addr = smem_u32(ring), q_addr = smem_u32(sQ), p_addr = smem_u32(sTP);
+      const int steps = (p.D + 15) >> 4;
+      bool ok = mbar_wait(q_full, 0, p.status);
+      for (int t = 0; t < n_tiles && ok; ++t) {
+        const int g0 = t * units;
+        for (int u = 0; u < units; ++u) {
+          const int s = (g0 + u) % Cfg::kSlots;
+          if (!mbar_wait_parked(&full[s], ((g0 + u) / Cfg::kSlots) & 1, p.status)) { ok = false; break; }
+          tcgen05_fence_after();
+          for (int k = u * 8; k < min(steps, u * 8 + 8); ++k) {
+            const int box = k >> 2, sub = (k & 3) * 32;
+            umma_f16(tmem_s, umma_desc_k_sw128(ring_addr + s * kLdUnit + (box & 1) * kLdBox + sub), umma_desc_k_sw128(q_addr + box * N * 128 + sub),
+                     idesc_s, k != 0);
+          }
+          if (u >= m_tiles) umma_commit(&empty[s]);     // no value columns in this unit
+        }
+        if (!ok) break;
+        umma_commit(s_full);
+        if (!mbar_wait_parked(p_full, t & 1, p.status)) break;
+        tcgen05_fence_after();
+        for (int m = 0; m < m_tiles; ++m) {
+          const int s = (g0 + m) % Cfg::kSlots;
 #pragma unroll
-      for (int i = 0; i < kRowKeys; ++i) {
-        const int key = sub + kRowThreads * i;
-        const float* src = sS + row * kSPitch + key;
-        s[i] = key < left ? (src[0] + src[kLdHeads * kSPitch] + src[2 * kLdHeads * kSPitch] + src[3 * kLdHeads * kSPitch]) * p.scale_log2 : -INFINITY;
-        mx = fmaxf(mx, s[i]);
+          for (int k = 0; k < kLdKeys / 16; ++k)
+            umma_f16(tmem_o + m * 2 * N, latent_v_desc(ring_addr + s * kLdUnit + k * 16 * 128),
+                     umma_desc_k_sw128(p_addr + (k >> 2) * 2 * N * 128 + (k & 3) * 32), idesc_o, (t | k) != 0);
+          umma_commit(&empty[s]);
+        }
+      }
+      if (ok) umma_commit(o_full);
+    }
+  } else {
+    const int quad = warp & 3, key = quad * 32 + lane;   // TMEM lane = key of the tile
+    const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
+    const int tid = key, head = tid / kHeadThreads, sub = tid % kHeadThreads;
+    float* sT = reinterpret_cast<float*>(sTP);
+    float m_ref = 0.f, l_run = 0.f;
+    bool ok = true;
+    for (int t = 0; t < n_tiles; ++t) {
+      // S of tile t is complete, and with it every product issued before: the weights of tile t - 1 may be overwritten
+      ok = mbar_wait(s_full, t & 1, p.status);
+      tcgen05_fence_after();
+      {
+        uint32_t v[N];
+        if constexpr (N == 16) tmem_ld_x16(tmem_s + lane_addr, v);
+        else tmem_ld_x32(tmem_s + lane_addr, v);
+        tmem_ld_wait();
+        const bool in = k_begin + t * kLdKeys + key < k_end;
+#pragma unroll
+        for (int h = 0; h < N; ++h) sT[h * Cfg::kTPitch + key] = in ? __uint_as_float(v[h]) * p.scale_log2 : -INFINITY;
+      }
+      if (tid == 0) s_grow[(t + 1) & 1] = 0;
+      named_barrier_sync(1, 128);
+      float x[kHeadKeys], mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < kHeadKeys; i += 4) {           // keys 8 (sub + kHeadThreads j) .. + 7: whole 16-byte chunks of the weight rows
+        const int at = ((i >> 3) * kHeadThreads + sub) * 8 + (i & 7);
+        const float4 f = *reinterpret_cast<const float4*>(sT + head * Cfg::kTPitch + at);
+        x[i] = f.x;
+        x[i + 1] = f.y;
+        x[i + 2] = f.z;
+        x[i + 3] = f.w;
+        mx = fmaxf(mx, fmaxf(fmaxf(f.x, f.y), fmaxf(f.z, f.w)));
       }
 #pragma unroll
-      for (int off = kRowThreads / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      const float m_new = fmaxf(m_run, mx);                            // finite: a tile holds at least one visible key
-      const float alpha = exp2f(m_run - m_new);
-      m_run = m_new;
+      for (int off = kHeadThreads / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      float alpha = 1.f;                                 // mx is finite: a tile holds at least one visible key
+      if (t == 0) {
+        m_ref = mx;
+      } else if (mx - m_ref > 8.f) {
+        alpha = exp2f(m_ref - mx);
+        m_ref = mx;
+        s_grow[t & 1] = 1;
+      }
+      if (sub == 0) s_scale[head] = alpha;
       l_run *= alpha;
+      named_barrier_sync(1, 128);                        // scores are in registers, scales and the flag are set
+      if (t > 0 && s_grow[t & 1]) {
+#pragma unroll 1
+        for (int c = 0; c < m_tiles * 2 * N; c += 32) {
+          uint32_t o[32];
+          tmem_ld_x32(tmem_o + lane_addr + c, o);
+          tmem_ld_wait();
 #pragma unroll
-      for (int i = 0; i < kRowKeys; ++i) {
-        const float w = exp2f(s[i] - m_new);
-        l_run += w;
-        float hi, lo;
-        split_bf16(w, hi, lo);
-        sP[row * kPPitch + sub + kRowThreads * i] = __float2bfloat16_rn(hi);
-        sP[(kLdHeads + row) * kPPitch + sub + kRowThreads * i] = __float2bfloat16_rn(lo);
-      }
-      if (sub == 0) sAlpha[row] = alpha;
-    }
-    __syncthreads();
-#pragma unroll
-    for (int m = 0; m < kMT; ++m) {
-      const float a0 = sAlpha[m * 16 + (lane >> 2)], a1 = sAlpha[m * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int i = 0; i < kLdMaxPairs; ++i)
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          acc[m][i][j][0] *= a0;
-          acc[m][i][j][1] *= a0;
-          acc[m][i][j][2] *= a1;
-          acc[m][i][j][3] *= a1;
+          for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_scale[i % N]);
+          tmem_st_x32(tmem_o + lane_addr + c, o);
         }
-    }
-#pragma unroll
-    for (int ks = 0; ks < kTile / 16; ++ks) {
-      uint32_t ph[kMT][4], pl[kMT][4];
-#pragma unroll
-      for (int m = 0; m < kMT; ++m) {
-        const uint32_t at = smem_u32(sP) + ((m * 16 + (lane & 15)) * kPPitch + ks * 16 + (lane >> 4) * 8) * 2;
-        ldsm_x4(at, ph[m]);
-        ldsm_x4(at + kLdHeads * kPPitch * 2, pl[m]);
+        tmem_st_wait();
       }
 #pragma unroll
-      for (int i = 0; i < kLdMaxPairs; ++i) {
-        const int pair = warp + i * 8;
-        if (pair < pairs) {
-          uint32_t b[4];
-          const int r = ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
-          ldsm_x4_trans(kv + (r * pitch + pair * 16 + (lane >> 4) * 8) * 2, b);
+      for (int i = 0; i < kHeadKeys; i += 8) {
+        uint32_t hi[4], lo[4];
 #pragma unroll
-          for (int m = 0; m < kMT; ++m) {
-            mma16816(acc[m][i][0], ph[m], b[0], b[1]);
-            mma16816(acc[m][i][1], ph[m], b[2], b[3]);
-            mma16816(acc[m][i][0], pl[m], b[0], b[1]);
-            mma16816(acc[m][i][1], pl[m], b[2], b[3]);
-          }
+        for (int e = 0; e < 4; ++e) {
+          const float p0 = ex2_approx(x[i + 2 * e] - m_ref), p1 = ex2_approx(x[i + 2 * e + 1] - m_ref);
+          l_run += p0 + p1;
+          hi[e] = pack_bf16x2(p0, p1);
+          lo[e] = pack_bf16x2(p0 - bf16_lo(hi[e]), p1 - bf16_hi(hi[e]));
         }
+        const int c = (i >> 3) * kHeadThreads + sub;     // 16-byte chunk of the 128 keys: box c / 8, chunk c % 8
+        uint8_t* row = sTP + (c >> 3) * 2 * N * 128 + head * 128 + (((c & 7) ^ (head & 7)) << 4);
+        *reinterpret_cast<uint4*>(row) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(row + N * 128) = make_uint4(lo[0], lo[1], lo[2], lo[3]);    // N is a multiple of 8: same swizzle phase
+      }
+      fence_proxy_async_smem();
+      tcgen05_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_full);
+    }
+#pragma unroll
+    for (int off = kHeadThreads / 2; off > 0; off >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
+    if (sub == 0) {
+      s_scale[head] = p.max_chunks == 1 ? 1.f / l_run : 1.f;
+      if (p.max_chunks > 1 && h0 + head < p.heads) {
+        float* ml = p.part_ml + ((static_cast<size_t>(seq) * p.heads + h0 + head) * p.max_chunks + ch) * 2;
+        ml[0] = m_ref;
+        ml[1] = l_run;
+      }
+    }
+    if (ok) ok = mbar_wait(o_full, 0, p.status);
+    named_barrier_sync(1, 128);
+    tcgen05_fence_after();
+    for (int m = 0; m < m_tiles; ++m) {
+      __syncwarp();
+      uint32_t hi[N], lo[N];
+      if constexpr (N == 16) {
+        tmem_ld_x16(tmem_o + lane_addr + m * 2 * N, hi);
+        tmem_ld_x16(tmem_o + lane_addr + m * 2 * N + N, lo);
+      } else {
+        tmem_ld_x32(tmem_o + lane_addr + m * 2 * N, hi);
+        tmem_ld_x32(tmem_o + lane_addr + m * 2 * N + N, lo);
+      }
+      tmem_ld_wait();
+      const int d = m * 128 + key;
+      if (d >= p.R) continue;
+#pragma unroll
+      for (int h = 0; h < N; ++h) {
+        if (h0 + h >= p.heads) continue;
+        const float v = __uint_as_float(hi[h]) + __uint_as_float(lo[h]);
+        const size_t hr = static_cast<size_t>(seq) * p.heads + h0 + h;
+        if (p.max_chunks == 1) p.o[hr * p.R + d] = __float2bfloat16_rn(v * s_scale[h]);
+        else p.part_o[(hr * p.max_chunks + ch) * p.R + d] = v;
       }
     }
   }
-#pragma unroll
-  for (int off = kRowThreads / 2; off > 0; off >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
-  if (p.max_chunks == 1) {
-    __syncthreads();
-    if (sub == 0) sAlpha[row] = 1.f / l_run;
-    __syncthreads();
-  } else if (sub == 0 && h0 + row < p.heads) {
-    float* ml = p.part_ml + ((static_cast<size_t>(seq) * p.heads + h0 + row) * p.max_chunks + ch) * 2;
-    ml[0] = m_run;
-    ml[1] = l_run;
+
+  tcgen05_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tcgen05_fence_after();
+    tmem_dealloc(tmem_s, 512);
   }
-#pragma unroll
-  for (int m = 0; m < kMT; ++m)
-#pragma unroll
-    for (int i = 0; i < kLdMaxPairs; ++i) {
-      const int pair = warp + i * 8;
-      if (pair >= pairs) continue;
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int r = m * 16 + (lane >> 2) + e * 8, c = pair * 16 + j * 8 + 2 * (lane & 3);
-          if (h0 + r >= p.heads) continue;
-          const float v0 = acc[m][i][j][2 * e], v1 = acc[m][i][j][2 * e + 1];
-          const size_t hr = static_cast<size_t>(seq) * p.heads + h0 + r;
-          if (p.max_chunks == 1)
-            *reinterpret_cast<uint32_t*>(p.o + hr * p.R + c) = pack_bf16x2(v0 * sAlpha[r], v1 * sAlpha[r]);
-          else
-            *reinterpret_cast<float2*>(p.part_o + (hr * p.max_chunks + ch) * p.R + c) = make_float2(v0, v1);
-        }
-    }
 }
 
 // One CTA per (head, sequence): the chunks' partial sums, weighted by their maxima.
@@ -288,39 +337,41 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
   }
 }
 
-template <int kTile, int kMT, int kStages>
-static int launch_latent_decode(const LatentDecodeArgs& p, int seqs, cudaStream_t stream) {
-  constexpr int kHeads = 16 * kMT;
-  auto smem = [](int D) {
-    return static_cast<int>((kHeads + kStages * kTile) * latent_pitch(D) * 2 + 4 * kHeads * (kTile + 4) * 4 + 2 * kHeads * (kTile + 8) * 2 +
-                            kHeads * 4 + kLdMaxBlocks * 4);
-  };
-  auto kern = latent_decode_kernel<kTile, kMT, kStages>;
-  FORGE_ENSURE_DYN_SMEM(kern, smem(64 * kLdMaxSteps));
-  return launch_kernel(kern, dim3(p.max_chunks, (p.heads + kHeads - 1) / kHeads, seqs), dim3(kLdThreads), smem(p.D), stream, 0, p) == cudaSuccess ? 0 : -2;
-}
+extern "C" int forge_make_tmap_2d(CUtensorMap* tm, const void* base, uint64_t rows, uint64_t cols, uint64_t ld,
+                                  uint32_t box_rows, int elem_bytes);
 
 // 1 if the kernel takes these sizes (else: latent_attend_any).
 extern "C" int forge_latent_decode_ok(int R, int rot, int block_size) {
-  return R % 16 == 0 && rot % 16 == 0 && R >= 16 && R <= 16 * 8 * kLdMaxPairs && R + rot <= 64 * kLdMaxSteps && block_size >= 16 && (block_size & (block_size - 1)) == 0;
+  return R >= 8 && R <= 512 && R % 8 == 0 && rot % 8 == 0 && R + rot <= kLdMaxD && block_size >= 16 && (block_size & (block_size - 1)) == 0;
 }
 
-// qa [seqs][heads][R + rot] bf16; lens = keys visible per sequence; part_* needed when max_chunks > 1.
+template <int N>
+static int launch_latent_decode(const CUtensorMap& tm_q, const CUtensorMap& tm_kv, const LatentDecodeArgs& p, int seqs, cudaStream_t stream) {
+  auto kern = latent_decode_kernel<N>;
+  FORGE_ENSURE_DYN_SMEM(kern, LatentDecodeCfg<N>::kSmem);
+  return launch_kernel(kern, dim3(p.max_chunks, (p.heads + N - 1) / N, seqs), dim3(kLdThreads), LatentDecodeCfg<N>::kSmem, stream, 0, tm_q, tm_kv,
+                       p) == cudaSuccess ? 0 : -2;
+}
+
+// qa [seqs][heads][R + rot] bf16; lens = keys visible per sequence; chunk a multiple of 128; part_* needed when max_chunks > 1.
 extern "C" int forge_latent_decode(const void* qa, const void* cache, const int* block_tables, const int* lens, void* o, float* part_o,
                                    float* part_ml, int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size,
-                                   int chunk, int max_chunks, int tile, float scale, unsigned* status, cudaStream_t stream) {
+                                   int chunk, int max_chunks, float scale, unsigned* status, cudaStream_t stream) {
   if (seqs <= 0) return 0;
-  if (!forge_latent_decode_ok(R, rot, block_size) || chunk < 64 || chunk % 64 || chunk > kLdMaxChunk || (tile != 32 && tile != 64) || seqs > 65535 ||
-      (reinterpret_cast<uintptr_t>(qa) & 15) || (reinterpret_cast<uintptr_t>(cache) & 15))
+  if (!forge_latent_decode_ok(R, rot, block_size) || chunk < kLdKeys || chunk % kLdKeys || seqs > 65535 ||
+      (reinterpret_cast<uintptr_t>(qa) & 15) || (reinterpret_cast<uintptr_t>(cache) & 15) ||
+      static_cast<long long>(num_blocks) * block_size >= (1ll << 31))
     return -1;
   int shift = 0;
   while ((1 << shift) < block_size) ++shift;
-  const LatentDecodeArgs p = {static_cast<const bf16*>(qa), static_cast<const bf16*>(cache), block_tables, lens, static_cast<bf16*>(o), part_o,
-                              part_ml, table_width, num_blocks, shift, heads, R, R + rot, chunk, max_chunks, scale * 1.4426950408889634f, status};
-  const int rc = heads > 16 ? launch_latent_decode<32, 2, 3>(p, seqs, stream)
-                 : tile == 32 ? launch_latent_decode<32, 1, 2>(p, seqs, stream) : launch_latent_decode<64, 1, 2>(p, seqs, stream);
-  if (rc != 0) return rc;
-  if (max_chunks == 1) return 0;
+  const int D = R + rot, n = heads > 16 ? 32 : 16;
+  const LatentDecodeArgs p = {block_tables, lens, static_cast<bf16*>(o), part_o, part_ml, table_width, num_blocks, shift, heads, R, D, chunk,
+                              max_chunks, scale * 1.4426950408889634f, status};
+  CUtensorMap tm_q, tm_kv;
+  if (forge_make_tmap_2d(&tm_q, qa, static_cast<uint64_t>(seqs) * heads, D, D, n, 2) != 0) return -2;
+  if (forge_make_tmap_2d(&tm_kv, cache, static_cast<uint64_t>(num_blocks) * block_size, D, D, block_size < kLdKeys ? block_size : kLdKeys, 2) != 0) return -2;
+  const int rc = n == 32 ? launch_latent_decode<32>(tm_q, tm_kv, p, seqs, stream) : launch_latent_decode<16>(tm_q, tm_kv, p, seqs, stream);
+  if (rc != 0 || max_chunks == 1) return rc;
   return launch_kernel(latent_merge_kernel, dim3(heads, seqs), dim3(128), 0, stream, 0, part_o, part_ml, lens, static_cast<bf16*>(o), heads, R,
                        chunk, max_chunks, table_width * block_size) == cudaSuccess ? 0 : -2;
 }

@@ -40,7 +40,7 @@ int forge_head_linear(const void* x, long long x_tok, long long x_head, const vo
 int forge_latent_decode_ok(int R, int rot, int block_size);
 int forge_latent_decode(const void* qa, const void* cache, const int* block_tables, const int* lens, void* o, float* part_o, float* part_ml,
                         int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size, int chunk, int max_chunks,
-                        int tile, float scale, unsigned* status, cudaStream_t stream);
+                        float scale, unsigned* status, cudaStream_t stream);
 int forge_latent_prefill_qcols(int dim, int rot, int vdim);
 int forge_latent_prefill(const void* q, const void* kv, const void* kr, const int* cu_q, const int* cu_k, void* out, int tokens, int tok0,
                          int keys, int num_seqs, int max_q, int heads, int dim, int rot, int vdim, float scale, unsigned* status,
@@ -321,7 +321,7 @@ void head_linear(const Tensor& x, const Tensor& w, Tensor& out) {
 }
 
 void latent_decode(const Tensor& qa, const Tensor& cache, const Tensor& block_tables, const Tensor& lens, Tensor& o, const OptTensor& part_o,
-                   const OptTensor& part_ml, int64_t chunk, int64_t max_chunks, int64_t tile, double scale, const Tensor& status) {
+                   const OptTensor& part_ml, int64_t chunk, int64_t max_chunks, double scale, const Tensor& status) {
   TORCH_CHECK(qa.dim() == 3 && cache.dim() == 3 && block_tables.dim() == 2 && o.dim() == 3, "latent_decode: ranks");
   const int64_t B = qa.size(0), H = qa.size(1), D = qa.size(2), R = o.size(2);
   TORCH_CHECK(cache.size(2) == D && R <= D && o.size(0) == B && o.size(1) == H && block_tables.size(0) >= B && max_chunks >= 1, "latent_decode: shapes");
@@ -334,7 +334,7 @@ void latent_decode(const Tensor& qa, const Tensor& cache, const Tensor& block_ta
   const c10::cuda::CUDAGuard guard(qa.device());
   check_rc(forge_latent_decode(data(qa, kBf16, 0, "qa"), data(cache, kBf16, 0, "cache"), ints(block_tables, 0, "block_tables"), ints(lens, B, "lens"),
                                data(o, kBf16, 0, "o"), po, pml, i32(B), i32(H), i32(R), i32(D - R), i32(block_tables.size(1)), i32(cache.size(0)),
-                               i32(cache.size(1)), i32(chunk), i32(max_chunks), i32(tile), static_cast<float>(scale), status_word(status),
+                               i32(cache.size(1)), i32(chunk), i32(max_chunks), static_cast<float>(scale), status_word(status),
                                stream_of(qa)),
            "forge_latent_decode");
 }

@@ -113,7 +113,7 @@ def test_head_linear(ops, M, H, N, K):
 
 
 # ------------------------------------------------------------------------------------------------ latent attention
-def latent_setup(ops, ranges, block, dtype, s, seed=0, decode=False, pad=0, needle=None):
+def latent_setup(ops, ranges, block, dtype, s, seed=0, decode=False, pad=0, needle=None, grow=False):
     """Random latents for whole sequences in the cache, queries for the ranges; what the oracle's softmax attention gives.
     ``needle(position) -> key``: the query of that position points at that key (unrotated and rotated part alike)."""
     b = Batch(ranges, block, decode=decode, pad=pad, seed=seed)
@@ -124,6 +124,8 @@ def latent_setup(ops, ranges, block, dtype, s, seed=0, decode=False, pad=0, need
     q_all, outs = [], []
     for i, (lo, hi) in enumerate(ranges):
         c = rnd(hi, R, seed=100 * seed + i + 5, dtype=dtype)
+        if grow:                                                # the same direction, longer and longer
+            c = (c[:1].double() * torch.linspace(0.1, 6, hi, dtype=torch.float64)[:, None]).to(dtype)
         k_pre = rnd(hi, 1, r, seed=100 * seed + i + 6)
         kr = rotated(k_pre.double(), 10000.0, r)[:, 0].to(dtype)
         rows = torch.cat([c, kr], 1)
@@ -136,6 +138,9 @@ def latent_setup(ops, ranges, block, dtype, s, seed=0, decode=False, pad=0, need
             for n in range(hi - lo):
                 j = needle(lo + n)
                 q[n] = torch.cat([k_un[j] * 3, rotated(kr[j].double().view(1, 1, r).expand(1, H, r), 10000.0, r, -(lo + n))[0] * 3], -1)
+        if grow:
+            q[:, :, :s.dim] = k_un[-1] / k_un[-1].norm(dim=-1, keepdim=True) * 6
+            q[:, :, s.dim:] *= 0.1
         q = q.to(dtype)
         qr = rotated(q[:, :, s.dim:].double(), 10000.0, r, lo)
         k = torch.cat([k_un, kr.double()[:, None].expand(hi, H, r)], -1)
@@ -183,19 +188,30 @@ def test_latent_prompts(ops, name, dtype):
     close(got, want, 1e-5 if dtype == F32 else 1.5e-2)
 
 
-@pytest.mark.parametrize("tile", [32, 64])
-@pytest.mark.parametrize("name", ["real", "groups", "small", "odd"])
-def test_latent_decode(ops, name, tile):
-    lens = (1, 2, 63, 64, 65, 128, 129, 1000, 257, 700)
-    old = ops.latent_tile
-    ops.latent_tile = tile
-    try:
-        got, want = latent_setup(ops, [(n - 1, n) for n in lens], 64, BF, LATENT[name], seed=2, decode=True, pad=3)
-        close(got, want, 1.5e-2)
-        got, want = latent_setup(ops, [(n - 1, n) for n in (2500, 3, 2049)], 256, BF, LATENT[name], seed=3, decode=True)
-        close(got, want, 1.5e-2)
-    finally:
-        ops.latent_tile = old
+@pytest.mark.parametrize("block", [16, 64, 256])
+@pytest.mark.parametrize("name", list(LATENT))
+def test_latent_decode(ops, name, block):
+    lens = (1, 2, 63, 64, 65, 127, 128, 129, 256, 1000, 257, 700)
+    got, want = latent_setup(ops, [(n - 1, n) for n in lens], block, BF, LATENT[name], seed=2, decode=True, pad=3)
+    close(got, want, 1.5e-2)
+    got, want = latent_setup(ops, [(n - 1, n) for n in (2500, 3, 2049)], block, BF, LATENT[name], seed=3, decode=True)
+    close(got, want, 1.5e-2)
+
+
+@pytest.mark.parametrize("heads", [1, 16, 17, 32, 33, 70])
+def test_latent_decode_head_groups(ops, heads):
+    s = Spec(**{**LATENT["groups"].__dict__, "heads": heads})
+    got, want = latent_setup(ops, [(n - 1, n) for n in (5, 300, 140)], 64, BF, s, seed=7, decode=True)
+    close(got, want, 1.5e-2)
+
+
+def test_latent_decode_rescales_growing_maxima(ops):
+    """Keys whose scores grow along the context: the accumulators are rescaled several times on the way, head by head."""
+    s = Spec(**{**LATENT["groups"].__dict__, "scale": 1.5})
+    got, want = latent_setup(ops, [(n - 1, n) for n in (1000, 600, 129)], 64, BF, s, seed=8, decode=True, needle=lambda p: p)
+    close(got, want, 2.5e-2)
+    got, want = latent_setup(ops, [(899, 900)], 64, BF, Spec(**{**s.__dict__, "scale": 0.5}), seed=9, decode=True, grow=True)
+    close(got, want, 2.5e-2)
 
 
 @pytest.mark.parametrize("name", ["real", "small", "odd"])

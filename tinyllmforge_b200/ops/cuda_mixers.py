@@ -18,8 +18,6 @@ class Routed:
 class MixerOps:
     """Mixed into ``CudaOps`` (uses its ``C``, ``status``, ``device`` and GEMM methods)."""
 
-    latent_tile = 32                # keys per tile of the decode kernel (32: two CTAs per SM, 64: one)
-
     # ------------------------------------------------------------------ residual stream
     def stream_update(self, x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None):
         n = x.shape[0] if rows is None else rows.shape[0]
@@ -74,11 +72,10 @@ class MixerOps:
         return out
 
     def latent_chunking(self, seqs: int, heads: int, max_len: int) -> tuple[int, int]:
-        """(keys per chunk, chunks) of the decode kernel: enough chunks to fill the GPU once or
-        twice, from shapes known at capture time."""
-        ctas = seqs * (-(-heads // 32) if heads > 16 else 1)      # 16 heads per CTA and two CTAs per SM, or 32 and one
-        want = -(-self.num_sms * (1 if heads > 16 else 2) // ctas)
-        chunk = 64
+        """(keys per chunk, chunks) of the decode kernel: enough chunks to fill the GPU, from
+        shapes known at capture time."""
+        want = -(-self.num_sms // (seqs * -(-heads // 32)))       # one CTA per SM, up to 32 heads each
+        chunk = 128
         while chunk < 1024 and -(-max_len // (2 * chunk)) >= want:
             chunk *= 2
         return chunk, max(1, -(-max_len // chunk))
@@ -100,7 +97,7 @@ class MixerOps:
             if chunks > 1:
                 part_o = torch.empty(n * H * chunks * R, dtype=torch.float32, device=q.device)
                 part_ml = torch.empty(n * H * chunks * 2, dtype=torch.float32, device=q.device)
-            self.C.latent_decode(qa, cache, batch.block_tables, batch.context_lens, o, part_o, part_ml, chunk, chunks, self.latent_tile,
+            self.C.latent_decode(qa, cache, batch.block_tables, batch.context_lens, o, part_o, part_ml, chunk, chunks,
                                  spec.scale, self.status)
         else:
             self.C.latent_attend_any(qa, cache, o, 0, batch.cu_seqlens_q, batch.padded_seqs, batch.positions, batch.block_tables,

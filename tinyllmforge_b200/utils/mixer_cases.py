@@ -42,7 +42,7 @@ def _latent_decode(ops, heads, B=64, ctx=2048):
     chunk, n = ops.latent_chunking(B, heads, ctx)
     po = torch.empty(B * heads * n * R, device="cuda")
     pml = torch.empty(B * heads * n * 2, device="cuda")
-    return (lambda: ops.C.latent_decode(qa, cache, bt, lens, o, po, pml, chunk, n, ops.latent_tile, LATENT.scale, ops.status),
+    return (lambda: ops.C.latent_decode(qa, cache, bt, lens, o, po, pml, chunk, n, LATENT.scale, ops.status),
             B * ctx * (R + r) * 2 + B * heads * (2 * R + r) * 2, 2 * B * heads * ctx * (2 * R + r))
 
 
