@@ -2,15 +2,18 @@
 // [blocks][block_size][R + rot].
 //
 // The queries come folded (W_k^T q | rotated part), so all heads of a token share one key row per cached token (its whole
-// latent row) and one value row (the first R entries of the SAME row): a tile of 128 keys is read from memory once and serves
+// latent row) and one value row (the first R entries of the SAME row): a tile of 64 keys is read from memory once and serves
 // both products for up to 32 heads.  The keys and latents are the UMMA's 128-row side, the heads ride the N side:
 //
-//   S^T = K Q^T     A = the key tile as TMA delivers it (K-major boxes of 64 columns), B = the queries
+//   S^T = K Q^T     A = the key tile as TMA delivers it (K-major boxes of 64 columns; rows 64 .. 127 are whatever follows in
+//                   shared memory, their scores are not read: the tensor pipe is far from busy), B = the queries
 //   O^T += V^T P^T  A = the same boxes read the other way (MN-major: rows = latent columns), B = the softmax weights.  They are
 //                   fp32 and enter as bf16 hi and lo halves side by side on N (16 mantissa bits); hi and lo sums meet at the end
 //
-// CTA = (context chunk, group of heads, sequence).  A tile is ceil((R + rot) / 128) units of two boxes; a ring of units runs
-// across tiles, and a unit is free again as soon as its 128 latent columns have been multiplied.  Warp roles (192 threads): warp
+// CTA = (context chunk, group of heads, sequence).  A tile is ceil((R + rot) / 128) units of two boxes; a ring of two tiles' units
+// keeps loads in flight, and a unit is free again as soon as its 128 latent columns have been multiplied.  The products of tile
+// t + 1's scores and of tile t's O alternate unit by unit: the softmax of tile t overlaps the first scores of tile t + 1, and
+// tile t gives its units back early.  Warp roles (192 threads): warp
 // 0 = TMA producer, warp 1 = TMEM owner + UMMA issuer, warps 2..5 = softmax: scores go through shared memory to change from
 // one key per thread to a share of one head's keys per thread.  O is rescaled only when a head's maximum has grown by 2^8.
 // All waits are bounded (ptx.cuh).  Chunks are merged by a second kernel.
@@ -19,7 +22,7 @@
 
 namespace forge {
 
-constexpr int kLdKeys = 128, kLdThreads = 192, kLdBox = kLdKeys * 128, kLdUnit = 2 * kLdBox, kLdMaxD = 576;
+constexpr int kLdKeys = 64, kLdThreads = 192, kLdBox = kLdKeys * 128, kLdUnit = 2 * kLdBox, kLdMaxD = 576;
 
 struct LatentDecodeArgs {
   const int* block_tables;   // [seqs][table_width]
@@ -34,12 +37,12 @@ struct LatentDecodeArgs {
 
 template <int N>
 struct LatentDecodeCfg {
-  static constexpr int kSlots = N == 16 ? 6 : 5;
+  static constexpr int kSlots = N == 16 ? 12 : 11;
   static constexpr int kTPitch = kLdKeys + 4;                        // floats per head of the transposed scores
   static constexpr int kQBytes = (kLdMaxD / 64) * N * 128;
-  static constexpr int kTBytes = (N * kTPitch * 4 + 1023) / 1024 * 1024;      // also holds the weights: 2 boxes of 2N rows x 128 bytes
+  static constexpr int kTBytes = (N * kTPitch * 4 + 1023) / 1024 * 1024;      // also holds the weights: 2N rows x 128 bytes
   static constexpr int kSmem = kSlots * kLdUnit + kQBytes + kTBytes + 512 + 1024;
-  static_assert(kTBytes >= 2 * 2 * N * 128 && kSmem <= 227 * 1024, "shared memory");
+  static_assert(kTBytes >= 2 * N * 128 && kSlots >= 2 * ((kLdMaxD + 127) / 128) && kSmem <= 227 * 1024, "shared memory");
 };
 
 // MN-major operand with the 128-byte swizzle: rows of 64 MN elements, 8 K rows 1024 bytes apart, the next 64 MN elements one box on.
@@ -53,12 +56,12 @@ __device__ __forceinline__ uint64_t latent_v_desc(uint32_t smem_addr) {
   return d;
 }
 
-// tm_q: [seqs * heads, D], box N x 64; tm_kv: [blocks * block_size, D], box min(128, block_size) x 64.
+// tm_q: [seqs * heads, D], box N x 64; tm_kv: [blocks * block_size, D], box min(64, block_size) x 64.
 template <int N>
 __global__ void __launch_bounds__(kLdThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const LatentDecodeArgs p) {
   using Cfg = LatentDecodeCfg<N>;
-  constexpr int kHeadThreads = 128 / N, kHeadKeys = kLdKeys / kHeadThreads;   // 8 x 16 or 4 x 32
+  constexpr int kHeadThreads = 128 / N, kHeadKeys = kLdKeys / kHeadThreads;   // 8 x 8 or 4 x 16
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* ring = smem;
@@ -68,10 +71,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   uint64_t* full = bars;                                // [kSlots]
   uint64_t* empty = full + Cfg::kSlots;                 // [kSlots]
   uint64_t* q_full = empty + Cfg::kSlots;
-  uint64_t* s_full = q_full + 1;
-  uint64_t* p_full = q_full + 2;                        // one arrival per softmax warp
-  uint64_t* o_full = q_full + 3;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 4);
+  uint64_t* s_full = q_full + 1;                        // [2]
+  uint64_t* p_full = q_full + 3;                        // one arrival per softmax warp
+  uint64_t* o_full = q_full + 4;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 5);
   int* s_grow = reinterpret_cast<int*>(tmem_slot + 1);  // [2]: some head's maximum has grown (by tile parity)
   float* s_scale = reinterpret_cast<float*>(s_grow + 3);       // [N]
 
@@ -98,20 +101,21 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       mbar_init(&empty[s], 1);
     }
     mbar_init(q_full, 1);
-    mbar_init(s_full, 1);
+    mbar_init(&s_full[0], 1);
+    mbar_init(&s_full[1], 1);
     mbar_init(p_full, 4);
     mbar_init(o_full, 1);
     s_grow[0] = s_grow[1] = 0;
     fence_mbar_init();
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, 512);                         // S (N columns) | O: m_tiles x (hi N, lo N) from column 32
+    tmem_alloc(tmem_slot, 512);                         // S0 | S1 (N columns each) | O: m_tiles x (hi N, lo N) from column 64
     tmem_relinquish();
   }
   tcgen05_fence_before();
   __syncthreads();
   tcgen05_fence_after();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 32;
+  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 64;
 
   if (warp == 0) {
     if (lane == 0) {
@@ -150,62 +154,75 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       }
     }
   } else if (warp == 1) {
-    if (lane == 0) {
-      constexpr uint32_t idesc_s = umma_idesc(kLdKeys, N, 1, 1);
-      constexpr uint32_t idesc_o = umma_idesc(128, 2 * N, 1, 1) | (1u << 15);         // A (= V^T) MN-major
-      const uint32_t ring_addr = smem_u32(ring), q_addr = smem_u32(sQ), p_addr = smem_u32(sTP);
-      const int steps = (p.D + 15) >> 4;
-      bool ok = mbar_wait(q_full, 0, p.status);
-      for (int t = 0; t < n_tiles && ok; ++t) {
-        const int g0 = t * units;
-        for (int u = 0; u < units; ++u) {
-          const int s = (g0 + u) % Cfg::kSlots;
-          if (!mbar_wait_parked(&full[s], ((g0 + u) / Cfg::kSlots) & 1, p.status)) { ok = false; break; }
-          tcgen05_fence_after();
-          for (int k = u * 8; k < min(steps, u * 8 + 8); ++k) {
-            const int box = k >> 2, sub = (k & 3) * 32;
-            umma_f16(tmem_s, umma_desc_k_sw128(ring_addr + s * kLdUnit + (box & 1) * kLdBox + sub), umma_desc_k_sw128(q_addr + box * N * 128 + sub),
-                     idesc_s, k != 0);
-          }
-          if (u >= m_tiles) umma_commit(&empty[s]);     // no value columns in this unit
-        }
-        if (!ok) break;
-        umma_commit(s_full);
-        if (!mbar_wait_parked(p_full, t & 1, p.status)) break;
-        tcgen05_fence_after();
-        for (int m = 0; m < m_tiles; ++m) {
-          const int s = (g0 + m) % Cfg::kSlots;
+    // Many small products: the instructions around each count.  Descriptors are a base plus (bytes >> 4), and the whole warp issues.
+    constexpr uint32_t idesc_s = umma_idesc(128, N, 1, 1);
+    constexpr uint32_t idesc_o = umma_idesc(128, 2 * N, 1, 1) | (1u << 15);           // A (= V^T) MN-major
+    const uint64_t k_desc = umma_desc_k_sw128(smem_u32(ring)), v_desc = latent_v_desc(smem_u32(ring));
+    const uint64_t q_desc = umma_desc_k_sw128(smem_u32(sQ)), p_desc = umma_desc_k_sw128(smem_u32(sTP));
+    const int steps = (p.D + 15) >> 4;
+    int s_slot = 0, o_slot = 0;                         // unit that comes next for S and for O
+    uint32_t s_phase = 0;
+    bool ok = __all_sync(0xffffffffu, mbar_wait(q_full, 0, p.status));
+    auto issue_s = [&](int t, int u) {                  // unit u of tile t's scores
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(&full[s_slot], s_phase, p.status));
+      if (!ok) return;
+      tcgen05_fence_after();
+      const uint32_t d = tmem_s + (t & 1) * N;
+      const uint64_t ad = k_desc + static_cast<uint32_t>(s_slot * (kLdUnit >> 4)), bd = q_desc + static_cast<uint32_t>(u * (2 * N * 128 >> 4));
+      const int n = steps - u * 8;
 #pragma unroll
-          for (int k = 0; k < kLdKeys / 16; ++k)
-            umma_f16(tmem_o + m * 2 * N, latent_v_desc(ring_addr + s * kLdUnit + k * 16 * 128),
-                     umma_desc_k_sw128(p_addr + (k >> 2) * 2 * N * 128 + (k & 3) * 32), idesc_o, (t | k) != 0);
-          umma_commit(&empty[s]);
-        }
+      for (int k = 0; k < 8; ++k)
+        if (k < n)
+          umma_f16_warp(d, ad + (((k >> 2) * kLdBox + (k & 3) * 32) >> 4), bd + (((k >> 2) * N * 128 + (k & 3) * 32) >> 4), idesc_s, (u | k) != 0);
+      if (u >= m_tiles) umma_commit_warp(&empty[s_slot]);        // no value columns in this unit
+      if (++s_slot == Cfg::kSlots) { s_slot = 0; s_phase ^= 1; }
+    };
+    for (int u = 0; u < units; ++u) issue_s(0, u);
+    if (ok) umma_commit_warp(&s_full[0]);
+    for (int t = 0; t < n_tiles && ok; ++t) {
+      const bool more = t + 1 < n_tiles;
+      int u = 0;
+      for (; more && u < min(2, units); ++u) issue_s(t + 1, u);
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(p_full, t & 1, p.status));
+      if (!ok) break;
+      tcgen05_fence_after();
+      int s = o_slot;
+      for (int m = 0; m < m_tiles; ++m) {
+        const uint64_t ad = v_desc + static_cast<uint32_t>(s * (kLdUnit >> 4));
+#pragma unroll
+        for (int k = 0; k < kLdKeys / 16; ++k)
+          umma_f16_warp(tmem_o + m * 2 * N, ad + (k * 16 * 128 >> 4), p_desc + (k * 32 >> 4), idesc_o, (t | k) != 0);
+        umma_commit_warp(&empty[s]);
+        if (++s == Cfg::kSlots) s = 0;
+        if (more && u < units) issue_s(t + 1, u++);
       }
-      if (ok) umma_commit(o_full);
+      for (; more && u < units; ++u) issue_s(t + 1, u);
+      if (ok) umma_commit_warp(more ? &s_full[(t + 1) & 1] : o_full);
+      o_slot += units;
+      if (o_slot >= Cfg::kSlots) o_slot -= Cfg::kSlots;
     }
   } else {
     const int quad = warp & 3, key = quad * 32 + lane;   // TMEM lane = key of the tile
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const int tid = key, head = tid / kHeadThreads, sub = tid % kHeadThreads;
-    float* sT = reinterpret_cast<float*>(sTP);
     float m_ref = 0.f, l_run = 0.f;
-    bool ok = true;
+    // a wait that runs out is in the status word; the loop goes on, so that all four warps meet at the barriers
     for (int t = 0; t < n_tiles; ++t) {
-      // S of tile t is complete, and with it every product issued before: the weights of tile t - 1 may be overwritten
-      ok = mbar_wait(s_full, t & 1, p.status);
+      // S of tile t is complete, and with it every product issued before, O of tile t - 1 among them: the weights may be overwritten
+      mbar_wait(&s_full[t & 1], (t >> 1) & 1, p.status);
       tcgen05_fence_after();
-      {
+      float* sT = reinterpret_cast<float*>(sTP);
+      if (quad < 2) {
         uint32_t v[N];
-        if constexpr (N == 16) tmem_ld_x16(tmem_s + lane_addr, v);
-        else tmem_ld_x32(tmem_s + lane_addr, v);
+        if constexpr (N == 16) tmem_ld_x16(tmem_s + (t & 1) * N + lane_addr, v);
+        else tmem_ld_x32(tmem_s + (t & 1) * N + lane_addr, v);
         tmem_ld_wait();
         const bool in = k_begin + t * kLdKeys + key < k_end;
 #pragma unroll
         for (int h = 0; h < N; ++h) sT[h * Cfg::kTPitch + key] = in ? __uint_as_float(v[h]) * p.scale_log2 : -INFINITY;
       }
-      if (tid == 0) s_grow[(t + 1) & 1] = 0;
       named_barrier_sync(1, 128);
+      if (tid == 0) s_grow[(t + 1) & 1] = 0;             // last read in tile t - 1, which everyone has left
       float x[kHeadKeys], mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < kHeadKeys; i += 4) {           // keys 8 (sub + kHeadThreads j) .. + 7: whole 16-byte chunks of the weight rows
@@ -252,8 +269,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           hi[e] = pack_bf16x2(p0, p1);
           lo[e] = pack_bf16x2(p0 - bf16_lo(hi[e]), p1 - bf16_hi(hi[e]));
         }
-        const int c = (i >> 3) * kHeadThreads + sub;     // 16-byte chunk of the 128 keys: box c / 8, chunk c % 8
-        uint8_t* row = sTP + (c >> 3) * 2 * N * 128 + head * 128 + (((c & 7) ^ (head & 7)) << 4);
+        const int c = (i >> 3) * kHeadThreads + sub;     // 16-byte chunk of the 64 keys
+        uint8_t* row = sTP + head * 128 + ((c ^ (head & 7)) << 4);
         *reinterpret_cast<uint4*>(row) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
         *reinterpret_cast<uint4*>(row + N * 128) = make_uint4(lo[0], lo[1], lo[2], lo[3]);    // N is a multiple of 8: same swizzle phase
       }
@@ -272,7 +289,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         ml[1] = l_run;
       }
     }
-    if (ok) ok = mbar_wait(o_full, 0, p.status);
+    mbar_wait(o_full, 0, p.status);
     named_barrier_sync(1, 128);
     tcgen05_fence_after();
     for (int m = 0; m < m_tiles; ++m) {

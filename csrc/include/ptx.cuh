@@ -201,6 +201,26 @@ __device__ __forceinline__ void umma_commit(uint64_t* bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
 }
 
+// The same two issued by a whole converged warp: one elected lane (the same one every time) executes the instruction.  The
+// operands stay warp-uniform for the compiler, so they need no per-instruction move into uniform registers; this halves the
+// issue time where small UMMAs follow each other closely.
+__device__ __forceinline__ void umma_f16_warp(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}\n"
+      ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+__device__ __forceinline__ void umma_commit_warp(uint64_t* bar) {
+  asm volatile(
+      "{\n\t.reg .pred e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
+      "@e tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}\n"
+      ::"r"(smem_u32(bar)) : "memory");
+}
+
 // ---- CTA pairs (cta_group::2) ----------------------------------------------------------------------------
 // Two CTAs of a cluster (ranks 2i, 2i + 1) on the two SMs of a pair work on one UMMA: M = 256 rows (128 per CTA), each
 // CTA keeps its own half of A and its own half of the N rows of B in its shared memory, at the same offsets, and gets the
