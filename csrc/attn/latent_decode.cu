@@ -11,18 +11,18 @@
 //                   fp32 and enter as bf16 hi and lo halves side by side on N (16 mantissa bits); hi and lo sums meet at the end
 //
 // CTA = (context chunk, group of heads, sequence).  A tile is ceil((R + rot) / 128) units of two boxes; a ring of two tiles' units
-// keeps loads in flight, and a unit is free again as soon as its 128 latent columns have been multiplied.  The products of tile
-// t + 1's scores and of tile t's O alternate unit by unit: the softmax of tile t overlaps the first scores of tile t + 1, and
-// tile t gives its units back early.  Warp roles (192 threads): warp
-// 0 = TMA producer, warp 1 = TMEM owner + UMMA issuer, warps 2..5 = softmax: scores go through shared memory to change from
-// one key per thread to a share of one head's keys per thread.  O is rescaled only when a head's maximum has grown by 2^8.
-// All waits are bounded (ptx.cuh).  Chunks are merged by a second kernel.
+// or more keeps loads in flight, and a unit is free again as soon as its 128 latent columns have been multiplied.  The products are
+// small (N = 16 .. 64), so issuing them is what costs: S and O have an issuing warp each, both S and P are double-buffered, and
+// the softmax of a tile overlaps the scores of the next and the sums of the one before.  Warp roles (224 threads): warp 0 = TMA
+// producer, warp 1 = TMEM owner + issuer of S, warp 2 = issuer of O, warps 3..6 = softmax: scores go through shared memory to
+// change from one key per thread to a share of one head's keys per thread.  O is rescaled only when a head's maximum has grown by
+// 2^8.  All waits are bounded (ptx.cuh).  Chunks are merged by a second kernel.
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
 namespace forge {
 
-constexpr int kLdKeys = 64, kLdThreads = 192, kLdBox = kLdKeys * 128, kLdUnit = 2 * kLdBox, kLdMaxD = 576;
+constexpr int kLdKeys = 64, kLdThreads = 224, kLdBox = kLdKeys * 128, kLdUnit = 2 * kLdBox, kLdMaxD = 576;
 
 struct LatentDecodeArgs {
   const int* block_tables;   // [seqs][table_width]
@@ -37,11 +37,11 @@ struct LatentDecodeArgs {
 
 template <int N>
 struct LatentDecodeCfg {
-  static constexpr int kSlots = N == 16 ? 12 : 11;
+  static constexpr int kSlots = N == 16 ? 12 : 10;
   static constexpr int kTPitch = kLdKeys + 4;                        // floats per head of the transposed scores
   static constexpr int kQBytes = (kLdMaxD / 64) * N * 128;
-  static constexpr int kTBytes = (N * kTPitch * 4 + 1023) / 1024 * 1024;      // also holds the weights: 2N rows x 128 bytes
-  static constexpr int kSmem = kSlots * kLdUnit + kQBytes + kTBytes + 512 + 1024;
+  static constexpr int kTBytes = (N * kTPitch * 4 + 1023) / 1024 * 1024;      // per buffer; also holds the weights: 2N rows x 128 bytes
+  static constexpr int kSmem = kSlots * kLdUnit + kQBytes + 2 * kTBytes + 512 + 1024;
   static_assert(kTBytes >= 2 * N * 128 && kSlots >= 2 * ((kLdMaxD + 127) / 128) && kSmem <= 227 * 1024, "shared memory");
 };
 
@@ -56,6 +56,12 @@ __device__ __forceinline__ uint64_t latent_v_desc(uint32_t smem_addr) {
   return d;
 }
 
+// A bounded wait by a whole warp, and a value that is the same in all its lanes (UMMA operands live in uniform registers).
+__device__ __forceinline__ bool warp_wait(uint64_t* bar, uint32_t parity, unsigned* status) {
+  return __all_sync(0xffffffffu, mbar_wait(bar, parity, status));
+}
+__device__ __forceinline__ uint32_t warp_uniform(uint32_t x) { return __shfl_sync(0xffffffffu, x, 0); }
+
 // tm_q: [seqs * heads, D], box N x 64; tm_kv: [blocks * block_size, D], box min(64, block_size) x 64.
 template <int N>
 __global__ void __launch_bounds__(kLdThreads, 1)
@@ -66,15 +72,17 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* ring = smem;
   uint8_t* sQ = ring + Cfg::kSlots * kLdUnit;
-  uint8_t* sTP = sQ + Cfg::kQBytes;                     // scores [N][kTPitch] fp32, then weights
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sTP + Cfg::kTBytes);
+  uint8_t* sTP = sQ + Cfg::kQBytes;                     // [2]: scores [N][kTPitch] fp32, then weights
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sTP + 2 * Cfg::kTBytes);
   uint64_t* full = bars;                                // [kSlots]
   uint64_t* empty = full + Cfg::kSlots;                 // [kSlots]
   uint64_t* q_full = empty + Cfg::kSlots;
   uint64_t* s_full = q_full + 1;                        // [2]
-  uint64_t* p_full = q_full + 3;                        // one arrival per softmax warp
-  uint64_t* o_full = q_full + 4;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 5);
+  uint64_t* s_empty = q_full + 3;                       // [2], one arrival per softmax warp that reads scores (two of them)
+  uint64_t* p_full = q_full + 5;                        // [2], one arrival per softmax warp
+  uint64_t* pv_done = q_full + 7;                       // [2]: O += of the tile that used this weights' buffer is complete
+  uint64_t* o_full = q_full + 9;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 10);
   int* s_grow = reinterpret_cast<int*>(tmem_slot + 1);  // [2]: some head's maximum has grown (by tile parity)
   float* s_scale = reinterpret_cast<float*>(s_grow + 3);       // [N]
 
@@ -101,9 +109,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       mbar_init(&empty[s], 1);
     }
     mbar_init(q_full, 1);
-    mbar_init(&s_full[0], 1);
-    mbar_init(&s_full[1], 1);
-    mbar_init(p_full, 4);
+    for (int b = 0; b < 2; ++b) {
+      mbar_init(&s_full[b], 1);
+      mbar_init(&s_empty[b], 2);
+      mbar_init(&p_full[b], 4);
+      mbar_init(&pv_done[b], 1);
+    }
     mbar_init(o_full, 1);
     s_grow[0] = s_grow[1] = 0;
     fence_mbar_init();
@@ -154,53 +165,62 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       }
     }
   } else if (warp == 1) {
-    // Many small products: the instructions around each count.  Descriptors are a base plus (bytes >> 4), and the whole warp issues.
     constexpr uint32_t idesc_s = umma_idesc(128, N, 1, 1);
-    constexpr uint32_t idesc_o = umma_idesc(128, 2 * N, 1, 1) | (1u << 15);           // A (= V^T) MN-major
-    const uint64_t k_desc = umma_desc_k_sw128(smem_u32(ring)), v_desc = latent_v_desc(smem_u32(ring));
-    const uint64_t q_desc = umma_desc_k_sw128(smem_u32(sQ)), p_desc = umma_desc_k_sw128(smem_u32(sTP));
+    const uint64_t k_desc = umma_desc_k_sw128(smem_u32(ring)), q_desc = umma_desc_k_sw128(smem_u32(sQ));
     const int steps = (p.D + 15) >> 4;
-    int s_slot = 0, o_slot = 0;                         // unit that comes next for S and for O
-    uint32_t s_phase = 0;
-    bool ok = __all_sync(0xffffffffu, mbar_wait(q_full, 0, p.status));
-    auto issue_s = [&](int t, int u) {                  // unit u of tile t's scores
-      ok = ok && __all_sync(0xffffffffu, mbar_wait(&full[s_slot], s_phase, p.status));
-      if (!ok) return;
-      tcgen05_fence_after();
-      const uint32_t d = tmem_s + (t & 1) * N;
-      const uint64_t ad = k_desc + static_cast<uint32_t>(s_slot * (kLdUnit >> 4)), bd = q_desc + static_cast<uint32_t>(u * (2 * N * 128 >> 4));
-      const int n = steps - u * 8;
-#pragma unroll
-      for (int k = 0; k < 8; ++k)
-        if (k < n)
-          umma_f16_warp(d, ad + (((k >> 2) * kLdBox + (k & 3) * 32) >> 4), bd + (((k >> 2) * N * 128 + (k & 3) * 32) >> 4), idesc_s, (u | k) != 0);
-      if (u >= m_tiles) umma_commit_warp(&empty[s_slot]);        // no value columns in this unit
-      if (++s_slot == Cfg::kSlots) { s_slot = 0; s_phase ^= 1; }
-    };
-    for (int u = 0; u < units; ++u) issue_s(0, u);
-    if (ok) umma_commit_warp(&s_full[0]);
+    int slot = 0;
+    uint32_t phase = 0;
+    bool ok = warp_wait(q_full, 0, p.status);
     for (int t = 0; t < n_tiles && ok; ++t) {
-      const bool more = t + 1 < n_tiles;
-      int u = 0;
-      for (; more && u < min(2, units); ++u) issue_s(t + 1, u);
-      ok = ok && __all_sync(0xffffffffu, mbar_wait(p_full, t & 1, p.status));
+      if (t >= 2) ok = warp_wait(&s_empty[t & 1], ((t >> 1) - 1) & 1, p.status);         // softmax has read S of tile t - 2
+      const uint32_t d = warp_uniform(tmem_s + (t & 1) * N);
+      for (int u = 0; u < units && ok; ++u) {
+        ok = warp_wait(&full[slot], phase, p.status);
+        if (!ok) break;
+        tcgen05_fence_after();
+        const uint32_t bt = warp_uniform(u * (2 * N * 128 >> 4));
+        const uint64_t ad = k_desc + warp_uniform(slot * (kLdUnit >> 4)), bd = q_desc + bt;
+        const int n = steps - u * 8;
+        auto product = [&](int k) {
+          umma_f16_warp(d, ad + (((k >> 2) * kLdBox + (k & 3) * 32) >> 4), bd + (((k >> 2) * N * 128 + (k & 3) * 32) >> 4), idesc_s, k != 0 || bt != 0);
+        };
+        if (n >= 8) {
+#pragma unroll
+          for (int k = 0; k < 8; ++k) product(k);
+        } else {
+#pragma unroll
+          for (int k = 0; k < 7; ++k)
+            if (k < n) product(k);
+        }
+        if (u >= m_tiles) umma_commit_warp(&empty[slot]);        // no value columns in this unit
+        if (++slot == Cfg::kSlots) { slot = 0; phase ^= 1; }
+      }
+      if (ok) umma_commit_warp(&s_full[t & 1]);
+    }
+  } else if (warp == 2) {
+    constexpr uint32_t idesc_o = umma_idesc(128, 2 * N, 1, 1) | (1u << 15);           // A (= V^T) MN-major
+    const uint64_t v_desc = latent_v_desc(smem_u32(ring)), p_desc = umma_desc_k_sw128(smem_u32(sTP));
+    int slot0 = 0;                                      // first unit of the tile
+    bool ok = true;
+    for (int t = 0; t < n_tiles && ok; ++t) {
+      ok = warp_wait(&p_full[t & 1], (t >> 1) & 1, p.status);    // and with it: the tile's units are in place
       if (!ok) break;
       tcgen05_fence_after();
-      int s = o_slot;
+      const uint64_t bd = p_desc + warp_uniform((t & 1) * (Cfg::kTBytes >> 4));
+      int slot = slot0;
       for (int m = 0; m < m_tiles; ++m) {
-        const uint64_t ad = v_desc + static_cast<uint32_t>(s * (kLdUnit >> 4));
+        const uint32_t d = warp_uniform(tmem_o + m * 2 * N);
+        const uint64_t ad = v_desc + warp_uniform(slot * (kLdUnit >> 4));
 #pragma unroll
-        for (int k = 0; k < kLdKeys / 16; ++k)
-          umma_f16_warp(tmem_o + m * 2 * N, ad + (k * 16 * 128 >> 4), p_desc + (k * 32 >> 4), idesc_o, (t | k) != 0);
-        umma_commit_warp(&empty[s]);
-        if (++s == Cfg::kSlots) s = 0;
-        if (more && u < units) issue_s(t + 1, u++);
+        for (int k = 0; k < kLdKeys / 16; ++k) umma_f16_warp(d, ad + (k * 16 * 128 >> 4), bd + (k * 32 >> 4), idesc_o, k != 0 || t != 0);
+        umma_commit_warp(&empty[slot]);
+        if (++slot == Cfg::kSlots) slot = 0;
       }
-      for (; more && u < units; ++u) issue_s(t + 1, u);
-      if (ok) umma_commit_warp(more ? &s_full[(t + 1) & 1] : o_full);
-      o_slot += units;
-      if (o_slot >= Cfg::kSlots) o_slot -= Cfg::kSlots;
+      umma_commit_warp(&pv_done[t & 1]);
+      slot0 += units;
+      if (slot0 >= Cfg::kSlots) slot0 -= Cfg::kSlots;
     }
+    if (ok) umma_commit_warp(o_full);
   } else {
     const int quad = warp & 3, key = quad * 32 + lane;   // TMEM lane = key of the tile
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
@@ -208,15 +228,19 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     float m_ref = 0.f, l_run = 0.f;
     // a wait that runs out is in the status word; the loop goes on, so that all four warps meet at the barriers
     for (int t = 0; t < n_tiles; ++t) {
-      // S of tile t is complete, and with it every product issued before, O of tile t - 1 among them: the weights may be overwritten
       mbar_wait(&s_full[t & 1], (t >> 1) & 1, p.status);
+      if (t >= 2) mbar_wait(&pv_done[t & 1], ((t >> 1) - 1) & 1, p.status);     // the buffer's weights (tile t - 2) have been used
       tcgen05_fence_after();
-      float* sT = reinterpret_cast<float*>(sTP);
+      uint8_t* tp = sTP + (t & 1) * Cfg::kTBytes;
+      float* sT = reinterpret_cast<float*>(tp);
       if (quad < 2) {
         uint32_t v[N];
         if constexpr (N == 16) tmem_ld_x16(tmem_s + (t & 1) * N + lane_addr, v);
         else tmem_ld_x32(tmem_s + (t & 1) * N + lane_addr, v);
         tmem_ld_wait();
+        tcgen05_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&s_empty[t & 1]);
         const bool in = k_begin + t * kLdKeys + key < k_end;
 #pragma unroll
         for (int h = 0; h < N; ++h) sT[h * Cfg::kTPitch + key] = in ? __uint_as_float(v[h]) * p.scale_log2 : -INFINITY;
@@ -248,6 +272,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       l_run *= alpha;
       named_barrier_sync(1, 128);                        // scores are in registers, scales and the flag are set
       if (t > 0 && s_grow[t & 1]) {
+        mbar_wait(&pv_done[(t - 1) & 1], ((t - 1) >> 1) & 1, p.status);         // every earlier product has landed in O
+        tcgen05_fence_after();
 #pragma unroll 1
         for (int c = 0; c < m_tiles * 2 * N; c += 32) {
           uint32_t o[32];
@@ -270,14 +296,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           lo[e] = pack_bf16x2(p0 - bf16_lo(hi[e]), p1 - bf16_hi(hi[e]));
         }
         const int c = (i >> 3) * kHeadThreads + sub;     // 16-byte chunk of the 64 keys
-        uint8_t* row = sTP + head * 128 + ((c ^ (head & 7)) << 4);
+        uint8_t* row = tp + head * 128 + ((c ^ (head & 7)) << 4);
         *reinterpret_cast<uint4*>(row) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
         *reinterpret_cast<uint4*>(row + N * 128) = make_uint4(lo[0], lo[1], lo[2], lo[3]);    // N is a multiple of 8: same swizzle phase
       }
       fence_proxy_async_smem();
       tcgen05_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_full);
+      if (lane == 0) mbar_arrive(&p_full[t & 1]);
     }
 #pragma unroll
     for (int off = kHeadThreads / 2; off > 0; off >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
