@@ -38,9 +38,10 @@ int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int
 int forge_head_linear(const void* x, long long x_tok, long long x_head, const void* w, void* out, long long o_tok, long long o_head, int M,
                       int heads, int N, int K, cudaStream_t stream);
 int forge_latent_decode_ok(int R, int rot, int block_size);
-int forge_latent_decode(const void* qa, const void* cache, const int* block_tables, const int* lens, void* o, float* part_o, float* part_ml,
-                        int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size, int chunk, int max_chunks,
-                        float scale, unsigned* status, cudaStream_t stream);
+long long forge_latent_decode_scratch(int heads, int R, int ctas);
+int forge_latent_decode(const void* qa, const void* cache, const int* block_tables, const int* lens, void* o, float* scratch, int ctas,
+                        int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size, float scale, unsigned* status,
+                        cudaStream_t stream);
 int forge_latent_prefill_qcols(int dim, int rot, int vdim);
 int forge_latent_prefill(const void* q, const void* kv, const void* kr, const int* cu_q, const int* cu_k, void* out, int tokens, int tok0,
                          int keys, int num_seqs, int max_q, int heads, int dim, int rot, int vdim, float scale, unsigned* status,
@@ -320,22 +321,17 @@ void head_linear(const Tensor& x, const Tensor& w, Tensor& out) {
            "forge_head_linear");
 }
 
-void latent_decode(const Tensor& qa, const Tensor& cache, const Tensor& block_tables, const Tensor& lens, Tensor& o, const OptTensor& part_o,
-                   const OptTensor& part_ml, int64_t chunk, int64_t max_chunks, double scale, const Tensor& status) {
+// scratch: fp32, latent_decode_scratch(heads, R, ctas) elements
+void latent_decode(const Tensor& qa, const Tensor& cache, const Tensor& block_tables, const Tensor& lens, Tensor& o, Tensor& scratch, int64_t ctas,
+                   double scale, const Tensor& status) {
   TORCH_CHECK(qa.dim() == 3 && cache.dim() == 3 && block_tables.dim() == 2 && o.dim() == 3, "latent_decode: ranks");
   const int64_t B = qa.size(0), H = qa.size(1), D = qa.size(2), R = o.size(2);
-  TORCH_CHECK(cache.size(2) == D && R <= D && o.size(0) == B && o.size(1) == H && block_tables.size(0) >= B && max_chunks >= 1, "latent_decode: shapes");
-  float *po = nullptr, *pml = nullptr;
-  if (max_chunks > 1) {
-    TORCH_CHECK(part_o.has_value() && part_ml.has_value(), "latent_decode: scratch");
-    po = floats(*part_o, B * H * max_chunks * R, "part_o");
-    pml = floats(*part_ml, B * H * max_chunks * 2, "part_ml");
-  }
+  TORCH_CHECK(cache.size(2) == D && R <= D && o.size(0) == B && o.size(1) == H && block_tables.size(0) >= B, "latent_decode: shapes");
   const c10::cuda::CUDAGuard guard(qa.device());
   check_rc(forge_latent_decode(data(qa, kBf16, 0, "qa"), data(cache, kBf16, 0, "cache"), ints(block_tables, 0, "block_tables"), ints(lens, B, "lens"),
-                               data(o, kBf16, 0, "o"), po, pml, i32(B), i32(H), i32(R), i32(D - R), i32(block_tables.size(1)), i32(cache.size(0)),
-                               i32(cache.size(1)), i32(chunk), i32(max_chunks), static_cast<float>(scale), status_word(status),
-                               stream_of(qa)),
+                               data(o, kBf16, 0, "o"), floats(scratch, forge_latent_decode_scratch(i32(H), i32(R), i32(ctas)), "scratch"), i32(ctas),
+                               i32(B), i32(H), i32(R), i32(D - R), i32(block_tables.size(1)), i32(cache.size(0)), i32(cache.size(1)),
+                               static_cast<float>(scale), status_word(status), stream_of(qa)),
            "forge_latent_decode");
 }
 
@@ -416,6 +412,7 @@ void register_mixers(pybind11::module& m) {
   m.def("grouped_gemm", &grouped_gemm);
   m.def("head_linear", &head_linear);
   m.def("latent_decode", &latent_decode);
+  m.def("latent_decode_scratch", [](int64_t H, int64_t R, int64_t ctas) { return static_cast<int64_t>(forge_latent_decode_scratch(i32(H), i32(R), i32(ctas))); });
   m.def("latent_decode_ok", [](int64_t R, int64_t rot, int64_t bs) { return forge_latent_decode_ok(i32(R), i32(rot), i32(bs)) != 0; });
   m.def("latent_gather", &latent_gather);
   m.def("latent_pack_q", &latent_pack_q);

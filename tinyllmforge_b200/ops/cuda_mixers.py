@@ -71,15 +71,6 @@ class MixerOps:
         self._latent_folded(q, weights, cache, batch, table, spec, out, n1)
         return out
 
-    def latent_chunking(self, seqs: int, heads: int, max_len: int) -> tuple[int, int]:
-        """(keys per chunk, chunks) of the decode kernel: enough chunks to fill the GPU, from
-        shapes known at capture time."""
-        want = -(-self.num_sms // (seqs * -(-heads // 32)))       # one CTA per SM, up to 32 heads each
-        chunk = 128
-        while chunk < 1024 and -(-max_len // (2 * chunk)) >= want:
-            chunk *= 2
-        return chunk, max(1, -(-max_len // chunk))
-
     def _latent_folded(self, q, weights, cache, batch, table, spec, out, n) -> None:
         """The first n tokens of the step."""
         H, d, r, dv, R = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
@@ -91,14 +82,9 @@ class MixerOps:
         self.C.latent_rotate_q(q, qa, d, R, table, batch.positions[:n])
         o = torch.empty(n, H, R, dtype=q.dtype, device=q.device)
         singles = n == (batch.num_single if batch.is_prefill else batch.padded_seqs)
-        if singles and q.dtype == torch.bfloat16 and self.C.latent_decode_ok(R, r, cache.shape[1]):
-            chunk, chunks = self.latent_chunking(n, H, batch.table_width * cache.shape[1])
-            part_o = part_ml = None
-            if chunks > 1:
-                part_o = torch.empty(n * H * chunks * R, dtype=torch.float32, device=q.device)
-                part_ml = torch.empty(n * H * chunks * 2, dtype=torch.float32, device=q.device)
-            self.C.latent_decode(qa, cache, batch.block_tables, batch.context_lens, o, part_o, part_ml, chunk, chunks,
-                                 spec.scale, self.status)
+        if singles and q.dtype == torch.bfloat16 and n <= 1024 and self.C.latent_decode_ok(R, r, cache.shape[1]):
+            scratch = torch.empty(self.C.latent_decode_scratch(H, R, self.num_sms), dtype=torch.float32, device=q.device)
+            self.C.latent_decode(qa, cache, batch.block_tables, batch.context_lens, o, scratch, self.num_sms, spec.scale, self.status)
         else:
             self.C.latent_attend_any(qa, cache, o, 0, batch.cu_seqlens_q, batch.padded_seqs, batch.positions, batch.block_tables,
                                      spec.scale, self.status)

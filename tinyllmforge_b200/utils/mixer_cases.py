@@ -39,10 +39,8 @@ def _latent_decode(ops, heads, B=64, ctx=2048):
     bt = torch.randperm(B * ctx // bs, dtype=torch.int32).view(B, -1).cuda()
     lens = _ints([ctx] * B)
     qa, o = _rand(B, heads, R + r), _rand(B, heads, R)
-    chunk, n = ops.latent_chunking(B, heads, ctx)
-    po = torch.empty(B * heads * n * R, device="cuda")
-    pml = torch.empty(B * heads * n * 2, device="cuda")
-    return (lambda: ops.C.latent_decode(qa, cache, bt, lens, o, po, pml, chunk, n, LATENT.scale, ops.status),
+    scratch = torch.empty(ops.C.latent_decode_scratch(heads, R, ops.num_sms), device="cuda")
+    return (lambda: ops.C.latent_decode(qa, cache, bt, lens, o, scratch, ops.num_sms, LATENT.scale, ops.status),
             B * ctx * (R + r) * 2 + B * heads * (2 * R + r) * 2, 2 * B * heads * ctx * (2 * R + r))
 
 
