@@ -15,9 +15,10 @@
 // result, partial ones leave sums that a second kernel merges.  Lengths are read on the device, so a captured graph serves
 // any.  A tile is ceil((R + rot) / 128) units of two boxes; a ring of two tiles' units
 // or more keeps loads in flight, and a unit is free again as soon as its 128 latent columns have been multiplied.  The products are
-// small (N = 16 .. 64), so issuing them is what costs: S and O have an issuing warp each, both S and P are double-buffered, and
-// the softmax of a tile overlaps the scores of the next and the sums of the one before.  Warp roles (224 threads): warp 0 = TMA
-// producer, warp 1 = TMEM owner + issuer of S, warp 2 = issuer of O, warps 3..6 = softmax: scores go through shared memory to
+// small (N = 16 .. 64), so issuing them is what costs: S has two issuing warps (even and odd units, an accumulator each, added by
+// the softmax), O has one, both S and P are double-buffered, and the softmax of a tile overlaps the scores of the next and the
+// sums of the one before.  Warp roles (256 threads): warp 0 = TMA producer, warps 1, 2 = issuers of S (1 owns tensor memory),
+// warp 3 = issuer of O, warps 4..7 = softmax: scores go through shared memory to
 // change from one key per thread to a share of one head's keys per thread.  O is rescaled only when a head's maximum has grown by
 // 2^8.  All waits are bounded (ptx.cuh).
 #include "../include/launch.cuh"
@@ -25,7 +26,7 @@
 
 namespace forge {
 
-constexpr int kLdKeys = 64, kLdThreads = 224, kLdBox = kLdKeys * 128, kLdUnit = 2 * kLdBox, kLdMaxD = 576;
+constexpr int kLdKeys = 64, kLdThreads = 256, kLdBox = kLdKeys * 128, kLdUnit = 2 * kLdBox, kLdMaxD = 576;
 
 struct LatentDecodeArgs {
   const int* block_tables;   // [seqs][table_width]
@@ -162,10 +163,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       mbar_init(&empty[s], 1);
     }
     mbar_init(q_full, 1);
-    mbar_init(q_empty, 1);
+    mbar_init(q_empty, min(units, 2));
     mbar_init(o_empty, 4);
     for (int b = 0; b < 2; ++b) {
-      mbar_init(&s_full[b], 1);
+      mbar_init(&s_full[b], min(units, 2));
       mbar_init(&s_empty[b], 2);
       mbar_init(&p_full[b], 4);
       mbar_init(&pv_done[b], 1);
@@ -175,13 +176,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     fence_mbar_init();
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, 512);                         // S0 | S1 (N columns each) | O: m_tiles x (hi N, lo N) from column 64
+    tmem_alloc(tmem_slot, 512);                         // S: two buffers x two parts of N columns | O: m_tiles x (hi N, lo N) from column 128
     tmem_relinquish();
   }
   tcgen05_fence_before();
   __syncthreads();
   tcgen05_fence_after();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 64;
+  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 128;
 
   if (warp == 0) {
     if (lane == 0) {
@@ -225,45 +226,49 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         }
       }
     }
-  } else if (warp == 1) {
+  } else if (warp <= 2) {
+    const int part = warp - 1;                          // units part, part + 2, ...
     constexpr uint32_t idesc_s = umma_idesc(128, N, 1, 1);
     const uint64_t k_desc = umma_desc_k_sw128(smem_u32(ring)), q_desc = umma_desc_k_sw128(smem_u32(sQ));
     const int steps = (p.D + 15) >> 4;
-    int slot = 0;
-    uint32_t phase = 0;
-    int t = 0, n_piece = 0;                             // tiles and pieces of this CTA so far
-    bool ok = true;
+    int slot0 = 0, t = 0, n_piece = 0;                  // first unit of the tile; tiles and pieces of this CTA so far
+    uint32_t phase0 = 0;
+    bool ok = part < units;
     for (; ok && pc.next(before, p.seqs, p.groups); ++n_piece) {
-    ok = warp_wait(q_full, n_piece & 1, p.status);
-    for (int left = pc.tiles; left > 0 && ok; --left, ++t) {
-      if (t >= 2) ok = warp_wait(&s_empty[t & 1], ((t >> 1) - 1) & 1, p.status);         // softmax has read S of tile t - 2
-      const uint32_t d = warp_uniform(tmem_s + (t & 1) * N);
-      for (int u = 0; u < units && ok; ++u) {
-        ok = warp_wait(&full[slot], phase, p.status);
-        if (!ok) break;
-        tcgen05_fence_after();
-        const uint32_t bt = warp_uniform(u * (2 * N * 128 >> 4));
-        const uint64_t ad = k_desc + warp_uniform(slot * (kLdUnit >> 4)), bd = q_desc + bt;
-        const int n = steps - u * 8;
-        auto product = [&](int k) {
-          umma_f16_warp(d, ad + (((k >> 2) * kLdBox + (k & 3) * 32) >> 4), bd + (((k >> 2) * N * 128 + (k & 3) * 32) >> 4), idesc_s, k != 0 || bt != 0);
-        };
-        if (n >= 8) {
+      ok = warp_wait(q_full, n_piece & 1, p.status);
+      for (int left = pc.tiles; left > 0 && ok; --left, ++t) {
+        if (t >= 2) ok = warp_wait(&s_empty[t & 1], ((t >> 1) - 1) & 1, p.status);       // softmax has read S of tile t - 2
+        const uint32_t d = warp_uniform(tmem_s + ((t & 1) * 2 + part) * N);
+        for (int u = part; u < units && ok; u += 2) {
+          int slot = slot0 + u;
+          uint32_t phase = phase0;
+          if (slot >= Cfg::kSlots) { slot -= Cfg::kSlots; phase ^= 1; }
+          ok = warp_wait(&full[slot], phase, p.status);
+          if (!ok) break;
+          tcgen05_fence_after();
+          const uint64_t ad = k_desc + warp_uniform(slot * (kLdUnit >> 4)), bd = q_desc + warp_uniform(u * (2 * N * 128 >> 4));
+          const uint32_t more = warp_uniform(u != part);
+          const int n = steps - u * 8;
+          auto product = [&](int k) {
+            umma_f16_warp(d, ad + (((k >> 2) * kLdBox + (k & 3) * 32) >> 4), bd + (((k >> 2) * N * 128 + (k & 3) * 32) >> 4), idesc_s, k != 0 ? 1 : more);
+          };
+          if (n >= 8) {
 #pragma unroll
-          for (int k = 0; k < 8; ++k) product(k);
-        } else {
+            for (int k = 0; k < 8; ++k) product(k);
+          } else {
 #pragma unroll
-          for (int k = 0; k < 7; ++k)
-            if (k < n) product(k);
+            for (int k = 0; k < 7; ++k)
+              if (k < n) product(k);
+          }
+          if (u >= m_tiles) umma_commit_warp(&empty[slot]);      // no value columns in this unit
         }
-        if (u >= m_tiles) umma_commit_warp(&empty[slot]);        // no value columns in this unit
-        if (++slot == Cfg::kSlots) { slot = 0; phase ^= 1; }
+        if (ok) umma_commit_warp(&s_full[t & 1]);
+        slot0 += units;
+        if (slot0 >= Cfg::kSlots) { slot0 -= Cfg::kSlots; phase0 ^= 1; }
       }
-      if (ok) umma_commit_warp(&s_full[t & 1]);
+      if (ok) umma_commit_warp(q_empty);
     }
-    if (ok) umma_commit_warp(q_empty);
-    }
-  } else if (warp == 2) {
+  } else if (warp == 3) {
     constexpr uint32_t idesc_o = umma_idesc(128, 2 * N, 1, 1) | (1u << 15);           // A (= V^T) MN-major
     const uint64_t v_desc = latent_v_desc(smem_u32(ring)), p_desc = umma_desc_k_sw128(smem_u32(sTP));
     int slot0 = 0, t = 0, n_piece = 0;                  // first unit of the tile; tiles and pieces so far
@@ -306,10 +311,20 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       uint8_t* tp = sTP + (t & 1) * Cfg::kTBytes;
       float* sT = reinterpret_cast<float*>(tp);
       if (quad < 2) {
-        uint32_t v[N];
-        if constexpr (N == 16) tmem_ld_x16(tmem_s + (t & 1) * N + lane_addr, v);
-        else tmem_ld_x32(tmem_s + (t & 1) * N + lane_addr, v);
+        uint32_t v[N], w[N];
+        const uint32_t at = tmem_s + (t & 1) * 2 * N + lane_addr;
+        if constexpr (N == 16) {
+          tmem_ld_x16(at, v);
+          tmem_ld_x16(at + N, w);
+        } else {
+          tmem_ld_x32(at, v);
+          tmem_ld_x32(at + N, w);
+        }
         tmem_ld_wait();
+        if (units > 1) {
+#pragma unroll
+          for (int h = 0; h < N; ++h) v[h] = __float_as_uint(__uint_as_float(v[h]) + __uint_as_float(w[h]));
+        }
         tcgen05_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&s_empty[t & 1]);
