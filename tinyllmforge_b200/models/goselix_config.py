@@ -191,3 +191,19 @@ class GoselixConfig:
     def prefix_cacheable(self) -> bool:
         """A recurrent state cannot be picked up in the middle of a prompt from cached blocks alone."""
         return self.num_recurrent_runs == 0
+
+
+def example_dict(width: int, layers: int = 4, vocab: int = 32000) -> dict:
+    """A configuration with the proportions of a real model of this width (16 heads of 128 per 2048 columns, latents of 512, feed-forwards of
+    three times the width, 32 experts of which four take the dense one's work together): latent attention and retention in
+    turn, dense and expert layers in turn two by two."""
+    heads = max(8, width // 128)
+    latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 3 * width // 8, "kv_rank": 512, "scale": 192 ** -0.5,
+              "rot": {"base": 1e6, "dims": 64}}
+    n = max(4, width // 256)
+    retention = {"heads": n, "dim": 128, "vdim": 256, "decay": [1.0 - 2.0 ** (-4 - 6.0 * h / n) for h in range(n)], "rot": {"base": 1e4, "dims": 128}}
+    dense = {"kind": "dense", "ff": 3 * width}
+    moe = {"kind": "moe", "router": {"experts": 32, "top": 4}, "expert": {"ff": 3 * width // 4}}
+    kinds = [("latent_attention", latent, dense), ("retention", retention, moe), ("latent_attention", latent, moe), ("retention", retention, dense)]
+    return {"architecture": "Goselix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [dict(zip(("type", "mixer", "mlp"), kinds[i % 4])) for i in range(layers)]}
