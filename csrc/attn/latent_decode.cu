@@ -274,26 +274,26 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     int slot0 = 0, t = 0, n_piece = 0;                  // first unit of the tile; tiles and pieces so far
     bool ok = true;
     for (; ok && pc.next(before, p.seqs, p.groups); ++n_piece) {
-    if (n_piece > 0) ok = warp_wait(o_empty, (n_piece - 1) & 1, p.status);            // the piece before has been read
-    for (int i = 0; i < pc.tiles && ok; ++i, ++t) {
-      ok = warp_wait(&p_full[t & 1], (t >> 1) & 1, p.status);    // and with it: the tile's units are in place
-      if (!ok) break;
-      tcgen05_fence_after();
-      const uint64_t bd = p_desc + warp_uniform((t & 1) * (Cfg::kTBytes >> 4));
-      int slot = slot0;
-      for (int m = 0; m < m_tiles; ++m) {
-        const uint32_t d = warp_uniform(tmem_o + m * 2 * N);
-        const uint64_t ad = v_desc + warp_uniform(slot * (kLdUnit >> 4));
+      if (n_piece > 0) ok = warp_wait(o_empty, (n_piece - 1) & 1, p.status);            // the piece before has been read
+      for (int i = 0; i < pc.tiles && ok; ++i, ++t) {
+        ok = warp_wait(&p_full[t & 1], (t >> 1) & 1, p.status);    // and with it: the tile's units are in place
+        if (!ok) break;
+        tcgen05_fence_after();
+        const uint64_t bd = p_desc + warp_uniform((t & 1) * (Cfg::kTBytes >> 4));
+        int slot = slot0;
+        for (int m = 0; m < m_tiles; ++m) {
+          const uint32_t d = warp_uniform(tmem_o + m * 2 * N);
+          const uint64_t ad = v_desc + warp_uniform(slot * (kLdUnit >> 4));
 #pragma unroll
-        for (int k = 0; k < kLdKeys / 16; ++k) umma_f16_warp(d, ad + (k * 16 * 128 >> 4), bd + (k * 32 >> 4), idesc_o, k != 0 || i != 0);
-        umma_commit_warp(&empty[slot]);
-        if (++slot == Cfg::kSlots) slot = 0;
+          for (int k = 0; k < kLdKeys / 16; ++k) umma_f16_warp(d, ad + (k * 16 * 128 >> 4), bd + (k * 32 >> 4), idesc_o, k != 0 || i != 0);
+          umma_commit_warp(&empty[slot]);
+          if (++slot == Cfg::kSlots) slot = 0;
+        }
+        umma_commit_warp(&pv_done[t & 1]);
+        slot0 += units;
+        if (slot0 >= Cfg::kSlots) slot0 -= Cfg::kSlots;
       }
-      umma_commit_warp(&pv_done[t & 1]);
-      slot0 += units;
-      if (slot0 >= Cfg::kSlots) slot0 -= Cfg::kSlots;
-    }
-    if (ok) umma_commit_warp(o_full);
+      if (ok) umma_commit_warp(o_full);
     }
   } else {
     const int quad = warp & 3, key = quad * 32 + lane;   // TMEM lane = key of the tile
@@ -301,137 +301,137 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     const int tid = key, head = tid / kHeadThreads, sub = tid % kHeadThreads;
     int t = 0, n_piece = 0;                              // tiles and pieces of this CTA so far
     for (; pc.next(before, p.seqs, p.groups); ++n_piece) {
-    const int len = min(p.lens[pc.seq], p.table_width << p.block_shift), h0 = pc.group * N;
-    float m_ref = 0.f, l_run = 0.f;
-    // a wait that runs out is in the status word; the loop goes on, so that all four warps meet at the barriers
-    for (int i_tile = 0; i_tile < pc.tiles; ++i_tile, ++t) {
-      mbar_wait_parked(&s_full[t & 1], (t >> 1) & 1, p.status);
-      if (t >= 2) mbar_wait_parked(&pv_done[t & 1], ((t >> 1) - 1) & 1, p.status);     // the buffer's weights (tile t - 2) have been used
-      tcgen05_fence_after();
-      uint8_t* tp = sTP + (t & 1) * Cfg::kTBytes;
-      float* sT = reinterpret_cast<float*>(tp);
-      if (quad < 2) {
-        uint32_t v[N], w[N];
-        const uint32_t at = tmem_s + (t & 1) * 2 * N + lane_addr;
-        if constexpr (N == 16) {
-          tmem_ld_x16(at, v);
-          tmem_ld_x16(at + N, w);
-        } else {
-          tmem_ld_x32(at, v);
-          tmem_ld_x32(at + N, w);
-        }
-        tmem_ld_wait();
-        if (units > 1) {
+      const int len = min(p.lens[pc.seq], p.table_width << p.block_shift), h0 = pc.group * N;
+      float m_ref = 0.f, l_run = 0.f;
+      // a wait that runs out is in the status word; the loop goes on, so that all four warps meet at the barriers
+      for (int i_tile = 0; i_tile < pc.tiles; ++i_tile, ++t) {
+        mbar_wait_parked(&s_full[t & 1], (t >> 1) & 1, p.status);
+        if (t >= 2) mbar_wait_parked(&pv_done[t & 1], ((t >> 1) - 1) & 1, p.status);     // the buffer's weights (tile t - 2) have been used
+        tcgen05_fence_after();
+        uint8_t* tp = sTP + (t & 1) * Cfg::kTBytes;
+        float* sT = reinterpret_cast<float*>(tp);
+        if (quad < 2) {
+          uint32_t v[N], w[N];
+          const uint32_t at = tmem_s + (t & 1) * 2 * N + lane_addr;
+          if constexpr (N == 16) {
+            tmem_ld_x16(at, v);
+            tmem_ld_x16(at + N, w);
+          } else {
+            tmem_ld_x32(at, v);
+            tmem_ld_x32(at + N, w);
+          }
+          tmem_ld_wait();
+          if (units > 1) {
 #pragma unroll
-          for (int h = 0; h < N; ++h) v[h] = __float_as_uint(__uint_as_float(v[h]) + __uint_as_float(w[h]));
+            for (int h = 0; h < N; ++h) v[h] = __float_as_uint(__uint_as_float(v[h]) + __uint_as_float(w[h]));
+          }
+          tcgen05_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&s_empty[t & 1]);
+          const bool in = (pc.tile + i_tile) * kLdKeys + key < len;
+#pragma unroll
+          for (int h = 0; h < N; ++h) sT[h * Cfg::kTPitch + key] = in ? __uint_as_float(v[h]) * p.scale_log2 : -INFINITY;
         }
+        named_barrier_sync(1, 128);
+        if (tid == 0) s_grow[(t + 1) & 1] = 0;             // last read in tile t - 1, which everyone has left
+        float x[kHeadKeys], mx = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < kHeadKeys; i += 4) {           // keys 8 (sub + kHeadThreads j) .. + 7: whole 16-byte chunks of the weight rows
+          const int at = ((i >> 3) * kHeadThreads + sub) * 8 + (i & 7);
+          const float4 f = *reinterpret_cast<const float4*>(sT + head * Cfg::kTPitch + at);
+          x[i] = f.x;
+          x[i + 1] = f.y;
+          x[i + 2] = f.z;
+          x[i + 3] = f.w;
+          mx = fmaxf(mx, fmaxf(fmaxf(f.x, f.y), fmaxf(f.z, f.w)));
+        }
+#pragma unroll
+        for (int off = kHeadThreads / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+        float alpha = 1.f;                                 // mx is finite: a tile holds at least one visible key
+        if (i_tile == 0) {
+          m_ref = mx;
+        } else if (mx - m_ref > 8.f) {
+          alpha = exp2f(m_ref - mx);
+          m_ref = mx;
+          s_grow[t & 1] = 1;
+        }
+        if (sub == 0) s_scale[head] = alpha;
+        l_run *= alpha;
+        named_barrier_sync(1, 128);                        // scores are in registers, scales and the flag are set
+        if (i_tile > 0 && s_grow[t & 1]) {
+          mbar_wait_parked(&pv_done[(t - 1) & 1], ((t - 1) >> 1) & 1, p.status);         // every earlier product has landed in O
+          tcgen05_fence_after();
+#pragma unroll 1
+          for (int c = 0; c < m_tiles * 2 * N; c += 32) {
+            uint32_t o[32];
+            tmem_ld_x32(tmem_o + lane_addr + c, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_scale[i % N]);
+            tmem_st_x32(tmem_o + lane_addr + c, o);
+          }
+          tmem_st_wait();
+        }
+#pragma unroll
+        for (int i = 0; i < kHeadKeys; i += 8) {
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float p0 = ex2_approx(x[i + 2 * e] - m_ref), p1 = ex2_approx(x[i + 2 * e + 1] - m_ref);
+            l_run += p0 + p1;
+            hi[e] = pack_bf16x2(p0, p1);
+            lo[e] = pack_bf16x2(p0 - bf16_lo(hi[e]), p1 - bf16_hi(hi[e]));
+          }
+          const int c = (i >> 3) * kHeadThreads + sub;     // 16-byte chunk of the 64 keys
+          uint8_t* row = tp + head * 128 + ((c ^ (head & 7)) << 4);
+          *reinterpret_cast<uint4*>(row) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(row + N * 128) = make_uint4(lo[0], lo[1], lo[2], lo[3]);    // N is a multiple of 8: same swizzle phase
+        }
+        fence_proxy_async_smem();
         tcgen05_fence_before();
         __syncwarp();
-        if (lane == 0) mbar_arrive(&s_empty[t & 1]);
-        const bool in = (pc.tile + i_tile) * kLdKeys + key < len;
+        if (lane == 0) mbar_arrive(&p_full[t & 1]);
+      }
 #pragma unroll
-        for (int h = 0; h < N; ++h) sT[h * Cfg::kTPitch + key] = in ? __uint_as_float(v[h]) * p.scale_log2 : -INFINITY;
+      for (int off = kHeadThreads / 2; off > 0; off >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
+      const bool whole = pc.starts && pc.ends;
+      const size_t part = static_cast<size_t>(blockIdx.x) * 2 + (pc.starts ? 1 : 0);
+      mbar_wait_parked(o_full, n_piece & 1, p.status);     // and with it: every warp is past its last use of s_scale
+      if (sub == 0) {
+        s_scale[head] = whole ? 1.f / l_run : 1.f;
+        if (!whole) {
+          p.part_ml[(part * N + head) * 2] = m_ref;
+          p.part_ml[(part * N + head) * 2 + 1] = l_run;
+        }
       }
       named_barrier_sync(1, 128);
-      if (tid == 0) s_grow[(t + 1) & 1] = 0;             // last read in tile t - 1, which everyone has left
-      float x[kHeadKeys], mx = -INFINITY;
-#pragma unroll
-      for (int i = 0; i < kHeadKeys; i += 4) {           // keys 8 (sub + kHeadThreads j) .. + 7: whole 16-byte chunks of the weight rows
-        const int at = ((i >> 3) * kHeadThreads + sub) * 8 + (i & 7);
-        const float4 f = *reinterpret_cast<const float4*>(sT + head * Cfg::kTPitch + at);
-        x[i] = f.x;
-        x[i + 1] = f.y;
-        x[i + 2] = f.z;
-        x[i + 3] = f.w;
-        mx = fmaxf(mx, fmaxf(fmaxf(f.x, f.y), fmaxf(f.z, f.w)));
-      }
-#pragma unroll
-      for (int off = kHeadThreads / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      float alpha = 1.f;                                 // mx is finite: a tile holds at least one visible key
-      if (i_tile == 0) {
-        m_ref = mx;
-      } else if (mx - m_ref > 8.f) {
-        alpha = exp2f(m_ref - mx);
-        m_ref = mx;
-        s_grow[t & 1] = 1;
-      }
-      if (sub == 0) s_scale[head] = alpha;
-      l_run *= alpha;
-      named_barrier_sync(1, 128);                        // scores are in registers, scales and the flag are set
-      if (i_tile > 0 && s_grow[t & 1]) {
-        mbar_wait_parked(&pv_done[(t - 1) & 1], ((t - 1) >> 1) & 1, p.status);         // every earlier product has landed in O
-        tcgen05_fence_after();
-#pragma unroll 1
-        for (int c = 0; c < m_tiles * 2 * N; c += 32) {
-          uint32_t o[32];
-          tmem_ld_x32(tmem_o + lane_addr + c, o);
-          tmem_ld_wait();
-#pragma unroll
-          for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_scale[i % N]);
-          tmem_st_x32(tmem_o + lane_addr + c, o);
-        }
-        tmem_st_wait();
-      }
-#pragma unroll
-      for (int i = 0; i < kHeadKeys; i += 8) {
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float p0 = ex2_approx(x[i + 2 * e] - m_ref), p1 = ex2_approx(x[i + 2 * e + 1] - m_ref);
-          l_run += p0 + p1;
-          hi[e] = pack_bf16x2(p0, p1);
-          lo[e] = pack_bf16x2(p0 - bf16_lo(hi[e]), p1 - bf16_hi(hi[e]));
-        }
-        const int c = (i >> 3) * kHeadThreads + sub;     // 16-byte chunk of the 64 keys
-        uint8_t* row = tp + head * 128 + ((c ^ (head & 7)) << 4);
-        *reinterpret_cast<uint4*>(row) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        *reinterpret_cast<uint4*>(row + N * 128) = make_uint4(lo[0], lo[1], lo[2], lo[3]);    // N is a multiple of 8: same swizzle phase
-      }
-      fence_proxy_async_smem();
-      tcgen05_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&p_full[t & 1]);
-    }
-#pragma unroll
-    for (int off = kHeadThreads / 2; off > 0; off >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, off);
-    const bool whole = pc.starts && pc.ends;
-    const size_t part = static_cast<size_t>(blockIdx.x) * 2 + (pc.starts ? 1 : 0);
-    mbar_wait_parked(o_full, n_piece & 1, p.status);     // and with it: every warp is past its last use of s_scale
-    if (sub == 0) {
-      s_scale[head] = whole ? 1.f / l_run : 1.f;
-      if (!whole) {
-        p.part_ml[(part * N + head) * 2] = m_ref;
-        p.part_ml[(part * N + head) * 2 + 1] = l_run;
-      }
-    }
-    named_barrier_sync(1, 128);
-    tcgen05_fence_after();
-    for (int m = 0; m < m_tiles; ++m) {
-      __syncwarp();
-      uint32_t hi[N], lo[N];
-      if constexpr (N == 16) {
-        tmem_ld_x16(tmem_o + lane_addr + m * 2 * N, hi);
-        tmem_ld_x16(tmem_o + lane_addr + m * 2 * N + N, lo);
-      } else {
-        tmem_ld_x32(tmem_o + lane_addr + m * 2 * N, hi);
-        tmem_ld_x32(tmem_o + lane_addr + m * 2 * N + N, lo);
-      }
-      tmem_ld_wait();
-      if (m + 1 == m_tiles) {                            // O is in registers: the next piece may begin
-        tcgen05_fence_before();
+      tcgen05_fence_after();
+      for (int m = 0; m < m_tiles; ++m) {
         __syncwarp();
-        if (lane == 0) mbar_arrive(o_empty);
-      }
-      const int d = m * 128 + key;
-      if (d >= p.R) continue;
+        uint32_t hi[N], lo[N];
+        if constexpr (N == 16) {
+          tmem_ld_x16(tmem_o + lane_addr + m * 2 * N, hi);
+          tmem_ld_x16(tmem_o + lane_addr + m * 2 * N + N, lo);
+        } else {
+          tmem_ld_x32(tmem_o + lane_addr + m * 2 * N, hi);
+          tmem_ld_x32(tmem_o + lane_addr + m * 2 * N + N, lo);
+        }
+        tmem_ld_wait();
+        if (m + 1 == m_tiles) {                            // O is in registers: the next piece may begin
+          tcgen05_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(o_empty);
+        }
+        const int d = m * 128 + key;
+        if (d >= p.R) continue;
 #pragma unroll
-      for (int h = 0; h < N; ++h) {
-        const float v = __uint_as_float(hi[h]) + __uint_as_float(lo[h]);
-        if (!whole) p.part_o[(part * N + h) * p.R + d] = v;
-        else if (h0 + h < p.heads) p.o[(static_cast<size_t>(pc.seq) * p.heads + h0 + h) * p.R + d] = __float2bfloat16_rn(v * s_scale[h]);
+        for (int h = 0; h < N; ++h) {
+          const float v = __uint_as_float(hi[h]) + __uint_as_float(lo[h]);
+          if (!whole) p.part_o[(part * N + h) * p.R + d] = v;
+          else if (h0 + h < p.heads) p.o[(static_cast<size_t>(pc.seq) * p.heads + h0 + h) * p.R + d] = __float2bfloat16_rn(v * s_scale[h]);
+        }
       }
-    }
-    named_barrier_sync(1, 128);                          // s_scale has been read
+      named_barrier_sync(1, 128);                          // s_scale has been read
     }
   }
 

@@ -153,6 +153,8 @@ class Worker:
                 stats = torch.cuda.memory_stats()
                 peak, cur = stats["allocated_bytes.all.peak"], stats["allocated_bytes.all.current"]
                 budget = int(total * cfg.gpu_memory_utilization) - (total - free) - (peak - cur) - self.num_slots * self.model.state_bytes()
+                # chunked prefill: a late portion of a long prompt sees more keys than the warm-up's whole prompts did
+                budget -= self.model.expansion_bytes(max(0, cfg.max_model_len - cfg.max_num_batched_tokens))
                 # a model whose layers are all recurrent pages nothing: the blocks then only bound the tokens of live requests
                 n = budget // block_bytes if block_bytes else cfg.max_num_seqs * self.table_width
                 if budget <= 0:

@@ -60,6 +60,11 @@ class LatentAttention:
     def bytes_per_sequence(self) -> int:
         return 0
 
+    def expansion_bytes(self) -> int:
+        """Workspace per key that a portion of a prompt sees."""
+        s = self.spec
+        return (s.heads * (s.dim + s.vdim) + s.kv_rank + s.rot_dim) * self.o.element_size()
+
     def new_memory(self, num_blocks: int, block_size: int, num_slots: int):
         return torch.zeros(num_blocks, block_size, self.spec.kv_rank + self.spec.rot_dim, dtype=self.o.dtype, device=self.o.device)
 
@@ -95,6 +100,9 @@ class Retention:
         pass
 
     def bytes_per_token(self) -> int:
+        return 0
+
+    def expansion_bytes(self) -> int:
         return 0
 
     def bytes_per_sequence(self) -> int:

@@ -92,6 +92,10 @@ class GoselixForCausalLM:
         """Recurrent state of one sequence."""
         return sum(self.layers[i].mix.bytes_per_sequence() for i, _ in self.runs)
 
+    def expansion_bytes(self, tokens: int) -> int:
+        """Largest workspace that ``tokens`` cached keys take when a portion of a prompt sees them (keys and values rebuilt per head)."""
+        return tokens * max((l.mix.expansion_bytes() for l in self.layers), default=0)
+
     def bind_cache(self, num_blocks: int, block_size: int, num_slots: int) -> None:
         """Every layer run (each pass of a looped layer) has a cache or state of its own; all share block and slot numbers."""
         self.memory = [self.layers[i].mix.new_memory(num_blocks, block_size, num_slots) for i, _ in self.runs]

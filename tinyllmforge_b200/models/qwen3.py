@@ -115,6 +115,9 @@ class Qwen3ForCausalLM:
         """Per-sequence state beside the paged cache: none."""
         return 0
 
+    def expansion_bytes(self, tokens: int) -> int:
+        return 0
+
     def bind_cache(self, num_blocks: int, block_size: int, num_slots: int = 0) -> None:
         self.bind_kv_cache(torch.zeros(len(self.layers), 2, num_blocks, self.num_kv_heads, block_size, self.head_dim, dtype=self.dtype,
                                        device=self.device))
