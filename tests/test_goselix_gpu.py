@@ -322,7 +322,8 @@ def test_retention_segments(ops, name):
 
 # ------------------------------------------------------------------------------------------------ experts
 @pytest.mark.parametrize("dtype,T,E,top,W,F", [(F32, 33, 5, 2, 50, 11), (BF, 33, 5, 2, 50, 11), (F32, 200, 3, 3, 64, 40), (BF, 1, 8, 1, 64, 32),
-                                               (BF, 3, 64, 4, 256, 96), (BF, 70, 16, 2, 512, 200), (BF, 500, 9, 4, 192, 136), (BF, 1500, 4, 3, 256, 320)])
+                                               (BF, 3, 64, 4, 256, 96), (BF, 70, 16, 2, 512, 200), (BF, 500, 9, 4, 192, 136), (BF, 1500, 4, 3, 256, 320), (BF, 1100, 20, 5, 96, 48), (BF, 1030, 64, 2, 160, 32),
+                                               (BF, 2100, 100, 2, 64, 16), (BF, 40, 200, 3, 64, 16), (BF, 20, 300, 2, 64, 16)])
 def test_experts(ops, dtype, T, E, top, W, F):
     h = rnd(T, W, seed=1, dtype=dtype)
     w = {"router": rnd(E, W, seed=2, scale=2 * W ** -0.5, dtype=dtype)}
