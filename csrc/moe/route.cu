@@ -254,7 +254,7 @@ constexpr int kPlanThreads = 1024;
 // One CTA.  smem: counts [E], next row [E].
 __global__ void __launch_bounds__(kPlanThreads) moe_plan_kernel(const int* __restrict__ experts, int n, int E, int tile, int max_tiles,
                                                                 int* __restrict__ pos, int* __restrict__ tile_expert,
-                                                                int* __restrict__ num_tiles) {
+                                                                int* __restrict__ num_tiles, unsigned* status) {
   extern __shared__ int sm_plan[];
   int* count = sm_plan;
   int* next = sm_plan + E;
@@ -262,7 +262,13 @@ __global__ void __launch_bounds__(kPlanThreads) moe_plan_kernel(const int* __res
   pdl_wait();
   for (int e = threadIdx.x; e < E; e += kPlanThreads) count[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < n; i += kPlanThreads) atomicAdd(&count[experts[i]], 1);
+  auto expert_of = [&](int i) {                   // an index out of range is reported and becomes expert 0
+    const int e = experts[i];
+    if (e >= 0 && e < E) return e;
+    set_status(status, kStatusBadIndex);
+    return 0;
+  };
+  for (int i = threadIdx.x; i < n; i += kPlanThreads) atomicAdd(&count[expert_of(i)], 1);
   __syncthreads();
   if (threadIdx.x < 32) {                         // running sum of tiles, 32 experts at a time
     int base = 0;
@@ -283,23 +289,24 @@ __global__ void __launch_bounds__(kPlanThreads) moe_plan_kernel(const int* __res
   for (int i = threadIdx.x; i < max_tiles; i += kPlanThreads) tile_expert[i] = -1;
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += kPlanThreads)
-    for (int k = 0; k < (count[e] + tile - 1) / tile; ++k) tile_expert[next[e] / tile + k] = e;
+    for (int k = 0; k < (count[e] + tile - 1) / tile && next[e] / tile + k < max_tiles; ++k) tile_expert[next[e] / tile + k] = e;
   __syncthreads();
-  for (int i = threadIdx.x; i < n; i += kPlanThreads) pos[i] = atomicAdd(&next[experts[i]], 1);
+  for (int i = threadIdx.x; i < n; i += kPlanThreads) pos[i] = atomicAdd(&next[expert_of(i)], 1);
 }
 
 // max_tiles >= n / tile + E rounded up: the caller's buffer has max_tiles * tile rows.
 extern "C" int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles,
-                              cudaStream_t stream) {
+                              unsigned* status, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (E > 4096 || tile < 1) return -1;
   return launch_kernel(moe_plan_kernel, dim3(1), dim3(kPlanThreads), static_cast<size_t>(E) * 8, stream, 0, experts, n, E, tile, max_tiles,
-                       pos, tile_expert, num_tiles) == cudaSuccess ? 0 : -2;
+                       pos, tile_expert, num_tiles, status) == cudaSuccess ? 0 : -2;
 }
 
 template <typename T, int N>
 __global__ void __launch_bounds__(256) moe_scatter_kernel(const T* __restrict__ h, const int* __restrict__ pos,
-                                                          const float* __restrict__ weights, int top, int W, T* __restrict__ xs) {
+                                                          const float* __restrict__ weights, int top, int W, T* __restrict__ xs,
+                                                          int xs_rows, unsigned* status) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
@@ -308,24 +315,29 @@ __global__ void __launch_bounds__(256) moe_scatter_kernel(const T* __restrict__ 
     load_n<N>(h + t * W + c, v);
     for (int j = 0; j < top; ++j) {
       const float s = weights[t * top + j];
+      const int row = pos[t * top + j];
+      if (row < 0 || row >= xs_rows) {
+        set_status(status, kStatusBadIndex);
+        continue;
+      }
       float x[N];
 #pragma unroll
       for (int e = 0; e < N; ++e) x[e] = s * v[e];
-      store_n<N>(xs + static_cast<size_t>(pos[t * top + j]) * W + c, x);
+      store_n<N>(xs + static_cast<size_t>(row) * W + c, x);
     }
   }
 }
 
-extern "C" int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs,
-                                 cudaStream_t stream) {
+extern "C" int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs, int xs_rows,
+                                 unsigned* status, cudaStream_t stream) {
   if (n <= 0) return 0;
   const bool v4 = (W & 3) == 0;
   if (fp32) {
     auto k = v4 ? moe_scatter_kernel<float, 4> : moe_scatter_kernel<float, 1>;
-    return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const float*>(h), pos, weights, top, W, static_cast<float*>(xs)) == cudaSuccess ? 0 : -2;
+    return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const float*>(h), pos, weights, top, W, static_cast<float*>(xs), xs_rows, status) == cudaSuccess ? 0 : -2;
   }
   auto k = v4 ? moe_scatter_kernel<bf16, 4> : moe_scatter_kernel<bf16, 1>;
-  return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const bf16*>(h), pos, weights, top, W, static_cast<bf16*>(xs)) == cudaSuccess ? 0 : -2;
+  return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const bf16*>(h), pos, weights, top, W, static_cast<bf16*>(xs), xs_rows, status) == cudaSuccess ? 0 : -2;
 }
 
 }  // namespace forge
