@@ -17,7 +17,7 @@ struct StreamArgs {
   const T* a;
   const T* b;
   const int* b_rows;     // null: b is [rows][W]; else b is indexed by b_rows[row * top + j], j < top
-  int top, b_n;          // b_n: rows of b
+  int top;
   const int* ids;
   const T* embed;
   int vocab;
@@ -29,7 +29,6 @@ struct StreamArgs {
   const int* rows;
   int n_rows, W, start;
   float eps;
-  unsigned* status;
 };
 
 template <typename T, int N>
@@ -71,12 +70,7 @@ __global__ void __launch_bounds__(256) stream_update_kernel(const StreamArgs<T> 
         for (int e = 0; e < N; ++e) s[e] += v[e];
       } else {
         for (int j = 0; j < p.top; ++j) {
-          const int row = p.b_rows[static_cast<size_t>(r) * p.top + j];
-          if (row < 0 || row >= p.b_n) {
-            set_status(p.status, kStatusBadIndex);
-            continue;
-          }
-          load_n<N>(p.b + static_cast<size_t>(row) * p.W + i, v);
+          load_n<N>(p.b + static_cast<size_t>(p.b_rows[static_cast<size_t>(r) * p.top + j]) * p.W + i, v);
 #pragma unroll
           for (int e = 0; e < N; ++e) s[e] += v[e];
         }
@@ -136,21 +130,21 @@ static int stream_update(int out_rows, const StreamArgs<T>& p, cudaStream_t stre
   return launch_kernel(k, dim3(out_rows), dim3(threads), smem, stream, 0, p) == cudaSuccess ? 0 : -2;
 }
 
-extern "C" int forge_stream_update(int fp32, float* x, const void* a, const void* b, const int* b_rows, int top, int b_n, const int* ids,
+extern "C" int forge_stream_update(int fp32, float* x, const void* a, const void* b, const int* b_rows, int top, const int* ids,
                                    const void* embed, int vocab, const void* vec, const void* w1, const void* w2, void* h1, void* h2,
-                                   const int* rows, int out_rows, int n_rows, int W, int start, float eps, unsigned* status, cudaStream_t stream) {
+                                   const int* rows, int out_rows, int n_rows, int W, int start, float eps, cudaStream_t stream) {
   if (out_rows <= 0) return 0;
   if (fp32) {
     using T = float;
-    const StreamArgs<T> p = {x, static_cast<const T*>(a), static_cast<const T*>(b), b_rows, top, b_n, ids, static_cast<const T*>(embed), vocab,
+    const StreamArgs<T> p = {x, static_cast<const T*>(a), static_cast<const T*>(b), b_rows, top, ids, static_cast<const T*>(embed), vocab,
                              static_cast<const T*>(vec), static_cast<const T*>(w1), static_cast<const T*>(w2), static_cast<T*>(h1),
-                             static_cast<T*>(h2), rows, n_rows, W, start, eps, status};
+                             static_cast<T*>(h2), rows, n_rows, W, start, eps};
     return stream_update<T>(out_rows, p, stream);
   }
   using T = bf16;
-  const StreamArgs<T> p = {x, static_cast<const T*>(a), static_cast<const T*>(b), b_rows, top, b_n, ids, static_cast<const T*>(embed), vocab,
+  const StreamArgs<T> p = {x, static_cast<const T*>(a), static_cast<const T*>(b), b_rows, top, ids, static_cast<const T*>(embed), vocab,
                            static_cast<const T*>(vec), static_cast<const T*>(w1), static_cast<const T*>(w2), static_cast<T*>(h1),
-                           static_cast<T*>(h2), rows, n_rows, W, start, eps, status};
+                           static_cast<T*>(h2), rows, n_rows, W, start, eps};
   return stream_update<T>(out_rows, p, stream);
 }
 

@@ -9,9 +9,9 @@
 #include <cstdint>
 
 extern "C" {
-int forge_stream_update(int fp32, float* x, const void* a, const void* b, const int* b_rows, int top, int b_n, const int* ids, const void* embed,
+int forge_stream_update(int fp32, float* x, const void* a, const void* b, const int* b_rows, int top, const int* ids, const void* embed,
                         int vocab, const void* vec, const void* w1, const void* w2, void* h1, void* h2, const int* rows, int out_rows,
-                        int n_rows, int W, int start, float eps, unsigned* status, cudaStream_t stream);
+                        int n_rows, int W, int start, float eps, cudaStream_t stream);
 int forge_silu_mul_any(int fp32, const void* x, void* out, long long rows, int I, cudaStream_t stream);
 int forge_gemm_simt(int fp32, const void* x, long long ldx, long long x_batch, const void* w, long long ldw, long long w_batch, void* out,
                     long long ldo, long long o_batch, int M, int N, int K, int batch, const int* tile_expert, cudaStream_t stream);
@@ -32,8 +32,7 @@ int forge_retention_scan(int fp32, const void* qkvg, int ld, const float* decay,
 int forge_retention_gate(int fp32, const float* o, const void* qkvg, int ld, int gate_at, void* y, int tok0, int tokens, int heads, int dv,
                          float eps, cudaStream_t stream);
 int forge_router(int fp32, const void* h, const void* w, int T, int W, int E, int top, int* experts, float* weights, cudaStream_t stream);
-int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles, unsigned* status,
-                   cudaStream_t stream);
+int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles, cudaStream_t stream);
 int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int n_out, int K, int gated, int tile, const int* tile_expert,
                        const int* num_tiles, int max_tiles, unsigned* status, cudaStream_t stream);
 int forge_head_linear(const void* x, long long x_tok, long long x_head, const void* w, void* out, long long o_tok, long long o_head, int M,
@@ -56,8 +55,7 @@ int forge_retention_chunk_cols(int dk, int dv);
 int forge_retention_chunk(void* qkvg, int ld, const float* decay, float* state, const int* slots, const int* positions, const float* rope,
                           int rope_rows, int rd, const int* cu, int seqs, int tok0, int tokens, int heads, int dk, int dv, int num_slots,
                           float* o, float* ws, int segs, int seg_len, unsigned* status, cudaStream_t stream);
-int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs, int xs_rows,
-                      unsigned* status, cudaStream_t stream);
+int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs, cudaStream_t stream);
 }
 
 namespace {
@@ -101,7 +99,7 @@ int i32(int64_t v) {
 // outputs whose rows b_rows[r, :] are summed.  rows (int32): norms of these rows only, x unchanged.
 void stream_update(Tensor& x, const OptTensor& a, const OptTensor& b, const OptTensor& b_rows, const OptTensor& ids, const OptTensor& embed,
                    const OptTensor& vec, const OptTensor& w1, const OptTensor& w2, const OptTensor& h1, const OptTensor& h2,
-                   const OptTensor& rows, bool start, double eps, bool fp32, const Tensor& status) {
+                   const OptTensor& rows, bool start, double eps, bool fp32) {
   TORCH_CHECK(x.dim() == 2, "stream_update: x must be [rows, width]");
   const int64_t R = x.size(0), W = x.size(1);
   const auto dt = fp32 ? at::kFloat : at::kBFloat16;
@@ -140,8 +138,8 @@ void stream_update(Tensor& x, const OptTensor& a, const OptTensor& b, const OptT
     h2p = data(*h2, dt, out_rows * W, "h2");
   }
   const c10::cuda::CUDAGuard guard(x.device());
-  check_rc(forge_stream_update(fp32, xp, ap, bp, brp, i32(top), brp != nullptr ? i32(b->size(0)) : 0, idp, ep, i32(vocab), vp, w1p, w2p, h1p, h2p, rp, i32(out_rows), i32(R), i32(W),
-                               start ? 1 : 0, static_cast<float>(eps), status_word(status), stream_of(x)),
+  check_rc(forge_stream_update(fp32, xp, ap, bp, brp, i32(top), idp, ep, i32(vocab), vp, w1p, w2p, h1p, h2p, rp, i32(out_rows), i32(R), i32(W),
+                               start ? 1 : 0, static_cast<float>(eps), stream_of(x)),
            "forge_stream_update");
 }
 
@@ -275,24 +273,24 @@ void router(const Tensor& h, const Tensor& w, Tensor& experts, Tensor& weights) 
            "forge_router");
 }
 
-void moe_plan(const Tensor& experts, int64_t E, int64_t tile, Tensor& pos, Tensor& tile_expert, Tensor& num_tiles, const Tensor& status) {
+void moe_plan(const Tensor& experts, int64_t E, int64_t tile, Tensor& pos, Tensor& tile_expert, Tensor& num_tiles) {
   const int64_t n = experts.numel();
   // an expert with c rows takes ceil(c / tile) tiles, at least one row each
   const int64_t worst = std::min(n, n / tile + E);
   const c10::cuda::CUDAGuard guard(experts.device());
   check_rc(forge_moe_plan(ints(experts, n, "experts"), i32(n), i32(E), i32(tile), i32(tile_expert.numel()),
                           const_cast<int*>(ints(pos, n, "pos")), const_cast<int*>(ints(tile_expert, worst, "tile_expert")),
-                          const_cast<int*>(ints(num_tiles, 1, "num_tiles")), status_word(status), stream_of(experts)),
+                          const_cast<int*>(ints(num_tiles, 1, "num_tiles")), stream_of(experts)),
            "forge_moe_plan");
 }
 
-void moe_scatter(const Tensor& h, const Tensor& pos, const Tensor& weights, Tensor& xs, const Tensor& status) {
+void moe_scatter(const Tensor& h, const Tensor& pos, const Tensor& weights, Tensor& xs) {
   const int f = elem(h);
   TORCH_CHECK(h.dim() == 2 && pos.dim() == 2 && pos.size(0) == h.size(0) && xs.dim() == 2 && xs.size(1) == h.size(1), "moe_scatter: shapes");
   const int64_t n = pos.numel();
   const c10::cuda::CUDAGuard guard(h.device());
   check_rc(forge_moe_scatter(f, data(h, h.scalar_type(), 0, "h"), ints(pos, n, "pos"), floats(weights, n, "weights"), i32(n), i32(pos.size(1)),
-                             i32(h.size(1)), data(xs, h.scalar_type(), 0, "xs"), i32(xs.size(0)), status_word(status), stream_of(h)),
+                             i32(h.size(1)), data(xs, h.scalar_type(), 0, "xs"), stream_of(h)),
            "forge_moe_scatter");
 }
 

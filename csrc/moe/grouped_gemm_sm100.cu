@@ -8,8 +8,7 @@
 //
 // Operands are swapped as in the decode GEMM: the UMMA's 128-row side is a tile of 128 weight rows and the rows of x ride
 // the N side, so a tile holds 16 to 128 of them and few tokens per expert waste no tensor work.  One CTA per SM walks the
-// output tiles in groups of 16 row tiles, row tiles fastest within a group: a group's rows of x (8 MB at width 2048) and the weights of
-// its one or two experts stay in L2 until all their features are done.  The TMA
+// (feature tile, row tile) pairs, row tiles fastest: CTAs that run at the same time share an expert's weight tiles in L2.  The TMA
 // ring does not drain between tiles, and tensor memory holds two accumulator sets, so the epilogue of a tile overlaps the
 // main loop of the next.  The number of row tiles in use and their experts are read on the device (no host round trip, a
 // captured graph serves every routing).
@@ -38,14 +37,6 @@ struct GroupedCfg {
   static constexpr int kSmemBytes = kStages * kStageBytes + 1024 + 256;
   static_assert(kTok % 16 == 0 && kTok <= 128 && 2 * kAccCols <= 512, "UMMA N and tensor memory");
 };
-
-// Output tile `tile` -> (feature tile, row tile).
-__device__ __forceinline__ void grouped_tile(int tile, int row_tiles, int feat_tiles, int& ft, int& rt) {
-  constexpr int kRows = 16;
-  const int group = tile / (kRows * feat_tiles), rem = tile - group * kRows * feat_tiles, rows = min(kRows, row_tiles - group * kRows);
-  ft = rem / rows;
-  rt = group * kRows + rem % rows;
-}
 
 template <int kTok, int kMode>
 __global__ void __launch_bounds__(kGThreads, 1)
@@ -98,9 +89,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
       uint32_t ph = 0;
       bool ok = true;
       for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
-        int ft, rt;
-        grouped_tile(tile, row_tiles, feat_tiles, ft, rt);
-        const int f0 = ft * Cfg::kTileFeat;
+        const int rt = tile % row_tiles, f0 = (tile / row_tiles) * Cfg::kTileFeat;
         const int wrow = max(tile_expert[rt], 0) * w_rows + f0;
         for (int kb = 0; kb < num_kb; ++kb) {
           if (!mbar_wait_parked(&empty_bar[s], ph ^ 1, status)) { ok = false; break; }
@@ -148,9 +137,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
     int n = 0;
     for (int tile = blockIdx.x; tile < total; tile += gridDim.x, ++n) {
       const int b = n & 1;
-      int ft, rt;
-      grouped_tile(tile, row_tiles, feat_tiles, ft, rt);
-      const int f = ft * Cfg::kTileFeat + quad * 32 + lane;
+      const int rt = tile % row_tiles, f = (tile / row_tiles) * Cfg::kTileFeat + quad * 32 + lane;
       if (!mbar_wait(&acc_full[b], (n >> 1) & 1, status)) break;
       tcgen05_fence_after();
       const uint32_t acc = tmem_base + lane_addr + b * Cfg::kAccCols;

@@ -100,98 +100,6 @@ __global__ void __launch_bounds__(256) router_mma_kernel(const bf16* __restrict_
   }
 }
 
-// The same for many tokens and at most 64 experts: CTA = 128 tokens, a warp owns 16 of them over the whole width; the router matrix
-// passes through shared memory, 128 columns at a time, so it is read once per 128 tokens.  A token's scores end up in the four
-// lanes of its row, which choose the experts among themselves.
-constexpr int kRtCols = 128, kRtPitch = kRtCols + 32;       // a row stride of 4 (mod 8) 16-byte units: conflict-free 16-byte reads
-
-template <int NB>
-__global__ void __launch_bounds__(256) router_tall_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w, int T, int W, int E, int top,
-                                                          int* __restrict__ experts, float* __restrict__ weights) {
-  __shared__ __align__(16) bf16 sw[2][NB * 8][kRtPitch];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
-  const int t0 = blockIdx.x * 128 + warp * 16;
-  auto load_w = [&](int c0, int st) {
-    for (int i = threadIdx.x; i < NB * 8 * (kRtCols / 8); i += 256) {
-      const int e = i / (kRtCols / 8), u = i % (kRtCols / 8);
-      const bool in = e < E && c0 + u * 8 < W;
-      cp_async16(smem_u32(&sw[st][e][u * 8]), in ? w + static_cast<size_t>(e) * W + c0 + u * 8 : w, in ? 16 : 0);
-    }
-    cp_async_commit();
-  };
-  pdl_launch_dependents();
-  load_w(0, 0);                                     // weights do not depend on the kernel before
-  pdl_wait();
-  const bf16* rows[2] = {h + static_cast<size_t>(min(t0 + g, T - 1)) * W + q * 8, h + static_cast<size_t>(min(t0 + 8 + g, T - 1)) * W + q * 8};
-  uint4 next[4][2];                                 // the tokens' columns of the next 128
-  auto load_h = [&](int c0) {
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) next[i][r] = c0 + i * 32 < W ? *reinterpret_cast<const uint4*>(rows[r] + c0 + i * 32) : make_uint4(0, 0, 0, 0);
-  };
-  load_h(0);
-  float acc[NB][4];
-#pragma unroll
-  for (int n = 0; n < NB; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-  int st = 0;
-  for (int c0 = 0; c0 < W; c0 += kRtCols, st ^= 1) {
-    cp_async_wait<0>();
-    __syncthreads();                                // the columns are here; everyone is done with the other stage
-    if (c0 + kRtCols < W) load_w(c0 + kRtCols, st ^ 1);
-    uint4 a[4][2];
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) a[i][r] = next[i][r];
-    if (c0 + kRtCols < W) load_h(c0 + kRtCols);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const uint32_t lo[4] = {a[i][0].x, a[i][1].x, a[i][0].y, a[i][1].y}, hi[4] = {a[i][0].z, a[i][1].z, a[i][0].w, a[i][1].w};
-#pragma unroll
-      for (int n = 0; n < NB; ++n) {
-        const uint4 b = *reinterpret_cast<const uint4*>(&sw[st][n * 8 + g][i * 32 + q * 8]);
-        mma16816(acc[n], lo, b.x, b.y);
-        mma16816(acc[n], hi, b.z, b.w);
-      }
-    }
-  }
-  // lane (g, q) holds the logits of tokens g and g + 8 for experts 8 n + 2 q, + 1
-#pragma unroll
-  for (int n = 0; n < NB; ++n)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) acc[n][e] = n * 8 + 2 * q + (e & 1) < E ? 1.f / (1.f + expf(-acc[n][e])) : -2.f;
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    const int t = t0 + r * 8 + g;
-    for (int j = 0; j < top; ++j) {
-      float best = -1.f;
-      int at = E;
-#pragma unroll
-      for (int n = 0; n < NB; ++n)
-#pragma unroll
-        for (int e = 0; e < 2; ++e)
-          if (acc[n][2 * r + e] > best) { best = acc[n][2 * r + e]; at = n * 8 + 2 * q + e; }
-#pragma unroll
-      for (int off = 1; off < 4; off <<= 1) {
-        const float v = __shfl_xor_sync(0xffffffffu, best, off);
-        const int i = __shfl_xor_sync(0xffffffffu, at, off);
-        if (v > best || (v == best && i < at)) { best = v; at = i; }
-      }
-      if (at >= E) at = 0;                          // only if every score is NaN
-#pragma unroll
-      for (int n = 0; n < NB; ++n)
-#pragma unroll
-        for (int e = 0; e < 2; ++e)
-          if (n * 8 + 2 * q + e == at) acc[n][2 * r + e] = -2.f;
-      if (q == 0 && t < T) {
-        experts[static_cast<size_t>(t) * top + j] = at;
-        weights[static_cast<size_t>(t) * top + j] = best;
-      }
-    }
-  }
-}
-
 // CTA = one token; one warp per expert at a time.
 template <typename T, int N>
 __global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, const T* __restrict__ w, int W, int E, int top,
@@ -230,10 +138,6 @@ extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int 
     return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
   }
   if (W % 32 == 0 && E <= 256 && (reinterpret_cast<uintptr_t>(h) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
-    if (T_ >= 1024 && E <= 64) {
-      auto k = E <= 16 ? router_tall_kernel<2> : E <= 32 ? router_tall_kernel<4> : router_tall_kernel<8>;
-      return launch_kernel(k, dim3((T_ + 127) / 128), dim3(256), 0, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
-    }
     const int Ep = (E + 7) & ~7;
     const bool two = T_ > 2048 && E <= 128;        // more tokens per CTA halve the reads of the router matrix
     const dim3 grid((T_ + (two ? 31 : 15)) / (two ? 32 : 16));
@@ -254,7 +158,7 @@ constexpr int kPlanThreads = 1024;
 // One CTA.  smem: counts [E], next row [E].
 __global__ void __launch_bounds__(kPlanThreads) moe_plan_kernel(const int* __restrict__ experts, int n, int E, int tile, int max_tiles,
                                                                 int* __restrict__ pos, int* __restrict__ tile_expert,
-                                                                int* __restrict__ num_tiles, unsigned* status) {
+                                                                int* __restrict__ num_tiles) {
   extern __shared__ int sm_plan[];
   int* count = sm_plan;
   int* next = sm_plan + E;
@@ -262,13 +166,7 @@ __global__ void __launch_bounds__(kPlanThreads) moe_plan_kernel(const int* __res
   pdl_wait();
   for (int e = threadIdx.x; e < E; e += kPlanThreads) count[e] = 0;
   __syncthreads();
-  auto expert_of = [&](int i) {                   // an index out of range is reported and becomes expert 0
-    const int e = experts[i];
-    if (e >= 0 && e < E) return e;
-    set_status(status, kStatusBadIndex);
-    return 0;
-  };
-  for (int i = threadIdx.x; i < n; i += kPlanThreads) atomicAdd(&count[expert_of(i)], 1);
+  for (int i = threadIdx.x; i < n; i += kPlanThreads) atomicAdd(&count[experts[i]], 1);
   __syncthreads();
   if (threadIdx.x < 32) {                         // running sum of tiles, 32 experts at a time
     int base = 0;
@@ -289,24 +187,23 @@ __global__ void __launch_bounds__(kPlanThreads) moe_plan_kernel(const int* __res
   for (int i = threadIdx.x; i < max_tiles; i += kPlanThreads) tile_expert[i] = -1;
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += kPlanThreads)
-    for (int k = 0; k < (count[e] + tile - 1) / tile && next[e] / tile + k < max_tiles; ++k) tile_expert[next[e] / tile + k] = e;
+    for (int k = 0; k < (count[e] + tile - 1) / tile; ++k) tile_expert[next[e] / tile + k] = e;
   __syncthreads();
-  for (int i = threadIdx.x; i < n; i += kPlanThreads) pos[i] = atomicAdd(&next[expert_of(i)], 1);
+  for (int i = threadIdx.x; i < n; i += kPlanThreads) pos[i] = atomicAdd(&next[experts[i]], 1);
 }
 
 // max_tiles >= n / tile + E rounded up: the caller's buffer has max_tiles * tile rows.
 extern "C" int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles,
-                              unsigned* status, cudaStream_t stream) {
+                              cudaStream_t stream) {
   if (n <= 0) return 0;
   if (E > 4096 || tile < 1) return -1;
   return launch_kernel(moe_plan_kernel, dim3(1), dim3(kPlanThreads), static_cast<size_t>(E) * 8, stream, 0, experts, n, E, tile, max_tiles,
-                       pos, tile_expert, num_tiles, status) == cudaSuccess ? 0 : -2;
+                       pos, tile_expert, num_tiles) == cudaSuccess ? 0 : -2;
 }
 
 template <typename T, int N>
 __global__ void __launch_bounds__(256) moe_scatter_kernel(const T* __restrict__ h, const int* __restrict__ pos,
-                                                          const float* __restrict__ weights, int top, int W, T* __restrict__ xs,
-                                                          int xs_rows, unsigned* status) {
+                                                          const float* __restrict__ weights, int top, int W, T* __restrict__ xs) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
@@ -315,29 +212,24 @@ __global__ void __launch_bounds__(256) moe_scatter_kernel(const T* __restrict__ 
     load_n<N>(h + t * W + c, v);
     for (int j = 0; j < top; ++j) {
       const float s = weights[t * top + j];
-      const int row = pos[t * top + j];
-      if (row < 0 || row >= xs_rows) {
-        set_status(status, kStatusBadIndex);
-        continue;
-      }
       float x[N];
 #pragma unroll
       for (int e = 0; e < N; ++e) x[e] = s * v[e];
-      store_n<N>(xs + static_cast<size_t>(row) * W + c, x);
+      store_n<N>(xs + static_cast<size_t>(pos[t * top + j]) * W + c, x);
     }
   }
 }
 
-extern "C" int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs, int xs_rows,
-                                 unsigned* status, cudaStream_t stream) {
+extern "C" int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weights, int n, int top, int W, void* xs,
+                                 cudaStream_t stream) {
   if (n <= 0) return 0;
   const bool v4 = (W & 3) == 0;
   if (fp32) {
     auto k = v4 ? moe_scatter_kernel<float, 4> : moe_scatter_kernel<float, 1>;
-    return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const float*>(h), pos, weights, top, W, static_cast<float*>(xs), xs_rows, status) == cudaSuccess ? 0 : -2;
+    return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const float*>(h), pos, weights, top, W, static_cast<float*>(xs)) == cudaSuccess ? 0 : -2;
   }
   auto k = v4 ? moe_scatter_kernel<bf16, 4> : moe_scatter_kernel<bf16, 1>;
-  return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const bf16*>(h), pos, weights, top, W, static_cast<bf16*>(xs), xs_rows, status) == cudaSuccess ? 0 : -2;
+  return launch_kernel(k, dim3(n / top), dim3(256), 0, stream, 0, static_cast<const bf16*>(h), pos, weights, top, W, static_cast<bf16*>(xs)) == cudaSuccess ? 0 : -2;
 }
 
 }  // namespace forge

@@ -26,7 +26,7 @@ class MixerOps:
         if isinstance(b, Routed):
             b, b_rows = b.y, b.rows
         self.C.stream_update(x, a, b, b_rows, ids, embed, vec, norms[0] if norms else None, norms[1] if len(norms) > 1 else None,
-                             outs[0] if outs else None, outs[1] if len(outs) > 1 else None, rows, start, eps, dtype == torch.float32, self.status)
+                             outs[0] if outs else None, outs[1] if len(outs) > 1 else None, rows, start, eps, dtype == torch.float32)
         return outs
 
     # ------------------------------------------------------------------ products outside the tcgen05 GEMMs' reach
@@ -155,9 +155,9 @@ class MixerOps:
         rows = torch.empty(T, top, dtype=torch.int32, device=h.device)
         tile_expert = torch.empty(tiles, dtype=torch.int32, device=h.device)
         num_tiles = torch.empty(1, dtype=torch.int32, device=h.device)
-        self.C.moe_plan(experts, E, tile, rows, tile_expert, num_tiles, self.status)
+        self.C.moe_plan(experts, E, tile, rows, tile_expert, num_tiles)
         xs = torch.empty(tiles * tile, W, dtype=h.dtype, device=h.device)
-        self.C.moe_scatter(h, rows, weights, xs, self.status)
+        self.C.moe_scatter(h, rows, weights, xs)
         y = torch.empty(tiles * tile, W, dtype=h.dtype, device=h.device)
         if fast:
             g = torch.empty(tiles * tile, down.shape[2], dtype=h.dtype, device=h.device)

@@ -93,11 +93,11 @@ def _experts(ops, T, part):
     rows = torch.empty(T, TOP, dtype=torch.int32, device="cuda")
     te, nt = torch.empty(tiles, dtype=torch.int32, device="cuda"), torch.empty(1, dtype=torch.int32, device="cuda")
     if part == "plan":
-        return lambda: ops.C.moe_plan(experts, EXPERTS, tile, rows, te, nt, ops.status), 3 * n * 4, 0
-    ops.C.moe_plan(experts, EXPERTS, tile, rows, te, nt, ops.status)
+        return lambda: ops.C.moe_plan(experts, EXPERTS, tile, rows, te, nt), 3 * n * 4, 0
+    ops.C.moe_plan(experts, EXPERTS, tile, rows, te, nt)
     xs = torch.zeros(tiles * tile, WIDTH, device="cuda", dtype=BF)
     if part == "scatter":
-        return lambda: ops.C.moe_scatter(h, rows, weights, xs, ops.status), (T + n) * WIDTH * 2, 0
+        return lambda: ops.C.moe_scatter(h, rows, weights, xs), (T + n) * WIDTH * 2, 0
     used = int((torch.bincount(experts.view(-1).long(), minlength=EXPERTS) > 0).sum())
     if part == "gate_up":
         w, out = _rand(EXPERTS, 2 * FF, WIDTH, scale=0.02), _rand(tiles * tile, FF)
