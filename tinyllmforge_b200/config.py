@@ -164,7 +164,7 @@ class Config:
     gpu_memory_utilization: float = 0.9
     tensor_parallel_size: int = 1
     enforce_eager: bool = False
-    hf_config: Optional[Any] = None          # a configuration class of models/registry.py (ModelConfig, GoselixConfig) or its dict
+    hf_config: Optional[Any] = None          # a configuration class of models/registry.py (ModelConfig, GoselixConfig, ...) or its dict
     eos: int = -1
     kvcache_block_size: int = 256
     num_kvcache_blocks: int = -1

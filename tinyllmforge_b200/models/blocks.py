@@ -118,10 +118,10 @@ class Retention:
 
 
 class GatedFeedForward:
-    """down(silu(gate h) * (up h))"""
+    """down(act(gate h) * (up h))"""
 
     def __init__(self, spec, width: int, dtype, device):
-        self.ff = spec.ff
+        self.ff, self.act = spec.ff, spec.act
         self.gate_up = _empty((2 * spec.ff, width), dtype, device)
         self.down = _empty((width, spec.ff), dtype, device)
 
@@ -131,11 +131,11 @@ class GatedFeedForward:
         yield p + "down", self.down
 
     def forward(self, ops, h):
-        return ops.linear(ops.linear_silu_mul(h, self.gate_up), self.down)
+        return ops.linear(ops.linear_act_mul(h, self.gate_up, self.act), self.down)
 
 
 class RoutedFeedForward:
-    """Experts chosen per token by the largest sigmoid scores; the score multiplies the expert's input."""
+    """Experts chosen per token; how their weights are made and applied is the spec's (see ``MoeSpec``)."""
 
     def __init__(self, spec, width: int, dtype, device):
         self.spec = spec
@@ -151,4 +151,5 @@ class RoutedFeedForward:
             yield f"{p}e{e}.down", self.down[e]
 
     def forward(self, ops, h):
-        return ops.moe(h, self.router, self.gate_up, self.down, self.spec.top)
+        s = self.spec
+        return ops.moe(h, self.router, self.gate_up, self.down, s.top, score=s.score, weigh=s.weigh, act=s.act, limit=s.limit)

@@ -7,35 +7,10 @@ checkpoint: a missing size is an error, an unknown key a warning.
 """
 from __future__ import annotations
 
-import warnings
 from dataclasses import dataclass
 
 from ..config import parse_dtype
-
-
-def _take(d: dict, what: str, keys: dict) -> dict:
-    """The values of ``keys`` (name -> converter) in ``d``."""
-    missing = [k for k in keys if k not in d]
-    if missing:
-        raise ValueError(f"{what}: missing {missing}")
-    extra = sorted(set(d) - set(keys))
-    if extra:
-        warnings.warn(f"{what}: keys not used by this model: {extra}")
-    return {k: conv(d[k]) for k, conv in keys.items()}
-
-
-@dataclass(frozen=True)
-class Rotation:
-    """Pairs (i, i + dims / 2) of the first ``dims`` entries of a head, angle = position * base ** (-2 i / dims)."""
-    base: float
-    dims: int
-
-    @classmethod
-    def from_dict(cls, d: dict) -> "Rotation":
-        r = cls(**_take(d, "rot", {"base": float, "dims": int}))
-        if r.dims < 0 or r.dims % 2:
-            raise ValueError("rot.dims must be even")
-        return r
+from .specs import DenseSpec, MoeSpec, Rotation, take
 
 
 @dataclass(frozen=True)
@@ -51,7 +26,7 @@ class LatentAttentionSpec:
 
     @classmethod
     def from_dict(cls, d: dict) -> "LatentAttentionSpec":
-        s = cls(**_take(d, "latent_attention", {"heads": int, "dim": int, "rot_dim": int, "vdim": int, "q_rank": int, "kv_rank": int,
+        s = cls(**take(d, "latent_attention", {"heads": int, "dim": int, "rot_dim": int, "vdim": int, "q_rank": int, "kv_rank": int,
                                                 "scale": float, "rot": Rotation.from_dict}))
         if s.rot.dims != s.rot_dim:
             raise ValueError("latent_attention: the whole rotated part is rotated (rot.dims == rot_dim)")
@@ -68,7 +43,7 @@ class RetentionSpec:
 
     @classmethod
     def from_dict(cls, d: dict) -> "RetentionSpec":
-        s = cls(**_take(d, "retention", {"heads": int, "dim": int, "vdim": int, "decay": lambda v: tuple(float(x) for x in v),
+        s = cls(**take(d, "retention", {"heads": int, "dim": int, "vdim": int, "decay": lambda v: tuple(float(x) for x in v),
                                          "rot": Rotation.from_dict}))
         if len(s.decay) != s.heads:
             raise ValueError("retention: one decay per head")
@@ -79,18 +54,6 @@ class RetentionSpec:
         return s
 
 
-@dataclass(frozen=True)
-class DenseSpec:
-    ff: int
-
-
-@dataclass(frozen=True)
-class MoeSpec:
-    experts: int
-    top: int
-    ff: int
-
-
 def _mlp_from_dict(d):
     if d is None:
         return None
@@ -98,11 +61,8 @@ def _mlp_from_dict(d):
     if kind == "dense":
         return DenseSpec(int(d["ff"]))
     if kind == "moe":
-        router = _take(d["router"], "mlp.router", {"experts": int, "top": int})
-        spec = MoeSpec(router["experts"], router["top"], int(d["expert"]["ff"]))
-        if not 1 <= spec.top <= spec.experts:
-            raise ValueError("mlp.router: top must lie between 1 and experts")
-        return spec
+        router = take(d["router"], "mlp.router", {"experts": int, "top": int})
+        return MoeSpec(router["experts"], router["top"], int(d["expert"]["ff"]))
     raise ValueError(f"unknown feed-forward kind {kind!r}; known: dense, moe")
 
 
@@ -150,7 +110,7 @@ class GoselixConfig:
                 raise ValueError(f"Goselix config: missing {key!r}")
         loop = d.get("loop")
         cfg = cls(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), tuple(LayerSpec.from_dict(l) for l in d["layers"]),
-                  LoopSpec(**_take(loop, "loop", {"start": int, "stop": int, "times": int})) if loop else None,
+                  LoopSpec(**take(loop, "loop", {"start": int, "stop": int, "times": int})) if loop else None,
                   torch_dtype=str(d.get("torch_dtype") or d.get("dtype") or "bfloat16").replace("torch.", ""))
         if d.get("eos_token_id") is not None:
             eos = d["eos_token_id"]

@@ -24,6 +24,8 @@ import numpy as np
 import torch
 import torch.nn.functional as F
 
+from . import ref_hybrid
+
 
 # ----------------------------------------------------------------------------- norms
 def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
@@ -78,6 +80,19 @@ def linear(x: torch.Tensor, w) -> torch.Tensor:
 
 def linear_silu_mul(x: torch.Tensor, w_gate_up) -> torch.Tensor:
     return silu_mul(linear(x, w_gate_up))
+
+
+# gate and up projections (fp32) and a limit -> the feed-forward's inner activation
+ACTIVATIONS = {
+    "silu": lambda g, u, limit: F.silu(g) * u,
+    "gelu_tanh": lambda g, u, limit: F.gelu(g, approximate="tanh") * u,
+    "clamped_swish": lambda g, u, limit: (gc := g.clamp(max=limit)) * torch.sigmoid(1.702 * gc) * (u.clamp(-limit, limit) + 1.0),
+}
+
+
+def linear_act_mul(x: torch.Tensor, w_gate_up, act: str, limit: float = 0.0) -> torch.Tensor:
+    g, u = linear(x, w_gate_up).float().chunk(2, dim=-1)
+    return ACTIVATIONS[act](g, u, limit).to(x.dtype)
 
 
 # ----------------------------------------------------------------------------- KV cache
@@ -151,14 +166,21 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_
 
 
 # ----------------------------------------------------------------------------- 32-bit residual stream
-def stream_update(x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None):
+def stream_update(x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None,
+                  a_bias=None, post=None, mult=1.0, offset=0.0):
     """The residual stream between two layers: x += a + b (the two branches of a parallel layer), += embed[ids], += vec,
     all in fp32; then one RMS norm per weight in ``norms``, each rounded once to ``dtype``.  ``start``: x begins at zero.
-    ``rows``: norms of these rows only, and x is left as it was."""
+    ``rows``: norms of these rows only, and x is left as it was.  ``a_bias`` is added to a.  ``post``: a is normed with this
+    weight and multiplied by ``mult`` on its way into x.  ``offset`` is added to every norm weight (weights stored around zero)."""
+    def norm(v, w):
+        return v * torch.rsqrt(v.pow(2).mean(dim=-1, keepdim=True) + eps) * (w.float() + offset)
+
     s = torch.zeros_like(x) if start else x
-    for term in (a, b):
-        if term is not None:
-            s = s + term.float()
+    if a is not None:
+        a = a.float() if a_bias is None else a.float() + a_bias
+        s = s + (a if post is None else mult * norm(a, post))
+    if b is not None:
+        s = s + b.float()
     if ids is not None:
         s = s + F.embedding(ids.long(), embed).float()
     if vec is not None:
@@ -167,8 +189,7 @@ def stream_update(x, dtype, eps, norms, start=False, a=None, b=None, ids=None, e
         x.copy_(s)
     else:
         s = s[rows.long()]
-    inv = torch.rsqrt(s.pow(2).mean(dim=-1, keepdim=True) + eps)
-    return [(s * inv * w.float()).to(dtype) for w in norms]
+    return [norm(s, w).to(dtype) for w in norms]
 
 
 def apply_partial_rope(x: torch.Tensor, positions: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
@@ -243,17 +264,19 @@ def retention(qkvg, decay, state, batch, table, spec, eps):
 
 
 # ----------------------------------------------------------------------------- mixture of experts
-def moe(h, router, gate_up, down, top):
-    """Sigmoid-scored top-k experts; the score multiplies the expert's INPUT.  gate_up [experts, 2 ff, width], down [experts,
-    width, ff]."""
-    score = torch.sigmoid(h.float() @ router.float().t())
-    w, e = torch.sort(score, dim=-1, descending=True, stable=True)
+def moe(h, router, gate_up, down, top, score="sigmoid", weigh="input", act="silu", limit=0.0):
+    """Top-k experts.  ``score``: sigmoid of each logit, or softmax over the chosen logits; ``weigh``: the score multiplies the
+    expert's input or its output.  gate_up [experts, 2 ff, width], down [experts, width, ff]."""
+    z, e = torch.sort(h.float() @ router.float().t(), dim=-1, descending=True, stable=True)
+    w = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z[:, :top], dim=-1)
     out = torch.zeros(h.shape[0], down.shape[1], device=h.device)
     for j in range(top):
         for x in e[:, j].unique().tolist():
             rows = (e[:, j] == x).nonzero()[:, 0]
-            hx = (h[rows].float() * w[rows, j, None]).to(h.dtype)
-            out[rows] += linear(linear_silu_mul(hx, gate_up[x]), down[x]).float()
+            hx, wx = h[rows], w[rows, j, None]
+            if weigh == "input":
+                hx, wx = (hx.float() * wx).to(h.dtype), 1.0
+            out[rows] += wx * linear(linear_act_mul(hx, gate_up[x], act, limit), down[x]).float()
     return out
 
 
@@ -361,13 +384,14 @@ def sample(logits: torch.Tensor, temperatures: torch.Tensor, seed: int, step: in
 
 
 # ----------------------------------------------------------------------------- op set
-class RefOps:
+class RefOps(ref_hybrid.RefHybridOps):
     """The op set the model calls, stated with the functions above (CPU path and oracle)."""
 
     name = "ref"
 
     linear = staticmethod(linear)
     linear_silu_mul = staticmethod(linear_silu_mul)
+    linear_act_mul = staticmethod(linear_act_mul)
     embedding = staticmethod(embedding)
     add_rms_norm = staticmethod(add_rms_norm)
     rms_norm = staticmethod(rms_norm)
