@@ -66,6 +66,8 @@ struct GemmFuse {
   float* out_ssq;
   int out_parts;
   int w_dynamic;      // weight-tile kernel only: W was written by the kernel launched just before, do not prefetch it early
+  int act;            // gated epilogue: GateAct and its limit
+  float limit;
 };
 
 __device__ __forceinline__ float fuse_row_scale(const GemmFuse& f, int row, int rows) {
@@ -316,7 +318,7 @@ __device__ __forceinline__ void tile_epilogue(uint32_t tacc, bool whole, const S
 #pragma unroll
     for (int j = 0; j < kChunk; ++j) {
       f[j] = __uint_as_float(v[j]) * row_scale;
-      if constexpr (kEpi == kEpiSiluMul) f[j] = silu(f[j]) * (__uint_as_float(u[j]) * row_scale);
+      if constexpr (kEpi == kEpiSiluMul) f[j] = gated_act<false>(fuse.act, fuse.limit, f[j], __uint_as_float(u[j]) * row_scale);
     }
     const int c = c0 + cc;
     if (r < m_total) {
@@ -981,8 +983,10 @@ __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const SplitKFin
       float4 f;
       f.x = acc[0] * row_scale; f.y = acc[1] * row_scale; f.z = acc[2] * row_scale; f.w = acc[3] * row_scale;
       if constexpr (kEpi == kEpiSiluMul) {
-        f.x = silu(f.x) * (up[0] * row_scale); f.y = silu(f.y) * (up[1] * row_scale);
-        f.z = silu(f.z) * (up[2] * row_scale); f.w = silu(f.w) * (up[3] * row_scale);
+        f.x = gated_act<false>(fuse.act, fuse.limit, f.x, up[0] * row_scale);
+        f.y = gated_act<false>(fuse.act, fuse.limit, f.y, up[1] * row_scale);
+        f.z = gated_act<false>(fuse.act, fuse.limit, f.z, up[2] * row_scale);
+        f.w = gated_act<false>(fuse.act, fuse.limit, f.w, up[3] * row_scale);
       }
       *reinterpret_cast<float4*>(&s_val[lane][cg * 4]) = f;
     }
@@ -1222,7 +1226,7 @@ gemm_weights_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_const
 #pragma unroll
               for (int j = 0; j < kChunk; ++j) {
                 const float sc = fuse_io.in_ssq != nullptr ? col_scale[cc + j] : 1.f;     // column = token
-                v[j] = __float_as_uint(silu(__uint_as_float(v[j]) * sc) * (__uint_as_float(u[j]) * sc));
+                v[j] = __float_as_uint(gated_act<false>(fuse_io.act, fuse_io.limit, __uint_as_float(v[j]) * sc, __uint_as_float(u[j]) * sc));
               }
             }
           }
@@ -1285,8 +1289,10 @@ gemm_weights_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_const
                   continue;
                 }
                 const float4 gv = *g;
-                v.x = silu(gv.x * sc) * (v.x * sc); v.y = silu(gv.y * sc) * (v.y * sc);
-                v.z = silu(gv.z * sc) * (v.z * sc); v.w = silu(gv.w * sc) * (v.w * sc);
+                v.x = gated_act<false>(fuse_io.act, fuse_io.limit, gv.x * sc, v.x * sc);
+                v.y = gated_act<false>(fuse_io.act, fuse_io.limit, gv.y * sc, v.y * sc);
+                v.z = gated_act<false>(fuse_io.act, fuse_io.limit, gv.z * sc, v.z * sc);
+                v.w = gated_act<false>(fuse_io.act, fuse_io.limit, gv.w * sc, v.w * sc);
               }
             } else {
               v.x *= sc; v.y *= sc; v.z *= sc; v.w *= sc;
@@ -1748,6 +1754,16 @@ extern "C" int forge_gemm_bf16(const void* x, int ldx, const void* w, int ldw, v
                                int K, int epi, int force_mode, int tune, unsigned* status, cudaStream_t stream) {
   TpPush none = {};
   return gemm_dispatch(x, ldx, w, ldw, out, ldo, M, n_out, K, epi, force_mode, tune, status, stream, none);
+}
+
+// The gated epilogue (epi = 1) with another activation (GateAct) than silu.
+extern "C" int forge_gemm_bf16_act(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int n_out, int K, int act,
+                                   float limit, unsigned* status, cudaStream_t stream) {
+  TpPush none = {};
+  GemmFuse fuse = {};
+  fuse.act = act;
+  fuse.limit = limit;
+  return gemm_dispatch(x, ldx, w, ldw, out, ldo, M, n_out, K, kEpiSiluMul, 0, 0, status, stream, none, fuse);
 }
 
 // Row-parallel GEMM under tensor parallelism: `out` is this rank's partial buffer in symmetric memory (row stride ldo);

@@ -667,11 +667,13 @@ void tp_sample_pairs(const Tensor& vals, const Tensor& ids, int64_t tp_rank, con
 
 }  // namespace
 
-void register_mixers(pybind11::module& m);      // bindings_mixers.cpp
+void register_mixers(pybind11::module& m);
+void register_hybrid(pybind11::module& m);      // bindings_mixers.cpp
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.doc() = "tinyllmforge_b200 sm_100a kernels";
   register_mixers(m);
+  register_hybrid(m);
   m.def("gemm", &gemm);
   m.def("gemm_fused", &gemm_fused);
   m.def("gemm_sample", &gemm_sample);

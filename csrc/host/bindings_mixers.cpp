@@ -8,11 +8,18 @@
 #include <algorithm>
 #include <cstdint>
 
+#include "checks.h"
+
 extern "C" {
 int forge_stream_update(int fp32, float* x, const void* a, const void* b, const int* b_rows, int top, const int* ids, const void* embed,
                         int vocab, const void* vec, const void* w1, const void* w2, void* h1, void* h2, const int* rows, int out_rows,
                         int n_rows, int W, int start, float eps, cudaStream_t stream);
-int forge_silu_mul_any(int fp32, const void* x, void* out, long long rows, int I, cudaStream_t stream);
+int forge_stream_sandwich(int fp32, float* x, const void* a, const int* a_rows, const float* a_weights, int top, const float* a_bias,
+                          const void* post, float mult, float offset, const int* ids, const void* embed, int vocab, const void* w, void* h,
+                          const int* rows, int out_rows, int n_rows, int W, int start, float eps, cudaStream_t stream);
+int forge_act_mul_any(int fp32, const void* x, void* out, long long rows, int I, int act, float limit, cudaStream_t stream);
+int forge_gemm_bf16_act(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int n_out, int K, int act, float limit,
+                        unsigned* status, cudaStream_t stream);
 int forge_gemm_simt(int fp32, const void* x, long long ldx, long long x_batch, const void* w, long long ldw, long long w_batch, void* out,
                     long long ldo, long long o_batch, int M, int N, int K, int batch, const int* tile_expert, cudaStream_t stream);
 int forge_latent_prepare(int fp32, const void* proj, int T, int q_rank, int kv_rank, int rot, const void* qw, const void* kw, float eps,
@@ -31,10 +38,11 @@ int forge_retention_scan(int fp32, const void* qkvg, int ld, const float* decay,
                          float* o, unsigned* status, cudaStream_t stream);
 int forge_retention_gate(int fp32, const float* o, const void* qkvg, int ld, int gate_at, void* y, int tok0, int tokens, int heads, int dv,
                          float eps, cudaStream_t stream);
-int forge_router(int fp32, const void* h, const void* w, int T, int W, int E, int top, int* experts, float* weights, cudaStream_t stream);
+int forge_router(int fp32, const void* h, const void* w, int T, int W, int E, int top, int softmax, int* experts, float* weights,
+                 cudaStream_t stream);
 int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles, cudaStream_t stream);
-int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int n_out, int K, int gated, int tile, const int* tile_expert,
-                       const int* num_tiles, int max_tiles, unsigned* status, cudaStream_t stream);
+int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int n_out, int K, int gated, int tile, int act, float limit,
+                       const int* tile_expert, const int* num_tiles, int max_tiles, unsigned* status, cudaStream_t stream);
 int forge_head_linear(const void* x, long long x_tok, long long x_head, const void* w, void* out, long long o_tok, long long o_head, int M,
                       int heads, int N, int K, cudaStream_t stream);
 int forge_latent_decode_ok(int R, int rot, int block_size);
@@ -59,41 +67,6 @@ int forge_moe_scatter(int fp32, const void* h, const int* pos, const float* weig
 }
 
 namespace {
-
-using torch::Tensor;
-using OptTensor = c10::optional<Tensor>;
-
-void check_rc(int rc, const char* what) { TORCH_CHECK(rc == 0, what, " failed with code ", rc); }
-cudaStream_t stream_of(const Tensor& t) { return at::cuda::getCurrentCUDAStream(t.get_device()).stream(); }
-unsigned* status_word(const Tensor& status) {
-  TORCH_CHECK(status.is_cuda() && status.scalar_type() == at::kInt && status.numel() >= 1, "status must be a CUDA int32 tensor");
-  return reinterpret_cast<unsigned*>(status.data_ptr<int>());
-}
-// 1: fp32, 0: bf16
-int elem(const Tensor& t) {
-  TORCH_CHECK(t.scalar_type() == at::kFloat || t.scalar_type() == at::kBFloat16, "element type must be bfloat16 or float32");
-  return t.scalar_type() == at::kFloat ? 1 : 0;
-}
-void need(const Tensor& t, at::ScalarType dtype, int64_t min_numel, const char* what) {
-  TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.scalar_type() == dtype, what, ": contiguous CUDA tensor of the right type expected");
-  TORCH_CHECK(t.numel() >= min_numel, what, ": too few elements (", t.numel(), " of ", min_numel, ")");
-}
-const int* ints(const Tensor& t, int64_t n, const char* what) {
-  need(t, at::kInt, n, what);
-  return t.data_ptr<int>();
-}
-float* floats(const Tensor& t, int64_t n, const char* what) {
-  need(t, at::kFloat, n, what);
-  return t.data_ptr<float>();
-}
-void* data(const Tensor& t, at::ScalarType dtype, int64_t n, const char* what) {
-  need(t, dtype, n, what);
-  return t.data_ptr();
-}
-int i32(int64_t v) {
-  TORCH_CHECK(v >= INT32_MIN && v <= INT32_MAX, "value does not fit 32 bits");
-  return static_cast<int>(v);
-}
 
 // x fp32 [rows, W]; a, b, embed, vec, w1, w2, h1, h2 of one element type.  b_rows (int32 [rows, top]): b is a buffer of expert
 // outputs whose rows b_rows[r, :] are summed.  rows (int32): norms of these rows only, x unchanged.
@@ -143,13 +116,74 @@ void stream_update(Tensor& x, const OptTensor& a, const OptTensor& b, const OptT
            "forge_stream_update");
 }
 
-void silu_mul_any(const Tensor& x, Tensor& out) {
+// x fp32 [rows, W]; a, post, embed, w, h of one element type.  a_rows (int32 [rows, top]) with a_weights (fp32, or none: 1): a is
+// a buffer of expert outputs.  rows (int32): these rows only, x unchanged.
+void stream_sandwich(Tensor& x, const OptTensor& a, const OptTensor& a_rows, const OptTensor& a_weights, const OptTensor& a_bias,
+                     const OptTensor& post, double mult, double offset, const OptTensor& ids, const OptTensor& embed, const OptTensor& w,
+                     const OptTensor& h, const OptTensor& rows, bool start, double eps, bool fp32) {
+  TORCH_CHECK(x.dim() == 2, "stream_sandwich: x must be [rows, width]");
+  const int64_t R = x.size(0), W = x.size(1);
+  const auto dt = fp32 ? at::kFloat : at::kBFloat16;
+  float* xp = floats(x, R * W, "x");
+  const void *ap = nullptr, *pp = nullptr, *ep = nullptr, *wp = nullptr;
+  void* hp = nullptr;
+  const int *arp = nullptr, *idp = nullptr, *rp = nullptr;
+  const float *awp = nullptr, *abp = nullptr;
+  int64_t top = 0, vocab = 0, out_rows = R;
+  if (rows.has_value()) { rp = ints(*rows, 0, "rows"); out_rows = rows->numel(); }
+  if (a.has_value()) {
+    if (a_rows.has_value()) {
+      TORCH_CHECK(a_rows->dim() == 2 && a_rows->size(0) == R && a->dim() == 2 && a->size(1) == W, "stream_sandwich: routed a");
+      top = a_rows->size(1);
+      arp = ints(*a_rows, R * top, "a_rows");
+      ap = data(*a, dt, W, "a");
+      if (a_weights.has_value()) awp = floats(*a_weights, R * top, "a_weights");
+    } else {
+      ap = data(*a, dt, R * W, "a");
+    }
+    if (a_bias.has_value()) abp = floats(*a_bias, W, "a_bias");
+  }
+  if (post.has_value()) {
+    TORCH_CHECK(a.has_value(), "stream_sandwich: post belongs to a");
+    pp = data(*post, dt, W, "post");
+  }
+  if (ids.has_value()) {
+    TORCH_CHECK(embed.has_value() && embed->dim() == 2 && embed->size(1) == W, "stream_sandwich: embed");
+    idp = ints(*ids, R, "ids");
+    vocab = embed->size(0);
+    ep = data(*embed, dt, W, "embed");
+  }
+  if (w.has_value()) {
+    TORCH_CHECK(h.has_value(), "stream_sandwich: h");
+    wp = data(*w, dt, W, "w");
+    hp = data(*h, dt, out_rows * W, "h");
+  }
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_stream_sandwich(fp32, xp, ap, arp, awp, i32(top), abp, pp, static_cast<float>(mult), static_cast<float>(offset), idp, ep,
+                                 i32(vocab), wp, hp, rp, i32(out_rows), i32(R), i32(W), start ? 1 : 0, static_cast<float>(eps), stream_of(x)),
+           "forge_stream_sandwich");
+}
+
+// out = act(x w_gate^T, x w_up^T) for w = gate rows, up rows (bf16, tcgen05)
+void gemm_act(const Tensor& x, const Tensor& w, Tensor& out, int64_t act, double limit, const Tensor& status) {
+  TORCH_CHECK(x.is_cuda() && w.is_cuda() && out.is_cuda() && x.scalar_type() == at::kBFloat16 && w.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16,
+              "gemm_act: bf16 CUDA tensors expected");
+  TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && out.dim() == 2 && x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1, "gemm_act: ranks and strides");
+  TORCH_CHECK(w.size(1) == x.size(1) && w.size(0) % 2 == 0 && out.size(0) == x.size(0) && out.size(1) == w.size(0) / 2 && act >= 0 && act <= 2, "gemm_act: shapes");
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_gemm_bf16_act(x.data_ptr(), i32(x.stride(0)), w.data_ptr(), i32(w.stride(0)), out.data_ptr(), i32(out.stride(0)), i32(x.size(0)),
+                               i32(out.size(1)), i32(x.size(1)), i32(act), static_cast<float>(limit), status_word(status), stream_of(x)),
+           "forge_gemm_bf16_act");
+}
+
+void act_mul_any(const Tensor& x, Tensor& out, int64_t act, double limit) {
   const int f = elem(x);
-  TORCH_CHECK(x.dim() == 2 && x.size(1) % 2 == 0, "silu_mul_any: x [rows, 2 I]");
+  TORCH_CHECK(x.dim() == 2 && x.size(1) % 2 == 0, "act_mul_any: x [rows, 2 I]");
   const int64_t rows = x.size(0), I = x.size(1) / 2;
   const c10::cuda::CUDAGuard guard(x.device());
-  check_rc(forge_silu_mul_any(f, data(x, x.scalar_type(), rows * 2 * I, "x"), data(out, x.scalar_type(), rows * I, "out"), rows, i32(I), stream_of(x)),
-           "forge_silu_mul_any");
+  check_rc(forge_act_mul_any(f, data(x, x.scalar_type(), rows * 2 * I, "x"), data(out, x.scalar_type(), rows * I, "out"), rows, i32(I), i32(act),
+                             static_cast<float>(limit), stream_of(x)),
+           "forge_act_mul_any");
 }
 
 // out[b] = x[b] w[b]^T for 3-D views [batch, M, K], [batch, N, K], [batch, M, N] with unit inner strides (2-D: one product).
@@ -263,12 +297,12 @@ void retention_gate(const Tensor& o, const Tensor& qkvg, Tensor& y, int64_t tok0
            "forge_retention_gate");
 }
 
-void router(const Tensor& h, const Tensor& w, Tensor& experts, Tensor& weights) {
+void router(const Tensor& h, const Tensor& w, Tensor& experts, Tensor& weights, bool softmax) {
   const int f = elem(h);
   TORCH_CHECK(h.dim() == 2 && w.dim() == 2 && w.size(1) == h.size(1) && experts.dim() == 2 && experts.size(0) == h.size(0), "router: shapes");
   const int64_t T = h.size(0), W = h.size(1), E = w.size(0), top = experts.size(1);
   const c10::cuda::CUDAGuard guard(h.device());
-  check_rc(forge_router(f, data(h, h.scalar_type(), 0, "h"), data(w, h.scalar_type(), 0, "w"), i32(T), i32(W), i32(E), i32(top),
+  check_rc(forge_router(f, data(h, h.scalar_type(), 0, "h"), data(w, h.scalar_type(), 0, "w"), i32(T), i32(W), i32(E), i32(top), softmax ? 1 : 0,
                         const_cast<int*>(ints(experts, T * top, "experts")), floats(weights, T * top, "weights"), stream_of(h)),
            "forge_router");
 }
@@ -284,12 +318,12 @@ void moe_plan(const Tensor& experts, int64_t E, int64_t tile, Tensor& pos, Tenso
            "forge_moe_plan");
 }
 
-void moe_scatter(const Tensor& h, const Tensor& pos, const Tensor& weights, Tensor& xs) {
+void moe_scatter(const Tensor& h, const Tensor& pos, const OptTensor& weights, Tensor& xs) {
   const int f = elem(h);
   TORCH_CHECK(h.dim() == 2 && pos.dim() == 2 && pos.size(0) == h.size(0) && xs.dim() == 2 && xs.size(1) == h.size(1), "moe_scatter: shapes");
   const int64_t n = pos.numel();
   const c10::cuda::CUDAGuard guard(h.device());
-  check_rc(forge_moe_scatter(f, data(h, h.scalar_type(), 0, "h"), ints(pos, n, "pos"), floats(weights, n, "weights"), i32(n), i32(pos.size(1)),
+  check_rc(forge_moe_scatter(f, data(h, h.scalar_type(), 0, "h"), ints(pos, n, "pos"), weights.has_value() ? floats(*weights, n, "weights") : nullptr, i32(n), i32(pos.size(1)),
                              i32(h.size(1)), data(xs, h.scalar_type(), 0, "xs"), stream_of(h)),
            "forge_moe_scatter");
 }
@@ -298,13 +332,13 @@ void moe_scatter(const Tensor& h, const Tensor& pos, const Tensor& weights, Tens
 constexpr auto kBf16 = at::kBFloat16;
 
 void grouped_gemm(const Tensor& x, const Tensor& w, Tensor& out, bool gated, int64_t tile, const Tensor& tile_expert, const Tensor& num_tiles,
-                  const Tensor& status) {
+                  int64_t act, double limit, const Tensor& status) {
   TORCH_CHECK(x.dim() == 2 && w.dim() == 3 && out.dim() == 2 && w.size(2) == x.size(1), "grouped_gemm: ranks");
   const int64_t rows = x.size(0), K = x.size(1), N = gated ? w.size(1) / 2 : w.size(1), tiles = tile_expert.numel();
   TORCH_CHECK(rows == tiles * tile && out.size(0) == rows && out.size(1) == N, "grouped_gemm: shapes");
   const c10::cuda::CUDAGuard guard(x.device());
   check_rc(forge_grouped_gemm(data(x, kBf16, 0, "x"), data(w, kBf16, 0, "w"), data(out, kBf16, 0, "out"), i32(w.size(0)), i32(N), i32(K),
-                              gated ? 1 : 0, i32(tile), ints(tile_expert, 0, "tile_expert"), ints(num_tiles, 1, "num_tiles"), i32(tiles),
+                              gated ? 1 : 0, i32(tile), i32(act), static_cast<float>(limit), ints(tile_expert, 0, "tile_expert"), ints(num_tiles, 1, "num_tiles"), i32(tiles),
                               status_word(status), stream_of(x)),
            "forge_grouped_gemm");
 }
@@ -398,7 +432,9 @@ void retention_chunk(Tensor& qkvg, const Tensor& decay, Tensor& state, const Ten
 
 void register_mixers(pybind11::module& m) {
   m.def("stream_update", &stream_update);
-  m.def("silu_mul_any", &silu_mul_any);
+  m.def("stream_sandwich", &stream_sandwich);
+  m.def("gemm_act", &gemm_act);
+  m.def("act_mul_any", &act_mul_any);
   m.def("gemm_simt", &gemm_simt);
   m.def("latent_prepare", &latent_prepare);
   m.def("latent_rotate_q", &latent_rotate_q);

@@ -363,4 +363,23 @@ __device__ __forceinline__ float bf16_hi(uint32_t v) { return __uint_as_float(v 
 // measured 13 -> 20 us on a 256 x 6144 x 1024 GEMM epilogue whose accumulators were zero.
 __device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 
+// The inner activation of a gated feed-forward from its gate and up projections.
+//   silu            g sigmoid(g) u
+//   gelu_tanh       gelu(g) u; 0.5 (1 + tanh(y)) is sigmoid(2 y)
+//   clamped_swish   g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+enum GateAct { kActSilu = 0, kActGeluTanh = 1, kActClampedSwish = 2 };
+
+// z sigmoid(y); accurate: fp32 models.
+template <bool kAccurate>
+__device__ __forceinline__ float times_sigmoid(float z, float y) {
+  return kAccurate ? z / (1.f + expf(-y)) : __fdividef(z, 1.0f + __expf(-y));
+}
+template <bool kAccurate>
+__device__ __forceinline__ float gated_act(int act, float limit, float g, float u) {
+  if (act == kActSilu) return times_sigmoid<kAccurate>(g, g) * u;
+  if (act == kActGeluTanh) return times_sigmoid<kAccurate>(g, 1.5957691216057308f * (g + 0.044715f * g * g * g)) * u;
+  g = fminf(g, limit);
+  return times_sigmoid<kAccurate>(g, 1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+}
+
 }  // namespace forge

@@ -67,6 +67,15 @@ __device__ __forceinline__ float silu_t(float x) {
   else return silu(x);
 }
 
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) {
+  if constexpr (sizeof(T) == 4) return 1.f / (1.f + expf(-x));
+  else return __fdividef(1.f, 1.f + __expf(-x));
+}
+
+// log(1 + e^x) without overflow.
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
 // x = hi + lo with both halves in bf16 (|x - hi - lo| <= 2^-17 |x|): an fp32 factor as two tensor-core operands.
 __device__ __forceinline__ void split_bf16(float x, float& hi, float& lo) {
   hi = __bfloat162float(__float2bfloat16_rn(x));

@@ -1,7 +1,7 @@
 // Expert GEMM on the 5th-generation tensor cores: rows sorted by expert (moe_plan), every tile of kTok rows has one expert.
 //
 //   plain   y[r, f]  = x[r, :] . w[e, f, :]                               (down)
-//   gated   y[r, f]  = silu(x[r, :] . w[e, f, :]) * (x[r, :] . w[e, F + f, :])   (gate and up rows of one packed matrix)
+//   gated   y[r, f]  = act(x[r, :] . w[e, f, :], x[r, :] . w[e, F + f, :])       (gate and up rows of one packed matrix; GateAct)
 //
 // With many rows the plain form takes two feature tiles per row tile, as the gated form does by nature: a tile of x is loaded
 // once for both, which is what keeps the loads from L2 below the tensor cores' pace.
@@ -42,7 +42,7 @@ template <int kTok, int kMode>
 __global__ void __launch_bounds__(kGThreads, 1)
 grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_w, bf16* __restrict__ out,
                     int ldo, int n_out, int w_rows, int K, const int* __restrict__ tile_expert, const int* __restrict__ num_tiles,
-                    int max_tiles, unsigned* status) {
+                    int max_tiles, int act, float limit, unsigned* status) {
   using Cfg = GroupedCfg<kTok, kMode>;
   constexpr bool kTwo = Cfg::kNumA == 2, kGated = kMode == kGGated;
   extern __shared__ uint8_t smem_raw[];
@@ -163,7 +163,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
 #pragma unroll
           for (int j = 0; j < kChunk; ++j) {
             float v = __uint_as_float(g[j]);
-            if (kGated) v = silu(v) * __uint_as_float(u[j]);
+            if (kGated) v = gated_act<false>(act, limit, v, __uint_as_float(u[j]));
             dst[static_cast<size_t>(c + j) * ldo] = __float2bfloat16_rn(v);
           }
         }
@@ -188,7 +188,7 @@ extern "C" int forge_make_tmap_2d(CUtensorMap* tm, const void* base, uint64_t ro
 
 template <int kTok, int kMode>
 static int launch_grouped(const void* x, const void* w, void* out, int experts, int n_out, int K, const int* tile_expert, const int* num_tiles,
-                          int max_tiles, unsigned* status, cudaStream_t stream) {
+                          int max_tiles, int act, float limit, unsigned* status, cudaStream_t stream) {
   using Cfg = GroupedCfg<kTok, kMode>;
   const int w_rows = kMode == kGGated ? 2 * n_out : n_out;
   CUtensorMap tm_x, tm_w;
@@ -199,19 +199,19 @@ static int launch_grouped(const void* x, const void* w, void* out, int experts, 
   const long long tiles = static_cast<long long>(max_tiles) * ((n_out + Cfg::kTileFeat - 1) / Cfg::kTileFeat);
   const int grid = tiles < device_sm_count() ? static_cast<int>(tiles) : device_sm_count();
   return launch_kernel(kern, dim3(grid), dim3(kGThreads), Cfg::kSmemBytes, stream, 0, tm_x, tm_w, static_cast<bf16*>(out), n_out, n_out,
-                       w_rows, K, tile_expert, num_tiles, max_tiles, status) == cudaSuccess ? 0 : -5;
+                       w_rows, K, tile_expert, num_tiles, max_tiles, act, limit, status) == cudaSuccess ? 0 : -5;
 }
 
 // x [max_tiles * tile, K] bf16, w [experts, n_out or 2 n_out (gated), K], out [max_tiles * tile, n_out]; K a multiple of 8.
-extern "C" int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int n_out, int K, int gated, int tile,
-                                  const int* tile_expert, const int* num_tiles, int max_tiles, unsigned* status, cudaStream_t stream) {
+extern "C" int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int n_out, int K, int gated, int tile, int act,
+                                  float limit, const int* tile_expert, const int* num_tiles, int max_tiles, unsigned* status, cudaStream_t stream) {
   if (max_tiles <= 0 || n_out <= 0 || K <= 0) return 0;
   if ((K & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return -1;
   if (static_cast<long long>(experts) * n_out * 2 >= (1ll << 31)) return -1;
 #define FORGE_G(TOK, PLAIN)                                                                                                       \
   case TOK:                                                                                                                       \
-    return gated ? launch_grouped<TOK, kGGated>(x, w, out, experts, n_out, K, tile_expert, num_tiles, max_tiles, status, stream)  \
-                 : launch_grouped<TOK, PLAIN>(x, w, out, experts, n_out, K, tile_expert, num_tiles, max_tiles, status, stream);
+    return gated ? launch_grouped<TOK, kGGated>(x, w, out, experts, n_out, K, tile_expert, num_tiles, max_tiles, act, limit, status, stream)  \
+                 : launch_grouped<TOK, PLAIN>(x, w, out, experts, n_out, K, tile_expert, num_tiles, max_tiles, act, limit, status, stream);
   switch (tile) {
     FORGE_G(16, kGPlain)
     FORGE_G(32, kGPlain)

@@ -1,9 +1,10 @@
 // Mixture of experts: routing and the shuffling of rows.
 //
-//   router          logits (fp32) -> sigmoid -> the `top` largest scores of a token (ties: the lower expert)
+//   router          logits (fp32) -> the `top` largest of a token (ties: the lower expert), weighted by the sigmoid of each or
+//                   by the softmax over the chosen ones
 //   moe_plan        (token, choice) -> row of the expert-sorted buffer; every expert's rows start on a multiple of `tile`, so
 //                   a tile of rows has one expert (tile_expert; -1 past the last tile in use)
-//   moe_scatter     row = score * token, the score in fp32: it multiplies the expert's INPUT
+//   moe_scatter     row = token, or weight * token (weight in fp32) where the weight multiplies the expert's INPUT
 //
 // Rows between an expert's last token and its next tile boundary are never written nor read back.
 #include "../include/launch.cuh"
@@ -12,10 +13,12 @@
 
 namespace forge {
 
-// The `top` largest of a token's scores, by one warp; the scores in shared memory are used up.
-__device__ __forceinline__ void choose_top(float* score, int E, int top, int lane, int* experts, float* weights) {
+// The `top` largest of a token's scores, by one warp; the scores in shared memory are used up.  softmax: the weights are the
+// softmax over the chosen scores, else the scores themselves.
+__device__ __forceinline__ void choose_top(float* score, int E, int top, bool softmax, int lane, int* experts, float* weights) {
+  float first = 0.f, sum = 0.f;
   for (int j = 0; j < top; ++j) {
-    float best = -1.f;
+    float best = -INFINITY;
     int at = E;
     for (int e = lane; e < E; e += 32)
       if (score[e] > best) { best = score[e]; at = e; }
@@ -29,17 +32,21 @@ __device__ __forceinline__ void choose_top(float* score, int E, int top, int lan
     if (lane == 0) {
       experts[j] = at;
       weights[j] = best;
-      score[at] = -2.f;
+      score[at] = -INFINITY;
     }
+    if (j == 0) first = best;
+    sum += expf(best - first);
     __syncwarp();
   }
+  if (softmax)
+    for (int j = lane; j < top; j += 32) weights[j] = expf(weights[j] - first) / sum;
 }
 
 // bf16, W a multiple of 32, E <= 256: CTA = 16 MT tokens, the eight warps split W.  The order of the columns in a dot product is
 // free, so a lane loads eight consecutive columns of its row (16 bytes) and uses them as the four column pairs of two mma
 // k-steps, for tokens and experts alike: no shared memory on the way in.  The warps' partial logits are added in a fixed order.
 template <int MT>
-__global__ void __launch_bounds__(256) router_mma_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w, int T, int W, int E, int top,
+__global__ void __launch_bounds__(256) router_mma_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w, int T, int W, int E, int top, bool softmax,
                                                          int* __restrict__ experts, float* __restrict__ weights) {
   extern __shared__ float sm_part[];               // [8][16 MT][Ep]
   constexpr int kTok = 16 * MT, kGroup = 8;        // 8-expert blocks per pass
@@ -93,16 +100,16 @@ __global__ void __launch_bounds__(256) router_mma_kernel(const bf16* __restrict_
       float z = score[e];
 #pragma unroll
       for (int k = 1; k < 8; ++k) z += score[static_cast<size_t>(k) * kTok * Ep + e];
-      score[e] = 1.f / (1.f + expf(-z));
+      score[e] = softmax ? z : 1.f / (1.f + expf(-z));
     }
     __syncwarp();
-    choose_top(score, E, top, lane, experts + static_cast<size_t>(t0 + t) * top, weights + static_cast<size_t>(t0 + t) * top);
+    choose_top(score, E, top, softmax, lane, experts + static_cast<size_t>(t0 + t) * top, weights + static_cast<size_t>(t0 + t) * top);
   }
 }
 
 // CTA = one token; one warp per expert at a time.
 template <typename T, int N>
-__global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, const T* __restrict__ w, int W, int E, int top,
+__global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, const T* __restrict__ w, int W, int E, int top, bool softmax,
                                                      int* __restrict__ experts, float* __restrict__ weights) {
   extern __shared__ float score[];
   pdl_launch_dependents();
@@ -121,13 +128,13 @@ __global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, co
       for (int q = 0; q < N; ++q) z = fmaf(a[q], b[q], z);
     }
     z = warp_sum_f(z);
-    if (lane == 0) score[e] = 1.f / (1.f + expf(-z));
+    if (lane == 0) score[e] = softmax ? z : 1.f / (1.f + expf(-z));
   }
   __syncthreads();
-  if (warp == 0) choose_top(score, E, top, lane, experts + t * top, weights + t * top);
+  if (warp == 0) choose_top(score, E, top, softmax, lane, experts + t * top, weights + t * top);
 }
 
-extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int W, int E, int top, int* experts, float* weights,
+extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int W, int E, int top, int softmax, int* experts, float* weights,
                             cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (E > 4096 || top < 1 || top > E) return -1;
@@ -135,7 +142,7 @@ extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int 
   const size_t smem = static_cast<size_t>(E) * 4;
   if (fp32) {
     auto k = v4 ? router_kernel<float, 4> : router_kernel<float, 1>;
-    return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+    return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
   }
   if (W % 32 == 0 && E <= 256 && (reinterpret_cast<uintptr_t>(h) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
     const int Ep = (E + 7) & ~7;
@@ -144,13 +151,13 @@ extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int 
     const size_t part = static_cast<size_t>(8) * (two ? 32 : 16) * Ep * 4;
     if (two) {
       FORGE_ENSURE_DYN_SMEM(router_mma_kernel<2>, 8 * 32 * 128 * 4);
-      return launch_kernel(router_mma_kernel<2>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+      return launch_kernel(router_mma_kernel<2>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
     }
     FORGE_ENSURE_DYN_SMEM(router_mma_kernel<1>, 8 * 16 * 256 * 4);
-    return launch_kernel(router_mma_kernel<1>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+    return launch_kernel(router_mma_kernel<1>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
   }
   auto k = v4 ? router_kernel<bf16, 4> : router_kernel<bf16, 1>;
-  return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, experts, weights) == cudaSuccess ? 0 : -2;
+  return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
 }
 
 constexpr int kPlanThreads = 1024;
@@ -211,7 +218,7 @@ __global__ void __launch_bounds__(256) moe_scatter_kernel(const T* __restrict__ 
     float v[N];
     load_n<N>(h + t * W + c, v);
     for (int j = 0; j < top; ++j) {
-      const float s = weights[t * top + j];
+      const float s = weights != nullptr ? weights[t * top + j] : 1.f;
       float x[N];
 #pragma unroll
       for (int e = 0; e < N; ++e) x[e] = s * v[e];

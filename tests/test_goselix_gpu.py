@@ -353,7 +353,7 @@ def test_experts(ops, dtype, T, E, top, W, F):
 def test_equal_scores_choose_the_lower_expert(ops):
     h, router = torch.ones(3, 64, dtype=BF, device="cuda"), torch.ones(40, 64, dtype=BF, device="cuda")
     e, w = torch.empty(3, 4, dtype=torch.int32, device="cuda"), torch.empty(3, 4, device="cuda")
-    ops.C.router(h, router, e, w)
+    ops.C.router(h, router, e, w, False)
     assert e.tolist() == [[0, 1, 2, 3]] * 3
 
 

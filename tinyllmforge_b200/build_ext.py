@@ -64,6 +64,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
     os.makedirs(BUILD, exist_ok=True)
     headers = glob.glob(os.path.join(CSRC, "include", "*"))
     cu_files = sorted(glob.glob(os.path.join(CSRC, "**", "*.cu"), recursive=True))
+    host_headers = glob.glob(os.path.join(CSRC, "host", "*.h"))
     cpp_files = sorted(glob.glob(os.path.join(CSRC, "host", "*.cpp")))
     cuda_inc = os.path.join(os.path.dirname(os.path.dirname(_nvcc())), "include") if os.path.sep in _nvcc() else "/usr/local/cuda/include"
 
@@ -78,7 +79,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
                  f"-D_GLIBCXX_USE_CXX11_ABI={int(torch._C._GLIBCXX_USE_CXX11_ABI)}"]
     incs = [f"-I{p}" for p in cpp_extension.include_paths()] + [f"-I{sysconfig.get_paths()['include']}", f"-I{cuda_inc}"]
     for src in cpp_files:
-        tag = _digest([src], " ".join(cxx_flags) + torch.__version__)
+        tag = _digest([src] + host_headers, " ".join(cxx_flags) + torch.__version__)
         obj = os.path.join(BUILD, os.path.basename(src) + "." + tag + ".o")
         objs.append(obj)
         if force or not os.path.exists(obj):

@@ -17,6 +17,7 @@ import torch
 
 from ..config import Config
 from ..parallel.comm import TPGroup
+from .cuda_hybrid import HybridOps
 from .cuda_mixers import MixerOps
 from .quant import Fp8BlockWeight
 
@@ -77,7 +78,7 @@ def _streamk_workspace(C, device, num_sms: int) -> None:
     _STREAMK_WS[key] = (ws, counters)
 
 
-class CudaOps(MixerOps):
+class CudaOps(MixerOps, HybridOps):
     name = "cuda"
 
     def __init__(self, config: Config | None = None, tp: TPGroup | None = None, device=None):
@@ -152,7 +153,7 @@ class CudaOps(MixerOps):
                 return self.silu_mul(self.linear_fp8(x, w_gate_up))
             w_gate_up, force_deep = self._expand_fp8(w_gate_up), force_deep | W_DYNAMIC
         if not self.tma_ok(x, w_gate_up):
-            return self.silu_mul_any(self.linear_simt(x, w_gate_up))
+            return self.act_mul_any(self.linear_simt(x, w_gate_up))
         out = torch.empty(x.shape[0], w_gate_up.shape[0] // 2, dtype=x.dtype, device=x.device)
         self.C.gemm(x, w_gate_up, out, 1, force_mode, force_splits | (force_block_c << 8) | (force_deep << 16), self.status)
         return out

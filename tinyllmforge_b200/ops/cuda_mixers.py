@@ -9,21 +9,37 @@ import torch
 
 
 class Routed:
-    """The output of an expert layer before it is summed: row ``rows[t, j]`` of ``y`` belongs to token t's j-th expert."""
+    """The output of an expert layer before it is summed: row ``rows[t, j]`` of ``y`` belongs to token t's j-th expert and
+    counts ``weights[t, j]`` times (None: once)."""
 
-    def __init__(self, y: torch.Tensor, rows: torch.Tensor):
-        self.y, self.rows = y, rows
+    def __init__(self, y: torch.Tensor, rows: torch.Tensor, weights: torch.Tensor | None = None):
+        self.y, self.rows, self.weights = y, rows, weights
+
+
+ACTS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
 
 
 class MixerOps:
     """Mixed into ``CudaOps`` (uses its ``C``, ``status``, ``device`` and GEMM methods)."""
 
     # ------------------------------------------------------------------ residual stream
-    def stream_update(self, x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None):
+    def stream_update(self, x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None,
+                      a_bias=None, post=None, mult=1.0, offset=0.0):
         n = x.shape[0] if rows is None else rows.shape[0]
         outs = [torch.empty(n, x.shape[1], dtype=dtype, device=x.device) for _ in norms]
+        if post is not None or offset or isinstance(a, Routed):
+            if b is not None or vec is not None or len(norms) > 1:
+                raise ValueError("stream_update: one branch and one norm where a is normed or norm weights have an offset")
+            a_rows = a_weights = None
+            if isinstance(a, Routed):
+                a, a_rows, a_weights = a.y, a.rows, a.weights
+            self.C.stream_sandwich(x, a, a_rows, a_weights, a_bias, post, mult, offset, ids, embed, norms[0] if norms else None,
+                                   outs[0] if outs else None, rows, start, eps, dtype == torch.float32)
+            return outs
         b_rows = None
         if isinstance(b, Routed):
+            if b.weights is not None:
+                raise ValueError("stream_update: b is summed without weights")
             b, b_rows = b.y, b.rows
         self.C.stream_update(x, a, b, b_rows, ids, embed, vec, norms[0] if norms else None, norms[1] if len(norms) > 1 else None,
                              outs[0] if outs else None, outs[1] if len(outs) > 1 else None, rows, start, eps, dtype == torch.float32)
@@ -41,9 +57,19 @@ class MixerOps:
         self.C.gemm_simt(x, w, out, None)
         return out
 
-    def silu_mul_any(self, x):
+    def act_mul_any(self, x, act="silu", limit=0.0):
         out = torch.empty(x.shape[0], x.shape[1] // 2, dtype=x.dtype, device=x.device)
-        self.C.silu_mul_any(x, out)
+        self.C.act_mul_any(x, out, ACTS[act], limit)
+        return out
+
+    def linear_act_mul(self, x, w_gate_up, act: str, limit: float = 0.0):
+        """act(x @ w_gate.T, x @ w_up.T) for w_gate_up = gate rows, up rows."""
+        if act == "silu":
+            return self.linear_silu_mul(x, w_gate_up)
+        if not self.tma_ok(x, w_gate_up):
+            return self.act_mul_any(self.linear_simt(x, w_gate_up), act, limit)
+        out = torch.empty(x.shape[0], w_gate_up.shape[0] // 2, dtype=x.dtype, device=x.device)
+        self.C.gemm_act(x, w_gate_up, out, ACTS[act], limit, self.status)
         return out
 
     def head_linear(self, x, w, out) -> None:
@@ -143,12 +169,12 @@ class MixerOps:
         """Rows per tile of the tensor-core kernel (16 to 128): about what an expert gets."""
         return next((t for t in (16, 32, 64) if rows <= t * experts), 128)
 
-    def moe(self, h, router, gate_up, down, top):
+    def moe(self, h, router, gate_up, down, top, score="sigmoid", weigh="input", act="silu", limit=0.0):
         T, W = h.shape
         E, n = router.shape[0], T * top
         experts = torch.empty(T, top, dtype=torch.int32, device=h.device)
         weights = torch.empty(T, top, dtype=torch.float32, device=h.device)
-        self.C.router(h, router, experts, weights)
+        self.C.router(h, router, experts, weights, score == "softmax")
         fast = h.dtype == torch.bfloat16 and W % 8 == 0 and down.shape[2] % 8 == 0
         tile = self.expert_tile(n, E) if fast else 64
         tiles = min(n, n // tile + E)
@@ -157,14 +183,14 @@ class MixerOps:
         num_tiles = torch.empty(1, dtype=torch.int32, device=h.device)
         self.C.moe_plan(experts, E, tile, rows, tile_expert, num_tiles)
         xs = torch.empty(tiles * tile, W, dtype=h.dtype, device=h.device)
-        self.C.moe_scatter(h, rows, weights, xs)
+        self.C.moe_scatter(h, rows, weights if weigh == "input" else None, xs)
         y = torch.empty(tiles * tile, W, dtype=h.dtype, device=h.device)
         if fast:
             g = torch.empty(tiles * tile, down.shape[2], dtype=h.dtype, device=h.device)
-            self.C.grouped_gemm(xs, gate_up, g, True, tile, tile_expert, num_tiles, self.status)
-            self.C.grouped_gemm(g, down, y, False, tile, tile_expert, num_tiles, self.status)
+            self.C.grouped_gemm(xs, gate_up, g, True, tile, tile_expert, num_tiles, ACTS[act], limit, self.status)
+            self.C.grouped_gemm(g, down, y, False, tile, tile_expert, num_tiles, 0, 0.0, self.status)
         else:
             gu = torch.empty(tiles * tile, gate_up.shape[1], dtype=h.dtype, device=h.device)
             self.C.gemm_simt(xs, gate_up, gu, tile_expert)
-            self.C.gemm_simt(self.silu_mul_any(gu), down, y, tile_expert)
-        return Routed(y, rows)
+            self.C.gemm_simt(self.act_mul_any(gu, act, limit), down, y, tile_expert)
+        return Routed(y, rows, weights if weigh == "output" else None)

@@ -85,8 +85,8 @@ def _experts(ops, T, part):
     experts = torch.empty(T, TOP, dtype=torch.int32, device="cuda")
     weights = torch.empty(T, TOP, device="cuda")
     if part == "router":
-        return lambda: ops.C.router(h, router, experts, weights), T * WIDTH * 2, 2 * T * WIDTH * EXPERTS
-    ops.C.router(h, router, experts, weights)
+        return lambda: ops.C.router(h, router, experts, weights, False), T * WIDTH * 2, 2 * T * WIDTH * EXPERTS
+    ops.C.router(h, router, experts, weights, False)
     n = T * TOP
     tile = ops.expert_tile(n, EXPERTS)
     tiles = min(n, n // tile + EXPERTS)
@@ -101,10 +101,10 @@ def _experts(ops, T, part):
     used = int((torch.bincount(experts.view(-1).long(), minlength=EXPERTS) > 0).sum())
     if part == "gate_up":
         w, out = _rand(EXPERTS, 2 * FF, WIDTH, scale=0.02), _rand(tiles * tile, FF)
-        return (lambda: ops.C.grouped_gemm(xs, w, out, True, tile, te, nt, ops.status),
+        return (lambda: ops.C.grouped_gemm(xs, w, out, True, tile, te, nt, 0, 0.0, ops.status),
                 (used * 2 * FF * WIDTH + n * (WIDTH + FF)) * 2, 4 * n * WIDTH * FF)
     g, w, out = _rand(tiles * tile, FF), _rand(EXPERTS, WIDTH, FF, scale=0.02), _rand(tiles * tile, WIDTH)
-    return (lambda: ops.C.grouped_gemm(g, w, out, False, tile, te, nt, ops.status), (used * FF * WIDTH + n * (WIDTH + FF)) * 2, 2 * n * WIDTH * FF)
+    return (lambda: ops.C.grouped_gemm(g, w, out, False, tile, te, nt, 0, 0.0, ops.status), (used * FF * WIDTH + n * (WIDTH + FF)) * 2, 2 * n * WIDTH * FF)
 
 
 def _stream(ops, T, W=WIDTH):
