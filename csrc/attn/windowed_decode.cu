@@ -1,0 +1,297 @@
+// Decode attention over a sliding window of the paged cache (bf16): one query token per sequence, grouped queries.
+//
+// CTA = (key/value head and up to 16 of its query heads, sequence, chunk of the window).  Its four warps are independent: each
+// takes every fourth tile of 16 keys, brings it into a ring of its own with 16-byte asynchronous copies, multiplies it with all
+// query heads at once (mma.sync: heads on the 16-row side) and keeps its own running maximum, sum and output.  Softmax
+// weights are fp32 and enter the second product as bf16 hi + lo halves.  The warps' states are merged through shared memory;
+// with more than one chunk, partial outputs go to scratch and a second kernel merges them.  Lengths are read on the device and
+// the grid depends on the batch bucket only, so the launch is CUDA-graph safe.
+#include "../include/launch.cuh"
+#include "../include/mma_sync.cuh"
+#include "../include/scalar.cuh"
+
+namespace forge {
+
+constexpr int kWDKeys = 16, kWDWarps = 4;
+
+struct WindowedDecode {
+  const bf16* q;            // [seqs][H][q_pitch]
+  const bf16* k_cache;      // [blocks][G][block_size][d]
+  const bf16* v_cache;      // [blocks][G][block_size][dv]
+  const int* tables;        // [seqs][width]
+  const int* lens;          // [seqs]
+  bf16* out;                // [seqs][ldo]
+  long long ldo;
+  float* part_o;            // [seqs][H][chunks][dv]
+  float* part_ml;           // [seqs][H][chunks][2]
+  int width, num_blocks, block_size, H, G, d, dv, q_pitch, window, chunk, max_chunks, stages, slices;
+  float scale_log2, out_scale;
+  unsigned* status;
+};
+
+// Row pitch in elements: an odd number of 16-byte units (conflict-free ldmatrix) with room for 16-column reads.
+__host__ __device__ __forceinline__ int wd_pitch(int cols) {
+  const int u = cols >> 3;
+  return ((u & 1) ? u + 2 : u + 1) * 8;
+}
+
+struct WindowRange {
+  int begin, lo, end;       // first key of the first 16-key tile, first visible key, end of the visible keys
+};
+__device__ __forceinline__ WindowRange window_range(const WindowedDecode& p, int s, unsigned* status) {
+  int len = p.lens[s];
+  const int cap = p.width * p.block_size;
+  if (len > cap) {
+    set_status(status, kStatusBadIndex);
+    len = cap;
+  }
+  WindowRange r;
+  r.end = max(len, 0);
+  r.lo = max(r.end - p.window, 0);
+  r.begin = r.lo & ~(kWDKeys - 1);
+  return r;
+}
+
+template <int NV>           // blocks of 8 value columns
+__global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const WindowedDecode p) {
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  const int kp = wd_pitch(p.d), vp = wd_pitch(p.dv);
+  const int stage = kWDKeys * (kp + vp);                       // elements per warp and stage
+  bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                // [16][kp]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, q2 = 2 * (lane & 3);
+  bf16* ring = sQ + 16 * kp + static_cast<size_t>(warp) * p.stages * stage;
+
+  pdl_launch_dependents();
+  pdl_wait();
+  const int s = blockIdx.y, g = blockIdx.x / p.slices, slice = blockIdx.x % p.slices, chunk = blockIdx.z;
+  const int per = p.H / p.G, h0 = g * per + slice * 16, nh = min(16, per - slice * 16);
+  const WindowRange w = window_range(p, s, chunk == 0 ? p.status : nullptr);
+  const int c_begin = w.begin + chunk * p.chunk, c_end = min(c_begin + p.chunk, w.end);
+  const int n_chunks = (w.end - w.begin + p.chunk - 1) / p.chunk;
+  if (c_begin >= c_end) {                                      // uniform for the CTA
+    if (chunk == 0)                                            // padding row: defined output
+      for (int i = threadIdx.x; i < nh * p.dv; i += blockDim.x)
+        p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h0) * p.dv + i] = __float2bfloat16_rn(0.f);
+    return;
+  }
+  const int dpad = (p.d + 15) & ~15, ku = p.d >> 3, vu = p.dv >> 3, qu = dpad >> 3;
+  for (int i = threadIdx.x; i < 16 * qu; i += blockDim.x) {
+    const int r = i / qu, u = i % qu;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (r < nh && u < ku) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<size_t>(s) * p.H + h0 + r) * p.q_pitch + u * 8);
+    *reinterpret_cast<uint4*>(sQ + r * kp + u * 8) = v;
+  }
+  if (dpad != p.d)                                             // the key columns that complete a 16-column step stay zero
+    for (int r = lane; r < p.stages * kWDKeys; r += 32)
+      *reinterpret_cast<uint4*>(ring + static_cast<size_t>(r / kWDKeys) * stage + (r % kWDKeys) * kp + p.d) = make_uint4(0, 0, 0, 0);
+  __syncthreads();
+
+  const int tiles = (c_end - c_begin + kWDKeys - 1) / kWDKeys;
+  const int mine = tiles > warp ? (tiles - warp + kWDWarps - 1) / kWDWarps : 0;
+  auto load = [&](int i) {                                     // this warp's tile i
+    if (i < mine) {
+      const int key = c_begin + (i * kWDWarps + warp) * kWDKeys;
+      int blk = p.tables[static_cast<size_t>(s) * p.width + key / p.block_size];
+      if (blk < 0 || blk >= p.num_blocks) {
+        if (lane == 0) set_status(p.status, kStatusBadIndex);
+        blk = 0;
+      }
+      const size_t row = (static_cast<size_t>(blk) * p.G + g) * p.block_size + key % p.block_size;   // 16 keys never straddle a block
+      bf16* sk = ring + static_cast<size_t>(i % p.stages) * stage;
+      bf16* sv = sk + kWDKeys * kp;
+      for (int u = lane; u < kWDKeys * ku; u += 32) cp_async16(smem_u32(sk + (u / ku) * kp + (u % ku) * 8), p.k_cache + row * p.d + u * 8, 16);
+      for (int u = lane; u < kWDKeys * vu; u += 32) cp_async16(smem_u32(sv + (u / vu) * vp + (u % vu) * 8), p.v_cache + row * p.dv + u * 8, 16);
+    }
+    cp_async_commit();
+  };
+
+  float o[NV][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+  for (int nb = 0; nb < NV; ++nb) o[nb][0] = o[nb][1] = o[nb][2] = o[nb][3] = 0.f;
+  for (int i = 0; i + 1 < p.stages; ++i) load(i);
+  for (int i = 0; i < mine; ++i) {
+    __syncwarp();                                              // every lane has read the stage that is filled next
+    load(i + p.stages - 1);
+    if (p.stages == 4) cp_async_wait<3>();
+    else if (p.stages == 3) cp_async_wait<2>();
+    else cp_async_wait<1>();
+    __syncwarp();
+    const bf16* sk = ring + static_cast<size_t>(i % p.stages) * stage;
+    const bf16* sv = sk + kWDKeys * kp;
+    float x[2][4] = {};
+    for (int k = 0; k < dpad >> 4; ++k) {
+      uint32_t a[4], b[4];
+      ldsm_x4(smem_u32(sQ + (lane & 15) * kp + k * 16 + (lane >> 4) * 8), a);
+      ldsm_x4(smem_u32(sk + ((lane & 7) + (lane >> 4) * 8) * kp + k * 16 + ((lane >> 3) & 1) * 8), b);
+      mma16816(x[0], a, b[0], b[1]);
+      mma16816(x[1], a, b[2], b[3]);
+    }
+    const int key = c_begin + (i * kWDWarps + warp) * kWDKeys;
+    float mt[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j = key + n * 8 + q2 + (e & 1);
+        x[n][e] = j >= w.lo && j < c_end ? x[n][e] * p.scale_log2 : -INFINITY;
+        mt[e >> 1] = fmaxf(mt[e >> 1], x[n][e]);
+      }
+    float alpha[2];
+    bool moved = false;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 1));
+      mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 2));
+      const float m_new = fmaxf(m[r], mt[r]);
+      moved |= m_new != m[r];
+      alpha[r] = m_new == -INFINITY ? 1.f : exp2f(m[r] - m_new);          // nothing visible so far
+      m[r] = m_new;
+    }
+    if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+      for (int nb = 0; nb < NV; ++nb) {
+        o[nb][0] *= alpha[0]; o[nb][1] *= alpha[0];
+        o[nb][2] *= alpha[1]; o[nb][3] *= alpha[1];
+      }
+      l[0] *= alpha[0];
+      l[1] *= alpha[1];
+    }
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const float ref = m[r] == -INFINITY ? 0.f : m[r];
+        const float a = ex2_approx(x[n][2 * r] - ref), b = ex2_approx(x[n][2 * r + 1] - ref);
+        l[r] += a + b;
+        const uint32_t h = pack_bf16x2(a, b);
+        hi[n * 2 + r] = h;
+        lo[n * 2 + r] = pack_bf16x2(a - bf16_lo(h), b - bf16_hi(h));
+      }
+    const bf16* vr = sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * vp + (lane >> 4) * 8;
+#pragma unroll
+    for (int nb = 0; nb < NV; nb += 2) {
+      if (nb * 8 < p.dv) {
+        uint32_t b[4];
+        ldsm_x4_trans(smem_u32(vr + nb * 8), b);
+        mma16816(o[nb], hi, b[0], b[1]);
+        mma16816(o[nb], lo, b[0], b[1]);
+        mma16816(o[nb + 1], hi, b[2], b[3]);
+        mma16816(o[nb + 1], lo, b[2], b[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  // merge the warps: [4][16][8 NV + 2] floats over the rings
+  float* merge = reinterpret_cast<float*>(smem_raw);
+  const int mp = NV * 8 + 2;
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    float* row = merge + (warp * 16 + g4 + r * 8) * mp;
+#pragma unroll
+    for (int nb = 0; nb < NV; ++nb) {
+      row[nb * 8 + q2] = o[nb][2 * r];
+      row[nb * 8 + q2 + 1] = o[nb][2 * r + 1];
+    }
+    if ((lane & 3) == 0) {
+      row[NV * 8] = m[r];
+      row[NV * 8 + 1] = l[r];
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nh * p.dv; i += blockDim.x) {
+    const int r = i / p.dv, c = i % p.dv;
+    float M = -INFINITY;
+#pragma unroll
+    for (int k = 0; k < kWDWarps; ++k) M = fmaxf(M, merge[(k * 16 + r) * mp + NV * 8]);
+    float L = 0.f, O = 0.f;
+#pragma unroll
+    for (int k = 0; k < kWDWarps; ++k) {
+      const float* row = merge + (k * 16 + r) * mp;
+      const float f = row[NV * 8] == -INFINITY ? 0.f : exp2f(row[NV * 8] - M);
+      L = fmaf(f, row[NV * 8 + 1], L);
+      O = fmaf(f, row[c], O);
+    }
+    if (n_chunks == 1) {
+      p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h0 + r) * p.dv + c] = __float2bfloat16_rn(L > 0.f ? p.out_scale * O / L : 0.f);
+    } else {
+      const size_t at = (static_cast<size_t>(s) * p.H + h0 + r) * p.max_chunks + chunk;
+      p.part_o[at * p.dv + c] = O;
+      if (c == 0) {
+        p.part_ml[at * 2] = M;
+        p.part_ml[at * 2 + 1] = L;
+      }
+    }
+  }
+}
+
+// CTA = (query head, sequence): merges the chunks of a window that has more than one.
+__global__ void __launch_bounds__(128) windowed_merge_kernel(const WindowedDecode p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, s = blockIdx.y;
+  const WindowRange w = window_range(p, s, nullptr);
+  const int n = (w.end - w.begin + p.chunk - 1) / p.chunk;
+  if (n <= 1) return;
+  const size_t base = (static_cast<size_t>(s) * p.H + h) * p.max_chunks;
+  float M = -INFINITY;
+  for (int c = 0; c < n; ++c) M = fmaxf(M, p.part_ml[(base + c) * 2]);
+  for (int i = threadIdx.x; i < p.dv; i += blockDim.x) {
+    float L = 0.f, O = 0.f;
+    for (int c = 0; c < n; ++c) {
+      const float m = p.part_ml[(base + c) * 2], f = m == -INFINITY ? 0.f : exp2f(m - M);
+      L = fmaf(f, p.part_ml[(base + c) * 2 + 1], L);
+      O = fmaf(f, p.part_o[(base + c) * p.dv + i], O);
+    }
+    p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h) * p.dv + i] = __float2bfloat16_rn(L > 0.f ? p.out_scale * O / L : 0.f);
+  }
+}
+
+static size_t wd_smem(int d, int dv, int nv, int stages) {
+  const size_t ring = static_cast<size_t>(16 * wd_pitch(d) + kWDWarps * stages * kWDKeys * (wd_pitch(d) + wd_pitch(dv))) * 2;
+  const size_t merge = static_cast<size_t>(kWDWarps) * 16 * (nv * 8 + 2) * 4;
+  return ring > merge ? ring : merge;
+}
+
+// 1 if the kernel takes these sizes (else: windowed_attend_any).
+extern "C" int forge_windowed_decode_ok(int d, int dv, int block_size) {
+  return (d & 7) == 0 && (dv & 7) == 0 && d >= 8 && dv >= 8 && d <= 256 && dv <= 256 && block_size % kWDKeys == 0;
+}
+
+// q [seqs][H][q_pitch], one token per sequence; out rows of ldo elements.  chunk: a multiple of 16; max_chunks * chunk must cover
+// min(window, width * block_size) + 15 keys.  part_o, part_ml: fp32 scratch, needed when max_chunks > 1.
+extern "C" int forge_windowed_decode(const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* tables, const int* lens,
+                                     int seqs, int width, int num_blocks, int block_size, void* out, long long ldo, float* part_o, float* part_ml,
+                                     int chunk, int max_chunks, int H, int G, int d, int dv, int window, float scale, float out_scale,
+                                     unsigned* status, cudaStream_t stream) {
+  if (seqs <= 0) return 0;
+  if (!forge_windowed_decode_ok(d, dv, block_size) || (q_pitch & 7) || seqs > 65535 || max_chunks > 65535 || chunk % kWDKeys || chunk < kWDKeys || window < 1)
+    return -1;
+  const long long cap = static_cast<long long>(width) * block_size, span = (window < cap ? window : cap) + kWDKeys - 1;
+  if (static_cast<long long>(max_chunks) * chunk < span || (max_chunks > 1 && (part_o == nullptr || part_ml == nullptr))) return -1;
+  WindowedDecode p = {static_cast<const bf16*>(q), static_cast<const bf16*>(k_cache), static_cast<const bf16*>(v_cache), tables, lens,
+                      static_cast<bf16*>(out), ldo, part_o, part_ml, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, chunk, max_chunks,
+                      0, (H / G + 15) / 16, scale * 1.4426950408889634f, out_scale, status};
+  const dim3 grid(G * p.slices, seqs, max_chunks);
+#define FORGE_WD(NV)                                                                                                                   \
+  {                                                                                                                                    \
+    p.stages = 4;                                                                                                                      \
+    while (p.stages > 2 && wd_smem(d, dv, NV, p.stages) > 112 * 1024) --p.stages;                                                      \
+    const size_t smem = wd_smem(d, dv, NV, p.stages);                                                                                  \
+    if (smem > 227 * 1024) return -1;                                                                                                  \
+    FORGE_ENSURE_DYN_SMEM(windowed_decode_kernel<NV>, 227 * 1024);                                                                     \
+    if (launch_kernel(windowed_decode_kernel<NV>, grid, dim3(32 * kWDWarps), smem, stream, 0, p) != cudaSuccess) return -2;            \
+  }
+  if (dv <= 64) FORGE_WD(8) else if (dv <= 128) FORGE_WD(16) else if (dv <= 192) FORGE_WD(24) else FORGE_WD(32)
+#undef FORGE_WD
+  if (max_chunks > 1 && launch_kernel(windowed_merge_kernel, dim3(H, seqs), dim3(128), 0, stream, 0, p) != cudaSuccess) return -2;
+  return 0;
+}
+
+}  // namespace forge

@@ -1,0 +1,349 @@
+// Attention of prompts over a sliding window on the 5th-generation tensor cores: variable length, grouped queries, keys and
+// values read from the paged cache, key and value heads of different width (multiples of 8 up to 256).
+//
+//   S = Q K^T   K-major boxes of 64 columns; q rows are zero-padded to whole boxes, TMA fills the missing key columns with zeros
+//   O += P V    P = softmax weights in fp32, as bf16 hi + lo halves (two products: 16 mantissa bits), V as TMA delivers it
+//               (rows = keys, MN-major)
+//
+// CTA = 128 query rows of one (sequence, head), key tiles of 64 from the tile that holds the first row's oldest visible key to
+// the tile of the last row's own.  A row may see nothing of its CTA's first tiles: its reference maximum is set by the first
+// key it does see, and nothing of O needs scaling then.  Warp roles, double-buffered S, the reference maximum that is only
+// raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu; P is double-buffered where shared memory allows.
+#include "../include/launch.cuh"
+#include "../include/scalar.cuh"
+
+namespace forge {
+
+constexpr int kXM = 128, kXN = 64, kXThreads = 192;
+constexpr int kXQBox = kXM * 128;           // bytes of a 128-row x 64-column box
+constexpr int kXKBox = kXN * 128;           // bytes of a 64-row x 64-column box
+
+__device__ __forceinline__ uint64_t windowed_desc_mn(uint32_t smem_addr, uint32_t mn_block_bytes) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((smem_addr & 0x3FFFFu) >> 4);
+  d |= static_cast<uint64_t>((mn_block_bytes >> 4) & 0x3FFFu) << 16;   // next 64 elements along MN
+  d |= static_cast<uint64_t>(1024 >> 4) << 32;                         // next 8 rows along K
+  d |= static_cast<uint64_t>(1) << 46;
+  d |= static_cast<uint64_t>(2) << 61;                                 // SWIZZLE_128B
+  return d;
+}
+
+// kMasked: only keys kbase + i in [lo, limit) count.
+template <bool kMasked>
+__device__ __forceinline__ float windowed_row_max(const uint32_t (&v)[kXN], int kbase, int lo, int limit) {
+  float m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+  for (int i = 0; i < kXN; i += 4)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float x = __uint_as_float(v[i + e]);
+      const int key = kbase + i + e;
+      m[e] = fmaxf(m[e], (!kMasked || (key >= lo && key < limit)) ? x : -INFINITY);
+    }
+  return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
+}
+
+// p = 2^(s scale - m_ref) of one row -> hi and lo bf16 halves in shared memory (K-major, 128-byte swizzle); returns the row sum.
+template <bool kMasked>
+__device__ __forceinline__ float windowed_probs(const uint32_t (&v)[kXN], int kbase, int lo, int limit, float scale_log2, float m_ref,
+                                                uint8_t* p_row, int r) {
+  float ps[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int c = 0; c < kXN; c += 8) {
+    uint32_t hi[4], lw[4];
+#pragma unroll
+    for (int i = 0; i < 8; i += 2) {
+      const int key = kbase + c + i;
+      float p0 = ex2_approx(fmaf(__uint_as_float(v[c + i]), scale_log2, -m_ref));
+      float p1 = ex2_approx(fmaf(__uint_as_float(v[c + i + 1]), scale_log2, -m_ref));
+      if (kMasked) {
+        p0 = key >= lo && key < limit ? p0 : 0.f;
+        p1 = key + 1 >= lo && key + 1 < limit ? p1 : 0.f;
+      }
+      ps[i >> 1] += p0 + p1;
+      const uint32_t h = pack_bf16x2(p0, p1);
+      hi[i >> 1] = h;
+      lw[i >> 1] = pack_bf16x2(p0 - bf16_lo(h), p1 - bf16_hi(h));
+    }
+    const int at = ((c >> 3) ^ (r & 7)) << 4;
+    *reinterpret_cast<uint4*>(p_row + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4*>(p_row + kXQBox + at) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+  }
+  return (ps[0] + ps[1]) + (ps[2] + ps[3]);
+}
+
+struct WindowedPrefill {
+  int H, G, d, dv, nq, nv, p_bufs;          // nq, nv: boxes of 64 columns of keys and of values
+  int window, block_size, table_width, num_blocks;
+  long long ldo;
+  float scale_log2, out_scale;
+};
+
+// tm_q: [tokens, H * 64 nq], box 128 x 64; tm_k / tm_v: [blocks * G * block_size, d / dv], box 64 x 64.
+__global__ void __launch_bounds__(kXThreads, 1)
+windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
+                        const int* __restrict__ cu_q, const int* __restrict__ context_lens, const int* __restrict__ tables,
+                        bf16* __restrict__ out, const WindowedPrefill z, unsigned* status) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const uint32_t k_stage = z.nq * kXKBox, v_stage = z.nv * kXKBox;
+  uint8_t* sQ = smem;
+  uint8_t* sK = sQ + z.nq * kXQBox;                   // [2 stages]
+  uint8_t* sV = sK + 2 * k_stage;                     // [2 stages]
+  uint8_t* sP = sV + 2 * v_stage;                     // [p_bufs][hi, lo]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + z.p_bufs * 2 * kXQBox);
+  uint64_t* q_full = bars;
+  uint64_t* k_full = bars + 1;
+  uint64_t* k_empty = bars + 3;
+  uint64_t* v_full = bars + 5;
+  uint64_t* v_empty = bars + 7;
+  uint64_t* s_full = bars + 9;
+  uint64_t* s_empty = bars + 11;                      // one arrival per softmax warp
+  uint64_t* p_full = bars + 13;                       // one arrival per softmax warp
+  uint64_t* pv_done = bars + 15;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
+
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.z, h = blockIdx.y, g = h / (z.H / z.G);
+  const int q_begin = cu_q[seq], q_len = cu_q[seq + 1] - q_begin;
+  const int k_len = min(context_lens[seq], z.table_width * z.block_size);
+  const int m0 = (gridDim.x - 1 - blockIdx.x) * kXM;  // late tiles, which see more keys, first
+  if (m0 >= q_len) return;                            // uniform for the CTA, before anything is allocated
+  const int past = max(k_len - q_len, 0);
+  const int kv_end = min(k_len, past + m0 + kXM);
+  const int tile0 = max(past + m0 - z.window + 1, 0) / kXN;
+  const int n_tiles = (kv_end + kXN - 1) / kXN - tile0;
+  if (n_tiles <= 0) return;
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp == 0 && lane == 0) {
+    prefetch_tensormap(&tm_q);
+    prefetch_tensormap(&tm_k);
+    prefetch_tensormap(&tm_v);
+    mbar_init(q_full, 1);
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(&k_full[s], 1);
+      mbar_init(&k_empty[s], 1);
+      mbar_init(&v_full[s], 1);
+      mbar_init(&v_empty[s], 1);
+      mbar_init(&s_full[s], 1);
+      mbar_init(&s_empty[s], 4);
+      mbar_init(&p_full[s], 4);
+      mbar_init(&pv_done[s], 1);
+    }
+    fence_mbar_init();
+  }
+  const uint32_t tmem_cols = z.nv > 2 ? 512 : 256;    // S0 | S1 | O
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, tmem_cols);
+    tmem_relinquish();
+  }
+  tcgen05_fence_before();
+  __syncthreads();
+  tcgen05_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  const uint32_t tmem_o = tmem_base + 2 * kXN;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      mbar_expect_tx(q_full, z.nq * kXQBox);
+      for (int b = 0; b < z.nq; ++b) tma_load_2d(sQ + b * kXQBox, &tm_q, q_full, (h * z.nq + b) * 64, q_begin + m0);
+      for (int j = 0; j < n_tiles; ++j) {
+        const int s = j & 1, tok = (tile0 + j) * kXN;
+        const uint32_t ph = (j >> 1) & 1;
+        int blk = tables[static_cast<size_t>(seq) * z.table_width + tok / z.block_size];
+        if (blk < 0 || blk >= z.num_blocks) {
+          set_status(status, kStatusBadIndex);
+          blk = 0;
+        }
+        const int row = (blk * z.G + g) * z.block_size + tok % z.block_size;       // a tile never straddles a block
+        if (!mbar_wait_parked(&k_empty[s], ph ^ 1, status)) break;
+        mbar_expect_tx(&k_full[s], k_stage);
+        for (int b = 0; b < z.nq; ++b) tma_load_2d(sK + s * k_stage + b * kXKBox, &tm_k, &k_full[s], b * 64, row);
+        if (!mbar_wait_parked(&v_empty[s], ph ^ 1, status)) break;
+        mbar_expect_tx(&v_full[s], v_stage);
+        for (int b = 0; b < z.nv; ++b) tma_load_2d(sV + s * v_stage + b * kXKBox, &tm_v, &v_full[s], b * 64, row);
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = umma_idesc(kXM, kXN, 1, 1);
+      const uint32_t idesc_o = umma_idesc(kXM, z.nv * 64, 1, 1) | (1u << 16);         // B (= V) MN-major
+      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
+      const int steps = (z.d + 15) >> 4;
+      bool ok = mbar_wait(q_full, 0, status);
+      auto issue_s = [&](int j) -> bool {
+        const int s = j & 1;
+        if (!mbar_wait_parked(&k_full[s], (j >> 1) & 1, status)) return false;
+        if (!mbar_wait_parked(&s_empty[s], ((j >> 1) & 1) ^ 1, status)) return false; // softmax has read S of tile j - 2
+        tcgen05_fence_after();
+        const uint32_t k_addr = smem_u32(sK + s * k_stage);
+        for (int k = 0; k < steps; ++k)
+          umma_f16(tmem_base + s * kXN, umma_desc_k_sw128(q_addr + (k >> 2) * kXQBox + (k & 3) * 32),
+                   umma_desc_k_sw128(k_addr + (k >> 2) * kXKBox + (k & 3) * 32), idesc_s, k != 0);
+        umma_commit(&s_full[s]);
+        umma_commit(&k_empty[s]);
+        return true;
+      };
+      ok = ok && issue_s(0);
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        if (j + 1 < n_tiles) ok = issue_s(j + 1);
+        if (!ok) break;
+        const int s = j & 1;
+        const uint32_t ph = (j >> 1) & 1;
+        if (!mbar_wait_parked(&v_full[s], ph, status) || !mbar_wait_parked(&p_full[s], ph, status)) {
+          ok = false;
+          break;
+        }
+        tcgen05_fence_after();
+        const uint32_t v_addr = smem_u32(sV + s * v_stage);
+        const uint32_t pj_addr = p_addr + (j % z.p_bufs) * 2 * kXQBox;
+#pragma unroll
+        for (int k = 0; k < kXN / 16; ++k) {
+          const uint64_t vd = windowed_desc_mn(v_addr + k * 16 * 128, kXKBox);
+          umma_f16(tmem_o, umma_desc_k_sw128(pj_addr + k * 32), vd, idesc_o, (j | k) != 0);
+          umma_f16(tmem_o, umma_desc_k_sw128(pj_addr + kXQBox + k * 32), vd, idesc_o, 1);
+        }
+        umma_commit(&pv_done[s]);
+        umma_commit(&v_empty[s]);
+      }
+    }
+  } else {
+    const int quad = warp & 3;
+    const int r = quad * 32 + lane;
+    const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
+    const int qpos = past + m0 + r;
+    const int limit = min(qpos + 1, k_len), lo = max(qpos - z.window + 1, 0);          // visible keys: [lo, limit)
+    const int o_cols = z.nv * 64;
+    float m_ref = 0.f, l_run = 0.f;
+    bool seen = false, ok = true;
+    for (int j = 0; j < n_tiles; ++j) {
+      ok = mbar_wait(&s_full[j & 1], (j >> 1) & 1, status);
+      if (!ok) break;
+      tcgen05_fence_after();
+      const uint32_t s_addr = tmem_base + lane_addr + (j & 1) * kXN;
+      const int kbase = (tile0 + j) * kXN;
+      uint32_t v[kXN];
+#pragma unroll
+      for (int c = 0; c < kXN; c += 32) tmem_ld_x32(s_addr + c, v + c);
+      tmem_ld_wait();
+      tcgen05_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&s_empty[j & 1]);
+      const bool masked = !__all_sync(0xffffffffu, kbase >= lo && kbase + kXN <= limit);
+      float mt = masked ? windowed_row_max<true>(v, kbase, lo, limit) : windowed_row_max<false>(v, kbase, lo, limit);
+      mt *= z.scale_log2;                                // scale > 0: max commutes with the scaling
+      if (!seen && mt != -INFINITY) {                    // nothing of this row is in O yet, or only zeros
+        m_ref = mt;
+        seen = true;
+      }
+      if (j > 0) {
+        const bool grow = seen && mt - m_ref > 8.f;
+        if (__any_sync(0xffffffffu, grow)) {
+          ok = mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1, status);
+          if (!ok) break;
+          tcgen05_fence_after();
+          const float m_new = seen ? fmaxf(m_ref, mt) : m_ref;
+          const float alpha = exp2f(m_ref - m_new);
+#pragma unroll 1
+          for (int c = 0; c < o_cols; c += 32) {
+            uint32_t o[32];
+            tmem_ld_x32(tmem_o + lane_addr + c, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+            tmem_st_x32(tmem_o + lane_addr + c, o);
+          }
+          tmem_st_wait();
+          tcgen05_fence_before();
+          l_run *= alpha;
+          m_ref = m_new;
+        }
+      }
+      if (j >= z.p_bufs) {                               // this P buffer was last read by P V of tile j - p_bufs
+        const int jj = j - z.p_bufs;
+        ok = mbar_wait(&pv_done[jj & 1], (jj >> 1) & 1, status);
+        if (!ok) break;
+      }
+      uint8_t* p_row = sP + (j % z.p_bufs) * 2 * kXQBox + r * 128;
+      l_run += masked ? windowed_probs<true>(v, kbase, lo, limit, z.scale_log2, m_ref, p_row, r)
+                      : windowed_probs<false>(v, kbase, lo, limit, z.scale_log2, m_ref, p_row, r);
+      fence_proxy_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[j & 1]);
+    }
+    if (ok) ok = mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, status);
+    if (ok) {
+      tcgen05_fence_after();
+      const float inv = l_run > 0.f ? z.out_scale / l_run : 0.f;
+      const bool store = m0 + r < q_len;
+      bf16* dst = out + static_cast<size_t>(q_begin + m0 + r) * z.ldo + static_cast<size_t>(h) * z.dv;
+#pragma unroll 1
+      for (int c = 0; c < o_cols; c += 32) {
+        uint32_t o[32];
+        tmem_ld_x32(tmem_o + lane_addr + c, o);
+        tmem_ld_wait();
+        if (store) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 8) {
+            if (c + i >= z.dv) continue;                 // dv is a multiple of 8
+            uint4 pk;
+            pk.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
+            pk.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
+            pk.z = pack_bf16x2(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv);
+            pk.w = pack_bf16x2(__uint_as_float(o[i + 6]) * inv, __uint_as_float(o[i + 7]) * inv);
+            *reinterpret_cast<uint4*>(dst + c + i) = pk;
+          }
+        }
+      }
+    }
+  }
+
+  tcgen05_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tcgen05_fence_after();
+    tmem_dealloc(tmem_base, tmem_cols);
+  }
+}
+
+static int windowed_prefill_smem(int nq, int nv, int p_bufs) {
+  return nq * (kXQBox + 2 * kXKBox) + 2 * nv * kXKBox + p_bufs * 2 * kXQBox + 256 + 1024;
+}
+
+// Columns of one head's padded query row, or 0 when the kernel does not take these sizes (else: windowed_attend_any).
+extern "C" int forge_windowed_prefill_qcols(int d, int dv, int block_size) {
+  if ((d & 7) || (dv & 7) || d < 8 || dv < 8 || d > 256 || dv > 256 || block_size % kXN) return 0;
+  return 64 * ((d + 63) / 64);
+}
+
+extern "C" int forge_make_tmap_2d(CUtensorMap* tm, const void* base, uint64_t rows, uint64_t cols, uint64_t ld,
+                                  uint32_t box_rows, int elem_bytes);
+
+// q [tokens][H][q_pitch], q_pitch = forge_windowed_prefill_qcols; sequence s has the step's tokens cu_q[s] .. cu_q[s + 1] (its last
+// ones) and context_lens[s] keys; out rows of ldo elements (a multiple of 8), 16-byte aligned.
+extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_cache, const void* v_cache, const int* cu_q, const int* context_lens,
+                                      const int* tables, int table_width, int num_blocks, int block_size, void* out, long long ldo, int num_seqs,
+                                      int max_q, int H, int G, int d, int dv, int window, float scale, float out_scale, unsigned* status,
+                                      cudaStream_t stream) {
+  if (tokens <= 0 || num_seqs <= 0 || max_q <= 0) return 0;
+  const int qcols = forge_windowed_prefill_qcols(d, dv, block_size);
+  if (qcols == 0 || num_seqs > 65535 || H > 65535 || H % G || window < 1 || !(scale > 0.f) || (ldo & 7) || (reinterpret_cast<uintptr_t>(out) & 15)) return -1;
+  if (static_cast<long long>(num_blocks) * G * block_size >= (1ll << 31)) return -1;
+  const int nq = qcols / 64, nv = (dv + 63) / 64;
+  const int p_bufs = windowed_prefill_smem(nq, nv, 2) <= 227 * 1024 ? 2 : 1;
+  const int smem = windowed_prefill_smem(nq, nv, p_bufs);
+  if (smem > 227 * 1024) return -1;
+  const WindowedPrefill z = {H, G, d, dv, nq, nv, p_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale};
+  CUtensorMap tm_q, tm_k, tm_v;
+  const uint64_t qw = static_cast<uint64_t>(H) * qcols, rows = static_cast<uint64_t>(num_blocks) * G * block_size;
+  if (forge_make_tmap_2d(&tm_q, q, tokens, qw, qw, kXM, 2) != 0) return -2;
+  if (forge_make_tmap_2d(&tm_k, k_cache, rows, d, d, kXN, 2) != 0) return -2;
+  if (forge_make_tmap_2d(&tm_v, v_cache, rows, dv, dv, kXN, 2) != 0) return -2;
+  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel, 227 * 1024);
+  return launch_kernel(windowed_prefill_kernel, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v,
+                       cu_q, context_lens, tables, static_cast<bf16*>(out), z, status) == cudaSuccess ? 0 : -5;
+}
+
+}  // namespace forge
