@@ -1,10 +1,12 @@
-// Retention over runs of tokens on the tensor cores, 64 tokens at a time (bf16 projections, fp32 state).
+// Retention, and the state-space recurrence (recurrence.cuh), over runs of tokens on the tensor cores, 64 tokens at a time (bf16
+// operands, fp32 state).
 //
 // With g the head's decay and S the state before a chunk of L tokens:
 //
 //   o_i = g^(i+1) S^T q_i + sum_{j <= i} g^(i-j) (q_i . k_j) v_j            S <- g^L S + sum_j g^(L-1-j) k_j v_j^T
 //
-// (k_j carries dim^-1/2, applied in fp32 to the weights).  Everything of the recurrence stays in fp32: the state lives in
+// (k_j carries dim^-1/2, applied in fp32 to the weights).  The state-space form (kGated) has a decay per token: with c_i the running
+// sum of the logarithms of the decays in the chunk, g^(i-j) becomes exp(c_i - c_j), k_j carries dt_j instead, and D x_i is added.  Everything of the recurrence stays in fp32: the state lives in
 // accumulator registers; where it, the decayed scores or the decayed keys are operands of a product they enter as bf16
 // hi + lo halves (two products, 16 mantissa bits).  q and k come rotated (retention_rotate, in place).
 //
@@ -14,16 +16,23 @@
 // state, and then all segments compute their outputs at the same time.
 #include "../include/launch.cuh"
 #include "../include/mma_sync.cuh"
-#include "../include/scalar.cuh"
+#include "../include/recurrence.cuh"
 
 namespace forge {
 
 constexpr int kRC = 64, kRPP = kRC + 8;      // tokens per chunk; row pitch of the decayed scores (odd number of 16-byte units)
 
 struct RetentionChunk {
-  const bf16* qkvg;         // [tokens][ld], q and k rotated
-  int ld;
-  const float* decay;
+  const bf16* q;            // [tokens][ld] (rotated), head h at (h / share) * dk
+  const bf16* k;            // the same
+  const bf16* v;            // [tokens][ld], head h at h * dv
+  int ld, share;
+  const float* decay;       // one per head, or
+  const float* cum;         // [heads][ldt]: running sum of log2 of the decays in the token's chunk,
+  const float* weight;      // [heads][ldt]: the factor of k_j,
+  long long ldt;
+  const float* skip;        // [heads]: the factor of v_i in o_i,
+  float* seg_decay;         // [seqs][segs][heads]: log2 of a segment's decay
   float* state;             // [slots][heads][dk][dv]
   const int* slots;         // [seqs]
   const int* positions;     // [tokens]
@@ -45,7 +54,7 @@ __device__ __forceinline__ void weigh_split(const uint32_t* a, float w0, float w
 }
 
 // kWide: 16 warps, 128 columns, two stages; else 8 warps, 64 columns, one stage.  MT: 16-row tiles of the state per warp.
-template <int MT, bool kStateOnly, bool kWide>
+template <int MT, bool kStateOnly, bool kWide, bool kGated>
 __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) retention_chunk_kernel(const RetentionChunk p) {
   constexpr int kWarps = kWide ? 16 : 8, kQuarters = kWarps / 4, kCols = 32 * kQuarters, kRPitch = kCols + 8, kStages = kWide ? 2 : 1;
   constexpr int kKB = 8 / kQuarters;                                   // 8-key blocks of the scores per warp
@@ -54,7 +63,7 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
   const int stage = kRC * (2 * kp + kRPitch);                          // elements: q [64][kp], k [64][kp], v [64][kRPitch]
   bf16* sS = reinterpret_cast<bf16*>(smem_raw) + kStages * stage;      // [hi, lo][dk][kRPitch]
   bf16* sP = sS + 2 * p.dk * kRPitch;                                  // [hi, lo][64][kRPP]
-  float* pw = reinterpret_cast<float*>(sP + 2 * kRC * kRPP);           // [65]: g^i
+  float* pw = reinterpret_cast<float*>(sP + 2 * kRC * kRPP);           // [65]: g^i; kGated: [stages][c_i, weight][64]
 
   pdl_launch_dependents();
   pdl_wait();
@@ -72,7 +81,8 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g4 = lane >> 2, q2 = 2 * (lane & 3);
   const float ks = rsqrtf(static_cast<float>(p.dk));
-  if (threadIdx.x <= kRC) pw[threadIdx.x] = powf(p.decay[h], static_cast<float>(threadIdx.x));
+  if (!kGated && threadIdx.x <= kRC) pw[threadIdx.x] = powf(p.decay[h], static_cast<float>(threadIdx.x));
+  float total = 0.f;                                                   // log2 of the decay so far (kGated)
 
   const int steps = p.dk >> 4;
   const bool both = steps > 4;                     // a warp owns two 32-column parts of its state rows, or one
@@ -105,18 +115,24 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
     bf16* sv = sk + kRC * kp;
     for (int r = warp; r < kRC; r += kWarps) {
       const bool in = t0 + r < t_end;
-      const bf16* row = p.qkvg + static_cast<size_t>(in ? t0 + r : t0) * p.ld;
-      const bf16* qr = row + h * p.dk;
-      const bf16* kr = row + (p.heads + h) * p.dk;
-      const bf16* vr = row + 2 * p.heads * p.dk + h * p.dv + c0;
+      const size_t row = static_cast<size_t>(in ? t0 + r : t0) * p.ld;
+      const bf16* qr = p.q + row + (h / p.share) * p.dk;
+      const bf16* kr = p.k + row + (h / p.share) * p.dk;
+      const bf16* vr = p.v + row + h * p.dv + c0;
       for (int u = lane; u < units; u += 32) {
         if (!kStateOnly) cp_async16(smem_u32(sq + r * kp + u * 8), qr + u * 8, in ? 16 : 0);
         cp_async16(smem_u32(sk + r * kp + u * 8), kr + u * 8, in ? 16 : 0);
       }
       if (lane < kCols / 8) {
         const bool vin = in && c0 + lane * 8 < p.dv;
-        cp_async16(smem_u32(sv + r * kRPitch + lane * 8), vin ? vr + lane * 8 : row, vin ? 16 : 0);
+        cp_async16(smem_u32(sv + r * kRPitch + lane * 8), vin ? vr + lane * 8 : qr, vin ? 16 : 0);
       }
+    }
+    if (kGated && threadIdx.x < 2 * kRC) {
+      const int r = threadIdx.x & (kRC - 1);
+      const bool in = t0 + r < t_end;
+      const float* src = (threadIdx.x < kRC ? p.cum : p.weight) + h * p.ldt + (in ? t0 + r : t0);
+      cp_async4(smem_u32(pw + st * 2 * kRC + threadIdx.x), src, in ? 4 : 0);
     }
   };
   if (kStages == 2) {
@@ -124,6 +140,7 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
     cp_async_commit();
   }
   int st_now = 0;
+  const float skip = kGated ? p.skip[h] : 0.f;
   for (int t0 = t_begin; t0 < t_end; t0 += kRC) {
     const int L = min(kRC, t_end - t0);
     __syncthreads();                                                   // the chunk before is done with shared memory
@@ -133,6 +150,8 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
     const bf16* sq = reinterpret_cast<bf16*>(smem_raw) + st_now * stage;
     const bf16* sk = sq + kRC * kp;
     const bf16* sv = sk + kRC * kp;
+    const float* cum = pw + st_now * 2 * kRC;
+    const float* wgt = cum + kRC;
     st_now ^= kStages - 1;
     if (!kStateOnly) {                                                 // the state before this chunk as hi and lo operands
 #pragma unroll
@@ -191,17 +210,24 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
 #pragma unroll
         for (int nb = 0; nb < kKB; ++nb) {
           const int j = nh * 8 * kKB + nb * 8 + q2;
-          const float x = j <= i ? s[nb][2 * e] * (pw[i - j] * ks) : 0.f;
-          const float y = j + 1 <= i ? s[nb][2 * e + 1] * (pw[i - j - 1] * ks) : 0.f;
+          float x = 0.f, y = 0.f;
+          if (kGated) {
+            if (j <= i) x = s[nb][2 * e] * (ex2_approx(cum[i] - cum[j]) * wgt[j]);
+            if (j + 1 <= i) y = s[nb][2 * e + 1] * (ex2_approx(cum[i] - cum[j + 1]) * wgt[j + 1]);
+          } else {
+            if (j <= i) x = s[nb][2 * e] * (pw[i - j] * ks);
+            if (j + 1 <= i) y = s[nb][2 * e + 1] * (pw[i - j - 1] * ks);
+          }
           const uint32_t hi = pack_bf16x2(x, y);
           bf16* dst = sP + i * kRPP + j;
           *reinterpret_cast<uint32_t*>(dst) = hi;
           *reinterpret_cast<uint32_t*>(dst + kRC * kRPP) = pack_bf16x2(x - bf16_lo(hi), y - bf16_hi(hi));
         }
+        const float past = kGated ? ex2_approx(cum[i]) : pw[i + 1];
 #pragma unroll
         for (int nb = 0; nb < 4; ++nb) {
-          o[nb][2 * e] *= pw[i + 1];
-          o[nb][2 * e + 1] *= pw[i + 1];
+          o[nb][2 * e] *= past;
+          o[nb][2 * e + 1] *= past;
         }
       }
       __syncthreads();
@@ -225,12 +251,18 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int i = mt * 16 + g4 + e * 8, c = c0 + nh * 32 + nb * 8 + q2;
+          if (kGated) {
+            const uint32_t x = *reinterpret_cast<const uint32_t*>(sv + i * kRPitch + nh * 32 + nb * 8 + q2);
+            o[nb][2 * e] = fmaf(skip, bf16_lo(x), o[nb][2 * e]);
+            o[nb][2 * e + 1] = fmaf(skip, bf16_hi(x), o[nb][2 * e + 1]);
+          }
           if (i < L && c < p.dv)
             *reinterpret_cast<float2*>(p.o + (static_cast<size_t>(t0 + i) * p.heads + h) * p.dv + c) = make_float2(o[nb][2 * e], o[nb][2 * e + 1]);
         }
     }
 
-    const float keep = pw[L];
+    const float keep = kGated ? ex2_approx(cum[L - 1]) : pw[L];
+    if (kGated) total += cum[L - 1];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -246,7 +278,7 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int j = k * 16 + q2 + (e & 1) + (e >> 1) * 8;
-        w[e] = j < L ? pw[L - 1 - j] * ks : 0.f;
+        w[e] = j >= L ? 0.f : kGated ? ex2_approx(cum[L - 1] - cum[j]) * wgt[j] : pw[L - 1 - j] * ks;
       }
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
@@ -271,6 +303,8 @@ __global__ void __launch_bounds__(kWide ? 512 : 256, kWide || MT == 2 ? 1 : 2) r
     }
   }
 
+  if (kGated && kStateOnly && blockIdx.x == 0 && threadIdx.x == 0)
+    p.seg_decay[(static_cast<size_t>(seq) * p.segs + seg) * p.heads + h] = total;
   float* dst = kStateOnly ? seg_state : (seg == n_segs - 1 ? slot_state : nullptr);
   if (dst == nullptr) return;
 #pragma unroll
@@ -298,7 +332,7 @@ __global__ void __launch_bounds__(256) retention_segments_kernel(const Retention
   const int n_segs = min((run + p.seg_len - 1) / p.seg_len, p.segs);
   const int n = p.dk * p.dv, i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
   if (i >= n) return;
-  const float g = powf(p.decay[h], static_cast<float>(p.seg_len));
+  const float g = p.cum != nullptr ? 0.f : powf(p.decay[h], static_cast<float>(p.seg_len));
   float s[4] = {0.f, 0.f, 0.f, 0.f};
   if (p.positions[p.cu[seq]] != 0) load_n<4>(p.state + (static_cast<size_t>(slot) * p.heads + h) * n + i, s);
   for (int seg = 0; seg < n_segs; ++seg) {
@@ -307,8 +341,9 @@ __global__ void __launch_bounds__(256) retention_segments_kernel(const Retention
     if (seg + 1 < n_segs) load_n<4>(w, own);
     store_n<4>(w, s);
     if (seg + 1 < n_segs) {
+      const float f = p.cum != nullptr ? exp2f(p.seg_decay[(static_cast<size_t>(seq) * p.segs + seg) * p.heads + h]) : g;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[e] = fmaf(g, s[e], own[e]);
+      for (int e = 0; e < 4; ++e) s[e] = fmaf(f, s[e], own[e]);
     }
   }
 }
@@ -342,7 +377,7 @@ __global__ void __launch_bounds__(128) retention_rotate_kernel(bf16* __restrict_
 
 static size_t retention_chunk_smem(int dk, bool wide) {
   const int pitch = wide ? 136 : 72;
-  return static_cast<size_t>((wide ? 2 : 1) * kRC * (2 * (dk + 8) + pitch) + 2 * dk * pitch + 2 * kRC * kRPP) * 2 + (kRC + 1) * 4;
+  return static_cast<size_t>((wide ? 2 : 1) * kRC * (2 * (dk + 8) + pitch) + 2 * dk * pitch + 2 * kRC * kRPP) * 2 + 4 * kRC * 4;
 }
 
 // Value columns per CTA for these sizes.
@@ -351,6 +386,27 @@ extern "C" int forge_retention_chunk_cols(int dk, int dv) { return dk <= 128 && 
 // 1 if the kernels take these sizes (else: retention_scan).
 extern "C" int forge_retention_chunk_ok(int heads, int dk, int dv, int rd) {
   return dk % 16 == 0 && dk >= 16 && dk <= 256 && dv % 8 == 0 && rd % 8 == 0 && heads > 0 && (2 * heads * (dk + dv)) % 8 == 0;
+}
+
+template <bool kGated>
+static int run_chunks(const RetentionChunk& p, int seqs, cudaStream_t stream) {
+  const int cols = forge_retention_chunk_cols(p.dk, p.dv);
+  const bool wide = cols == 128;
+  const dim3 grid((p.dv + cols - 1) / cols, p.heads, seqs * p.segs);
+  const size_t smem = retention_chunk_smem(p.dk, wide);
+#define FORGE_RC(MT, ONLY, WIDE)                                                                                           \
+  {                                                                                                                        \
+    auto k = retention_chunk_kernel<MT, ONLY, WIDE, kGated>;                                                               \
+    FORGE_ENSURE_DYN_SMEM(k, static_cast<int>(retention_chunk_smem(128 * MT, WIDE)));                                      \
+    if (launch_kernel(k, grid, dim3(WIDE ? 512 : 256), smem, stream, 0, p) != cudaSuccess) return -2;                      \
+  }
+  if (p.segs > 1) {
+    if (wide) FORGE_RC(1, true, true) else if (p.dk <= 128) FORGE_RC(1, true, false) else FORGE_RC(2, true, false)
+    if (launch_kernel(retention_segments_kernel, dim3((p.dk * p.dv / 4 + 255) / 256, p.heads, seqs), dim3(256), 0, stream, 0, p) != cudaSuccess) return -2;
+  }
+  if (wide) FORGE_RC(1, false, true) else if (p.dk <= 128) FORGE_RC(1, false, false) else FORGE_RC(2, false, false)
+#undef FORGE_RC
+  return 0;
 }
 
 // Rotates q and k of qkvg in place, then runs sequence s over the step's tokens cu[s] .. cu[s + 1] (cu[0] == tok0, cu[seqs] == tokens).
@@ -366,24 +422,72 @@ extern "C" int forge_retention_chunk(void* qkvg, int ld, const float* decay, flo
   if (rd > 0 && launch_kernel(retention_rotate_kernel, dim3(tokens - tok0), dim3(128), 0, stream, 0, static_cast<bf16*>(qkvg), ld, tok0, 2 * heads,
                               dk, rd, rope, rope_rows, positions) != cudaSuccess)
     return -2;
-  const RetentionChunk p = {static_cast<const bf16*>(qkvg), ld, decay, state, slots, positions, cu, ws, o, heads, dk, dv, num_slots, segs, seg_len, status};
-  const int cols = forge_retention_chunk_cols(dk, dv);
-  const bool wide = cols == 128;
-  const dim3 grid((dv + cols - 1) / cols, heads, seqs * segs);
-  const size_t smem = retention_chunk_smem(dk, wide);
-#define FORGE_RC(MT, ONLY, WIDE)                                                                                           \
-  {                                                                                                                        \
-    auto k = retention_chunk_kernel<MT, ONLY, WIDE>;                                                                       \
-    FORGE_ENSURE_DYN_SMEM(k, static_cast<int>(retention_chunk_smem(128 * MT, WIDE)));                                      \
-    if (launch_kernel(k, grid, dim3(WIDE ? 512 : 256), smem, stream, 0, p) != cudaSuccess) return -2;                      \
+  const bf16* rows = static_cast<const bf16*>(qkvg);
+  return run_chunks<false>({rows, rows + heads * dk, rows + 2 * heads * dk, ld, 1, decay, nullptr, nullptr, 0, nullptr, nullptr, state, slots, positions,
+                            cu, ws, o, heads, dk, dv, num_slots, segs, seg_len, status}, seqs, stream);
+}
+
+// The same for the state-space recurrence: q, k [tokens][ld] with head h at (h / share) * dk, v with head h at h * dv; cum, weight
+// [heads][ldt] as recurrence_gates leaves them.
+extern "C" int forge_state_space_chunk(const void* q, const void* k, const void* v, long long ld, int share, const float* cum, const float* weight,
+                                       long long ldt, const float* skip, float* state, const int* slots, const int* positions, const int* cu,
+                                       int seqs, int heads, int dk, int dv, int num_slots, float* o, float* ws, float* seg_decay, int segs,
+                                       int seg_len, unsigned* status, cudaStream_t stream) {
+  if (seqs <= 0) return 0;
+  const uintptr_t any = reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v);
+  if (!forge_retention_chunk_ok(heads, dk, dv, 0) || segs < 1 || static_cast<long long>(seqs) * segs > 65535 || (ld & 7) || ld >= (1ll << 31) ||
+      (any & 15) || (segs > 1 && (ws == nullptr || seg_decay == nullptr || seg_len < kRC || seg_len % kRC)))
+    return -1;
+  return run_chunks<true>({static_cast<const bf16*>(q), static_cast<const bf16*>(k), static_cast<const bf16*>(v), static_cast<int>(ld), share, nullptr, cum,
+                           weight, ldt, skip, seg_decay, state, slots, positions, cu, ws, o, heads, dk, dv, num_slots, segs, seg_len, status},
+                          seqs, stream);
+}
+
+// CTA = (64-token chunk of a sequence's run, sequence); a warp takes a head at a time, a lane two tokens.
+template <typename T>
+__global__ void __launch_bounds__(256) recurrence_gates_kernel(const Recurrence<T> p, const int* __restrict__ cu, float* __restrict__ cum,
+                                                               float* __restrict__ weight, long long ldt) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int s = blockIdx.y, t0 = cu[s] + blockIdx.x * kRC, end = min(cu[s + 1], t0 + kRC);
+  if (t0 >= end) return;
+  const int lane = threadIdx.x & 31, a = t0 + 2 * lane;
+  for (int h = threadIdx.x >> 5; h < p.heads; h += blockDim.x >> 5) {
+    TokenGates x = {0.f, 0.f}, y = {0.f, 0.f};
+    if (a < end) x = token_gates(p, a, h);
+    if (a + 1 < end) y = token_gates(p, a + 1, h);
+    float sum = x.log_g + y.log_g;
+#pragma unroll
+    for (int off = 1; off < 32; off <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, sum, off);
+      if (lane >= off) sum += v;
+    }
+    const float before = sum - y.log_g;
+    if (a < end) {
+      cum[h * ldt + a] = before * 1.4426950408889634f;
+      weight[h * ldt + a] = x.w;
+    }
+    if (a + 1 < end) {
+      cum[h * ldt + a + 1] = sum * 1.4426950408889634f;
+      weight[h * ldt + a + 1] = y.w;
+    }
   }
-  if (segs > 1) {
-    if (wide) FORGE_RC(1, true, true) else if (dk <= 128) FORGE_RC(1, true, false) else FORGE_RC(2, true, false)
-    if (launch_kernel(retention_segments_kernel, dim3((dk * dv / 4 + 255) / 256, heads, seqs), dim3(256), 0, stream, 0, p) != cudaSuccess) return -2;
-  }
-  if (wide) FORGE_RC(1, false, true) else if (dk <= 128) FORGE_RC(1, false, false) else FORGE_RC(2, false, false)
-#undef FORGE_RC
-  return 0;
+}
+
+// cum, weight [heads][ldt] for the tokens of the runs: the running sum of log2 of the decays within 64-token chunks counted from
+// the run's first token, and dt (state-space) or beta (delta).
+extern "C" int forge_recurrence_gates(const void* dt, const void* beta, long long ld_raw, const float* A_log, const float* dt_bias, const int* cu,
+                                      int seqs, int max_q, int heads, float* cum, float* weight, long long ldt, cudaStream_t stream) {
+  if (seqs <= 0 || max_q <= 0) return 0;
+  if (seqs > 65535) return -1;
+  Recurrence<bf16> p = {};
+  p.dt = static_cast<const bf16*>(dt);
+  p.beta = static_cast<const bf16*>(beta);
+  p.ld_raw = ld_raw;
+  p.A_log = A_log;
+  p.dt_bias = dt_bias;
+  p.heads = heads;
+  return launch_kernel(recurrence_gates_kernel<bf16>, dim3((max_q + kRC - 1) / kRC, seqs), dim3(256), 0, stream, 0, p, cu, cum, weight, ldt) == cudaSuccess ? 0 : -2;
 }
 
 }  // namespace forge

@@ -17,6 +17,27 @@ int forge_recurrence(int fp32, const void* q, const void* k, const void* v, long
                      const float* A_log, const float* dt_bias, const float* D, float* state, const int* slots, const int* positions,
                      const int* cu, int seqs, int heads, int share, int dk, int dv, int num_slots, float* o, unsigned* status,
                      cudaStream_t stream);
+int forge_windowed_decode_ok(int d, int dv, int block_size);
+int forge_windowed_decode(const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* tables, const int* lens, int seqs,
+                          int width, int num_blocks, int block_size, void* out, long long ldo, float* part_o, float* part_ml, int chunk,
+                          int max_chunks, int H, int G, int d, int dv, int window, float scale, float out_scale, unsigned* status,
+                          cudaStream_t stream);
+int forge_windowed_prefill_qcols(int d, int dv, int block_size);
+int forge_windowed_prefill(const void* q, int tokens, const void* k_cache, const void* v_cache, const int* cu_q, const int* context_lens,
+                           const int* tables, int table_width, int num_blocks, int block_size, void* out, long long ldo, int num_seqs, int max_q,
+                           int H, int G, int d, int dv, int window, float scale, float out_scale, unsigned* status, cudaStream_t stream);
+int forge_recurrence_gates(const void* dt, const void* beta, long long ld_raw, const float* A_log, const float* dt_bias, const int* cu, int seqs,
+                           int max_q, int heads, float* cum, float* weight, long long ldt, cudaStream_t stream);
+int forge_retention_chunk_ok(int heads, int dk, int dv, int rd);
+int forge_state_space_chunk(const void* q, const void* k, const void* v, long long ld, int share, const float* cum, const float* weight,
+                            long long ldt, const float* skip, float* state, const int* slots, const int* positions, const int* cu, int seqs,
+                            int heads, int dk, int dv, int num_slots, float* o, float* ws, float* seg_decay, int segs, int seg_len,
+                            unsigned* status, cudaStream_t stream);
+int forge_delta_chunk_ok(int dk, int dv);
+long long forge_delta_chunk_scratch(int tokens, int seqs, int heads, int which);
+int forge_delta_chunk(const void* q, const void* k, const void* v, long long ld, int share, const float* cum, const float* beta, long long ldt,
+                      float* state, const int* slots, const int* positions, const int* cu, int seqs, int max_q, int heads, int dk, int dv,
+                      int num_slots, void* mats, float* factors, float* o, unsigned* status, cudaStream_t stream);
 int forge_gated_norm(int fp32, const float* o, const void* gate, long long ldg, const float* weight, int weight_period, void* out, long long ldo,
                      int tokens, int groups, int n, int gate_first, float factor, float eps, cudaStream_t stream);
 }
@@ -77,6 +98,42 @@ void windowed_attend_any(const Tensor& q, const Tensor& k_cache, const Tensor& v
            "forge_windowed_attend_any");
 }
 
+constexpr auto kBf16 = at::kBFloat16;
+
+// One token per sequence: rows 0 .. seqs - 1 of q and out.
+void windowed_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& tables, const Tensor& lens, int64_t seqs,
+                     Tensor& out, const OptTensor& part_o, const OptTensor& part_ml, int64_t chunk, int64_t max_chunks, int64_t window,
+                     double scale, double out_scale, const Tensor& status) {
+  TORCH_CHECK(q.scalar_type() == kBf16 && seqs <= q.size(0), "windowed_decode: q");
+  const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
+  float *po = nullptr, *pm = nullptr;
+  if (max_chunks > 1) {
+    TORCH_CHECK(part_o.has_value() && part_ml.has_value(), "windowed_decode: scratch");
+    po = floats(*part_o, seqs * a.H * max_chunks * a.c.dv, "part_o");
+    pm = floats(*part_ml, seqs * a.H * max_chunks * 2, "part_ml");
+  }
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_rc(forge_windowed_decode(q.data_ptr(), i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), ints(tables, 0, "tables"), ints(lens, seqs, "lens"),
+                                 i32(seqs), i32(tables.size(1)), i32(a.c.blocks), i32(a.c.block_size), out.data_ptr(), out.stride(0), po, pm, i32(chunk),
+                                 i32(max_chunks), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window), static_cast<float>(scale),
+                                 static_cast<float>(out_scale), status_word(status), stream_of(q)),
+           "forge_windowed_decode");
+}
+
+// Sequence s: the rows cu[s] .. cu[s + 1] of q and out, its last ones; context_lens[s] keys.
+void windowed_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu, const Tensor& context_lens, const Tensor& tables,
+                      int64_t seqs, int64_t max_q, Tensor& out, int64_t window, double scale, double out_scale, const Tensor& status) {
+  TORCH_CHECK(q.scalar_type() == kBf16, "windowed_prefill: q");
+  const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
+  TORCH_CHECK(q.size(2) == forge_windowed_prefill_qcols(i32(a.c.d), i32(a.c.dv), i32(a.c.block_size)), "windowed_prefill: q columns");
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_rc(forge_windowed_prefill(q.data_ptr(), i32(a.T), k_cache.data_ptr(), v_cache.data_ptr(), ints(cu, seqs + 1, "cu"), ints(context_lens, seqs, "lens"),
+                                  ints(tables, 0, "tables"), i32(tables.size(1)), i32(a.c.blocks), i32(a.c.block_size), out.data_ptr(), out.stride(0),
+                                  i32(seqs), i32(max_q), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window), static_cast<float>(scale),
+                                  static_cast<float>(out_scale), status_word(status), stream_of(q)),
+           "forge_windowed_prefill");
+}
+
 // x [tokens, channels] (a view), taps [channels, n], state [slots, n - 1, channels], out [tokens, channels]
 void short_conv(const Tensor& x, const Tensor& taps, const OptTensor& bias, Tensor& state, const Tensor& slots, const Tensor& positions,
                 const Tensor& cu, int64_t seqs, int64_t max_q, Tensor& out, const Tensor& status) {
@@ -130,6 +187,58 @@ void recurrence(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor&
            "forge_recurrence");
 }
 
+// cum, weight fp32 [heads, tokens]
+void recurrence_gates(const Tensor& dt, const OptTensor& beta, const Tensor& A_log, const Tensor& dt_bias, const Tensor& cu, int64_t seqs, int64_t max_q,
+                      Tensor& cum, Tensor& weight) {
+  TORCH_CHECK(cum.dim() == 2 && weight.sizes() == cum.sizes(), "recurrence_gates: ranks");
+  const int64_t H = cum.size(0), T = cum.size(1);
+  view2(dt, kBf16, T, H, "dt");
+  if (beta.has_value()) {
+    view2(*beta, kBf16, T, H, "beta");
+    TORCH_CHECK(beta->stride(0) == dt.stride(0), "recurrence_gates: row strides");
+  }
+  const c10::cuda::CUDAGuard guard(dt.device());
+  check_rc(forge_recurrence_gates(dt.data_ptr(), beta.has_value() ? beta->data_ptr() : nullptr, dt.stride(0), floats(A_log, H, "A_log"),
+                                  floats(dt_bias, H, "dt_bias"), ints(cu, seqs + 1, "cu"), i32(seqs), i32(max_q), i32(H), floats(cum, H * T, "cum"),
+                                  floats(weight, H * T, "weight"), T, stream_of(dt)),
+           "forge_recurrence_gates");
+}
+
+// The runs cu[s] .. cu[s + 1]; q, k, v as in recurrence; cum, weight from recurrence_gates; o fp32 [tokens, heads, dv]
+void state_space_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& cum, const Tensor& weight, const Tensor& skip, Tensor& state,
+                       const Tensor& slots, const Tensor& positions, const Tensor& cu, int64_t seqs, Tensor& o, const OptTensor& ws,
+                       const OptTensor& seg_decay, int64_t segs, int64_t seg_len, const Tensor& status) {
+  TORCH_CHECK(q.scalar_type() == kBf16 && state.dim() == 4 && cum.dim() == 2 && cum.size(0) == state.size(1) && cum.size(1) == q.size(0), "state_space_chunk: sizes");
+  const Rec r = recurrence_sizes(q, k, v, v.slice(1, 0, state.size(1)), c10::nullopt, state);
+  float *wp = nullptr, *sp = nullptr;
+  if (segs > 1) {
+    TORCH_CHECK(ws.has_value() && seg_decay.has_value(), "state_space_chunk: scratch");
+    wp = floats(*ws, seqs * segs * r.H * r.dk * r.dv, "ws");
+    sp = floats(*seg_decay, seqs * segs * r.H, "seg_decay");
+  }
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_rc(forge_state_space_chunk(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), i32(r.share), floats(cum, r.H * r.T, "cum"),
+                                   floats(weight, r.H * r.T, "weight"), r.T, floats(skip, r.H, "skip"), floats(state, 0, "state"),
+                                   ints(slots, seqs, "slots"), ints(positions, r.T, "positions"), ints(cu, seqs + 1, "cu"), i32(seqs), i32(r.H),
+                                   i32(r.dk), i32(r.dv), i32(r.slots), floats(o, r.T * r.H * r.dv, "o"), wp, sp, i32(segs), i32(seg_len),
+                                   status_word(status), stream_of(q)),
+           "forge_state_space_chunk");
+}
+
+void delta_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& cum, const Tensor& beta, Tensor& state, const Tensor& slots,
+                 const Tensor& positions, const Tensor& cu, int64_t seqs, int64_t max_q, Tensor& mats, Tensor& factors, Tensor& o, const Tensor& status) {
+  TORCH_CHECK(q.scalar_type() == kBf16 && state.dim() == 4 && cum.dim() == 2 && cum.size(0) == state.size(1) && cum.size(1) == q.size(0), "delta_chunk: sizes");
+  const Rec r = recurrence_sizes(q, k, v, v.slice(1, 0, state.size(1)), c10::nullopt, state);
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_rc(forge_delta_chunk(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), i32(r.share), floats(cum, r.H * r.T, "cum"),
+                             floats(beta, r.H * r.T, "beta"), r.T, floats(state, 0, "state"), ints(slots, seqs, "slots"),
+                             ints(positions, r.T, "positions"), ints(cu, seqs + 1, "cu"), i32(seqs), i32(max_q), i32(r.H), i32(r.dk), i32(r.dv),
+                             i32(r.slots), data(mats, kBf16, forge_delta_chunk_scratch(i32(r.T), i32(seqs), i32(r.H), 0), "mats"),
+                             floats(factors, forge_delta_chunk_scratch(i32(r.T), i32(seqs), i32(r.H), 1), "factors"),
+                             floats(o, r.T * r.H * r.dv, "o"), status_word(status), stream_of(q)),
+           "forge_delta_chunk");
+}
+
 // o fp32 [tokens, groups n], gate and out [tokens, groups n] (views); weight fp32, repeated along the row
 void gated_norm(const Tensor& o, const Tensor& gate, const Tensor& weight, Tensor& out, int64_t groups, bool gate_first, double factor, double eps) {
   const int f = elem(gate);
@@ -147,6 +256,16 @@ void gated_norm(const Tensor& o, const Tensor& gate, const Tensor& weight, Tenso
 void register_hybrid(pybind11::module& m) {
   m.def("bias_rope_store", &bias_rope_store);
   m.def("windowed_attend_any", &windowed_attend_any);
+  m.def("windowed_decode", &windowed_decode);
+  m.def("windowed_decode_ok", [](int64_t d, int64_t dv, int64_t bs) { return forge_windowed_decode_ok(i32(d), i32(dv), i32(bs)) != 0; });
+  m.def("windowed_prefill", &windowed_prefill);
+  m.def("windowed_prefill_qcols", [](int64_t d, int64_t dv, int64_t bs) { return forge_windowed_prefill_qcols(i32(d), i32(dv), i32(bs)); });
+  m.def("recurrence_gates", &recurrence_gates);
+  m.def("state_space_chunk", &state_space_chunk);
+  m.def("state_space_chunk_ok", [](int64_t dk, int64_t dv) { return forge_retention_chunk_ok(1, i32(dk), i32(dv), 0) != 0; });
+  m.def("delta_chunk", &delta_chunk);
+  m.def("delta_chunk_ok", [](int64_t dk, int64_t dv) { return forge_delta_chunk_ok(i32(dk), i32(dv)) != 0; });
+  m.def("delta_chunk_scratch", [](int64_t T, int64_t S, int64_t H, int64_t which) { return static_cast<int64_t>(forge_delta_chunk_scratch(i32(T), i32(S), i32(H), i32(which))); });
   m.def("short_conv", &short_conv);
   m.def("recurrence", &recurrence);
   m.def("recurrence_decode_ok", [](int64_t dk, int64_t dv) { return forge_recurrence_decode_ok(i32(dk), i32(dv)) != 0; });
