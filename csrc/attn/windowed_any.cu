@@ -28,82 +28,92 @@ struct QkvArgs {
   unsigned* status;
 };
 
-// CTA = one token.  N entries of a rotated pair half at a time.
-template <typename T, int N>
-__global__ void __launch_bounds__(256) bias_rope_store_kernel(const QkvArgs<T> p) {
+// CTA = kTok tokens.  The work of a token is a list of items of N entries: per query and key head the rotated pairs, then the
+// entries that pass (and a query's padding); then the values.  A thread keeps its item's bias for all tokens.
+template <typename T, int N, int kTok>
+__global__ void __launch_bounds__(512) bias_rope_store_kernel(const QkvArgs<T> p, int tokens, uint32_t magic) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x;
-  const T* row = p.proj + static_cast<size_t>(t) * p.ld;
-  int pos = p.positions[t];
-  pos = pos < 0 ? 0 : (pos >= p.rope_rows ? p.rope_rows - 1 : pos);
-  const float* cs = p.rope + static_cast<size_t>(pos) * p.rd;
-  const long long slot = p.slots[t];
-  const bool store = slot >= 0 && slot < p.num_slots;
-  if (slot >= p.num_slots && threadIdx.x == 0) set_status(p.status, kStatusBadIndex);
-  const int half = p.rd >> 1, heads = p.H + p.G;
-  const size_t blk = store ? slot / p.block_size : 0, off = store ? slot % p.block_size : 0;
-  auto dest = [&](int h) -> T* {
-    if (h < p.H) return p.q + (static_cast<size_t>(t) * p.H + h) * p.q_pitch;
-    return p.k_cache + ((blk * p.G + (h - p.H)) * p.block_size + off) * p.d;
-  };
-  // rotated pairs
-  const int pairs = half / N;
-  for (int i = threadIdx.x; i < heads * pairs; i += blockDim.x) {
-    const int h = i / pairs, c = (i % pairs) * N;
-    const size_t at = static_cast<size_t>(h) * p.d + c;
-    float a[N], b[N], ab[N], bb[N], co[N], si[N], x[N], y[N];
-    load_n<N>(row + at, a);
-    load_n<N>(row + at + half, b);
-    load_n<N>(p.bias + at, ab);
-    load_n<N>(p.bias + at + half, bb);
-    load_n<N>(cs + c, co);
-    load_n<N>(cs + half + c, si);
+  const int half = p.rd >> 1, pairs = half / N, rest = (p.d - p.rd) / N, per = pairs + (p.q_pitch - p.rd) / N, heads = p.H + p.G;
+  const int vper = p.dv / N, items = heads * per + p.G * vper;
+  for (int i = threadIdx.x; i < items; i += blockDim.x) {
+    const bool value = i >= heads * per;
+    const int h = value ? heads + (i - heads * per) / vper : per == 1 ? i : static_cast<int>(__umulhi(static_cast<uint32_t>(i), magic));
+    const int k = value ? (i - heads * per) % vper : i - h * per;
+    const bool pair = !value && k < pairs, pad = !value && k >= pairs + rest, query = h < p.H;
+    if (pad && !query) continue;
+    const int c = value ? k * N : pair ? k * N : p.rd + (k - pairs) * N;
+    const size_t at = value ? static_cast<size_t>(heads) * p.d + static_cast<size_t>(h - heads) * p.dv + c : static_cast<size_t>(h) * p.d + c;
+    float ab[N], bb[N];
 #pragma unroll
-    for (int e = 0; e < N; ++e) {
-      a[e] += ab[e];
-      b[e] += bb[e];
-      x[e] = a[e] * co[e] - b[e] * si[e];
-      y[e] = b[e] * co[e] + a[e] * si[e];
+    for (int e = 0; e < N; ++e) ab[e] = bb[e] = 0.f;
+    if (!pad) load_n<N>(p.bias + at, ab);
+    if (pair) load_n<N>(p.bias + at + half, bb);
+#pragma unroll
+    for (int u = 0; u < kTok; ++u) {
+      const int t = blockIdx.x * kTok + u;
+      if (t >= tokens) break;
+      const T* src = p.proj + static_cast<size_t>(t) * p.ld + at;
+      T* dst;
+      if (query) {
+        dst = p.q + (static_cast<size_t>(t) * p.H + h) * p.q_pitch + c;
+      } else {
+        const long long slot = p.slots[t];
+        if (slot < 0) continue;
+        if (slot >= p.num_slots) {
+          set_status(p.status, kStatusBadIndex);
+          continue;
+        }
+        const size_t blk = slot / p.block_size, off = slot % p.block_size;
+        dst = value ? p.v_cache + ((blk * p.G + (h - heads)) * p.block_size + off) * p.dv + c
+                    : p.k_cache + ((blk * p.G + (h - p.H)) * p.block_size + off) * p.d + c;
+      }
+      float a[N];
+#pragma unroll
+      for (int e = 0; e < N; ++e) a[e] = 0.f;
+      if (!pad) load_n<N>(src, a);
+#pragma unroll
+      for (int e = 0; e < N; ++e) a[e] += ab[e];
+      if (pair) {
+        int pos = p.positions[t];
+        pos = pos < 0 ? 0 : (pos >= p.rope_rows ? p.rope_rows - 1 : pos);
+        const float* cs = p.rope + static_cast<size_t>(pos) * p.rd + c;
+        float b[N], co[N], si[N], y[N];
+        load_n<N>(src + half, b);
+        load_n<N>(cs, co);
+        load_n<N>(cs + half, si);
+#pragma unroll
+        for (int e = 0; e < N; ++e) {
+          b[e] += bb[e];
+          y[e] = b[e] * co[e] + a[e] * si[e];
+          a[e] = a[e] * co[e] - b[e] * si[e];
+        }
+        store_n<N>(dst + half, y);
+      }
+      store_n<N>(dst, a);
     }
-    if (h < p.H || store) {
-      T* dst = dest(h) + c;
-      store_n<N>(dst, x);
-      store_n<N>(dst + half, y);
-    }
   }
-  // the entries that pass, and the padding of q
-  const int rest = p.d - p.rd, per = rest / N;
-  for (int i = threadIdx.x; i < heads * per; i += blockDim.x) {
-    const int h = i / per, c = p.rd + (i % per) * N;
-    const size_t at = static_cast<size_t>(h) * p.d + c;
-    float a[N], b[N];
-    load_n<N>(row + at, a);
-    load_n<N>(p.bias + at, b);
-#pragma unroll
-    for (int e = 0; e < N; ++e) a[e] += b[e];
-    if (h < p.H || store) store_n<N>(dest(h) + c, a);
-  }
-  const int pad = p.q_pitch - p.d;
-  for (int i = threadIdx.x; i < p.H * pad; i += blockDim.x) store_f(dest(i / pad) + p.d + i % pad, 0.f);
-  // values
-  if (!store) return;
-  const int vat = heads * p.d, vper = p.dv / N;
-  for (int i = threadIdx.x; i < p.G * vper; i += blockDim.x) {
-    const int g = i / vper, c = (i % vper) * N;
-    float a[N], b[N];
-    load_n<N>(row + vat + g * p.dv + c, a);
-    load_n<N>(p.bias + vat + g * p.dv + c, b);
-#pragma unroll
-    for (int e = 0; e < N; ++e) a[e] += b[e];
-    store_n<N>(p.v_cache + ((blk * p.G + g) * p.block_size + off) * p.dv + c, a);
-  }
+}
+
+template <typename T, int N>
+static int bias_rope_store_n(const QkvArgs<T>& p, int tokens, cudaStream_t stream) {
+  const int per = (p.rd >> 1) / N + (p.q_pitch - p.rd) / N, items = (p.H + p.G) * per + p.G * (p.dv / N);
+  if (per < 1) return -1;
+  const uint32_t magic = per == 1 ? 0u : static_cast<uint32_t>(((1ull << 32) + per - 1) / per);    // exact for the item counts of a token
+  const int threads = items >= 512 ? 512 : ((items + 31) / 32) * 32;
+  if (static_cast<long long>(items) * per >= (1ll << 32)) return -1;
+  if (tokens >= 2048)
+    return launch_kernel(bias_rope_store_kernel<T, N, 4>, dim3((tokens + 3) / 4), dim3(threads), 0, stream, 0, p, tokens, magic) == cudaSuccess ? 0 : -2;
+  return launch_kernel(bias_rope_store_kernel<T, N, 1>, dim3(tokens), dim3(threads), 0, stream, 0, p, tokens, magic) == cudaSuccess ? 0 : -2;
 }
 
 template <typename T>
 static int bias_rope_store(const QkvArgs<T>& p, int tokens, cudaStream_t stream) {
-  const bool v4 = ((p.rd >> 1) & 3) == 0 && ((p.d | p.dv | p.q_pitch) & 3) == 0 && (p.ld & 3) == 0 && (reinterpret_cast<uintptr_t>(p.proj) & (4 * sizeof(T) - 1)) == 0;
-  return launch_kernel(v4 ? bias_rope_store_kernel<T, 4> : bias_rope_store_kernel<T, 1>, dim3(tokens), dim3(256), 0, stream, 0, p) == cudaSuccess ? 0 : -2;
+  const uintptr_t proj = reinterpret_cast<uintptr_t>(p.proj);
+  const int all = (p.rd >> 1) | p.d | p.dv | p.q_pitch | static_cast<int>(p.ld & 7);
+  if (sizeof(T) == 2 && (all & 7) == 0 && (proj & 15) == 0) return bias_rope_store_n<T, 8>(p, tokens, stream);
+  if ((all & 3) == 0 && (proj & (4 * sizeof(T) - 1)) == 0) return bias_rope_store_n<T, 4>(p, tokens, stream);
+  return bias_rope_store_n<T, 1>(p, tokens, stream);
 }
 
 extern "C" int forge_bias_rope_store(int fp32, const void* proj, long long ld, int tokens, const float* bias, const float* rope, int rope_rows,

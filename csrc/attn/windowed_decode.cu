@@ -52,6 +52,17 @@ __device__ __forceinline__ WindowRange window_range(const WindowedDecode& p, int
   return r;
 }
 
+// 16 rows of `cols` elements: 2^lanes_log2 lanes to a row, a 16-byte unit each.
+__device__ __forceinline__ void wd_load_rows(uint32_t dst, int pitch, const bf16* src, int cols, int lanes_log2, int lane) {
+  const int u = lane & ((1 << lanes_log2) - 1), r0 = lane >> lanes_log2, step = 32 >> lanes_log2;
+  if (u * 8 >= cols) return;
+  dst += (r0 * pitch + u * 8) * 2;
+  src += r0 * cols + u * 8;
+#pragma unroll 8
+  for (int r = r0; r < kWDKeys; r += step, dst += step * pitch * 2, src += step * cols) cp_async16(dst, src, 16);
+}
+__device__ __forceinline__ int wd_lanes_log2(int units) { return units <= 1 ? 0 : 32 - __clz(units - 1); }
+
 template <int NV>           // blocks of 8 value columns
 __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const WindowedDecode p) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -74,7 +85,7 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
         p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h0) * p.dv + i] = __float2bfloat16_rn(0.f);
     return;
   }
-  const int dpad = (p.d + 15) & ~15, ku = p.d >> 3, vu = p.dv >> 3, qu = dpad >> 3;
+  const int dpad = (p.d + 15) & ~15, ku = p.d >> 3, qu = dpad >> 3, kl = wd_lanes_log2(ku), vl = wd_lanes_log2(p.dv >> 3);
   for (int i = threadIdx.x; i < 16 * qu; i += blockDim.x) {
     const int r = i / qu, u = i % qu;
     uint4 v = make_uint4(0, 0, 0, 0);
@@ -98,9 +109,8 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
       }
       const size_t row = (static_cast<size_t>(blk) * p.G + g) * p.block_size + key % p.block_size;   // 16 keys never straddle a block
       bf16* sk = ring + static_cast<size_t>(i % p.stages) * stage;
-      bf16* sv = sk + kWDKeys * kp;
-      for (int u = lane; u < kWDKeys * ku; u += 32) cp_async16(smem_u32(sk + (u / ku) * kp + (u % ku) * 8), p.k_cache + row * p.d + u * 8, 16);
-      for (int u = lane; u < kWDKeys * vu; u += 32) cp_async16(smem_u32(sv + (u / vu) * vp + (u % vu) * 8), p.v_cache + row * p.dv + u * 8, 16);
+      wd_load_rows(smem_u32(sk), kp, p.k_cache + row * p.d, p.d, kl, lane);
+      wd_load_rows(smem_u32(sk + kWDKeys * kp), vp, p.v_cache + row * p.dv, p.dv, vl, lane);
     }
     cp_async_commit();
   };
@@ -144,7 +154,7 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
       mt[r] = fmaxf(mt[r], __shfl_xor_sync(0xffffffffu, mt[r], 2));
       const float m_new = fmaxf(m[r], mt[r]);
       moved |= m_new != m[r];
-      alpha[r] = m_new == -INFINITY ? 1.f : exp2f(m[r] - m_new);          // nothing visible so far
+      alpha[r] = m_new == -INFINITY ? 1.f : ex2_approx(m[r] - m_new);          // nothing visible so far
       m[r] = m_new;
     }
     if (__any_sync(0xffffffffu, moved)) {

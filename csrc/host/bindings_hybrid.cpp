@@ -37,7 +37,7 @@ int forge_delta_chunk_ok(int dk, int dv);
 long long forge_delta_chunk_scratch(int tokens, int seqs, int heads, int which);
 int forge_delta_chunk(const void* q, const void* k, const void* v, long long ld, int share, const float* cum, const float* beta, long long ldt,
                       float* state, const int* slots, const int* positions, const int* cu, int seqs, int max_q, int heads, int dk, int dv,
-                      int num_slots, void* mats, float* factors, float* o, unsigned* status, cudaStream_t stream);
+                      int num_slots, void* mats, float* factors, float* o, int cols, unsigned* status, cudaStream_t stream);
 int forge_gated_norm(int fp32, const float* o, const void* gate, long long ldg, const float* weight, int weight_period, void* out, long long ldo,
                      int tokens, int groups, int n, int gate_first, float factor, float eps, cudaStream_t stream);
 }
@@ -226,7 +226,8 @@ void state_space_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const 
 }
 
 void delta_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& cum, const Tensor& beta, Tensor& state, const Tensor& slots,
-                 const Tensor& positions, const Tensor& cu, int64_t seqs, int64_t max_q, Tensor& mats, Tensor& factors, Tensor& o, const Tensor& status) {
+                 const Tensor& positions, const Tensor& cu, int64_t seqs, int64_t max_q, Tensor& mats, Tensor& factors, Tensor& o, int64_t cols,
+                 const Tensor& status) {
   TORCH_CHECK(q.scalar_type() == kBf16 && state.dim() == 4 && cum.dim() == 2 && cum.size(0) == state.size(1) && cum.size(1) == q.size(0), "delta_chunk: sizes");
   const Rec r = recurrence_sizes(q, k, v, v.slice(1, 0, state.size(1)), c10::nullopt, state);
   const c10::cuda::CUDAGuard guard(q.device());
@@ -235,7 +236,7 @@ void delta_chunk(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor
                              ints(positions, r.T, "positions"), ints(cu, seqs + 1, "cu"), i32(seqs), i32(max_q), i32(r.H), i32(r.dk), i32(r.dv),
                              i32(r.slots), data(mats, kBf16, forge_delta_chunk_scratch(i32(r.T), i32(seqs), i32(r.H), 0), "mats"),
                              floats(factors, forge_delta_chunk_scratch(i32(r.T), i32(seqs), i32(r.H), 1), "factors"),
-                             floats(o, r.T * r.H * r.dv, "o"), status_word(status), stream_of(q)),
+                             floats(o, r.T * r.H * r.dv, "o"), i32(cols), status_word(status), stream_of(q)),
            "forge_delta_chunk");
 }
 

@@ -13,10 +13,13 @@ __device__ __forceinline__ float load_f(const bf16* p) { return __bfloat162float
 __device__ __forceinline__ void store_f(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_f(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-// N consecutive elements (N = 1 or 4; 4 needs 16-byte / 8-byte alignment).
+// N consecutive elements (N = 1, 4 or 8; 4 fp32 or 8 bf16 need 16-byte alignment, 4 bf16 8-byte).
 template <int N>
 __device__ __forceinline__ void load_n(const float* p, float* v) {
-  if constexpr (N == 4) {
+  if constexpr (N == 8) {
+    load_n<4>(p, v);
+    load_n<4>(p + 4, v + 4);
+  } else if constexpr (N == 4) {
     const float4 a = *reinterpret_cast<const float4*>(p);
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
   } else {
@@ -25,7 +28,11 @@ __device__ __forceinline__ void load_n(const float* p, float* v) {
 }
 template <int N>
 __device__ __forceinline__ void load_n(const bf16* p, float* v) {
-  if constexpr (N == 4) {
+  if constexpr (N == 8) {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    v[0] = bf16_lo(a.x); v[1] = bf16_hi(a.x); v[2] = bf16_lo(a.y); v[3] = bf16_hi(a.y);
+    v[4] = bf16_lo(a.z); v[5] = bf16_hi(a.z); v[6] = bf16_lo(a.w); v[7] = bf16_hi(a.w);
+  } else if constexpr (N == 4) {
     const uint2 a = *reinterpret_cast<const uint2*>(p);
     v[0] = bf16_lo(a.x); v[1] = bf16_hi(a.x); v[2] = bf16_lo(a.y); v[3] = bf16_hi(a.y);
   } else {
@@ -34,12 +41,17 @@ __device__ __forceinline__ void load_n(const bf16* p, float* v) {
 }
 template <int N>
 __device__ __forceinline__ void store_n(float* p, const float* v) {
-  if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  if constexpr (N == 8) {
+    store_n<4>(p, v);
+    store_n<4>(p + 4, v + 4);
+  } else if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
   else *p = v[0];
 }
 template <int N>
 __device__ __forceinline__ void store_n(bf16* p, const float* v) {
-  if constexpr (N == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  if constexpr (N == 8)
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  else if constexpr (N == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
   else *p = __float2bfloat16_rn(v[0]);
 }
 

@@ -299,7 +299,8 @@ extern "C" int forge_recurrence(int fp32, const void* q, const void* k, const vo
 }
 
 // One warp per (token, group of n entries).  kGateFirst: a = o silu(z), out = a / rms(a) weight; else out = o / rms(o) weight silu(z).
-template <typename T, int N, bool kGateFirst>
+// A lane holds up to R pieces of N entries; R = 0: any n, read twice.
+template <typename T, int N, int R, bool kGateFirst>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ldg,
                                                          const float* __restrict__ weight, int weight_period, T* __restrict__ out, long long ldo,
                                                          long long work, int groups, int n, float factor, float eps) {
@@ -307,36 +308,69 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
   pdl_wait();
   const long long w = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (w >= work) return;
-  const int lane = threadIdx.x & 31, g = static_cast<int>(w % groups);
+  const int lane = threadIdx.x & 31;
   const long long t = w / groups;
-  const float* src = o + t * groups * n + static_cast<long long>(g) * n;
+  const int g = static_cast<int>(w - t * groups);
+  const float* src = o + w * n;
+  const float* w0 = weight + static_cast<long long>(g) * n % weight_period;
   const T* z = gate + t * ldg + static_cast<long long>(g) * n;
   T* dst = out + t * ldo + static_cast<long long>(g) * n;
   float ss = 0.f;
-  for (int c = lane * N; c < n; c += 32 * N) {
-    float v[N], s[N];
-    load_n<N>(src + c, v);
-    if (kGateFirst) {
-      load_n<N>(z + c, s);
+  if constexpr (R > 0) {
+    float v[R][N], s[R][N], m[R][N];
 #pragma unroll
-      for (int e = 0; e < N; ++e) v[e] *= silu_t<T>(s[e]);
+    for (int r = 0; r < R; ++r) {
+      const int c = (r * 32 + lane) * N;
+      if (c < n) {
+        load_n<N>(src + c, v[r]);
+        load_n<N>(z + c, s[r]);
+        load_n<N>(w0 + c, m[r]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < N; ++e) v[r][e] = s[r][e] = m[r][e] = 0.f;
+      }
     }
 #pragma unroll
-    for (int e = 0; e < N; ++e) ss += v[e] * v[e];
-  }
-  const float inv = factor * rsqrtf(warp_sum_f(ss) / static_cast<float>(n) + eps);
-  for (int c = lane * N; c < n; c += 32 * N) {
-    float v[N], s[N], m[N];
-    load_n<N>(src + c, v);
-    load_n<N>(z + c, s);
-    load_n<N>(weight + (g * n + c) % weight_period, m);
+    for (int r = 0; r < R; ++r)
 #pragma unroll
-    for (int e = 0; e < N; ++e) v[e] *= inv * m[e] * silu_t<T>(s[e]);
-    store_n<N>(dst + c, v);
+      for (int e = 0; e < N; ++e) {
+        if (kGateFirst) v[r][e] *= silu_t<T>(s[r][e]);
+        ss += v[r][e] * v[r][e];
+        m[r][e] *= kGateFirst ? v[r][e] : v[r][e] * silu_t<T>(s[r][e]);
+      }
+    const float inv = factor * rsqrtf(warp_sum_f(ss) / static_cast<float>(n) + eps);
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int c = (r * 32 + lane) * N;
+#pragma unroll
+      for (int e = 0; e < N; ++e) m[r][e] *= inv;
+      if (c < n) store_n<N>(dst + c, m[r]);
+    }
+  } else {
+    for (int c = lane * N; c < n; c += 32 * N) {
+      float v[N], s[N];
+      load_n<N>(src + c, v);
+      load_n<N>(z + c, s);
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        if (kGateFirst) v[e] *= silu_t<T>(s[e]);
+        ss += v[e] * v[e];
+      }
+    }
+    const float inv = factor * rsqrtf(warp_sum_f(ss) / static_cast<float>(n) + eps);
+    for (int c = lane * N; c < n; c += 32 * N) {
+      float v[N], s[N], m[N];
+      load_n<N>(src + c, v);
+      load_n<N>(z + c, s);
+      load_n<N>(w0 + c, m);
+#pragma unroll
+      for (int e = 0; e < N; ++e) v[e] *= inv * m[e] * silu_t<T>(s[e]);
+      store_n<N>(dst + c, v);
+    }
   }
 }
 
-// o fp32 [tokens][groups n], gate [tokens][ldg], out [tokens][ldo]; the weight repeats every weight_period entries.
+// o fp32 [tokens][groups n], gate [tokens][ldg], out [tokens][ldo]; the weight repeats every weight_period entries, a multiple of n.
 template <typename T>
 static int gated_norm(const float* o, const T* gate, long long ldg, const float* weight, int weight_period, T* out, long long ldo, int tokens,
                       int groups, int n, bool gate_first, float factor, float eps, cudaStream_t stream) {
@@ -344,15 +378,20 @@ static int gated_norm(const float* o, const T* gate, long long ldg, const float*
   const dim3 grid(static_cast<unsigned>((work + 7) / 8));
   const uintptr_t mask = 4 * sizeof(T) - 1;
   const bool v4 = ((n | weight_period) & 3) == 0 && ((ldg | ldo) & 3) == 0 && (reinterpret_cast<uintptr_t>(gate) & mask) == 0 && (reinterpret_cast<uintptr_t>(out) & mask) == 0;
-  auto k = v4 ? (gate_first ? gated_norm_kernel<T, 4, true> : gated_norm_kernel<T, 4, false>)
-              : (gate_first ? gated_norm_kernel<T, 1, true> : gated_norm_kernel<T, 1, false>);
-  return launch_kernel(k, grid, dim3(256), 0, stream, 0, o, gate, ldg, weight, weight_period, out, ldo, work, groups, n, factor, eps) == cudaSuccess ? 0 : -2;
+#define FORGE_GN(N, R)                                                                                                                         \
+  return launch_kernel(gate_first ? gated_norm_kernel<T, N, R, true> : gated_norm_kernel<T, N, R, false>, grid, dim3(256), 0, stream, 0, o, gate, \
+                       ldg, weight, weight_period, out, ldo, work, groups, n, factor, eps) == cudaSuccess ? 0 : -2
+  if (!v4) FORGE_GN(1, 0);
+  if (n <= 128) FORGE_GN(4, 1);
+  if (n <= 256) FORGE_GN(4, 2);
+  FORGE_GN(4, 0);
+#undef FORGE_GN
 }
 
 extern "C" int forge_gated_norm(int fp32, const float* o, const void* gate, long long ldg, const float* weight, int weight_period, void* out,
                                 long long ldo, int tokens, int groups, int n, int gate_first, float factor, float eps, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (groups < 1 || n < 1 || weight_period < 1) return -1;
+  if (groups < 1 || n < 1 || weight_period < n || weight_period % n) return -1;
   return fp32 ? gated_norm<float>(o, static_cast<const float*>(gate), ldg, weight, weight_period, static_cast<float*>(out), ldo, tokens, groups, n, gate_first != 0, factor, eps, stream)
               : gated_norm<bf16>(o, static_cast<const bf16*>(gate), ldg, weight, weight_period, static_cast<bf16*>(out), ldo, tokens, groups, n, gate_first != 0, factor, eps, stream);
 }

@@ -10,7 +10,7 @@
 
 namespace forge {
 
-constexpr int kConvMaxTaps = 8;
+constexpr int kConvMaxTaps = 8, kConvBatch = 4;
 
 template <typename T>
 struct ConvArgs {
@@ -74,30 +74,35 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ConvArgs<T> p) {
     for (int i = 0; i < kTaps - 1; ++i)
       if (i < taps - 1) store_n<N>(st + static_cast<size_t>(i) * p.channels, keep[i]);
   }
-  for (int t = t0; t < t1; ++t) {
-    float y[N];
-    load_n<N>(p.x + static_cast<size_t>(t) * p.ldx + c, y);
+  for (int ta = t0; ta < t1; ta += kConvBatch) {
+    float x[kConvBatch][N];                      // loads of several tokens in flight
 #pragma unroll
-    for (int i = 0; i < kTaps; ++i)
-      if (i == taps - 1) {
+    for (int k = 0; k < kConvBatch; ++k) load_n<N>(p.x + static_cast<size_t>(min(ta + k, t1 - 1)) * p.ldx + c, x[k]);
 #pragma unroll
-        for (int e = 0; e < N; ++e) win[i][e] = y[e];
-      }
-#pragma unroll
-    for (int e = 0; e < N; ++e) {
-      float a = b[e];
+    for (int k = 0; k < kConvBatch; ++k) {
 #pragma unroll
       for (int i = 0; i < kTaps; ++i)
-        if (i < taps) a = fmaf(w[i][e], win[i][e], a);
-      y[e] = silu_t<T>(a);
-    }
-    store_n<N>(p.out + static_cast<size_t>(t) * p.channels + c, y);
+        if (i == taps - 1) {
 #pragma unroll
-    for (int i = 0; i + 1 < kTaps; ++i)
-      if (i + 1 < taps) {
+          for (int e = 0; e < N; ++e) win[i][e] = x[k][e];
+        }
+      float y[N];
 #pragma unroll
-        for (int e = 0; e < N; ++e) win[i][e] = win[i + 1][e];
+      for (int e = 0; e < N; ++e) {
+        float a = b[e];
+#pragma unroll
+        for (int i = 0; i < kTaps; ++i)
+          if (i < taps) a = fmaf(w[i][e], win[i][e], a);
+        y[e] = silu_t<T>(a);
       }
+      if (ta + k < t1) store_n<N>(p.out + static_cast<size_t>(ta + k) * p.channels + c, y);
+#pragma unroll
+      for (int i = 0; i + 1 < kTaps; ++i)
+        if (i + 1 < taps) {
+#pragma unroll
+          for (int e = 0; e < N; ++e) win[i][e] = win[i + 1][e];
+        }
+    }
   }
 }
 
@@ -121,7 +126,7 @@ extern "C" int forge_short_conv(int fp32, const void* x, long long ldx, const fl
                                 unsigned* status, cudaStream_t stream) {
   if (seqs <= 0 || max_q <= 0) return 0;
   if (taps_n < 1 || taps_n > kConvMaxTaps) return -1;
-  const int tile = 32;
+  const int tile = max_q > 64 ? 64 : 32;
   if (fp32)
     return short_conv<float>({static_cast<const float*>(x), ldx, taps, bias, static_cast<float*>(state), slots, positions, cu, static_cast<float*>(out),
                               channels, taps_n, num_slots, tile, status}, seqs, max_q, stream);

@@ -103,8 +103,13 @@ class HybridOps:
         else:
             mats = torch.empty(self.C.delta_chunk_scratch(T, seqs, H, 0), dtype=torch.bfloat16, device=q.device)
             factors = torch.empty(self.C.delta_chunk_scratch(T, seqs, H, 1), dtype=torch.float32, device=q.device)
-            self.C.delta_chunk(q, k, v, cum, weight, state, slots, batch.positions, cu, seqs, batch.max_seqlen_q, mats, factors, o, self.status)
+            self.C.delta_chunk(q, k, v, cum, weight, state, slots, batch.positions, cu, seqs, batch.max_seqlen_q, mats, factors, o,
+                               self.delta_columns(seqs, H, dv), self.status)
         return o
+
+    def delta_columns(self, seqs: int, heads: int, dv: int) -> int:
+        """Value columns per CTA of the chunked delta rule: narrow slices where wide ones leave half of the SMs idle."""
+        return 64 if 2 * seqs * heads * -(-dv // 64) > self.num_sms else 32
 
     def state_space(self, xbc, z, dt, block, state, batch, out, scale) -> None:
         s = block.spec

@@ -1,6 +1,7 @@
-"""Prefill and decode throughput of Goselix beside Qwen3 at equal width, head size, feed-forward work and number of layers.
+"""Prefill and decode throughput of a design beside others at equal width, head size, feed-forward work and number of layers:
+Goselix beside Qwen3, Tonapel beside Goselix and Qwen3.
 
-    python bench.py --design goselix [--steps K] [--warmup W]
+    python bench.py --design goselix|tonapel [--steps K] [--warmup W]
 
 A few layers of each (random weights, bf16), through the engine's own step: packed step buffer, model, sampling, CUDA graph for
 decode steps.  Device time per step (CUDA events); ahead of every timed step a buffer larger than L2 is written.  One JSON line
@@ -17,13 +18,17 @@ LAYERS, VOCAB = 4, 32000
 WORKLOADS = [("prefill", 8, 1024), ("prefill", 1, 8192), ("decode", 64, 1024), ("decode", 16, 4096), ("decode", 1, 4096)]
 
 
-def _configs(width: int):
+def _configs(design: str, width: int):
     from ..config import ModelConfig
-    from ..models.goselix_config import GoselixConfig, example_dict
+    from ..models import goselix_config, tonapel_config
     heads = max(8, width // 128)
     qwen = ModelConfig(hidden_size=width, num_hidden_layers=LAYERS, num_attention_heads=heads, num_key_value_heads=max(2, heads // 2) if width < 4096 else 8,
                        head_dim=128, intermediate_size=3 * width, vocab_size=VOCAB, tie_word_embeddings=False)
-    return [("goselix", GoselixConfig.from_dict(example_dict(width, LAYERS, VOCAB))), ("qwen3", qwen)]
+    goselix = goselix_config.GoselixConfig.from_dict(goselix_config.example_dict(width, LAYERS, VOCAB))
+    models = [("goselix", goselix), ("qwen3", qwen)]
+    if design == "tonapel":
+        models.insert(0, ("tonapel", tonapel_config.TonapelConfig.from_dict(tonapel_config.example_dict(width, LAYERS, VOCAB))))
+    return models
 
 
 def _requests(worker, seqs: int, tokens: int):
@@ -39,12 +44,12 @@ def _requests(worker, seqs: int, tokens: int):
     return out
 
 
-def run(steps: int, warmup: int, clock_sampler=None) -> None:
+def run(design: str, steps: int, warmup: int, clock_sampler=None) -> None:
     from .. import LLM
     from ..engine.step_batch import build_decode, build_prefill
     flush = torch.empty(1 << 30, dtype=torch.uint8, device="cuda")
     for width in SIZES:
-        for name, cfg in _configs(width):
+        for name, cfg in _configs(design, width):
             llm = LLM(name, hf_config=cfg, load_format="dummy", skip_tokenizer_init=True, max_model_len=8448, max_num_batched_tokens=8448,
                       max_num_seqs=64, num_kvcache_blocks=5 * 64 + 64, extra={"device_timing": True})
             w = llm.worker

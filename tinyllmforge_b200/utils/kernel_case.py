@@ -8,7 +8,7 @@ gemm_prefill_8b (8192 x 6144 x 4096), gemm_silu, gemm_fp8 (256 x 6144 x 4096, bl
 epilogue), gemm_scaled (qkv-like GEMM with the folded-norm row scale), gemm_decode_8b_down (256 x 4096 x 12288 with the residual
 epilogue: K split over CTA pairs + the reduce kernel), lm_head_sample (LM head + sampling in one kernel),
 rms_norm, qk_norm_rope_store, sampler; and those of ``mixer_cases.CASES`` (latent attention, retention, experts, residual
-stream).  Several cases may be given, separated by commas.
+stream) and ``hybrid_cases.CASES`` (windowed attention, short convolution, state-space and delta recurrences, sandwich norms).  Several cases may be given, separated by commas.
 ``--lib`` runs the library kernel the reference would use on the same case instead (cuBLAS through torch.matmul for the
 GEMMs, flash-attn 2 for the attention cases), for a same-box comparison.
 Prints the mean device time per launch (CUDA events) and the achieved fraction of the roofline denominator that applies:
@@ -23,9 +23,11 @@ import os
 
 import torch
 
-from .mixer_cases import CASES
+from .hybrid_cases import CASES as HYBRID_CASES
+from .mixer_cases import CASES as MIXER_CASES
 
 BF = torch.bfloat16
+CASES = {**MIXER_CASES, **HYBRID_CASES}
 
 
 def _peaks(path):
