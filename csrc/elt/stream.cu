@@ -232,8 +232,107 @@ __global__ void __launch_bounds__(256) stream_sandwich_kernel(const SandwichArgs
   }
 }
 
+// The same for rows that fit the registers of a CTA: R pieces of N entries per thread, no pass through shared memory.
+template <typename T, int N, int R>
+__global__ void __launch_bounds__(256) stream_sandwich_reg_kernel(const SandwichArgs<T> p) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  int r = blockIdx.x;
+  if (p.rows != nullptr) {
+    r = p.rows[r];
+    r = r < 0 ? 0 : (r >= p.n_rows ? p.n_rows - 1 : r);
+  }
+  const size_t base = static_cast<size_t>(r) * p.W;
+  const T* emb = nullptr;
+  if (p.ids != nullptr) {
+    int id = p.ids[r];
+    id = id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id);
+    emb = p.embed + static_cast<size_t>(id) * p.W;
+  }
+  float x[R][N], y[R][N], ss = 0.f;
+#pragma unroll
+  for (int q = 0; q < R; ++q) {
+    const int i = (q * blockDim.x + threadIdx.x) * N;
+#pragma unroll
+    for (int e = 0; e < N; ++e) x[q][e] = y[q][e] = 0.f;
+    if (i >= p.W) continue;
+    if (!p.start) load_n<N>(p.x + base + i, x[q]);
+    if (p.a != nullptr && p.a_rows == nullptr) load_n<N>(p.a + base + i, y[q]);
+  }
+#pragma unroll
+  for (int q = 0; q < R; ++q) {
+    const int i = (q * blockDim.x + threadIdx.x) * N;
+    if (i >= p.W) continue;
+    float v[N];
+    if (p.a != nullptr && p.a_rows != nullptr) {
+#pragma unroll 4
+      for (int j = 0; j < p.top; ++j) {
+        const size_t at = static_cast<size_t>(r) * p.top + j;
+        const float s = p.a_weights != nullptr ? p.a_weights[at] : 1.f;
+        load_n<N>(p.a + static_cast<size_t>(p.a_rows[at]) * p.W + i, v);
+#pragma unroll
+        for (int e = 0; e < N; ++e) y[q][e] = fmaf(s, v[e], y[q][e]);
+      }
+    }
+    if (p.a_bias != nullptr) {
+      load_n<N>(p.a_bias + i, v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) y[q][e] += v[e];
+    }
+    if (emb != nullptr) {
+      load_n<N>(emb + i, v);
+#pragma unroll
+      for (int e = 0; e < N; ++e) x[q][e] += v[e];
+    }
+#pragma unroll
+    for (int e = 0; e < N; ++e) ss += y[q][e] * y[q][e];
+  }
+  float f = 1.f;
+  if (p.a != nullptr && p.post != nullptr) f = p.mult * rsqrtf(block_sum_f(ss, red) / static_cast<float>(p.W) + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int q = 0; q < R; ++q) {
+    const int i = (q * blockDim.x + threadIdx.x) * N;
+    if (i >= p.W) continue;
+    float g[N];
+#pragma unroll
+    for (int e = 0; e < N; ++e) g[e] = 1.f;
+    if (p.post != nullptr) {
+      load_n<N>(p.post + i, g);
+#pragma unroll
+      for (int e = 0; e < N; ++e) g[e] += p.offset;
+    }
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      x[q][e] = fmaf(f * y[q][e], g[e], x[q][e]);
+      ss += x[q][e] * x[q][e];
+    }
+    if (p.rows == nullptr) store_n<N>(p.x + base + i, x[q]);
+  }
+  if (p.w == nullptr) return;
+  const float inv = rsqrtf(block_sum_f(ss, red) / static_cast<float>(p.W) + p.eps);
+  const size_t out = static_cast<size_t>(blockIdx.x) * p.W;
+#pragma unroll
+  for (int q = 0; q < R; ++q) {
+    const int i = (q * blockDim.x + threadIdx.x) * N;
+    if (i >= p.W) continue;
+    float g[N];
+    load_n<N>(p.w + i, g);
+#pragma unroll
+    for (int e = 0; e < N; ++e) g[e] = x[q][e] * inv * (g[e] + p.offset);
+    store_n<N>(p.h + out + i, g);
+  }
+}
+
 template <typename T>
 static int stream_sandwich(int out_rows, const SandwichArgs<T>& p, cudaStream_t stream) {
+  if ((p.W & 7) == 0 && p.W <= 4096) {
+    const int pieces = p.W <= 2048 ? 1 : 2, per = 8 * pieces;
+    const int threads = ((p.W + per - 1) / per + 31) / 32 * 32;
+    auto k = pieces == 1 ? stream_sandwich_reg_kernel<T, 8, 1> : stream_sandwich_reg_kernel<T, 8, 2>;
+    return launch_kernel(k, dim3(out_rows), dim3(threads), 0, stream, 0, p) == cudaSuccess ? 0 : -2;
+  }
   const size_t smem = static_cast<size_t>(p.W) * 8;
   if (smem > 200 * 1024) return -1;
   const bool v4 = (p.W & 3) == 0;

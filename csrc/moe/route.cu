@@ -120,6 +120,7 @@ __global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, co
   for (int e = warp; e < E; e += blockDim.x >> 5) {
     const T* we = w + static_cast<size_t>(e) * W;
     float z = 0.f;
+#pragma unroll 4
     for (int i = lane * N; i < W; i += 32 * N) {
       float a[N], b[N];
       load_n<N>(row + i, a);
@@ -144,6 +145,10 @@ extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int 
     auto k = v4 ? router_kernel<float, 4> : router_kernel<float, 1>;
     return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
   }
+  const bool aligned = ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(w)) & 15) == 0;
+  // a few tokens would occupy a few CTAs of the kernel below: one CTA per token spreads them
+  if (T_ <= 128 && (W & 7) == 0 && aligned)
+    return launch_kernel(router_kernel<bf16, 8>, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
   if (W % 32 == 0 && E <= 256 && (reinterpret_cast<uintptr_t>(h) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
     const int Ep = (E + 7) & ~7;
     const bool two = T_ > 2048 && E <= 128;        // more tokens per CTA halve the reads of the router matrix
