@@ -56,11 +56,11 @@ class HybridOps:
                                        spec.scale, scale, self.status)
 
     def windowed_chunks(self, seqs: int, spec, capacity: int) -> tuple[int, int]:
-        """(keys per chunk, chunks): the window is cut until there are about four CTAs per SM.  Depends only on shapes known at
+        """(keys per chunk, chunks): the window is cut until the two CTAs that an SM holds are busy.  Depends only on shapes known at
         graph-capture time."""
         span = min(spec.window, capacity) + 15
         ctas = seqs * spec.kv_heads * -(-(spec.heads // spec.kv_heads) // 16)
-        parts = max(1, min(4 * self.num_sms // ctas, span // 128))
+        parts = max(1, min(2 * self.num_sms // ctas, span // 128))
         chunk = -(-(-(-span // parts)) // 64) * 64
         return chunk, -(-span // chunk)
 
