@@ -8,7 +8,8 @@
 // CTA = 128 query rows of one (sequence, head), key tiles of 64 from the tile that holds the first row's oldest visible key to
 // the tile of the last row's own.  A row may see nothing of its CTA's first tiles: its reference maximum is set by the first
 // key it does see, and nothing of O needs scaling then.  Warp roles, double-buffered S, the reference maximum that is only
-// raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu; P is double-buffered where shared memory allows.
+// raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu.  P and V are double-buffered where that leaves room for
+// two CTAs per SM (whose softmax warps hide each other's latency), else single-buffered, else as shared memory allows.
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
@@ -73,24 +74,23 @@ __device__ __forceinline__ float windowed_probs(const uint32_t (&v)[kXN], int kb
 }
 
 struct WindowedPrefill {
-  int H, G, d, dv, nq, nv, p_bufs;          // nq, nv: boxes of 64 columns of keys and of values
+  int H, G, d, dv, nq, nv, p_bufs, v_bufs;  // nq, nv: boxes of 64 columns of keys and of values
   int window, block_size, table_width, num_blocks;
   long long ldo;
   float scale_log2, out_scale;
 };
 
 // tm_q: [tokens, H * 64 nq], box 128 x 64; tm_k / tm_v: [blocks * G * block_size, d / dv], box 64 x 64.
-__global__ void __launch_bounds__(kXThreads, 1)
+__global__ void __launch_bounds__(kXThreads, 2)
 windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                         const int* __restrict__ cu_q, const int* __restrict__ context_lens, const int* __restrict__ tables,
                         bf16* __restrict__ out, const WindowedPrefill z, unsigned* status) {
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  extern __shared__ __align__(1024) uint8_t smem[];   // the swizzled boxes start on multiples of 1024 bytes
   const uint32_t k_stage = z.nq * kXKBox, v_stage = z.nv * kXKBox;
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + z.nq * kXQBox;                   // [2 stages]
-  uint8_t* sV = sK + 2 * k_stage;                     // [2 stages]
-  uint8_t* sP = sV + 2 * v_stage;                     // [p_bufs][hi, lo]
+  uint8_t* sV = sK + 2 * k_stage;                     // [v_bufs]
+  uint8_t* sP = sV + z.v_bufs * v_stage;              // [p_bufs][hi, lo]
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + z.p_bufs * 2 * kXQBox);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;
@@ -105,6 +105,10 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 
   pdl_launch_dependents();
   pdl_wait();
+  if (smem_u32(smem) & 1023) {
+    if (threadIdx.x == 0) set_status(status, kStatusBadShape);
+    return;
+  }
   const int seq = blockIdx.z, h = blockIdx.y, g = h / (z.H / z.G);
   const int q_begin = cu_q[seq], q_len = cu_q[seq + 1] - q_begin;
   const int k_len = min(context_lens[seq], z.table_width * z.block_size);
@@ -161,9 +165,10 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         if (!mbar_wait_parked(&k_empty[s], ph ^ 1, status)) break;
         mbar_expect_tx(&k_full[s], k_stage);
         for (int b = 0; b < z.nq; ++b) tma_load_2d(sK + s * k_stage + b * kXKBox, &tm_k, &k_full[s], b * 64, row);
-        if (!mbar_wait_parked(&v_empty[s], ph ^ 1, status)) break;
-        mbar_expect_tx(&v_full[s], v_stage);
-        for (int b = 0; b < z.nv; ++b) tma_load_2d(sV + s * v_stage + b * kXKBox, &tm_v, &v_full[s], b * 64, row);
+        const int vs = j % z.v_bufs;
+        if (!mbar_wait_parked(&v_empty[vs], ((j / z.v_bufs) & 1) ^ 1, status)) break;
+        mbar_expect_tx(&v_full[vs], v_stage);
+        for (int b = 0; b < z.nv; ++b) tma_load_2d(sV + vs * v_stage + b * kXKBox, &tm_v, &v_full[vs], b * 64, row);
       }
     }
   } else if (warp == 1) {
@@ -190,14 +195,14 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       for (int j = 0; j < n_tiles && ok; ++j) {
         if (j + 1 < n_tiles) ok = issue_s(j + 1);
         if (!ok) break;
-        const int s = j & 1;
+        const int s = j & 1, vs = j % z.v_bufs;
         const uint32_t ph = (j >> 1) & 1;
-        if (!mbar_wait_parked(&v_full[s], ph, status) || !mbar_wait_parked(&p_full[s], ph, status)) {
+        if (!mbar_wait_parked(&v_full[vs], (j / z.v_bufs) & 1, status) || !mbar_wait_parked(&p_full[s], ph, status)) {
           ok = false;
           break;
         }
         tcgen05_fence_after();
-        const uint32_t v_addr = smem_u32(sV + s * v_stage);
+        const uint32_t v_addr = smem_u32(sV + vs * v_stage);
         const uint32_t pj_addr = p_addr + (j % z.p_bufs) * 2 * kXQBox;
 #pragma unroll
         for (int k = 0; k < kXN / 16; ++k) {
@@ -206,7 +211,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
           umma_f16(tmem_o, umma_desc_k_sw128(pj_addr + kXQBox + k * 32), vd, idesc_o, 1);
         }
         umma_commit(&pv_done[s]);
-        umma_commit(&v_empty[s]);
+        umma_commit(&v_empty[vs]);
       }
     }
   } else {
@@ -308,8 +313,8 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   }
 }
 
-static int windowed_prefill_smem(int nq, int nv, int p_bufs) {
-  return nq * (kXQBox + 2 * kXKBox) + 2 * nv * kXKBox + p_bufs * 2 * kXQBox + 256 + 1024;
+static int windowed_prefill_smem(int nq, int nv, int p_bufs, int v_bufs) {
+  return nq * (kXQBox + 2 * kXKBox) + v_bufs * nv * kXKBox + p_bufs * 2 * kXQBox + 256;
 }
 
 // Columns of one head's padded query row, or 0 when the kernel does not take these sizes (else: windowed_attend_any).
@@ -332,10 +337,18 @@ extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_c
   if (qcols == 0 || num_seqs > 65535 || H > 65535 || H % G || window < 1 || !(scale > 0.f) || (ldo & 7) || (reinterpret_cast<uintptr_t>(out) & 15)) return -1;
   if (static_cast<long long>(num_blocks) * G * block_size >= (1ll << 31)) return -1;
   const int nq = qcols / 64, nv = (dv + 63) / 64;
-  const int p_bufs = windowed_prefill_smem(nq, nv, 2) <= 227 * 1024 ? 2 : 1;
-  const int smem = windowed_prefill_smem(nq, nv, p_bufs);
-  if (smem > 227 * 1024) return -1;
-  const WindowedPrefill z = {H, G, d, dv, nq, nv, p_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale};
+  constexpr int kHalf = 113 * 1024, kAll = 227 * 1024;        // two CTAs per SM, one
+  const int bufs[3][2] = {{2, 2}, {1, 2}, {1, 1}};            // of P, of V
+  int smem = 0, p_bufs = 1, v_bufs = 1;
+  for (int limit = nv > 2 ? kAll : kHalf; smem == 0 && limit <= kAll; limit += kAll - kHalf)
+    for (int i = 0; i < 3 && smem == 0; ++i)
+      if (windowed_prefill_smem(nq, nv, bufs[i][0], bufs[i][1]) <= limit) {
+        p_bufs = bufs[i][0];
+        v_bufs = bufs[i][1];
+        smem = windowed_prefill_smem(nq, nv, p_bufs, v_bufs);
+      }
+  if (smem == 0) return -1;
+  const WindowedPrefill z = {H, G, d, dv, nq, nv, p_bufs, v_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale};
   CUtensorMap tm_q, tm_k, tm_v;
   const uint64_t qw = static_cast<uint64_t>(H) * qcols, rows = static_cast<uint64_t>(num_blocks) * G * block_size;
   if (forge_make_tmap_2d(&tm_q, q, tokens, qw, qw, kXM, 2) != 0) return -2;
