@@ -25,6 +25,8 @@ Layout (all int32 words, every section starts on a 16-byte boundary):
     state_slots[padded_seqs] row of the recurrent-state arrays that belongs to the sequence; -1: none (padding, or a model
                              without recurrent layers)
     cu_seqlens_k[padded_seqs + 1]  running sum of the keys visible to the sequences from ``num_single`` on (0 before)
+    prev_ids[padded_tokens]  the token before each of input_ids in its sequence, -1 before a sequence's first (models whose embedding
+                             reads pairs of tokens)
 
 A prefill step may mix portions of prompts with single tokens of running requests.  ``num_single`` counts its LEADING
 sequences with one query token: a model may give them to its decode kernels and the rest to its prefill kernels;
@@ -43,7 +45,7 @@ HEADER_WORDS = 16
 H_MAGIC, H_PREFILL, H_NSEQ, H_NTOK, H_PSEQ, H_PTOK, H_WIDTH, H_MAXQ, H_MAXK, H_STEP, H_SEEDLO, H_SEEDHI, H_NSINGLE, H_KVROWS = range(14)
 
 SECTIONS = ("input_ids", "positions", "slot_mapping", "cu_seqlens_q", "context_lens", "last_index",
-            "temperatures", "block_tables", "src_rows", "state_slots", "cu_seqlens_k")
+            "temperatures", "block_tables", "src_rows", "state_slots", "cu_seqlens_k", "prev_ids")
 
 
 def _align4(n: int) -> int:
@@ -57,6 +59,7 @@ def section_offsets(padded_tokens: int, padded_seqs: int, table_width: int) -> t
         "cu_seqlens_q": padded_seqs + 1, "context_lens": padded_seqs, "last_index": padded_seqs,
         "temperatures": padded_seqs, "block_tables": padded_seqs * table_width, "src_rows": padded_seqs,
         "state_slots": padded_seqs, "cu_seqlens_k": padded_seqs + 1,
+        "prev_ids": padded_tokens,
     }
     off = HEADER_WORDS
     out = {}
@@ -142,7 +145,7 @@ def build_prefill(reqs, block_size: int, step_index: int = 0, seed: int = 0) -> 
         o, n = offs[name]
         return buf[o:o + n]
 
-    ids, pos, slots = sec("input_ids"), sec("positions"), sec("slot_mapping")
+    ids, prev, pos, slots = sec("input_ids"), sec("prev_ids"), sec("positions"), sec("slot_mapping")
     tables = sec("block_tables").reshape(S, width)
     tables[:] = -1
     t = 0
@@ -150,6 +153,8 @@ def build_prefill(reqs, block_size: int, step_index: int = 0, seed: int = 0) -> 
         c, n = starts[i], ends[i]
         q = n - c
         ids[t:t + q] = r.token_ids[c:n]
+        prev[t] = r.token_ids[c - 1] if c > 0 else -1
+        prev[t + 1:t + q] = ids[t:t + q - 1]
         p = np.arange(c, n, dtype=np.int64)
         pos[t:t + q] = p
         bt = np.asarray(r.block_table, dtype=np.int64)
@@ -172,6 +177,12 @@ def build_prefill(reqs, block_size: int, step_index: int = 0, seed: int = 0) -> 
     return StepBatch(buf)
 
 
+def _previous(r) -> int:
+    """The token before a request's newest.  It is known when a decode step is built, also in the loop that runs one step ahead of the
+    tokens it has read back (where the newest itself is not)."""
+    return r.token_ids[-2] if len(r.token_ids) > 1 else -1
+
+
 def build_decode(reqs, block_size: int, step_index: int = 0, seed: int = 0,
                  pad_to: int | None = None, table_width: int | None = None) -> StepBatch:
     """Decode step: one token per request, optionally padded to a graph bucket."""
@@ -186,6 +197,9 @@ def build_decode(reqs, block_size: int, step_index: int = 0, seed: int = 0,
         return buf[o:o + n]
 
     sec("input_ids")[:S] = [r.token_ids[-1] for r in reqs]
+    prev = sec("prev_ids")
+    prev[:] = -1
+    prev[:S] = [_previous(r) for r in reqs]
     sec("positions")[:S] = lens - 1
     last_block = np.fromiter((r.block_table[-1] for r in reqs), dtype=np.int64, count=S)
     slots = sec("slot_mapping")
@@ -243,6 +257,8 @@ class DecodeBuilder:
                 buf[H_MAXK] = int(lens.max())
                 o, _ = sb.offsets["input_ids"]
                 buf[o:o + S] = [r.token_ids[-1] for r in reqs]
+                o, _ = sb.offsets["prev_ids"]
+                buf[o:o + S] = [_previous(r) for r in reqs]
                 o, _ = sb.offsets["positions"]
                 buf[o:o + S] = lens - 1
                 o, _ = sb.offsets["context_lens"]

@@ -10,7 +10,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 
 from ..config import parse_dtype
-from .specs import DenseSpec, MoeSpec, Rotation, take
+from .specs import DenseSpec, LoopSpec, MoeSpec, Rotation, layer_runs, take
 
 
 @dataclass(frozen=True)
@@ -82,14 +82,6 @@ class LayerSpec:
         return cls(d["type"], MIXER_SPECS[d["type"]].from_dict(d["mixer"]), _mlp_from_dict(d.get("mlp")))
 
 
-@dataclass(frozen=True)
-class LoopSpec:
-    """Layers start .. stop - 1 run ``times`` times in a row before the rest follow."""
-    start: int
-    stop: int
-    times: int
-
-
 @dataclass
 class GoselixConfig:
     vocab_size: int
@@ -108,9 +100,8 @@ class GoselixConfig:
         for key in ("vocab", "width", "norm", "layers"):
             if key not in d:
                 raise ValueError(f"Goselix config: missing {key!r}")
-        loop = d.get("loop")
         cfg = cls(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), tuple(LayerSpec.from_dict(l) for l in d["layers"]),
-                  LoopSpec(**take(loop, "loop", {"start": int, "stop": int, "times": int})) if loop else None,
+                  LoopSpec.from_dict(d["loop"], len(d["layers"])) if d.get("loop") else None,
                   torch_dtype=str(d.get("torch_dtype") or d.get("dtype") or "bfloat16").replace("torch.", ""))
         if d.get("eos_token_id") is not None:
             eos = d["eos_token_id"]
@@ -123,8 +114,6 @@ class GoselixConfig:
     def validate(self) -> None:
         if not self.layers:
             raise ValueError("Goselix config: no layers")
-        if self.loop is not None and not (0 <= self.loop.start < self.loop.stop <= len(self.layers) and self.loop.times >= 1):
-            raise ValueError("Goselix config: loop must name a range of layers and at least one pass")
 
     def validate_tp(self, size: int) -> None:
         if size != 1:
@@ -132,12 +121,7 @@ class GoselixConfig:
 
     def layer_runs(self) -> list:
         """[(layer, pass)] in the order of computation; pass is None for a layer outside the loop."""
-        n, loop = len(self.layers), self.loop
-        if loop is None:
-            return [(i, None) for i in range(n)]
-        return ([(i, None) for i in range(loop.start)]
-                + [(i, t) for t in range(loop.times) for i in range(loop.start, loop.stop)]
-                + [(i, None) for i in range(loop.stop, n)])
+        return layer_runs(len(self.layers), self.loop)
 
     @property
     def dtype(self):

@@ -1,7 +1,7 @@
 """What decoders whose layers are listed one by one have in common: embedding and head, memory per layer run, sampling.
 
-A design derives from ``LayeredDecoder``, fills ``layers`` (each with ``mix``, a block of ``blocks.py`` or
-``hybrid_blocks.py``) and ``runs`` (the layer runs in order of computation), and states its residual stream in ``forward``.
+A design derives from ``LayeredDecoder``, fills ``layers`` (each with ``mix``, a block of ``blocks.py``,
+``hybrid_blocks.py`` or ``attention_blocks.py``) and ``runs`` (the layer runs in order of computation), and states its residual stream in ``forward``.
 """
 from __future__ import annotations
 
@@ -26,7 +26,7 @@ class LayeredDecoder:
 
         def rope(rot):                           # layers with the same rotation share one table
             if rot not in tables:
-                tables[rot] = ref_ops.rope_table(positions, rot.dims, rot.base, self.device, torch.float64)
+                tables[rot] = ref_ops.rotation_table(positions, rot.frequencies, rot.amplitude, self.device)
             return tables[rot]
 
         self.rope = rope

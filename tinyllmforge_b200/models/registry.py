@@ -1,8 +1,8 @@
 """Model registry: from a ``config.json`` to its configuration class and its model class.
 
 An entry names the configuration class (a dataclass with ``from_dict``) and the model class.  A checkpoint of
-Goselix or Tonapel names its design under ``architecture``; everything else is a Hugging Face configuration whose ``model_type`` the configuration
-class checks itself.
+Goselix, Tonapel or Mezapel names its design under ``architecture``; everything else is a Hugging Face configuration whose
+``model_type`` the configuration class checks itself.
 """
 from __future__ import annotations
 
@@ -15,6 +15,7 @@ _ENTRIES = {
     "qwen3": ("tinyllmforge_b200.config:ModelConfig", "tinyllmforge_b200.models.qwen3:Qwen3ForCausalLM"),
     "Goselix": ("tinyllmforge_b200.models.goselix_config:GoselixConfig", "tinyllmforge_b200.models.goselix:GoselixForCausalLM"),
     "Tonapel": ("tinyllmforge_b200.models.tonapel_config:TonapelConfig", "tinyllmforge_b200.models.tonapel:TonapelForCausalLM"),
+    "Mezapel": ("tinyllmforge_b200.models.mezapel_config:MezapelConfig", "tinyllmforge_b200.models.mezapel:MezapelForCausalLM"),
 }
 
 

@@ -53,6 +53,12 @@ def rope_table(max_positions: int, head_dim: int, theta: float, device="cpu", an
     return torch.cat((freqs.cos(), freqs.sin()), dim=-1).float().to(device)
 
 
+def rotation_table(max_positions: int, frequencies: list, amplitude: float = 1.0, device="cpu") -> torch.Tensor:
+    """The same from given frequencies (one per pair of entries), angles in fp64; cos and sin times ``amplitude``."""
+    angles = torch.outer(torch.arange(max_positions, dtype=torch.float64), torch.tensor(frequencies, dtype=torch.float64))
+    return (amplitude * torch.cat((angles.cos(), angles.sin()), dim=-1)).float().to(device)
+
+
 def apply_rope(x: torch.Tensor, positions: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
     """x: [T, heads, d]; rotates pairs (i, i + d/2)."""
     d = x.shape[-1]
@@ -190,6 +196,30 @@ def stream_update(x, dtype, eps, norms, start=False, a=None, b=None, ids=None, e
     else:
         s = s[rows.long()]
     return [norm(s, w).to(dtype) for w in norms]
+
+
+def stream_mix(x, dtype, eps, into, norm, bias, y=None, mix=None, out=None, ids=None, prev=None, embed=None, scale=1.0, pairs=None,
+               mul_prev=0, mul_cur=0, rows=None):
+    """Several residual streams x [T, streams, W] (fp32) between two sublayers.  First the streams take up a sublayer's result, all at
+    once: x_t <- sum_s mix[s, t] x_s + out[t] y; or, with ``ids``, every stream begins as scale * embed[id] + the pair table's row
+    (prev * mul_prev + id * mul_cur) mod (rows - 1), the last row where prev < 0.  Then sum_s into[s] x_s goes through a
+    layer norm (weight, bias) and is rounded once to ``dtype``.  norm=None: no result.  ``rows``: results of these rows only, and
+    x is left as it was."""
+    if ids is not None:
+        last = pairs.shape[0] - 1
+        at = torch.where(prev < 0, last, (prev.long() * mul_prev + ids.long() * mul_cur) % last)
+        s = (scale * F.embedding(ids.long(), embed).float() + pairs[at].float())[:, None].expand_as(x)
+    else:
+        s = torch.einsum("nsw,st->ntw", x, mix) + out[:, None] * y.float()[:, None, :]
+    if rows is None:
+        x.copy_(s)
+    else:
+        s = s[rows.long()]
+    if norm is None:
+        return None
+    u = torch.einsum("nsw,s->nw", s, into)
+    u = u - u.mean(dim=-1, keepdim=True)
+    return (u * torch.rsqrt(u.pow(2).mean(dim=-1, keepdim=True) + eps) * norm.float() + bias.float()).to(dtype)
 
 
 def apply_partial_rope(x: torch.Tensor, positions: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
@@ -397,6 +427,7 @@ class RefOps(ref_hybrid.RefHybridOps):
     rms_norm = staticmethod(rms_norm)
     qk_norm_rope_store = staticmethod(qk_norm_rope_store)
     stream_update = staticmethod(stream_update)
+    stream_mix = staticmethod(stream_mix)
     latent_prepare = staticmethod(latent_prepare)
     retention = staticmethod(retention)
     moe = staticmethod(moe)

@@ -26,8 +26,25 @@ def bias_rope_store(proj, bias, spec, table, positions, slot_mapping, k_cache, v
     return q.to(proj.dtype)
 
 
-def windowed_attention(q, k_cache, v_cache, batch, spec, out, scale):
-    """out [T, heads * vdim] <- scale * attention of q over the keys at most ``window - 1`` positions back."""
+def norm_rope_store(proj, q_norm, k_norm, eps, spec, table, positions, slot_mapping, k_cache, v_cache):
+    """proj [T, q | k | v] -> q [T, heads, dim] normed and rotated; keys (the same) and values go to the paged caches.  A norm weight of
+    ``dim`` entries belongs to every head, one of all entries to the projection as a whole."""
+    from .ref import apply_partial_rope, store_kv
+    T, H, G, d = proj.shape[0], spec.heads, spec.kv_heads, spec.dim
+
+    def normed(x, w, heads):
+        x = x.float().reshape((T, heads, d) if spec.norm == "head" else (T, heads * d))
+        return apply_partial_rope((x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps) * w).view(T, heads, d), positions, table)
+
+    q, k, v = proj.split([H * d, G * d, G * spec.vdim], dim=-1)
+    store_kv(normed(k, k_norm, G), v.reshape(T, G, spec.vdim), k_cache, v_cache, slot_mapping)
+    return normed(q, q_norm, H).to(proj.dtype)
+
+
+def windowed_attention(q, k_cache, v_cache, batch, spec, out, scale, chunked=False, softcap=0.0, sink=None, gate=None):
+    """out [T, heads * vdim] <- scale * attention of q over the keys at most ``window - 1`` positions back, or (``chunked``) over those of
+    the query's own chunk of ``window`` positions.  ``softcap`` bounds the scores; ``sink`` [heads]: one more score per head, of
+    the denominator alone; ``gate`` [T, heads] or [T, heads * vdim]: its sigmoid multiplies the result."""
     from .ref import _gather_kv
     H, G = spec.heads, spec.kv_heads
     cu, lens = batch.cu_seqlens_q.tolist(), batch.context_lens.tolist()
@@ -36,22 +53,30 @@ def windowed_attention(q, k_cache, v_cache, batch, spec, out, scale):
         k = _gather_kv(k_cache, batch.block_tables[s], n).float().repeat_interleave(H // G, dim=0)
         v = _gather_kv(v_cache, batch.block_tables[s], n).float().repeat_interleave(H // G, dim=0)
         scores = torch.einsum("qhd,hkd->hqk", q[a:b].float(), k) * spec.scale
-        back = batch.positions[a:b].long()[:, None] - torch.arange(n, device=q.device)[None, :]
-        scores.masked_fill_((back < 0) | (back >= spec.window), float("-inf"))
-        o = torch.einsum("hqk,hke->qhe", torch.softmax(scores, dim=-1), v)
+        if softcap:
+            scores = softcap * torch.tanh(scores / softcap)
+        pos, keys = batch.positions[a:b].long()[:, None], torch.arange(n, device=q.device)[None, :]
+        oldest = pos // spec.window * spec.window if chunked else pos - spec.window + 1
+        scores.masked_fill_((keys > pos) | (keys < oldest), float("-inf"))
+        if sink is not None:
+            scores = torch.cat((scores, sink[:, None, None].expand(H, b - a, 1)), dim=-1)
+        o = torch.einsum("hqk,hke->qhe", torch.softmax(scores, dim=-1)[..., :n], v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[a:b].float()).view(b - a, H, -1)
         out[a:b] = (scale * o.reshape(b - a, -1)).to(out.dtype)
 
 
-def short_conv(x, taps, bias, state, batch):
-    """silu of a causal convolution over time, per channel.  x [T, channels], taps [channels, n] (last column: the token
-    itself), state [slots, n - 1, channels]: the inputs before the step's first token, replaced by the last ones."""
+def short_conv(x, taps, bias, state, batch, act="silu"):
+    """A causal convolution over time, per channel, then silu (``act="none"``: nothing).  x [T, channels], taps [channels, n] (last column:
+    the token itself), state [slots, n - 1, channels]: the inputs before the step's first token, replaced by the last ones."""
     n = taps.shape[1]
     out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     for a, b, slot, fresh in _runs(batch):
-        past = state[slot] if not fresh else torch.zeros_like(state[slot])
+        past = state[slot] if not fresh and n > 1 else torch.zeros(state.shape[1:], dtype=state.dtype, device=state.device)
         seq = torch.cat([past, x[a:b]]).float()
         y = sum(seq[i:i + b - a] * taps[:, i] for i in range(n))
-        out[a:b] = F.silu(y if bias is None else y + bias).to(x.dtype)
+        y = y if bias is None else y + bias
+        out[a:b] = (F.silu(y) if act == "silu" else y).to(x.dtype)
         if n > 1:
             state[slot] = seq[seq.shape[0] - (n - 1):].to(state.dtype)
     return out
@@ -108,6 +133,7 @@ def gated_delta(qkv, gate, ba, block, state, batch):
 class RefHybridOps:
     """Mixed into ``RefOps``."""
     bias_rope_store = staticmethod(bias_rope_store)
+    norm_rope_store = staticmethod(norm_rope_store)
     windowed_attention = staticmethod(windowed_attention)
     short_conv = staticmethod(short_conv)
     state_space = staticmethod(state_space)
