@@ -2,10 +2,12 @@
 //
 //   bias_rope_store     q | k | v of a token + biases; q and k rotated (first rd entries of a head, entry i with i + rd / 2); q to
 //                       [token][head][q_pitch] (padding columns zero), k and v to the caches [block][kv_head][block_size][dim / vdim]
-//   windowed_attend_any softmax attention of a token over itself and the window - 1 tokens before it, bf16 or fp32, any sizes: one
-//                       warp per query token, eight tokens of one head per CTA share key and value tiles of 32
+//   windowed_attend_any softmax attention of a token over itself and the window - 1 tokens before it (or the tokens of its chunk of
+//                       the sequence), with the options of attend_options.cuh, bf16 or fp32, any sizes: one warp per query token,
+//                       eight tokens of one head per CTA share key and value tiles of 32
 //
 // Scores, weights and sums are fp32.
+#include "../include/attend_options.cuh"
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
@@ -142,6 +144,7 @@ struct AttendAny {
   long long ldo;
   int width, num_blocks, block_size, H, G, d, dv, q_pitch, window;
   float scale, out_scale;
+  AttendOptions<T> opt;
   unsigned* status;
 };
 
@@ -165,7 +168,7 @@ __global__ void __launch_bounds__(256) windowed_attend_any_kernel(const AttendAn
     sq[i] = load_f(p.q + (static_cast<size_t>(t0 + i / p.d) * p.H + h) * p.q_pitch + i % p.d);
   const int first = p.positions[t0], pos = live ? p.positions[t] : -1;
   const int last = first + n - 1, cap = p.width * p.block_size;
-  const int lo = max(first - p.window + 1, 0);
+  const int lo = oldest_visible(first, p.window, p.opt.chunked), mine = live ? oldest_visible(pos, p.window, p.opt.chunked) : 0;
   float m = -INFINITY, l = 0.f, acc[kWMaxCols];
 #pragma unroll
   for (int c = 0; c < kWMaxCols; ++c) acc[c] = 0.f;
@@ -190,7 +193,9 @@ __global__ void __launch_bounds__(256) windowed_attend_any_kernel(const AttendAn
     const int j = j0 + lane;
     float x = 0.f;
     for (int c = 0; c < p.d; ++c) x = fmaf(sq[warp * p.d + c], sk[lane * kp + c], x);
-    x = j <= pos && pos - j < p.window ? x * p.scale : -INFINITY;
+    x *= p.scale;
+    if (p.opt.softcap > 0.f) x = p.opt.softcap * tanhf(x / p.opt.softcap);
+    if (j > pos || j < mine) x = -INFINITY;
     float mt = x;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, o));
@@ -208,11 +213,16 @@ __global__ void __launch_bounds__(256) windowed_attend_any_kernel(const AttendAn
     }
   }
   if (!live) return;
-  const float inv = l > 0.f ? p.out_scale / l : 0.f;
+  float top = m;
+  if (p.opt.sink != nullptr) {                     // one more score, of the denominator alone
+    top = fmaxf(m, p.opt.sink[h]);
+    l = l * expf(m - top) + expf(p.opt.sink[h] - top);
+  }
+  const float inv = l > 0.f ? p.out_scale * expf(m - top) / l : 0.f;
   T* dst = p.out + static_cast<size_t>(t) * p.ldo + static_cast<size_t>(h) * p.dv;
 #pragma unroll
   for (int c = 0; c < kWMaxCols; ++c)
-    if (c * 32 + lane < p.dv) store_f(dst + c * 32 + lane, acc[c] * inv);
+    if (c * 32 + lane < p.dv) store_f(dst + c * 32 + lane, acc[c] * inv * output_gate(p.opt, t, h, c * 32 + lane));
 }
 
 template <typename T>
@@ -228,15 +238,19 @@ static int windowed_attend_any(const AttendAny<T>& p, int seqs, int max_q, cudaS
 extern "C" int forge_windowed_attend_any(int fp32, const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* cu, int seqs,
                                          int max_q, const int* positions, const int* tables, int width, int num_blocks, int block_size,
                                          void* out, long long ldo, int H, int G, int d, int dv, int window, float scale, float out_scale,
-                                         unsigned* status, cudaStream_t stream) {
+                                         int chunked, float softcap, const float* sink, const void* gate, long long ldg, int gate_head,
+                                         int gate_col, unsigned* status, cudaStream_t stream) {
   if (seqs <= 0 || max_q <= 0) return 0;
+  if (window < 1) return -1;
   if (seqs > 65535 || H > 65535) return -1;
   if (fp32)
     return windowed_attend_any<float>({static_cast<const float*>(q), static_cast<const float*>(k_cache), static_cast<const float*>(v_cache), cu, positions,
-                                       tables, static_cast<float*>(out), ldo, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, scale, out_scale, status},
+                                       tables, static_cast<float*>(out), ldo, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, scale, out_scale,
+                                       {chunked, softcap, sink, static_cast<const float*>(gate), ldg, gate_head, gate_col}, status},
                                       seqs, max_q, stream);
   return windowed_attend_any<bf16>({static_cast<const bf16*>(q), static_cast<const bf16*>(k_cache), static_cast<const bf16*>(v_cache), cu, positions,
-                                    tables, static_cast<bf16*>(out), ldo, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, scale, out_scale, status},
+                                    tables, static_cast<bf16*>(out), ldo, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, scale, out_scale,
+                                    {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}, status},
                                    seqs, max_q, stream);
 }
 

@@ -5,7 +5,8 @@
 // query heads at once (mma.sync: heads on the 16-row side) and keeps its own running maximum, sum and output.  Softmax
 // weights are fp32 and enter the second product as bf16 hi + lo halves.  The warps' states are merged through shared memory;
 // with more than one chunk, partial outputs go to scratch and a second kernel merges them.  Lengths are read on the device and
-// the grid depends on the batch bucket only, so the launch is CUDA-graph safe.
+// the grid depends on the batch bucket only, so the launch is CUDA-graph safe.  Options: attend_options.cuh.
+#include "../include/attend_options.cuh"
 #include "../include/launch.cuh"
 #include "../include/mma_sync.cuh"
 #include "../include/scalar.cuh"
@@ -25,7 +26,8 @@ struct WindowedDecode {
   float* part_o;            // [seqs][H][chunks][dv]
   float* part_ml;           // [seqs][H][chunks][2]
   int width, num_blocks, block_size, H, G, d, dv, q_pitch, window, chunk, max_chunks, stages, slices;
-  float scale_log2, out_scale;
+  float scale_log2, out_scale, cap_pre, cap_post;
+  AttendOptions<bf16> opt;
   unsigned* status;
 };
 
@@ -47,7 +49,7 @@ __device__ __forceinline__ WindowRange window_range(const WindowedDecode& p, int
   }
   WindowRange r;
   r.end = max(len, 0);
-  r.lo = max(r.end - p.window, 0);
+  r.lo = r.end > 0 ? oldest_visible(r.end - 1, p.window, p.opt.chunked) : 0;
   r.begin = r.lo & ~(kWDKeys - 1);
   return r;
 }
@@ -63,7 +65,17 @@ __device__ __forceinline__ void wd_load_rows(uint32_t dst, int pitch, const bf16
 }
 __device__ __forceinline__ int wd_lanes_log2(int units) { return units <= 1 ? 0 : 32 - __clz(units - 1); }
 
-template <int NV>           // blocks of 8 value columns
+// Output entry from sums O and L that are relative to the maximum M (base-2 logarithms).
+__device__ __forceinline__ float wd_finish(const WindowedDecode& p, int s, int h, int c, float M, float L, float O) {
+  if (p.opt.sink != nullptr) {
+    const float sink = p.opt.sink[h] * 1.4426950408889634f, top = fmaxf(M, sink), f = exp2f(M - top);
+    L = fmaf(L, f, exp2f(sink - top));
+    O *= f;
+  }
+  return L > 0.f ? p.out_scale * O / L * output_gate(p.opt, s, h, c) : 0.f;
+}
+
+template <int NV, bool kCap>           // blocks of 8 value columns; bounded scores
 __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const WindowedDecode p) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int kp = wd_pitch(p.d), vp = wd_pitch(p.dv);
@@ -143,7 +155,8 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int j = key + n * 8 + q2 + (e & 1);
-        x[n][e] = j >= w.lo && j < c_end ? x[n][e] * p.scale_log2 : -INFINITY;
+        const float y = kCap ? softcap_log2(x[n][e], p.cap_pre, p.cap_post) : x[n][e] * p.scale_log2;
+        x[n][e] = j >= w.lo && j < c_end ? y : -INFINITY;
         mt[e >> 1] = fmaxf(mt[e >> 1], x[n][e]);
       }
     float alpha[2];
@@ -229,7 +242,7 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
       O = fmaf(f, row[c], O);
     }
     if (n_chunks == 1) {
-      p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h0 + r) * p.dv + c] = __float2bfloat16_rn(L > 0.f ? p.out_scale * O / L : 0.f);
+      p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h0 + r) * p.dv + c] = __float2bfloat16_rn(wd_finish(p, s, h0 + r, c, M, L, O));
     } else {
       const size_t at = (static_cast<size_t>(s) * p.H + h0 + r) * p.max_chunks + chunk;
       p.part_o[at * p.dv + c] = O;
@@ -259,7 +272,7 @@ __global__ void __launch_bounds__(128) windowed_merge_kernel(const WindowedDecod
       L = fmaf(f, p.part_ml[(base + c) * 2 + 1], L);
       O = fmaf(f, p.part_o[(base + c) * p.dv + i], O);
     }
-    p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h) * p.dv + i] = __float2bfloat16_rn(L > 0.f ? p.out_scale * O / L : 0.f);
+    p.out[static_cast<size_t>(s) * p.ldo + static_cast<size_t>(h) * p.dv + i] = __float2bfloat16_rn(wd_finish(p, s, h, i, M, L, O));
   }
 }
 
@@ -279,6 +292,7 @@ extern "C" int forge_windowed_decode_ok(int d, int dv, int block_size) {
 extern "C" int forge_windowed_decode(const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* tables, const int* lens,
                                      int seqs, int width, int num_blocks, int block_size, void* out, long long ldo, float* part_o, float* part_ml,
                                      int chunk, int max_chunks, int H, int G, int d, int dv, int window, float scale, float out_scale,
+                                     int chunked, float softcap, const float* sink, const void* gate, long long ldg, int gate_head, int gate_col,
                                      unsigned* status, cudaStream_t stream) {
   if (seqs <= 0) return 0;
   if (!forge_windowed_decode_ok(d, dv, block_size) || (q_pitch & 7) || seqs > 65535 || max_chunks > 65535 || chunk % kWDKeys || chunk < kWDKeys || window < 1)
@@ -287,7 +301,9 @@ extern "C" int forge_windowed_decode(const void* q, int q_pitch, const void* k_c
   if (static_cast<long long>(max_chunks) * chunk < span || (max_chunks > 1 && (part_o == nullptr || part_ml == nullptr))) return -1;
   WindowedDecode p = {static_cast<const bf16*>(q), static_cast<const bf16*>(k_cache), static_cast<const bf16*>(v_cache), tables, lens,
                       static_cast<bf16*>(out), ldo, part_o, part_ml, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, chunk, max_chunks,
-                      0, (H / G + 15) / 16, scale * 1.4426950408889634f, out_scale, status};
+                      0, (H / G + 15) / 16, scale * 1.4426950408889634f, out_scale,
+                      softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f, softcap * 1.4426950408889634f,
+                      {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}, status};
   const dim3 grid(G * p.slices, seqs, max_chunks);
 #define FORGE_WD(NV)                                                                                                                   \
   {                                                                                                                                    \
@@ -295,8 +311,10 @@ extern "C" int forge_windowed_decode(const void* q, int q_pitch, const void* k_c
     while (p.stages > 2 && wd_smem(d, dv, NV, p.stages) > 112 * 1024) --p.stages;                                                      \
     const size_t smem = wd_smem(d, dv, NV, p.stages);                                                                                  \
     if (smem > 227 * 1024) return -1;                                                                                                  \
-    FORGE_ENSURE_DYN_SMEM(windowed_decode_kernel<NV>, 227 * 1024);                                                                     \
-    if (launch_kernel(windowed_decode_kernel<NV>, grid, dim3(32 * kWDWarps), smem, stream, 0, p) != cudaSuccess) return -2;            \
+    FORGE_ENSURE_DYN_SMEM((windowed_decode_kernel<NV, false>), 227 * 1024);                                                            \
+    FORGE_ENSURE_DYN_SMEM((windowed_decode_kernel<NV, true>), 227 * 1024);                                                             \
+    auto k = softcap > 0.f ? windowed_decode_kernel<NV, true> : windowed_decode_kernel<NV, false>;                                     \
+    if (launch_kernel(k, grid, dim3(32 * kWDWarps), smem, stream, 0, p) != cudaSuccess) return -2;                                         \
   }
   if (dv <= 64) FORGE_WD(8) else if (dv <= 128) FORGE_WD(16) else if (dv <= 192) FORGE_WD(24) else FORGE_WD(32)
 #undef FORGE_WD

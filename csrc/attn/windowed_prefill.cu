@@ -10,6 +10,8 @@
 // key it does see, and nothing of O needs scaling then.  Warp roles, double-buffered S, the reference maximum that is only
 // raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu.  P and V are double-buffered where that leaves room for
 // two CTAs per SM (whose softmax warps hide each other's latency), else single-buffered, else as shared memory allows.
+// Options (chunks, bounded scores, sinks, gated output): attend_options.cuh.
+#include "../include/attend_options.cuh"
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
@@ -44,9 +46,9 @@ __device__ __forceinline__ float windowed_row_max(const uint32_t (&v)[kXN], int 
   return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
 }
 
-// p = 2^(s scale - m_ref) of one row -> hi and lo bf16 halves in shared memory (K-major, 128-byte swizzle); returns the row sum.
-template <bool kMasked>
-__device__ __forceinline__ float windowed_probs(const uint32_t (&v)[kXN], int kbase, int lo, int limit, float scale_log2, float m_ref,
+// p = 2^(s scale - m_ref) of one row (kCap: of its bounded scores, s = raw, scale = the two factors of softcap_log2) -> hi and lo bf16 halves in shared memory (K-major, 128-byte swizzle); returns the row sum.
+template <bool kMasked, bool kCap>
+__device__ __forceinline__ float windowed_probs(const uint32_t (&v)[kXN], int kbase, int lo, int limit, float scale_log2, float cap_post, float m_ref,
                                                 uint8_t* p_row, int r) {
   float ps[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -55,8 +57,9 @@ __device__ __forceinline__ float windowed_probs(const uint32_t (&v)[kXN], int kb
 #pragma unroll
     for (int i = 0; i < 8; i += 2) {
       const int key = kbase + c + i;
-      float p0 = ex2_approx(fmaf(__uint_as_float(v[c + i]), scale_log2, -m_ref));
-      float p1 = ex2_approx(fmaf(__uint_as_float(v[c + i + 1]), scale_log2, -m_ref));
+      const float s0 = __uint_as_float(v[c + i]), s1 = __uint_as_float(v[c + i + 1]);
+      float p0 = ex2_approx(kCap ? softcap_log2(s0, scale_log2, cap_post) - m_ref : fmaf(s0, scale_log2, -m_ref));
+      float p1 = ex2_approx(kCap ? softcap_log2(s1, scale_log2, cap_post) - m_ref : fmaf(s1, scale_log2, -m_ref));
       if (kMasked) {
         p0 = key >= lo && key < limit ? p0 : 0.f;
         p1 = key + 1 >= lo && key + 1 < limit ? p1 : 0.f;
@@ -77,10 +80,12 @@ struct WindowedPrefill {
   int H, G, d, dv, nq, nv, p_bufs, v_bufs;  // nq, nv: boxes of 64 columns of keys and of values
   int window, block_size, table_width, num_blocks;
   long long ldo;
-  float scale_log2, out_scale;
+  float scale_log2, out_scale, cap_pre, cap_post;
+  AttendOptions<bf16> opt;
 };
 
 // tm_q: [tokens, H * 64 nq], box 128 x 64; tm_k / tm_v: [blocks * G * block_size, d / dv], box 64 x 64.
+template <bool kCap>
 __global__ void __launch_bounds__(kXThreads, 2)
 windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                         const int* __restrict__ cu_q, const int* __restrict__ context_lens, const int* __restrict__ tables,
@@ -116,7 +121,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   if (m0 >= q_len) return;                            // uniform for the CTA, before anything is allocated
   const int past = max(k_len - q_len, 0);
   const int kv_end = min(k_len, past + m0 + kXM);
-  const int tile0 = max(past + m0 - z.window + 1, 0) / kXN;
+  const int tile0 = oldest_visible(past + m0, z.window, z.opt.chunked) / kXN;
   const int n_tiles = (kv_end + kXN - 1) / kXN - tile0;
   if (n_tiles <= 0) return;
 
@@ -219,7 +224,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const int r = quad * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const int qpos = past + m0 + r;
-    const int limit = min(qpos + 1, k_len), lo = max(qpos - z.window + 1, 0);          // visible keys: [lo, limit)
+    const int limit = min(qpos + 1, k_len), lo = oldest_visible(qpos, z.window, z.opt.chunked);          // visible keys: [lo, limit)
     const int o_cols = z.nv * 64;
     float m_ref = 0.f, l_run = 0.f;
     bool seen = false, ok = true;
@@ -238,7 +243,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       if (lane == 0) mbar_arrive(&s_empty[j & 1]);
       const bool masked = !__all_sync(0xffffffffu, kbase >= lo && kbase + kXN <= limit);
       float mt = masked ? windowed_row_max<true>(v, kbase, lo, limit) : windowed_row_max<false>(v, kbase, lo, limit);
-      mt *= z.scale_log2;                                // scale > 0: max commutes with the scaling
+      mt = kCap && mt != -INFINITY ? softcap_log2(mt, z.cap_pre, z.cap_post) : mt * z.scale_log2;      // scale > 0: both keep the order
       if (!seen && mt != -INFINITY) {                    // nothing of this row is in O yet, or only zeros
         m_ref = mt;
         seen = true;
@@ -272,8 +277,9 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         if (!ok) break;
       }
       uint8_t* p_row = sP + (j % z.p_bufs) * 2 * kXQBox + r * 128;
-      l_run += masked ? windowed_probs<true>(v, kbase, lo, limit, z.scale_log2, m_ref, p_row, r)
-                      : windowed_probs<false>(v, kbase, lo, limit, z.scale_log2, m_ref, p_row, r);
+      const float factor = kCap ? z.cap_pre : z.scale_log2;
+      l_run += masked ? windowed_probs<true, kCap>(v, kbase, lo, limit, factor, z.cap_post, m_ref, p_row, r)
+                      : windowed_probs<false, kCap>(v, kbase, lo, limit, factor, z.cap_post, m_ref, p_row, r);
       fence_proxy_async_smem();
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_full[j & 1]);
@@ -281,8 +287,19 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     if (ok) ok = mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, status);
     if (ok) {
       tcgen05_fence_after();
-      const float inv = l_run > 0.f ? z.out_scale / l_run : 0.f;
+      float top = m_ref;
+      if (z.opt.sink != nullptr) {                       // one more score, of the denominator alone
+        const float sink = z.opt.sink[h] * 1.4426950408889634f;
+        top = fmaxf(m_ref, sink);
+        l_run = fmaf(l_run, exp2f(m_ref - top), exp2f(sink - top));
+      }
       const bool store = m0 + r < q_len;
+      float inv = l_run > 0.f ? z.out_scale * exp2f(m_ref - top) / l_run : 0.f;
+      const bf16* gate = z.opt.gate == nullptr || !store ? nullptr : z.opt.gate + static_cast<size_t>(q_begin + m0 + r) * z.opt.ldg + static_cast<size_t>(h) * z.opt.gate_head;
+      if (gate != nullptr && z.opt.gate_col == 0) {      // one gate per head
+        inv *= sigmoid_t<bf16>(load_f(gate));
+        gate = nullptr;
+      }
       bf16* dst = out + static_cast<size_t>(q_begin + m0 + r) * z.ldo + static_cast<size_t>(h) * z.dv;
 #pragma unroll 1
       for (int c = 0; c < o_cols; c += 32) {
@@ -293,12 +310,11 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             if (c + i >= z.dv) continue;                 // dv is a multiple of 8
-            uint4 pk;
-            pk.x = pack_bf16x2(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
-            pk.y = pack_bf16x2(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
-            pk.z = pack_bf16x2(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv);
-            pk.w = pack_bf16x2(__uint_as_float(o[i + 6]) * inv, __uint_as_float(o[i + 7]) * inv);
-            *reinterpret_cast<uint4*>(dst + c + i) = pk;
+            float f[8];
+            if (gate != nullptr) load_n<8>(gate + c + i, f);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(o[i + e]) * inv * (gate != nullptr ? sigmoid_t<bf16>(f[e]) : 1.f);
+            store_n<8>(dst + c + i, f);
           }
         }
       }
@@ -327,15 +343,17 @@ extern "C" int forge_make_tmap_2d(CUtensorMap* tm, const void* base, uint64_t ro
                                   uint32_t box_rows, int elem_bytes);
 
 // q [tokens][H][q_pitch], q_pitch = forge_windowed_prefill_qcols; sequence s has the step's tokens cu_q[s] .. cu_q[s + 1] (its last
-// ones) and context_lens[s] keys; out rows of ldo elements (a multiple of 8), 16-byte aligned.
+// ones) and context_lens[s] keys; out rows of ldo elements (a multiple of 8), 16-byte aligned; a gate per element likewise.
 extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_cache, const void* v_cache, const int* cu_q, const int* context_lens,
                                       const int* tables, int table_width, int num_blocks, int block_size, void* out, long long ldo, int num_seqs,
-                                      int max_q, int H, int G, int d, int dv, int window, float scale, float out_scale, unsigned* status,
+                                      int max_q, int H, int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap,
+                                      const float* sink, const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status,
                                       cudaStream_t stream) {
   if (tokens <= 0 || num_seqs <= 0 || max_q <= 0) return 0;
   const int qcols = forge_windowed_prefill_qcols(d, dv, block_size);
   if (qcols == 0 || num_seqs > 65535 || H > 65535 || H % G || window < 1 || !(scale > 0.f) || (ldo & 7) || (reinterpret_cast<uintptr_t>(out) & 15)) return -1;
   if (static_cast<long long>(num_blocks) * G * block_size >= (1ll << 31)) return -1;
+  if (gate != nullptr && gate_col != 0 && (gate_col != 1 || ((ldg | gate_head) & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -1;
   const int nq = qcols / 64, nv = (dv + 63) / 64;
   constexpr int kHalf = 113 * 1024, kAll = 227 * 1024;        // two CTAs per SM, one
   const int bufs[3][2] = {{2, 2}, {1, 2}, {1, 1}};            // of P, of V
@@ -348,14 +366,17 @@ extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_c
         smem = windowed_prefill_smem(nq, nv, p_bufs, v_bufs);
       }
   if (smem == 0) return -1;
-  const WindowedPrefill z = {H, G, d, dv, nq, nv, p_bufs, v_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale};
+  const WindowedPrefill z = {H, G, d, dv, nq, nv, p_bufs, v_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale,
+                             softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f, softcap * 1.4426950408889634f,
+                             {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}};
   CUtensorMap tm_q, tm_k, tm_v;
   const uint64_t qw = static_cast<uint64_t>(H) * qcols, rows = static_cast<uint64_t>(num_blocks) * G * block_size;
   if (forge_make_tmap_2d(&tm_q, q, tokens, qw, qw, kXM, 2) != 0) return -2;
   if (forge_make_tmap_2d(&tm_k, k_cache, rows, d, d, kXN, 2) != 0) return -2;
   if (forge_make_tmap_2d(&tm_v, v_cache, rows, dv, dv, kXN, 2) != 0) return -2;
-  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel, 227 * 1024);
-  return launch_kernel(windowed_prefill_kernel, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v,
+  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<false>, 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<true>, 227 * 1024);
+  return launch_kernel(softcap > 0.f ? windowed_prefill_kernel<true> : windowed_prefill_kernel<false>, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v,
                        cu_q, context_lens, tables, static_cast<bf16*>(out), z, status) == cudaSuccess ? 0 : -5;
 }
 

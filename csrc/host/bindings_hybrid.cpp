@@ -8,10 +8,17 @@ int forge_bias_rope_store(int fp32, const void* proj, long long ld, int tokens, 
                           int block_size, int H, int G, int d, int dv, unsigned* status, cudaStream_t stream);
 int forge_windowed_attend_any(int fp32, const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* cu, int seqs, int max_q,
                               const int* positions, const int* tables, int width, int num_blocks, int block_size, void* out, long long ldo, int H,
-                              int G, int d, int dv, int window, float scale, float out_scale, unsigned* status, cudaStream_t stream);
+                              int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap, const float* sink,
+                              const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status, cudaStream_t stream);
+int forge_norm_rope_store(int fp32, const void* proj, long long ld, int tokens, const float* q_norm, const float* k_norm, int whole, float eps,
+                          const float* rope, int rope_rows, int rd, const int* positions, const int* slots, void* q, int q_pitch, void* k_cache,
+                          void* v_cache, long long num_slots, int block_size, int H, int G, int d, int dv, unsigned* status, cudaStream_t stream);
+int forge_stream_mix(int fp32, float* x, const void* y, const float* mix, const float* out, const int* ids, const int* prev, const void* embed,
+                     int vocab, float scale, const void* pairs, int buckets, long long mul_prev, long long mul_cur, const float* into, const void* w,
+                     const void* b, void* h, const int* rows, int out_rows, int n_rows, int W, int S, float eps, cudaStream_t stream);
 int forge_short_conv(int fp32, const void* x, long long ldx, const float* taps, const float* bias, void* state, const int* slots,
                      const int* positions, const int* cu, int seqs, int max_q, void* out, int channels, int taps_n, int num_slots,
-                     unsigned* status, cudaStream_t stream);
+                     int silu, unsigned* status, cudaStream_t stream);
 int forge_recurrence_decode_ok(int dk, int dv);
 int forge_recurrence(int fp32, const void* q, const void* k, const void* v, long long ld, const void* dt, const void* beta, long long ld_raw,
                      const float* A_log, const float* dt_bias, const float* D, float* state, const int* slots, const int* positions,
@@ -20,12 +27,13 @@ int forge_recurrence(int fp32, const void* q, const void* k, const void* v, long
 int forge_windowed_decode_ok(int d, int dv, int block_size);
 int forge_windowed_decode(const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* tables, const int* lens, int seqs,
                           int width, int num_blocks, int block_size, void* out, long long ldo, float* part_o, float* part_ml, int chunk,
-                          int max_chunks, int H, int G, int d, int dv, int window, float scale, float out_scale, unsigned* status,
-                          cudaStream_t stream);
+                          int max_chunks, int H, int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap,
+                          const float* sink, const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status, cudaStream_t stream);
 int forge_windowed_prefill_qcols(int d, int dv, int block_size);
 int forge_windowed_prefill(const void* q, int tokens, const void* k_cache, const void* v_cache, const int* cu_q, const int* context_lens,
                            const int* tables, int table_width, int num_blocks, int block_size, void* out, long long ldo, int num_seqs, int max_q,
-                           int H, int G, int d, int dv, int window, float scale, float out_scale, unsigned* status, cudaStream_t stream);
+                           int H, int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap, const float* sink,
+                           const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status, cudaStream_t stream);
 int forge_recurrence_gates(const void* dt, const void* beta, long long ld_raw, const float* A_log, const float* dt_bias, const int* cu, int seqs,
                            int max_q, int heads, float* cum, float* weight, long long ldt, cudaStream_t stream);
 int forge_retention_chunk_ok(int heads, int dk, int dv, int rd);
@@ -71,10 +79,87 @@ void bias_rope_store(const Tensor& proj, const Tensor& bias, const Tensor& rope,
            "forge_bias_rope_store");
 }
 
+// The same with norms of q and k ahead of the rotation and no biases; norm weights of dim entries (per head) or of all rows
+void norm_rope_store(const Tensor& proj, const Tensor& q_norm, const Tensor& k_norm, bool whole, double eps, const Tensor& rope, const Tensor& positions,
+                     const Tensor& slots, Tensor& q, Tensor& k_cache, Tensor& v_cache, const Tensor& status) {
+  const int f = elem(proj);
+  const auto dt = proj.scalar_type();
+  const Caches c = cache_sizes(k_cache, v_cache, dt);
+  TORCH_CHECK(q.dim() == 3 && q.size(0) == proj.size(0) && rope.dim() == 2 && rope.size(1) % 2 == 0 && rope.size(1) <= c.d && q.size(2) >= c.d, "norm_rope_store: sizes");
+  const int64_t T = proj.size(0), H = q.size(1), rows = (H + c.G) * c.d + c.G * c.dv;
+  const c10::cuda::CUDAGuard guard(proj.device());
+  check_rc(forge_norm_rope_store(f, view2(proj, dt, T, rows, "proj"), proj.stride(0), i32(T), floats(q_norm, whole ? H * c.d : c.d, "q_norm"),
+                                 floats(k_norm, whole ? c.G * c.d : c.d, "k_norm"), whole ? 1 : 0, static_cast<float>(eps), floats(rope, 0, "rope"),
+                                 i32(rope.size(0)), i32(rope.size(1)), ints(positions, T, "positions"), ints(slots, T, "slots"), data(q, dt, 0, "q"),
+                                 i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), static_cast<long long>(c.blocks) * c.block_size,
+                                 i32(c.block_size), i32(H), i32(c.G), i32(c.d), i32(c.dv), status_word(status), stream_of(proj)),
+           "forge_norm_rope_store");
+}
+
+// x fp32 [tokens, streams, width].  With y [tokens, width]: mix [streams, streams], out [streams]; without: the streams begin as embeddings
+void stream_mix(Tensor& x, const OptTensor& y, const OptTensor& mix, const OptTensor& out, const OptTensor& ids, const OptTensor& prev,
+                const OptTensor& embed, double scale, const OptTensor& pairs, int64_t mul_prev, int64_t mul_cur, const Tensor& into, const OptTensor& w,
+                const OptTensor& b, const OptTensor& h, const OptTensor& rows, double eps, bool fp32) {
+  TORCH_CHECK(x.dim() == 3, "stream_mix: x [tokens, streams, width] expected");
+  const int64_t T = x.size(0), S = x.size(1), W = x.size(2), n = rows.has_value() ? rows->numel() : T;
+  const auto dt = fp32 ? at::kFloat : at::kBFloat16;
+  const void *yp = nullptr, *ep = nullptr, *pp = nullptr;
+  const float *mp = nullptr, *op = nullptr;
+  const int *ip = nullptr, *vp = nullptr;
+  int64_t vocab = 0, buckets = 0;
+  if (y.has_value()) {
+    TORCH_CHECK(mix.has_value() && out.has_value(), "stream_mix: y comes with mix and out");
+    yp = view2(*y, dt, T, W, "y");
+    need(*y, dt, 0, "y");
+    mp = floats(*mix, S * S, "mix");
+    op = floats(*out, S, "out");
+  } else {
+    TORCH_CHECK(ids.has_value() && prev.has_value() && embed.has_value() && pairs.has_value(), "stream_mix: y or tokens and tables expected");
+    ip = ints(*ids, T, "ids");
+    vp = ints(*prev, T, "prev");
+    TORCH_CHECK(embed->dim() == 2 && embed->size(1) == W && pairs->dim() == 2 && pairs->size(1) == W && pairs->size(0) >= 2, "stream_mix: tables");
+    ep = data(*embed, dt, 0, "embed");
+    pp = data(*pairs, dt, 0, "pairs");
+    vocab = embed->size(0);
+    buckets = pairs->size(0) - 1;
+  }
+  const bool normed = w.has_value();
+  TORCH_CHECK(!normed || (b.has_value() && h.has_value()), "stream_mix: a norm has a bias and a result");
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_stream_mix(fp32 ? 1 : 0, floats(x, 0, "x"), yp, mp, op, ip, vp, ep, i32(vocab), static_cast<float>(scale), pp, i32(buckets), mul_prev,
+                            mul_cur, floats(into, S, "into"), normed ? data(*w, dt, W, "w") : nullptr, normed ? data(*b, dt, W, "b") : nullptr,
+                            normed ? data(*h, dt, n * W, "h") : nullptr, rows.has_value() ? ints(*rows, n, "rows") : nullptr, i32(n), i32(T), i32(W), i32(S),
+                            static_cast<float>(eps), stream_of(x)),
+           "forge_stream_mix");
+}
+
 struct Attend {
   int64_t T, H;
   Caches c;
 };
+
+// sink fp32 [heads]; gate [tokens, heads] or [tokens, heads dv] (a view)
+struct Options {
+  int chunked;
+  float softcap;
+  const float* sink;
+  const void* gate;
+  long long ldg;
+  int gate_head, gate_col;
+};
+Options attend_options(bool chunked, double softcap, const OptTensor& sink, const OptTensor& gate, const Attend& a, at::ScalarType dt) {
+  TORCH_CHECK(softcap >= 0, "windowed attention: softcap");
+  Options o{chunked ? 1 : 0, static_cast<float>(softcap), nullptr, nullptr, 0, 0, 0};
+  if (sink.has_value()) o.sink = floats(*sink, a.H, "sink");
+  if (gate.has_value()) {
+    const bool element = gate->dim() == 2 && gate->size(1) == a.H * a.c.dv;
+    o.gate = view2(*gate, dt, a.T, element ? a.H * a.c.dv : a.H, "gate");
+    o.ldg = gate->stride(0);
+    o.gate_head = element ? i32(a.c.dv) : 1;
+    o.gate_col = element ? 1 : 0;
+  }
+  return o;
+}
 Attend attend_sizes(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& out, const Tensor& tables, int64_t seqs) {
   const auto dt = q.scalar_type();
   const Caches c = cache_sizes(k_cache, v_cache, dt);
@@ -87,14 +172,16 @@ Attend attend_sizes(const Tensor& q, const Tensor& k_cache, const Tensor& v_cach
 // q [tokens, H, q_pitch], out [tokens, H dv] (a view); sequence s: query rows cu[s] .. cu[s + 1]
 void windowed_attend_any(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu, int64_t seqs, int64_t max_q,
                          const Tensor& positions, const Tensor& tables, Tensor& out, int64_t window, double scale, double out_scale,
-                         const Tensor& status) {
+                         bool chunked, double softcap, const OptTensor& sink, const OptTensor& gate, const Tensor& status) {
   const int f = elem(q);
   const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
+  const Options x = attend_options(chunked, softcap, sink, gate, a, q.scalar_type());
   const c10::cuda::CUDAGuard guard(q.device());
   check_rc(forge_windowed_attend_any(f, q.data_ptr(), i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), ints(cu, seqs + 1, "cu"), i32(seqs),
                                      i32(max_q), ints(positions, a.T, "positions"), ints(tables, 0, "tables"), i32(tables.size(1)), i32(a.c.blocks),
                                      i32(a.c.block_size), out.data_ptr(), out.stride(0), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window),
-                                     static_cast<float>(scale), static_cast<float>(out_scale), status_word(status), stream_of(q)),
+                                     static_cast<float>(scale), static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head,
+                                     x.gate_col, status_word(status), stream_of(q)),
            "forge_windowed_attend_any");
 }
 
@@ -103,9 +190,10 @@ constexpr auto kBf16 = at::kBFloat16;
 // One token per sequence: rows 0 .. seqs - 1 of q and out.
 void windowed_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& tables, const Tensor& lens, int64_t seqs,
                      Tensor& out, const OptTensor& part_o, const OptTensor& part_ml, int64_t chunk, int64_t max_chunks, int64_t window,
-                     double scale, double out_scale, const Tensor& status) {
+                     double scale, double out_scale, bool chunked, double softcap, const OptTensor& sink, const OptTensor& gate, const Tensor& status) {
   TORCH_CHECK(q.scalar_type() == kBf16 && seqs <= q.size(0), "windowed_decode: q");
   const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
+  const Options x = attend_options(chunked, softcap, sink, gate, a, q.scalar_type());
   float *po = nullptr, *pm = nullptr;
   if (max_chunks > 1) {
     TORCH_CHECK(part_o.has_value() && part_ml.has_value(), "windowed_decode: scratch");
@@ -116,27 +204,31 @@ void windowed_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cac
   check_rc(forge_windowed_decode(q.data_ptr(), i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), ints(tables, 0, "tables"), ints(lens, seqs, "lens"),
                                  i32(seqs), i32(tables.size(1)), i32(a.c.blocks), i32(a.c.block_size), out.data_ptr(), out.stride(0), po, pm, i32(chunk),
                                  i32(max_chunks), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window), static_cast<float>(scale),
-                                 static_cast<float>(out_scale), status_word(status), stream_of(q)),
+                                 static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head, x.gate_col, status_word(status),
+                                 stream_of(q)),
            "forge_windowed_decode");
 }
 
 // Sequence s: the rows cu[s] .. cu[s + 1] of q and out, its last ones; context_lens[s] keys.
 void windowed_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu, const Tensor& context_lens, const Tensor& tables,
-                      int64_t seqs, int64_t max_q, Tensor& out, int64_t window, double scale, double out_scale, const Tensor& status) {
+                      int64_t seqs, int64_t max_q, Tensor& out, int64_t window, double scale, double out_scale, bool chunked, double softcap,
+                      const OptTensor& sink, const OptTensor& gate, const Tensor& status) {
   TORCH_CHECK(q.scalar_type() == kBf16, "windowed_prefill: q");
   const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
+  const Options x = attend_options(chunked, softcap, sink, gate, a, q.scalar_type());
   TORCH_CHECK(q.size(2) == forge_windowed_prefill_qcols(i32(a.c.d), i32(a.c.dv), i32(a.c.block_size)), "windowed_prefill: q columns");
   const c10::cuda::CUDAGuard guard(q.device());
   check_rc(forge_windowed_prefill(q.data_ptr(), i32(a.T), k_cache.data_ptr(), v_cache.data_ptr(), ints(cu, seqs + 1, "cu"), ints(context_lens, seqs, "lens"),
                                   ints(tables, 0, "tables"), i32(tables.size(1)), i32(a.c.blocks), i32(a.c.block_size), out.data_ptr(), out.stride(0),
                                   i32(seqs), i32(max_q), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window), static_cast<float>(scale),
-                                  static_cast<float>(out_scale), status_word(status), stream_of(q)),
+                                  static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head, x.gate_col, status_word(status),
+                                  stream_of(q)),
            "forge_windowed_prefill");
 }
 
 // x [tokens, channels] (a view), taps [channels, n], state [slots, n - 1, channels], out [tokens, channels]
 void short_conv(const Tensor& x, const Tensor& taps, const OptTensor& bias, Tensor& state, const Tensor& slots, const Tensor& positions,
-                const Tensor& cu, int64_t seqs, int64_t max_q, Tensor& out, const Tensor& status) {
+                const Tensor& cu, int64_t seqs, int64_t max_q, Tensor& out, bool silu, const Tensor& status) {
   const int f = elem(x);
   const auto dt = x.scalar_type();
   TORCH_CHECK(taps.dim() == 2 && state.dim() == 3 && state.size(1) == taps.size(1) - 1 && state.size(2) == taps.size(0), "short_conv: sizes");
@@ -144,7 +236,7 @@ void short_conv(const Tensor& x, const Tensor& taps, const OptTensor& bias, Tens
   const c10::cuda::CUDAGuard guard(x.device());
   check_rc(forge_short_conv(f, view2(x, dt, T, C, "x"), x.stride(0), floats(taps, 0, "taps"), bias.has_value() ? floats(*bias, C, "bias") : nullptr,
                             data(state, dt, 0, "state"), ints(slots, seqs, "slots"), ints(positions, T, "positions"), ints(cu, seqs + 1, "cu"),
-                            i32(seqs), i32(max_q), data(out, dt, T * C, "out"), i32(C), i32(taps.size(1)), i32(state.size(0)), status_word(status),
+                            i32(seqs), i32(max_q), data(out, dt, T * C, "out"), i32(C), i32(taps.size(1)), i32(state.size(0)), silu ? 1 : 0, status_word(status),
                             stream_of(x)),
            "forge_short_conv");
 }
@@ -256,6 +348,8 @@ void gated_norm(const Tensor& o, const Tensor& gate, const Tensor& weight, Tenso
 
 void register_hybrid(pybind11::module& m) {
   m.def("bias_rope_store", &bias_rope_store);
+  m.def("norm_rope_store", &norm_rope_store);
+  m.def("stream_mix", &stream_mix);
   m.def("windowed_attend_any", &windowed_attend_any);
   m.def("windowed_decode", &windowed_decode);
   m.def("windowed_decode_ok", [](int64_t d, int64_t dv, int64_t bs) { return forge_windowed_decode_ok(i32(d), i32(dv), i32(bs)) != 0; });

@@ -1,4 +1,4 @@
-// silu of a causal convolution over time, per channel, with the last taps - 1 inputs of every sequence kept in its slot.
+// A causal convolution over time, per channel (and its silu, if asked), with the last taps - 1 inputs of every sequence kept in its slot.
 //
 // x [tokens][ldx] are the step's inputs, out [tokens][channels]; state [slots][taps - 1][channels] holds the inputs before
 // the step's first token (a sequence at position 0 has zeros before it, whatever its slot holds) and receives the last ones.
@@ -10,7 +10,7 @@
 
 namespace forge {
 
-constexpr int kConvMaxTaps = 8, kConvBatch = 4;
+constexpr int kConvMaxTaps = 8, kConvManyTaps = 32, kConvBatch = 4;
 
 template <typename T>
 struct ConvArgs {
@@ -23,22 +23,22 @@ struct ConvArgs {
   const int* positions;     // [tokens]
   const int* cu;            // [seqs + 1]
   T* out;
-  int channels, taps_n, num_slots, tile;
+  int channels, taps_n, num_slots, tile, silu;
   unsigned* status;
 };
 
-template <typename T, int N, int K>       // K: taps (0: any up to kConvMaxTaps)
+template <typename T, int N, int K>       // K: taps (0: any up to kConvMaxTaps; -1: up to kConvManyTaps)
 __global__ void __launch_bounds__(128) short_conv_kernel(const ConvArgs<T> p) {
-  constexpr int kTaps = K ? K : kConvMaxTaps;
-  const int taps = K ? K : p.taps_n;
+  constexpr int kTaps = K > 0 ? K : K == 0 ? kConvMaxTaps : kConvManyTaps;
+  const int taps = K > 0 ? K : p.taps_n;
   pdl_launch_dependents();
   pdl_wait();
   const int s = blockIdx.y, begin = p.cu[s], end = p.cu[s + 1];
   const int t0 = begin + blockIdx.x * p.tile, t1 = min(t0 + p.tile, end);
   const int c = (blockIdx.z * blockDim.x + threadIdx.x) * N;
   if (t0 >= end || c >= p.channels) return;
-  const int slot = p.slots[s];
-  const bool bad = slot < 0 || slot >= p.num_slots;
+  const int slot = taps > 1 ? p.slots[s] : 0;    // one tap: nothing is kept
+  const bool bad = taps > 1 && (slot < 0 || slot >= p.num_slots);
   if (bad) {                                     // padding rows have empty ranges: this is a corrupted step
     if (threadIdx.x == 0) set_status(p.status, kStatusBadIndex);
     return;
@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ConvArgs<T> p) {
 #pragma unroll
         for (int i = 0; i < kTaps; ++i)
           if (i < taps) a = fmaf(w[i][e], win[i][e], a);
-        y[e] = silu_t<T>(a);
+        y[e] = p.silu ? silu_t<T>(a) : a;
       }
       if (ta + k < t1) store_n<N>(p.out + static_cast<size_t>(ta + k) * p.channels + c, y);
 #pragma unroll
@@ -117,21 +117,22 @@ static int short_conv(const ConvArgs<T>& p, int seqs, int max_q, cudaStream_t st
   if (p.taps_n == 4) FORGE_CONV(4);
   if (p.taps_n == 3) FORGE_CONV(3);
   if (p.taps_n == 2) FORGE_CONV(2);
-  FORGE_CONV(0);
+  if (p.taps_n <= kConvMaxTaps) FORGE_CONV(0);
 #undef FORGE_CONV
+  return launch_kernel(short_conv_kernel<T, 1, -1>, dim3(grid.x, seqs, (p.channels + 127) / 128), dim3(128), 0, stream, 0, p) == cudaSuccess ? 0 : -2;
 }
 
 extern "C" int forge_short_conv(int fp32, const void* x, long long ldx, const float* taps, const float* bias, void* state, const int* slots,
                                 const int* positions, const int* cu, int seqs, int max_q, void* out, int channels, int taps_n, int num_slots,
-                                unsigned* status, cudaStream_t stream) {
+                                int silu, unsigned* status, cudaStream_t stream) {
   if (seqs <= 0 || max_q <= 0) return 0;
-  if (taps_n < 1 || taps_n > kConvMaxTaps) return -1;
+  if (taps_n < 1 || taps_n > kConvManyTaps) return -1;
   const int tile = max_q > 64 ? 64 : 32;
   if (fp32)
     return short_conv<float>({static_cast<const float*>(x), ldx, taps, bias, static_cast<float*>(state), slots, positions, cu, static_cast<float*>(out),
-                              channels, taps_n, num_slots, tile, status}, seqs, max_q, stream);
+                              channels, taps_n, num_slots, tile, silu, status}, seqs, max_q, stream);
   return short_conv<bf16>({static_cast<const bf16*>(x), ldx, taps, bias, static_cast<bf16*>(state), slots, positions, cu, static_cast<bf16*>(out),
-                           channels, taps_n, num_slots, tile, status}, seqs, max_q, stream);
+                           channels, taps_n, num_slots, tile, silu, status}, seqs, max_q, stream);
 }
 
 }  // namespace forge

@@ -30,10 +30,18 @@ class HybridOps:
         self.C.bias_rope_store(proj, bias, table, positions, slot_mapping, q, k_cache, v_cache, self.status)
         return q
 
-    def windowed_attention(self, q, k_cache, v_cache, batch, spec, out, scale) -> None:
-        """out (a view [T, heads * vdim]) <- scale * attention over the last ``spec.window`` tokens."""
+    def norm_rope_store(self, proj, q_norm, k_norm, eps, spec, table, positions, slot_mapping, k_cache, v_cache):
+        """q [T, heads, columns]: the columns from ``dim`` on are zero."""
+        cols = self.C.windowed_prefill_qcols(spec.dim, spec.vdim, k_cache.shape[2]) if proj.dtype == torch.bfloat16 else 0
+        q = torch.empty(proj.shape[0], spec.heads, cols or spec.dim, dtype=proj.dtype, device=proj.device)
+        self.C.norm_rope_store(proj, q_norm, k_norm, spec.norm == "all", eps, table, positions, slot_mapping, q, k_cache, v_cache, self.status)
+        return q
+
+    def windowed_attention(self, q, k_cache, v_cache, batch, spec, out, scale, chunked=False, softcap=0.0, sink=None, gate=None) -> None:
+        """out (a view [T, heads * vdim]) <- scale * attention over the last ``spec.window`` tokens, or inside chunks of that many."""
         d, dv, bs = spec.dim, spec.vdim, k_cache.shape[2]
         bf16, seqs = q.dtype == torch.bfloat16, batch.padded_seqs
+        options = (spec.window, spec.scale, scale, chunked, softcap, sink, gate, self.status)
         n1 = self._singles(batch)
         if n1 and bf16 and self.C.windowed_decode_ok(d, dv, bs):
             chunk, chunks = self.windowed_chunks(n1, spec, batch.table_width * bs)
@@ -41,19 +49,17 @@ class HybridOps:
             if chunks > 1:
                 part_o = torch.empty(n1 * spec.heads * chunks * dv, dtype=torch.float32, device=q.device)
                 part_ml = torch.empty(n1 * spec.heads * chunks * 2, dtype=torch.float32, device=q.device)
-            self.C.windowed_decode(q, k_cache, v_cache, batch.block_tables, batch.context_lens, n1, out, part_o, part_ml, chunk, chunks,
-                                   spec.window, spec.scale, scale, self.status)
+            self.C.windowed_decode(q, k_cache, v_cache, batch.block_tables, batch.context_lens, n1, out, part_o, part_ml, chunk, chunks, *options)
         else:
             n1 = 0
         if seqs == n1:
             return
         cu, tables = batch.cu_seqlens_q[n1:], batch.block_tables[n1:]
-        if bf16 and spec.scale > 0 and batch.is_prefill and q.shape[2] == self.C.windowed_prefill_qcols(d, dv, bs) and _aligned(out):
-            self.C.windowed_prefill(q, k_cache, v_cache, cu, batch.context_lens[n1:], tables, seqs - n1, batch.max_seqlen_q, out, spec.window,
-                                    spec.scale, scale, self.status)
+        rows = (out,) if gate is None or gate.shape[1] == spec.heads else (out, gate)
+        if bf16 and spec.scale > 0 and batch.is_prefill and q.shape[2] == self.C.windowed_prefill_qcols(d, dv, bs) and _aligned(*rows):
+            self.C.windowed_prefill(q, k_cache, v_cache, cu, batch.context_lens[n1:], tables, seqs - n1, batch.max_seqlen_q, out, *options)
         else:
-            self.C.windowed_attend_any(q, k_cache, v_cache, cu, seqs - n1, batch.max_seqlen_q, batch.positions, tables, out, spec.window,
-                                       spec.scale, scale, self.status)
+            self.C.windowed_attend_any(q, k_cache, v_cache, cu, seqs - n1, batch.max_seqlen_q, batch.positions, tables, out, *options)
 
     def windowed_chunks(self, seqs: int, spec, capacity: int) -> tuple[int, int]:
         """(keys per chunk, chunks): the window is cut until the two CTAs that an SM holds are busy.  Depends only on shapes known at
@@ -65,10 +71,10 @@ class HybridOps:
         return chunk, -(-span // chunk)
 
     # ------------------------------------------------------------------ recurrences
-    def short_conv(self, x, taps, bias, state, batch):
+    def short_conv(self, x, taps, bias, state, batch, act="silu"):
         out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
         self.C.short_conv(x, taps, bias, state, batch.state_slots, batch.positions, batch.cu_seqlens_q, batch.padded_seqs, batch.max_seqlen_q,
-                          out, self.status)
+                          out, act == "silu", self.status)
         return out
 
     def recur(self, q, k, v, dt, beta, block, state, batch):

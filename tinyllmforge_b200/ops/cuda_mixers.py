@@ -45,6 +45,14 @@ class MixerOps:
                              outs[0] if outs else None, outs[1] if len(outs) > 1 else None, rows, start, eps, dtype == torch.float32)
         return outs
 
+    def stream_mix(self, x, dtype, eps, into, norm, bias, y=None, mix=None, out=None, ids=None, prev=None, embed=None, scale=1.0, pairs=None,
+                   mul_prev=0, mul_cur=0, rows=None):
+        h = None
+        if norm is not None:
+            h = torch.empty(x.shape[0] if rows is None else rows.shape[0], x.shape[2], dtype=dtype, device=x.device)
+        self.C.stream_mix(x, y, mix, out, ids, prev, embed, scale, pairs, mul_prev, mul_cur, into, norm, bias, h, rows, eps, dtype == torch.float32)
+        return h
+
     # ------------------------------------------------------------------ products outside the tcgen05 GEMMs' reach
     @staticmethod
     def tma_ok(x: torch.Tensor, w: torch.Tensor) -> bool:
