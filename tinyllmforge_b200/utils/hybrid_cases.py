@@ -1,5 +1,5 @@
 """One-kernel cases of hybrid decoders (see ``kernel_case``): windowed attention, short convolution, recurrences with a decay per
-token, sandwich norms; sizes of a layer of width 2048.  Bytes and flops are those of the operation, as in ``mixer_cases``: the
+token, sandwich norms, attention with its options, several residual streams; sizes of a layer of width 2048.  Bytes and flops are those of the operation, as in ``mixer_cases``: the
 recurrences count the token-by-token products of their chunked form (chunks of 64)."""
 from __future__ import annotations
 
@@ -30,14 +30,20 @@ def _caches(b, s, block=256):
     return _rand(b.num_blocks, s.kv_heads, block, s.dim), _rand(b.num_blocks, s.kv_heads, block, s.vdim)
 
 
-def _attention(ops, seqs, q_len, ctx, window=None, heads=16):
+def _attention(ops, seqs, q_len, ctx, window=None, heads=16, kind=None):
+    """``kind``: None, "chunked" (chunks, sink, a gate per head) or "capped" (window, sink, bounded scores, a gate per element)."""
     s = Spec(**{**ATTENTION.__dict__, "heads": heads, "window": window or ATTENTION.window})
     b = _Batch(seqs, q_len, ctx)
     kc, vc = _caches(b, s)
     q, out = _rand(seqs * q_len, s.heads, s.dim), _rand(seqs * q_len, s.heads * s.vdim)
-    keys = sum(min(p + 1, s.window) for p in range(ctx - q_len, ctx)) * seqs            # (query, key) pairs per head
-    cached = seqs * min(ctx, s.window + q_len - 1) * s.kv_heads * (s.dim + s.vdim) * 2
-    return (lambda: ops.windowed_attention(q, kc, vc, b, s, out, 0.7), cached + seqs * q_len * s.heads * (s.dim + s.vdim) * 2,
+    oldest = (lambda p: p // s.window * s.window) if kind == "chunked" else (lambda p: max(p - s.window + 1, 0))
+    keys = sum(p + 1 - oldest(p) for p in range(ctx - q_len, ctx)) * seqs               # (query, key) pairs per head
+    cached = seqs * (ctx - oldest(ctx - q_len)) * s.kv_heads * (s.dim + s.vdim) * 2
+    options, gates = {}, 0
+    if kind is not None:
+        gates = {"chunked": s.heads, "capped": s.heads * s.vdim}[kind]
+        options = dict(chunked=kind == "chunked", softcap=50.0 if kind == "capped" else 0.0, sink=torch.zeros(s.heads, device="cuda"), gate=_rand(seqs * q_len, gates))
+    return (lambda: ops.windowed_attention(q, kc, vc, b, s, out, 0.7, **options), cached + seqs * q_len * (s.heads * (s.dim + s.vdim) + gates) * 2,
             2 * keys * s.heads * (s.dim + s.vdim) if q_len > 1 else 0)
 
 
@@ -48,6 +54,30 @@ def _bias_rope_store(ops, T):
     n = (s.heads + s.kv_heads) * s.dim + s.kv_heads * s.vdim
     proj, bias, table = _rand(T, n), torch.randn(n, device="cuda"), _rope(T, 64)
     return lambda: ops.bias_rope_store(proj, bias, s, table, b.positions, b.slot_mapping, kc, vc), 4 * T * n, 0
+
+
+def _norm_rope_store(ops, T, whole, rd):
+    s = Spec(**{**ATTENTION.__dict__, "norm": "all" if whole else "head"})
+    b = _Batch(1, T, T)
+    kc, vc = _caches(b, s)
+    n = (s.heads + s.kv_heads) * s.dim + s.kv_heads * s.vdim
+    proj, table = _rand(T, n), _rope(T, rd)
+    qw, kw = (torch.ones(h * s.dim if whole else s.dim, device="cuda") for h in (s.heads, s.kv_heads))
+    return lambda: ops.norm_rope_store(proj, qw, kw, 1e-6, s, table, b.positions, b.slot_mapping, kc, vc), 4 * T * n, 0
+
+
+def _stream_mix(ops, T, streams):
+    x, y, w, W = torch.randn(T, streams, WIDTH, device="cuda"), _rand(T, WIDTH), _rand(WIDTH), WIDTH
+    into, mix = torch.ones(streams, device="cuda"), torch.eye(streams, device="cuda")
+    return lambda: ops.stream_mix(x, BF, 1e-6, into, w, w, y=y, mix=mix, out=into), (8 * streams + 4) * T * W, 0
+
+
+def _stream_start(ops, T, streams):
+    x, embed, pairs, w, W = torch.empty(T, streams, WIDTH, device="cuda"), _rand(32000, WIDTH), _rand(8192, WIDTH), _rand(WIDTH), WIDTH
+    ids, prev = (torch.randint(0, 32000, (T,), dtype=torch.int32, device="cuda") for _ in range(2))
+    into = torch.ones(streams, device="cuda")
+    return (lambda: ops.stream_mix(x, BF, 1e-6, into, w, w, ids=ids, prev=prev, embed=embed, scale=45.0, pairs=pairs, mul_prev=31, mul_cur=7),
+            (4 * streams + 6) * T * W, 0)
 
 
 def _operands(s, T):
@@ -71,11 +101,11 @@ def _recurrence(ops, s, delta, seqs, q_len):
     return lambda: ops.recur(q, k, v, dt, beta if delta else None, block, state, b), moved, T * s.heads * per
 
 
-def _short_conv(ops, seqs, q_len):
-    C, T = 4096, seqs * q_len
+def _short_conv(ops, seqs, q_len, C=4096, act="silu"):
+    T = seqs * q_len
     b = _Batch(seqs, q_len, q_len if q_len > 1 else 700)
     x, taps, state = _rand(T, C), torch.randn(C, 4, device="cuda"), _rand(seqs, 3, C)
-    return lambda: ops.short_conv(x, taps, None, state, b), (4 * T * C if q_len > 1 else seqs * C * (4 + 12)), 0
+    return lambda: ops.short_conv(x, taps, None, state, b, act=act), (4 * T * C if q_len > 1 else seqs * C * (4 + 12)), 0
 
 
 def _gated_norm(ops, T, groups, first):
@@ -119,6 +149,20 @@ CASES = {
     "windowed_prefill": lambda ops: _attention(ops, 8, 2048, 2048),
     "windowed_prefill_long": lambda ops: _attention(ops, 1, 8192, 8192),
     "windowed_prefill_full": lambda ops: _attention(ops, 8, 2048, 2048, 2048),
+    "chunked_decode": lambda ops: _attention(ops, 64, 1, 2048, 4096, kind="chunked"),
+    "chunked_decode_b8": lambda ops: _attention(ops, 8, 1, 16384, 16384, kind="chunked"),
+    "capped_decode": lambda ops: _attention(ops, 64, 1, 2048, kind="capped"),
+    "capped_decode_b256": lambda ops: _attention(ops, 256, 1, 1500, kind="capped"),
+    "chunked_prefill": lambda ops: _attention(ops, 8, 2048, 2048, 4096, kind="chunked"),
+    "chunked_prefill_long": lambda ops: _attention(ops, 1, 8192, 8192, 4096, kind="chunked"),
+    "capped_prefill": lambda ops: _attention(ops, 8, 2048, 2048, kind="capped"),
+    "capped_prefill_long": lambda ops: _attention(ops, 1, 8192, 8192, kind="capped"),
+    "norm_rope_heads": lambda ops: _norm_rope_store(ops, 16384, False, 128),
+    "norm_rope_whole": lambda ops: _norm_rope_store(ops, 16384, True, 64),
+    "stream_mix2": lambda ops: _stream_mix(ops, 16384, 2),
+    "stream_mix4": lambda ops: _stream_mix(ops, 16384, 4),
+    "stream_start2": lambda ops: _stream_start(ops, 16384, 2),
+    "short_conv_plain": lambda ops: _short_conv(ops, 8, 2048, 3072, "none"),
     "bias_rope_store": lambda ops: _bias_rope_store(ops, 16384),
     "state_space_prefill": lambda ops: _recurrence(ops, SSD, False, 8, 2048),
     "state_space_prefill_long": lambda ops: _recurrence(ops, SSD, False, 1, 16384),
