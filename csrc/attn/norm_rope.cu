@@ -3,9 +3,8 @@
 // a head, entry i with i + rd / 2); q to [token][head][q_pitch] (padding columns zero), k and v to the caches
 // [block][kv_head][block_size][d / dv].
 //
-// CTA = a few tokens, one after the other.  L lanes (a power of two) share a head: a lane owns an item of N rotated pairs or of N
-// entries that pass.  Where every lane has one item at most and all heads fit the CTA (kOnce), weights stay in registers and the
-// row is read once; else rows are read again after the norm's sum.
+// CTA = one token.  L lanes (a power of two) share a head: a lane owns an item of N rotated pairs or of N entries that pass, of one
+// head or of several.
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
@@ -31,131 +30,179 @@ struct NormRope {
 };
 
 template <typename T, int N>
-struct RopeItem {
-  float a[N], b[N];
+struct alignas(sizeof(T) * N) Piece {       // N consecutive elements as they lie in memory
+  T v[N];
 };
+template <typename T, int N>
+__device__ __forceinline__ Piece<T, N> load_piece(const T* p) { return *reinterpret_cast<const Piece<T, N>*>(p); }
+template <typename T, int N>
+__device__ __forceinline__ Piece<T, N> zero_piece() {
+  Piece<T, N> r;
+#pragma unroll
+  for (int e = 0; e < N; ++e) store_f(&r.v[e], 0.f);
+  return r;
+}
 
-template <typename T, int N, bool kOnce, int kTok>
-__global__ void __launch_bounds__(512) norm_rope_kernel(const NormRope<T> p, int tokens) {
+// One token's sums of squares over all rows of q and of k -> their reciprocal root mean squares, for all threads.
+__device__ __forceinline__ void whole_norms(float& sq, float& sk, float (*red)[32], float nq, float nk, float eps) {
+  const int wl = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  sq = warp_sum_f(sq);
+  sk = warp_sum_f(sk);
+  if (wl == 0) {
+    red[0][warp] = sq;
+    red[1][warp] = sk;
+  }
+  __syncthreads();
+  sq = rsqrtf(warp_sum_f(wl < nw ? red[0][wl] : 0.f) / nq + eps);
+  sk = rsqrtf(warp_sum_f(wl < nw ? red[1][wl] : 0.f) / nk + eps);
+}
+
+template <typename T>
+struct TokenPlace {
+  bool stored;
+  size_t blk, off;
+  const float* rope;
+};
+template <typename T>
+__device__ __forceinline__ TokenPlace<T> token_place(const NormRope<T>& p, int t) {
+  const long long slot = p.slots[t];
+  int pos = p.positions[t];
+  pos = pos < 0 ? 0 : (pos >= p.rope_rows ? p.rope_rows - 1 : pos);
+  TokenPlace<T> r;
+  r.stored = slot >= 0 && slot < p.num_slots;
+  if (slot >= p.num_slots && threadIdx.x == 0) set_status(p.status, kStatusBadIndex);
+  const unsigned s = r.stored ? static_cast<unsigned>(slot) : 0u;      // num_slots fits 31 bits
+  r.blk = s / static_cast<unsigned>(p.block_size);
+  r.off = s % static_cast<unsigned>(p.block_size);
+  r.rope = p.rope + static_cast<size_t>(pos) * p.rd;
+  return r;
+}
+
+// R > 0: every lane has one item at most of each of up to R heads; all of the token's loads are under way before the first
+// sum.  R = 0: any sizes, items are read again after the norm's sum.
+template <typename T, int N, int R>
+__global__ void __launch_bounds__(512) norm_rope_kernel(const NormRope<T> p) {
   __shared__ float red[2][32];
   const int lane = threadIdx.x & ((1 << p.lanes_log2) - 1), L = 1 << p.lanes_log2;
   const int group = threadIdx.x >> p.lanes_log2, groups = blockDim.x >> p.lanes_log2, heads = p.H + p.G;
   const int half = p.rd >> 1, pairs = half / N, items = pairs + (p.d - p.rd) / N, padded = items + (p.q_pitch - p.d) / N;
   const int rounds = (heads + groups - 1) / groups;                    // the same for all threads: shuffles stay converged
-  auto load = [&](const T* row, int i, float* a, float* b) {           // item i of a head's row
-#pragma unroll
-    for (int e = 0; e < N; ++e) a[e] = b[e] = 0.f;
-    if (i < pairs) {
-      load_n<N>(row + i * N, a);
-      load_n<N>(row + i * N + half, b);
-    } else if (i < items) {
-      load_n<N>(row + p.rd + (i - pairs) * N, a);
-    }
-  };
-  auto weight = [&](int h, int i, float* wa, float* wb) {
-    const float* w = h < p.H ? p.q_norm + (p.whole ? static_cast<size_t>(h) * p.d : 0) : p.k_norm + (p.whole ? static_cast<size_t>(h - p.H) * p.d : 0);
-    if (i < pairs) {
-      load_n<N>(w + i * N, wa);
-      load_n<N>(w + i * N + half, wb);
-    } else if (i < items) {
-      load_n<N>(w + p.rd + (i - pairs) * N, wa);
-    }
-  };
-  float wa[N], wb[N];
-#pragma unroll
-  for (int e = 0; e < N; ++e) wa[e] = wb[e] = 0.f;
-  if (kOnce && group < heads) weight(group, lane, wa, wb);             // weights do not come from the kernel before
+  const int t = blockIdx.x;
+  const T* src = p.proj + static_cast<size_t>(t) * p.ld;
+  auto first = [&](int i) { return i < pairs ? i * N : p.rd + (i - pairs) * N; };
   pdl_launch_dependents();
   pdl_wait();
-  for (int u = 0; u < kTok; ++u) {
-    const int t = blockIdx.x * kTok + u;
-    if (t >= tokens) break;                                            // uniform for the CTA
-    const T* src = p.proj + static_cast<size_t>(t) * p.ld;
-    const long long slot = p.slots[t];
-    int pos = p.positions[t];
-    pos = pos < 0 ? 0 : (pos >= p.rope_rows ? p.rope_rows - 1 : pos);
-    const bool stored = slot >= 0 && slot < p.num_slots;
-    if (slot >= p.num_slots && threadIdx.x == 0) set_status(p.status, kStatusBadIndex);
-    const size_t blk = stored ? slot / p.block_size : 0, off = stored ? slot % p.block_size : 0;
-    float a[N], b[N];
+  using P = Piece<T, N>;
+  auto load = [&](int h, int i, P& a, P& b) {                          // item i of head h
+    const T* row = src + static_cast<size_t>(h) * p.d + first(i);
+    a = i < items ? load_piece<T, N>(row) : zero_piece<T, N>();
+    b = i < pairs ? load_piece<T, N>(row + half) : zero_piece<T, N>();
+  };
+  auto squares = [&](const P& a, const P& b) {
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < N; ++e) s = fmaf(load_f(&a.v[e]), load_f(&a.v[e]), fmaf(load_f(&b.v[e]), load_f(&b.v[e]), s));
+    return s;
+  };
+  auto store = [&](const TokenPlace<T>& at, int h, int i, const P& a, const P& b, float inv) {
+    const bool query = h < p.H;
+    if (i >= (query ? padded : items) || (!query && !at.stored)) return;
+    T* dst = (query ? p.q + (static_cast<size_t>(t) * p.H + h) * p.q_pitch : p.k_cache + ((at.blk * p.G + (h - p.H)) * p.block_size + at.off) * p.d) + first(i);
+    const float* w = (query ? p.q_norm + (p.whole ? h * p.d : 0) : p.k_norm + (p.whole ? (h - p.H) * p.d : 0)) + first(i);
+    float x[N], g[N];
+    if (i < items) load_n<N>(w, g);
+#pragma unroll
+    for (int e = 0; e < N; ++e) x[e] = i < items ? load_f(&a.v[e]) * inv * g[e] : 0.f;
+    if (i < pairs) {
+      float co[N], si[N], y[N];
+      load_n<N>(w + half, g);
+      load_n<N>(at.rope + i * N, co);
+      load_n<N>(at.rope + i * N + half, si);
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        const float z = load_f(&b.v[e]) * inv * g[e];
+        y[e] = z * co[e] + x[e] * si[e];
+        x[e] = x[e] * co[e] - z * si[e];
+      }
+      store_n<N>(dst + half, y);
+    }
+    store_n<N>(dst, x);
+  };
+  const T* values = src + static_cast<size_t>(heads) * p.d;
+  const int n_values = p.G * p.dv;
+  auto value_at = [&](const TokenPlace<T>& at, int i) { return p.v_cache + ((at.blk * p.G + i / p.dv) * p.block_size + at.off) * p.dv + i % p.dv; };
+
+  if constexpr (R > 0) {
+    P a[R], b[R], v;
+    float s[R], sq = 0.f, sk = 0.f;
+    const int vi = threadIdx.x * N;
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+      const int h = k * groups + group;
+      if (h < heads) load(h, lane, a[k], b[k]);
+      else a[k] = b[k] = zero_piece<T, N>();
+    }
+    v = vi < n_values ? load_piece<T, N>(values + vi) : zero_piece<T, N>();
+    const TokenPlace<T> at = token_place(p, t);
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+      s[k] = squares(a[k], b[k]);
+      if (k * groups + group < p.H) sq += s[k];
+      else sk += s[k];
+    }
+    if (at.stored) {
+      if (vi < n_values) *reinterpret_cast<P*>(value_at(at, vi)) = v;
+      for (int i = vi + blockDim.x * N; i < n_values; i += blockDim.x * N) *reinterpret_cast<P*>(value_at(at, i)) = load_piece<T, N>(values + i);
+    }
+    if (p.whole) whole_norms(sq, sk, red, static_cast<float>(p.H * p.d), static_cast<float>(p.G * p.d), p.eps);
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+      const int h = k * groups + group;
+      float inv = h < p.H ? sq : sk;
+      if (!p.whole) {
+        for (int o = L >> 1; o > 0; o >>= 1) s[k] += __shfl_xor_sync(0xffffffffu, s[k], o);
+        inv = rsqrtf(s[k] / static_cast<float>(p.d) + p.eps);
+      }
+      if (h < heads) store(at, h, lane, a[k], b[k], inv);
+    }
+  } else {
+    const TokenPlace<T> at = token_place(p, t);
+    P a, b;
+    auto head_sum = [&](int h) {
+      float s = 0.f;
+      if (h < heads)
+        for (int i = lane; i < items; i += L) {
+          load(h, i, a, b);
+          s += squares(a, b);
+        }
+      return s;
+    };
     float sq = 0.f, sk = 0.f;
-    if (kOnce && group < heads) load(src + static_cast<size_t>(group) * p.d, lane, a, b);
-    if (p.whole) {                                                     // uniform
+    if (p.whole) {
       for (int k = 0; k < rounds; ++k) {
         const int h = k * groups + group;
-        if (h >= heads) break;
-        float s = 0.f;
-        for (int i = lane; i < items; i += L) {
-          if (!kOnce) load(src + static_cast<size_t>(h) * p.d, i, a, b);
-#pragma unroll
-          for (int e = 0; e < N; ++e) s = fmaf(a[e], a[e], fmaf(b[e], b[e], s));
-        }
+        const float s = head_sum(h);
         if (h < p.H) sq += s;
         else sk += s;
       }
-      const int wl = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-      sq = warp_sum_f(sq);
-      sk = warp_sum_f(sk);
-      if (wl == 0) {
-        red[0][warp] = sq;
-        red[1][warp] = sk;
-      }
-      __syncthreads();
-      sq = rsqrtf(warp_sum_f(wl < nw ? red[0][wl] : 0.f) / static_cast<float>(p.H * p.d) + p.eps);
-      sk = rsqrtf(warp_sum_f(wl < nw ? red[1][wl] : 0.f) / static_cast<float>(p.G * p.d) + p.eps);
-      if (u + 1 < kTok) __syncthreads();
+      whole_norms(sq, sk, red, static_cast<float>(p.H * p.d), static_cast<float>(p.G * p.d), p.eps);
     }
     for (int k = 0; k < rounds; ++k) {
       const int h = k * groups + group;
-      const bool live = h < heads;
-      const T* row = src + static_cast<size_t>(live ? h : 0) * p.d;
       float inv = h < p.H ? sq : sk;
       if (!p.whole) {
-        float s = 0.f;
-        if (live)
-          for (int i = lane; i < items; i += L) {
-            if (!kOnce) load(row, i, a, b);
-#pragma unroll
-            for (int e = 0; e < N; ++e) s = fmaf(a[e], a[e], fmaf(b[e], b[e], s));
-          }
+        float s = head_sum(h);
         for (int o = L >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
         inv = rsqrtf(s / static_cast<float>(p.d) + p.eps);
       }
-      if (!live || (h >= p.H && !stored)) continue;
-      T* dst = h < p.H ? p.q + (static_cast<size_t>(t) * p.H + h) * p.q_pitch
-                       : p.k_cache + ((blk * p.G + (h - p.H)) * p.block_size + off) * p.d;
+      if (h >= heads) continue;
       for (int i = lane; i < (h < p.H ? padded : items); i += L) {
-        if (!kOnce) {
-          load(row, i, a, b);
-          weight(h, i, wa, wb);
-        }
-        if (i < pairs) {
-          const float* cs = p.rope + static_cast<size_t>(pos) * p.rd + i * N;
-          float co[N], si[N], x[N], y[N];
-          load_n<N>(cs, co);
-          load_n<N>(cs + half, si);
-#pragma unroll
-          for (int e = 0; e < N; ++e) {
-            const float v = a[e] * inv * wa[e], z = b[e] * inv * wb[e];
-            x[e] = v * co[e] - z * si[e];
-            y[e] = z * co[e] + v * si[e];
-          }
-          store_n<N>(dst + i * N, x);
-          store_n<N>(dst + i * N + half, y);
-        } else {
-          float x[N];
-#pragma unroll
-          for (int e = 0; e < N; ++e) x[e] = i < items ? a[e] * inv * wa[e] : 0.f;
-          store_n<N>(dst + p.rd + (i - pairs) * N, x);
-        }
+        load(h, i, a, b);
+        store(at, h, i, a, b, inv);
       }
     }
-    if (stored)
-      for (int i = threadIdx.x * N; i < p.G * p.dv; i += blockDim.x * N) {
-        float x[N];
-        load_n<N>(src + static_cast<size_t>(heads) * p.d + i, x);
-        store_n<N>(p.v_cache + ((blk * p.G + i / p.dv) * p.block_size + off) * p.dv + i % p.dv, x);
-      }
+    if (at.stored)
+      for (int i = threadIdx.x * N; i < n_values; i += blockDim.x * N) *reinterpret_cast<P*>(value_at(at, i)) = load_piece<T, N>(values + i);
   }
 }
 
@@ -165,13 +212,15 @@ static int norm_rope_n(NormRope<T> p, int tokens, cudaStream_t stream) {
   p.lanes_log2 = 0;
   while ((1 << p.lanes_log2) < items && p.lanes_log2 < 5) ++p.lanes_log2;
   const int L = 1 << p.lanes_log2;
-  const long long all = static_cast<long long>(heads) * L;
-  const bool once = items <= L && all <= 512;
-  const int threads = all >= 512 ? 512 : static_cast<int>((all + 31) / 32 * 32);
-  const bool four = tokens >= 2048;
-  auto k = once ? (four ? norm_rope_kernel<T, N, true, 4> : norm_rope_kernel<T, N, true, 1>)
-                : (four ? norm_rope_kernel<T, N, false, 4> : norm_rope_kernel<T, N, false, 1>);
-  return launch_kernel(k, dim3(four ? (tokens + 3) / 4 : tokens), dim3(threads), 0, stream, 0, p, tokens) == cudaSuccess ? 0 : -2;
+  // heads per lane: few threads and many tokens per SM where there are many tokens
+  int r = tokens >= 1024 ? 4 : 1;
+  auto threads_for = [&](int rounds) { return static_cast<int>((static_cast<long long>((heads + rounds - 1) / rounds) * L + 31) / 32 * 32); };
+  if (items > L) r = 0;
+  while (r > 0 && r < 4 && threads_for(r) > 512) r *= 2;
+  if (r > 0 && threads_for(r) > 512) r = 0;
+  const int threads = r > 0 ? threads_for(r) : heads >= 512 / L ? 512 : static_cast<int>((static_cast<long long>(heads) * L + 31) / 32 * 32);
+  auto k = r == 0 ? norm_rope_kernel<T, N, 0> : r == 1 ? norm_rope_kernel<T, N, 1> : r == 2 ? norm_rope_kernel<T, N, 2> : norm_rope_kernel<T, N, 4>;
+  return launch_kernel(k, dim3(tokens), dim3(threads), 0, stream, 0, p) == cudaSuccess ? 0 : -2;
 }
 
 template <typename T>
@@ -189,7 +238,7 @@ extern "C" int forge_norm_rope_store(int fp32, const void* proj, long long ld, i
                                      int q_pitch, void* k_cache, void* v_cache, long long num_slots, int block_size, int H, int G, int d, int dv,
                                      unsigned* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (rd < 0 || (rd & 1) || rd > d || q_pitch < d || (rd > 0 && rope_rows < 1)) return -1;
+  if (rd < 0 || (rd & 1) || rd > d || q_pitch < d || (rd > 0 && rope_rows < 1) || num_slots >= (1ll << 31)) return -1;
 #define FORGE_NORM_ROPE(T)                                                                                                             \
   return norm_rope<T>({static_cast<const T*>(proj), ld, q_norm, k_norm, rope, rope_rows, rd, positions, slots, static_cast<T*>(q),     \
                        static_cast<T*>(k_cache), static_cast<T*>(v_cache), num_slots, H, G, d, dv, q_pitch, block_size, whole, 0, eps, status}, tokens, stream)

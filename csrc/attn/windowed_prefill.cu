@@ -15,6 +15,8 @@
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
+#include <type_traits>
+
 namespace forge {
 
 constexpr int kXM = 128, kXN = 64, kXThreads = 192;
@@ -31,47 +33,86 @@ __device__ __forceinline__ uint64_t windowed_desc_mn(uint32_t smem_addr, uint32_
   return d;
 }
 
-// kMasked: only keys kbase + i in [lo, limit) count.
-template <bool kMasked>
-__device__ __forceinline__ float windowed_row_max(const uint32_t (&v)[kXN], int kbase, int lo, int limit) {
-  float m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+// Bounded scores: none; by an odd polynomial, where no score of the tile passes the bound before it is applied (|z| <= 1 in
+// cap tanh(z)), which is nearly always; by the exponential.  The exponential and the reciprocal of tanh would take three times the
+// special-function slots of the softmax itself.
+enum { kCapNone, kCapPoly, kCapExp };
+
+struct CapFactors {
+  float z, pre, post, c[7];   // z = raw * z; softcap_log2(raw, pre, post) = z (c0 + c1 z^2 + ...)
+};
+
+template <int kCap>
+__device__ __forceinline__ float windowed_exponent(float raw, float scale_log2, const CapFactors& f, float m_ref) {
+  if constexpr (kCap == kCapPoly) {
+    const float z = raw * f.z, t = z * z;
+    float y = f.c[6];
 #pragma unroll
-  for (int i = 0; i < kXN; i += 4)
+    for (int i = 5; i >= 0; --i) y = fmaf(y, t, f.c[i]);
+    return fmaf(z, y, -m_ref);
+  } else if constexpr (kCap == kCapExp) {
+    return softcap_log2(raw, f.pre, f.post) - m_ref;
+  } else {
+    return fmaf(raw, scale_log2, -m_ref);
+  }
+}
+
+// The scores of a tile are read from tensor memory twice, a few columns at a time: the loops stay short enough for the instruction
+// caches (unrolled over 64 columns, half of the issue slots went by waiting for instructions).
+constexpr int kXCols = 16;
+
+// Maximum of a row's scores over the keys kbase + i in [lo, limit) (kMasked) or all of the tile; `size`: the largest |score|, masked or not.
+template <bool kMasked, bool kSize>
+__device__ __forceinline__ float windowed_row_max(uint32_t s_addr, int kbase, int lo, int limit, float& size) {
+  float m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}, a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 1
+  for (int c = 0; c < kXN; c += 32) {
+    uint32_t v[32];
+    tmem_ld_x32(s_addr + c, v);
+    tmem_ld_wait();
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float x = __uint_as_float(v[i + e]);
-      const int key = kbase + i + e;
-      m[e] = fmaxf(m[e], (!kMasked || (key >= lo && key < limit)) ? x : -INFINITY);
+    for (int i = 0; i < 32; ++i) {
+      const float x = __uint_as_float(v[i]);
+      const int key = kbase + c + i;
+      m[i & 3] = fmaxf(m[i & 3], (!kMasked || (key >= lo && key < limit)) ? x : -INFINITY);
+      if (kSize) a[i & 3] = fmaxf(a[i & 3], fabsf(x));
     }
+  }
+  size = fmaxf(fmaxf(a[0], a[1]), fmaxf(a[2], a[3]));
   return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
 }
 
-// p = 2^(s scale - m_ref) of one row (kCap: of its bounded scores, s = raw, scale = the two factors of softcap_log2) -> hi and lo bf16 halves in shared memory (K-major, 128-byte swizzle); returns the row sum.
-template <bool kMasked, bool kCap>
-__device__ __forceinline__ float windowed_probs(const uint32_t (&v)[kXN], int kbase, int lo, int limit, float scale_log2, float cap_post, float m_ref,
+// p = 2^(s scale - m_ref) of one row -> hi and lo bf16 halves in shared memory (K-major, 128-byte swizzle); returns the row sum.
+template <bool kMasked, int kCap>
+__device__ __forceinline__ float windowed_probs(uint32_t s_addr, int kbase, int lo, int limit, float scale_log2, const CapFactors& cap, float m_ref,
                                                 uint8_t* p_row, int r) {
   float ps[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 1
+  for (int c0 = 0; c0 < kXN; c0 += kXCols) {
+    uint32_t v[kXCols];
+    tmem_ld_x16(s_addr + c0, v);
+    tmem_ld_wait();
 #pragma unroll
-  for (int c = 0; c < kXN; c += 8) {
-    uint32_t hi[4], lw[4];
+    for (int c = 0; c < kXCols; c += 8) {
+      uint32_t hi[4], lw[4];
 #pragma unroll
-    for (int i = 0; i < 8; i += 2) {
-      const int key = kbase + c + i;
-      const float s0 = __uint_as_float(v[c + i]), s1 = __uint_as_float(v[c + i + 1]);
-      float p0 = ex2_approx(kCap ? softcap_log2(s0, scale_log2, cap_post) - m_ref : fmaf(s0, scale_log2, -m_ref));
-      float p1 = ex2_approx(kCap ? softcap_log2(s1, scale_log2, cap_post) - m_ref : fmaf(s1, scale_log2, -m_ref));
-      if (kMasked) {
-        p0 = key >= lo && key < limit ? p0 : 0.f;
-        p1 = key + 1 >= lo && key + 1 < limit ? p1 : 0.f;
+      for (int i = 0; i < 8; i += 2) {
+        const int key = kbase + c0 + c + i;
+        float p0 = ex2_approx(windowed_exponent<kCap>(__uint_as_float(v[c + i]), scale_log2, cap, m_ref));
+        float p1 = ex2_approx(windowed_exponent<kCap>(__uint_as_float(v[c + i + 1]), scale_log2, cap, m_ref));
+        if (kMasked) {
+          p0 = key >= lo && key < limit ? p0 : 0.f;
+          p1 = key + 1 >= lo && key + 1 < limit ? p1 : 0.f;
+        }
+        ps[i >> 1] += p0 + p1;
+        const uint32_t h = pack_bf16x2(p0, p1);
+        hi[i >> 1] = h;
+        lw[i >> 1] = pack_bf16x2(p0 - bf16_lo(h), p1 - bf16_hi(h));
       }
-      ps[i >> 1] += p0 + p1;
-      const uint32_t h = pack_bf16x2(p0, p1);
-      hi[i >> 1] = h;
-      lw[i >> 1] = pack_bf16x2(p0 - bf16_lo(h), p1 - bf16_hi(h));
+      const int at = (((c0 + c) >> 3) ^ (r & 7)) << 4;
+      *reinterpret_cast<uint4*>(p_row + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(p_row + kXQBox + at) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
     }
-    const int at = ((c >> 3) ^ (r & 7)) << 4;
-    *reinterpret_cast<uint4*>(p_row + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-    *reinterpret_cast<uint4*>(p_row + kXQBox + at) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
   }
   return (ps[0] + ps[1]) + (ps[2] + ps[3]);
 }
@@ -80,16 +121,19 @@ struct WindowedPrefill {
   int H, G, d, dv, nq, nv, p_bufs, v_bufs;  // nq, nv: boxes of 64 columns of keys and of values
   int window, block_size, table_width, num_blocks;
   long long ldo;
-  float scale_log2, out_scale, cap_pre, cap_post;
+  float scale_log2, out_scale;
+  CapFactors cap;
   AttendOptions<bf16> opt;
 };
 
 // tm_q: [tokens, H * 64 nq], box 128 x 64; tm_k / tm_v: [blocks * G * block_size, d / dv], box 64 x 64.
-template <bool kCap>
+// kOptions 0: none; 1: chunks, sinks, gates; 2: these and bounded scores.
+template <int kOptions>
 __global__ void __launch_bounds__(kXThreads, 2)
 windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                         const int* __restrict__ cu_q, const int* __restrict__ context_lens, const int* __restrict__ tables,
                         bf16* __restrict__ out, const WindowedPrefill z, unsigned* status) {
+  constexpr bool kCap = kOptions == 2;
   extern __shared__ __align__(1024) uint8_t smem[];   // the swizzled boxes start on multiples of 1024 bytes
   const uint32_t k_stage = z.nq * kXKBox, v_stage = z.nv * kXKBox;
   uint8_t* sQ = smem;
@@ -121,7 +165,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   if (m0 >= q_len) return;                            // uniform for the CTA, before anything is allocated
   const int past = max(k_len - q_len, 0);
   const int kv_end = min(k_len, past + m0 + kXM);
-  const int tile0 = oldest_visible(past + m0, z.window, z.opt.chunked) / kXN;
+  const int tile0 = oldest_visible(past + m0, z.window, kOptions && z.opt.chunked) / kXN;
   const int n_tiles = (kv_end + kXN - 1) / kXN - tile0;
   if (n_tiles <= 0) return;
 
@@ -224,7 +268,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const int r = quad * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const int qpos = past + m0 + r;
-    const int limit = min(qpos + 1, k_len), lo = oldest_visible(qpos, z.window, z.opt.chunked);          // visible keys: [lo, limit)
+    const int limit = min(qpos + 1, k_len), lo = oldest_visible(qpos, z.window, kOptions && z.opt.chunked);          // visible keys: [lo, limit)
     const int o_cols = z.nv * 64;
     float m_ref = 0.f, l_run = 0.f;
     bool seen = false, ok = true;
@@ -234,16 +278,10 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       tcgen05_fence_after();
       const uint32_t s_addr = tmem_base + lane_addr + (j & 1) * kXN;
       const int kbase = (tile0 + j) * kXN;
-      uint32_t v[kXN];
-#pragma unroll
-      for (int c = 0; c < kXN; c += 32) tmem_ld_x32(s_addr + c, v + c);
-      tmem_ld_wait();
-      tcgen05_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&s_empty[j & 1]);
       const bool masked = !__all_sync(0xffffffffu, kbase >= lo && kbase + kXN <= limit);
-      float mt = masked ? windowed_row_max<true>(v, kbase, lo, limit) : windowed_row_max<false>(v, kbase, lo, limit);
-      mt = kCap && mt != -INFINITY ? softcap_log2(mt, z.cap_pre, z.cap_post) : mt * z.scale_log2;      // scale > 0: both keep the order
+      float size;
+      float mt = masked ? windowed_row_max<true, kCap>(s_addr, kbase, lo, limit, size) : windowed_row_max<false, kCap>(s_addr, kbase, lo, limit, size);
+      mt = kCap && mt != -INFINITY ? softcap_log2(mt, z.cap.pre, z.cap.post) : mt * z.scale_log2;      // scale > 0: both keep the order
       if (!seen && mt != -INFINITY) {                    // nothing of this row is in O yet, or only zeros
         m_ref = mt;
         seen = true;
@@ -277,25 +315,36 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         if (!ok) break;
       }
       uint8_t* p_row = sP + (j % z.p_bufs) * 2 * kXQBox + r * 128;
-      const float factor = kCap ? z.cap_pre : z.scale_log2;
-      l_run += masked ? windowed_probs<true, kCap>(v, kbase, lo, limit, factor, z.cap_post, m_ref, p_row, r)
-                      : windowed_probs<false, kCap>(v, kbase, lo, limit, factor, z.cap_post, m_ref, p_row, r);
+      auto probs = [&](auto masked_c, auto cap_c) {
+        return windowed_probs<decltype(masked_c)::value, decltype(cap_c)::value>(s_addr, kbase, lo, limit, z.scale_log2, z.cap, m_ref, p_row, r);
+      };
+      auto either = [&](auto cap_c) { return masked ? probs(std::true_type{}, cap_c) : probs(std::false_type{}, cap_c); };
+      if constexpr (kCap) {
+        const bool small = __all_sync(0xffffffffu, size * z.cap.z <= 1.f);
+        l_run += small ? either(std::integral_constant<int, kCapPoly>{}) : either(std::integral_constant<int, kCapExp>{});
+      } else {
+        l_run += either(std::integral_constant<int, kCapNone>{});
+      }
+      tcgen05_fence_before();
       fence_proxy_async_smem();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&p_full[j & 1]);
+      if (lane == 0) {
+        mbar_arrive(&s_empty[j & 1]);
+        mbar_arrive(&p_full[j & 1]);
+      }
     }
     if (ok) ok = mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, status);
     if (ok) {
       tcgen05_fence_after();
       float top = m_ref;
-      if (z.opt.sink != nullptr) {                       // one more score, of the denominator alone
+      if (kOptions && z.opt.sink != nullptr) {                       // one more score, of the denominator alone
         const float sink = z.opt.sink[h] * 1.4426950408889634f;
         top = fmaxf(m_ref, sink);
         l_run = fmaf(l_run, exp2f(m_ref - top), exp2f(sink - top));
       }
       const bool store = m0 + r < q_len;
       float inv = l_run > 0.f ? z.out_scale * exp2f(m_ref - top) / l_run : 0.f;
-      const bf16* gate = z.opt.gate == nullptr || !store ? nullptr : z.opt.gate + static_cast<size_t>(q_begin + m0 + r) * z.opt.ldg + static_cast<size_t>(h) * z.opt.gate_head;
+      const bf16* gate = !kOptions || z.opt.gate == nullptr || !store ? nullptr : z.opt.gate + static_cast<size_t>(q_begin + m0 + r) * z.opt.ldg + static_cast<size_t>(h) * z.opt.gate_head;
       if (gate != nullptr && z.opt.gate_col == 0) {      // one gate per head
         inv *= sigmoid_t<bf16>(load_f(gate));
         gate = nullptr;
@@ -327,6 +376,19 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     tcgen05_fence_after();
     tmem_dealloc(tmem_base, tmem_cols);
   }
+}
+
+static CapFactors cap_factors(float scale, float cap) {
+  CapFactors f = {};
+  if (cap > 0.f) {
+    // tanh(z) / z over z^2 <= 1: weighted least squares, refitted until the largest error of tanh was even (7e-8 in fp32)
+    constexpr float c[7] = {0.9999997020f, -0.3333213031f, 0.1331958175f, -0.0532657616f, 0.0199731588f, -0.0059511801f, 0.0009637412f};
+    f.z = scale / cap;
+    f.post = cap * 1.4426950408889634f;
+    f.pre = 2.f * 1.4426950408889634f * f.z;
+    for (int i = 0; i < 7; ++i) f.c[i] = f.post * c[i];
+  }
+  return f;
 }
 
 static int windowed_prefill_smem(int nq, int nv, int p_bufs, int v_bufs) {
@@ -367,16 +429,18 @@ extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_c
       }
   if (smem == 0) return -1;
   const WindowedPrefill z = {H, G, d, dv, nq, nv, p_bufs, v_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale,
-                             softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f, softcap * 1.4426950408889634f,
+                             cap_factors(scale, softcap),
                              {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}};
   CUtensorMap tm_q, tm_k, tm_v;
   const uint64_t qw = static_cast<uint64_t>(H) * qcols, rows = static_cast<uint64_t>(num_blocks) * G * block_size;
   if (forge_make_tmap_2d(&tm_q, q, tokens, qw, qw, kXM, 2) != 0) return -2;
   if (forge_make_tmap_2d(&tm_k, k_cache, rows, d, d, kXN, 2) != 0) return -2;
   if (forge_make_tmap_2d(&tm_v, v_cache, rows, dv, dv, kXN, 2) != 0) return -2;
-  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<false>, 227 * 1024);
-  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<true>, 227 * 1024);
-  return launch_kernel(softcap > 0.f ? windowed_prefill_kernel<true> : windowed_prefill_kernel<false>, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v,
+  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<0>, 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<1>, 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<2>, 227 * 1024);
+  auto k = softcap > 0.f ? windowed_prefill_kernel<2> : chunked || sink != nullptr || gate != nullptr ? windowed_prefill_kernel<1> : windowed_prefill_kernel<0>;
+  return launch_kernel(k, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v,
                        cu_q, context_lens, tables, static_cast<bf16*>(out), z, status) == cudaSuccess ? 0 : -5;
 }
 
