@@ -2,14 +2,14 @@
 // values read from the paged cache, key and value heads of different width (multiples of 8 up to 256).
 //
 //   S = Q K^T   K-major boxes of 64 columns; q rows are zero-padded to whole boxes, TMA fills the missing key columns with zeros
-//   O += P V    P = softmax weights in fp32, as bf16 hi + lo halves (two products: 16 mantissa bits), V as TMA delivers it
-//               (rows = keys, MN-major)
+//   O += P V    P = softmax weights in fp32, as bf16 hi + lo halves (two products: 16 mantissa bits) that take the place of S in
+//               tensor memory, V as TMA delivers it (rows = keys, MN-major)
 //
 // CTA = 128 query rows of one (sequence, head), key tiles of 64 from the tile that holds the first row's oldest visible key to
 // the tile of the last row's own.  A row may see nothing of its CTA's first tiles: its reference maximum is set by the first
 // key it does see, and nothing of O needs scaling then.  Warp roles, double-buffered S, the reference maximum that is only
-// raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu.  P and V are double-buffered where that leaves room for
-// two CTAs per SM (whose softmax warps hide each other's latency), else single-buffered, else as shared memory allows.
+// raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu.  V is double-buffered where that leaves room for two CTAs per
+// SM (whose softmax warps hide each other's latency), else single-buffered, else as shared memory allows.
 // Options (chunks, bounded scores, sinks, gated output): attend_options.cuh.
 #include "../include/attend_options.cuh"
 #include "../include/launch.cuh"
@@ -82,43 +82,37 @@ __device__ __forceinline__ float windowed_row_max(uint32_t s_addr, int kbase, in
   return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
 }
 
-// p = 2^(s scale - m_ref) of one row -> hi and lo bf16 halves in shared memory (K-major, 128-byte swizzle); returns the row sum.
+// p = 2^(s scale - m_ref) of one row, in place of its scores in tensor memory: the 16 columns of 16 keys take 8 columns of hi halves, then
+// 8 of lo halves, each an A operand of 16 entries.  Returns the row sum.
 template <bool kMasked, int kCap>
-__device__ __forceinline__ float windowed_probs(uint32_t s_addr, int kbase, int lo, int limit, float scale_log2, const CapFactors& cap, float m_ref,
-                                                uint8_t* p_row, int r) {
+__device__ __forceinline__ float windowed_probs(uint32_t s_addr, int kbase, int lo, int limit, float scale_log2, const CapFactors& cap, float m_ref) {
   float ps[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 1
-  for (int c0 = 0; c0 < kXN; c0 += kXCols) {
-    uint32_t v[kXCols];
-    tmem_ld_x16(s_addr + c0, v);
+  for (int c = 0; c < kXN; c += kXCols) {
+    uint32_t v[kXCols], w[kXCols];
+    tmem_ld_x16(s_addr + c, v);
     tmem_ld_wait();
 #pragma unroll
-    for (int c = 0; c < kXCols; c += 8) {
-      uint32_t hi[4], lw[4];
-#pragma unroll
-      for (int i = 0; i < 8; i += 2) {
-        const int key = kbase + c0 + c + i;
-        float p0 = ex2_approx(windowed_exponent<kCap>(__uint_as_float(v[c + i]), scale_log2, cap, m_ref));
-        float p1 = ex2_approx(windowed_exponent<kCap>(__uint_as_float(v[c + i + 1]), scale_log2, cap, m_ref));
-        if (kMasked) {
-          p0 = key >= lo && key < limit ? p0 : 0.f;
-          p1 = key + 1 >= lo && key + 1 < limit ? p1 : 0.f;
-        }
-        ps[i >> 1] += p0 + p1;
-        const uint32_t h = pack_bf16x2(p0, p1);
-        hi[i >> 1] = h;
-        lw[i >> 1] = pack_bf16x2(p0 - bf16_lo(h), p1 - bf16_hi(h));
+    for (int i = 0; i < kXCols; i += 2) {
+      const int key = kbase + c + i;
+      float p0 = ex2_approx(windowed_exponent<kCap>(__uint_as_float(v[i]), scale_log2, cap, m_ref));
+      float p1 = ex2_approx(windowed_exponent<kCap>(__uint_as_float(v[i + 1]), scale_log2, cap, m_ref));
+      if (kMasked) {
+        p0 = key >= lo && key < limit ? p0 : 0.f;
+        p1 = key + 1 >= lo && key + 1 < limit ? p1 : 0.f;
       }
-      const int at = (((c0 + c) >> 3) ^ (r & 7)) << 4;
-      *reinterpret_cast<uint4*>(p_row + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4*>(p_row + kXQBox + at) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+      ps[(i >> 1) & 3] += p0 + p1;
+      const uint32_t h = pack_bf16x2(p0, p1);
+      w[i >> 1] = h;
+      w[8 + (i >> 1)] = pack_bf16x2(p0 - bf16_lo(h), p1 - bf16_hi(h));
     }
+    tmem_st_x16(s_addr + c, w);
   }
   return (ps[0] + ps[1]) + (ps[2] + ps[3]);
 }
 
 struct WindowedPrefill {
-  int H, G, d, dv, nq, nv, p_bufs, v_bufs;  // nq, nv: boxes of 64 columns of keys and of values
+  int H, G, d, dv, nq, nv, v_bufs;          // nq, nv: boxes of 64 columns of keys and of values
   int window, block_size, table_width, num_blocks;
   long long ldo;
   float scale_log2, out_scale;
@@ -139,18 +133,16 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + z.nq * kXQBox;                   // [2 stages]
   uint8_t* sV = sK + 2 * k_stage;                     // [v_bufs]
-  uint8_t* sP = sV + z.v_bufs * v_stage;              // [p_bufs][hi, lo]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + z.p_bufs * 2 * kXQBox);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + z.v_bufs * v_stage);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;
   uint64_t* k_empty = bars + 3;
   uint64_t* v_full = bars + 5;
   uint64_t* v_empty = bars + 7;
   uint64_t* s_full = bars + 9;
-  uint64_t* s_empty = bars + 11;                      // one arrival per softmax warp
-  uint64_t* p_full = bars + 13;                       // one arrival per softmax warp
-  uint64_t* pv_done = bars + 15;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
+  uint64_t* p_full = bars + 11;                       // one arrival per softmax warp
+  uint64_t* pv_done = bars + 13;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
 
   pdl_launch_dependents();
   pdl_wait();
@@ -181,13 +173,12 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       mbar_init(&v_full[s], 1);
       mbar_init(&v_empty[s], 1);
       mbar_init(&s_full[s], 1);
-      mbar_init(&s_empty[s], 4);
       mbar_init(&p_full[s], 4);
       mbar_init(&pv_done[s], 1);
     }
     fence_mbar_init();
   }
-  const uint32_t tmem_cols = z.nv > 2 ? 512 : 256;    // S0 | S1 | O
+  const uint32_t tmem_cols = z.nv > 2 ? 512 : 256;    // S0 (P0) | S1 (P1) | O
   if (warp == 1) {
     tmem_alloc(tmem_slot, tmem_cols);
     tmem_relinquish();
@@ -224,13 +215,14 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc(kXM, kXN, 1, 1);
       const uint32_t idesc_o = umma_idesc(kXM, z.nv * 64, 1, 1) | (1u << 16);         // B (= V) MN-major
-      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
+      const uint32_t q_addr = smem_u32(sQ);
       const int steps = (z.d + 15) >> 4;
       bool ok = mbar_wait(q_full, 0, status);
       auto issue_s = [&](int j) -> bool {
         const int s = j & 1;
         if (!mbar_wait_parked(&k_full[s], (j >> 1) & 1, status)) return false;
-        if (!mbar_wait_parked(&s_empty[s], ((j >> 1) & 1) ^ 1, status)) return false; // softmax has read S of tile j - 2
+        // P V of tile j - 2 has read these columns
+        if (j >= 2 && !mbar_wait_parked(&pv_done[s], ((j - 2) >> 1) & 1, status)) return false;
         tcgen05_fence_after();
         const uint32_t k_addr = smem_u32(sK + s * k_stage);
         for (int k = 0; k < steps; ++k)
@@ -252,12 +244,12 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
         }
         tcgen05_fence_after();
         const uint32_t v_addr = smem_u32(sV + vs * v_stage);
-        const uint32_t pj_addr = p_addr + (j % z.p_bufs) * 2 * kXQBox;
+        const uint32_t p_addr = tmem_base + s * kXN;
 #pragma unroll
         for (int k = 0; k < kXN / 16; ++k) {
           const uint64_t vd = windowed_desc_mn(v_addr + k * 16 * 128, kXKBox);
-          umma_f16(tmem_o, umma_desc_k_sw128(pj_addr + k * 32), vd, idesc_o, (j | k) != 0);
-          umma_f16(tmem_o, umma_desc_k_sw128(pj_addr + kXQBox + k * 32), vd, idesc_o, 1);
+          umma_f16_ts(tmem_o, p_addr + k * 16, vd, idesc_o, (j | k) != 0);
+          umma_f16_ts(tmem_o, p_addr + k * 16 + 8, vd, idesc_o, 1);
         }
         umma_commit(&pv_done[s]);
         umma_commit(&v_empty[vs]);
@@ -309,14 +301,8 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
           m_ref = m_new;
         }
       }
-      if (j >= z.p_bufs) {                               // this P buffer was last read by P V of tile j - p_bufs
-        const int jj = j - z.p_bufs;
-        ok = mbar_wait(&pv_done[jj & 1], (jj >> 1) & 1, status);
-        if (!ok) break;
-      }
-      uint8_t* p_row = sP + (j % z.p_bufs) * 2 * kXQBox + r * 128;
       auto probs = [&](auto masked_c, auto cap_c) {
-        return windowed_probs<decltype(masked_c)::value, decltype(cap_c)::value>(s_addr, kbase, lo, limit, z.scale_log2, z.cap, m_ref, p_row, r);
+        return windowed_probs<decltype(masked_c)::value, decltype(cap_c)::value>(s_addr, kbase, lo, limit, z.scale_log2, z.cap, m_ref);
       };
       auto either = [&](auto cap_c) { return masked ? probs(std::true_type{}, cap_c) : probs(std::false_type{}, cap_c); };
       if constexpr (kCap) {
@@ -325,13 +311,10 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       } else {
         l_run += either(std::integral_constant<int, kCapNone>{});
       }
+      tmem_st_wait();
       tcgen05_fence_before();
-      fence_proxy_async_smem();
       __syncwarp();
-      if (lane == 0) {
-        mbar_arrive(&s_empty[j & 1]);
-        mbar_arrive(&p_full[j & 1]);
-      }
+      if (lane == 0) mbar_arrive(&p_full[j & 1]);
     }
     if (ok) ok = mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, status);
     if (ok) {
@@ -391,9 +374,7 @@ static CapFactors cap_factors(float scale, float cap) {
   return f;
 }
 
-static int windowed_prefill_smem(int nq, int nv, int p_bufs, int v_bufs) {
-  return nq * (kXQBox + 2 * kXKBox) + v_bufs * nv * kXKBox + p_bufs * 2 * kXQBox + 256;
-}
+static int windowed_prefill_smem(int nq, int nv, int v_bufs) { return nq * (kXQBox + 2 * kXKBox) + v_bufs * nv * kXKBox + 256; }
 
 // Columns of one head's padded query row, or 0 when the kernel does not take these sizes (else: windowed_attend_any).
 extern "C" int forge_windowed_prefill_qcols(int d, int dv, int block_size) {
@@ -418,17 +399,12 @@ extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_c
   if (gate != nullptr && gate_col != 0 && (gate_col != 1 || ((ldg | gate_head) & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -1;
   const int nq = qcols / 64, nv = (dv + 63) / 64;
   constexpr int kHalf = 113 * 1024, kAll = 227 * 1024;        // two CTAs per SM, one
-  const int bufs[3][2] = {{2, 2}, {1, 2}, {1, 1}};            // of P, of V
-  int smem = 0, p_bufs = 1, v_bufs = 1;
-  for (int limit = nv > 2 ? kAll : kHalf; smem == 0 && limit <= kAll; limit += kAll - kHalf)
-    for (int i = 0; i < 3 && smem == 0; ++i)
-      if (windowed_prefill_smem(nq, nv, bufs[i][0], bufs[i][1]) <= limit) {
-        p_bufs = bufs[i][0];
-        v_bufs = bufs[i][1];
-        smem = windowed_prefill_smem(nq, nv, p_bufs, v_bufs);
-      }
-  if (smem == 0) return -1;
-  const WindowedPrefill z = {H, G, d, dv, nq, nv, p_bufs, v_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale,
+  int v_bufs = 2;
+  if (nv <= 2 && windowed_prefill_smem(nq, nv, 2) > kHalf && windowed_prefill_smem(nq, nv, 1) <= kHalf) v_bufs = 1;
+  if (windowed_prefill_smem(nq, nv, v_bufs) > kAll) v_bufs = 1;
+  const int smem = windowed_prefill_smem(nq, nv, v_bufs);
+  if (smem > kAll) return -1;
+  const WindowedPrefill z = {H, G, d, dv, nq, nv, v_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale,
                              cap_factors(scale, softcap),
                              {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}};
   CUtensorMap tm_q, tm_k, tm_v;
