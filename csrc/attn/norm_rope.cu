@@ -3,8 +3,7 @@
 // a head, entry i with i + rd / 2); q to [token][head][q_pitch] (padding columns zero), k and v to the caches
 // [block][kv_head][block_size][d / dv].
 //
-// CTA = one token.  L lanes (a power of two) share a head: a lane owns an item of N rotated pairs or of N entries that pass, of one
-// head or of several.
+// The work of a token is a list of items: N rotated pairs or N entries that pass of a head, or N values.
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
@@ -14,8 +13,8 @@ template <typename T>
 struct NormRope {
   const T* proj;            // [tokens][ld]
   long long ld;
-  const float* q_norm;      // [d], or [H d] with `whole`
-  const float* k_norm;      // [d], or [G d]
+  const T* q_norm;          // [d], or [H d] with `whole`
+  const T* k_norm;          // [d], or [G d]
   const float* rope;        // [rope_rows][rd]
   int rope_rows, rd;
   const int* positions;
@@ -43,20 +42,6 @@ __device__ __forceinline__ Piece<T, N> zero_piece() {
   return r;
 }
 
-// One token's sums of squares over all rows of q and of k -> their reciprocal root mean squares, for all threads.
-__device__ __forceinline__ void whole_norms(float& sq, float& sk, float (*red)[32], float nq, float nk, float eps) {
-  const int wl = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  sq = warp_sum_f(sq);
-  sk = warp_sum_f(sk);
-  if (wl == 0) {
-    red[0][warp] = sq;
-    red[1][warp] = sk;
-  }
-  __syncthreads();
-  sq = rsqrtf(warp_sum_f(wl < nw ? red[0][wl] : 0.f) / nq + eps);
-  sk = rsqrtf(warp_sum_f(wl < nw ? red[1][wl] : 0.f) / nk + eps);
-}
-
 template <typename T>
 struct TokenPlace {
   bool stored;
@@ -70,7 +55,7 @@ __device__ __forceinline__ TokenPlace<T> token_place(const NormRope<T>& p, int t
   pos = pos < 0 ? 0 : (pos >= p.rope_rows ? p.rope_rows - 1 : pos);
   TokenPlace<T> r;
   r.stored = slot >= 0 && slot < p.num_slots;
-  if (slot >= p.num_slots && threadIdx.x == 0) set_status(p.status, kStatusBadIndex);
+  if (slot >= p.num_slots) set_status(p.status, kStatusBadIndex);
   const unsigned s = r.stored ? static_cast<unsigned>(slot) : 0u;      // num_slots fits 31 bits
   r.blk = s / static_cast<unsigned>(p.block_size);
   r.off = s % static_cast<unsigned>(p.block_size);
@@ -78,149 +63,276 @@ __device__ __forceinline__ TokenPlace<T> token_place(const NormRope<T>& p, int t
   return r;
 }
 
-// R > 0: every lane has one item at most of each of up to R heads; all of the token's loads are under way before the first
-// sum.  R = 0: any sizes, items are read again after the norm's sum.
-template <typename T, int N, int R>
-__global__ void __launch_bounds__(512) norm_rope_kernel(const NormRope<T> p) {
-  __shared__ float red[2][32];
-  const int lane = threadIdx.x & ((1 << p.lanes_log2) - 1), L = 1 << p.lanes_log2;
-  const int group = threadIdx.x >> p.lanes_log2, groups = blockDim.x >> p.lanes_log2, heads = p.H + p.G;
-  const int half = p.rd >> 1, pairs = half / N, items = pairs + (p.d - p.rd) / N, padded = items + (p.q_pitch - p.d) / N;
-  const int rounds = (heads + groups - 1) / groups;                    // the same for all threads: shuffles stay converged
-  const int t = blockIdx.x;
-  const T* src = p.proj + static_cast<size_t>(t) * p.ld;
-  auto first = [&](int i) { return i < pairs ? i * N : p.rd + (i - pairs) * N; };
-  pdl_launch_dependents();
-  pdl_wait();
-  using P = Piece<T, N>;
-  auto load = [&](int h, int i, P& a, P& b) {                          // item i of head h
-    const T* row = src + static_cast<size_t>(h) * p.d + first(i);
-    a = i < items ? load_piece<T, N>(row) : zero_piece<T, N>();
-    b = i < pairs ? load_piece<T, N>(row + half) : zero_piece<T, N>();
-  };
-  auto squares = [&](const P& a, const P& b) {
+// The items of a head: item i < pairs is N rotated pairs, i < items N entries that pass, i < padded (queries) N padding columns.
+template <typename T, int N>
+struct HeadItems {
+  int half, pairs, items, padded;
+  __device__ explicit HeadItems(const NormRope<T>& p)
+      : half(p.rd >> 1), pairs(half / N), items(pairs + (p.d - p.rd) / N), padded(items + (p.q_pitch - p.d) / N) {}
+  __device__ int first(const NormRope<T>& p, int i) const { return i < pairs ? i * N : p.rd + (i - pairs) * N; }
+};
+
+template <typename T, int N>
+struct Item {
+  Piece<T, N> a, b;         // entries at first and at first + half
+  Piece<T, N> wa, wb;       // their norm weights
+  int c;                    // first
+
+  __device__ __forceinline__ void weights(const NormRope<T>& p, const HeadItems<T, N>& z, int h, int i) {
+    const T* w = (h < p.H ? p.q_norm + (p.whole ? h * p.d : 0) : p.k_norm + (p.whole ? (h - p.H) * p.d : 0)) + z.first(p, i);
+    wa = i < z.items ? load_piece<T, N>(w) : zero_piece<T, N>();
+    wb = i < z.pairs ? load_piece<T, N>(w + z.half) : zero_piece<T, N>();
+  }
+  __device__ __forceinline__ void load(const NormRope<T>& p, const HeadItems<T, N>& z, const T* head, int i) {
+    c = z.first(p, i);
+    a = i < z.items ? load_piece<T, N>(head + c) : zero_piece<T, N>();
+    b = i < z.pairs ? load_piece<T, N>(head + c + z.half) : zero_piece<T, N>();
+  }
+  __device__ __forceinline__ float squares() const {
     float s = 0.f;
 #pragma unroll
     for (int e = 0; e < N; ++e) s = fmaf(load_f(&a.v[e]), load_f(&a.v[e]), fmaf(load_f(&b.v[e]), load_f(&b.v[e]), s));
     return s;
-  };
-  auto store = [&](const TokenPlace<T>& at, int h, int i, const P& a, const P& b, float inv) {
-    const bool query = h < p.H;
-    if (i >= (query ? padded : items) || (!query && !at.stored)) return;
-    T* dst = (query ? p.q + (static_cast<size_t>(t) * p.H + h) * p.q_pitch : p.k_cache + ((at.blk * p.G + (h - p.H)) * p.block_size + at.off) * p.d) + first(i);
-    const float* w = (query ? p.q_norm + (p.whole ? h * p.d : 0) : p.k_norm + (p.whole ? (h - p.H) * p.d : 0)) + first(i);
-    float x[N], g[N];
-    if (i < items) load_n<N>(w, g);
+  }
+  // co, si: the rotation of a pair item
+  __device__ __forceinline__ void store(const HeadItems<T, N>& z, T* dst, int i, float inv, const float* co, const float* si) const {
+    float x[N], y[N];
 #pragma unroll
-    for (int e = 0; e < N; ++e) x[e] = i < items ? load_f(&a.v[e]) * inv * g[e] : 0.f;
-    if (i < pairs) {
-      float co[N], si[N], y[N];
-      load_n<N>(w + half, g);
-      load_n<N>(at.rope + i * N, co);
-      load_n<N>(at.rope + i * N + half, si);
+    for (int e = 0; e < N; ++e) {
+      x[e] = load_f(&a.v[e]) * inv * load_f(&wa.v[e]);
+      y[e] = load_f(&b.v[e]) * inv * load_f(&wb.v[e]);
+    }
+    if (i < z.pairs) {
+      float u[N];
 #pragma unroll
       for (int e = 0; e < N; ++e) {
-        const float z = load_f(&b.v[e]) * inv * g[e];
-        y[e] = z * co[e] + x[e] * si[e];
-        x[e] = x[e] * co[e] - z * si[e];
+        u[e] = x[e] * co[e] - y[e] * si[e];
+        y[e] = y[e] * co[e] + x[e] * si[e];
       }
-      store_n<N>(dst + half, y);
+      store_n<N>(dst + c, u);
+      store_n<N>(dst + c + z.half, y);
+    } else {
+      store_n<N>(dst + c, x);
     }
-    store_n<N>(dst, x);
-  };
-  const T* values = src + static_cast<size_t>(heads) * p.d;
-  const int n_values = p.G * p.dv;
-  auto value_at = [&](const TokenPlace<T>& at, int i) { return p.v_cache + ((at.blk * p.G + i / p.dv) * p.block_size + at.off) * p.dv + i % p.dv; };
-
-  if constexpr (R > 0) {
-    P a[R], b[R], v;
-    float s[R], sq = 0.f, sk = 0.f;
-    const int vi = threadIdx.x * N;
-#pragma unroll
-    for (int k = 0; k < R; ++k) {
-      const int h = k * groups + group;
-      if (h < heads) load(h, lane, a[k], b[k]);
-      else a[k] = b[k] = zero_piece<T, N>();
-    }
-    v = vi < n_values ? load_piece<T, N>(values + vi) : zero_piece<T, N>();
-    const TokenPlace<T> at = token_place(p, t);
-#pragma unroll
-    for (int k = 0; k < R; ++k) {
-      s[k] = squares(a[k], b[k]);
-      if (k * groups + group < p.H) sq += s[k];
-      else sk += s[k];
-    }
-    if (at.stored) {
-      if (vi < n_values) *reinterpret_cast<P*>(value_at(at, vi)) = v;
-      for (int i = vi + blockDim.x * N; i < n_values; i += blockDim.x * N) *reinterpret_cast<P*>(value_at(at, i)) = load_piece<T, N>(values + i);
-    }
-    if (p.whole) whole_norms(sq, sk, red, static_cast<float>(p.H * p.d), static_cast<float>(p.G * p.d), p.eps);
-#pragma unroll
-    for (int k = 0; k < R; ++k) {
-      const int h = k * groups + group;
-      float inv = h < p.H ? sq : sk;
-      if (!p.whole) {
-        for (int o = L >> 1; o > 0; o >>= 1) s[k] += __shfl_xor_sync(0xffffffffu, s[k], o);
-        inv = rsqrtf(s[k] / static_cast<float>(p.d) + p.eps);
-      }
-      if (h < heads) store(at, h, lane, a[k], b[k], inv);
-    }
-  } else {
-    const TokenPlace<T> at = token_place(p, t);
-    P a, b;
-    auto head_sum = [&](int h) {
-      float s = 0.f;
-      if (h < heads)
-        for (int i = lane; i < items; i += L) {
-          load(h, i, a, b);
-          s += squares(a, b);
-        }
-      return s;
-    };
-    float sq = 0.f, sk = 0.f;
-    if (p.whole) {
-      for (int k = 0; k < rounds; ++k) {
-        const int h = k * groups + group;
-        const float s = head_sum(h);
-        if (h < p.H) sq += s;
-        else sk += s;
-      }
-      whole_norms(sq, sk, red, static_cast<float>(p.H * p.d), static_cast<float>(p.G * p.d), p.eps);
-    }
-    for (int k = 0; k < rounds; ++k) {
-      const int h = k * groups + group;
-      float inv = h < p.H ? sq : sk;
-      if (!p.whole) {
-        float s = head_sum(h);
-        for (int o = L >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-        inv = rsqrtf(s / static_cast<float>(p.d) + p.eps);
-      }
-      if (h >= heads) continue;
-      for (int i = lane; i < (h < p.H ? padded : items); i += L) {
-        load(h, i, a, b);
-        store(at, h, i, a, b, inv);
-      }
-    }
-    if (at.stored)
-      for (int i = threadIdx.x * N; i < n_values; i += blockDim.x * N) *reinterpret_cast<P*>(value_at(at, i)) = load_piece<T, N>(values + i);
   }
+};
+
+template <typename T>
+__device__ __forceinline__ T* head_place(const NormRope<T>& p, const TokenPlace<T>& at, int t, int h) {
+  return h < p.H ? p.q + (static_cast<size_t>(t) * p.H + h) * p.q_pitch : p.k_cache + ((at.blk * p.G + (h - p.H)) * p.block_size + at.off) * p.d;
+}
+template <typename T>
+__device__ __forceinline__ T* value_place(const NormRope<T>& p, const TokenPlace<T>& at, int i) {
+  return p.v_cache + ((at.blk * p.G + i / p.dv) * p.block_size + at.off) * p.dv + i % p.dv;
+}
+
+// A norm per head: L lanes take a head of a token (or its share of the values), whatever the token.  kOnce: one item per lane.
+template <typename T, int N, bool kOnce>
+__global__ void __launch_bounds__(256) norm_rope_heads_kernel(const NormRope<T> p, int units) {
+  const HeadItems<T, N> z(p);
+  const int L = 1 << p.lanes_log2, lane = threadIdx.x & (L - 1), all = p.H + 2 * p.G;
+  const int unit = blockIdx.x * (blockDim.x >> p.lanes_log2) + (threadIdx.x >> p.lanes_log2);
+  const bool live = unit < units;
+  const int t = live ? unit / all : 0, h = live ? unit % all : all;
+  const bool value = h >= p.H + p.G;
+  Item<T, N> it;
+  if (kOnce && !value) it.weights(p, z, h, lane);                      // weights do not come from the kernel before
+  pdl_launch_dependents();
+  pdl_wait();
+  const T* src = p.proj + static_cast<size_t>(t) * p.ld + (value ? static_cast<size_t>(p.H + p.G) * p.d + static_cast<size_t>(h - p.H - p.G) * p.dv
+                                                                 : static_cast<size_t>(h) * p.d);
+  float s = 0.f;
+  TokenPlace<T> at = {};
+  if (live) {
+    if (!value)
+      for (int i = lane; i < z.items; i += L) {
+        it.load(p, z, src, i);
+        s += it.squares();
+      }
+    if (kOnce && lane >= z.items) it.load(p, z, src, lane);
+    at = token_place(p, t);
+  }
+  float co[N], si[N];
+  if (kOnce && live && !value && lane < z.pairs) {
+    load_n<N>(at.rope + lane * N, co);
+    load_n<N>(at.rope + lane * N + z.half, si);
+  }
+  for (int o = L >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+  if (!live || (h >= p.H && !at.stored)) return;
+  if (value) {
+    for (int i = lane * N; i < p.dv; i += L * N)
+      *reinterpret_cast<Piece<T, N>*>(value_place(p, at, (h - p.H - p.G) * p.dv + i)) = load_piece<T, N>(src + i);
+    return;
+  }
+  const float inv = rsqrtf(s / static_cast<float>(p.d) + p.eps);
+  T* dst = head_place(p, at, t, h);
+  const int last = h < p.H ? z.padded : z.items;
+  if (kOnce) {
+    if (lane < last) it.store(z, dst, lane, inv, co, si);
+    return;
+  }
+  for (int i = lane; i < last; i += L) {
+    it.load(p, z, src, i);
+    it.weights(p, z, h, i);
+    if (i < z.pairs) {
+      load_n<N>(at.rope + i * N, co);
+      load_n<N>(at.rope + i * N + z.half, si);
+    }
+    it.store(z, dst, i, inv, co, si);
+  }
+}
+
+// A norm over all rows of q and one over all rows of k: CTA = one token.  kOnce: a thread has one item (or one piece of the values).
+template <typename T, int N, bool kOnce>
+__global__ void __launch_bounds__(kOnce ? 1024 : 512) norm_rope_whole_kernel(const NormRope<T> p) {
+  __shared__ float red[2][32];
+  const HeadItems<T, N> z(p);
+  const int heads = p.H + p.G, head_items = p.H * z.padded + p.G * z.items, items = head_items + p.G * p.dv / N, t = blockIdx.x;
+  auto split = [&](int k, int& h, int& i) {                            // item k of the token: of which head
+    const int kk = k - p.H * z.padded;
+    h = kk < 0 ? k / z.padded : p.H + kk / z.items;
+    i = kk < 0 ? k % z.padded : kk % z.items;
+  };
+  Item<T, N> it;
+  int h = 0, i = 0;
+  const int mine = threadIdx.x;
+  if (kOnce && mine < head_items) {
+    split(mine, h, i);
+    it.weights(p, z, h, i);
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  const T* src = p.proj + static_cast<size_t>(t) * p.ld;
+  const T* values = src + static_cast<size_t>(heads) * p.d;
+  float sq = 0.f, sk = 0.f;
+  for (int k = mine; k < (kOnce ? min(items, mine + 1) : head_items); k += blockDim.x) {
+    if (k < head_items) {
+      if (!kOnce) split(k, h, i);
+      it.load(p, z, src + static_cast<size_t>(h) * p.d, i);
+      const float s = it.squares();
+      if (h < p.H) sq += s;
+      else sk += s;
+    } else {
+      it.a = load_piece<T, N>(values + (k - head_items) * N);
+    }
+  }
+  const TokenPlace<T> at = token_place(p, t);
+  float co[N], si[N];
+  if (kOnce && mine < head_items && i < z.pairs) {
+    load_n<N>(at.rope + i * N, co);
+    load_n<N>(at.rope + i * N + z.half, si);
+  }
+  const int wl = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  sq = warp_sum_f(sq);
+  sk = warp_sum_f(sk);
+  if (wl == 0) {
+    red[0][warp] = sq;
+    red[1][warp] = sk;
+  }
+  __syncthreads();
+  sq = rsqrtf(warp_sum_f(wl < nw ? red[0][wl] : 0.f) / static_cast<float>(p.H * p.d) + p.eps);
+  sk = rsqrtf(warp_sum_f(wl < nw ? red[1][wl] : 0.f) / static_cast<float>(p.G * p.d) + p.eps);
+  for (int k = mine; k < (kOnce ? min(items, mine + 1) : items); k += blockDim.x) {
+    if (k >= head_items) {
+      const int v = (k - head_items) * N;
+      if (!kOnce) it.a = load_piece<T, N>(values + v);
+      if (at.stored) *reinterpret_cast<Piece<T, N>*>(value_place(p, at, v)) = it.a;
+      continue;
+    }
+    if (!kOnce) {
+      split(k, h, i);
+      it.load(p, z, src + static_cast<size_t>(h) * p.d, i);
+      it.weights(p, z, h, i);
+      if (i < z.pairs) {
+        load_n<N>(at.rope + i * N, co);
+        load_n<N>(at.rope + i * N + z.half, si);
+      }
+    }
+    if (h < p.H || at.stored) it.store(z, head_place(p, at, t, h), i, h < p.H ? sq : sk, co, si);
+  }
+}
+
+// Many tokens: a warp takes a token, L lanes a head at a time, one item per lane; the rotation and a head's weights stay in registers, the
+// next heads' entries are under way while these are stored.  With kWhole a first round over the heads takes the sums.
+template <typename T, int N, bool kWhole>
+__global__ void __launch_bounds__(256) norm_rope_warp_kernel(const NormRope<T> p, int tokens) {
+  const HeadItems<T, N> z(p);
+  const int L = 1 << p.lanes_log2, warp_lane = threadIdx.x & 31, lane = warp_lane & (L - 1), group = warp_lane >> p.lanes_log2, step = 32 >> p.lanes_log2;
+  const int heads = p.H + p.G, t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  Item<T, N> it, next;
+  if (!kWhole) it.weights(p, z, 0, lane);                              // weights do not come from the kernel before
+  pdl_launch_dependents();
+  pdl_wait();
+  if (t >= tokens) return;                                             // uniform for the warp
+  const T* src = p.proj + static_cast<size_t>(t) * p.ld;
+  const TokenPlace<T> at = token_place(p, t);
+  float sq = 0.f, sk = 0.f;
+  if (kWhole) {
+#pragma unroll 4
+    for (int h = group; h < heads; h += step) {
+      next.load(p, z, src + static_cast<size_t>(h) * p.d, lane);
+      const float s = next.squares();
+      if (h < p.H) sq += s;
+      else sk += s;
+    }
+    sq = rsqrtf(warp_sum_f(sq) / static_cast<float>(p.H * p.d) + p.eps);
+    sk = rsqrtf(warp_sum_f(sk) / static_cast<float>(p.G * p.d) + p.eps);
+  }
+  float co[N], si[N];
+#pragma unroll
+  for (int e = 0; e < N; ++e) co[e] = si[e] = 0.f;
+  if (lane < z.pairs) {
+    load_n<N>(at.rope + lane * N, co);
+    load_n<N>(at.rope + lane * N + z.half, si);
+  }
+  next.load(p, z, src + static_cast<size_t>(min(group, heads - 1)) * p.d, lane);
+  bool keys = false;
+  for (int h0 = 0; h0 < heads; h0 += step) {                           // the same for all lanes: shuffles stay converged
+    const int h = h0 + group;
+    it.a = next.a;
+    it.b = next.b;
+    it.c = next.c;
+    if (h0 + step < heads) next.load(p, z, src + static_cast<size_t>(min(h + step, heads - 1)) * p.d, lane);
+    float inv = h < p.H ? sq : sk;
+    if (!kWhole) {
+      float s = it.squares();
+      for (int o = L >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      inv = rsqrtf(s / static_cast<float>(p.d) + p.eps);
+    }
+    if (h >= heads || (h >= p.H && !at.stored)) continue;
+    if (kWhole || (h >= p.H && !keys)) {
+      it.weights(p, z, h, lane);
+      keys = h >= p.H;
+    }
+    if (lane < (h < p.H ? z.padded : z.items)) it.store(z, head_place(p, at, t, h), lane, inv, co, si);
+  }
+  if (!at.stored) return;
+  const T* values = src + static_cast<size_t>(heads) * p.d;
+  for (int i = warp_lane * N; i < p.G * p.dv; i += 32 * N) *reinterpret_cast<Piece<T, N>*>(value_place(p, at, i)) = load_piece<T, N>(values + i);
 }
 
 template <typename T, int N>
 static int norm_rope_n(NormRope<T> p, int tokens, cudaStream_t stream) {
-  const int items = (p.rd >> 1) / N + (p.q_pitch - p.rd) / N, heads = p.H + p.G;
+  const int pairs = (p.rd >> 1) / N, items = pairs + (p.d - p.rd) / N, padded = pairs + (p.q_pitch - p.rd) / N;
   p.lanes_log2 = 0;
-  while ((1 << p.lanes_log2) < items && p.lanes_log2 < 5) ++p.lanes_log2;
-  const int L = 1 << p.lanes_log2;
-  // heads per lane: few threads and many tokens per SM where there are many tokens
-  int r = tokens >= 1024 ? 4 : 1;
-  auto threads_for = [&](int rounds) { return static_cast<int>((static_cast<long long>((heads + rounds - 1) / rounds) * L + 31) / 32 * 32); };
-  if (items > L) r = 0;
-  while (r > 0 && r < 4 && threads_for(r) > 512) r *= 2;
-  if (r > 0 && threads_for(r) > 512) r = 0;
-  const int threads = r > 0 ? threads_for(r) : heads >= 512 / L ? 512 : static_cast<int>((static_cast<long long>(heads) * L + 31) / 32 * 32);
-  auto k = r == 0 ? norm_rope_kernel<T, N, 0> : r == 1 ? norm_rope_kernel<T, N, 1> : r == 2 ? norm_rope_kernel<T, N, 2> : norm_rope_kernel<T, N, 4>;
-  return launch_kernel(k, dim3(tokens), dim3(threads), 0, stream, 0, p) == cudaSuccess ? 0 : -2;
+  while ((1 << p.lanes_log2) < padded && p.lanes_log2 < 5) ++p.lanes_log2;
+  if (tokens >= 2048 && padded <= (1 << p.lanes_log2)) {
+    auto k = p.whole ? norm_rope_warp_kernel<T, N, true> : norm_rope_warp_kernel<T, N, false>;
+    return launch_kernel(k, dim3((tokens + 7) / 8), dim3(256), 0, stream, 0, p, tokens) == cudaSuccess ? 0 : -2;
+  }
+  if (p.whole) {
+    const long long all = static_cast<long long>(p.H) * padded + static_cast<long long>(p.G) * items + static_cast<long long>(p.G) * p.dv / N;
+    if (all >= (1ll << 31)) return -1;
+    const bool once = all <= 1024;
+    const int threads = all >= 512 && !once ? 512 : static_cast<int>((all + 31) / 32 * 32);
+    auto k = once ? norm_rope_whole_kernel<T, N, true> : norm_rope_whole_kernel<T, N, false>;
+    return launch_kernel(k, dim3(tokens), dim3(threads), 0, stream, 0, p) == cudaSuccess ? 0 : -2;
+  }
+  const long long units = static_cast<long long>(tokens) * (p.H + 2 * p.G);
+  const int per = 256 >> p.lanes_log2;
+  if (units >= (1ll << 31) - 256) return -1;
+  auto k = padded <= (1 << p.lanes_log2) ? norm_rope_heads_kernel<T, N, true> : norm_rope_heads_kernel<T, N, false>;
+  return launch_kernel(k, dim3(static_cast<unsigned>((units + per - 1) / per)), dim3(256), 0, stream, 0, p, static_cast<int>(units)) == cudaSuccess ? 0 : -2;
 }
 
 template <typename T>
@@ -233,14 +345,14 @@ static int norm_rope(const NormRope<T>& p, int tokens, cudaStream_t stream) {
 }
 
 // whole: the norms run over all rows of q and of k at once (weights [H d] and [G d]), else over each head (weights [d]).
-extern "C" int forge_norm_rope_store(int fp32, const void* proj, long long ld, int tokens, const float* q_norm, const float* k_norm, int whole,
+extern "C" int forge_norm_rope_store(int fp32, const void* proj, long long ld, int tokens, const void* q_norm, const void* k_norm, int whole,
                                      float eps, const float* rope, int rope_rows, int rd, const int* positions, const int* slots, void* q,
                                      int q_pitch, void* k_cache, void* v_cache, long long num_slots, int block_size, int H, int G, int d, int dv,
                                      unsigned* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (rd < 0 || (rd & 1) || rd > d || q_pitch < d || (rd > 0 && rope_rows < 1) || num_slots >= (1ll << 31)) return -1;
 #define FORGE_NORM_ROPE(T)                                                                                                             \
-  return norm_rope<T>({static_cast<const T*>(proj), ld, q_norm, k_norm, rope, rope_rows, rd, positions, slots, static_cast<T*>(q),     \
+  return norm_rope<T>({static_cast<const T*>(proj), ld, static_cast<const T*>(q_norm), static_cast<const T*>(k_norm), rope, rope_rows, rd, positions, slots, static_cast<T*>(q),     \
                        static_cast<T*>(k_cache), static_cast<T*>(v_cache), num_slots, H, G, d, dv, q_pitch, block_size, whole, 0, eps, status}, tokens, stream)
   if (fp32) FORGE_NORM_ROPE(float);
   FORGE_NORM_ROPE(bf16);

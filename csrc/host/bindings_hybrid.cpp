@@ -10,7 +10,7 @@ int forge_windowed_attend_any(int fp32, const void* q, int q_pitch, const void* 
                               const int* positions, const int* tables, int width, int num_blocks, int block_size, void* out, long long ldo, int H,
                               int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap, const float* sink,
                               const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status, cudaStream_t stream);
-int forge_norm_rope_store(int fp32, const void* proj, long long ld, int tokens, const float* q_norm, const float* k_norm, int whole, float eps,
+int forge_norm_rope_store(int fp32, const void* proj, long long ld, int tokens, const void* q_norm, const void* k_norm, int whole, float eps,
                           const float* rope, int rope_rows, int rd, const int* positions, const int* slots, void* q, int q_pitch, void* k_cache,
                           void* v_cache, long long num_slots, int block_size, int H, int G, int d, int dv, unsigned* status, cudaStream_t stream);
 int forge_stream_mix(int fp32, float* x, const void* y, const float* mix, const float* out, const int* ids, const int* prev, const void* embed,
@@ -88,8 +88,8 @@ void norm_rope_store(const Tensor& proj, const Tensor& q_norm, const Tensor& k_n
   TORCH_CHECK(q.dim() == 3 && q.size(0) == proj.size(0) && rope.dim() == 2 && rope.size(1) % 2 == 0 && rope.size(1) <= c.d && q.size(2) >= c.d, "norm_rope_store: sizes");
   const int64_t T = proj.size(0), H = q.size(1), rows = (H + c.G) * c.d + c.G * c.dv;
   const c10::cuda::CUDAGuard guard(proj.device());
-  check_rc(forge_norm_rope_store(f, view2(proj, dt, T, rows, "proj"), proj.stride(0), i32(T), floats(q_norm, whole ? H * c.d : c.d, "q_norm"),
-                                 floats(k_norm, whole ? c.G * c.d : c.d, "k_norm"), whole ? 1 : 0, static_cast<float>(eps), floats(rope, 0, "rope"),
+  check_rc(forge_norm_rope_store(f, view2(proj, dt, T, rows, "proj"), proj.stride(0), i32(T), data(q_norm, dt, whole ? H * c.d : c.d, "q_norm"),
+                                 data(k_norm, dt, whole ? c.G * c.d : c.d, "k_norm"), whole ? 1 : 0, static_cast<float>(eps), floats(rope, 0, "rope"),
                                  i32(rope.size(0)), i32(rope.size(1)), ints(positions, T, "positions"), ints(slots, T, "slots"), data(q, dt, 0, "q"),
                                  i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), static_cast<long long>(c.blocks) * c.block_size,
                                  i32(c.block_size), i32(H), i32(c.G), i32(c.d), i32(c.dv), status_word(status), stream_of(proj)),

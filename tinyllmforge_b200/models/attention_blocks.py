@@ -22,7 +22,7 @@ class NormedAttention:
         self.channels = sum(n for _, n in self.sizes)
         self.inp = _packed(self.channels + s.gate_columns, width, dtype, device)
         self.conv = _f32((self.channels, s.conv), device) if s.conv else None
-        self.q_norm, self.k_norm = (_f32(s.dim if s.norm == "head" else n, device) for _, n in self.sizes[:2])
+        self.q_norm, self.k_norm = (torch.ones(s.dim if s.norm == "head" else n, dtype=dtype, device=device) for _, n in self.sizes[:2])
         self.sink = None if s.sink is None else torch.zeros(s.heads, dtype=torch.float32, device=device)
         self.o = _empty((width, s.heads * s.vdim), dtype, device)
         self.rope = rope(s.rot)

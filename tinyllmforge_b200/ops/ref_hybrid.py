@@ -34,7 +34,7 @@ def norm_rope_store(proj, q_norm, k_norm, eps, spec, table, positions, slot_mapp
 
     def normed(x, w, heads):
         x = x.float().reshape((T, heads, d) if spec.norm == "head" else (T, heads * d))
-        return apply_partial_rope((x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps) * w).view(T, heads, d), positions, table)
+        return apply_partial_rope((x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps) * w.float()).view(T, heads, d), positions, table)
 
     q, k, v = proj.split([H * d, G * d, G * spec.vdim], dim=-1)
     store_kv(normed(k, k_norm, G), v.reshape(T, G, spec.vdim), k_cache, v_cache, slot_mapping)

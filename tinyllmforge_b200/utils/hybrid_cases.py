@@ -62,7 +62,7 @@ def _norm_rope_store(ops, T, whole, rd):
     kc, vc = _caches(b, s)
     n = (s.heads + s.kv_heads) * s.dim + s.kv_heads * s.vdim
     proj, table = _rand(T, n), _rope(T, rd)
-    qw, kw = (torch.ones(h * s.dim if whole else s.dim, device="cuda") for h in (s.heads, s.kv_heads))
+    qw, kw = (_rand(h * s.dim if whole else s.dim) for h in (s.heads, s.kv_heads))
     return lambda: ops.norm_rope_store(proj, qw, kw, 1e-6, s, table, b.positions, b.slot_mapping, kc, vc), 4 * T * n, 0
 
 
