@@ -3,7 +3,7 @@
 // a head, entry i with i + rd / 2); q to [token][head][q_pitch] (padding columns zero), k and v to the caches
 // [block][kv_head][block_size][d / dv].
 //
-// The work of a token is a list of items: N rotated pairs or N entries that pass of a head, or N values.
+// The work of a token is a list of items: N rotated pairs or 2 N entries that pass of a head, or N values.
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
@@ -63,30 +63,35 @@ __device__ __forceinline__ TokenPlace<T> token_place(const NormRope<T>& p, int t
   return r;
 }
 
-// The items of a head: item i < pairs is N rotated pairs, i < items N entries that pass, i < padded (queries) N padding columns.
+// The items of a head, two pieces of N entries each: item i < pairs is N rotated pairs, i < items two neighbouring pieces that pass (the
+// second may be missing), i < padded (queries) reaches into the padding columns.
+__host__ __device__ __forceinline__ int items_of(int pairs, int passing) { return pairs + ((passing + 1) >> 1); }
+
 template <typename T, int N>
 struct HeadItems {
-  int half, pairs, items, padded;
+  int pairs, items, padded;
   __device__ explicit HeadItems(const NormRope<T>& p)
-      : half(p.rd >> 1), pairs(half / N), items(pairs + (p.d - p.rd) / N), padded(items + (p.q_pitch - p.d) / N) {}
-  __device__ int first(const NormRope<T>& p, int i) const { return i < pairs ? i * N : p.rd + (i - pairs) * N; }
+      : pairs((p.rd >> 1) / N), items(items_of(pairs, (p.d - p.rd) / N)), padded(items_of(pairs, (p.q_pitch - p.rd) / N)) {}
 };
 
 template <typename T, int N>
 struct Item {
-  Piece<T, N> a, b;         // entries at first and at first + half
+  Piece<T, N> a, b;         // entries at c and at c2
   Piece<T, N> wa, wb;       // their norm weights
-  int c;                    // first
+  int c, c2;
 
-  __device__ __forceinline__ void weights(const NormRope<T>& p, const HeadItems<T, N>& z, int h, int i) {
-    const T* w = (h < p.H ? p.q_norm + (p.whole ? h * p.d : 0) : p.k_norm + (p.whole ? (h - p.H) * p.d : 0)) + z.first(p, i);
-    wa = i < z.items ? load_piece<T, N>(w) : zero_piece<T, N>();
-    wb = i < z.pairs ? load_piece<T, N>(w + z.half) : zero_piece<T, N>();
+  __device__ __forceinline__ void place(const NormRope<T>& p, const HeadItems<T, N>& z, int i) {
+    c = i < z.pairs ? i * N : p.rd + 2 * (i - z.pairs) * N;
+    c2 = c + (i < z.pairs ? p.rd >> 1 : N);
   }
-  __device__ __forceinline__ void load(const NormRope<T>& p, const HeadItems<T, N>& z, const T* head, int i) {
-    c = z.first(p, i);
-    a = i < z.items ? load_piece<T, N>(head + c) : zero_piece<T, N>();
-    b = i < z.pairs ? load_piece<T, N>(head + c + z.half) : zero_piece<T, N>();
+  __device__ __forceinline__ void weights(const NormRope<T>& p, int h) {
+    const T* w = h < p.H ? p.q_norm + (p.whole ? h * p.d : 0) : p.k_norm + (p.whole ? (h - p.H) * p.d : 0);
+    wa = c < p.d ? load_piece<T, N>(w + c) : zero_piece<T, N>();
+    wb = c2 < p.d ? load_piece<T, N>(w + c2) : zero_piece<T, N>();
+  }
+  __device__ __forceinline__ void load(const NormRope<T>& p, const T* head) {
+    a = c < p.d ? load_piece<T, N>(head + c) : zero_piece<T, N>();
+    b = c2 < p.d ? load_piece<T, N>(head + c2) : zero_piece<T, N>();
   }
   __device__ __forceinline__ float squares() const {
     float s = 0.f;
@@ -94,28 +99,33 @@ struct Item {
     for (int e = 0; e < N; ++e) s = fmaf(load_f(&a.v[e]), load_f(&a.v[e]), fmaf(load_f(&b.v[e]), load_f(&b.v[e]), s));
     return s;
   }
-  // co, si: the rotation of a pair item
-  __device__ __forceinline__ void store(const HeadItems<T, N>& z, T* dst, int i, float inv, const float* co, const float* si) const {
+  // co, si: 1 and 0 where the entries pass; cols: columns of a row at dst
+  __device__ __forceinline__ void store(T* dst, int cols, float inv, const float* co, const float* si) const {
     float x[N], y[N];
 #pragma unroll
     for (int e = 0; e < N; ++e) {
-      x[e] = load_f(&a.v[e]) * inv * load_f(&wa.v[e]);
-      y[e] = load_f(&b.v[e]) * inv * load_f(&wb.v[e]);
+      const float u = load_f(&a.v[e]) * inv * load_f(&wa.v[e]), v = load_f(&b.v[e]) * inv * load_f(&wb.v[e]);
+      x[e] = u * co[e] - v * si[e];
+      y[e] = v * co[e] + u * si[e];
     }
-    if (i < z.pairs) {
-      float u[N];
-#pragma unroll
-      for (int e = 0; e < N; ++e) {
-        u[e] = x[e] * co[e] - y[e] * si[e];
-        y[e] = y[e] * co[e] + x[e] * si[e];
-      }
-      store_n<N>(dst + c, u);
-      store_n<N>(dst + c + z.half, y);
-    } else {
-      store_n<N>(dst + c, x);
-    }
+    if (c < cols) store_n<N>(dst + c, x);
+    if (c2 < cols) store_n<N>(dst + c2, y);
   }
 };
+
+// Cos and sin of item i.
+template <typename T, int N>
+__device__ __forceinline__ void item_rotation(const NormRope<T>& p, const HeadItems<T, N>& z, const float* row, int i, float* co, float* si) {
+#pragma unroll
+  for (int e = 0; e < N; ++e) {
+    co[e] = 1.f;
+    si[e] = 0.f;
+  }
+  if (i < z.pairs) {
+    load_n<N>(row + i * N, co);
+    load_n<N>(row + i * N + (p.rd >> 1), si);
+  }
+}
 
 template <typename T>
 __device__ __forceinline__ T* head_place(const NormRope<T>& p, const TokenPlace<T>& at, int t, int h) {
@@ -136,7 +146,8 @@ __global__ void __launch_bounds__(256) norm_rope_heads_kernel(const NormRope<T> 
   const int t = live ? unit / all : 0, h = live ? unit % all : all;
   const bool value = h >= p.H + p.G;
   Item<T, N> it;
-  if (kOnce && !value) it.weights(p, z, h, lane);                      // weights do not come from the kernel before
+  it.place(p, z, lane);
+  if (kOnce && !value) it.weights(p, h);                               // weights do not come from the kernel before
   pdl_launch_dependents();
   pdl_wait();
   const T* src = p.proj + static_cast<size_t>(t) * p.ld + (value ? static_cast<size_t>(p.H + p.G) * p.d + static_cast<size_t>(h - p.H - p.G) * p.dv
@@ -144,19 +155,20 @@ __global__ void __launch_bounds__(256) norm_rope_heads_kernel(const NormRope<T> 
   float s = 0.f;
   TokenPlace<T> at = {};
   if (live) {
-    if (!value)
+    if (kOnce && !value) {
+      it.load(p, src);
+      s = it.squares();
+    }
+    if (!kOnce && !value)
       for (int i = lane; i < z.items; i += L) {
-        it.load(p, z, src, i);
+        it.place(p, z, i);
+        it.load(p, src);
         s += it.squares();
       }
-    if (kOnce && lane >= z.items) it.load(p, z, src, lane);
     at = token_place(p, t);
   }
   float co[N], si[N];
-  if (kOnce && live && !value && lane < z.pairs) {
-    load_n<N>(at.rope + lane * N, co);
-    load_n<N>(at.rope + lane * N + z.half, si);
-  }
+  if (kOnce) item_rotation(p, z, at.rope, live && !value ? lane : z.pairs, co, si);
   for (int o = L >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
   if (!live || (h >= p.H && !at.stored)) return;
   if (value) {
@@ -166,19 +178,17 @@ __global__ void __launch_bounds__(256) norm_rope_heads_kernel(const NormRope<T> 
   }
   const float inv = rsqrtf(s / static_cast<float>(p.d) + p.eps);
   T* dst = head_place(p, at, t, h);
-  const int last = h < p.H ? z.padded : z.items;
+  const int cols = h < p.H ? p.q_pitch : p.d;
   if (kOnce) {
-    if (lane < last) it.store(z, dst, lane, inv, co, si);
+    it.store(dst, cols, inv, co, si);
     return;
   }
-  for (int i = lane; i < last; i += L) {
-    it.load(p, z, src, i);
-    it.weights(p, z, h, i);
-    if (i < z.pairs) {
-      load_n<N>(at.rope + i * N, co);
-      load_n<N>(at.rope + i * N + z.half, si);
-    }
-    it.store(z, dst, i, inv, co, si);
+  for (int i = lane; i < z.padded; i += L) {
+    it.place(p, z, i);
+    it.load(p, src);
+    it.weights(p, h);
+    item_rotation(p, z, at.rope, i, co, si);
+    it.store(dst, cols, inv, co, si);
   }
 }
 
@@ -198,7 +208,8 @@ __global__ void __launch_bounds__(kOnce ? 1024 : 512) norm_rope_whole_kernel(con
   const int mine = threadIdx.x;
   if (kOnce && mine < head_items) {
     split(mine, h, i);
-    it.weights(p, z, h, i);
+    it.place(p, z, i);
+    it.weights(p, h);
   }
   pdl_launch_dependents();
   pdl_wait();
@@ -207,8 +218,11 @@ __global__ void __launch_bounds__(kOnce ? 1024 : 512) norm_rope_whole_kernel(con
   float sq = 0.f, sk = 0.f;
   for (int k = mine; k < (kOnce ? min(items, mine + 1) : head_items); k += blockDim.x) {
     if (k < head_items) {
-      if (!kOnce) split(k, h, i);
-      it.load(p, z, src + static_cast<size_t>(h) * p.d, i);
+      if (!kOnce) {
+        split(k, h, i);
+        it.place(p, z, i);
+      }
+      it.load(p, src + static_cast<size_t>(h) * p.d);
       const float s = it.squares();
       if (h < p.H) sq += s;
       else sk += s;
@@ -218,10 +232,7 @@ __global__ void __launch_bounds__(kOnce ? 1024 : 512) norm_rope_whole_kernel(con
   }
   const TokenPlace<T> at = token_place(p, t);
   float co[N], si[N];
-  if (kOnce && mine < head_items && i < z.pairs) {
-    load_n<N>(at.rope + i * N, co);
-    load_n<N>(at.rope + i * N + z.half, si);
-  }
+  if (kOnce) item_rotation(p, z, at.rope, mine < head_items ? i : z.pairs, co, si);
   const int wl = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   sq = warp_sum_f(sq);
   sk = warp_sum_f(sk);
@@ -241,14 +252,12 @@ __global__ void __launch_bounds__(kOnce ? 1024 : 512) norm_rope_whole_kernel(con
     }
     if (!kOnce) {
       split(k, h, i);
-      it.load(p, z, src + static_cast<size_t>(h) * p.d, i);
-      it.weights(p, z, h, i);
-      if (i < z.pairs) {
-        load_n<N>(at.rope + i * N, co);
-        load_n<N>(at.rope + i * N + z.half, si);
-      }
+      it.place(p, z, i);
+      it.load(p, src + static_cast<size_t>(h) * p.d);
+      it.weights(p, h);
+      item_rotation(p, z, at.rope, i, co, si);
     }
-    if (h < p.H || at.stored) it.store(z, head_place(p, at, t, h), i, h < p.H ? sq : sk, co, si);
+    if (h < p.H || at.stored) it.store(head_place(p, at, t, h), h < p.H ? p.q_pitch : p.d, h < p.H ? sq : sk, co, si);
   }
 }
 
@@ -260,7 +269,9 @@ __global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2) norm_rope_warp_ke
   const int L = 1 << p.lanes_log2, warp_lane = threadIdx.x & 31, lane = warp_lane & (L - 1), group = warp_lane >> p.lanes_log2, step = 32 >> p.lanes_log2;
   const int heads = p.H + p.G, t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   Item<T, N> it, next;
-  if (!kWhole) it.weights(p, z, 0, lane);                              // weights do not come from the kernel before
+  it.place(p, z, lane);
+  next.place(p, z, lane);
+  if (!kWhole) it.weights(p, 0);                                       // weights do not come from the kernel before
   pdl_launch_dependents();
   pdl_wait();
   if (t >= tokens) return;                                             // uniform for the warp
@@ -270,7 +281,7 @@ __global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2) norm_rope_warp_ke
   if (kWhole) {
 #pragma unroll 4
     for (int h = group; h < heads; h += step) {
-      next.load(p, z, src + static_cast<size_t>(h) * p.d, lane);
+      next.load(p, src + static_cast<size_t>(h) * p.d);
       const float s = next.squares();
       if (h < p.H) sq += s;
       else sk += s;
@@ -279,20 +290,14 @@ __global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2) norm_rope_warp_ke
     sk = rsqrtf(warp_sum_f(sk) / static_cast<float>(p.G * p.d) + p.eps);
   }
   float co[N], si[N];
-#pragma unroll
-  for (int e = 0; e < N; ++e) co[e] = si[e] = 0.f;
-  if (lane < z.pairs) {
-    load_n<N>(at.rope + lane * N, co);
-    load_n<N>(at.rope + lane * N + z.half, si);
-  }
-  next.load(p, z, src + static_cast<size_t>(min(group, heads - 1)) * p.d, lane);
+  item_rotation(p, z, at.rope, lane, co, si);
+  next.load(p, src + static_cast<size_t>(min(group, heads - 1)) * p.d);
   bool keys = false;
   for (int h0 = 0; h0 < heads; h0 += step) {                           // the same for all lanes: shuffles stay converged
     const int h = h0 + group;
     it.a = next.a;
     it.b = next.b;
-    it.c = next.c;
-    if (h0 + step < heads) next.load(p, z, src + static_cast<size_t>(min(h + step, heads - 1)) * p.d, lane);
+    if (h0 + step < heads) next.load(p, src + static_cast<size_t>(min(h + step, heads - 1)) * p.d);
     float inv = h < p.H ? sq : sk;
     if (!kWhole) {
       float s = it.squares();
@@ -301,10 +306,10 @@ __global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2) norm_rope_warp_ke
     }
     if (h >= heads || (h >= p.H && !at.stored)) continue;
     if (kWhole || (h >= p.H && !keys)) {
-      it.weights(p, z, h, lane);
+      it.weights(p, h);
       keys = h >= p.H;
     }
-    if (lane < (h < p.H ? z.padded : z.items)) it.store(z, head_place(p, at, t, h), lane, inv, co, si);
+    it.store(head_place(p, at, t, h), h < p.H ? p.q_pitch : p.d, inv, co, si);
   }
   if (!at.stored) return;
   const T* values = src + static_cast<size_t>(heads) * p.d;
@@ -313,7 +318,7 @@ __global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2) norm_rope_warp_ke
 
 template <typename T, int N>
 static int norm_rope_n(NormRope<T> p, int tokens, cudaStream_t stream) {
-  const int pairs = (p.rd >> 1) / N, items = pairs + (p.d - p.rd) / N, padded = pairs + (p.q_pitch - p.rd) / N;
+  const int pairs = (p.rd >> 1) / N, items = items_of(pairs, (p.d - p.rd) / N), padded = items_of(pairs, (p.q_pitch - p.rd) / N);
   p.lanes_log2 = 0;
   while ((1 << p.lanes_log2) < padded && p.lanes_log2 < 5) ++p.lanes_log2;
   if (tokens >= 2048 && padded <= (1 << p.lanes_log2)) {
