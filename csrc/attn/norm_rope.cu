@@ -262,7 +262,7 @@ __global__ void __launch_bounds__(kOnce ? 1024 : 512) norm_rope_whole_kernel(con
 }
 
 // Many tokens: a warp takes a token, L lanes a head at a time, one item per lane; the rotation and a head's weights stay in registers, the
-// next heads' entries are under way while these are stored.  With kWhole a first round over the heads takes the sums.
+// next heads' entries are under way while these are stored.  With kWhole a first pass over the heads takes the sums.
 template <typename T, int N, bool kWhole>
 __global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2) norm_rope_warp_kernel(const NormRope<T> p, int tokens) {
   const HeadItems<T, N> z(p);

@@ -49,7 +49,7 @@ CONFIGS = {
     # short, for generation; everything looped
     "short": _model(130, 64, 2, [
         _window(2, 1, 32, 16, 5, 0.2, 32, 4, 8.0, _dense(64)),
-        _chunk(2, 2, 16, 32, 12, 0.3, 16, _dense(48))], (0, 2, 2), buckets=1009, mul_prev=131, mul_cur=17),
+        _chunk(2, 2, 16, 32, 12, 0.3, 16, _dense(48))], (0, 2, 2), buckets=1009, mul_prev=141, mul_cur=19),
     # one stream, one kind of attention, nothing looped: no state per sequence, so cached prefixes are found again
     "chunks": _model(90, 48, 1, [
         _chunk(3, 1, 16, 16, 32, 0.3, 16, _dense(40)),
