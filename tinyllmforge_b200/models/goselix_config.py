@@ -10,27 +10,15 @@ from __future__ import annotations
 from dataclasses import dataclass
 
 from ..config import parse_dtype
-from .specs import DenseSpec, LoopSpec, MoeSpec, Rotation, layer_runs, take
+from .specs import DenseSpec, LatentAttentionSpec, LoopSpec, MoeSpec, Rotation, layer_runs, take
 
 
-@dataclass(frozen=True)
-class LatentAttentionSpec:
-    heads: int
-    dim: int
-    rot_dim: int
-    vdim: int
-    q_rank: int
-    kv_rank: int
-    scale: float
-    rot: Rotation
-
-    @classmethod
-    def from_dict(cls, d: dict) -> "LatentAttentionSpec":
-        s = cls(**take(d, "latent_attention", {"heads": int, "dim": int, "rot_dim": int, "vdim": int, "q_rank": int, "kv_rank": int,
-                                                "scale": float, "rot": Rotation.from_dict}))
-        if s.rot.dims != s.rot_dim:
-            raise ValueError("latent_attention: the whole rotated part is rotated (rot.dims == rot_dim)")
-        return s
+def _latent_attention(d: dict) -> LatentAttentionSpec:
+    s = LatentAttentionSpec(**take(d, "latent_attention", {"heads": int, "dim": int, "rot_dim": int, "vdim": int, "q_rank": int, "kv_rank": int,
+                                                           "scale": float, "rot": Rotation.from_dict}))
+    if s.q_rank < 1:
+        raise ValueError("latent_attention: sizes must be positive")
+    return s
 
 
 @dataclass(frozen=True)
@@ -66,7 +54,7 @@ def _mlp_from_dict(d):
     raise ValueError(f"unknown feed-forward kind {kind!r}; known: dense, moe")
 
 
-MIXER_SPECS = {"latent_attention": LatentAttentionSpec, "retention": RetentionSpec}
+MIXER_SPECS = {"latent_attention": _latent_attention, "retention": RetentionSpec.from_dict}
 
 
 @dataclass(frozen=True)
@@ -79,7 +67,7 @@ class LayerSpec:
     def from_dict(cls, d: dict) -> "LayerSpec":
         if d.get("type") not in MIXER_SPECS:
             raise ValueError(f"unknown layer type {d.get('type')!r}; known: {sorted(MIXER_SPECS)}")
-        return cls(d["type"], MIXER_SPECS[d["type"]].from_dict(d["mixer"]), _mlp_from_dict(d.get("mlp")))
+        return cls(d["type"], MIXER_SPECS[d["type"]](d["mixer"]), _mlp_from_dict(d.get("mlp")))
 
 
 @dataclass

@@ -13,6 +13,8 @@ from ..parallel.tp_layers import ParallelLMHead, VocabParallelEmbedding
 
 
 class LayeredDecoder:
+    tied, logit_scale, logit_softcap = False, 1.0, 0.0      # the embedding table is the head; logits <- bounded by softcap (scale * logits)
+
     def __init__(self, cfg, tp: TPGroup | None = None, dtype=None, device="cpu", ops=None, max_positions: int | None = None):
         self.cfg = cfg
         self.tp = tp or TPGroup()
@@ -32,7 +34,8 @@ class LayeredDecoder:
         self.rope = rope
         self.embed = VocabParallelEmbedding(cfg.vocab_size, cfg.hidden_size, self.tp, self.dtype, self.device)
         self.final_norm = torch.ones(cfg.hidden_size, dtype=self.dtype, device=self.device)
-        self.head = ParallelLMHead(cfg.vocab_size, cfg.hidden_size, self.tp, self.dtype, self.device)
+        self.head = ParallelLMHead(cfg.vocab_size, cfg.hidden_size, self.tp, self.dtype, self.device, tied=self.embed if self.tied else None,
+                                   scale=self.logit_scale, softcap=self.logit_softcap)
         self.layers: list = []
         self.runs: list = []                     # index into ``layers`` of every layer run
         self.memory: list = []                   # per layer run: paged cache, recurrent state, or both
@@ -53,7 +56,8 @@ class LayeredDecoder:
             for name, t in self.layer_parameters(i):
                 yield name, t, None, None
         yield "final.norm", self.final_norm, None, None
-        yield "head", self.head.weight, self.head, None
+        if not self.tied:
+            yield "head", self.head.weight, self.head, None
 
     def num_parameter_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for _, t, _, _ in self.named_parameters())
@@ -64,7 +68,8 @@ class LayeredDecoder:
 
     # ------------------------------------------------------------------ cache and state
     def kv_block_bytes(self, block_size: int) -> int:
-        return block_size * sum(self.layers[i].mix.bytes_per_token() for i in self.runs)
+        return sum(block_size * m.bytes_per_token() + (m.pool_bytes(block_size) if hasattr(m, "pool_bytes") else 0)
+                   for m in (self.layers[i].mix for i in self.runs))
 
     def state_bytes(self) -> int:
         """Recurrent state of one sequence."""
@@ -75,8 +80,13 @@ class LayeredDecoder:
         return tokens * max((l.mix.expansion_bytes() for l in self.layers), default=0)
 
     def bind_cache(self, num_blocks: int, block_size: int, num_slots: int) -> None:
-        """Every layer run has a cache or state of its own; all share block and slot numbers."""
-        self.memory = [self.layers[i].mix.new_memory(num_blocks, block_size, num_slots) for i in self.runs]
+        """Every layer run has a cache or state of its own, or borrows an earlier layer's; all share block and slot numbers."""
+        self.memory, latest = [], {}
+        for i in self.runs:
+            mix = self.layers[i].mix
+            lender = getattr(mix, "lender", None)
+            latest[i] = mix.new_memory(num_blocks, block_size, num_slots, **({} if lender is None else {"lent": latest[lender]}))
+            self.memory.append(latest[i])
 
     def drop_cache(self) -> None:
         self.memory = []
@@ -100,6 +110,6 @@ class LayeredDecoder:
         hidden = self.forward(batch, batch.last_index)
         ops, head = self.ops, self.head
         if hasattr(ops, "can_sample_in_lm_head") and ops.can_sample_in_lm_head(hidden.shape[0], head.weight):
-            ids, best = ops.lm_head_sample_shard(hidden, head.weight, batch.temperatures, batch.header, 0)
+            ids, best = ops.lm_head_sample_shard(hidden, head.weight, batch.temperatures, batch.header, 0, head.scale, head.softcap)
             return ops.merge_ranks(ids, best, self.tp)
         return ops.sample(head.forward(ops, hidden), batch, 0, self.tp)

@@ -1,7 +1,7 @@
 """Model registry: from a ``config.json`` to its configuration class and its model class.
 
 An entry names the configuration class (a dataclass with ``from_dict``) and the model class.  A checkpoint of
-Goselix, Tonapel or Mezapel names its design under ``architecture``; everything else is a Hugging Face configuration whose
+Goselix, Tonapel, Mezapel or Galupel names its design under ``architecture``; everything else is a Hugging Face configuration whose
 ``model_type`` the configuration class checks itself.
 """
 from __future__ import annotations
@@ -16,6 +16,7 @@ _ENTRIES = {
     "Goselix": ("tinyllmforge_b200.models.goselix_config:GoselixConfig", "tinyllmforge_b200.models.goselix:GoselixForCausalLM"),
     "Tonapel": ("tinyllmforge_b200.models.tonapel_config:TonapelConfig", "tinyllmforge_b200.models.tonapel:TonapelForCausalLM"),
     "Mezapel": ("tinyllmforge_b200.models.mezapel_config:MezapelConfig", "tinyllmforge_b200.models.mezapel:MezapelForCausalLM"),
+    "Galupel": ("tinyllmforge_b200.models.galupel_config:GalupelConfig", "tinyllmforge_b200.models.galupel:GalupelForCausalLM"),
 }
 
 

@@ -73,19 +73,20 @@ class BandScaling:
 
 @dataclass(frozen=True)
 class Rotation:
-    """Pairs (i, i + dims / 2) of the first ``dims`` entries of a head, angle = position * base ** (-2 i / dims), with the
-    frequencies changed by ``scaling`` if there is one."""
+    """Pairs (i, i + dims / 2) of the first ``dims`` entries of a head, or neighbours (2 i, 2 i + 1) if ``interleaved``; angle =
+    position * base ** (-2 i / dims), with the frequencies changed by ``scaling`` if there is one."""
     base: float
     dims: int
     scaling: object = None
+    interleaved: bool = False
 
     @classmethod
-    def from_dict(cls, d: dict, scaling=None) -> "Rotation":
+    def from_dict(cls, d: dict, scaling=None, interleaved: bool = False) -> "Rotation":
         """``scaling``: the class that reads ``rot.scaling`` in this design, None if it knows none."""
         keys = {"base": float, "dims": int}
         if scaling is not None and d.get("scaling") is not None:
             keys["scaling"] = scaling.from_dict
-        r = cls(**take(d, "rot", keys))
+        r = cls(**take(d, "rot", keys), interleaved=interleaved)
         if r.dims < 0 or r.dims % 2:
             raise ValueError("rot.dims must be even")
         return r
@@ -99,6 +100,9 @@ class Rotation:
     def amplitude(self) -> float:
         """Factor of cos and sin."""
         return 1.0 if self.scaling is None else self.scaling.amplitude
+
+
+NO_ROTATION = Rotation(1.0, 0)
 
 
 @dataclass(frozen=True)
@@ -131,7 +135,9 @@ class AttentionSpec:
     positions (``chunked``) or the last ``window`` tokens.  ``conv``: taps of the short convolutions ahead of the norms (0: none).
     ``norm``: over each "head" or over "all" rows of a projection at once.  ``sink``: a score that only the denominator
     sees, "learned" per head, "zero", or None.  ``softcap``: bound of the scores (0: none).  ``gate``: one sigmoid per "head" or per
-    "element" of the output, or None."""
+    "element" of the output, or None.  ``pool``: behind the window, one key and value (the means) for every whole block of that many
+    tokens of the sequence that lies before the window (0: none).  ``temper``: a learned factor of the scores per head.  ``kv_from``: the
+    layer whose keys and values are used instead of own ones."""
     heads: int
     kv_heads: int
     dim: int
@@ -145,6 +151,9 @@ class AttentionSpec:
     sink: str | None = None
     softcap: float = 0.0
     gate: str | None = None
+    pool: int = 0
+    temper: bool = False
+    kv_from: int | None = None
 
     def __post_init__(self):
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1:
@@ -155,10 +164,38 @@ class AttentionSpec:
             raise ValueError("attention: rot.dims cannot exceed dim")
         if self.window < 1:
             raise ValueError("attention: mask.size: a token sees at least itself")
+        if self.pool < 0 or (self.pool and self.chunked):
+            raise ValueError("attention: mask.pool: blocks of at least one token behind a sliding window")
+        if self.kv_from is not None and (self.conv or self.norm != "head"):
+            raise ValueError("attention: kv_from goes with norms per head and no convolutions")
 
     @property
     def gate_columns(self) -> int:
         return {None: 0, "head": self.heads, "element": self.heads * self.vdim}[self.gate]
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Attention over one latent of ``kv_rank`` entries per token, from which keys and values of every head are made, and one rotated key
+    part of ``rot_dim`` entries for all heads.  ``q_rank``: size of a latent of the queries (0: queries come from the input itself).
+    ``window``: a token sees the last ``window`` tokens (0: all)."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot: Rotation
+    q_rank: int = 0
+    window: int = 0
+
+    def __post_init__(self):
+        if min(self.heads, self.dim, self.vdim, self.kv_rank) < 1 or self.q_rank < 0:
+            raise ValueError("latent_attention: sizes must be positive")
+        if self.rot.dims != self.rot_dim:
+            raise ValueError("latent_attention: the whole rotated part is rotated (rot.dims == rot_dim)")
+        if self.window < 0:
+            raise ValueError("latent_attention: mask.size: a token sees at least itself")
 
 
 @dataclass(frozen=True)
@@ -170,7 +207,10 @@ class DenseSpec:
 @dataclass(frozen=True)
 class MoeSpec:
     """``score``: "sigmoid" (each logit on its own) or "softmax" (over the chosen logits only).  ``weigh``: whether the weight
-    multiplies an expert's "input" or its "output".  ``limit`` belongs to the activations that clamp."""
+    multiplies an expert's "input" or its "output".  ``limit`` belongs to the activations that clamp.  ``gated``: an expert is
+    down(act(gate h, up h)), else down(act(up h)).  ``correction``: a learned number per expert is added to the scores that choose, not to those
+    that weigh.  ``groups``: experts form that many groups of neighbours, and only those of the ``keep`` groups whose two best experts are
+    best together can be chosen."""
     experts: int
     top: int
     ff: int
@@ -178,7 +218,17 @@ class MoeSpec:
     limit: float = 0.0
     score: str = "sigmoid"
     weigh: str = "input"
+    gated: bool = True
+    correction: bool = False
+    groups: int = 1
+    keep: int = 1
 
     def __post_init__(self):
         if not 1 <= self.top <= self.experts:
             raise ValueError("mlp.router: top must lie between 1 and experts")
+        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            raise ValueError("mlp.router: groups.count must divide experts, groups.keep lie between 1 and groups.count")
+        if self.top > self.keep * (self.experts // self.groups):
+            raise ValueError("mlp.router: the groups kept must hold at least top experts")
+        if self.score == "softmax" and (self.correction or self.groups > 1):
+            raise ValueError("mlp.router: corrections and groups go with sigmoid scores")

@@ -101,6 +101,20 @@ def linear_act_mul(x: torch.Tensor, w_gate_up, act: str, limit: float = 0.0) -> 
     return ACTIVATIONS[act](g, u, limit).to(x.dtype)
 
 
+# the inner activation of a feed-forward without gates
+PLAIN_ACTIVATIONS = {"gelu": lambda u, limit: F.gelu(u)}
+
+
+def linear_act(x: torch.Tensor, w_up, act: str, limit: float = 0.0) -> torch.Tensor:
+    return PLAIN_ACTIVATIONS[act](linear(x, w_up).float(), limit).to(x.dtype)
+
+
+def bound_logits(x: torch.Tensor, scale: float, softcap: float) -> torch.Tensor:
+    """softcap * tanh(scale * x / softcap); without a softcap scale * x."""
+    z = x.float() * scale
+    return (softcap * torch.tanh(z / softcap) if softcap else z).to(x.dtype)
+
+
 # ----------------------------------------------------------------------------- KV cache
 def store_kv(k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
              slot_mapping: torch.Tensor) -> None:
@@ -173,15 +187,22 @@ def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_
 
 # ----------------------------------------------------------------------------- 32-bit residual stream
 def stream_update(x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None,
-                  a_bias=None, post=None, mult=1.0, offset=0.0):
+                  a_bias=None, post=None, mult=1.0, offset=0.0, groups=1):
     """The residual stream between two layers: x += a + b (the two branches of a parallel layer), += embed[ids], += vec,
-    all in fp32; then one RMS norm per weight in ``norms``, each rounded once to ``dtype``.  ``start``: x begins at zero.
-    ``rows``: norms of these rows only, and x is left as it was.  ``a_bias`` is added to a.  ``post``: a is normed with this
-    weight and multiplied by ``mult`` on its way into x.  ``offset`` is added to every norm weight (weights stored around zero)."""
+    all in fp32; then one RMS norm per weight in ``norms``, each rounded once to ``dtype`` (None: the stream itself, rounded).  ``start``: x
+    begins at zero.  ``rows``: norms of these rows only, and x is left as it was.  ``a_bias`` is added to a.  ``post``: a (without
+    a: the embedding) is normed with this weight and multiplied by ``mult`` on its way into x.  ``offset`` is added to every norm
+    weight (weights stored around zero).  ``groups``: a norm divides every one of that many equal parts of a row by its own root mean
+    square."""
     def norm(v, w):
-        return v * torch.rsqrt(v.pow(2).mean(dim=-1, keepdim=True) + eps) * (w.float() + offset)
+        if w is None:
+            return v
+        parts = v.view(v.shape[0], groups, -1)
+        return (parts * torch.rsqrt(parts.pow(2).mean(dim=-1, keepdim=True) + eps)).view(v.shape) * (w.float() + offset)
 
     s = torch.zeros_like(x) if start else x
+    if a is None and post is not None:
+        s, ids = s + mult * norm(F.embedding(ids.long(), embed).float(), post), None
     if a is not None:
         a = a.float() if a_bias is None else a.float() + a_bias
         s = s + (a if post is None else mult * norm(a, post))
@@ -231,13 +252,14 @@ def apply_partial_rope(x: torch.Tensor, positions: torch.Tensor, table: torch.Te
 # ----------------------------------------------------------------------------- latent attention
 def latent_prepare(proj, q_rank, kv_rank, q_norm, kv_norm, eps, table, positions, slot_mapping, cache):
     """proj [T, q_rank + kv_rank + rot] -> the normed query latent; the normed key/value latent and the rotated shared key
-    part go to the paged cache [blocks, block_size, kv_rank + rot]."""
+    part go to the paged cache [blocks, block_size, kv_rank + rot].  Without ``q_norm`` the first ``q_rank`` columns are passed over and
+    nothing is returned; columns after the rotated part are padding."""
     def norm(v, w):
         v = v.float()
         return v * torch.rsqrt(v.pow(2).mean(dim=-1, keepdim=True) + eps) * w.float()
-    cq = norm(proj[:, :q_rank], q_norm).to(proj.dtype)
+    cq = None if q_norm is None else norm(proj[:, :q_rank], q_norm).to(proj.dtype)
     c = norm(proj[:, q_rank:q_rank + kv_rank], kv_norm)
-    kr = apply_partial_rope(proj[:, None, q_rank + kv_rank:], positions, table)[:, 0]
+    kr = apply_partial_rope(proj[:, None, q_rank + kv_rank:q_rank + cache.shape[-1]], positions, table)[:, 0]
     slots = slot_mapping.long()
     keep = slots >= 0
     flat = cache.view(-1, cache.shape[-1])
@@ -249,7 +271,7 @@ def latent_attention(q, wkv, cache, batch, table, spec):
     """q [T, heads * (dim + rot)] before rotation; wkv [heads * (dim + vdim), kv_rank] = key rows, then value rows."""
     H, d, r, dv, R = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
     T = q.shape[0]
-    q = q.view(T, H, d + r).float()
+    q = q.reshape(T, H, d + r).float()
     q = torch.cat((q[..., :d], apply_partial_rope(q[..., d:], batch.positions, table)), dim=-1)
     out = torch.zeros(T, H, dv, dtype=cache.dtype, device=cache.device)
     w = wkv.float()
@@ -263,7 +285,8 @@ def latent_attention(q, wkv, cache, batch, table, spec):
         k = torch.cat((kv[:, :H * d].view(n, H, d), rows[:, None, R:].expand(n, H, r)), dim=-1)
         scores = torch.einsum("qhd,khd->hqk", q[a:b], k) * spec.scale
         pos = batch.positions[a:b].long()
-        scores.masked_fill_(torch.arange(n, device=q.device)[None, None, :] > pos[None, :, None], float("-inf"))
+        back = pos[:, None] - torch.arange(n, device=q.device)[None, :]
+        scores.masked_fill_((back < 0) | (back >= (spec.window or n)), float("-inf"))
         out[a:b] = torch.einsum("hqk,khe->qhe", torch.softmax(scores, dim=-1), kv[:, H * d:].view(n, H, dv)).to(out.dtype)
     return out.view(T, H * dv)
 
@@ -294,11 +317,29 @@ def retention(qkvg, decay, state, batch, table, spec, eps):
 
 
 # ----------------------------------------------------------------------------- mixture of experts
-def moe(h, router, gate_up, down, top, score="sigmoid", weigh="input", act="silu", limit=0.0):
+def choose_experts(scores, correction, groups, keep):
+    """Experts of every token, best first, by scores + correction within the ``keep`` best groups of neighbours (a group's worth: its two
+    best experts together); ties go to the lower number."""
+    c = scores if correction is None else scores + correction
+    if groups > 1:
+        parts = c.view(c.shape[0], groups, -1)
+        worth = parts.topk(min(2, parts.shape[-1]), dim=-1).values.sum(dim=-1)
+        best = torch.sort(worth, dim=-1, descending=True, stable=True).indices[:, :keep]
+        out = torch.ones_like(worth, dtype=torch.bool).scatter_(1, best, False)
+        c = parts.masked_fill(out[:, :, None], float("-inf")).view(c.shape)
+    return torch.sort(c, dim=-1, descending=True, stable=True).indices
+
+
+def moe(h, router, up, down, top, score="sigmoid", weigh="input", act="silu", limit=0.0, gated=True, correction=None, groups=1, keep=1):
     """Top-k experts.  ``score``: sigmoid of each logit, or softmax over the chosen logits; ``weigh``: the score multiplies the
-    expert's input or its output.  gate_up [experts, 2 ff, width], down [experts, width, ff]."""
-    z, e = torch.sort(h.float() @ router.float().t(), dim=-1, descending=True, stable=True)
-    w = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z[:, :top], dim=-1)
+    expert's input or its output.  up [experts, 2 ff (gate, up), width], or with ``gated=False`` [experts, ff, width]; down [experts, width,
+    ff].  ``correction``, ``groups``, ``keep``: see ``choose_experts``; weights are the scores without the correction."""
+    z = h.float() @ router.float().t()
+    if score == "sigmoid":
+        z = torch.sigmoid(z)
+    e = choose_experts(z, correction, groups, keep)
+    w = z.gather(1, e) if score == "sigmoid" else torch.softmax(z.gather(1, e)[:, :top], dim=-1)
+    inner = linear_act_mul if gated else linear_act
     out = torch.zeros(h.shape[0], down.shape[1], device=h.device)
     for j in range(top):
         for x in e[:, j].unique().tolist():
@@ -306,7 +347,7 @@ def moe(h, router, gate_up, down, top, score="sigmoid", weigh="input", act="silu
             hx, wx = h[rows], w[rows, j, None]
             if weigh == "input":
                 hx, wx = (hx.float() * wx).to(h.dtype), 1.0
-            out[rows] += wx * linear(linear_act_mul(hx, gate_up[x], act, limit), down[x]).float()
+            out[rows] += wx * linear(inner(hx, up[x], act, limit), down[x]).float()
     return out
 
 
@@ -422,6 +463,7 @@ class RefOps(ref_hybrid.RefHybridOps):
     linear = staticmethod(linear)
     linear_silu_mul = staticmethod(linear_silu_mul)
     linear_act_mul = staticmethod(linear_act_mul)
+    bound_logits = staticmethod(bound_logits)
     embedding = staticmethod(embedding)
     add_rms_norm = staticmethod(add_rms_norm)
     rms_norm = staticmethod(rms_norm)

@@ -26,9 +26,10 @@ def bias_rope_store(proj, bias, spec, table, positions, slot_mapping, k_cache, v
     return q.to(proj.dtype)
 
 
-def norm_rope_store(proj, q_norm, k_norm, eps, spec, table, positions, slot_mapping, k_cache, v_cache):
+def norm_rope_store(proj, q_norm, k_norm, eps, spec, table, positions, slot_mapping, k_cache, v_cache, temper=None):
     """proj [T, q | k | v] -> q [T, heads, dim] normed and rotated; keys (the same) and values go to the paged caches.  A norm weight of
-    ``dim`` entries belongs to every head, one of all entries to the projection as a whole."""
+    ``dim`` entries belongs to every head, one of all entries to the projection as a whole.  Without ``k_norm`` proj is q alone and
+    nothing is stored.  ``temper`` [heads]: a factor of the queries."""
     from .ref import apply_partial_rope, store_kv
     T, H, G, d = proj.shape[0], spec.heads, spec.kv_heads, spec.dim
 
@@ -36,28 +37,65 @@ def norm_rope_store(proj, q_norm, k_norm, eps, spec, table, positions, slot_mapp
         x = x.float().reshape((T, heads, d) if spec.norm == "head" else (T, heads * d))
         return apply_partial_rope((x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps) * w.float()).view(T, heads, d), positions, table)
 
-    q, k, v = proj.split([H * d, G * d, G * spec.vdim], dim=-1)
-    store_kv(normed(k, k_norm, G), v.reshape(T, G, spec.vdim), k_cache, v_cache, slot_mapping)
-    return normed(q, q_norm, H).to(proj.dtype)
+    q = proj[:, :H * d]
+    if k_norm is not None:
+        k, v = proj[:, H * d:].split([G * d, G * spec.vdim], dim=-1)
+        store_kv(normed(k, k_norm, G), v.reshape(T, G, spec.vdim), k_cache, v_cache, slot_mapping)
+    q = normed(q, q_norm, H)
+    return (q if temper is None else q * temper[:, None]).to(proj.dtype)
 
 
-def windowed_attention(q, k_cache, v_cache, batch, spec, out, scale, chunked=False, softcap=0.0, sink=None, gate=None):
+def pool_place(block, size: int, block_size: int):
+    """Where the mean of block ``block`` (an index tensor) of ``size`` tokens lies: page of the sequence, row of the page."""
+    page = (block * size + size - 1) // block_size
+    return page, block - page * block_size // size
+
+
+def pool_blocks(k_cache, v_cache, pool, batch) -> None:
+    """Means of the keys and values of the blocks that end among the step's tokens, into their places."""
+    from .ref import _gather_kv
+    cu, lens, bs = batch.cu_seqlens_q.tolist(), batch.context_lens.tolist(), k_cache.shape[2]
+    for s in range(batch.num_seqs):
+        first, end = (lens[s] - (cu[s + 1] - cu[s])) // pool.size, lens[s] // pool.size
+        if first >= end:
+            continue
+        page, row = pool_place(torch.arange(first, end, device=k_cache.device), pool.size, bs)
+        page = batch.block_tables[s].long()[page]
+        for cache, means in ((k_cache, pool.k), (v_cache, pool.v)):
+            x = _gather_kv(cache, batch.block_tables[s], end * pool.size)[:, first * pool.size:].float()
+            means[page, :, row] = x.reshape(x.shape[0], end - first, pool.size, -1).mean(dim=2).transpose(0, 1).to(means.dtype)
+
+
+def windowed_attention(q, k_cache, v_cache, batch, spec, out, scale, chunked=False, softcap=0.0, sink=None, gate=None, pool=None):
     """out [T, heads * vdim] <- scale * attention of q over the keys at most ``window - 1`` positions back, or (``chunked``) over those of
     the query's own chunk of ``window`` positions.  ``softcap`` bounds the scores; ``sink`` [heads]: one more score per head, of
-    the denominator alone; ``gate`` [T, heads] or [T, heads * vdim]: its sigmoid multiplies the result."""
+    the denominator alone; ``gate`` [T, heads] or [T, heads * vdim]: its sigmoid multiplies the result.  ``pool`` (see
+    ``PooledCache``): the blocks that end in this step get their means, and every query also sees the means of the blocks that end before
+    its window."""
     from .ref import _gather_kv
     H, G = spec.heads, spec.kv_heads
     cu, lens = batch.cu_seqlens_q.tolist(), batch.context_lens.tolist()
+    if pool is not None and pool.own:
+        pool_blocks(k_cache, v_cache, pool, batch)
     for s in range(batch.num_seqs):
         a, b, n = cu[s], cu[s + 1], lens[s]
-        k = _gather_kv(k_cache, batch.block_tables[s], n).float().repeat_interleave(H // G, dim=0)
-        v = _gather_kv(v_cache, batch.block_tables[s], n).float().repeat_interleave(H // G, dim=0)
+        k = _gather_kv(k_cache, batch.block_tables[s], n).float()
+        v = _gather_kv(v_cache, batch.block_tables[s], n).float()
+        pos, keys = batch.positions[a:b].long()[:, None], torch.arange(n, device=q.device)[None, :]
+        oldest = pos // spec.window * spec.window if chunked else pos - spec.window + 1
+        hidden = (keys > pos) | (keys < oldest)
+        if pool is not None:
+            blocks = torch.arange(n // pool.size, device=q.device)
+            page, row = pool_place(blocks, pool.size, k_cache.shape[2])
+            page = batch.block_tables[s].long()[page]
+            k, v = (torch.cat((x, means[page, :, row].float().transpose(0, 1)), dim=1) for x, means in ((k, pool.k), (v, pool.v)))
+            hidden = torch.cat((hidden, blocks[None, :] * pool.size + pool.size > oldest), dim=1)
+            n = hidden.shape[1]
+        k, v = k.repeat_interleave(H // G, dim=0), v.repeat_interleave(H // G, dim=0)
         scores = torch.einsum("qhd,hkd->hqk", q[a:b].float(), k) * spec.scale
         if softcap:
             scores = softcap * torch.tanh(scores / softcap)
-        pos, keys = batch.positions[a:b].long()[:, None], torch.arange(n, device=q.device)[None, :]
-        oldest = pos // spec.window * spec.window if chunked else pos - spec.window + 1
-        scores.masked_fill_((keys > pos) | (keys < oldest), float("-inf"))
+        scores.masked_fill_(hidden, float("-inf"))
         if sink is not None:
             scores = torch.cat((scores, sink[:, None, None].expand(H, b - a, 1)), dim=-1)
         o = torch.einsum("hqk,hke->qhe", torch.softmax(scores, dim=-1)[..., :n], v)

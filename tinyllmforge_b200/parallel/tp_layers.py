@@ -145,10 +145,19 @@ class ParallelLMHead(VocabParallelEmbedding):
     """Vocab-sharded output projection.  ``forward`` returns this rank's logits shard
     ``[rows, vocab / tp]``; ``ops.sample`` then reduces each shard to one (score, id) pair per row and
     only those pairs cross ranks.  ``full_logits`` is the materialising variant (the reference gathers
-    whole shards to rank 0: tinyvllm/layers/embed_head.py:63-70)."""
+    whole shards to rank 0: tinyvllm/layers/embed_head.py:63-70).  ``tied``: the embedding whose table this is.  ``scale`` and
+    ``softcap``: logits <- softcap * tanh(scale * logits / softcap), or scale * logits without a softcap."""
+
+    def __init__(self, vocab_size, hidden_size, tp: TPGroup, dtype, device, tied=None, scale: float = 1.0, softcap: float = 0.0):
+        if tied is None:
+            super().__init__(vocab_size, hidden_size, tp, dtype, device)
+        else:
+            self.tp, self.vocab_size, self.shard, self.vocab_start, self.weight = tp, vocab_size, tied.shard, tied.vocab_start, tied.weight
+        self.scale, self.softcap = scale, softcap
 
     def forward(self, ops, hidden):
-        return ops.linear(hidden, self.weight)
+        logits = ops.linear(hidden, self.weight)
+        return logits if self.scale == 1.0 and not self.softcap else ops.bound_logits(logits, self.scale, self.softcap)
 
     def full_logits(self, ops, hidden):
-        return self.tp.all_gather_cat(ops.linear(hidden, self.weight), dim=-1)
+        return self.tp.all_gather_cat(self.forward(ops, hidden), dim=-1)
