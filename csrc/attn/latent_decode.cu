@@ -34,7 +34,7 @@ struct LatentDecodeArgs {
   bf16* o;                   // [seqs][heads][R]
   float* part_o;             // [CTAs][2][N][R]: slot 0 = a piece that starts inside a sequence, 1 = one that only ends there
   float* part_ml;            // [CTAs][2][N][2]
-  int table_width, num_blocks, block_shift, heads, R, D, seqs, groups;
+  int table_width, num_blocks, block_shift, heads, R, D, seqs, groups, window;
   float scale_log2;
   unsigned* status;
 };
@@ -44,8 +44,12 @@ constexpr int kLdMaxSeqs = 1024;
 // Share of CTA c of G in U tiles: [ld_start(c), ld_start(c + 1)); ld_owner is its inverse.
 __device__ __forceinline__ int ld_start(int c, int G, int U) { return static_cast<int>(static_cast<long long>(U) * c / G); }
 __device__ __forceinline__ int ld_owner(int u, int G, int U) { return static_cast<int>((static_cast<long long>(u + 1) * G - 1) / U); }
+// A sequence's visible keys are [lo, len); its tiles begin with the one that holds key lo.
+__device__ __forceinline__ int ld_len(const LatentDecodeArgs& p, int seq) { return max(min(p.lens[seq], p.table_width << p.block_shift), 0); }
+__device__ __forceinline__ int ld_lo(const LatentDecodeArgs& p, int len) { return p.window > 0 ? max(len - p.window, 0) : 0; }
 __device__ __forceinline__ int ld_tiles(const LatentDecodeArgs& p, int seq) {
-  return (max(min(p.lens[seq], p.table_width << p.block_shift), 0) + kLdKeys - 1) / kLdKeys;
+  const int len = ld_len(p, seq);
+  return (len + kLdKeys - 1) / kLdKeys - ld_lo(p, len) / kLdKeys;
 }
 
 // A CTA's walk over its pieces, the same in every warp role.
@@ -196,13 +200,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         mbar_expect_tx(q_full, boxes * N * 128);
         for (int b = 0; b < boxes; ++b) tma_load_2d(sQ + b * N * 128, &tm_q, q_full, b * 64, pc.seq * p.heads + pc.group * N);
         const int* table = p.block_tables + static_cast<size_t>(pc.seq) * p.table_width;
-        const int len = min(p.lens[pc.seq], p.table_width << p.block_shift);
+        const int len = ld_len(p, pc.seq), tile0 = ld_lo(p, len) / kLdKeys + pc.tile;
         for (int t = 0; t < pc.tiles && ok; ++t) {
           int rows[4];                                  // cache row of every box_rows keys of the tile
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             rows[i] = 0;
-            const int key = (pc.tile + t) * kLdKeys + i * box_rows;
+            const int key = (tile0 + t) * kLdKeys + i * box_rows;
             if (i * box_rows < kLdKeys && key < len) {  // past the end: any rows will do, their weights are zero
               int blk = table[key >> p.block_shift];
               if (blk < 0 || blk >= p.num_blocks) {
@@ -301,7 +305,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     const int tid = key, head = tid / kHeadThreads, sub = tid % kHeadThreads;
     int t = 0, n_piece = 0;                              // tiles and pieces of this CTA so far
     for (; pc.next(before, p.seqs, p.groups); ++n_piece) {
-      const int len = min(p.lens[pc.seq], p.table_width << p.block_shift), h0 = pc.group * N;
+      const int len = ld_len(p, pc.seq), lo = ld_lo(p, len), tile0 = lo / kLdKeys + pc.tile, h0 = pc.group * N;
       float m_ref = 0.f, l_run = 0.f;
       // a wait that runs out is in the status word; the loop goes on, so that all four warps meet at the barriers
       for (int i_tile = 0; i_tile < pc.tiles; ++i_tile, ++t) {
@@ -328,7 +332,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           tcgen05_fence_before();
           __syncwarp();
           if (lane == 0) mbar_arrive(&s_empty[t & 1]);
-          const bool in = (pc.tile + i_tile) * kLdKeys + key < len;
+          const int at_key = (tile0 + i_tile) * kLdKeys + key;
+          const bool in = at_key >= lo && at_key < len;
 #pragma unroll
           for (int h = 0; h < N; ++h) sT[h * Cfg::kTPitch + key] = in ? __uint_as_float(v[h]) * p.scale_log2 : -INFINITY;
         }
@@ -513,10 +518,10 @@ static int launch_latent_decode(const CUtensorMap& tm_q, const CUtensorMap& tm_k
   return launch_kernel(kern, dim3(ctas), dim3(kLdThreads), LatentDecodeCfg<N>::kSmem, stream, 0, tm_q, tm_kv, p) == cudaSuccess ? 0 : -2;
 }
 
-// qa [seqs][heads][R + rot] bf16; lens = keys visible per sequence; scratch: forge_latent_decode_scratch floats, 16-byte aligned.
+// qa [seqs][heads][R + rot] bf16; lens = keys per sequence, of which the last `window` are visible (0: all); scratch: forge_latent_decode_scratch floats, 16-byte aligned.
 extern "C" int forge_latent_decode(const void* qa, const void* cache, const int* block_tables, const int* lens, void* o, float* scratch,
                                    int ctas, int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size,
-                                   float scale, unsigned* status, cudaStream_t stream) {
+                                   int window, float scale, unsigned* status, cudaStream_t stream) {
   if (seqs <= 0) return 0;
   const int D = R + rot, n = latent_decode_group(heads), groups = (heads + n - 1) / n;
   if (!forge_latent_decode_ok(R, rot, block_size) || seqs > kLdMaxSeqs || ctas < 1 || (reinterpret_cast<uintptr_t>(qa) & 15) ||
@@ -527,7 +532,7 @@ extern "C" int forge_latent_decode(const void* qa, const void* cache, const int*
   int shift = 0;
   while ((1 << shift) < block_size) ++shift;
   const LatentDecodeArgs p = {block_tables, lens, static_cast<bf16*>(o), scratch, scratch + 2ll * ctas * n * R, table_width, num_blocks, shift,
-                              heads, R, D, seqs, groups, scale * 1.4426950408889634f, status};
+                              heads, R, D, seqs, groups, window, scale * 1.4426950408889634f, status};
   CUtensorMap tm_q, tm_kv;
   if (forge_make_tmap_2d(&tm_q, qa, static_cast<uint64_t>(seqs) * heads, D, D, n, 2) != 0) return -2;
   if (forge_make_tmap_2d(&tm_kv, cache, static_cast<uint64_t>(num_blocks) * block_size, D, D, block_size < kLdKeys ? block_size : kLdKeys, 2) != 0) return -2;

@@ -2,7 +2,8 @@
 // the cached latents of the step's sequences are gathered into one contiguous buffer (latent_gather), one GEMM with the packed
 // key / value matrices expands them, and the kernel below attends.  Two little kernels put the operands in shape:
 //
-//   latent_gather     paged rows [c | rotated key part] -> c [keys][R] and k_rot [keys][rot], sequences one after another
+//   latent_gather     paged rows [c | rotated key part] -> c [keys][R] and k_rot [keys][rot], sequences one after another, of each the
+//                     last keys (all that its queries see)
 //   latent_pack_q     q [tokens][heads][dim + rot] -> [tokens][heads][Dq]: the rotated part rotated, both parts zero-padded to
 //                     multiples of 64 columns, so that a 64-column box of keys may run into its neighbour's columns
 //
@@ -11,7 +12,8 @@
 //                           delivers it (rows = keys, MN-major)
 //
 // CTA = 128 query rows of one (sequence, head), key tiles of 64.  Warp roles, double-buffered S and P, the reference maximum
-// that is only raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu.
+// that is only raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu.  With a window the key tiles begin with the one
+// that holds the first row's oldest visible key; a row may see nothing of them, as in windowed_prefill.cu.
 #include "../include/launch.cuh"
 #include "../include/scalar.cuh"
 
@@ -33,21 +35,21 @@ __device__ __forceinline__ uint64_t latent_desc_mn(uint32_t smem_addr, uint32_t 
 }
 
 template <bool kMasked>
-__device__ __forceinline__ float latent_row_max(const uint32_t (&v)[kVN], int kbase, int limit) {
+__device__ __forceinline__ float latent_row_max(const uint32_t (&v)[kVN], int kbase, int lo, int limit) {
   float m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
   for (int i = 0; i < kVN; i += 4)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float x = __uint_as_float(v[i + e]);
-      m[e] = fmaxf(m[e], (!kMasked || kbase + i + e < limit) ? x : -INFINITY);
+      m[e] = fmaxf(m[e], (!kMasked || (kbase + i + e >= lo && kbase + i + e < limit)) ? x : -INFINITY);
     }
   return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
 }
 
 // p = 2^(s scale - m_ref) of one row -> hi and lo bf16 halves in shared memory (K-major, 128-byte swizzle); returns the row sum.
 template <bool kMasked>
-__device__ __forceinline__ float latent_probs(const uint32_t (&v)[kVN], int kbase, int limit, float scale_log2, float m_ref, uint8_t* p_row,
+__device__ __forceinline__ float latent_probs(const uint32_t (&v)[kVN], int kbase, int first, int limit, float scale_log2, float m_ref, uint8_t* p_row,
                                               int r) {
   float ps[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -58,8 +60,8 @@ __device__ __forceinline__ float latent_probs(const uint32_t (&v)[kVN], int kbas
       float p0 = ex2_approx(fmaf(__uint_as_float(v[c + i]), scale_log2, -m_ref));
       float p1 = ex2_approx(fmaf(__uint_as_float(v[c + i + 1]), scale_log2, -m_ref));
       if (kMasked) {
-        p0 = kbase + c + i < limit ? p0 : 0.f;
-        p1 = kbase + c + i + 1 < limit ? p1 : 0.f;
+        p0 = kbase + c + i >= first && kbase + c + i < limit ? p0 : 0.f;
+        p1 = kbase + c + i + 1 >= first && kbase + c + i + 1 < limit ? p1 : 0.f;
       }
       ps[i >> 1] += p0 + p1;
       const uint32_t h = pack_bf16x2(p0, p1);
@@ -75,7 +77,7 @@ __device__ __forceinline__ float latent_probs(const uint32_t (&v)[kVN], int kbas
 
 // Boxes of 64 columns: nb1 of the unrotated part, nb2 of the rotated part, nv of the values.
 struct LatentPrefillSizes {
-  int heads, dim, rot, vdim, nb1, nb2, nv, tok0;
+  int heads, dim, rot, vdim, nb1, nb2, nv, tok0, window;
 };
 
 // tm_q: [tokens, heads * 64 (nb1 + nb2)], box 128 x 64; tm_kv: [keys, heads * (dim + vdim)], tm_r: [keys, rot], box 64 x 64.
@@ -113,7 +115,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   if (m0 >= q_len) return;                            // uniform for the CTA, before anything is allocated
   const int past = k_len - q_len;
   const int kv_end = min(k_len, past + m0 + kVM);
-  const int n_tiles = (kv_end + kVN - 1) / kVN;
+  const int tile0 = z.window > 0 ? max(past + m0 - z.window + 1, 0) / kVN : 0;
+  const int n_tiles = (kv_end + kVN - 1) / kVN - tile0;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp == 0 && lane == 0) {
@@ -148,7 +151,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       mbar_expect_tx(q_full, nq * kVQBox);
       for (int b = 0; b < nq; ++b) tma_load_2d(sQ + b * kVQBox, &tm_q, q_full, (h * nq + b) * 64, q_begin - z.tok0 + m0);
       for (int j = 0; j < n_tiles; ++j) {
-        const int s = j & 1, row = k_row0 + j * kVN;
+        const int s = j & 1, row = k_row0 + (tile0 + j) * kVN;
         const uint32_t ph = (j >> 1) & 1;
         if (!mbar_wait_parked(&k_empty[s], ph ^ 1, status)) break;
         mbar_expect_tx(&k_full[s], k_stage);
@@ -210,16 +213,16 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const int quad = warp & 3;
     const int r = quad * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
-    const int limit = min(past + m0 + r + 1, k_len);   // visible keys: [0, limit)
+    const int limit = min(past + m0 + r + 1, k_len), lo = z.window > 0 ? past + m0 + r + 1 - z.window : 0;   // visible keys: [lo, limit)
     const int o_cols = z.nv * 64;
     float m_ref = 0.f, l_run = 0.f;
-    bool ok = true;
+    bool seen = false, ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       ok = mbar_wait(&s_full[j & 1], (j >> 1) & 1, status);
       if (!ok) break;
       tcgen05_fence_after();
       const uint32_t s_addr = tmem_base + lane_addr + (j & 1) * kVN;
-      const int kbase = j * kVN;
+      const int kbase = (tile0 + j) * kVN;
       uint32_t v[kVN];
 #pragma unroll
       for (int c = 0; c < kVN; c += 32) tmem_ld_x32(s_addr + c, v + c);
@@ -227,18 +230,20 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       tcgen05_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[j & 1]);
-      const bool masked = !__all_sync(0xffffffffu, kbase + kVN <= limit);
-      float mt = masked ? latent_row_max<true>(v, kbase, limit) : latent_row_max<false>(v, kbase, limit);
+      const bool masked = !__all_sync(0xffffffffu, kbase >= lo && kbase + kVN <= limit);
+      float mt = masked ? latent_row_max<true>(v, kbase, lo, limit) : latent_row_max<false>(v, kbase, lo, limit);
       mt *= scale_log2;
-      if (j == 0) {
-        m_ref = mt == -INFINITY ? 0.f : mt;
-      } else {
-        const bool grow = mt - m_ref > 8.f;
+      if (!seen && mt != -INFINITY) {                   // nothing of this row is in O yet, or only zeros
+        m_ref = mt;
+        seen = true;
+      }
+      if (j > 0) {
+        const bool grow = seen && mt - m_ref > 8.f;
         if (__any_sync(0xffffffffu, grow)) {
           ok = mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1, status);
           if (!ok) break;
           tcgen05_fence_after();
-          const float m_new = fmaxf(m_ref, mt);
+          const float m_new = seen ? fmaxf(m_ref, mt) : m_ref;
           const float alpha = exp2f(m_ref - m_new);
 #pragma unroll 1
           for (int c = 0; c < o_cols; c += 32) {
@@ -260,8 +265,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         if (!ok) break;
       }
       uint8_t* p_row = sP + (j & 1) * 2 * kVQBox + r * 128;
-      l_run += masked ? latent_probs<true>(v, kbase, limit, scale_log2, m_ref, p_row, r)
-                      : latent_probs<false>(v, kbase, limit, scale_log2, m_ref, p_row, r);
+      l_run += masked ? latent_probs<true>(v, kbase, lo, limit, scale_log2, m_ref, p_row, r)
+                      : latent_probs<false>(v, kbase, lo, limit, scale_log2, m_ref, p_row, r);
       fence_proxy_async_smem();
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_full[j & 1]);
@@ -301,8 +306,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   }
 }
 
-static LatentPrefillSizes latent_prefill_sizes(int heads, int dim, int rot, int vdim, int tok0) {
-  return LatentPrefillSizes{heads, dim, rot, vdim, (dim + 63) / 64, (rot + 63) / 64, (vdim + 63) / 64, tok0};
+static LatentPrefillSizes latent_prefill_sizes(int heads, int dim, int rot, int vdim, int tok0, int window) {
+  return LatentPrefillSizes{heads, dim, rot, vdim, (dim + 63) / 64, (rot + 63) / 64, (vdim + 63) / 64, tok0, window};
 }
 static int latent_prefill_smem(const LatentPrefillSizes& z) {
   return (z.nb1 + z.nb2) * (kVQBox + kVStages * kVKBox) + kVStages * z.nv * kVKBox + 4 * kVQBox + 256 + 1024;
@@ -311,7 +316,7 @@ static int latent_prefill_smem(const LatentPrefillSizes& z) {
 // Columns of one head's packed query row, or 0 when the kernel does not take these sizes (else: latent_attend_any).
 extern "C" int forge_latent_prefill_qcols(int dim, int rot, int vdim) {
   if ((dim & 7) || (rot & 7) || (vdim & 7) || dim < 8 || rot < 8 || vdim < 8 || vdim > 128) return 0;
-  const LatentPrefillSizes z = latent_prefill_sizes(1, dim, rot, vdim, 0);
+  const LatentPrefillSizes z = latent_prefill_sizes(1, dim, rot, vdim, 0, 0);
   return latent_prefill_smem(z) <= 227 * 1024 ? 64 * (z.nb1 + z.nb2) : 0;
 }
 
@@ -319,14 +324,15 @@ extern "C" int forge_make_tmap_2d(CUtensorMap* tm, const void* base, uint64_t ro
                                   uint32_t box_rows, int elem_bytes);
 
 // q [tokens - tok0][heads][qcols] (packed); kv [keys][heads * (dim + vdim)]; kr [keys][rot]; sequence s has the step's tokens
-// cu_q[s] .. cu_q[s + 1] (its last ones) and the keys cu_k[s] .. cu_k[s + 1]; out [tokens][heads * vdim].
+// cu_q[s] .. cu_q[s + 1] (its last ones) and the keys cu_k[s] .. cu_k[s + 1] (at least all that they see); out [tokens][heads * vdim].
+// Key rows past the last sequence's must hold numbers.
 extern "C" int forge_latent_prefill(const void* q, const void* kv, const void* kr, const int* cu_q, const int* cu_k, void* out, int tokens,
-                                    int tok0, int keys, int num_seqs, int max_q, int heads, int dim, int rot, int vdim, float scale,
+                                    int tok0, int keys, int num_seqs, int max_q, int heads, int dim, int rot, int vdim, int window, float scale,
                                     unsigned* status, cudaStream_t stream) {
   if (tokens <= tok0 || num_seqs <= 0) return 0;
   const int qcols = forge_latent_prefill_qcols(dim, rot, vdim);
   if (qcols == 0 || num_seqs > 65535 || heads > 65535) return -1;
-  const LatentPrefillSizes z = latent_prefill_sizes(heads, dim, rot, vdim, tok0);
+  const LatentPrefillSizes z = latent_prefill_sizes(heads, dim, rot, vdim, tok0, window);
   CUtensorMap tm_q, tm_kv, tm_r;
   const uint64_t qw = static_cast<uint64_t>(heads) * qcols, kw = static_cast<uint64_t>(heads) * (dim + vdim);
   if (forge_make_tmap_2d(&tm_q, q, tokens - tok0, qw, qw, kVM, 2) != 0) return -2;
@@ -338,8 +344,8 @@ extern "C" int forge_latent_prefill(const void* q, const void* kv, const void* k
                        static_cast<bf16*>(out), z, scale * 1.4426950408889634f, status) == cudaSuccess ? 0 : -5;
 }
 
-// One warp per key row, 16-byte units.
-__global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restrict__ cache, const int* __restrict__ cu_k, int num_seqs,
+// One warp per key row, 16-byte units.  Of a sequence of lens[s] keys the last cu_k[s + 1] - cu_k[s]; rows past the last sequence's are zero.
+__global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restrict__ cache, const int* __restrict__ cu_k, const int* __restrict__ lens, int num_seqs,
                                                             const int* __restrict__ block_tables, int table_width, int num_blocks,
                                                             int block_size, int R, int rot, int keys, bf16* __restrict__ c,
                                                             bf16* __restrict__ kr, unsigned* status) {
@@ -352,16 +358,20 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restri
     const int mid = (lo + hi) >> 1;
     if (cu_k[mid] <= row) lo = mid; else hi = mid;
   }
-  const int key = row - cu_k[lo];
+  uint4* dc = reinterpret_cast<uint4*>(c + static_cast<size_t>(row) * R);
+  uint4* dr = reinterpret_cast<uint4*>(kr + static_cast<size_t>(row) * rot);
+  const int uc = R >> 3, ur = rot >> 3;
+  if (row >= cu_k[num_seqs]) {
+    for (int u = lane; u < uc + ur; u += 32) (u < uc ? dc[u] : dr[u - uc]) = make_uint4(0, 0, 0, 0);
+    return;
+  }
+  const int key = max(lens[lo] - (cu_k[lo + 1] - cu_k[lo]), 0) + row - cu_k[lo];
   int blk = block_tables[static_cast<size_t>(lo) * table_width + min(key / block_size, table_width - 1)];
   if (blk < 0 || blk >= num_blocks) {
     if (lane == 0) set_status(status, kStatusBadIndex);
     blk = 0;
   }
   const uint4* src = reinterpret_cast<const uint4*>(cache + (static_cast<size_t>(blk) * block_size + key % block_size) * (R + rot));
-  uint4* dc = reinterpret_cast<uint4*>(c + static_cast<size_t>(row) * R);
-  uint4* dr = reinterpret_cast<uint4*>(kr + static_cast<size_t>(row) * rot);
-  const int uc = R >> 3, ur = rot >> 3;
   for (int u = lane; u < uc + ur; u += 32) {
     const uint4 v = src[u];
     if (u < uc) dc[u] = v;
@@ -369,17 +379,17 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restri
   }
 }
 
-extern "C" int forge_latent_gather(const void* cache, const int* cu_k, int num_seqs, const int* block_tables, int table_width, int num_blocks,
+extern "C" int forge_latent_gather(const void* cache, const int* cu_k, const int* lens, int num_seqs, const int* block_tables, int table_width, int num_blocks,
                                    int block_size, int R, int rot, int keys, void* c, void* kr, unsigned* status, cudaStream_t stream) {
   if (keys <= 0 || num_seqs <= 0) return 0;
   if ((R & 7) || (rot & 7)) return -1;
-  return launch_kernel(latent_gather_kernel, dim3((keys + 7) / 8), dim3(256), 0, stream, 0, static_cast<const bf16*>(cache), cu_k, num_seqs,
+  return launch_kernel(latent_gather_kernel, dim3((keys + 7) / 8), dim3(256), 0, stream, 0, static_cast<const bf16*>(cache), cu_k, lens, num_seqs,
                        block_tables, table_width, num_blocks, block_size, R, rot, keys, static_cast<bf16*>(c), static_cast<bf16*>(kr),
                        status) == cudaSuccess ? 0 : -2;
 }
 
-// q [tokens][heads][dim + rot] -> [tokens][heads][64 (nb1 + nb2)].  A thread moves 8 columns of the unrotated part or 4 pairs.
-__global__ void __launch_bounds__(128) latent_pack_q_kernel(const bf16* __restrict__ q, bf16* __restrict__ qp, int heads, int dim, int rot,
+// q [tokens][heads][dim + rot], tokens ld elements apart -> [tokens][heads][64 (nb1 + nb2)].  A thread moves 8 columns of the unrotated part or 4 pairs.
+__global__ void __launch_bounds__(128) latent_pack_q_kernel(const bf16* __restrict__ q, long long ld, bf16* __restrict__ qp, int heads, int dim, int rot,
                                                             int nb1, int nb2, const float* __restrict__ rope, int rope_rows,
                                                             const int* __restrict__ positions) {
   pdl_launch_dependents();
@@ -389,7 +399,7 @@ __global__ void __launch_bounds__(128) latent_pack_q_kernel(const bf16* __restri
   pos = pos < 0 ? 0 : (pos >= rope_rows ? rope_rows - 1 : pos);
   const float* cs = rope + static_cast<size_t>(pos) * rot;
   const int half = rot >> 1, u1 = nb1 * 8, pairs = half >> 2, pad = nb2 * 8 - (rot >> 3), per = u1 + pairs + pad;
-  const bf16* src0 = q + static_cast<size_t>(t) * heads * (dim + rot);
+  const bf16* src0 = q + static_cast<size_t>(t) * ld;
   bf16* dst0 = qp + static_cast<size_t>(t) * heads * (nb1 + nb2) * 64;
   for (int i = threadIdx.x; i < heads * per; i += blockDim.x) {
     const int h = i / per, u = i % per;
@@ -416,11 +426,11 @@ __global__ void __launch_bounds__(128) latent_pack_q_kernel(const bf16* __restri
   }
 }
 
-extern "C" int forge_latent_pack_q(const void* q, void* qp, int tokens, int heads, int dim, int rot, const float* rope, int rope_rows,
+extern "C" int forge_latent_pack_q(const void* q, long long ld, void* qp, int tokens, int heads, int dim, int rot, const float* rope, int rope_rows,
                                    const int* positions, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if ((dim & 7) || (rot & 7)) return -1;
-  return launch_kernel(latent_pack_q_kernel, dim3(tokens), dim3(128), 0, stream, 0, static_cast<const bf16*>(q), static_cast<bf16*>(qp), heads,
+  if ((dim & 7) || (rot & 7) || (ld & 7) || (reinterpret_cast<uintptr_t>(q) & 15)) return -1;
+  return launch_kernel(latent_pack_q_kernel, dim3(tokens), dim3(128), 0, stream, 0, static_cast<const bf16*>(q), ld, static_cast<bf16*>(qp), heads,
                        dim, rot, (dim + 63) / 64, (rot + 63) / 64, rope, rope_rows, positions) == cudaSuccess ? 0 : -2;
 }
 

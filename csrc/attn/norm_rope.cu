@@ -1,7 +1,7 @@
 // What stands before the attention of a decoder that norms its queries and keys: q | k | v of a token -> q and k normed (RMS over each
 // head with a weight of d entries, or over all rows of the projection at once with a weight per row) and rotated (first rd entries of
 // a head, entry i with i + rd / 2); q to [token][head][q_pitch] (padding columns zero), k and v to the caches
-// [block][kv_head][block_size][d / dv].
+// [block][kv_head][block_size][d / dv].  Without key/value heads (G = 0) there is q alone.  temper: one more factor per query head.
 //
 // The work of a token is a list of items: N rotated pairs or 2 N entries that pass of a head, or N values.
 #include "../include/launch.cuh"
@@ -25,8 +25,12 @@ struct NormRope {
   long long num_slots;
   int H, G, d, dv, q_pitch, block_size, whole, lanes_log2;
   float eps;
+  const float* temper;      // [H]; null: none
   unsigned* status;
 };
+
+template <typename T>
+__device__ __forceinline__ float head_factor(const NormRope<T>& p, int h) { return p.temper != nullptr && h < p.H ? p.temper[h] : 1.f; }
 
 template <typename T, int N>
 struct alignas(sizeof(T) * N) Piece {       // N consecutive elements as they lie in memory
@@ -55,7 +59,7 @@ __device__ __forceinline__ TokenPlace<T> token_place(const NormRope<T>& p, int t
   pos = pos < 0 ? 0 : (pos >= p.rope_rows ? p.rope_rows - 1 : pos);
   TokenPlace<T> r;
   r.stored = slot >= 0 && slot < p.num_slots;
-  if (slot >= p.num_slots) set_status(p.status, kStatusBadIndex);
+  if (slot >= p.num_slots && p.G > 0) set_status(p.status, kStatusBadIndex);
   const unsigned s = r.stored ? static_cast<unsigned>(slot) : 0u;      // num_slots fits 31 bits
   r.blk = s / static_cast<unsigned>(p.block_size);
   r.off = s % static_cast<unsigned>(p.block_size);
@@ -176,7 +180,7 @@ __global__ void __launch_bounds__(256) norm_rope_heads_kernel(const NormRope<T> 
       *reinterpret_cast<Piece<T, N>*>(value_place(p, at, (h - p.H - p.G) * p.dv + i)) = load_piece<T, N>(src + i);
     return;
   }
-  const float inv = rsqrtf(s / static_cast<float>(p.d) + p.eps);
+  const float inv = rsqrtf(s / static_cast<float>(p.d) + p.eps) * head_factor(p, h);
   T* dst = head_place(p, at, t, h);
   const int cols = h < p.H ? p.q_pitch : p.d;
   if (kOnce) {
@@ -257,7 +261,7 @@ __global__ void __launch_bounds__(kOnce ? 1024 : 512) norm_rope_whole_kernel(con
       it.weights(p, h);
       item_rotation(p, z, at.rope, i, co, si);
     }
-    if (h < p.H || at.stored) it.store(head_place(p, at, t, h), h < p.H ? p.q_pitch : p.d, h < p.H ? sq : sk, co, si);
+    if (h < p.H || at.stored) it.store(head_place(p, at, t, h), h < p.H ? p.q_pitch : p.d, (h < p.H ? sq : sk) * head_factor(p, h), co, si);
   }
 }
 
@@ -309,7 +313,7 @@ __global__ void __launch_bounds__(256, sizeof(T) == 2 ? 3 : 2) norm_rope_warp_ke
       it.weights(p, h);
       keys = h >= p.H;
     }
-    it.store(head_place(p, at, t, h), h < p.H ? p.q_pitch : p.d, inv, co, si);
+    it.store(head_place(p, at, t, h), h < p.H ? p.q_pitch : p.d, inv * head_factor(p, h), co, si);
   }
   if (!at.stored) return;
   const T* values = src + static_cast<size_t>(heads) * p.d;
@@ -353,12 +357,12 @@ static int norm_rope(const NormRope<T>& p, int tokens, cudaStream_t stream) {
 extern "C" int forge_norm_rope_store(int fp32, const void* proj, long long ld, int tokens, const void* q_norm, const void* k_norm, int whole,
                                      float eps, const float* rope, int rope_rows, int rd, const int* positions, const int* slots, void* q,
                                      int q_pitch, void* k_cache, void* v_cache, long long num_slots, int block_size, int H, int G, int d, int dv,
-                                     unsigned* status, cudaStream_t stream) {
+                                     const float* temper, unsigned* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (rd < 0 || (rd & 1) || rd > d || q_pitch < d || (rd > 0 && rope_rows < 1) || num_slots >= (1ll << 31)) return -1;
+  if (rd < 0 || (rd & 1) || rd > d || q_pitch < d || (rd > 0 && rope_rows < 1) || num_slots >= (1ll << 31) || block_size < 1 || (whole && G < 1)) return -1;
 #define FORGE_NORM_ROPE(T)                                                                                                             \
   return norm_rope<T>({static_cast<const T*>(proj), ld, static_cast<const T*>(q_norm), static_cast<const T*>(k_norm), rope, rope_rows, rd, positions, slots, static_cast<T*>(q),     \
-                       static_cast<T*>(k_cache), static_cast<T*>(v_cache), num_slots, H, G, d, dv, q_pitch, block_size, whole, 0, eps, status}, tokens, stream)
+                       static_cast<T*>(k_cache), static_cast<T*>(v_cache), num_slots, H, G, d, dv, q_pitch, block_size, whole, 0, eps, temper, status}, tokens, stream)
   if (fp32) FORGE_NORM_ROPE(float);
   FORGE_NORM_ROPE(bf16);
 #undef FORGE_NORM_ROPE

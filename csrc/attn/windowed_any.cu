@@ -4,11 +4,12 @@
 //                       [token][head][q_pitch] (padding columns zero), k and v to the caches [block][kv_head][block_size][dim / vdim]
 //   windowed_attend_any softmax attention of a token over itself and the window - 1 tokens before it (or the tokens of its chunk of
 //                       the sequence), with the options of attend_options.cuh, bf16 or fp32, any sizes: one warp per query token,
-//                       eight tokens of one head per CTA share key and value tiles of 32
+//                       eight tokens of one head per CTA share key and value tiles of 32; pooled blocks (pooled.cuh) come ahead of the window
 //
 // Scores, weights and sums are fp32.
 #include "../include/attend_options.cuh"
 #include "../include/launch.cuh"
+#include "../include/pooled.cuh"
 #include "../include/scalar.cuh"
 
 namespace forge {
@@ -145,6 +146,7 @@ struct AttendAny {
   int width, num_blocks, block_size, H, G, d, dv, q_pitch, window;
   float scale, out_scale;
   AttendOptions<T> opt;
+  PoolCache<T> pool;
   unsigned* status;
 };
 
@@ -175,18 +177,26 @@ __global__ void __launch_bounds__(256) windowed_attend_any_kernel(const AttendAn
   if (last >= cap) {
     if (threadIdx.x == 0) set_status(p.status, kStatusBadIndex);
   }
-  for (int j0 = lo / kWKeys * kWKeys; j0 <= last && j0 < cap; j0 += kWKeys) {
+  // entries of the pooled blocks that the last token sees, then the tokens of the windows
+  const int size = p.pool.size, blocks = size > 0 ? pool_visible(oldest_visible(min(last, cap - 1), p.window, 0), size) : 0;
+  const int pooled = (blocks + kWKeys - 1) / kWKeys * kWKeys, j_first = lo / kWKeys * kWKeys - pooled;
+  for (int i0 = 0; i0 < pooled || (j_first + i0 <= last && j_first + i0 < cap); i0 += kWKeys) {
+    const bool means = i0 < pooled;                // uniform for the CTA
+    const int j0 = means ? i0 : j_first + i0, end = means ? blocks : min(last + 1, cap), per = means ? p.pool.rows : p.block_size;
+    const T* k_src = means ? p.pool.k : p.k_cache;
+    const T* v_src = means ? p.pool.v : p.v_cache;
     __syncthreads();
     for (int r = warp; r < kWKeys; r += 8) {       // one key per warp at a time
-      const int j = j0 + r;
-      int blk = j <= last && j < cap ? p.tables[static_cast<size_t>(s) * p.width + j / p.block_size] : -1;
-      if (j <= last && (blk < 0 || blk >= p.num_blocks)) {
+      const int j = j0 + r, page = means ? pool_page(j, size, p.block_size) : j / p.block_size;
+      int blk = j < end ? p.tables[static_cast<size_t>(s) * p.width + page] : -1;
+      if (j < end && (blk < 0 || blk >= p.num_blocks)) {
         if (lane == 0) set_status(p.status, kStatusBadIndex);
         blk = -1;
       }
-      const size_t row = (static_cast<size_t>(max(blk, 0)) * p.G + g) * p.block_size + j % p.block_size;
-      for (int c = lane; c < p.d; c += 32) sk[r * kp + c] = blk < 0 ? 0.f : load_f(p.k_cache + row * p.d + c);
-      for (int c = lane; c < p.dv; c += 32) sv[r * p.dv + c] = blk < 0 ? 0.f : load_f(p.v_cache + row * p.dv + c);
+      const int at = blk < 0 ? 0 : means ? pool_row(j, page, size, p.block_size) : j % p.block_size;
+      const size_t row = (static_cast<size_t>(max(blk, 0)) * p.G + g) * per + at;
+      for (int c = lane; c < p.d; c += 32) sk[r * kp + c] = blk < 0 ? 0.f : load_f(k_src + row * p.d + c);
+      for (int c = lane; c < p.dv; c += 32) sv[r * p.dv + c] = blk < 0 ? 0.f : load_f(v_src + row * p.dv + c);
     }
     __syncthreads();
     if (!live) continue;
@@ -195,7 +205,7 @@ __global__ void __launch_bounds__(256) windowed_attend_any_kernel(const AttendAn
     for (int c = 0; c < p.d; ++c) x = fmaf(sq[warp * p.d + c], sk[lane * kp + c], x);
     x *= p.scale;
     if (p.opt.softcap > 0.f) x = p.opt.softcap * tanhf(x / p.opt.softcap);
-    if (j > pos || j < mine) x = -INFINITY;
+    if (means ? j >= pool_visible(mine, size) : j > pos || j < mine) x = -INFINITY;
     float mt = x;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, o));
@@ -239,18 +249,21 @@ extern "C" int forge_windowed_attend_any(int fp32, const void* q, int q_pitch, c
                                          int max_q, const int* positions, const int* tables, int width, int num_blocks, int block_size,
                                          void* out, long long ldo, int H, int G, int d, int dv, int window, float scale, float out_scale,
                                          int chunked, float softcap, const float* sink, const void* gate, long long ldg, int gate_head,
-                                         int gate_col, unsigned* status, cudaStream_t stream) {
+                                         int gate_col, const void* pool_k, const void* pool_v, int pool, unsigned* status, cudaStream_t stream) {
   if (seqs <= 0 || max_q <= 0) return 0;
-  if (window < 1) return -1;
+  if (window < 1 || pool < 0 || (pool > 0 && chunked)) return -1;
+  const int rows = pool > 0 ? (block_size + pool - 1) / pool : 0;
   if (seqs > 65535 || H > 65535) return -1;
   if (fp32)
     return windowed_attend_any<float>({static_cast<const float*>(q), static_cast<const float*>(k_cache), static_cast<const float*>(v_cache), cu, positions,
                                        tables, static_cast<float*>(out), ldo, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, scale, out_scale,
-                                       {chunked, softcap, sink, static_cast<const float*>(gate), ldg, gate_head, gate_col}, status},
+                                       {chunked, softcap, sink, static_cast<const float*>(gate), ldg, gate_head, gate_col},
+                                       {const_cast<float*>(static_cast<const float*>(pool_k)), const_cast<float*>(static_cast<const float*>(pool_v)), pool, rows}, status},
                                       seqs, max_q, stream);
   return windowed_attend_any<bf16>({static_cast<const bf16*>(q), static_cast<const bf16*>(k_cache), static_cast<const bf16*>(v_cache), cu, positions,
                                     tables, static_cast<bf16*>(out), ldo, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, scale, out_scale,
-                                    {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}, status},
+                                    {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col},
+                                    {const_cast<bf16*>(static_cast<const bf16*>(pool_k)), const_cast<bf16*>(static_cast<const bf16*>(pool_v)), pool, rows}, status},
                                    seqs, max_q, stream);
 }
 

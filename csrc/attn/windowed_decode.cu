@@ -6,9 +6,13 @@
 // weights are fp32 and enter the second product as bf16 hi + lo halves.  The warps' states are merged through shared memory;
 // with more than one chunk, partial outputs go to scratch and a second kernel merges them.  Lengths are read on the device and
 // the grid depends on the batch bucket only, so the launch is CUDA-graph safe.  Options: attend_options.cuh.
+//
+// Pooled blocks behind the window (pooled.cuh) come ahead of it as tiles of 16 entries.  A block that ends with the step's token gets its
+// entry here too: no token sees it before a later step.
 #include "../include/attend_options.cuh"
 #include "../include/launch.cuh"
 #include "../include/mma_sync.cuh"
+#include "../include/pooled.cuh"
 #include "../include/scalar.cuh"
 
 namespace forge {
@@ -28,6 +32,8 @@ struct WindowedDecode {
   int width, num_blocks, block_size, H, G, d, dv, q_pitch, window, chunk, max_chunks, stages, slices;
   float scale_log2, out_scale, cap_pre, cap_post;
   AttendOptions<bf16> opt;
+  PoolCache<bf16> pool;
+  int pool_own;             // entries of blocks that end here are made
   unsigned* status;
 };
 
@@ -39,6 +45,8 @@ __host__ __device__ __forceinline__ int wd_pitch(int cols) {
 
 struct WindowRange {
   int begin, lo, end;       // first key of the first 16-key tile, first visible key, end of the visible keys
+  int blocks, pooled;       // visible pooled blocks; the same in whole tiles
+  __device__ int all() const { return pooled + end - begin; }          // places: tiles of pooled blocks, then tiles of keys
 };
 __device__ __forceinline__ WindowRange window_range(const WindowedDecode& p, int s, unsigned* status) {
   int len = p.lens[s];
@@ -51,6 +59,8 @@ __device__ __forceinline__ WindowRange window_range(const WindowedDecode& p, int
   r.end = max(len, 0);
   r.lo = r.end > 0 ? oldest_visible(r.end - 1, p.window, p.opt.chunked) : 0;
   r.begin = r.lo & ~(kWDKeys - 1);
+  r.blocks = p.pool.size > 0 ? pool_visible(r.lo, p.pool.size) : 0;
+  r.pooled = (r.blocks + kWDKeys - 1) & ~(kWDKeys - 1);
   return r;
 }
 
@@ -62,6 +72,16 @@ __device__ __forceinline__ void wd_load_rows(uint32_t dst, int pitch, const bf16
   src += r0 * cols + u * 8;
 #pragma unroll 8
   for (int r = r0; r < kWDKeys; r += step, dst += step * pitch * 2, src += step * cols) cp_async16(dst, src, 16);
+}
+// The same with rows anywhere: lane r < 16 knows row r's place.
+__device__ __forceinline__ void wd_load_places(uint32_t dst, int pitch, const bf16* src, int cols, int lanes_log2, int lane, int place) {
+  const int u = lane & ((1 << lanes_log2) - 1), r0 = lane >> lanes_log2, step = 32 >> lanes_log2;
+  const bool in = u * 8 < cols;
+#pragma unroll 8
+  for (int r = 0; r < kWDKeys; r += step) {                    // the same for all lanes
+    const int at = __shfl_sync(0xffffffffu, place, (r + r0) & (kWDKeys - 1));
+    if (in && r + r0 < kWDKeys) cp_async16(dst + ((r + r0) * pitch + u * 8) * 2, src + static_cast<size_t>(at) * cols + u * 8, 16);
+  }
 }
 __device__ __forceinline__ int wd_lanes_log2(int units) { return units <= 1 ? 0 : 32 - __clz(units - 1); }
 
@@ -89,8 +109,8 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
   const int s = blockIdx.y, g = blockIdx.x / p.slices, slice = blockIdx.x % p.slices, chunk = blockIdx.z;
   const int per = p.H / p.G, h0 = g * per + slice * 16, nh = min(16, per - slice * 16);
   const WindowRange w = window_range(p, s, chunk == 0 ? p.status : nullptr);
-  const int c_begin = w.begin + chunk * p.chunk, c_end = min(c_begin + p.chunk, w.end);
-  const int n_chunks = (w.end - w.begin + p.chunk - 1) / p.chunk;
+  const int c_begin = chunk * p.chunk, c_end = min(c_begin + p.chunk, w.all());       // places of this CTA
+  const int n_chunks = (w.all() + p.chunk - 1) / p.chunk;
   if (c_begin >= c_end) {                                      // uniform for the CTA
     if (chunk == 0)                                            // padding row: defined output
       for (int i = threadIdx.x; i < nh * p.dv; i += blockDim.x)
@@ -113,14 +133,28 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
   const int mine = tiles > warp ? (tiles - warp + kWDWarps - 1) / kWDWarps : 0;
   auto load = [&](int i) {                                     // this warp's tile i
     if (i < mine) {
-      const int key = c_begin + (i * kWDWarps + warp) * kWDKeys;
+      const int at = c_begin + (i * kWDWarps + warp) * kWDKeys;
+      bf16* sk = ring + static_cast<size_t>(i % p.stages) * stage;
+      if (at < w.pooled) {                                     // uniform for the warp
+        const int b = min(at + (lane & (kWDKeys - 1)), w.blocks - 1), page = pool_page(b, p.pool.size, p.block_size);
+        int blk = p.tables[static_cast<size_t>(s) * p.width + page];
+        if (blk < 0 || blk >= p.num_blocks) {
+          set_status(p.status, kStatusBadIndex);
+          blk = 0;
+        }
+        const int place = (blk * p.G + g) * p.pool.rows + pool_row(b, page, p.pool.size, p.block_size);
+        wd_load_places(smem_u32(sk), kp, p.pool.k, p.d, kl, lane, place);
+        wd_load_places(smem_u32(sk + kWDKeys * kp), vp, p.pool.v, p.dv, vl, lane, place);
+        cp_async_commit();
+        return;
+      }
+      const int key = w.begin + at - w.pooled;
       int blk = p.tables[static_cast<size_t>(s) * p.width + key / p.block_size];
       if (blk < 0 || blk >= p.num_blocks) {
         if (lane == 0) set_status(p.status, kStatusBadIndex);
         blk = 0;
       }
       const size_t row = (static_cast<size_t>(blk) * p.G + g) * p.block_size + key % p.block_size;   // 16 keys never straddle a block
-      bf16* sk = ring + static_cast<size_t>(i % p.stages) * stage;
       wd_load_rows(smem_u32(sk), kp, p.k_cache + row * p.d, p.d, kl, lane);
       wd_load_rows(smem_u32(sk + kWDKeys * kp), vp, p.v_cache + row * p.dv, p.dv, vl, lane);
     }
@@ -148,7 +182,9 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
       mma16816(x[0], a, b[0], b[1]);
       mma16816(x[1], a, b[2], b[3]);
     }
-    const int key = c_begin + (i * kWDWarps + warp) * kWDKeys;
+    const int at = c_begin + (i * kWDWarps + warp) * kWDKeys;
+    const bool means = at < w.pooled;
+    const int key = means ? at : w.begin + at - w.pooled, lo = means ? 0 : w.lo, end = means ? w.blocks : w.end;     // visible: [lo, end)
     float mt[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int n = 0; n < 2; ++n)
@@ -156,7 +192,7 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
       for (int e = 0; e < 4; ++e) {
         const int j = key + n * 8 + q2 + (e & 1);
         const float y = kCap ? softcap_log2(x[n][e], p.cap_pre, p.cap_post) : x[n][e] * p.scale_log2;
-        x[n][e] = j >= w.lo && j < c_end ? y : -INFINITY;
+        x[n][e] = j >= lo && j < end ? y : -INFINITY;
         mt[e >> 1] = fmaxf(mt[e >> 1], x[n][e]);
       }
     float alpha[2];
@@ -179,7 +215,7 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
       l[0] *= alpha[0];
       l[1] *= alpha[1];
     }
-    uint32_t hi[4], lo[4];
+    uint32_t hi[4], low[4];
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -189,7 +225,7 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
         l[r] += a + b;
         const uint32_t h = pack_bf16x2(a, b);
         hi[n * 2 + r] = h;
-        lo[n * 2 + r] = pack_bf16x2(a - bf16_lo(h), b - bf16_hi(h));
+        low[n * 2 + r] = pack_bf16x2(a - bf16_lo(h), b - bf16_hi(h));
       }
     const bf16* vr = sv + ((lane & 7) + ((lane >> 3) & 1) * 8) * vp + (lane >> 4) * 8;
 #pragma unroll
@@ -198,9 +234,9 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
         uint32_t b[4];
         ldsm_x4_trans(smem_u32(vr + nb * 8), b);
         mma16816(o[nb], hi, b[0], b[1]);
-        mma16816(o[nb], lo, b[0], b[1]);
+        mma16816(o[nb], low, b[0], b[1]);
         mma16816(o[nb + 1], hi, b[2], b[3]);
-        mma16816(o[nb + 1], lo, b[2], b[3]);
+        mma16816(o[nb + 1], low, b[2], b[3]);
       }
     }
   }
@@ -252,6 +288,34 @@ __global__ void __launch_bounds__(32 * kWDWarps) windowed_decode_kernel(const Wi
       }
     }
   }
+  const int size = p.pool.size;
+  if (size > 0 && p.pool_own && chunk == 0 && slice == 0 && w.end % size == 0) {
+    const int b = w.end / size - 1, page = pool_page(b, size, p.block_size), ku_all = p.d >> 3, units = ku_all + (p.dv >> 3);
+    auto block_of = [&](int i) {
+      int blk = p.tables[static_cast<size_t>(s) * p.width + i];
+      if (blk < 0 || blk >= p.num_blocks) {
+        set_status(p.status, kStatusBadIndex);
+        blk = 0;
+      }
+      return static_cast<size_t>(blk) * p.G + g;
+    };
+    for (int u = threadIdx.x; u < units; u += blockDim.x) {
+      const bool value = u >= ku_all;
+      const int cols = value ? p.dv : p.d, c = (value ? u - ku_all : u) * 8;
+      const bf16* cache = value ? p.v_cache : p.k_cache;
+      float sum[8] = {};
+#pragma unroll 8
+      for (int t = b * size; t < w.end; ++t) {
+        float y[8];
+        load_n<8>(cache + (block_of(t / p.block_size) * p.block_size + t % p.block_size) * cols + c, y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum[e] += y[e];
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum[e] /= static_cast<float>(size);
+      store_n<8>((value ? p.pool.v : p.pool.k) + (block_of(page) * p.pool.rows + pool_row(b, page, size, p.block_size)) * cols + c, sum);
+    }
+  }
 }
 
 // CTA = (query head, sequence): merges the chunks of a window that has more than one.
@@ -260,7 +324,7 @@ __global__ void __launch_bounds__(128) windowed_merge_kernel(const WindowedDecod
   pdl_wait();
   const int h = blockIdx.x, s = blockIdx.y;
   const WindowRange w = window_range(p, s, nullptr);
-  const int n = (w.end - w.begin + p.chunk - 1) / p.chunk;
+  const int n = (w.all() + p.chunk - 1) / p.chunk;
   if (n <= 1) return;
   const size_t base = (static_cast<size_t>(s) * p.H + h) * p.max_chunks;
   float M = -INFINITY;
@@ -288,22 +352,26 @@ extern "C" int forge_windowed_decode_ok(int d, int dv, int block_size) {
 }
 
 // q [seqs][H][q_pitch], one token per sequence; out rows of ldo elements.  chunk: a multiple of 16; max_chunks * chunk must cover
-// min(window, width * block_size) + 15 keys.  part_o, part_ml: fp32 scratch, needed when max_chunks > 1.
+// min(window, width * block_size) + 15 keys and, with pooled blocks, width * block_size / pool + 15 entries.  part_o, part_ml: fp32 scratch, needed when max_chunks > 1.
 extern "C" int forge_windowed_decode(const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* tables, const int* lens,
                                      int seqs, int width, int num_blocks, int block_size, void* out, long long ldo, float* part_o, float* part_ml,
                                      int chunk, int max_chunks, int H, int G, int d, int dv, int window, float scale, float out_scale,
                                      int chunked, float softcap, const float* sink, const void* gate, long long ldg, int gate_head, int gate_col,
-                                     unsigned* status, cudaStream_t stream) {
+                                     void* pool_k, void* pool_v, int pool, int pool_own, unsigned* status, cudaStream_t stream) {
   if (seqs <= 0) return 0;
+  if (pool < 0 || (pool > 0 && chunked)) return -1;
+  const int pool_rows = pool > 0 ? (block_size + pool - 1) / pool : 0;
+  if (static_cast<long long>(num_blocks) * G * pool_rows >= (1ll << 31)) return -1;
   if (!forge_windowed_decode_ok(d, dv, block_size) || (q_pitch & 7) || seqs > 65535 || max_chunks > 65535 || chunk % kWDKeys || chunk < kWDKeys || window < 1)
     return -1;
-  const long long cap = static_cast<long long>(width) * block_size, span = (window < cap ? window : cap) + kWDKeys - 1;
+  const long long cap = static_cast<long long>(width) * block_size, span = (window < cap ? window : cap) + kWDKeys - 1 + (pool > 0 ? cap / pool + kWDKeys - 1 : 0);
   if (static_cast<long long>(max_chunks) * chunk < span || (max_chunks > 1 && (part_o == nullptr || part_ml == nullptr))) return -1;
   WindowedDecode p = {static_cast<const bf16*>(q), static_cast<const bf16*>(k_cache), static_cast<const bf16*>(v_cache), tables, lens,
                       static_cast<bf16*>(out), ldo, part_o, part_ml, width, num_blocks, block_size, H, G, d, dv, q_pitch, window, chunk, max_chunks,
                       0, (H / G + 15) / 16, scale * 1.4426950408889634f, out_scale,
                       softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f, softcap * 1.4426950408889634f,
-                      {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}, status};
+                      {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col},
+                      {static_cast<bf16*>(pool_k), static_cast<bf16*>(pool_v), pool, pool_rows}, pool_own, status};
   const dim3 grid(G * p.slices, seqs, max_chunks);
 #define FORGE_WD(NV)                                                                                                                   \
   {                                                                                                                                    \

@@ -10,9 +10,11 @@
 // key it does see, and nothing of O needs scaling then.  Warp roles, double-buffered S, the reference maximum that is only
 // raised when it has grown by 2^8, and bounded waits as in prefill_umma.cu.  V is double-buffered where that leaves room for two CTAs per
 // SM (whose softmax warps hide each other's latency), else single-buffered, else as shared memory allows.
-// Options (chunks, bounded scores, sinks, gated output): attend_options.cuh.
+// Options (chunks, bounded scores, sinks, gated output): attend_options.cuh.  Pooled blocks behind the window (pooled.cuh), gathered by
+// pool_blocks, are key tiles ahead of the others.
 #include "../include/attend_options.cuh"
 #include "../include/launch.cuh"
+#include "../include/pooled.cuh"
 #include "../include/scalar.cuh"
 
 #include <type_traits>
@@ -118,14 +120,16 @@ struct WindowedPrefill {
   float scale_log2, out_scale;
   CapFactors cap;
   AttendOptions<bf16> opt;
+  const int* pool_rows;                     // [seqs] first gathered entry of a sequence
+  int pool;                                 // tokens of a block; 0: no pooled blocks
 };
 
-// tm_q: [tokens, H * 64 nq], box 128 x 64; tm_k / tm_v: [blocks * G * block_size, d / dv], box 64 x 64.
-// kOptions 0: none; 1: chunks, sinks, gates; 2: these and bounded scores.
+// tm_q: [tokens, H * 64 nq], box 128 x 64; tm_k / tm_v: [blocks * G * block_size, d / dv], tm_pk / tm_pv: [entries, G d / G dv], box 64 x 64.
+// kOptions 0: none; 1: chunks, sinks, gates, pooled blocks; 2: these and bounded scores.
 template <int kOptions>
 __global__ void __launch_bounds__(kXThreads, 2)
 windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
-                        const int* __restrict__ cu_q, const int* __restrict__ context_lens, const int* __restrict__ tables,
+                        const __grid_constant__ CUtensorMap tm_pk, const __grid_constant__ CUtensorMap tm_pv, const int* __restrict__ cu_q, const int* __restrict__ context_lens, const int* __restrict__ tables,
                         bf16* __restrict__ out, const WindowedPrefill z, unsigned* status) {
   constexpr bool kCap = kOptions == 2;
   extern __shared__ __align__(1024) uint8_t smem[];   // the swizzled boxes start on multiples of 1024 bytes
@@ -158,8 +162,10 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   const int past = max(k_len - q_len, 0);
   const int kv_end = min(k_len, past + m0 + kXM);
   const int tile0 = oldest_visible(past + m0, z.window, kOptions && z.opt.chunked) / kXN;
-  const int n_tiles = (kv_end + kXN - 1) / kXN - tile0;
-  if (n_tiles <= 0) return;
+  int n_pool = 0;                                     // tiles of pooled blocks: what the CTA's last row sees
+  if (kOptions && z.pool > 0) n_pool = (pool_visible(oldest_visible(min(past + q_len, kv_end) - 1, z.window, 0), z.pool) + kXN - 1) / kXN;
+  const int n_tiles = n_pool + (kv_end + kXN - 1) / kXN - tile0;
+  if (n_tiles <= n_pool) return;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp == 0 && lane == 0) {
@@ -194,21 +200,31 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       mbar_expect_tx(q_full, z.nq * kXQBox);
       for (int b = 0; b < z.nq; ++b) tma_load_2d(sQ + b * kXQBox, &tm_q, q_full, (h * z.nq + b) * 64, q_begin + m0);
       for (int j = 0; j < n_tiles; ++j) {
-        const int s = j & 1, tok = (tile0 + j) * kXN;
+        const bool means = kOptions && j < n_pool;
+        const int s = j & 1, tok = (tile0 + j - n_pool) * kXN;
         const uint32_t ph = (j >> 1) & 1;
-        int blk = tables[static_cast<size_t>(seq) * z.table_width + tok / z.block_size];
-        if (blk < 0 || blk >= z.num_blocks) {
-          set_status(status, kStatusBadIndex);
-          blk = 0;
+        int row, k_col = 0, v_col = 0;
+        if (means) {                                                               // columns past a head's are its neighbour's: q is zero there
+          row = z.pool_rows[seq] + j * kXN;
+          k_col = g * z.d;
+          v_col = g * z.dv;
+        } else {
+          int blk = tables[static_cast<size_t>(seq) * z.table_width + tok / z.block_size];
+          if (blk < 0 || blk >= z.num_blocks) {
+            set_status(status, kStatusBadIndex);
+            blk = 0;
+          }
+          row = (blk * z.G + g) * z.block_size + tok % z.block_size;               // a tile never straddles a block
         }
-        const int row = (blk * z.G + g) * z.block_size + tok % z.block_size;       // a tile never straddles a block
+        const CUtensorMap* map_k = means ? &tm_pk : &tm_k;
+        const CUtensorMap* map_v = means ? &tm_pv : &tm_v;
         if (!mbar_wait_parked(&k_empty[s], ph ^ 1, status)) break;
         mbar_expect_tx(&k_full[s], k_stage);
-        for (int b = 0; b < z.nq; ++b) tma_load_2d(sK + s * k_stage + b * kXKBox, &tm_k, &k_full[s], b * 64, row);
+        for (int b = 0; b < z.nq; ++b) tma_load_2d(sK + s * k_stage + b * kXKBox, map_k, &k_full[s], k_col + b * 64, row);
         const int vs = j % z.v_bufs;
         if (!mbar_wait_parked(&v_empty[vs], ((j / z.v_bufs) & 1) ^ 1, status)) break;
         mbar_expect_tx(&v_full[vs], v_stage);
-        for (int b = 0; b < z.nv; ++b) tma_load_2d(sV + vs * v_stage + b * kXKBox, &tm_v, &v_full[vs], b * 64, row);
+        for (int b = 0; b < z.nv; ++b) tma_load_2d(sV + vs * v_stage + b * kXKBox, map_v, &v_full[vs], v_col + b * 64, row);
       }
     }
   } else if (warp == 1) {
@@ -260,7 +276,8 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const int r = quad * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const int qpos = past + m0 + r;
-    const int limit = min(qpos + 1, k_len), lo = oldest_visible(qpos, z.window, kOptions && z.opt.chunked);          // visible keys: [lo, limit)
+    const int key_limit = min(qpos + 1, k_len), key_lo = oldest_visible(qpos, z.window, kOptions && z.opt.chunked);  // visible keys
+    const int block_limit = kOptions && z.pool > 0 ? pool_visible(key_lo, z.pool) : 0;                             // visible blocks
     const int o_cols = z.nv * 64;
     float m_ref = 0.f, l_run = 0.f;
     bool seen = false, ok = true;
@@ -269,7 +286,9 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       if (!ok) break;
       tcgen05_fence_after();
       const uint32_t s_addr = tmem_base + lane_addr + (j & 1) * kXN;
-      const int kbase = (tile0 + j) * kXN;
+      const bool means = kOptions && j < n_pool;
+      const int kbase = means ? j * kXN : (tile0 + j - n_pool) * kXN;
+      const int lo = means ? 0 : key_lo, limit = means ? block_limit : key_limit;            // visible in this tile: [lo, limit)
       const bool masked = !__all_sync(0xffffffffu, kbase >= lo && kbase + kXN <= limit);
       float size;
       float mt = masked ? windowed_row_max<true, kCap>(s_addr, kbase, lo, limit, size) : windowed_row_max<false, kCap>(s_addr, kbase, lo, limit, size);
@@ -386,16 +405,18 @@ extern "C" int forge_make_tmap_2d(CUtensorMap* tm, const void* base, uint64_t ro
                                   uint32_t box_rows, int elem_bytes);
 
 // q [tokens][H][q_pitch], q_pitch = forge_windowed_prefill_qcols; sequence s has the step's tokens cu_q[s] .. cu_q[s + 1] (its last
-// ones) and context_lens[s] keys; out rows of ldo elements (a multiple of 8), 16-byte aligned; a gate per element likewise.
+// ones) and context_lens[s] keys; out rows of ldo elements (a multiple of 8), 16-byte aligned; a gate per element likewise.  pool: tokens of a
+// pooled block (0: none), pool_k / pool_v [pool_entries][G][d / dv] the gathered entries, pool_rows [seqs] where a sequence's begin.
 extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_cache, const void* v_cache, const int* cu_q, const int* context_lens,
                                       const int* tables, int table_width, int num_blocks, int block_size, void* out, long long ldo, int num_seqs,
                                       int max_q, int H, int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap,
-                                      const float* sink, const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status,
-                                      cudaStream_t stream) {
+                                      const float* sink, const void* gate, long long ldg, int gate_head, int gate_col, const void* pool_k,
+                                      const void* pool_v, const int* pool_rows, int pool_entries, int pool, unsigned* status, cudaStream_t stream) {
   if (tokens <= 0 || num_seqs <= 0 || max_q <= 0) return 0;
   const int qcols = forge_windowed_prefill_qcols(d, dv, block_size);
   if (qcols == 0 || num_seqs > 65535 || H > 65535 || H % G || window < 1 || !(scale > 0.f) || (ldo & 7) || (reinterpret_cast<uintptr_t>(out) & 15)) return -1;
   if (static_cast<long long>(num_blocks) * G * block_size >= (1ll << 31)) return -1;
+  if (pool < 0 || (pool > 0 && (chunked || pool_entries < 1 || pool_rows == nullptr))) return -1;
   if (gate != nullptr && gate_col != 0 && (gate_col != 1 || ((ldg | gate_head) & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -1;
   const int nq = qcols / 64, nv = (dv + 63) / 64;
   constexpr int kHalf = 113 * 1024, kAll = 227 * 1024;        // two CTAs per SM, one
@@ -406,17 +427,24 @@ extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_c
   if (smem > kAll) return -1;
   const WindowedPrefill z = {H, G, d, dv, nq, nv, v_bufs, window, block_size, table_width, num_blocks, ldo, scale * 1.4426950408889634f, out_scale,
                              cap_factors(scale, softcap),
-                             {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}};
-  CUtensorMap tm_q, tm_k, tm_v;
+                             {chunked, softcap, sink, static_cast<const bf16*>(gate), ldg, gate_head, gate_col}, pool_rows, pool};
+  CUtensorMap tm_q, tm_k, tm_v, tm_pk, tm_pv;
   const uint64_t qw = static_cast<uint64_t>(H) * qcols, rows = static_cast<uint64_t>(num_blocks) * G * block_size;
   if (forge_make_tmap_2d(&tm_q, q, tokens, qw, qw, kXM, 2) != 0) return -2;
   if (forge_make_tmap_2d(&tm_k, k_cache, rows, d, d, kXN, 2) != 0) return -2;
   if (forge_make_tmap_2d(&tm_v, v_cache, rows, dv, dv, kXN, 2) != 0) return -2;
+  tm_pk = tm_k;
+  tm_pv = tm_v;
+  if (pool > 0) {
+    const uint64_t kw = static_cast<uint64_t>(G) * d, vw = static_cast<uint64_t>(G) * dv;
+    if (forge_make_tmap_2d(&tm_pk, pool_k, pool_entries, kw, kw, kXN, 2) != 0) return -2;
+    if (forge_make_tmap_2d(&tm_pv, pool_v, pool_entries, vw, vw, kXN, 2) != 0) return -2;
+  }
   FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<0>, 227 * 1024);
   FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<1>, 227 * 1024);
   FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<2>, 227 * 1024);
-  auto k = softcap > 0.f ? windowed_prefill_kernel<2> : chunked || sink != nullptr || gate != nullptr ? windowed_prefill_kernel<1> : windowed_prefill_kernel<0>;
-  return launch_kernel(k, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v,
+  auto k = softcap > 0.f ? windowed_prefill_kernel<2> : chunked || sink != nullptr || gate != nullptr || pool > 0 ? windowed_prefill_kernel<1> : windowed_prefill_kernel<0>;
+  return launch_kernel(k, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v, tm_pk, tm_pv,
                        cu_q, context_lens, tables, static_cast<bf16*>(out), z, status) == cudaSuccess ? 0 : -5;
 }
 

@@ -396,6 +396,26 @@ extern "C" int forge_stream_update(int fp32, float* x, const void* a, const void
   return stream_update<T>(out_rows, p, stream);
 }
 
+// x <- act(x) elementwise (PlainAct), bf16 or fp32; logits <- cap tanh(scale logits / cap).
+template <typename T>
+__global__ void __launch_bounds__(256) act_any_kernel(T* __restrict__ x, long long n, int act, bool logits, float scale, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const float v = load_f(x + i);
+    store_f(x + i, logits ? bound_logit<sizeof(T) == 4>(v, scale, cap) : plain_act(act, v));
+  }
+}
+
+extern "C" int forge_act_any(int fp32, void* x, long long n, int act, int logits, float scale, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  long long grid = (n + 255) / 256;
+  if (grid > device_sm_count() * 16) grid = device_sm_count() * 16;
+  const dim3 g(static_cast<unsigned>(grid));
+  if (fp32) return launch_kernel(act_any_kernel<float>, g, dim3(256), 0, stream, 0, static_cast<float*>(x), n, act, logits != 0, scale, cap) == cudaSuccess ? 0 : -2;
+  return launch_kernel(act_any_kernel<bf16>, g, dim3(256), 0, stream, 0, static_cast<bf16*>(x), n, act, logits != 0, scale, cap) == cudaSuccess ? 0 : -2;
+}
+
 // out[r, :I] = act(x[r, :I], x[r, I:2I]) (GateAct), any I, bf16 or fp32 (the fused epilogue of the tcgen05 GEMMs needs no such pass).
 template <typename T>
 __global__ void __launch_bounds__(256) act_mul_any_kernel(const T* __restrict__ x, T* __restrict__ out, long long rows, int I, int act,

@@ -93,6 +93,7 @@ struct GemmSample {
   float* part_v;             // [rows][n_tiles]
   int* part_i;
   int n_tiles;
+  float scale, cap;          // logits <- bounded by cap (scale * logits); scale 1 and cap 0: as they are
 };
 
 // q/k-norm + rotary embedding + KV-cache store in the epilogue of the qkv projection (kEpiQkv; head_dim 128, tiles of 128
@@ -524,6 +525,7 @@ gemm_tokens_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_consta
           const float T = live ? samp.temps[r] : 0.f;
           const bool greedy = !(T > 0.f);
           const float inv_t = greedy ? 1.f : 1.f / T;
+          const bool bounded = samp.cap > 0.f || samp.scale != 1.f;
           const uint32_t step = static_cast<uint32_t>(samp.header[9]);
           const uint32_t k0 = static_cast<uint32_t>(samp.header[10]), k1 = static_cast<uint32_t>(samp.header[11]);
           Best best{-INFINITY, 0x7fffffff};              // best group of this tile: (score, group index)
@@ -546,6 +548,11 @@ gemm_tokens_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_consta
 #pragma unroll
                 for (int i = 0; i < kSampleGroup; ++i)
                   lv[i] = c0 + cc + h * kSampleGroup + i < n_total ? bf16_round_g(__uint_as_float(v[h * kSampleGroup + i])) : -INFINITY;
+                if (bounded) {
+#pragma unroll
+                  for (int i = 0; i < kSampleGroup; ++i)
+                    if (lv[i] != -INFINITY) lv[i] = bf16_round_g(bound_logit<false>(lv[i], samp.scale, samp.cap));
+                }
                 const float sg = sample_group_score(lv, inv_t, greedy, rnd[(g0 + h) & 3]);
                 if (sg > best.v) {                         // groups are visited in ascending order: ties keep the earlier one
                   best = Best{sg, g0 + h};
@@ -1777,7 +1784,7 @@ extern "C" int forge_sample_merge(const float* part_v, const int* part_i, int n,
 // ids; a 32-column chunk of the accumulator holds two whole groups).
 extern "C" int forge_gemm_bf16_sample(const void* x, int ldx, const void* w, int ldw, int M, int vocab, int K, int vocab_start,
                                       const float* temps, const int* header, float* part_v, int* part_i, int* out_i, float* out_v,
-                                      unsigned* status, cudaStream_t stream) {
+                                      float scale, float cap, unsigned* status, cudaStream_t stream) {
   if (M <= 0 || vocab <= 0) return 0;
   if ((K & 7) || (ldx & 7) || (ldw & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) ||
       (vocab_start & 31))
@@ -1789,6 +1796,8 @@ extern "C" int forge_gemm_bf16_sample(const void* x, int ldx, const void* w, int
   samp.part_v = part_v;
   samp.part_i = part_i;
   samp.n_tiles = (vocab + 255) / 256;
+  samp.scale = scale;
+  samp.cap = cap;
   TpPush none = {};
   GemmFuse plain = {};
   const int rc = launch_tokens<256, kEpiSample>(x, ldx, w, vocab, ldw, nullptr, 0, M, vocab, K, status, stream, none, plain, samp);

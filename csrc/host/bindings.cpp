@@ -14,7 +14,7 @@ int forge_gemm_bf16_fused(const void* x, int ldx, const void* w, int ldw, void* 
                           int force_mode, int tune, const float* in_ssq, int in_parts, float eps, int add_residual, float* out_ssq,
                           unsigned* status, cudaStream_t stream);
 int forge_gemm_bf16_sample(const void* x, int ldx, const void* w, int ldw, int M, int vocab, int K, int vocab_start, const float* temps,
-                           const int* header, float* part_v, int* part_i, int* out_i, float* out_v, unsigned* status,
+                           const int* header, float* part_v, int* part_i, int* out_i, float* out_v, float scale, float cap, unsigned* status,
                            cudaStream_t stream);
 int forge_gemm_set_trace(unsigned long long* buf);
 long long forge_launch_count();
@@ -166,9 +166,10 @@ void gemm_fused(const Tensor& x, const Tensor& w, Tensor& out, int64_t epi, int6
 }
 
 // LM head + sampling: x [rows, K] @ w [vocab, K]^T, sampled per row without writing the logits.  part_v / part_i: scratch of
-// rows * ceil(vocab / 256) entries; out_i / out_v: the winning global id and its score per row.
+// rows * ceil(vocab / 256) entries; out_i / out_v: the winning global id and its score per row; logits are bounded by cap
+// (scale * logits; cap 0: not).
 void gemm_sample(const Tensor& x, const Tensor& w, int64_t vocab_start, const Tensor& temps, const Tensor& header, Tensor& part_v,
-                 Tensor& part_i, Tensor& out_i, Tensor& out_v, const Tensor& status) {
+                 Tensor& part_i, Tensor& out_i, Tensor& out_v, double scale, double cap, const Tensor& status) {
   CHECK_BF16(x); CHECK_BF16(w); CHECK_CUDA_CONTIG(temps); CHECK_F32(temps); CHECK_CUDA_CONTIG(header); CHECK_I32(header);
   CHECK_CUDA_CONTIG(part_v); CHECK_F32(part_v); CHECK_CUDA_CONTIG(part_i); CHECK_I32(part_i);
   CHECK_CUDA_CONTIG(out_i); CHECK_I32(out_i); CHECK_CUDA_CONTIG(out_v); CHECK_F32(out_v);
@@ -183,7 +184,8 @@ void gemm_sample(const Tensor& x, const Tensor& w, int64_t vocab_start, const Te
   check(forge_gemm_bf16_sample(x.data_ptr(), static_cast<int>(x.stride(0)), w.data_ptr(), static_cast<int>(w.stride(0)),
                                static_cast<int>(rows), static_cast<int>(vocab), static_cast<int>(x.size(1)),
                                static_cast<int>(vocab_start), temps.data_ptr<float>(), header.data_ptr<int>(), part_v.data_ptr<float>(),
-                               part_i.data_ptr<int>(), out_i.data_ptr<int>(), out_v.data_ptr<float>(), status_ptr(status), stream_of(x)),
+                               part_i.data_ptr<int>(), out_i.data_ptr<int>(), out_v.data_ptr<float>(), static_cast<float>(scale),
+                               static_cast<float>(cap), status_ptr(status), stream_of(x)),
         "forge_gemm_bf16_sample");
 }
 

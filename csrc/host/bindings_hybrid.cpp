@@ -9,10 +9,16 @@ int forge_bias_rope_store(int fp32, const void* proj, long long ld, int tokens, 
 int forge_windowed_attend_any(int fp32, const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* cu, int seqs, int max_q,
                               const int* positions, const int* tables, int width, int num_blocks, int block_size, void* out, long long ldo, int H,
                               int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap, const float* sink,
-                              const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status, cudaStream_t stream);
+                              const void* gate, long long ldg, int gate_head, int gate_col, const void* pool_k, const void* pool_v, int pool,
+                              unsigned* status, cudaStream_t stream);
 int forge_norm_rope_store(int fp32, const void* proj, long long ld, int tokens, const void* q_norm, const void* k_norm, int whole, float eps,
                           const float* rope, int rope_rows, int rd, const int* positions, const int* slots, void* q, int q_pitch, void* k_cache,
-                          void* v_cache, long long num_slots, int block_size, int H, int G, int d, int dv, unsigned* status, cudaStream_t stream);
+                          void* v_cache, long long num_slots, int block_size, int H, int G, int d, int dv, const float* temper, unsigned* status,
+                          cudaStream_t stream);
+int forge_pool_blocks(int fp32, const void* k_cache, const void* v_cache, void* pool_k, void* pool_v, int size, int own, const int* cu, const int* lens,
+                      const int* tables, int seqs, int max_q, int max_k, const int* offsets, void* gk, void* gv, int bound, int width, int num_blocks,
+                      int block_size, int G, int d, int dv, unsigned* status, cudaStream_t stream);
+int forge_row_offsets(const int* cu, const int* lens, int seqs, int window, int size, int* out, cudaStream_t stream);
 int forge_stream_mix(int fp32, float* x, const void* y, const float* mix, const float* out, const int* ids, const int* prev, const void* embed,
                      int vocab, float scale, const void* pairs, int buckets, long long mul_prev, long long mul_cur, const float* into, const void* w,
                      const void* b, void* h, const int* rows, int out_rows, int n_rows, int W, int S, float eps, cudaStream_t stream);
@@ -28,12 +34,14 @@ int forge_windowed_decode_ok(int d, int dv, int block_size);
 int forge_windowed_decode(const void* q, int q_pitch, const void* k_cache, const void* v_cache, const int* tables, const int* lens, int seqs,
                           int width, int num_blocks, int block_size, void* out, long long ldo, float* part_o, float* part_ml, int chunk,
                           int max_chunks, int H, int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap,
-                          const float* sink, const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status, cudaStream_t stream);
+                          const float* sink, const void* gate, long long ldg, int gate_head, int gate_col, void* pool_k, void* pool_v, int pool,
+                          int pool_own, unsigned* status, cudaStream_t stream);
 int forge_windowed_prefill_qcols(int d, int dv, int block_size);
 int forge_windowed_prefill(const void* q, int tokens, const void* k_cache, const void* v_cache, const int* cu_q, const int* context_lens,
                            const int* tables, int table_width, int num_blocks, int block_size, void* out, long long ldo, int num_seqs, int max_q,
                            int H, int G, int d, int dv, int window, float scale, float out_scale, int chunked, float softcap, const float* sink,
-                           const void* gate, long long ldg, int gate_head, int gate_col, unsigned* status, cudaStream_t stream);
+                           const void* gate, long long ldg, int gate_head, int gate_col, const void* pool_k, const void* pool_v, const int* pool_rows,
+                           int pool_entries, int pool, unsigned* status, cudaStream_t stream);
 int forge_recurrence_gates(const void* dt, const void* beta, long long ld_raw, const float* A_log, const float* dt_bias, const int* cu, int seqs,
                            int max_q, int heads, float* cum, float* weight, long long ldt, cudaStream_t stream);
 int forge_retention_chunk_ok(int heads, int dk, int dv, int rd);
@@ -79,21 +87,77 @@ void bias_rope_store(const Tensor& proj, const Tensor& bias, const Tensor& rope,
            "forge_bias_rope_store");
 }
 
-// The same with norms of q and k ahead of the rotation and no biases; norm weights of dim entries (per head) or of all rows
-void norm_rope_store(const Tensor& proj, const Tensor& q_norm, const Tensor& k_norm, bool whole, double eps, const Tensor& rope, const Tensor& positions,
-                     const Tensor& slots, Tensor& q, Tensor& k_cache, Tensor& v_cache, const Tensor& status) {
+// The same with norms of q and k ahead of the rotation and no biases; norm weights of dim entries (per head) or of all rows.  Without k_norm
+// proj is q alone and nothing is stored.  temper fp32 [H]: one more factor of the queries
+void norm_rope_store(const Tensor& proj, const Tensor& q_norm, const OptTensor& k_norm, bool whole, double eps, const Tensor& rope, const Tensor& positions,
+                     const Tensor& slots, Tensor& q, Tensor& k_cache, Tensor& v_cache, const OptTensor& temper, const Tensor& status) {
   const int f = elem(proj);
   const auto dt = proj.scalar_type();
-  const Caches c = cache_sizes(k_cache, v_cache, dt);
+  Caches c = cache_sizes(k_cache, v_cache, dt);
+  if (!k_norm.has_value()) c.G = 0;
   TORCH_CHECK(q.dim() == 3 && q.size(0) == proj.size(0) && rope.dim() == 2 && rope.size(1) % 2 == 0 && rope.size(1) <= c.d && q.size(2) >= c.d, "norm_rope_store: sizes");
   const int64_t T = proj.size(0), H = q.size(1), rows = (H + c.G) * c.d + c.G * c.dv;
   const c10::cuda::CUDAGuard guard(proj.device());
   check_rc(forge_norm_rope_store(f, view2(proj, dt, T, rows, "proj"), proj.stride(0), i32(T), data(q_norm, dt, whole ? H * c.d : c.d, "q_norm"),
-                                 data(k_norm, dt, whole ? c.G * c.d : c.d, "k_norm"), whole ? 1 : 0, static_cast<float>(eps), floats(rope, 0, "rope"),
+                                 k_norm.has_value() ? data(*k_norm, dt, whole ? c.G * c.d : c.d, "k_norm") : nullptr, whole ? 1 : 0, static_cast<float>(eps), floats(rope, 0, "rope"),
                                  i32(rope.size(0)), i32(rope.size(1)), ints(positions, T, "positions"), ints(slots, T, "slots"), data(q, dt, 0, "q"),
                                  i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), static_cast<long long>(c.blocks) * c.block_size,
-                                 i32(c.block_size), i32(H), i32(c.G), i32(c.d), i32(c.dv), status_word(status), stream_of(proj)),
+                                 i32(c.block_size), i32(H), i32(c.G), i32(c.d), i32(c.dv), temper.has_value() ? floats(*temper, H, "temper") : nullptr,
+                                 status_word(status), stream_of(proj)),
            "forge_norm_rope_store");
+}
+
+// Means of blocks: caches [blocks, kv_heads, ceil(block_size / size), dim / vdim]
+struct Pool {
+  void* k = nullptr;
+  void* v = nullptr;
+};
+Pool pool_caches(const OptTensor& pool_k, const OptTensor& pool_v, int64_t size, const Caches& c, at::ScalarType dt) {
+  Pool p;
+  TORCH_CHECK(size >= 0 && (size == 0) == !pool_k.has_value(), "pooled blocks: size and caches");
+  if (size == 0) return p;
+  const int64_t rows = (c.block_size + size - 1) / size;
+  TORCH_CHECK(pool_v.has_value() && pool_k->dim() == 4 && pool_v->dim() == 4 && pool_k->size(0) == c.blocks && pool_k->size(1) == c.G && pool_k->size(2) == rows &&
+                  pool_k->size(3) == c.d && pool_v->size(0) == c.blocks && pool_v->size(1) == c.G && pool_v->size(2) == rows && pool_v->size(3) == c.dv,
+              "pooled blocks: caches [blocks, kv_heads, ceil(block_size / size), dim] and [.., vdim] expected");
+  p.k = data(*pool_k, dt, 0, "pool_k");
+  p.v = data(*pool_v, dt, 0, "pool_v");
+  return p;
+}
+
+// The entries of the blocks that end in the step's tokens (own), and with offsets all entries gathered to gk, gv [rows, kv_heads, dim / vdim]
+void pool_blocks(const Tensor& k_cache, const Tensor& v_cache, const Tensor& pool_k, const Tensor& pool_v, int64_t size, bool own, const Tensor& cu,
+                 const Tensor& lens, const Tensor& tables, int64_t seqs, int64_t max_q, int64_t max_k, const OptTensor& offsets, const OptTensor& gk,
+                 const OptTensor& gv, const Tensor& status) {
+  const int f = elem(k_cache);
+  const auto dt = k_cache.scalar_type();
+  const Caches c = cache_sizes(k_cache, v_cache, dt);
+  TORCH_CHECK(size >= 1 && tables.dim() == 2 && tables.size(0) >= seqs, "pool_blocks: sizes");
+  const Pool p = pool_caches(pool_k, pool_v, size, c, dt);
+  const int* op = nullptr;
+  void *kp = nullptr, *vp = nullptr;
+  int64_t bound = 0;
+  if (offsets.has_value()) {
+    TORCH_CHECK(gk.has_value() && gv.has_value() && gk->dim() == 3 && gv->dim() == 3, "pool_blocks: gather buffers");
+    bound = gk->size(0);
+    op = ints(*offsets, seqs + 1, "offsets");
+    kp = data(*gk, dt, bound * c.G * c.d, "gk");
+    vp = data(*gv, dt, bound * c.G * c.dv, "gv");
+  }
+  const c10::cuda::CUDAGuard guard(k_cache.device());
+  check_rc(forge_pool_blocks(f, k_cache.data_ptr(), v_cache.data_ptr(), p.k, p.v, i32(size), own ? 1 : 0, ints(cu, seqs + 1, "cu"), ints(lens, seqs, "lens"),
+                             ints(tables, 0, "tables"), i32(seqs), i32(max_q), i32(max_k), op, kp, vp, i32(bound), i32(tables.size(1)), i32(c.blocks),
+                             i32(c.block_size), i32(c.G), i32(c.d), i32(c.dv), status_word(status), stream_of(k_cache)),
+           "forge_pool_blocks");
+}
+
+// out [seqs + 1]: running sums of floor(keys / size) or, with size 0, of min(keys, queries + window - 1)
+void row_offsets(const Tensor& cu, const Tensor& lens, int64_t seqs, int64_t window, int64_t size, Tensor& out) {
+  TORCH_CHECK(size >= 0 && (size > 0 || window >= 1), "row_offsets: sizes");
+  const c10::cuda::CUDAGuard guard(cu.device());
+  check_rc(forge_row_offsets(ints(cu, seqs + 1, "cu"), ints(lens, seqs, "lens"), i32(seqs), i32(window), i32(size), const_cast<int*>(ints(out, seqs + 1, "out")),
+                             stream_of(cu)),
+           "forge_row_offsets");
 }
 
 // x fp32 [tokens, streams, width].  With y [tokens, width]: mix [streams, streams], out [streams]; without: the streams begin as embeddings
@@ -172,16 +236,18 @@ Attend attend_sizes(const Tensor& q, const Tensor& k_cache, const Tensor& v_cach
 // q [tokens, H, q_pitch], out [tokens, H dv] (a view); sequence s: query rows cu[s] .. cu[s + 1]
 void windowed_attend_any(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu, int64_t seqs, int64_t max_q,
                          const Tensor& positions, const Tensor& tables, Tensor& out, int64_t window, double scale, double out_scale,
-                         bool chunked, double softcap, const OptTensor& sink, const OptTensor& gate, const Tensor& status) {
+                         bool chunked, double softcap, const OptTensor& sink, const OptTensor& gate, const OptTensor& pool_k, const OptTensor& pool_v,
+                         int64_t pool, const Tensor& status) {
   const int f = elem(q);
   const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
+  const Pool m = pool_caches(pool_k, pool_v, pool, a.c, q.scalar_type());
   const Options x = attend_options(chunked, softcap, sink, gate, a, q.scalar_type());
   const c10::cuda::CUDAGuard guard(q.device());
   check_rc(forge_windowed_attend_any(f, q.data_ptr(), i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), ints(cu, seqs + 1, "cu"), i32(seqs),
                                      i32(max_q), ints(positions, a.T, "positions"), ints(tables, 0, "tables"), i32(tables.size(1)), i32(a.c.blocks),
                                      i32(a.c.block_size), out.data_ptr(), out.stride(0), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window),
                                      static_cast<float>(scale), static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head,
-                                     x.gate_col, status_word(status), stream_of(q)),
+                                     x.gate_col, m.k, m.v, i32(pool), status_word(status), stream_of(q)),
            "forge_windowed_attend_any");
 }
 
@@ -190,9 +256,11 @@ constexpr auto kBf16 = at::kBFloat16;
 // One token per sequence: rows 0 .. seqs - 1 of q and out.
 void windowed_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& tables, const Tensor& lens, int64_t seqs,
                      Tensor& out, const OptTensor& part_o, const OptTensor& part_ml, int64_t chunk, int64_t max_chunks, int64_t window,
-                     double scale, double out_scale, bool chunked, double softcap, const OptTensor& sink, const OptTensor& gate, const Tensor& status) {
+                     double scale, double out_scale, bool chunked, double softcap, const OptTensor& sink, const OptTensor& gate, const OptTensor& pool_k,
+                     const OptTensor& pool_v, int64_t pool, bool pool_own, const Tensor& status) {
   TORCH_CHECK(q.scalar_type() == kBf16 && seqs <= q.size(0), "windowed_decode: q");
   const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
+  const Pool m = pool_caches(pool_k, pool_v, pool, a.c, q.scalar_type());
   const Options x = attend_options(chunked, softcap, sink, gate, a, q.scalar_type());
   float *po = nullptr, *pm = nullptr;
   if (max_chunks > 1) {
@@ -204,25 +272,38 @@ void windowed_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cac
   check_rc(forge_windowed_decode(q.data_ptr(), i32(q.size(2)), k_cache.data_ptr(), v_cache.data_ptr(), ints(tables, 0, "tables"), ints(lens, seqs, "lens"),
                                  i32(seqs), i32(tables.size(1)), i32(a.c.blocks), i32(a.c.block_size), out.data_ptr(), out.stride(0), po, pm, i32(chunk),
                                  i32(max_chunks), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window), static_cast<float>(scale),
-                                 static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head, x.gate_col, status_word(status),
-                                 stream_of(q)),
+                                 static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head, x.gate_col, m.k, m.v, i32(pool),
+                                 pool_own ? 1 : 0, status_word(status), stream_of(q)),
            "forge_windowed_decode");
 }
 
-// Sequence s: the rows cu[s] .. cu[s + 1] of q and out, its last ones; context_lens[s] keys.
+// Sequence s: the rows cu[s] .. cu[s + 1] of q and out, its last ones; context_lens[s] keys.  gk, gv, offsets: entries of pooled blocks as
+// pool_blocks gathers them.
 void windowed_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const Tensor& cu, const Tensor& context_lens, const Tensor& tables,
                       int64_t seqs, int64_t max_q, Tensor& out, int64_t window, double scale, double out_scale, bool chunked, double softcap,
-                      const OptTensor& sink, const OptTensor& gate, const Tensor& status) {
+                      const OptTensor& sink, const OptTensor& gate, const OptTensor& gk, const OptTensor& gv, const OptTensor& offsets, int64_t pool,
+                      const Tensor& status) {
   TORCH_CHECK(q.scalar_type() == kBf16, "windowed_prefill: q");
   const Attend a = attend_sizes(q, k_cache, v_cache, out, tables, seqs);
   const Options x = attend_options(chunked, softcap, sink, gate, a, q.scalar_type());
   TORCH_CHECK(q.size(2) == forge_windowed_prefill_qcols(i32(a.c.d), i32(a.c.dv), i32(a.c.block_size)), "windowed_prefill: q columns");
+  const void *kp = nullptr, *vp = nullptr;
+  const int* op = nullptr;
+  int64_t entries = 0;
+  TORCH_CHECK(pool >= 0 && (pool == 0) == !gk.has_value(), "windowed_prefill: pooled blocks");
+  if (pool > 0) {
+    TORCH_CHECK(gv.has_value() && offsets.has_value(), "windowed_prefill: pooled blocks");
+    entries = gk->size(0);
+    kp = data(*gk, kBf16, entries * a.c.G * a.c.d, "gk");
+    vp = data(*gv, kBf16, entries * a.c.G * a.c.dv, "gv");
+    op = ints(*offsets, seqs + 1, "offsets");
+  }
   const c10::cuda::CUDAGuard guard(q.device());
   check_rc(forge_windowed_prefill(q.data_ptr(), i32(a.T), k_cache.data_ptr(), v_cache.data_ptr(), ints(cu, seqs + 1, "cu"), ints(context_lens, seqs, "lens"),
                                   ints(tables, 0, "tables"), i32(tables.size(1)), i32(a.c.blocks), i32(a.c.block_size), out.data_ptr(), out.stride(0),
                                   i32(seqs), i32(max_q), i32(a.H), i32(a.c.G), i32(a.c.d), i32(a.c.dv), i32(window), static_cast<float>(scale),
-                                  static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head, x.gate_col, status_word(status),
-                                  stream_of(q)),
+                                  static_cast<float>(out_scale), x.chunked, x.softcap, x.sink, x.gate, x.ldg, x.gate_head, x.gate_col, kp, vp, op,
+                                  i32(entries), i32(pool), status_word(status), stream_of(q)),
            "forge_windowed_prefill");
 }
 
@@ -350,6 +431,8 @@ void register_hybrid(pybind11::module& m) {
   m.def("bias_rope_store", &bias_rope_store);
   m.def("norm_rope_store", &norm_rope_store);
   m.def("stream_mix", &stream_mix);
+  m.def("pool_blocks", &pool_blocks);
+  m.def("row_offsets", &row_offsets);
   m.def("windowed_attend_any", &windowed_attend_any);
   m.def("windowed_decode", &windowed_decode);
   m.def("windowed_decode_ok", [](int64_t d, int64_t dv, int64_t bs) { return forge_windowed_decode_ok(i32(d), i32(dv), i32(bs)) != 0; });

@@ -17,19 +17,23 @@ int forge_stream_update(int fp32, float* x, const void* a, const void* b, const 
 int forge_stream_sandwich(int fp32, float* x, const void* a, const int* a_rows, const float* a_weights, int top, const float* a_bias,
                           const void* post, float mult, float offset, const int* ids, const void* embed, int vocab, const void* w, void* h,
                           const int* rows, int out_rows, int n_rows, int W, int start, float eps, cudaStream_t stream);
+int forge_stream_group(int fp32, float* x, const void* a, const int* a_rows, const float* a_weights, int top, const void* post, float mult,
+                       float offset, const int* ids, const void* embed, int vocab, const void* w, void* h, const int* rows, int out_rows, int n_rows,
+                       int W, int groups, int start, float eps, cudaStream_t stream);
+int forge_act_any(int fp32, void* x, long long n, int act, int logits, float scale, float cap, cudaStream_t stream);
 int forge_act_mul_any(int fp32, const void* x, void* out, long long rows, int I, int act, float limit, cudaStream_t stream);
 int forge_gemm_bf16_act(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int M, int n_out, int K, int act, float limit,
                         unsigned* status, cudaStream_t stream);
 int forge_gemm_simt(int fp32, const void* x, long long ldx, long long x_batch, const void* w, long long ldw, long long w_batch, void* out,
                     long long ldo, long long o_batch, int M, int N, int K, int batch, const int* tile_expert, cudaStream_t stream);
-int forge_latent_prepare(int fp32, const void* proj, int T, int q_rank, int kv_rank, int rot, const void* qw, const void* kw, float eps,
+int forge_latent_prepare(int fp32, const void* proj, long long ld, int T, int q_rank, int kv_rank, int rot, const void* qw, const void* kw, float eps,
                          const float* rope, int rope_rows, const int* positions, const int* slots, void* cq, void* cache,
                          long long num_slots, unsigned* status, cudaStream_t stream);
-int forge_latent_rotate_q(int fp32, const void* q, void* qa, int tokens, int heads, int dim, int rot, int kv_rank, const float* rope,
+int forge_latent_rotate_q(int fp32, const void* q, long long ld, void* qa, int tokens, int heads, int dim, int rot, int kv_rank, const float* rope,
                           int rope_rows, const int* positions, cudaStream_t stream);
 int forge_latent_attend_any(int fp32, const void* qa, const void* cache, void* o, int tok0, int tokens, const int* cu, int num_seqs,
                             const int* positions, const int* block_tables, int table_width, int num_blocks, int block_size, int heads,
-                            int kv_rank, int rot, float scale, unsigned* status, cudaStream_t stream);
+                            int kv_rank, int rot, int window, float scale, unsigned* status, cudaStream_t stream);
 int forge_retention_decode(int fp32, const void* qkvg, int ld, const float* decay, float* state, const int* slots, const int* positions,
                            const float* rope, int rope_rows, int rd, int seqs, int heads, int dk, int dv, int num_slots, void* y, float eps,
                            unsigned* status, cudaStream_t stream);
@@ -38,8 +42,8 @@ int forge_retention_scan(int fp32, const void* qkvg, int ld, const float* decay,
                          float* o, unsigned* status, cudaStream_t stream);
 int forge_retention_gate(int fp32, const float* o, const void* qkvg, int ld, int gate_at, void* y, int tok0, int tokens, int heads, int dv,
                          float eps, cudaStream_t stream);
-int forge_router(int fp32, const void* h, const void* w, int T, int W, int E, int top, int softmax, int* experts, float* weights,
-                 cudaStream_t stream);
+int forge_router(int fp32, const void* h, const void* w, int T, int W, int E, int top, int softmax, const float* correction, int groups, int keep,
+                 int* experts, float* weights, cudaStream_t stream);
 int forge_moe_plan(const int* experts, int n, int E, int tile, int max_tiles, int* pos, int* tile_expert, int* num_tiles, cudaStream_t stream);
 int forge_grouped_gemm(const void* x, const void* w, void* out, int experts, int n_out, int K, int gated, int tile, int act, float limit,
                        const int* tile_expert, const int* num_tiles, int max_tiles, unsigned* status, cudaStream_t stream);
@@ -48,15 +52,15 @@ int forge_head_linear(const void* x, long long x_tok, long long x_head, const vo
 int forge_latent_decode_ok(int R, int rot, int block_size);
 long long forge_latent_decode_scratch(int heads, int R, int ctas);
 int forge_latent_decode(const void* qa, const void* cache, const int* block_tables, const int* lens, void* o, float* scratch, int ctas,
-                        int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size, float scale, unsigned* status,
-                        cudaStream_t stream);
+                        int seqs, int heads, int R, int rot, int table_width, int num_blocks, int block_size, int window, float scale,
+                        unsigned* status, cudaStream_t stream);
 int forge_latent_prefill_qcols(int dim, int rot, int vdim);
 int forge_latent_prefill(const void* q, const void* kv, const void* kr, const int* cu_q, const int* cu_k, void* out, int tokens, int tok0,
-                         int keys, int num_seqs, int max_q, int heads, int dim, int rot, int vdim, float scale, unsigned* status,
+                         int keys, int num_seqs, int max_q, int heads, int dim, int rot, int vdim, int window, float scale, unsigned* status,
                          cudaStream_t stream);
-int forge_latent_gather(const void* cache, const int* cu_k, int num_seqs, const int* block_tables, int table_width, int num_blocks,
+int forge_latent_gather(const void* cache, const int* cu_k, const int* lens, int num_seqs, const int* block_tables, int table_width, int num_blocks,
                         int block_size, int R, int rot, int keys, void* c, void* kr, unsigned* status, cudaStream_t stream);
-int forge_latent_pack_q(const void* q, void* qp, int tokens, int heads, int dim, int rot, const float* rope, int rope_rows,
+int forge_latent_pack_q(const void* q, long long ld, void* qp, int tokens, int heads, int dim, int rot, const float* rope, int rope_rows,
                         const int* positions, cudaStream_t stream);
 int forge_retention_chunk_ok(int heads, int dk, int dv, int rd);
 int forge_retention_chunk_cols(int dk, int dv);
@@ -164,6 +168,59 @@ void stream_sandwich(Tensor& x, const OptTensor& a, const OptTensor& a_rows, con
            "forge_stream_sandwich");
 }
 
+// x fp32 [rows, W]; a or embed (with ids), post, w, h of one element type; the rest as in stream_sandwich.  Norms over `groups` equal parts of
+// a row; h without w: the row itself.
+void stream_group(Tensor& x, const OptTensor& a, const OptTensor& a_rows, const OptTensor& a_weights, const Tensor& post, double mult, double offset,
+                  const OptTensor& ids, const OptTensor& embed, const OptTensor& w, const OptTensor& h, const OptTensor& rows, int64_t groups, bool start,
+                  double eps, bool fp32) {
+  TORCH_CHECK(x.dim() == 2 && a.has_value() != ids.has_value() && groups >= 1 && x.size(1) % groups == 0, "stream_group: sizes and operands");
+  const int64_t R = x.size(0), W = x.size(1);
+  const auto dt = fp32 ? at::kFloat : at::kBFloat16;
+  float* xp = floats(x, R * W, "x");
+  const void *ap = nullptr, *ep = nullptr, *wp = nullptr;
+  void* hp = nullptr;
+  const int *arp = nullptr, *idp = nullptr, *rp = nullptr;
+  const float* awp = nullptr;
+  int64_t top = 0, vocab = 0, out_rows = R;
+  if (rows.has_value()) { rp = ints(*rows, 0, "rows"); out_rows = rows->numel(); }
+  if (a.has_value() && a_rows.has_value()) {
+    TORCH_CHECK(a_rows->dim() == 2 && a_rows->size(0) == R && a->dim() == 2 && a->size(1) == W, "stream_group: routed a");
+    top = a_rows->size(1);
+    arp = ints(*a_rows, R * top, "a_rows");
+    ap = data(*a, dt, W, "a");
+    if (a_weights.has_value()) awp = floats(*a_weights, R * top, "a_weights");
+  } else if (a.has_value()) {
+    ap = data(*a, dt, R * W, "a");
+  } else {
+    TORCH_CHECK(embed.has_value() && embed->dim() == 2 && embed->size(1) == W, "stream_group: embed");
+    idp = ints(*ids, R, "ids");
+    vocab = embed->size(0);
+    ep = data(*embed, dt, W, "embed");
+  }
+  if (w.has_value()) {
+    TORCH_CHECK(h.has_value(), "stream_group: h");
+    wp = data(*w, dt, W, "w");
+  }
+  if (h.has_value()) hp = data(*h, dt, out_rows * W, "h");
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_stream_group(fp32, xp, ap, arp, awp, i32(top), data(post, dt, W, "post"), static_cast<float>(mult), static_cast<float>(offset), idp, ep,
+                              i32(vocab), wp, hp, rp, i32(out_rows), i32(R), i32(W), i32(groups), start ? 1 : 0, static_cast<float>(eps), stream_of(x)),
+           "forge_stream_group");
+}
+
+// x <- act(x) in place
+void act_any(Tensor& x, int64_t act) {
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_act_any(elem(x), data(x, x.scalar_type(), 0, "x"), x.numel(), i32(act), 0, 1.f, 0.f, stream_of(x)), "forge_act_any");
+}
+
+// x <- cap tanh(scale x / cap) in place
+void bound_logits(Tensor& x, double scale, double cap) {
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_rc(forge_act_any(elem(x), data(x, x.scalar_type(), 0, "x"), x.numel(), 0, 1, static_cast<float>(scale), static_cast<float>(cap), stream_of(x)),
+           "forge_act_any");
+}
+
 // out = act(x w_gate^T, x w_up^T) for w = gate rows, up rows (bf16, tcgen05)
 void gemm_act(const Tensor& x, const Tensor& w, Tensor& out, int64_t act, double limit, const Tensor& status) {
   TORCH_CHECK(x.is_cuda() && w.is_cuda() && out.is_cuda() && x.scalar_type() == at::kBFloat16 && w.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16,
@@ -205,38 +262,42 @@ void gemm_simt(const Tensor& x, const Tensor& w, Tensor& out, const OptTensor& t
            "forge_gemm_simt");
 }
 
-void latent_prepare(const Tensor& proj, int64_t q_rank, int64_t kv_rank, const Tensor& qw, const Tensor& kw, double eps, const Tensor& rope,
-                    const Tensor& positions, const Tensor& slots, Tensor& cq, Tensor& cache, const Tensor& status) {
+// proj [tokens, >= q_rank + kv_rank + rot]; without qw the first q_rank columns are passed over and there is no cq
+void latent_prepare(const Tensor& proj, int64_t q_rank, int64_t kv_rank, const OptTensor& qw, const Tensor& kw, double eps, const Tensor& rope,
+                    const Tensor& positions, const Tensor& slots, const OptTensor& cq, Tensor& cache, const Tensor& status) {
   const int f = elem(proj);
   const auto dt = proj.scalar_type();
   TORCH_CHECK(proj.dim() == 2 && cache.dim() == 3 && rope.dim() == 2, "latent_prepare: ranks");
-  const int64_t T = proj.size(0), rot = proj.size(1) - q_rank - kv_rank;
-  TORCH_CHECK(q_rank > 0 && kv_rank > 0 && rot >= 0 && cache.size(2) == kv_rank + rot && rope.size(1) == rot, "latent_prepare: sizes");
+  const int64_t T = proj.size(0), rot = cache.size(2) - kv_rank;
+  TORCH_CHECK(q_rank > 0 && kv_rank > 0 && rot >= 0 && proj.size(1) >= q_rank + kv_rank + rot && rope.size(1) == rot && qw.has_value() == cq.has_value(),
+              "latent_prepare: sizes");
   const c10::cuda::CUDAGuard guard(proj.device());
-  check_rc(forge_latent_prepare(f, data(proj, dt, 0, "proj"), i32(T), i32(q_rank), i32(kv_rank), i32(rot), data(qw, dt, q_rank, "qw"),
+  check_rc(forge_latent_prepare(f, data(proj, dt, 0, "proj"), proj.size(1), i32(T), i32(q_rank), i32(kv_rank), i32(rot),
+                                qw.has_value() ? data(*qw, dt, q_rank, "qw") : nullptr,
                                 data(kw, dt, kv_rank, "kw"), static_cast<float>(eps), floats(rope, 0, "rope"), i32(rope.size(0)),
-                                ints(positions, T, "positions"), ints(slots, T, "slots"), data(cq, dt, T * q_rank, "cq"),
+                                ints(positions, T, "positions"), ints(slots, T, "slots"), cq.has_value() ? data(*cq, dt, T * q_rank, "cq") : nullptr,
                                 data(cache, dt, 0, "cache"), static_cast<long long>(cache.size(0)) * cache.size(1), status_word(status),
                                 stream_of(proj)),
            "forge_latent_prepare");
 }
 
-// q [tokens, heads * (dim + rot)] -> the rotated parts in qa [tokens, heads, kv_rank + rot]
+// q [tokens, heads * (dim + rot)] (a view) -> the rotated parts in qa [tokens, heads, kv_rank + rot]
 void latent_rotate_q(const Tensor& q, Tensor& qa, int64_t dim, int64_t kv_rank, const Tensor& rope, const Tensor& positions) {
   const int f = elem(q);
   TORCH_CHECK(q.dim() == 2 && qa.dim() == 3 && rope.dim() == 2, "latent_rotate_q: ranks");
   const int64_t T = q.size(0), H = qa.size(1), rot = rope.size(1);
   TORCH_CHECK(qa.size(0) == T && q.size(1) == H * (dim + rot) && qa.size(2) == kv_rank + rot, "latent_rotate_q: sizes");
   const c10::cuda::CUDAGuard guard(q.device());
-  check_rc(forge_latent_rotate_q(f, data(q, q.scalar_type(), 0, "q"), data(qa, q.scalar_type(), 0, "qa"), i32(T), i32(H), i32(dim), i32(rot),
+  check_rc(forge_latent_rotate_q(f, view2(q, q.scalar_type(), T, H * (dim + rot), "q"), q.stride(0), data(qa, q.scalar_type(), 0, "qa"), i32(T), i32(H), i32(dim), i32(rot),
                                  i32(kv_rank), floats(rope, 0, "rope"), i32(rope.size(0)), ints(positions, T, "positions"), stream_of(q)),
            "forge_latent_rotate_q");
 }
 
 // qa [tokens, heads, kv_rank + rot] = the step's tokens tok0 .. tok0 + tokens; o [tokens, heads, kv_rank]
 void latent_attend_any(const Tensor& qa, const Tensor& cache, Tensor& o, int64_t tok0, const Tensor& cu, int64_t num_seqs,
-                       const Tensor& positions, const Tensor& block_tables, double scale, const Tensor& status) {
+                       const Tensor& positions, const Tensor& block_tables, int64_t window, double scale, const Tensor& status) {
   const int f = elem(qa);
+  TORCH_CHECK(window >= 0, "latent_attend_any: window");
   TORCH_CHECK(qa.dim() == 3 && cache.dim() == 3 && o.dim() == 3 && block_tables.dim() == 2, "latent_attend_any: ranks");
   const int64_t T = qa.size(0), H = qa.size(1), R = o.size(2), D = qa.size(2);
   TORCH_CHECK(o.size(0) == T && o.size(1) == H && cache.size(2) == D && R <= D && block_tables.size(0) >= num_seqs, "latent_attend_any: sizes");
@@ -244,8 +305,8 @@ void latent_attend_any(const Tensor& qa, const Tensor& cache, Tensor& o, int64_t
   check_rc(forge_latent_attend_any(f, data(qa, qa.scalar_type(), 0, "qa"), data(cache, qa.scalar_type(), 0, "cache"),
                                    data(o, qa.scalar_type(), 0, "o"), i32(tok0), i32(T), ints(cu, num_seqs + 1, "cu_seqlens_q"), i32(num_seqs),
                                    ints(positions, tok0 + T, "positions"), ints(block_tables, 0, "block_tables"), i32(block_tables.size(1)),
-                                   i32(cache.size(0)), i32(cache.size(1)), i32(H), i32(R), i32(D - R), static_cast<float>(scale),
-                                   status_word(status), stream_of(qa)),
+                                   i32(cache.size(0)), i32(cache.size(1)), i32(H), i32(R), i32(D - R), i32(window),
+                                   static_cast<float>(scale), status_word(status), stream_of(qa)),
            "forge_latent_attend_any");
 }
 
@@ -297,13 +358,14 @@ void retention_gate(const Tensor& o, const Tensor& qkvg, Tensor& y, int64_t tok0
            "forge_retention_gate");
 }
 
-void router(const Tensor& h, const Tensor& w, Tensor& experts, Tensor& weights, bool softmax) {
+// correction fp32 [experts]; the experts of the `keep` best of `groups` groups can be chosen
+void router(const Tensor& h, const Tensor& w, Tensor& experts, Tensor& weights, bool softmax, const OptTensor& correction, int64_t groups, int64_t keep) {
   const int f = elem(h);
   TORCH_CHECK(h.dim() == 2 && w.dim() == 2 && w.size(1) == h.size(1) && experts.dim() == 2 && experts.size(0) == h.size(0), "router: shapes");
   const int64_t T = h.size(0), W = h.size(1), E = w.size(0), top = experts.size(1);
   const c10::cuda::CUDAGuard guard(h.device());
   check_rc(forge_router(f, data(h, h.scalar_type(), 0, "h"), data(w, h.scalar_type(), 0, "w"), i32(T), i32(W), i32(E), i32(top), softmax ? 1 : 0,
-                        const_cast<int*>(ints(experts, T * top, "experts")), floats(weights, T * top, "weights"), stream_of(h)),
+                        correction.has_value() ? floats(*correction, E, "correction") : nullptr, i32(groups), i32(keep), const_cast<int*>(ints(experts, T * top, "experts")), floats(weights, T * top, "weights"), stream_of(h)),
            "forge_router");
 }
 
@@ -357,7 +419,8 @@ void head_linear(const Tensor& x, const Tensor& w, Tensor& out) {
 
 // scratch: fp32, latent_decode_scratch(heads, R, ctas) elements
 void latent_decode(const Tensor& qa, const Tensor& cache, const Tensor& block_tables, const Tensor& lens, Tensor& o, Tensor& scratch, int64_t ctas,
-                   double scale, const Tensor& status) {
+                   int64_t window, double scale, const Tensor& status) {
+  TORCH_CHECK(window >= 0, "latent_decode: window");
   TORCH_CHECK(qa.dim() == 3 && cache.dim() == 3 && block_tables.dim() == 2 && o.dim() == 3, "latent_decode: ranks");
   const int64_t B = qa.size(0), H = qa.size(1), D = qa.size(2), R = o.size(2);
   TORCH_CHECK(cache.size(2) == D && R <= D && o.size(0) == B && o.size(1) == H && block_tables.size(0) >= B, "latent_decode: shapes");
@@ -365,17 +428,17 @@ void latent_decode(const Tensor& qa, const Tensor& cache, const Tensor& block_ta
   check_rc(forge_latent_decode(data(qa, kBf16, 0, "qa"), data(cache, kBf16, 0, "cache"), ints(block_tables, 0, "block_tables"), ints(lens, B, "lens"),
                                data(o, kBf16, 0, "o"), floats(scratch, forge_latent_decode_scratch(i32(H), i32(R), i32(ctas)), "scratch"), i32(ctas),
                                i32(B), i32(H), i32(R), i32(D - R), i32(block_tables.size(1)), i32(cache.size(0)), i32(cache.size(1)),
-                               static_cast<float>(scale), status_word(status), stream_of(qa)),
+                               i32(window), static_cast<float>(scale), status_word(status), stream_of(qa)),
            "forge_latent_decode");
 }
 
-// c [keys, R], kr [keys, rot] <- the cached rows of the sequences whose running key counts are cu_k
-void latent_gather(const Tensor& cache, const Tensor& cu_k, int64_t num_seqs, const Tensor& block_tables, Tensor& c, Tensor& kr, const Tensor& status) {
+// c [keys, R], kr [keys, rot] <- the cached rows of the sequences, of each the last cu_k[s + 1] - cu_k[s] of lens[s]; zeros after them
+void latent_gather(const Tensor& cache, const Tensor& cu_k, const Tensor& lens, int64_t num_seqs, const Tensor& block_tables, Tensor& c, Tensor& kr, const Tensor& status) {
   TORCH_CHECK(cache.dim() == 3 && block_tables.dim() == 2 && c.dim() == 2 && kr.dim() == 2, "latent_gather: ranks");
   const int64_t keys = c.size(0), R = c.size(1), rot = kr.size(1);
   TORCH_CHECK(kr.size(0) == keys && cache.size(2) == R + rot && block_tables.size(0) >= num_seqs, "latent_gather: shapes");
   const c10::cuda::CUDAGuard guard(cache.device());
-  check_rc(forge_latent_gather(data(cache, kBf16, 0, "cache"), ints(cu_k, num_seqs + 1, "cu_k"), i32(num_seqs), ints(block_tables, 0, "block_tables"),
+  check_rc(forge_latent_gather(data(cache, kBf16, 0, "cache"), ints(cu_k, num_seqs + 1, "cu_k"), ints(lens, num_seqs, "lens"), i32(num_seqs), ints(block_tables, 0, "block_tables"),
                                i32(block_tables.size(1)), i32(cache.size(0)), i32(cache.size(1)), i32(R), i32(rot), i32(keys),
                                data(c, kBf16, 0, "c"), data(kr, kBf16, 0, "kr"), status_word(status), stream_of(cache)),
            "forge_latent_gather");
@@ -387,14 +450,15 @@ void latent_pack_q(const Tensor& q, Tensor& qp, int64_t heads, int64_t dim, cons
   TORCH_CHECK(q.size(1) == heads * (dim + rot) && qp.size(0) == T && qp.size(1) == heads && qp.size(2) == 64 * ((dim + 63) / 64 + (rot + 63) / 64),
               "latent_pack_q: shapes");
   const c10::cuda::CUDAGuard guard(q.device());
-  check_rc(forge_latent_pack_q(data(q, kBf16, 0, "q"), data(qp, kBf16, 0, "qp"), i32(T), i32(heads), i32(dim), i32(rot), floats(rope, 0, "rope"),
+  check_rc(forge_latent_pack_q(view2(q, kBf16, T, heads * (dim + rot), "q"), q.stride(0), data(qp, kBf16, 0, "qp"), i32(T), i32(heads), i32(dim), i32(rot), floats(rope, 0, "rope"),
                                i32(rope.size(0)), ints(positions, T, "positions"), stream_of(q)),
            "forge_latent_pack_q");
 }
 
 // qp [tokens - tok0, heads, qcols], kv [keys, heads * (dim + vdim)], kr [keys, rot], out [tokens, heads * vdim]
 void latent_prefill(const Tensor& qp, const Tensor& kv, const Tensor& kr, const Tensor& cu_q, const Tensor& cu_k, Tensor& out, int64_t tok0,
-                    int64_t num_seqs, int64_t max_q, int64_t dim, int64_t vdim, double scale, const Tensor& status) {
+                    int64_t num_seqs, int64_t max_q, int64_t dim, int64_t vdim, int64_t window, double scale, const Tensor& status) {
+  TORCH_CHECK(window >= 0, "latent_prefill: window");
   TORCH_CHECK(qp.dim() == 3 && kv.dim() == 2 && kr.dim() == 2 && out.dim() == 2, "latent_prefill: ranks");
   const int64_t H = qp.size(1), T = out.size(0), keys = kv.size(0), rot = kr.size(1);
   TORCH_CHECK(qp.size(0) == T - tok0 && kv.size(1) == H * (dim + vdim) && kr.size(0) == keys && out.size(1) == H * vdim &&
@@ -403,7 +467,7 @@ void latent_prefill(const Tensor& qp, const Tensor& kv, const Tensor& kr, const 
   const c10::cuda::CUDAGuard guard(qp.device());
   check_rc(forge_latent_prefill(data(qp, kBf16, 0, "qp"), data(kv, kBf16, 0, "kv"), data(kr, kBf16, 0, "kr"), ints(cu_q, num_seqs + 1, "cu_q"),
                                 ints(cu_k, num_seqs + 1, "cu_k"), data(out, kBf16, 0, "out"), i32(T), i32(tok0), i32(keys), i32(num_seqs),
-                                i32(max_q), i32(H), i32(dim), i32(rot), i32(vdim), static_cast<float>(scale), status_word(status),
+                                i32(max_q), i32(H), i32(dim), i32(rot), i32(vdim), i32(window), static_cast<float>(scale), status_word(status),
                                 stream_of(qp)),
            "forge_latent_prefill");
 }
@@ -433,6 +497,9 @@ void retention_chunk(Tensor& qkvg, const Tensor& decay, Tensor& state, const Ten
 void register_mixers(pybind11::module& m) {
   m.def("stream_update", &stream_update);
   m.def("stream_sandwich", &stream_sandwich);
+  m.def("stream_group", &stream_group);
+  m.def("act_any", &act_any);
+  m.def("bound_logits", &bound_logits);
   m.def("gemm_act", &gemm_act);
   m.def("act_mul_any", &act_mul_any);
   m.def("gemm_simt", &gemm_simt);

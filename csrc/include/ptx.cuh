@@ -398,4 +398,17 @@ __device__ __forceinline__ float gated_act(int act, float limit, float g, float 
   return times_sigmoid<kAccurate>(g, 1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
 }
 
+// Activations of a feed-forward without gates.
+enum PlainAct { kPlainNone = 0, kPlainGelu = 1 };
+__device__ __forceinline__ float plain_act(int act, float u) { return act == kPlainGelu ? 0.5f * u * (1.f + erff(u * 0.70710678118654752f)) : u; }
+
+// cap tanh(scale x / cap), or scale x without a cap; accurate: fp32 logits (else to a few units in the last place of cap).
+template <bool kAccurate>
+__device__ __forceinline__ float bound_logit(float x, float scale, float cap) {
+  const float z = x * scale;
+  if (!(cap > 0.f)) return z;
+  if (kAccurate) return cap * tanhf(z / cap);
+  return fmaf(-2.f * cap, __fdividef(1.f, 1.f + __expf(2.f * z / cap)), cap);
+}
+
 }  // namespace forge

@@ -1,6 +1,6 @@
 // Expert GEMM on the 5th-generation tensor cores: rows sorted by expert (moe_plan), every tile of kTok rows has one expert.
 //
-//   plain   y[r, f]  = x[r, :] . w[e, f, :]                               (down)
+//   plain   y[r, f]  = act(x[r, :] . w[e, f, :])                          (down; up of experts without gates: PlainAct)
 //   gated   y[r, f]  = act(x[r, :] . w[e, f, :], x[r, :] . w[e, F + f, :])       (gate and up rows of one packed matrix; GateAct)
 //
 // With many rows the plain form takes two feature tiles per row tile, as the gated form does by nature: a tile of x is loaded
@@ -158,6 +158,13 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
           tcgen05_fence_before();
           __syncwarp();
           if (lane == 0) mbar_arrive(&acc_empty[b]);
+        }
+        if (!kGated && act != kPlainNone) {
+#pragma unroll
+          for (int j = 0; j < kChunk; ++j) {
+            g[j] = __float_as_uint(plain_act(act, __uint_as_float(g[j])));
+            if (kTwo) u[j] = __float_as_uint(plain_act(act, __uint_as_float(u[j])));
+          }
         }
         if (f < n_out) {
 #pragma unroll

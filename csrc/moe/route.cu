@@ -1,7 +1,8 @@
 // Mixture of experts: routing and the shuffling of rows.
 //
 //   router          logits (fp32) -> the `top` largest of a token (ties: the lower expert), weighted by the sigmoid of each or
-//                   by the softmax over the chosen ones
+//                   by the softmax over the chosen ones.  With sigmoids the choice may go by score + correction, and be limited to
+//                   the experts of the `keep` groups of neighbours whose two best experts are best together
 //   moe_plan        (token, choice) -> row of the expert-sorted buffer; every expert's rows start on a multiple of `tile`, so
 //                   a tile of rows has one expert (tile_expert; -1 past the last tile in use)
 //   moe_scatter     row = token, or weight * token (weight in fp32) where the weight multiplies the expert's INPUT
@@ -42,12 +43,58 @@ __device__ __forceinline__ void choose_top(float* score, int E, int top, bool so
     for (int j = lane; j < top; j += 32) weights[j] = expf(weights[j] - first) / sum;
 }
 
+// What the choice goes by beside the scores.
+struct RouterGroups {
+  const float* correction;  // [E]; null: none
+  int groups, keep;
+  __device__ __host__ bool plain() const { return correction == nullptr && groups == 1; }
+};
+
+// The same from choice[e] = score + correction within groups; score[e] is the weight, worth [groups] is scratch.  An expert's place is the
+// number of better ones, so every place is taken once (NaN counts as the smallest number).
+__device__ __forceinline__ void choose_grouped(float* choice, const float* score, float* worth, const RouterGroups& z, int E, int top, int lane,
+                                               int* experts, float* weights) {
+  constexpr float kLeast = -3.402823466e38f;
+  for (int e = lane; e < E; e += 32) choice[e] = fmaxf(score[e] + (z.correction != nullptr ? z.correction[e] : 0.f), kLeast);
+  __syncwarp();
+  if (z.groups > 1) {
+    const int size = E / z.groups;
+    for (int g = lane; g < z.groups; g += 32) {
+      float a = -INFINITY, b = -INFINITY;                 // the best and the second
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float v = choice[e];
+        b = fmaxf(b, fminf(a, v));
+        a = fmaxf(a, v);
+      }
+      worth[g] = size > 1 ? fmaxf(a + b, kLeast) : a;
+    }
+    __syncwarp();
+    for (int g = lane; g < z.groups; g += 32) {
+      int better = 0;
+      for (int i = 0; i < z.groups; ++i) better += worth[i] > worth[g] || (worth[i] == worth[g] && i < g);
+      if (better >= z.keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) choice[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  for (int e = lane; e < E; e += 32) {
+    const float v = choice[e];
+    if (v == -INFINITY) continue;
+    int better = 0;
+    for (int i = 0; i < E; ++i) better += choice[i] > v || (choice[i] == v && i < e);
+    if (better < top) {
+      experts[better] = e;
+      weights[better] = score[e];
+    }
+  }
+}
+
 // bf16, W a multiple of 32, E <= 256: CTA = 16 MT tokens, the eight warps split W.  The order of the columns in a dot product is
 // free, so a lane loads eight consecutive columns of its row (16 bytes) and uses them as the four column pairs of two mma
 // k-steps, for tokens and experts alike: no shared memory on the way in.  The warps' partial logits are added in a fixed order.
 template <int MT>
 __global__ void __launch_bounds__(256) router_mma_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w, int T, int W, int E, int top, bool softmax,
-                                                         int* __restrict__ experts, float* __restrict__ weights) {
+                                                         const RouterGroups groups, int* __restrict__ experts, float* __restrict__ weights) {
   extern __shared__ float sm_part[];               // [8][16 MT][Ep]
   constexpr int kTok = 16 * MT, kGroup = 8;        // 8-expert blocks per pass
   const int Ep = (E + 7) & ~7;
@@ -103,15 +150,20 @@ __global__ void __launch_bounds__(256) router_mma_kernel(const bf16* __restrict_
       score[e] = softmax ? z : 1.f / (1.f + expf(-z));
     }
     __syncwarp();
-    choose_top(score, E, top, softmax, lane, experts + static_cast<size_t>(t0 + t) * top, weights + static_cast<size_t>(t0 + t) * top);
+    int* chosen = experts + static_cast<size_t>(t0 + t) * top;
+    float* weigh = weights + static_cast<size_t>(t0 + t) * top;
+    if (groups.plain())
+      choose_top(score, E, top, softmax, lane, chosen, weigh);
+    else                                            // the token's other partial logits have been added up: their places are free
+      choose_grouped(score + static_cast<size_t>(kTok) * Ep, score, score + static_cast<size_t>(2 * kTok) * Ep, groups, E, top, lane, chosen, weigh);
   }
 }
 
 // CTA = one token; one warp per expert at a time.
 template <typename T, int N>
 __global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, const T* __restrict__ w, int W, int E, int top, bool softmax,
-                                                     int* __restrict__ experts, float* __restrict__ weights) {
-  extern __shared__ float score[];
+                                                     const RouterGroups groups, int* __restrict__ experts, float* __restrict__ weights) {
+  extern __shared__ float score[];                  // [E]; with groups or corrections [3][E]
   pdl_launch_dependents();
   pdl_wait();
   const size_t t = blockIdx.x;
@@ -132,23 +184,27 @@ __global__ void __launch_bounds__(256) router_kernel(const T* __restrict__ h, co
     if (lane == 0) score[e] = softmax ? z : 1.f / (1.f + expf(-z));
   }
   __syncthreads();
-  if (warp == 0) choose_top(score, E, top, softmax, lane, experts + t * top, weights + t * top);
+  if (warp != 0) return;
+  if (groups.plain()) choose_top(score, E, top, softmax, lane, experts + t * top, weights + t * top);
+  else choose_grouped(score + E, score, score + 2 * E, groups, E, top, lane, experts + t * top, weights + t * top);
 }
 
-extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int W, int E, int top, int softmax, int* experts, float* weights,
-                            cudaStream_t stream) {
+extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int W, int E, int top, int softmax, const float* correction,
+                            int num_groups, int keep, int* experts, float* weights, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (E > 4096 || top < 1 || top > E) return -1;
+  const RouterGroups groups = {correction, num_groups, keep};
+  if (num_groups < 1 || E % num_groups || keep < 1 || keep > num_groups || top > keep * (E / num_groups) || (softmax && !groups.plain())) return -1;
   const bool v4 = (W & 3) == 0;
-  const size_t smem = static_cast<size_t>(E) * 4;
+  const size_t smem = static_cast<size_t>(E) * 4 * (groups.plain() ? 1 : 3);      // at most 48 KB
   if (fp32) {
     auto k = v4 ? router_kernel<float, 4> : router_kernel<float, 1>;
-    return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
+    return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const float*>(h), static_cast<const float*>(w), W, E, top, softmax != 0, groups, experts, weights) == cudaSuccess ? 0 : -2;
   }
   const bool aligned = ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(w)) & 15) == 0;
   // a few tokens would occupy a few CTAs of the kernel below: one CTA per token spreads them
   if (T_ <= 128 && (W & 7) == 0 && aligned)
-    return launch_kernel(router_kernel<bf16, 8>, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
+    return launch_kernel(router_kernel<bf16, 8>, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, softmax != 0, groups, experts, weights) == cudaSuccess ? 0 : -2;
   if (W % 32 == 0 && E <= 256 && (reinterpret_cast<uintptr_t>(h) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
     const int Ep = (E + 7) & ~7;
     const bool two = T_ > 2048 && E <= 128;        // more tokens per CTA halve the reads of the router matrix
@@ -156,13 +212,13 @@ extern "C" int forge_router(int fp32, const void* h, const void* w, int T_, int 
     const size_t part = static_cast<size_t>(8) * (two ? 32 : 16) * Ep * 4;
     if (two) {
       FORGE_ENSURE_DYN_SMEM(router_mma_kernel<2>, 8 * 32 * 128 * 4);
-      return launch_kernel(router_mma_kernel<2>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
+      return launch_kernel(router_mma_kernel<2>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, softmax != 0, groups, experts, weights) == cudaSuccess ? 0 : -2;
     }
     FORGE_ENSURE_DYN_SMEM(router_mma_kernel<1>, 8 * 16 * 256 * 4);
-    return launch_kernel(router_mma_kernel<1>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
+    return launch_kernel(router_mma_kernel<1>, grid, dim3(256), part, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), T_, W, E, top, softmax != 0, groups, experts, weights) == cudaSuccess ? 0 : -2;
   }
   auto k = v4 ? router_kernel<bf16, 4> : router_kernel<bf16, 1>;
-  return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, softmax != 0, experts, weights) == cudaSuccess ? 0 : -2;
+  return launch_kernel(k, dim3(T_), dim3(256), smem, stream, 0, static_cast<const bf16*>(h), static_cast<const bf16*>(w), W, E, top, softmax != 0, groups, experts, weights) == cudaSuccess ? 0 : -2;
 }
 
 constexpr int kPlanThreads = 1024;

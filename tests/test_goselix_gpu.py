@@ -123,11 +123,11 @@ def test_vectorised_rotation_is_the_oracles():
 
 
 LATENT = {
-    "real": Spec(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5),
-    "groups": Spec(heads=20, dim=40, rot_dim=32, vdim=72, kv_rank=112, scale=0.13),
-    "small": Spec(heads=3, dim=24, rot_dim=16, vdim=40, kv_rank=48, scale=0.2),
-    "deep": Spec(heads=2, dim=192, rot_dim=64, vdim=128, kv_rank=256, scale=0.06),
-    "odd": Spec(heads=5, dim=9, rot_dim=6, vdim=7, kv_rank=13, scale=0.3),
+    "real": Spec(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, window=0),
+    "groups": Spec(heads=20, dim=40, rot_dim=32, vdim=72, kv_rank=112, scale=0.13, window=0),
+    "small": Spec(heads=3, dim=24, rot_dim=16, vdim=40, kv_rank=48, scale=0.2, window=0),
+    "deep": Spec(heads=2, dim=192, rot_dim=64, vdim=128, kv_rank=256, scale=0.06, window=0),
+    "odd": Spec(heads=5, dim=9, rot_dim=6, vdim=7, kv_rank=13, scale=0.3, window=0),
 }
 
 
@@ -304,7 +304,7 @@ def test_experts(ops, dtype, T, E, top, W, F):
 def test_equal_scores_choose_the_lower_expert(ops):
     h, router = torch.ones(3, 64, dtype=BF, device="cuda"), torch.ones(40, 64, dtype=BF, device="cuda")
     e, w = torch.empty(3, 4, dtype=torch.int32, device="cuda"), torch.empty(3, 4, device="cuda")
-    ops.C.router(h, router, e, w, False)
+    ops.C.router(h, router, e, w, False, None, 1, 1)
     assert e.tolist() == [[0, 1, 2, 3]] * 3
 
 

@@ -460,15 +460,20 @@ class CudaOps(MixerOps, HybridOps):
                 and weight.shape[1] % 8 == 0
                 and (weight.shape[0] + 127) // 128 >= 2 * self.num_sms)
 
-    def lm_head_sample_shard(self, hidden, weight, temperatures, header, vocab_start):
+    def bound_logits(self, logits, scale, softcap):
+        """softcap * tanh(scale * logits / softcap), in place (softcap 0: scale * logits)."""
+        self.C.bound_logits(logits, scale, softcap)
+        return logits
+
+    def lm_head_sample_shard(self, hidden, weight, temperatures, header, vocab_start, scale=1.0, softcap=0.0):
         """(ids int32 [rows], scores fp32 [rows]) of this vocab shard, sampled in the epilogue of the LM-head GEMM: the
-        ``[rows, vocab / tp]`` logits are never written.  Same tokens as ``linear`` + ``sample_shard``."""
+        ``[rows, vocab / tp]`` logits are never written.  Same tokens as ``linear`` (+ ``bound_logits``) + ``sample_shard``."""
         rows, tiles = hidden.shape[0], (weight.shape[0] + 255) // 256
         part_v = torch.empty(rows * tiles, dtype=torch.float32, device=hidden.device)
         part_i = torch.empty(rows * tiles, dtype=torch.int32, device=hidden.device)
         ids = torch.empty(rows, dtype=torch.int32, device=hidden.device)
         best = torch.empty(rows, dtype=torch.float32, device=hidden.device)
-        self.C.gemm_sample(hidden, weight, vocab_start, temperatures, header, part_v, part_i, ids, best, self.status)
+        self.C.gemm_sample(hidden, weight, vocab_start, temperatures, header, part_v, part_i, ids, best, scale, softcap, self.status)
         return ids, best
 
     def sample(self, logits, batch, vocab_start, tp):

@@ -30,41 +30,64 @@ class HybridOps:
         self.C.bias_rope_store(proj, bias, table, positions, slot_mapping, q, k_cache, v_cache, self.status)
         return q
 
-    def norm_rope_store(self, proj, q_norm, k_norm, eps, spec, table, positions, slot_mapping, k_cache, v_cache):
-        """q [T, heads, columns]: the columns from ``dim`` on are zero."""
+    def norm_rope_store(self, proj, q_norm, k_norm, eps, spec, table, positions, slot_mapping, k_cache, v_cache, temper=None):
+        """q [T, heads, columns]: the columns from ``dim`` on are zero.  Without ``k_norm`` proj is q alone."""
+        if k_norm is None:
+            proj = proj[:, :spec.heads * spec.dim]
         cols = self.C.windowed_prefill_qcols(spec.dim, spec.vdim, k_cache.shape[2]) if proj.dtype == torch.bfloat16 else 0
         q = torch.empty(proj.shape[0], spec.heads, cols or spec.dim, dtype=proj.dtype, device=proj.device)
-        self.C.norm_rope_store(proj, q_norm, k_norm, spec.norm == "all", eps, table, positions, slot_mapping, q, k_cache, v_cache, self.status)
+        self.C.norm_rope_store(proj, q_norm, k_norm, spec.norm == "all", eps, table, positions, slot_mapping, q, k_cache, v_cache, temper, self.status)
         return q
 
-    def windowed_attention(self, q, k_cache, v_cache, batch, spec, out, scale, chunked=False, softcap=0.0, sink=None, gate=None) -> None:
-        """out (a view [T, heads * vdim]) <- scale * attention over the last ``spec.window`` tokens, or inside chunks of that many."""
+    def windowed_attention(self, q, k_cache, v_cache, batch, spec, out, scale, chunked=False, softcap=0.0, sink=None, gate=None, pool=None) -> None:
+        """out (a view [T, heads * vdim]) <- scale * attention over the last ``spec.window`` tokens, or inside chunks of that many.  ``pool`` (a
+        ``PooledCache``): with the means of the blocks behind the window; blocks that end in this step get theirs."""
         d, dv, bs = spec.dim, spec.vdim, k_cache.shape[2]
         bf16, seqs = q.dtype == torch.bfloat16, batch.padded_seqs
-        options = (spec.window, spec.scale, scale, chunked, softcap, sink, gate, self.status)
+        options = (spec.window, spec.scale, scale, chunked, softcap, sink, gate)
+        size = 0 if pool is None else pool.size
+        means = (None, None, 0) if pool is None else (pool.k, pool.v, size)
         n1 = self._singles(batch)
         if n1 and bf16 and self.C.windowed_decode_ok(d, dv, bs):
-            chunk, chunks = self.windowed_chunks(n1, spec, batch.table_width * bs)
+            chunk, chunks = self.windowed_chunks(n1, spec, batch.table_width * bs, size)
             part_o = part_ml = None
             if chunks > 1:
                 part_o = torch.empty(n1 * spec.heads * chunks * dv, dtype=torch.float32, device=q.device)
                 part_ml = torch.empty(n1 * spec.heads * chunks * 2, dtype=torch.float32, device=q.device)
-            self.C.windowed_decode(q, k_cache, v_cache, batch.block_tables, batch.context_lens, n1, out, part_o, part_ml, chunk, chunks, *options)
+            self.C.windowed_decode(q, k_cache, v_cache, batch.block_tables, batch.context_lens, n1, out, part_o, part_ml, chunk, chunks, *options,
+                                   *means, pool is not None and pool.own, self.status)
         else:
             n1 = 0
         if seqs == n1:
             return
-        cu, tables = batch.cu_seqlens_q[n1:], batch.block_tables[n1:]
+        cu, tables, lens = batch.cu_seqlens_q[n1:], batch.block_tables[n1:], batch.context_lens[n1:]
         rows = (out,) if gate is None or gate.shape[1] == spec.heads else (out, gate)
         if bf16 and spec.scale > 0 and batch.is_prefill and q.shape[2] == self.C.windowed_prefill_qcols(d, dv, bs) and _aligned(*rows):
-            self.C.windowed_prefill(q, k_cache, v_cache, cu, batch.context_lens[n1:], tables, seqs - n1, batch.max_seqlen_q, out, *options)
+            gathered = self.pool_blocks(k_cache, v_cache, pool, batch, n1, cu, lens, tables, spec.window)
+            self.C.windowed_prefill(q, k_cache, v_cache, cu, lens, tables, seqs - n1, batch.max_seqlen_q, out, *options, *gathered, self.status)
         else:
-            self.C.windowed_attend_any(q, k_cache, v_cache, cu, seqs - n1, batch.max_seqlen_q, batch.positions, tables, out, *options)
+            self.pool_blocks(k_cache, v_cache, pool, batch, n1, cu, lens, tables)
+            self.C.windowed_attend_any(q, k_cache, v_cache, cu, seqs - n1, batch.max_seqlen_q, batch.positions, tables, out, *options, *means, self.status)
 
-    def windowed_chunks(self, seqs: int, spec, capacity: int) -> tuple[int, int]:
-        """(keys per chunk, chunks): the window is cut until the two CTAs that an SM holds are busy.  Depends only on shapes known at
-        graph-capture time."""
-        span = min(spec.window, capacity) + 15
+    def pool_blocks(self, k_cache, v_cache, pool, batch, n1, cu, lens, tables, window=None):
+        """The means of the blocks that end in the step's tokens, for the sequences from ``n1`` on; with ``window`` all their entries one after
+        another for a kernel whose tiles cannot gather them: (keys, values, first rows, size), or nothing where no token sees a block."""
+        if pool is None:
+            return None, None, None, 0
+        seqs, gather = batch.padded_seqs - n1, window is not None and batch.max_seqlen_k - window >= pool.size
+        offsets = gk = gv = None
+        if gather:
+            offsets = self.row_offsets(batch, n1, size=pool.size)
+            keys = batch.kv_rows if n1 == batch.num_single else seqs * batch.max_seqlen_k
+            gk, gv = (torch.empty(keys // pool.size, k_cache.shape[1], c.shape[3], dtype=k_cache.dtype, device=k_cache.device) for c in (k_cache, v_cache))
+        self.C.pool_blocks(k_cache, v_cache, pool.k, pool.v, pool.size, pool.own, cu, lens, tables, seqs, batch.max_seqlen_q, batch.max_seqlen_k,
+                           offsets, gk, gv, self.status)
+        return gk, gv, offsets, pool.size if gather else 0
+
+    def windowed_chunks(self, seqs: int, spec, capacity: int, pool: int = 0) -> tuple[int, int]:
+        """(keys per chunk, chunks): the window, and the pooled blocks ahead of it, are cut until the two CTAs that an SM holds are busy.
+        Depends only on shapes known at graph-capture time."""
+        span = min(spec.window, capacity) + 15 + (capacity // pool + 15 if pool else 0)
         ctas = seqs * spec.kv_heads * -(-(spec.heads // spec.kv_heads) // 16)
         parts = max(1, min(2 * self.num_sms // ctas, span // 128))
         chunk = -(-(-(-span // parts)) // 64) * 64

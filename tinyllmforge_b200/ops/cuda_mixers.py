@@ -17,6 +17,7 @@ class Routed:
 
 
 ACTS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
+PLAIN_ACTS = {"gelu": 1}                        # of feed-forwards without gates
 
 
 class MixerOps:
@@ -24,9 +25,18 @@ class MixerOps:
 
     # ------------------------------------------------------------------ residual stream
     def stream_update(self, x, dtype, eps, norms, start=False, a=None, b=None, ids=None, embed=None, vec=None, rows=None,
-                      a_bias=None, post=None, mult=1.0, offset=0.0):
+                      a_bias=None, post=None, mult=1.0, offset=0.0, groups=1):
         n = x.shape[0] if rows is None else rows.shape[0]
         outs = [torch.empty(n, x.shape[1], dtype=dtype, device=x.device) for _ in norms]
+        if groups > 1 or None in norms or (a is None and post is not None):
+            if b is not None or vec is not None or a_bias is not None or post is None or len(norms) > 1 or (a is not None and ids is not None):
+                raise ValueError("stream_update: grouped norms go with one branch, normed on its way in, and one result")
+            a_rows = a_weights = None
+            if isinstance(a, Routed):
+                a, a_rows, a_weights = a.y, a.rows, a.weights
+            self.C.stream_group(x, a, a_rows, a_weights, post, mult, offset, ids, embed, norms[0] if norms else None, outs[0] if outs else None, rows,
+                                groups, start, eps, dtype == torch.float32)
+            return outs
         if post is not None or offset or isinstance(a, Routed):
             if b is not None or vec is not None or len(norms) > 1:
                 raise ValueError("stream_update: one branch and one norm where a is normed or norm weights have an offset")
@@ -90,7 +100,7 @@ class MixerOps:
 
     # ------------------------------------------------------------------ latent attention
     def latent_prepare(self, proj, q_rank, kv_rank, q_norm, kv_norm, eps, table, positions, slot_mapping, cache):
-        cq = torch.empty(proj.shape[0], q_rank, dtype=proj.dtype, device=proj.device)
+        cq = None if q_norm is None else torch.empty(proj.shape[0], q_rank, dtype=proj.dtype, device=proj.device)
         self.C.latent_prepare(proj, q_rank, kv_rank, q_norm, kv_norm, eps, table, positions, slot_mapping, cq, cache, self.status)
         return cq
 
@@ -118,28 +128,40 @@ class MixerOps:
         singles = n == (batch.num_single if batch.is_prefill else batch.padded_seqs)
         if singles and q.dtype == torch.bfloat16 and n <= 1024 and self.C.latent_decode_ok(R, r, cache.shape[1]):
             scratch = torch.empty(self.C.latent_decode_scratch(H, R, self.num_sms), dtype=torch.float32, device=q.device)
-            self.C.latent_decode(qa, cache, batch.block_tables, batch.context_lens, o, scratch, self.num_sms, spec.scale, self.status)
+            self.C.latent_decode(qa, cache, batch.block_tables, batch.context_lens, o, scratch, self.num_sms, spec.window, spec.scale, self.status)
         else:
             self.C.latent_attend_any(qa, cache, o, 0, batch.cu_seqlens_q, batch.padded_seqs, batch.positions, batch.block_tables,
-                                     spec.scale, self.status)
+                                     spec.window, spec.scale, self.status)
         self.head_linear(o, weights.uv, out[:n].view(n, H, dv))
 
     def _latent_expanded(self, q, weights, cache, batch, table, spec, out, n1) -> bool:
         """The sequences from ``n1`` on (their tokens start at row n1).  False: these sizes have no kernel, nothing was done."""
         H, d, r, dv, R = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
         qcols = self.C.latent_prefill_qcols(d, r, dv)
-        if q.dtype != torch.bfloat16 or qcols == 0 or R % 8:
+        if q.dtype != torch.bfloat16 or qcols == 0 or R % 8 or q.stride(0) % 8 or q.data_ptr() % 16:
             return False
         T, seqs, keys = q.shape[0], batch.num_seqs - n1, batch.kv_rows
-        cu_q, cu_k, tables = batch.cu_seqlens_q[n1:], batch.cu_seqlens_k[n1:], batch.block_tables[n1:]
+        cu_q, cu_k, tables, lens = batch.cu_seqlens_q[n1:], batch.cu_seqlens_k[n1:], batch.block_tables[n1:], batch.context_lens[n1:]
+        if spec.window:                              # the keys that some query of the step sees, and no others
+            cu_k, keys = self.row_offsets(batch, n1, window=spec.window), min(keys, T - n1 + seqs * (spec.window - 1))
         c = torch.empty(keys, R, dtype=q.dtype, device=q.device)
         kr = torch.empty(keys, r, dtype=q.dtype, device=q.device)
-        self.C.latent_gather(cache, cu_k, seqs, tables, c, kr, self.status)
+        self.C.latent_gather(cache, cu_k, lens, seqs, tables, c, kr, self.status)
         kv = self.linear(c, weights.ukv)
         qp = torch.empty(T - n1, H, qcols, dtype=q.dtype, device=q.device)
         self.C.latent_pack_q(q[n1:], qp, H, d, table, batch.positions[n1:])
-        self.C.latent_prefill(qp, kv, kr, cu_q, cu_k, out, n1, seqs, batch.max_seqlen_q, d, dv, spec.scale, self.status)
+        self.C.latent_prefill(qp, kv, kr, cu_q, cu_k, out, n1, seqs, batch.max_seqlen_q, d, dv, spec.window, spec.scale, self.status)
         return True
+
+    def row_offsets(self, batch, n1: int, window: int = 0, size: int = 0) -> torch.Tensor:
+        """Where the rows of the sequences from ``n1`` on begin in a buffer that holds, of each, its last min(keys, queries + window - 1) keys or
+        its floor(keys / size) blocks.  The layers of a step share it."""
+        known = batch.__dict__.setdefault("_row_offsets", {})
+        if (n1, window, size) not in known:
+            seqs = batch.padded_seqs - n1
+            out = known[n1, window, size] = torch.empty(seqs + 1, dtype=torch.int32, device=self.device)
+            self.C.row_offsets(batch.cu_seqlens_q[n1:], batch.context_lens[n1:], seqs, window, size, out)
+        return known[n1, window, size]
 
     # ------------------------------------------------------------------ retention
     def retention(self, qkvg, decay, state, batch, table, spec, eps):
@@ -177,12 +199,12 @@ class MixerOps:
         """Rows per tile of the tensor-core kernel (16 to 128): about what an expert gets."""
         return next((t for t in (16, 32, 64) if rows <= t * experts), 128)
 
-    def moe(self, h, router, gate_up, down, top, score="sigmoid", weigh="input", act="silu", limit=0.0):
+    def moe(self, h, router, up, down, top, score="sigmoid", weigh="input", act="silu", limit=0.0, gated=True, correction=None, groups=1, keep=1):
         T, W = h.shape
         E, n = router.shape[0], T * top
         experts = torch.empty(T, top, dtype=torch.int32, device=h.device)
         weights = torch.empty(T, top, dtype=torch.float32, device=h.device)
-        self.C.router(h, router, experts, weights, score == "softmax")
+        self.C.router(h, router, experts, weights, score == "softmax", correction, groups, keep)
         fast = h.dtype == torch.bfloat16 and W % 8 == 0 and down.shape[2] % 8 == 0
         tile = self.expert_tile(n, E) if fast else 64
         tiles = min(n, n // tile + E)
@@ -195,10 +217,14 @@ class MixerOps:
         y = torch.empty(tiles * tile, W, dtype=h.dtype, device=h.device)
         if fast:
             g = torch.empty(tiles * tile, down.shape[2], dtype=h.dtype, device=h.device)
-            self.C.grouped_gemm(xs, gate_up, g, True, tile, tile_expert, num_tiles, ACTS[act], limit, self.status)
+            self.C.grouped_gemm(xs, up, g, gated, tile, tile_expert, num_tiles, (ACTS if gated else PLAIN_ACTS)[act], limit, self.status)
             self.C.grouped_gemm(g, down, y, False, tile, tile_expert, num_tiles, 0, 0.0, self.status)
         else:
-            gu = torch.empty(tiles * tile, gate_up.shape[1], dtype=h.dtype, device=h.device)
-            self.C.gemm_simt(xs, gate_up, gu, tile_expert)
-            self.C.gemm_simt(self.act_mul_any(gu, act, limit), down, y, tile_expert)
+            g = torch.empty(tiles * tile, up.shape[1], dtype=h.dtype, device=h.device)
+            self.C.gemm_simt(xs, up, g, tile_expert)
+            if gated:
+                g = self.act_mul_any(g, act, limit)
+            else:
+                self.C.act_any(g, PLAIN_ACTS[act])
+            self.C.gemm_simt(g, down, y, tile_expert)
         return Routed(y, rows, weights if weigh == "output" else None)

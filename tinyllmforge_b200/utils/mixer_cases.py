@@ -15,7 +15,7 @@ class Spec:
         self.__dict__.update(kw)
 
 
-LATENT = Spec(heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, scale=192 ** -0.5)
+LATENT = Spec(heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, scale=192 ** -0.5, window=0)
 RETENTION = Spec(heads=8, dim=128, vdim=256)
 WIDTH, EXPERTS, TOP, FF = 2048, 32, 4, 1536
 
@@ -85,8 +85,8 @@ def _experts(ops, T, part):
     experts = torch.empty(T, TOP, dtype=torch.int32, device="cuda")
     weights = torch.empty(T, TOP, device="cuda")
     if part == "router":
-        return lambda: ops.C.router(h, router, experts, weights, False), T * WIDTH * 2, 2 * T * WIDTH * EXPERTS
-    ops.C.router(h, router, experts, weights, False)
+        return lambda: ops.C.router(h, router, experts, weights, False, None, 1, 1), T * WIDTH * 2, 2 * T * WIDTH * EXPERTS
+    ops.C.router(h, router, experts, weights, False, None, 1, 1)
     n = T * TOP
     tile = ops.expert_tile(n, EXPERTS)
     tiles = min(n, n // tile + EXPERTS)
