@@ -17,7 +17,7 @@ bench.py:54-56).  Metric: output tokens per second = K * sum(max_tokens) / time.
 * ``extras``: the same workload on the Qwen3-8B architecture at the same N (2 passes after 1 warm-up, in a child
   process before the headline run) and, at N = 8, the prefix-cache and the decode-heavy 32B workloads.
 
-``--design goselix|tonapel|mezapel`` runs something else instead: see tinyllmforge_b200/utils/design_bench.py.
+``--design goselix|tonapel|mezapel|galupel`` runs something else instead: see tinyllmforge_b200/utils/design_bench.py.
 
 With N > 1 (launched by torchrun, one rank per GPU) the model runs tensor-parallel over the N GPUs.
 ``--impl reference`` runs the unmodified reference engine from ``baseline/_ref`` on the same workload.
@@ -504,7 +504,7 @@ def main():
     ap.add_argument("--extras-timeout", type=float, default=600.0, help="most seconds one extra workload's child process gets")
     ap.add_argument("--time-budget", type=float, default=800.0,
                     help="seconds the whole run should fit in: the extra workloads get what the headline's estimated time leaves")
-    ap.add_argument("--design", default=None, choices=["goselix", "tonapel", "mezapel"],
+    ap.add_argument("--design", default=None, choices=["goselix", "tonapel", "mezapel", "galupel"],
                     help="instead of the headline workload: prefill and decode of a few layers of this design beside the closest other models at equal size")
     args = ap.parse_args()
     if args.design:

@@ -403,7 +403,7 @@ __global__ void __launch_bounds__(256) act_any_kernel(T* __restrict__ x, long lo
   pdl_wait();
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const float v = load_f(x + i);
-    store_f(x + i, logits ? bound_logit<sizeof(T) == 4>(v, scale, cap) : plain_act(act, v));
+    store_f(x + i, logits ? bound_logit<sizeof(T) == 4>(v, scale, cap) : plain_act<sizeof(T) == 4>(act, v));
   }
 }
 

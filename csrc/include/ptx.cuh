@@ -398,9 +398,29 @@ __device__ __forceinline__ float gated_act(int act, float limit, float g, float 
   return times_sigmoid<kAccurate>(g, 1.702f * g) * (fminf(fmaxf(u, -limit), limit) + 1.f);
 }
 
+// u Phi(u), Phi the normal distribution.  Not accurate (bf16 results): erfc(z) = (a1 t + .. + a5 t^5) exp(-z^2), t = 1 / (1 + p z), for z >= 0,
+// Abramowitz and Stegun, Handbook of Mathematical Functions, 7.1.26 (within 1.5e-7).
+template <bool kAccurate>
+__device__ __forceinline__ float gelu_erf(float u) {
+  const float z = fabsf(u) * 0.70710678118654752f;
+  if constexpr (kAccurate) {
+    const float tail = 0.5f * u * erfcf(z);
+    return u > 0.f ? u - tail : tail;
+  } else {
+    const float t = __fdividef(1.f, fmaf(0.3275911f, z, 1.f));
+    float y = fmaf(1.061405429f, t, -1.453152027f);
+    y = fmaf(y, t, 1.421413741f);
+    y = fmaf(y, t, -0.284496736f);
+    y = fmaf(y, t, 0.254829592f);
+    const float tail = 0.5f * u * (y * t) * __expf(-z * z);
+    return u > 0.f ? u - tail : tail;
+  }
+}
+
 // Activations of a feed-forward without gates.
 enum PlainAct { kPlainNone = 0, kPlainGelu = 1 };
-__device__ __forceinline__ float plain_act(int act, float u) { return act == kPlainGelu ? 0.5f * u * (1.f + erff(u * 0.70710678118654752f)) : u; }
+template <bool kAccurate>
+__device__ __forceinline__ float plain_act(int act, float u) { return act == kPlainGelu ? gelu_erf<kAccurate>(u) : u; }
 
 // cap tanh(scale x / cap), or scale x without a cap; accurate: fp32 logits (else to a few units in the last place of cap).
 template <bool kAccurate>

@@ -162,8 +162,8 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
         if (!kGated && act != kPlainNone) {
 #pragma unroll
           for (int j = 0; j < kChunk; ++j) {
-            g[j] = __float_as_uint(plain_act(act, __uint_as_float(g[j])));
-            if (kTwo) u[j] = __float_as_uint(plain_act(act, __uint_as_float(u[j])));
+            g[j] = __float_as_uint(plain_act<false>(act, __uint_as_float(g[j])));
+            if (kTwo) u[j] = __float_as_uint(plain_act<false>(act, __uint_as_float(u[j])));
           }
         }
         if (f < n_out) {

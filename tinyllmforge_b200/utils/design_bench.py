@@ -1,7 +1,7 @@
 """Prefill and decode throughput of a design beside others at equal width, head size, feed-forward work and number of layers:
-Goselix beside Qwen3, Tonapel beside Goselix and Qwen3, Mezapel beside Tonapel and Qwen3.
+Goselix beside Qwen3, Tonapel beside Goselix and Qwen3, Mezapel beside Tonapel and Qwen3, Galupel beside Goselix, Mezapel and Qwen3.
 
-    python bench.py --design goselix|tonapel|mezapel [--steps K] [--warmup W]
+    python bench.py --design goselix|tonapel|mezapel|galupel [--steps K] [--warmup W]
 
 A few layers of each (random weights, bf16), through the engine's own step: packed step buffer, model, sampling, CUDA graph for
 decode steps.  Device time per step (CUDA events); ahead of every timed step a buffer larger than L2 is written.  One JSON line
@@ -20,13 +20,13 @@ WORKLOADS = [("prefill", 8, 1024), ("prefill", 1, 8192), ("decode", 64, 1024), (
 
 def _configs(design: str, width: int):
     from ..config import ModelConfig
-    from ..models import goselix_config, mezapel_config, tonapel_config
+    from ..models import galupel_config, goselix_config, mezapel_config, tonapel_config
     heads = max(8, width // 128)
     qwen = ModelConfig(hidden_size=width, num_hidden_layers=LAYERS, num_attention_heads=heads, num_key_value_heads=max(2, heads // 2) if width < 4096 else 8,
                        head_dim=128, intermediate_size=3 * width, vocab_size=VOCAB, tie_word_embeddings=False)
     known = {"goselix": (goselix_config.GoselixConfig, goselix_config.example_dict), "tonapel": (tonapel_config.TonapelConfig, tonapel_config.example_dict),
-             "mezapel": (mezapel_config.MezapelConfig, mezapel_config.example_dict)}
-    order = {"goselix": ["goselix"], "tonapel": ["tonapel", "goselix"], "mezapel": ["mezapel", "tonapel"]}[design]
+             "mezapel": (mezapel_config.MezapelConfig, mezapel_config.example_dict), "galupel": (galupel_config.GalupelConfig, galupel_config.example_dict)}
+    order = {"goselix": ["goselix"], "tonapel": ["tonapel", "goselix"], "mezapel": ["mezapel", "tonapel"], "galupel": ["galupel", "goselix", "mezapel"]}[design]
     return [(name, known[name][0].from_dict(known[name][1](width, LAYERS, VOCAB))) for name in order] + [("qwen3", qwen)]
 
 

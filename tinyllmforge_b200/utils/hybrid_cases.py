@@ -24,14 +24,16 @@ class _Batch:
         self.slot_mapping = _ints(list(range(seqs * q_len)))
         self.state_slots = _ints(list(range(seqs)))
         self.table_width, self.max_seqlen_q, self.num_blocks = n, q_len, seqs * n
+        self.max_seqlen_k, self.kv_rows = ctx, seqs * ctx
 
 
 def _caches(b, s, block=256):
     return _rand(b.num_blocks, s.kv_heads, block, s.dim), _rand(b.num_blocks, s.kv_heads, block, s.vdim)
 
 
-def _attention(ops, seqs, q_len, ctx, window=None, heads=16, kind=None):
-    """``kind``: None, "chunked" (chunks, sink, a gate per head) or "capped" (window, sink, bounded scores, a gate per element)."""
+def _attention(ops, seqs, q_len, ctx, window=None, heads=16, kind=None, pool=0):
+    """``kind``: None, "chunked" (chunks, sink, a gate per head) or "capped" (window, sink, bounded scores, a gate per element).  ``pool``:
+    blocks of that many tokens behind the window, whose means exist for all but the step's tokens."""
     s = Spec(**{**ATTENTION.__dict__, "heads": heads, "window": window or ATTENTION.window})
     b = _Batch(seqs, q_len, ctx)
     kc, vc = _caches(b, s)
@@ -40,6 +42,12 @@ def _attention(ops, seqs, q_len, ctx, window=None, heads=16, kind=None):
     keys = sum(p + 1 - oldest(p) for p in range(ctx - q_len, ctx)) * seqs               # (query, key) pairs per head
     cached = seqs * (ctx - oldest(ctx - q_len)) * s.kv_heads * (s.dim + s.vdim) * 2
     options, gates = {}, 0
+    if pool:
+        from ..models.attention_blocks import PooledCache
+        pk, pv = (torch.zeros(b.num_blocks, s.kv_heads, PooledCache.rows(256, pool), c.shape[3], dtype=BF, device="cuda") for c in (kc, vc))
+        options = dict(pool=PooledCache(pool, pk, pv))
+        keys += sum(oldest(p) // pool for p in range(ctx - q_len, ctx)) * seqs
+        cached += seqs * (oldest(ctx - 1) // pool + (q_len // pool if q_len > 1 else 0)) * s.kv_heads * (s.dim + s.vdim) * 2
     if kind is not None:
         gates = {"chunked": s.heads, "capped": s.heads * s.vdim}[kind]
         options = dict(chunked=kind == "chunked", softcap=50.0 if kind == "capped" else 0.0, sink=torch.zeros(s.heads, device="cuda"), gate=_rand(seqs * q_len, gates))
@@ -124,6 +132,23 @@ def _sandwich(ops, T, routed):
     return lambda: ops.stream_update(x, BF, 1e-6, [w], a=y, post=w, mult=0.5, offset=1.0), (10 + 2 * TOP) * T * W, 0
 
 
+def _pool_blocks(ops, seqs, q_len, pool):
+    from ..models.attention_blocks import PooledCache
+    s, b = ATTENTION, _Batch(seqs, q_len, q_len)
+    kc, vc = _caches(b, s)
+    pk, pv = (torch.zeros(b.num_blocks, s.kv_heads, PooledCache.rows(256, pool), c.shape[3], dtype=BF, device="cuda") for c in (kc, vc))
+    p, n = PooledCache(pool, pk, pv), s.kv_heads * (s.dim + s.vdim) * 2
+    return (lambda: ops.pool_blocks(kc, vc, p, b, 0, b.cu_seqlens_q, b.context_lens, b.block_tables, s.window),
+            seqs * (q_len * n + q_len // pool * 2 * n), 0)
+
+
+def _grouped(ops, T, routed):
+    from ..ops.cuda_mixers import Routed
+    x, w, W, top = torch.randn(T, WIDTH, device="cuda"), _rand(WIDTH), WIDTH, 8
+    y = Routed(_rand(T * top, W), torch.randperm(T * top, dtype=torch.int32).view(T, top).cuda(), torch.rand(T, top, device="cuda")) if routed else _rand(T, W)
+    return lambda: ops.stream_update(x, BF, 1e-6, [None], a=y, post=w, groups=4), (10 + 2 * (top if routed else 1)) * T * W, 0
+
+
 def _gelu_product(ops, M):
     ws = [_rand(6 * WIDTH, WIDTH, scale=0.02) for _ in range(3)]
     x, state = _rand(M, WIDTH), {"i": 0}
@@ -157,6 +182,14 @@ CASES = {
     "chunked_prefill_long": lambda ops: _attention(ops, 1, 8192, 8192, 4096, kind="chunked"),
     "capped_prefill": lambda ops: _attention(ops, 8, 2048, 2048, kind="capped"),
     "capped_prefill_long": lambda ops: _attention(ops, 1, 8192, 8192, kind="capped"),
+    "pooled_decode": lambda ops: _attention(ops, 64, 1, 4096, pool=16),
+    "pooled_decode_b256": lambda ops: _attention(ops, 256, 1, 3000, pool=16),
+    "pooled_decode_b8": lambda ops: _attention(ops, 8, 1, 32768, pool=8),
+    "pooled_prefill": lambda ops: _attention(ops, 8, 2048, 2048, pool=16),
+    "pooled_prefill_long": lambda ops: _attention(ops, 1, 8192, 8192, pool=16),
+    "pool_blocks": lambda ops: _pool_blocks(ops, 8, 16384, 16),
+    "grouped_norm": lambda ops: _grouped(ops, 16384, False),
+    "grouped_norm_routed": lambda ops: _grouped(ops, 16384, True),
     "norm_rope_heads": lambda ops: _norm_rope_store(ops, 16384, False, 128),
     "norm_rope_whole": lambda ops: _norm_rope_store(ops, 16384, True, 64),
     "stream_mix2": lambda ops: _stream_mix(ops, 16384, 2),

@@ -33,25 +33,27 @@ def _ints(x):
     return torch.tensor(x, dtype=torch.int32, device="cuda")
 
 
-def _latent_decode(ops, heads, B=64, ctx=2048):
+def _latent_decode(ops, heads, B=64, ctx=2048, window=0):
     R, r, bs = LATENT.kv_rank, LATENT.rot_dim, 256
     cache = _rand(B * ctx // bs, bs, R + r)
     bt = torch.randperm(B * ctx // bs, dtype=torch.int32).view(B, -1).cuda()
     lens = _ints([ctx] * B)
     qa, o = _rand(B, heads, R + r), _rand(B, heads, R)
     scratch = torch.empty(ops.C.latent_decode_scratch(heads, R, ops.num_sms), device="cuda")
-    return (lambda: ops.C.latent_decode(qa, cache, bt, lens, o, scratch, ops.num_sms, LATENT.scale, ops.status),
-            B * ctx * (R + r) * 2 + B * heads * (2 * R + r) * 2, 2 * B * heads * ctx * (2 * R + r))
+    keys = min(ctx, window or ctx)
+    return (lambda: ops.C.latent_decode(qa, cache, bt, lens, o, scratch, ops.num_sms, window, LATENT.scale, ops.status),
+            B * keys * (R + r) * 2 + B * heads * (2 * R + r) * 2, 2 * B * heads * keys * (2 * R + r))
 
 
-def _latent_prefill(ops, S, n):
+def _latent_prefill(ops, S, n, window=0):
     s = LATENT
     T = S * n
     qp, kv, kr = _rand(T, s.heads, 192), _rand(T, s.heads * (s.dim + s.vdim)), _rand(T, s.rot_dim)
     cu = _ints([i * n for i in range(S + 1)])
     out = _rand(T, s.heads * s.vdim)
-    return (lambda: ops.C.latent_prefill(qp, kv, kr, cu, cu, out, 0, S, n, s.dim, s.vdim, s.scale, ops.status),
-            T * s.heads * (192 + s.dim + 2 * s.vdim) * 2, 2 * S * s.heads * n * n // 2 * (s.dim + s.rot_dim + s.vdim))
+    seen = sum(min(i + 1, window or n) for i in range(n))
+    return (lambda: ops.C.latent_prefill(qp, kv, kr, cu, cu, out, 0, S, n, s.dim, s.vdim, window, s.scale, ops.status),
+            T * s.heads * (192 + s.dim + 2 * s.vdim) * 2, 2 * S * s.heads * seen * (s.dim + s.rot_dim + s.vdim))
 
 
 def _retention_prefill(ops, S, n):
@@ -78,6 +80,30 @@ def _retention_decode(ops, B):
     slots, pos, y, table = _ints(list(range(B))), _ints([700] * B), _rand(B, s.heads * s.vdim), _rope(1024, 128)
     return (lambda: ops.C.retention_decode(x, decay, state, slots, pos, table, B, y, 1e-6, ops.status),
             B * s.heads * s.dim * s.vdim * 8 + B * x.shape[1] * 2, 0)
+
+
+def _ungated(ops, T, part):
+    """Eight of 32 experts without gates, chosen within four of eight groups."""
+    E, top, ff = 32, 8, 9 * WIDTH // 16
+    h, router, corr = _rand(T, WIDTH), _rand(E, WIDTH, scale=0.02), torch.zeros(E, device="cuda")
+    experts, weights = torch.empty(T, top, dtype=torch.int32, device="cuda"), torch.empty(T, top, device="cuda")
+    choose = lambda: ops.C.router(h, router, experts, weights, False, corr, 8, 4)
+    if part == "router":
+        return choose, T * WIDTH * 2, 2 * T * WIDTH * E
+    choose()
+    n = T * top
+    tile = ops.expert_tile(n, E)
+    tiles = min(n, n // tile + E)
+    rows = torch.empty(T, top, dtype=torch.int32, device="cuda")
+    te, nt = torch.empty(tiles, dtype=torch.int32, device="cuda"), torch.empty(1, dtype=torch.int32, device="cuda")
+    ops.C.moe_plan(experts, E, tile, rows, te, nt)
+    used = int((torch.bincount(experts.view(-1).long(), minlength=E) > 0).sum())
+    xs, g, y = _rand(tiles * tile, WIDTH), _rand(tiles * tile, ff), _rand(tiles * tile, WIDTH)
+    up, down = _rand(E, ff, WIDTH, scale=0.02), _rand(E, WIDTH, ff, scale=0.02)
+    moved, flops = (used * ff * WIDTH + n * (WIDTH + ff)) * 2, 2 * n * WIDTH * ff
+    if part == "up":
+        return lambda: ops.C.grouped_gemm(xs, up, g, False, tile, te, nt, 1, 0.0, ops.status), moved, flops
+    return lambda: ops.C.grouped_gemm(g, down, y, False, tile, te, nt, 0, 0.0, ops.status), moved, flops
 
 
 def _experts(ops, T, part):
@@ -119,15 +145,19 @@ def _latent_small(ops, which, T):
     pos = _ints(list(range(T)))
     table = _rope(T, s.rot_dim)
     cache = _rand(-(-T // 256), 256, s.kv_rank + s.rot_dim)
+    if which == "prepare_direct":                     # queries come from the input itself
+        cols = s.heads * (s.dim + s.rot_dim)
+        proj, kw = _rand(T, cols + s.kv_rank + s.rot_dim), _rand(s.kv_rank)
+        return (lambda: ops.C.latent_prepare(proj, cols, s.kv_rank, None, kw, 1e-6, table, pos, pos, None, cache, ops.status)), 4 * T * (s.kv_rank + s.rot_dim), 0
     if which == "prepare":
         proj, qw, kw, cq = _rand(T, D), _rand(s.q_rank), _rand(s.kv_rank), _rand(T, s.q_rank)
         return (lambda: ops.C.latent_prepare(proj, s.q_rank, s.kv_rank, qw, kw, 1e-6, table, pos, pos, cq, cache, ops.status)), 4 * T * D, 0
     if which == "pack_q":
         q, qp = _rand(T, s.heads * 192), _rand(T, s.heads, 192)
         return (lambda: ops.C.latent_pack_q(q, qp, s.heads, s.dim, table, pos)), 4 * T * s.heads * 192, 0
-    cu, bt = _ints([0, T]), _ints([list(range(-(-T // 256)))])
+    cu, bt, lens = _ints([0, T]), _ints([list(range(-(-T // 256)))]), _ints([T])
     c, kr = _rand(T, s.kv_rank), _rand(T, s.rot_dim)
-    return (lambda: ops.C.latent_gather(cache, cu, 1, bt, c, kr, ops.status)), 4 * T * (s.kv_rank + s.rot_dim), 0
+    return (lambda: ops.C.latent_gather(cache, cu, lens, 1, bt, c, kr, ops.status)), 4 * T * (s.kv_rank + s.rot_dim), 0
 
 
 def _retention_small(ops, T):
@@ -143,6 +173,12 @@ CASES = {
     "latent_decode_b8": lambda ops: _latent_decode(ops, 16, 8, 16384),
     "latent_prefill": lambda ops: _latent_prefill(ops, 8, 2048),
     "latent_prefill_long": lambda ops: _latent_prefill(ops, 1, 8192),
+    "latent_decode_b8_short": lambda ops: _latent_decode(ops, 16, 8, 4096),
+    "latent_decode_window": lambda ops: _latent_decode(ops, 16, 64, 4096, 2048),
+    "latent_decode_window_b8": lambda ops: _latent_decode(ops, 16, 8, 16384, 4096),
+    "latent_prefill_window": lambda ops: _latent_prefill(ops, 1, 8192, 4096),
+    "latent_prefill_window_short": lambda ops: _latent_prefill(ops, 8, 2048, 512),
+    "latent_prepare_direct": lambda ops: _latent_small(ops, "prepare_direct", 65536),
     "latent_prepare": lambda ops: _latent_small(ops, "prepare", 65536),
     "latent_pack_q": lambda ops: _latent_small(ops, "pack_q", 16384),
     "latent_gather": lambda ops: _latent_small(ops, "gather", 131072),
@@ -158,5 +194,10 @@ CASES = {
     "expert_down": lambda ops: _experts(ops, 8192, "down"),
     "expert_gate_up_decode": lambda ops: _experts(ops, 64, "gate_up"),
     "expert_down_decode": lambda ops: _experts(ops, 64, "down"),
+    "grouped_router": lambda ops: _ungated(ops, 32768, "router"),
+    "ungated_up": lambda ops: _ungated(ops, 8192, "up"),
+    "ungated_down": lambda ops: _ungated(ops, 8192, "down"),
+    "ungated_up_decode": lambda ops: _ungated(ops, 64, "up"),
+    "ungated_down_decode": lambda ops: _ungated(ops, 64, "down"),
     "stream_update": lambda ops: _stream(ops, 16384),
 }
