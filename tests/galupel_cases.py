@@ -94,7 +94,7 @@ def random_weights(cfg, seed=0):
         t = torch.randn(shape, generator=g)
         last = name.split(".")[-1]
         if name.endswith(("q.norm", "k.norm")):
-            t = 1.8 * (1.0 + 0.3 * t)
+            t = 1.3 * (1.0 + 0.3 * t)
         elif last in ("norm", "norm1"):
             t = 1.0 + 0.4 * t
         elif last == "norm2":                   # small: where a rounded router's close call goes the other way, the rest still agrees
