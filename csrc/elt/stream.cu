@@ -397,23 +397,32 @@ extern "C" int forge_stream_update(int fp32, float* x, const void* a, const void
 }
 
 // x <- act(x) elementwise (PlainAct), bf16 or fp32; logits <- cap tanh(scale logits / cap).
-template <typename T>
+template <typename T, int N>
 __global__ void __launch_bounds__(256) act_any_kernel(T* __restrict__ x, long long n, int act, bool logits, float scale, float cap) {
   pdl_launch_dependents();
   pdl_wait();
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const float v = load_f(x + i);
-    store_f(x + i, logits ? bound_logit<sizeof(T) == 4>(v, scale, cap) : plain_act<sizeof(T) == 4>(act, v));
+  const long long step = static_cast<long long>(gridDim.x) * blockDim.x * N;
+  for (long long i = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * N; i < n; i += step) {
+    float v[N];
+    load_n<N>(x + i, v);
+#pragma unroll
+    for (int e = 0; e < N; ++e) v[e] = logits ? bound_logit<sizeof(T) == 4>(v[e], scale, cap) : plain_act<sizeof(T) == 4>(act, v[e]);
+    store_n<N>(x + i, v);
   }
+}
+
+template <typename T>
+static int act_any(T* x, long long n, int act, int logits, float scale, float cap, cudaStream_t stream) {
+  const bool wide = n % 8 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  long long grid = (n / (wide ? 8 : 1) + 255) / 256;
+  if (grid > device_sm_count() * 16) grid = device_sm_count() * 16;
+  auto k = wide ? act_any_kernel<T, 8> : act_any_kernel<T, 1>;
+  return launch_kernel(k, dim3(static_cast<unsigned>(grid)), dim3(256), 0, stream, 0, x, n, act, logits != 0, scale, cap) == cudaSuccess ? 0 : -2;
 }
 
 extern "C" int forge_act_any(int fp32, void* x, long long n, int act, int logits, float scale, float cap, cudaStream_t stream) {
   if (n <= 0) return 0;
-  long long grid = (n + 255) / 256;
-  if (grid > device_sm_count() * 16) grid = device_sm_count() * 16;
-  const dim3 g(static_cast<unsigned>(grid));
-  if (fp32) return launch_kernel(act_any_kernel<float>, g, dim3(256), 0, stream, 0, static_cast<float*>(x), n, act, logits != 0, scale, cap) == cudaSuccess ? 0 : -2;
-  return launch_kernel(act_any_kernel<bf16>, g, dim3(256), 0, stream, 0, static_cast<bf16*>(x), n, act, logits != 0, scale, cap) == cudaSuccess ? 0 : -2;
+  return fp32 ? act_any(static_cast<float*>(x), n, act, logits, scale, cap, stream) : act_any(static_cast<bf16*>(x), n, act, logits, scale, cap, stream);
 }
 
 // out[r, :I] = act(x[r, :I], x[r, I:2I]) (GateAct), any I, bf16 or fp32 (the fused epilogue of the tcgen05 GEMMs needs no such pass).

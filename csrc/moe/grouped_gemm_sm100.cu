@@ -91,12 +91,13 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
       for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
         const int rt = tile % row_tiles, f0 = (tile / row_tiles) * Cfg::kTileFeat;
         const int wrow = max(tile_expert[rt], 0) * w_rows + f0;
+        const bool two = kGated || (kTwo && f0 + kGFeat < n_out);          // the last pair of feature tiles may be half a pair
         for (int kb = 0; kb < num_kb; ++kb) {
           if (!mbar_wait_parked(&empty_bar[s], ph ^ 1, status)) { ok = false; break; }
           uint8_t* st = smem + s * Cfg::kStageBytes;
-          mbar_expect_tx(&full_bar[s], Cfg::kStageBytes);
+          mbar_expect_tx(&full_bar[s], Cfg::kStageBytes - (kTwo && !two ? Cfg::kABytes : 0));
           tma_load_2d(st, &tm_w, &full_bar[s], kb * kGK, wrow);
-          if (kTwo) tma_load_2d(st + Cfg::kABytes, &tm_w, &full_bar[s], kb * kGK, wrow + (kGated ? n_out : kGFeat));
+          if (two) tma_load_2d(st + Cfg::kABytes, &tm_w, &full_bar[s], kb * kGK, wrow + (kGated ? n_out : kGFeat));
           tma_load_2d(st + Cfg::kNumA * Cfg::kABytes, &tm_x, &full_bar[s], kb * kGK, rt * kTok);
           if (++s == Cfg::kStages) { s = 0; ph ^= 1; }
         }
@@ -113,6 +114,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
         if (!mbar_wait_parked(&acc_empty[b], ((n >> 1) & 1) ^ 1, status)) break;
         tcgen05_fence_after();
         const uint32_t acc = tmem_base + b * Cfg::kAccCols;
+        const bool two = kGated || (kTwo && (tile / row_tiles) * Cfg::kTileFeat + kGFeat < n_out);
         for (int kb = 0; kb < num_kb; ++kb) {
           if (!mbar_wait_parked(&full_bar[s], ph, status)) { ok = false; break; }
           tcgen05_fence_after();
@@ -121,7 +123,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_const
 #pragma unroll
           for (int k = 0; k < kGK / 16; ++k) {
             umma_f16(acc, umma_desc_k_sw128(a_addr + k * 32), umma_desc_k_sw128(b_addr + k * 32), idesc, (kb | k) != 0);
-            if (kTwo)
+            if (two)
               umma_f16(acc + kTok, umma_desc_k_sw128(a_addr + Cfg::kABytes + k * 32), umma_desc_k_sw128(b_addr + k * 32), idesc, (kb | k) != 0);
           }
           umma_commit(&empty_bar[s]);

@@ -190,6 +190,13 @@ def test_attention_edges(ops, name, pool, decode, kind):
         close(got, want, 2e-2 if dtype == BF else 2e-5)
 
 
+@pytest.mark.parametrize("ranges", [[(499, 500), (0, 2)], [(499, 500), (0, 7), (3, 5)], [(40, 41), (0, 17)]])
+def test_portions_without_a_whole_block_beside_long_requests(ops, ranges):
+    for dtype in (BF, F32):
+        got, want = attention_case(ops, ATTENTION["real"], 16, ranges, 64, dtype, seed=8)
+        close(got, want, 1e-5 if dtype == F32 else 8e-3)
+
+
 def test_blocks_go_with_the_other_options(ops):
     s = ATTENTION["real"]
     for ranges, decode in (([(0, 300), (290, 300)], False), ([(299, 300), (511, 512)], True)):

@@ -74,12 +74,13 @@ class HybridOps:
         another for a kernel whose tiles cannot gather them: (keys, values, first rows, size), or nothing where no token sees a block."""
         if pool is None:
             return None, None, None, 0
-        seqs, gather = batch.padded_seqs - n1, window is not None and batch.max_seqlen_k - window >= pool.size
+        seqs = batch.padded_seqs - n1
+        entries = (batch.kv_rows if n1 == batch.num_single else seqs * batch.max_seqlen_k) // pool.size
+        gather = window is not None and entries > 0 and batch.max_seqlen_k - window >= pool.size
         offsets = gk = gv = None
         if gather:
             offsets = self.row_offsets(batch, n1, size=pool.size)
-            keys = batch.kv_rows if n1 == batch.num_single else seqs * batch.max_seqlen_k
-            gk, gv = (torch.empty(keys // pool.size, k_cache.shape[1], c.shape[3], dtype=k_cache.dtype, device=k_cache.device) for c in (k_cache, v_cache))
+            gk, gv = (torch.empty(entries, k_cache.shape[1], c.shape[3], dtype=k_cache.dtype, device=k_cache.device) for c in (k_cache, v_cache))
         self.C.pool_blocks(k_cache, v_cache, pool.k, pool.v, pool.size, pool.own, cu, lens, tables, seqs, batch.max_seqlen_q, batch.max_seqlen_k,
                            offsets, gk, gv, self.status)
         return gk, gv, offsets, pool.size if gather else 0
