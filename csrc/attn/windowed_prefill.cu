@@ -125,8 +125,8 @@ struct WindowedPrefill {
 };
 
 // tm_q: [tokens, H * 64 nq], box 128 x 64; tm_k / tm_v: [blocks * G * block_size, d / dv], tm_pk / tm_pv: [entries, G d / G dv], box 64 x 64.
-// kOptions 0: none; 1: chunks, sinks, gates, pooled blocks; 2: these and bounded scores.
-template <int kOptions>
+// kOptions 0: none; 1: chunks, sinks, gates; 2: these and bounded scores.  kPool: pooled blocks behind the window.
+template <int kOptions, bool kPool>
 __global__ void __launch_bounds__(kXThreads, 2)
 windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                         const __grid_constant__ CUtensorMap tm_pk, const __grid_constant__ CUtensorMap tm_pv, const int* __restrict__ cu_q, const int* __restrict__ context_lens, const int* __restrict__ tables,
@@ -163,7 +163,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
   const int kv_end = min(k_len, past + m0 + kXM);
   const int tile0 = oldest_visible(past + m0, z.window, kOptions && z.opt.chunked) / kXN;
   int n_pool = 0;                                     // tiles of pooled blocks: what the CTA's last row sees
-  if (kOptions && z.pool > 0) n_pool = (pool_visible(oldest_visible(min(past + q_len, kv_end) - 1, z.window, 0), z.pool) + kXN - 1) / kXN;
+  if (kPool) n_pool = (pool_visible(oldest_visible(min(past + q_len, kv_end) - 1, z.window, 0), z.pool) + kXN - 1) / kXN;
   const int n_tiles = n_pool + (kv_end + kXN - 1) / kXN - tile0;
   if (n_tiles <= n_pool) return;
 
@@ -200,7 +200,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       mbar_expect_tx(q_full, z.nq * kXQBox);
       for (int b = 0; b < z.nq; ++b) tma_load_2d(sQ + b * kXQBox, &tm_q, q_full, (h * z.nq + b) * 64, q_begin + m0);
       for (int j = 0; j < n_tiles; ++j) {
-        const bool means = kOptions && j < n_pool;
+        const bool means = kPool && j < n_pool;
         const int s = j & 1, tok = (tile0 + j - n_pool) * kXN;
         const uint32_t ph = (j >> 1) & 1;
         int row, k_col = 0, v_col = 0;
@@ -277,7 +277,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const int qpos = past + m0 + r;
     const int key_limit = min(qpos + 1, k_len), key_lo = oldest_visible(qpos, z.window, kOptions && z.opt.chunked);  // visible keys
-    const int block_limit = kOptions && z.pool > 0 ? pool_visible(key_lo, z.pool) : 0;                             // visible blocks
+    const int block_limit = kPool ? pool_visible(key_lo, z.pool) : 0;                                              // visible blocks
     const int o_cols = z.nv * 64;
     float m_ref = 0.f, l_run = 0.f;
     bool seen = false, ok = true;
@@ -286,7 +286,7 @@ windowed_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_c
       if (!ok) break;
       tcgen05_fence_after();
       const uint32_t s_addr = tmem_base + lane_addr + (j & 1) * kXN;
-      const bool means = kOptions && j < n_pool;
+      const bool means = kPool && j < n_pool;
       const int kbase = means ? j * kXN : (tile0 + j - n_pool) * kXN;
       const int lo = means ? 0 : key_lo, limit = means ? block_limit : key_limit;            // visible in this tile: [lo, limit)
       const bool masked = !__all_sync(0xffffffffu, kbase >= lo && kbase + kXN <= limit);
@@ -440,10 +440,15 @@ extern "C" int forge_windowed_prefill(const void* q, int tokens, const void* k_c
     if (forge_make_tmap_2d(&tm_pk, pool_k, pool_entries, kw, kw, kXN, 2) != 0) return -2;
     if (forge_make_tmap_2d(&tm_pv, pool_v, pool_entries, vw, vw, kXN, 2) != 0) return -2;
   }
-  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<0>, 227 * 1024);
-  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<1>, 227 * 1024);
-  FORGE_ENSURE_DYN_SMEM(windowed_prefill_kernel<2>, 227 * 1024);
-  auto k = softcap > 0.f ? windowed_prefill_kernel<2> : chunked || sink != nullptr || gate != nullptr || pool > 0 ? windowed_prefill_kernel<1> : windowed_prefill_kernel<0>;
+  FORGE_ENSURE_DYN_SMEM((windowed_prefill_kernel<0, false>), 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM((windowed_prefill_kernel<1, false>), 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM((windowed_prefill_kernel<2, false>), 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM((windowed_prefill_kernel<0, true>), 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM((windowed_prefill_kernel<1, true>), 227 * 1024);
+  FORGE_ENSURE_DYN_SMEM((windowed_prefill_kernel<2, true>), 227 * 1024);
+  const int options = softcap > 0.f ? 2 : chunked || sink != nullptr || gate != nullptr ? 1 : 0;
+  auto k = pool > 0 ? (options == 2 ? windowed_prefill_kernel<2, true> : options == 1 ? windowed_prefill_kernel<1, true> : windowed_prefill_kernel<0, true>)
+                    : (options == 2 ? windowed_prefill_kernel<2, false> : options == 1 ? windowed_prefill_kernel<1, false> : windowed_prefill_kernel<0, false>);
   return launch_kernel(k, dim3((max_q + kXM - 1) / kXM, H, num_seqs), dim3(kXThreads), smem, stream, 0, tm_q, tm_k, tm_v, tm_pk, tm_pv,
                        cu_q, context_lens, tables, static_cast<bf16*>(out), z, status) == cudaSuccess ? 0 : -5;
 }
